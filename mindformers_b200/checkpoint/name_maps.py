@@ -108,7 +108,69 @@ def reverse_name_glm(name: str) -> str:
     return out
 
 
-FAMILIES = ("llama", "qwen2", "qwen2_5", "qwen2_moe", "qwen3", "qwen3_moe", "deepseek_v2", "deepseek_v3",
+# Mefesun checkpoints: ``l<i>.mix.*`` / ``l<i>.mlp.*`` / ``l<i>.norm1`` ..., a tensor's bias is its name with ``.b``.
+# The last component decides between weight and bias, so the names are mapped one by one (``None``: no suffix).
+_MEFESUN = {
+    "mix.q": ("self_attention.linear_q", "weight"), "mix.k": ("self_attention.linear_k", "weight"),
+    "mix.v": ("self_attention.linear_v", "weight"), "mix.o": ("self_attention.linear_proj", "weight"),
+    "mix.q.norm": ("self_attention.q_layernorm", "weight"), "mix.k.norm": ("self_attention.k_layernorm", "weight"),
+    "mix.sink": ("self_attention.sink", None), "mlp.up": ("mlp.linear_fc1", "weight"), "mlp.down": ("mlp.linear_fc2", "weight"),
+    "norm1": ("post_attn_layernorm", "weight"), "norm2": ("post_mlp_layernorm", "weight"),
+    "ls1": ("attn_layer_scale", None), "ls2": ("mlp_layer_scale", None),
+}
+_MEFESUN_TOP = {"embed": "embedding.word_embeddings.weight", "final.norm": "decoder.final_layernorm.weight",
+                "final.norm.b": "decoder.final_layernorm.bias"}
+_MEFESUN_LAYER = re.compile(r"^l(\d+)\.(.+)$")
+
+
+def is_mefesun_name(name: str) -> bool:
+    return bool(_MEFESUN_LAYER.match(name)) or name in _MEFESUN_TOP
+
+
+def convert_name_mefesun(name: str) -> str:
+    """Mefesun key → per-projection framework key."""
+    if name in _MEFESUN_TOP:
+        return _MEFESUN_TOP[name]
+    m = _MEFESUN_LAYER.match(name)
+    if not m:
+        return name
+    part, kind = (m[2][:-2], "bias") if m[2].endswith(".b") else (m[2], None)
+    if part not in _MEFESUN:
+        raise KeyError(f"{name}: no counterpart in the model")
+    base, suffix = _MEFESUN[part]
+    suffix = kind or suffix
+    return f"decoder.layers.{m[1]}.{base}" + (f".{suffix}" if suffix else "")
+
+
+def framework_to_mefesun(sd: Dict[str, torch.Tensor], config) -> Dict[str, torch.Tensor]:
+    """Fused framework names → Mefesun keys (the q, k and v rows of a layer have that layer's sizes)."""
+    top = {v: k for k, v in _MEFESUN_TOP.items()}
+    back = {base: part for part, (base, _) in _MEFESUN.items()}
+    out: Dict[str, torch.Tensor] = {}
+    for name, t in sd.items():
+        if name in top:
+            out[top[name]] = t
+            continue
+        m = re.match(r"^decoder\.layers\.(\d+)\.(.+)$", name)
+        if not m:
+            out[name] = t
+            continue
+        base, kind = m[2], ""
+        if base.endswith((".weight", ".bias")):
+            base, _, last = base.rpartition(".")
+            kind = ".b" if last == "bias" else ""
+        if base == "self_attention.linear_qkv":
+            c = config.for_layer(int(m[1]))
+            rows = (c.num_attention_heads * c.kv_channels, c.num_query_groups * c.kv_channels,
+                    c.num_query_groups * (c.v_channels or c.kv_channels))
+            for p, piece in zip("qkv", torch.split(t, rows, dim=0)):
+                out[f"l{m[1]}.mix.{p}{kind}"] = piece.contiguous()
+        else:
+            out[f"l{m[1]}.{back[base]}{kind}"] = t
+    return out
+
+
+FAMILIES = ("mefesun", "llama", "qwen2", "qwen2_5", "qwen2_moe", "qwen3", "qwen3_moe", "deepseek_v2", "deepseek_v3",
             "deepseekv3", "mixtral", "telechat", "glm")
 
 
@@ -116,6 +178,8 @@ def convert_name(hf_name: str, family: str = "llama") -> str:
     """HF key → per-projection framework key."""
     if family == "glm" and is_glm_name(hf_name):
         return convert_name_glm(hf_name)
+    if family == "mefesun":
+        return convert_name_mefesun(hf_name)
     out = hf_name
     for a, b in _COMMON:
         out = out.replace(a, b)
@@ -384,6 +448,9 @@ def framework_to_hf(sd: Dict[str, torch.Tensor], config, family: str = "llama", 
                 t = t.to(dtype)
             out[reverse_name_glm(name)] = t.contiguous()
         return out
+    if family == "mefesun":
+        return {k: (t if dtype is None or not t.is_floating_point() else t.to(dtype)).contiguous()
+                for k, t in framework_to_mefesun(sd, config).items()}
     for name, t in unfuse_state_dict(sd, config).items():
         if dtype is not None and t.is_floating_point():
             t = t.to(dtype)

@@ -31,16 +31,25 @@ class GenerationMixin:
     generation_config: Optional[GenerationConfig] = None
 
     # ---- cache --------------------------------------------------------------------------------------
-    def _set_kv_cache(self, batch_size: int, max_len: int, num_blocks: Optional[int] = None, extra_layers: int = 0):
+    def _set_kv_cache(self, batch_size: int, max_len: int, num_blocks: Optional[int] = None, extra_layers: int = 0,
+                      exact_blocks: bool = False):
+        """``num_blocks`` raises the pool above what ``batch_size`` sequences of ``max_len`` tokens need; with
+        ``exact_blocks`` the pool has exactly that many blocks (the sequences then share it)."""
         cfg = self.config
         block_size = int(getattr(cfg, "block_size", 16) or 16)
         need = batch_size * (-(-max_len // block_size))
-        num_blocks = max(int(num_blocks or 0), need)
+        num_blocks = int(num_blocks) if exact_blocks and num_blocks else max(int(num_blocks or 0), need)
         tp = ps.get_tensor_model_parallel_world_size()
         device = next(self.parameters()).device
         dtype = next(self.parameters()).dtype
-        n_layers = len(self.model.decoder.layers) + extra_layers      # extra: multi-token-prediction layers that draft
-        if getattr(cfg, "multi_latent_attention", False):
+        n_layers = self.model.decoder.num_runs + extra_layers      # extra: multi-token-prediction layers that draft
+        shapes = self.model.decoder.cache_shapes()
+        if shapes is not None:
+            if extra_layers:
+                raise NotImplementedError("draft layers share the cache shapes of the decoder")
+            ctx = KVCacheContext(n_layers, num_blocks, block_size, 0, 0, dtype, device, layer_shapes=shapes,
+                                 kv_cache_dtype=getattr(cfg, "kv_cache_dtype", None))
+        elif getattr(cfg, "multi_latent_attention", False):
             ctx = KVCacheContext(n_layers, num_blocks, block_size, 1, 0, dtype, device,
                                  mla_latent_dim=cfg.kv_lora_rank + cfg.qk_pos_emb_head_dim)
         else:
@@ -55,10 +64,12 @@ class GenerationMixin:
     @torch.no_grad()
     def _forward_step(self, tokens: List[List[int]], starts: List[int], ctx: KVCacheContext, tables: BlockTables,
                       prefill: bool, active: Optional[List[bool]] = None, all_logits: bool = False,
-                      return_hidden: bool = False) -> torch.Tensor:
+                      return_hidden: bool = False, rows: Optional[List[int]] = None) -> Optional[torch.Tensor]:
         """Run the model on the new ``tokens`` of every sequence (positions start at ``starts``).
         Returns logits ``[B, V]`` of the last new token of each sequence (``all_logits``: of every new token). With
-        ``return_hidden`` the result is ``(logits, hidden [T, H] of every new token, flat token ids, positions)``."""
+        ``return_hidden`` the result is ``(logits, hidden [T, H] of every new token, flat token ids, positions)``.
+        ``rows`` (prefill calls): the flat new tokens whose logits are wanted; with an empty list the output layer does not
+        run and the result is None."""
         device = next(self.parameters()).device
         lens = [len(t) for t in tokens]
         if hasattr(self, "set_phase"):
@@ -73,10 +84,15 @@ class GenerationMixin:
                      q_seq_lens=lens, device=device)
         if all_logits:       # draft verification: the logits of every new token are needed
             ctx.last_token_index = torch.arange(int(flat.numel()), dtype=torch.int64, device=device)
+        if rows is not None:
+            ctx.last_token_index = torch.tensor(rows, dtype=torch.int64, device=device)
         meta = AttnMeta(batch=1, seq_len=int(flat.numel()), positions=pos, cache=ctx)
         hook = getattr(self, "input_embeds_hook", None)     # multimodal models splice encoder outputs in here
         embeds = hook(flat, pos, prefill) if hook is not None else None
         hidden_all = None
+        if rows is not None and not len(rows):
+            self.model(flat.unsqueeze(0), attn_meta=meta, return_hidden=True, input_embeds=embeds)
+            return None
         if return_hidden:
             hidden_all = self.model(flat.unsqueeze(0), attn_meta=meta, return_hidden=True, input_embeds=embeds)
             rows = hidden_all if (all_logits or not prefill) else hidden_all.index_select(0, ctx.last_token_index)
@@ -85,7 +101,7 @@ class GenerationMixin:
             logits = self.model(flat.unsqueeze(0), attn_meta=meta, input_embeds=embeds)
         else:
             logits = self.model(flat.unsqueeze(0), attn_meta=meta)
-        if all_logits:
+        if all_logits or rows is not None:
             pass
         elif not prefill:
             pass  # decode: one row per sequence already
@@ -99,6 +115,24 @@ class GenerationMixin:
         if return_hidden:
             return logits[:, : self.config.vocab_size], hidden_all, flat, pos
         return logits[:, : self.config.vocab_size]
+
+    @torch.no_grad()
+    def _forward_sequences(self, input_ids: torch.Tensor, labels=None, loss_mask=None):
+        """Logits ``[B * S, V]`` (or the masked loss, when labels are given) of whole sequences through a cache made for
+        this call: the forward pass of models whose attention reads its keys from a paged cache. No gradients."""
+        ids = input_ids if input_ids.dim() == 2 else input_ids.unsqueeze(0)
+        B, S = ids.shape
+        ctx, tables = self._set_kv_cache(B, S)
+        tables.init_cache_engine(B)
+        logits = self._forward_step(ids.tolist(), [0] * B, ctx, tables, True, all_logits=True)
+        tables.clear_cache()
+        if labels is None:
+            return logits
+        if loss_mask is None:
+            loss_mask = (ids != self.config.pad_token_id) & (labels != self.config.ignore_token_id)
+        else:
+            loss_mask = loss_mask.to(torch.bool) & (labels != self.config.ignore_token_id)
+        return self.model.loss(logits, labels, loss_mask)
 
     # ---- decode step as a CUDA graph ---------------------------------------------------------------------
     def _graph_decoder(self, B: int, ctx: KVCacheContext, tables: BlockTables):

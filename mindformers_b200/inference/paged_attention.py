@@ -28,8 +28,11 @@ class KVCacheContext:
 
     def __init__(self, num_layers: int, num_blocks: int, block_size: int, kv_heads: int, head_dim: int,
                  dtype=torch.bfloat16, device="cuda", mla_latent_dim: Optional[int] = None,
-                 kv_cache_dtype: Optional[str] = None):
-        """``kv_cache_dtype="int8"`` stores keys and values as int8 codes with one fp32 scale per token and KV head
+                 kv_cache_dtype: Optional[str] = None, layer_shapes: Optional[list] = None):
+        """``layer_shapes``: ``(kv heads, key size, value size)`` of every layer's cache, for models whose layers differ or
+        whose keys and values differ in size; such a cache also carries the step metadata of ragged attention.
+
+        ``kv_cache_dtype="int8"`` stores keys and values as int8 codes with one fp32 scale per token and KV head
         (``key_scale`` / ``value_scale`` ``[num_blocks, block_size, kv_heads]``): half the bytes per cached token, read
         back by the decode kernel and by prefill with history. Not available for the multi-latent cache."""
         self.num_layers, self.num_blocks, self.block_size = num_layers, num_blocks, block_size
@@ -39,7 +42,14 @@ class KVCacheContext:
         self.compute_dtype = dtype
         if self.int8 and mla_latent_dim:
             raise ValueError("an int8 KV cache is not available for multi-latent attention")
-        if self.int8:
+        self.ragged = layer_shapes is not None
+        if self.ragged:
+            if self.int8 or mla_latent_dim or len(layer_shapes) != num_layers:
+                raise ValueError("per-layer cache shapes: one per layer, and no int8 or latent cache")
+            rows = (num_blocks, block_size)
+            self.key_cache = [torch.zeros(rows + (h, k), dtype=dtype, device=device) for h, k, _ in layer_shapes]
+            self.value_cache = [torch.zeros(rows + (h, v), dtype=dtype, device=device) for h, _, v in layer_shapes]
+        elif self.int8:
             shape = (num_blocks, block_size, kv_heads, head_dim)
             self.key_cache = [torch.zeros(shape, dtype=torch.int8, device=device) for _ in range(num_layers)]
             self.value_cache = [torch.zeros(shape, dtype=torch.int8, device=device) for _ in range(num_layers)]
@@ -61,6 +71,9 @@ class KVCacheContext:
         self.last_token_index = None  # int64 [B] row of the last new token of each sequence
         self.cu_q = None              # python list of cumulative q lengths
         self.layer_offset = 0
+        self.cu_q_dev = None          # int32 [B+1]: cu_q on the device (ragged caches, prefill steps)
+        self.prefill_work_dev = None  # int32 [n, 2]: work list of the ragged prefill kernel
+        self.n_prefill_work = self.n_single_rows = 0
 
     def set_step(self, *, is_prefill, block_tables, slot_mapping, context_lens, q_seq_lens, device):
         self.is_prefill = is_prefill
@@ -73,6 +86,12 @@ class KVCacheContext:
         for n in q:
             cu.append(cu[-1] + n)
         self.cu_q = cu
+        if self.ragged and is_prefill:
+            from .ragged_attention import prefill_work
+            work = prefill_work(q, [int(x) for x in context_lens])
+            self.n_prefill_work, self.n_single_rows = len(work), sum(n == 1 for n in q)
+            flat = torch.tensor(cu + [x for item in work for x in item], dtype=torch.int32).to(device)   # one copy
+            self.cu_q_dev, self.prefill_work_dev = flat[: len(cu)], flat[len(cu):]
         # sequences without new tokens in this step (finished prompts of a chunked prefill, idle serving slots) have
         # no row of their own: one entry per sequence that has tokens
         self.last_token_index = torch.as_tensor([c - 1 for c, n in zip(cu[1:], q) if n > 0], dtype=torch.int64,

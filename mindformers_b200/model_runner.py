@@ -105,11 +105,15 @@ class ModelRunner:
         first = next(self.model.parameters())
         self.device, self.dtype = first.device, first.dtype
         tp = ps.get_tensor_model_parallel_world_size()
-        self.n_layers = len(self.model.model.decoder.layers)
+        self.n_layers = self.model.model.decoder.num_runs
+        shapes = self.model.model.decoder.cache_shapes()
         mla = bool(getattr(cfg, "multi_latent_attention", False))
         if mla:
             self.kv_heads, self.head_dim, width = 1, cfg.kv_lora_rank + cfg.qk_pos_emb_head_dim, cfg.kv_lora_rank + cfg.qk_pos_emb_head_dim
             per_block = self.n_layers * self.block_size * width * first.element_size()
+        elif shapes is not None:
+            self.kv_heads = self.head_dim = 0
+            per_block = sum(h * (k + v) for h, k, v in shapes) * self.block_size * first.element_size()
         else:
             self.kv_heads = max(1, (cfg.num_query_groups or cfg.num_attention_heads) // tp)
             self.head_dim = cfg.kv_channels or cfg.hidden_size // cfg.num_attention_heads
@@ -117,7 +121,8 @@ class ModelRunner:
         self.num_npu_blocks = max(1, int(npu_mem_size * (1 << 30)) // per_block)
         self.num_cpu_blocks = max(0, int(cpu_mem_size * (1 << 30)) // per_block)
         self.cache = KVCacheContext(self.n_layers, self.num_npu_blocks, self.block_size, self.kv_heads,
-                                    0 if mla else self.head_dim, self.dtype, self.device, mla_latent_dim=self.head_dim if mla else None)
+                                    0 if mla else self.head_dim, self.dtype, self.device, mla_latent_dim=self.head_dim if mla else None,
+                                    layer_shapes=shapes)
         self.cache.layer_offset = self.model.model.decoder.layer_ids[0] if self.model.model.decoder.layer_ids else 0
         pin = torch.cuda.is_available()
         self.cpu_key = [torch.zeros((self.num_cpu_blocks,) + tuple(k.shape[1:]), dtype=self.dtype, pin_memory=pin) for k in self.cache.key_cache]

@@ -36,6 +36,8 @@ def _read_config_dict(path: str) -> dict:
 
 def _classes_for(d: dict):
     mt = d.get("model_type") or d.get("type")
+    if mt is None and isinstance(d.get("architecture"), str):      # designs named by one ``architecture`` key
+        mt = d["architecture"].lower()
     if mt in _EXTRA:
         return _EXTRA[mt]
     if mt in MODEL_TYPE_TO_CLASSES:

@@ -6,6 +6,8 @@ which here differ only in configuration defaults: all of them are instances of t
 """
 from __future__ import annotations
 
+import copy
+
 from ..tools.register import MindFormerModuleType, MindFormerRegister
 from .configuration_utils import PretrainedConfig
 from .modeling_utils import PreTrainedModel
@@ -141,6 +143,79 @@ MindFormerRegister.register_cls(ChatGLM2Config, MindFormerModuleType.CONFIG, ali
 MindFormerRegister.register_cls(ChatGLM2Config, MindFormerModuleType.CONFIG, alias="ChatGLM2Config", legacy=False)
 ChatGLM4Config = ChatGLM2Config
 
+
+
+class MefesunConfig(PretrainedConfig):
+    """Mefesun: a decoder described layer by layer, with norms on the sub-layer outputs only, layer scale, chunked
+    grouped-query attention with a softmax sink, q / k norm, YaRN rotary positions, squared-relu feed-forwards, optional
+    weight sharing between layers, a tied head and soft-capped logits.
+
+    Keys of ``config.json``: ``vocab``, ``width``, ``norm.eps``, ``logit_softcap`` and ``layers``, a list of ``{"type":
+    "attention", "mixer": {"heads", "kv_heads", "dim", "vdim", "scale", "mask": {"size"}, "rot": {"base", "dims",
+    "scaling": {"factor", "original", "fast", "slow"}}}, "mlp": {"kind": "dense", "ff"} | null, "weights_of"}``. Framework
+    keys (``seq_length``, ``block_size``, token ids) may stand beside them. ``to_transformer_dict`` translates."""
+
+    model_type = "mefesun"
+
+    @classmethod
+    def default_values(cls):
+        return dict(architecture="Mefesun", vocab=32000, width=1024, norm=dict(eps=1e-6), logit_softcap=30.0,
+                    layers=MefesunConfig.uniform_layers(12, heads=8, kv_heads=2, dim=128, ff=4096, chunk=2048),
+                    pad_token_id=0, bos_token_id=None, eos_token_id=None, block_size=64)
+
+    @staticmethod
+    def uniform_layers(n: int, heads: int, kv_heads: int, dim: int, ff: int, chunk: int, vdim=None, rot_dims=None,
+                       base: float = 500000.0, factor: float = 8.0, original: int = 8192, fast: float = 32.0,
+                       slow: float = 1.0, scale=None):
+        """The ``layers`` list of a model whose ``n`` layers are alike."""
+        mixer = dict(heads=heads, kv_heads=kv_heads, dim=dim, vdim=vdim or dim, scale=scale or dim ** -0.5,
+                     mask=dict(size=chunk), rot=dict(base=base, dims=rot_dims or dim,
+                                                     scaling=dict(factor=factor, original=original, fast=fast, slow=slow)))
+        return [dict(type="attention", mixer=copy.deepcopy(mixer), mlp=dict(kind="dense", ff=ff)) for _ in range(n)]
+
+    @staticmethod
+    def _layer_fields(i: int, layer: dict) -> dict:
+        if layer.get("type") != "attention":
+            raise ValueError(f"layer {i}: unknown mixer type {layer.get('type')!r}")
+        mix, mlp = layer["mixer"], layer.get("mlp")
+        if mlp and mlp.get("kind", "dense") != "dense":
+            raise ValueError(f"layer {i}: unknown feed-forward kind {mlp['kind']!r}")
+        rot = mix["rot"]
+        scaling = rot.get("scaling")
+        return dict(
+            num_attention_heads=int(mix["heads"]), num_query_groups=int(mix["kv_heads"]), kv_channels=int(mix["dim"]),
+            v_channels=int(mix["vdim"]), softmax_scale=float(mix["scale"]),
+            attention_chunk_size=int((mix.get("mask") or {}).get("size") or 0),
+            rotary_dim=int(rot["dims"]), rotary_base=float(rot["base"]),
+            rope_scaling=None if not scaling else dict(
+                type="yarn", factor=float(scaling["factor"]), original_max_position_embeddings=float(scaling["original"]),
+                beta_fast=float(scaling["fast"]), beta_slow=float(scaling["slow"])),
+            ffn_hidden_size=int(mlp["ff"]) if mlp else 0)
+
+    def to_transformer_dict(self) -> dict:
+        d = {k: v for k, v in self.to_dict().items()
+             if k not in ("architecture", "layers", "norm", "vocab", "width", "mlp", "mixer")}
+        fields = [self._layer_fields(i, layer) for i, layer in enumerate(self.layers)]
+        owners = []
+        for i, layer in enumerate(self.layers):
+            j = layer.get("weights_of")
+            owners.append(i if j is None else owners[int(j)])
+        d.update({k: v for k, v in fields[0].items() if k != "rope_scaling"})
+        d.setdefault("seq_length", max(int(f["rope_scaling"]["factor"] * f["rope_scaling"]["original_max_position_embeddings"])
+                                       if f["rope_scaling"] else 4096 for f in fields))
+        d.setdefault("max_position_embeddings", d["seq_length"])
+        d.update(vocab_size=int(self.vocab), hidden_size=int(self.width), num_layers=len(fields), layer_overrides=fields,
+                 layer_sharing=owners, layernorm_epsilon=float(self.norm["eps"]), normalization="LayerNorm",
+                 norm_placement="output", layer_scale=True, fp32_residual_connection=True, ragged_attention=True,
+                 qk_layernorm=True, add_qkv_bias=True, add_attention_output_bias=True, attention_sink=True,
+                 rotary_interleaved=True, gated_linear_unit=False, hidden_act="relu2", position_embedding_type="none",
+                 tie_word_embeddings=True, logit_softcap=float(self.logit_softcap) if self.logit_softcap else None)
+        return d
+
+
+for _legacy in (True, False):
+    MindFormerRegister.register_cls(MefesunConfig, MindFormerModuleType.CONFIG, alias="MefesunConfig", legacy=_legacy)
+
 LlamaForCausalLM = _model("LlamaForCausalLM", LlamaConfig, "llama")
 Qwen2ForCausalLM = _model("Qwen2ForCausalLM", Qwen2Config, "qwen2")
 Qwen3ForCausalLM = _model("Qwen3ForCausalLM", Qwen3Config, "qwen3")
@@ -150,6 +225,10 @@ DeepseekV2ForCausalLM = _model("DeepseekV2ForCausalLM", DeepseekV2Config, "deeps
 Qwen2MoeForCausalLM = _model("Qwen2MoeForCausalLM", Qwen2MoeConfig, "qwen2_moe")
 MixtralForCausalLM = _model("MixtralForCausalLM", MixtralConfig, "mixtral")
 TelechatForCausalLM = _model("TelechatForCausalLM", TelechatConfig, "telechat")
+MefesunForCausalLM = _model("MefesunForCausalLM", MefesunConfig, "mefesun")
+MefesunForCausalLM.kernel_sources = ("host_util", "elementwise", "gemm_tcgen05", "gemm_tcgen05_2cta", "gemm_bf16_decode",
+                                     "output_norm", "qkv_rope_cache", "paged_prefill_tc", "paged_decode_tc",
+                                     "paged_attention", "paged_attention_any", "decode_loop")
 ChatGLM2ForConditionalGeneration = _model("ChatGLM2ForConditionalGeneration", ChatGLM4Config, "glm")
 
 def _backbone(name, causal_cls):
@@ -219,5 +298,5 @@ MODEL_TYPE_TO_CLASSES = {
     "deepseek_v2": (DeepseekV2Config, DeepseekV2ForCausalLM), "deepseek2": (DeepseekV2Config, DeepseekV2ForCausalLM),
     "qwen2_moe": (Qwen2MoeConfig, Qwen2MoeForCausalLM),
     "telechat": (TelechatConfig, TelechatForCausalLM), "glm": (ChatGLM4Config, ChatGLM2ForConditionalGeneration),
-    "chatglm": (ChatGLM4Config, ChatGLM2ForConditionalGeneration),
+    "mefesun": (MefesunConfig, MefesunForCausalLM), "chatglm": (ChatGLM4Config, ChatGLM2ForConditionalGeneration),
 }

@@ -33,6 +33,7 @@ class PreTrainedModel(nn.Module, GenerationMixin, InferModelMixin):
     config_class = PretrainedConfig
     base_model_prefix = "model"
     weight_family = "llama"
+    kernel_sources = None        # kernel source files that serving needs (None: the full library)
 
     def __init__(self, config: PretrainedConfig, device=None, dtype=None, **kwargs):
         super().__init__()
@@ -61,6 +62,8 @@ class PreTrainedModel(nn.Module, GenerationMixin, InferModelMixin):
 
     # ---- forward ----------------------------------------------------------------------------------------
     def forward(self, input_ids, labels=None, loss_mask=None, position_ids=None, attn_meta=None, **kw):
+        if attn_meta is None and self.config.ragged_attention:       # attention of these models reads a paged cache
+            return self._forward_sequences(input_ids, labels, loss_mask)
         return self.model(input_ids, labels, loss_mask, position_ids, attn_meta,
                           input_embeds=kw.get("input_embeds"))
 

@@ -19,6 +19,7 @@ ABI_VERSION = 2
 
 _lock = threading.Lock()
 _lib = None
+_path = KERNEL_LIB_PATH
 _launch_count = 0  # kernels launched through this binding (read by the benchmark)
 
 c_void_p = ctypes.c_void_p
@@ -34,11 +35,12 @@ class KernelLibraryError(RuntimeError):
 
 
 def _declare(lib):
-    def sig(name, args):
+    def sig(name, args, restype=c_int):
+        if not hasattr(lib, name):        # a library of selected sources (``build.ensure``): calling what it lacks raises
+            return
         fn = getattr(lib, name)
         fn.argtypes = args
-        fn.restype = c_int
-        return fn
+        fn.restype = restype
 
     P, I, L, F = c_void_p, c_int, c_ll, c_float
     lib.mfb_last_error.restype = ctypes.c_char_p
@@ -46,9 +48,9 @@ def _declare(lib):
     sig("mfb_gemm_bf16", [P, P, P, I, I, I, I, I, I, I, I, I, I, I, P, P, P, I, P, I, P])
     sig("mfb_gemm_bf16_decode_supported", [I, I, I])
     sig("mfb_gemm_bf16_decode", [P, P, P, P, I, I, I, L, L, L, I, P, P])
+    sig("mfb_gemm_bf16_decode_ex", [P, P, P, P, I, I, I, L, L, L, I, I, I, F, P, P])
     sig("mfb_gemm_bf16_pair", [P, P, P, I, I, I, I, I, I, I, I, I, P, I, P, I, P])
-    lib.mfb_gemm_pair_workspace_bytes.argtypes = []
-    lib.mfb_gemm_pair_workspace_bytes.restype = L
+    sig("mfb_gemm_pair_workspace_bytes", [], L)
     sig("mfb_gemm_pair_plan", [I, I, I, I, I, P, P])
     sig("mfb_rmsnorm_fwd", [P, P, P, P, P, P, I, I, F, P])
     sig("mfb_rmsnorm_bwd_parts", [I])
@@ -71,44 +73,31 @@ def _declare(lib):
     sig("mfb_flash_attn_fwd", [P, P, P, P, P, I, I, I, I, I, L, L, L, L, I, F, P, P])
     sig("mfb_flash_attn_fwd2_varlen", [P, P, P, P, P, P, I, I, I, I, I, L, L, L, L, I, I, F, P, P])
     sig("mfb_flash_attn_bwd2_varlen", [P] * 12 + [I, I, I, I, I] + [L] * 8 + [I, I, F, P, P])
-    lib.mfb_tp_set_rs_interleave.argtypes = [I]
-    lib.mfb_tp_set_rs_interleave.restype = None
-    lib.mfb_tp_set_pair.argtypes = [I]
-    lib.mfb_tp_set_pair.restype = None
-    lib.mfb_flash_attn_set_bwd_variant.argtypes = [I]
-    lib.mfb_flash_attn_set_bwd_variant.restype = None
-    lib.mfb_flash_attn_bwd2_set_split.argtypes = [I]
-    lib.mfb_flash_attn_bwd2_set_split.restype = None
-    lib.mfb_flash_attn_bwd_scratch_bytes_ex.argtypes = [I, I, I, I, I]
-    lib.mfb_flash_attn_bwd_scratch_bytes_ex.restype = L
-    lib.mfb_flash_attn_set_fwd_variant.argtypes = [I]
-    lib.mfb_flash_attn_set_fwd_variant.restype = None
-    lib.mfb_flash_attn_fwd2_set_poly.argtypes = [I]
-    lib.mfb_flash_attn_fwd2_set_poly.restype = None
+    sig("mfb_tp_set_rs_interleave", [I], None)
+    sig("mfb_tp_set_pair", [I], None)
+    sig("mfb_flash_attn_set_bwd_variant", [I], None)
+    sig("mfb_flash_attn_bwd2_set_split", [I], None)
+    sig("mfb_flash_attn_bwd_scratch_bytes_ex", [I, I, I, I, I], L)
+    sig("mfb_flash_attn_set_fwd_variant", [I], None)
+    sig("mfb_flash_attn_fwd2_set_poly", [I], None)
     sig("mfb_flash_attn_fwd_mla", [P, P, P, P, P, I, I, I, I, I, L, L, L, L, I, I, F, P, P])
-    lib.mfb_flash_attn_bwd_scratch_bytes.argtypes = [I, I, I]
-    lib.mfb_flash_attn_bwd_scratch_bytes.restype = L
+    sig("mfb_flash_attn_bwd_scratch_bytes", [I, I, I], L)
     sig("mfb_flash_attn_bwd", [P] * 10 + [I, I, I, I] + [L] * 8 + [I, F, P, P])
     sig("mfb_reshape_and_cache", [P, P, P, P, P, L, I, L, L, P])
     sig("mfb_paged_decode_attention", [P, P, P, P, P, P, P, I, I, I, I, I, I, I, F, P])
     sig("mfb_paged_decode_splits", [I, I, I, I])
-    lib.mfb_paged_decode_scratch_bytes.argtypes = [I, I, I, I]
-    lib.mfb_paged_decode_scratch_bytes.restype = L
+    sig("mfb_paged_decode_scratch_bytes", [I, I, I, I], L)
     sig("mfb_gemm_fp8_decode", [P, P, P, P, L, P, I, I, I, L, L, L, I, I, P, P, P, P, P, P])
     sig("mfb_gemm_fp8_decode_supported", [I, I, I, I])
-    lib.mfb_gemm_fp8_enable_ksplit.argtypes = [I]
-    lib.mfb_gemm_fp8_enable_ksplit.restype = None
+    sig("mfb_gemm_fp8_enable_ksplit", [I], None)
     sig("mfb_gemm_fp8_ksplit", [I, I, I, I, L])
     sig("mfb_mla_decode_attention", [P, P, P, P, P, P, I, I, I, I, I, I, F, P, P])
     sig("mfb_mla_decode_splits", [I, I, I])
-    lib.mfb_mla_decode_set_variant.argtypes = [I]
-    lib.mfb_mla_decode_set_variant.restype = None
+    sig("mfb_mla_decode_set_variant", [I], None)
     sig("mfb_mla_decode_get_variant", [])
-    lib.mfb_mla_decode_scratch_bytes.argtypes = [I, I, I]
-    lib.mfb_mla_decode_scratch_bytes.restype = L
+    sig("mfb_mla_decode_scratch_bytes", [I, I, I], L)
     sig("mfb_gather_cache", [P, P, P, P, I, I, I, I, I, P])
-    lib.mfb_ll_allreduce_buffer_bytes.argtypes = [I, L]
-    lib.mfb_ll_allreduce_buffer_bytes.restype = L
+    sig("mfb_ll_allreduce_buffer_bytes", [I, L], L)
     sig("mfb_ll_allreduce_state_words", [])
     sig("mfb_ll_allreduce_init", [P, L, P])
     sig("mfb_ll_allreduce", [P, P, L, L, I, I, P, P, P, P])
@@ -138,11 +127,9 @@ def _declare(lib):
     sig("mfb_gemm_fp8_blockscaled", [P, P, P, P, L, P, I, I, I, L, L, L, I, I, P, P, P, P])
     sig("mfb_quant_act_1x128", [P, L, P, L, P, L, L, I, P])
     if hasattr(lib, "mfb_gemm_pair_set_band"):
-        lib.mfb_gemm_pair_set_band.argtypes = [I]
-        lib.mfb_gemm_pair_set_band.restype = None
+        sig("mfb_gemm_pair_set_band", [I], None)
     if hasattr(lib, "mfb_flash_attn_bwd2_set_probe"):
-        lib.mfb_flash_attn_bwd2_set_probe.argtypes = [I]
-        lib.mfb_flash_attn_bwd2_set_probe.restype = None
+        sig("mfb_flash_attn_bwd2_set_probe", [I], None)
     sig("mfb_reshape_and_cache_int8", [P, P, P, P, P, P, P, L, I, I, L, L, P])
     sig("mfb_gather_cache_int8", [P, P, P, P, P, I, I, I, I, I, I, P])
     sig("mfb_decode_advance", [P, I, I, I, P, P, P, P, P, I, I, P, I, P, P, P, P, P])
@@ -152,6 +139,16 @@ def _declare(lib):
     sig("mfb_paged_decode_attention_ex", [P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, F, P])
     sig("mfb_gemm_w8a8", [P, P, P, P, P, P, I, I, I, L, L, L, P, P])
     sig("mfb_quant_act_int8", [P, L, P, L, P, P, L, I, P])
+    sig("mfb_paged_decode_tc_supported_ex", [I, I, I, I, I])
+    sig("mfb_paged_decode_attention_tc_ex", [P] * 9 + [I] * 11 + [F, P, P])
+    sig("mfb_paged_prefill_tc_supported", [I, I, I, I, I])
+    sig("mfb_paged_prefill_tc", [P, P, P, P, I, P, P, P, P, P] + [I] * 9 + [F, P, P])
+    sig("mfb_paged_attention_any", [P] * 8 + [I] * 9 + [F, I, P])
+    sig("mfb_qkv_rope_cache", [P, L, P, P, P, F, P, F, I, I, P, P, P, P, P, I, I, I, I, I, I, P])
+    sig("mfb_add_normed", [P, L, P, P, P, P, P, I, P, P, I, I, I, F, I, P])
+    sig("mfb_norm_stream", [P, P, P, P, I, I, I, F, I, P])
+    sig("mfb_relu2", [P, P, L, I, L, I, P])
+    sig("mfb_softcap", [P, L, I, L, F, P])
     # optional entry points (present once their source file is part of the build)
     for name, args in _OPTIONAL.items():
         if hasattr(lib, name):
@@ -171,7 +168,15 @@ def optional_entry(name, args):
 
 
 def available() -> bool:
-    return os.path.exists(KERNEL_LIB_PATH)
+    return os.path.exists(_path)
+
+
+def use_library(path: str):
+    """Load the kernels from ``path`` (what ``build.ensure`` returned) instead of the full library."""
+    global _path
+    if _lib is not None and path != _path:
+        raise KernelLibraryError(f"the kernel library {_path} is loaded already")
+    _path = path
 
 
 def get_lib():
@@ -182,11 +187,11 @@ def get_lib():
     with _lock:
         if _lib is not None:
             return _lib
-        if not os.path.exists(KERNEL_LIB_PATH):
+        if not os.path.exists(_path):
             raise KernelLibraryError(
-                f"{KERNEL_LIB_PATH} is missing: run `python -m mindformers_b200.ops.build` "
+                f"{_path} is missing: run `python -m mindformers_b200.ops.build` "
                 "(the CUDA path never falls back to PyTorch on a GPU)")
-        lib = ctypes.CDLL(KERNEL_LIB_PATH)
+        lib = ctypes.CDLL(_path)
         got = lib.mfb_abi_version()
         if got != ABI_VERSION:
             raise KernelLibraryError(f"kernel library ABI {got} != expected {ABI_VERSION}; rebuild it")

@@ -40,7 +40,7 @@ def _digest(paths, extra=""):
     h = hashlib.sha256(extra.encode())
     for p in sorted(paths):
         with open(p, "rb") as f:
-            h.update(p.encode())
+            h.update(os.path.basename(p).encode())      # the same digest wherever the checkout lies
             h.update(f.read())
     return h.hexdigest()
 
@@ -62,23 +62,73 @@ def _compile_one(src: str, headers, log) -> str:
     return obj
 
 
+def _sources(names=None):
+    cu = sorted(f for f in os.listdir(CSRC) if f.endswith(".cu"))
+    if names is not None:
+        missing = sorted(set(names) - {f[:-3] for f in cu})
+        if missing:
+            raise ValueError(f"no kernel sources named {missing}")
+        cu = [f for f in cu if f[:-3] in names]
+    return [os.path.join(CSRC, f) for f in cu]
+
+
+def _headers():
+    return sorted(os.path.join(CSRC, f) for f in os.listdir(CSRC) if f.endswith((".cuh", ".h")))
+
+
+def _link(objs, out: str):
+    want = _digest(objs)
+    stamp = out + ".sha"
+    if os.path.exists(out) and os.path.exists(stamp) and open(stamp).read() == want:
+        return
+    cmd = [_nvcc(), "-shared", "-o", out + ".new"] + objs + ["-gencode", "arch=compute_100a,code=sm_100a"]
+    res = subprocess.run(cmd, capture_output=True, text=True)
+    if res.returncode != 0:
+        raise RuntimeError(f"link failed:\n{res.stderr[-4000:]}")
+    os.replace(out + ".new", out)
+    with open(stamp, "w") as f:
+        f.write(want)
+
+
+def _full_library_is_current() -> bool:
+    headers, objs = _headers(), []
+    for src in _sources():
+        obj = os.path.join(OBJ_DIR, os.path.splitext(os.path.basename(src))[0] + ".o")
+        stamp = obj + ".sha"
+        if not (os.path.exists(obj) and os.path.exists(stamp)
+                and open(stamp).read() == _digest([src] + headers, " ".join(NVCC_FLAGS))):
+            return False
+        objs.append(obj)
+    stamp = KERNEL_LIB + ".sha"
+    return os.path.exists(KERNEL_LIB) and os.path.exists(stamp) and open(stamp).read() == _digest(objs)
+
+
+def ensure(names=None, jobs: int | None = None) -> str:
+    """Path of a kernel library that holds the sources ``names`` (file names without extension; None: all), built if
+    need be: the full library when it is current, else a library of those sources alone, so that a program that serves
+    one model compiles what that model needs and no more. Objects are shared with ``build``."""
+    if names is None:
+        return build(jobs=jobs)["kernel_lib"]
+    if _full_library_is_current():
+        return KERNEL_LIB
+    os.makedirs(OBJ_DIR, exist_ok=True)
+    headers, log = _headers(), {}
+    with ThreadPoolExecutor(max_workers=jobs or min(8, os.cpu_count() or 2)) as ex:
+        objs = list(ex.map(lambda s: _compile_one(s, headers, log), _sources(names)))
+    key = hashlib.sha256(" ".join(sorted(names)).encode()).hexdigest()[:12]
+    out = os.path.join(LIB_DIR, f"libmfb200_{key}.so")
+    _link(objs, out)
+    return out
+
+
 def build(verbose: bool = False, jobs: int | None = None) -> dict:
     """Compile and link everything; returns {"kernel_lib": path, "data_lib": path}."""
     os.makedirs(OBJ_DIR, exist_ok=True)
-    cu = sorted(os.path.join(CSRC, f) for f in os.listdir(CSRC) if f.endswith(".cu"))
-    headers = sorted(os.path.join(CSRC, f) for f in os.listdir(CSRC) if f.endswith((".cuh", ".h")))
+    headers = _headers()
     log: dict = {}
     with ThreadPoolExecutor(max_workers=jobs or min(8, os.cpu_count() or 2)) as ex:
-        objs = list(ex.map(lambda s: _compile_one(s, headers, log), cu))
-    link_stamp = KERNEL_LIB + ".sha"
-    want = _digest(objs)
-    if not (os.path.exists(KERNEL_LIB) and os.path.exists(link_stamp) and open(link_stamp).read() == want):
-        cmd = [_nvcc(), "-shared", "-o", KERNEL_LIB] + objs + ["-gencode", "arch=compute_100a,code=sm_100a"]
-        res = subprocess.run(cmd, capture_output=True, text=True)
-        if res.returncode != 0:
-            raise RuntimeError(f"link failed:\n{res.stderr[-4000:]}")
-        with open(link_stamp, "w") as f:
-            f.write(want)
+        objs = list(ex.map(lambda s: _compile_one(s, headers, log), _sources()))
+    _link(objs, KERNEL_LIB)
     # CPU-side native helpers
     cpp = os.path.join(CSRC, "data_helpers.cpp")
     if os.path.exists(cpp):

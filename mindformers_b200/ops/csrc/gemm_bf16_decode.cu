@@ -15,7 +15,8 @@
 //   with fewer tiles than SMs the K range of a tile is split over the KS CTAs (2, 4 or 8) of a thread-block cluster,
 //   which reduce-scatter their 128 x NT partials through distributed shared memory (CTA c owns NT / KS token
 //   columns) and add them in rank order, so the result does not depend on timing;
-//   the result is written transposed, D[token j, n]: the 32 threads of a warp store 32 consecutive n of one token.
+//   the result is written transposed, D[token j, n]: the 32 threads of a warp store 32 consecutive n of one token;
+//   the epilogue can apply a squared relu or a tanh soft cap and can write fp32 (output heads).
 //
 // Roles (192 threads): warp 0 TMA producer, warp 1 MMA issuer and TMEM owner, warps 2..5 epilogue (one weight row per
 // thread). Every wait is bounded; after a timeout the status word is set and the CTA still runs through its cluster
@@ -31,10 +32,25 @@ constexpr int kWTile = 128 * 128;          // bytes of a weight stage: 128 rows 
 struct Args {
   int T, N, K, kblocks, n_tiles;
   const __nv_bfloat16* bias;      // [N] or null
-  __nv_bfloat16* D;
+  void* D;                        // bf16, or fp32 with out_f32
   long long ldd;
+  int out_f32;
+  int act;                        // 0 none, 1 max(x, 0)^2, 2 cap * tanh(x / cap)
+  float cap;
   int* status;
 };
+
+// activation and store of one output element; the value is rounded to bf16 once, at the store
+__device__ __forceinline__ void emit(const Args& a, long long idx, float v) {
+  if (a.act == 1) {
+    v = fmaxf(v, 0.f);
+    v *= v;
+  } else if (a.act == 2) {
+    v = a.cap * tanhf(v / a.cap);
+  }
+  if (a.out_f32) reinterpret_cast<float*>(a.D)[idx] = v;
+  else reinterpret_cast<__nv_bfloat16*>(a.D)[idx] = __float2bfloat16_rn(v);
+}
 
 // OCC = 2: half the stages, so that two CTAs share an SM (used when there are between one and two tiles per SM: all
 // of them are then resident at once and share the memory bandwidth evenly, instead of half the SMs doing two rounds).
@@ -210,7 +226,7 @@ gemm_bf16_decode_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_co
 #pragma unroll
           for (int j = 0; j < W; ++j) {
             const int t = krank * W + j;
-            if (t < args.T) args.D[(long long)t * args.ldd + n] = __float2bfloat16_rn(out[j] + bias);
+            if (t < args.T) emit(args, (long long)t * args.ldd + n, out[j] + bias);
           }
         }
         break;                                        // one tile per cluster
@@ -218,7 +234,7 @@ gemm_bf16_decode_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_co
         if (ok && n < args.N) {
 #pragma unroll
           for (int j = 0; j < NT; ++j)
-            if (j < args.T) args.D[(long long)j * args.ldd + n] = __float2bfloat16_rn(acc[j] + bias);
+            if (j < args.T) emit(args, (long long)j * args.ldd + n, acc[j] + bias);
         }
       }
     }
@@ -281,9 +297,10 @@ int mfb_gemm_bf16_decode_supported(int T, int N, int K) {
 
 // X [T, K] bf16 (row pitch ldx elements), W [N, K] bf16 (row pitch ldw), D [T, N] bf16 (row pitch ldd), bias [N] or null.
 // force_ks > 0 fixes the K split (1, 2, 4, 8) for measurements, force_ks 16 one tile per CTA with two CTAs per SM;
-// 0 lets the launcher choose.
-int mfb_gemm_bf16_decode(const void* X, const void* W, void* D, const void* bias, int T, int N, int K, long long ldx,
-                         long long ldw, long long ldd, int force_ks, int* status, cudaStream_t stream) {
+// 0 lets the launcher choose. out_f32: D is fp32. act: 0 none, 1 max(x, 0)^2, 2 cap * tanh(x / cap), after the bias.
+int mfb_gemm_bf16_decode_ex(const void* X, const void* W, void* D, const void* bias, int T, int N, int K, long long ldx,
+                            long long ldw, long long ldd, int force_ks, int out_f32, int act, float cap, int* status,
+                            cudaStream_t stream) {
   if (!mfb_gemm_bf16_decode_supported(T, N, K)) {
     mfb_host::set_error("gemm_bf16_decode: T=%d N=%d K=%d not supported", T, N, K);
     return 1;
@@ -296,7 +313,7 @@ int mfb_gemm_bf16_decode(const void* X, const void* W, void* D, const void* bias
   bd::Args a;
   a.T = T; a.N = N; a.K = K; a.kblocks = (K + 63) / 64; a.n_tiles = (N + 127) / 128;
   a.bias = reinterpret_cast<const __nv_bfloat16*>(bias);
-  a.D = reinterpret_cast<__nv_bfloat16*>(D); a.ldd = ldd; a.status = status;
+  a.D = D; a.ldd = ldd; a.status = status; a.out_f32 = out_f32; a.act = act; a.cap = cap;
   // Fewer tiles than SMs: split K over a cluster until about two thirds of the SMs stream (each slice keeping at
   // least 8 K blocks). Between one and two tiles per SM: two CTAs per SM, every tile resident at once. More: one
   // persistent CTA per SM, or two if that leaves the last round fuller.
@@ -319,6 +336,11 @@ int mfb_gemm_bf16_decode(const void* X, const void* W, void* D, const void* bias
   if (NT == 16) return bd::launch_ks<16>(tW, tX, a, ks, occ, stream);
   if (NT == 32) return bd::launch_ks<32>(tW, tX, a, ks, occ, stream);
   return bd::launch_ks<64>(tW, tX, a, ks, occ, stream);
+}
+
+int mfb_gemm_bf16_decode(const void* X, const void* W, void* D, const void* bias, int T, int N, int K, long long ldx,
+                         long long ldw, long long ldd, int force_ks, int* status, cudaStream_t stream) {
+  return mfb_gemm_bf16_decode_ex(X, W, D, bias, T, N, K, ldx, ldw, ldd, force_ks, 0, 0, 0.f, status, stream);
 }
 
 }  // extern "C"

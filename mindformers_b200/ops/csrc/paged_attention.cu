@@ -233,22 +233,32 @@ paged_decode_split_kernel(const __nv_bfloat16* __restrict__ q,        // [B, Hq,
   }
 }
 
-// out[b, h, :] = merge over splits of (acc, max, sum)
-template <int HD>
+// out[row, h, :] = merge over splits of (acc, max, sum). With cu_q [B + 1] the result of sequence b goes to row cu_q[b],
+// and only sequences with exactly one row are written; otherwise row b. sink [Hq] (or null) adds exp(sink_h) to the
+// denominator.
 __global__ void paged_combine_kernel(const float* __restrict__ part_acc, const float* __restrict__ part_ml,
-                                     __nv_bfloat16* __restrict__ out, int splits) {
+                                     __nv_bfloat16* __restrict__ out, int splits, int hd, int Hq,
+                                     const int* __restrict__ cu_q, const float* __restrict__ sink) {
   const size_t bh = blockIdx.x;
+  const int b = blockIdx.x / Hq, h = blockIdx.x - b * Hq;
+  size_t row = b;
+  if (cu_q) {
+    row = cu_q[b];
+    if (cu_q[b + 1] - cu_q[b] != 1) return;
+  }
   const int d = threadIdx.x;
-  float mx = -INFINITY;
+  if (d >= hd) return;
+  const float sk = sink ? sink[h] * 1.4426950408889634f : -INFINITY;
+  float mx = sk;
   for (int s2 = 0; s2 < splits; ++s2) mx = fmaxf(mx, part_ml[(bh * splits + s2) * 2]);
-  float num = 0.f, den = 0.f;
+  float num = 0.f, den = sink ? exp2f(sk - mx) : 0.f;
   for (int s2 = 0; s2 < splits; ++s2) {
     const float ms = part_ml[(bh * splits + s2) * 2];
     const float w = ms == -INFINITY ? 0.f : exp2f(ms - mx);
-    num += w * part_acc[(bh * splits + s2) * HD + d];
+    num += w * part_acc[(bh * splits + s2) * hd + d];
     den += w * part_ml[(bh * splits + s2) * 2 + 1];
   }
-  out[bh * HD + d] = __float2bfloat16(den > 0.f ? num / den : 0.f);
+  out[(row * Hq + h) * hd + d] = __float2bfloat16(den > 0.f ? num / den : 0.f);
 }
 
 // out[t, :] = cache[slot(t), :] gathered through the block table: token i of sequence b for i < lens[b],
@@ -369,21 +379,21 @@ int mfb_paged_decode_attention_ex(const void* q, const void* key_cache, const vo
       part_ml, Hq, Hkv, block_size, max_blocks, chunk, scale)
   if (hd == 128) {
     if (i8) MFB_PA_LAUNCH(128, true); else MFB_PA_LAUNCH(128, false);
-    paged_combine_kernel<128><<<B * Hq, 128, 0, stream>>>(part_acc, part_ml, (__nv_bfloat16*)out, splits);
+    paged_combine_kernel<<<B * Hq, 128, 0, stream>>>(part_acc, part_ml, (__nv_bfloat16*)out, splits, 128, Hq, nullptr, nullptr);
   } else {
     if (i8) MFB_PA_LAUNCH(64, true); else MFB_PA_LAUNCH(64, false);
-    paged_combine_kernel<64><<<B * Hq, 64, 0, stream>>>(part_acc, part_ml, (__nv_bfloat16*)out, splits);
+    paged_combine_kernel<<<B * Hq, 64, 0, stream>>>(part_acc, part_ml, (__nv_bfloat16*)out, splits, 64, Hq, nullptr, nullptr);
   }
 #undef MFB_PA_LAUNCH
   return cudaGetLastError() == cudaSuccess ? 0 : 2;
 }
 
-// out[row, :] = merge of the `splits` partial results of every (sequence, query head) row.
-int mfb_paged_combine(const float* part_acc, const float* part_ml, void* out, int splits, int rows, int hd,
-                      cudaStream_t stream) {
-  if (hd == 128) paged_combine_kernel<128><<<rows, 128, 0, stream>>>(part_acc, part_ml, (__nv_bfloat16*)out, splits);
-  else if (hd == 64) paged_combine_kernel<64><<<rows, 64, 0, stream>>>(part_acc, part_ml, (__nv_bfloat16*)out, splits);
-  else { mfb_host::set_error("paged_combine: head dim %d", hd); return 1; }
+// Merge of the `splits` partial results of every (sequence, query head): rows = sequences x Hq, hd up to 1024 columns.
+int mfb_paged_combine_ex(const float* part_acc, const float* part_ml, void* out, int splits, int rows, int hd, int Hq,
+                         const int* cu_q, const float* sink, cudaStream_t stream) {
+  if (hd < 1 || hd > 1024 || Hq < 1) { mfb_host::set_error("paged_combine: head dim %d", hd); return 1; }
+  paged_combine_kernel<<<rows, (hd + 31) / 32 * 32, 0, stream>>>(part_acc, part_ml, (__nv_bfloat16*)out, splits, hd, Hq, cu_q,
+                                                                sink);
   return cudaGetLastError() == cudaSuccess ? 0 : 2;
 }
 

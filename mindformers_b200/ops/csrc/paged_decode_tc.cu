@@ -1,8 +1,11 @@
-// Single-query (decode) attention over a paged bf16 KV cache on the tensor cores (sm_100a, tcgen05 + TMA), head
-// dim 128, grouped-query attention with up to 16 query heads per KV head.
+// Single-query (decode) attention over a paged bf16 KV cache on the tensor cores (sm_100a, tcgen05 + TMA), query / key
+// size and value size up to 128 each (multiples of 8), grouped-query attention (16 query heads of a KV head per CTA).
 //
-// Cache layout: key_cache / value_cache [num_blocks, block_size, kv_heads, 128]; a sequence's blocks come from its
-// block table. A CTA handles (split of the sequence, KV head, sequence) and walks its tokens in tiles of 128. As in
+// Cache layout: key_cache / value_cache [num_blocks, block_size, kv_heads, D | DV]; a sequence's blocks come from its
+// block table. With `chunk` > 0 only the keys of the query's own chunk of positions (counted from 0) are visited. The
+// tiles are 128 columns wide: q's columns past D are zero fill, so what a K tile holds there does not count, and the
+// value columns past DV reach only result rows that are not stored; 64-column halves that hold no head column are not
+// loaded. A CTA handles (split of the sequence, KV head, sequence) and walks its tokens in tiles of 128. As in
 // the latent-cache kernel the products are TRANSPOSED, so that the tokens, not the few query heads, fill the 128
 // rows of the tensor core:
 //     S^T [128 tokens x 16 heads] = K_tile [128 x 128] (A, K-major) . Q^T (B, K-major)            -> TMEM, 16 columns
@@ -41,9 +44,11 @@ constexpr int kSmem = kSlots * kUnit + kPBytes + kQBytes + 4 * kHeads * 4 + 16 *
 struct Args {
   const int* block_tables;   // [B, max_blocks]
   const int* context_lens;   // [B]
+  const int* cu_q;           // [B + 1] or null: only sequences with exactly one new row are computed, q row cu_q[b]
   int max_blocks, block_size, num_q_heads, num_kv_heads, group, splits;
+  int D, DV, chunk, head_blocks;   // head_blocks: CTAs of up to 16 query heads per KV head
   float scale_log2;
-  float* part_acc;           // [B, Hq, splits, 128] unnormalised
+  float* part_acc;           // [B, Hq, splits, DV] unnormalised
   float* part_ml;            // [B, Hq, splits, 2]: running max (log2 units), sum
   int* status;
 };
@@ -76,14 +81,26 @@ paged_decode_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_holder + 1);
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int split = blockIdx.x, kvh = blockIdx.y, b = blockIdx.z;
+  const int split = blockIdx.x, b = blockIdx.z;
+  const int kvh = static_cast<int>(blockIdx.y) / args.head_blocks, hb = static_cast<int>(blockIdx.y) % args.head_blocks;
+  int q_row = b;
+  if (args.cu_q) {
+    q_row = args.cu_q[b];
+    if (args.cu_q[b + 1] - q_row != 1) return;
+  }
   const int len = args.context_lens[b];
-  const int n_tiles_all = (len + kTile - 1) / kTile;
+  // first visible token: the start of the chunk that holds the query (position len - 1)
+  const int first_tok = (args.chunk > 0 && len > 0) ? len - 1 - (len - 1) % args.chunk : 0;
+  const int base_tile = first_tok / kTile;
+  const int n_tiles_all = (len + kTile - 1) / kTile - base_tile;
   const int per = (n_tiles_all + args.splits - 1) / args.splits;
-  const int t0 = split * per;
-  const int t1 = (t0 + per < n_tiles_all) ? t0 + per : n_tiles_all;
-  const int n_tiles = t1 > t0 ? t1 - t0 : 0;
-  const int head0 = kvh * args.group;
+  const int rel0 = split * per;
+  const int rel1 = (rel0 + per < n_tiles_all) ? rel0 + per : n_tiles_all;
+  const int n_tiles = rel1 > rel0 ? rel1 - rel0 : 0;
+  const int t0 = base_tile + rel0;
+  const int head0 = kvh * args.group + hb * kHeads;
+  const int n_heads = args.group - hb * kHeads < kHeads ? args.group - hb * kHeads : kHeads;
+  const int k_halves = args.D > 64 ? 2 : 1, v_halves = args.DV > 64 ? 2 : 1;
 
   if (threadIdx.x == 0) {
     *abort_flag = 0;
@@ -119,17 +136,16 @@ paged_decode_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
     // ------------------------------------ producer ------------------------------------
     if (lane == 0 && n_tiles > 0) {
       const uint32_t qb = smem_u32(q_full);
-      mbar_expect_tx(qb, kQBytes);
-      for (int c = 0; c < 2; ++c)
-        tma_load_2d(smem_u32(sQ) + c * (kHeads * 128), &tmQ, qb, c * 64, b * args.num_q_heads + head0);
+      mbar_expect_tx(qb, k_halves * (kHeads * 128));
+      for (int c = 0; c < k_halves; ++c)
+        tma_load_2d(smem_u32(sQ) + c * (kHeads * 128), &tmQ, qb, c * 64, q_row * args.num_q_heads + head0);
       const int bs = args.block_size;
       const int pages = kTile / bs;               // pages per tile (block_size divides 128)
       const int* table = args.block_tables + static_cast<size_t>(b) * args.max_blocks;
-      const int col0 = kvh * kHd;
       uint32_t unit = 0;
       bool ok = true;
       // one K or V tile into the next ring slot
-      auto load_tile = [&](const CUtensorMap* tm, int j) {
+      auto load_tile = [&](const CUtensorMap* tm, int j, int col0, int halves) {
         const int slot = unit % kSlots;
         const uint32_t ph = (unit / kSlots) & 1;
         ok = mbar_wait(smem_u32(&empty[slot]), ph ^ 1, abort_flag, args.status, kStatusWaitTimeoutProducer);
@@ -138,20 +154,21 @@ paged_decode_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
         const int first_page = table[tok0 / bs];
         const uint32_t fb = smem_u32(&full[slot]);
         const uint32_t dst = smem_u32(sRing + slot * kUnit);
-        mbar_expect_tx(fb, kUnit);
+        mbar_expect_tx(fb, halves * kSub);
         for (int i = 0; i < pages; ++i) {
           // pages past the end of the sequence may be unallocated: read the tile's first page instead (masked)
           int pg = (tok0 + i * bs < len) ? table[tok0 / bs + i] : first_page;
           if (pg < 0) pg = first_page;
           tma_load_2d(dst + i * bs * 128, tm, fb, col0, pg * bs);
-          tma_load_2d(dst + kSub + i * bs * 128, tm, fb, col0 + 64, pg * bs);
+          if (halves > 1) tma_load_2d(dst + kSub + i * bs * 128, tm, fb, col0 + 64, pg * bs);
         }
         ++unit;
       };
-      load_tile(&tmK, 0);
+      const int kcol = kvh * args.D, vcol = kvh * args.DV;
+      load_tile(&tmK, 0, kcol, k_halves);
       for (int j = 0; j < n_tiles && ok; ++j) {
-        if (j + 1 < n_tiles) load_tile(&tmK, j + 1);
-        if (ok) load_tile(&tmV, j);
+        if (j + 1 < n_tiles) load_tile(&tmK, j + 1, kcol, k_halves);
+        if (ok) load_tile(&tmV, j, vcol, v_halves);
       }
     }
     __syncwarp();
@@ -177,6 +194,7 @@ paged_decode_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
         const uint32_t ka = smem_u32(sRing + slot * kUnit);
 #pragma unroll
         for (int k = 0; k < 8; ++k) {
+          if (k >= 4 * k_halves) break;
           const uint64_t a_desc = umma_desc_kmajor_sw128(ka + (k >> 2) * kSub + (k & 3) * 32);
           const uint64_t b_desc = umma_desc_kmajor_sw128(qa + (k >> 2) * (kHeads * 128) + (k & 3) * 32);
           umma_f16_ss(tmem_S + sb * 32, a_desc, b_desc, IDESC_S, k > 0 ? 1u : 0u);
@@ -232,7 +250,8 @@ paged_decode_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       tc_fence_before();
       mbar_arrive(smem_u32(&s_empty[sb]));
       float s[kHeads];
-      const bool valid = (t0 + j) * kTile + row < len;
+      const int tok = (t0 + j) * kTile + row;
+      const bool valid = tok < len && tok >= first_tok;
 #pragma unroll
       for (int h = 0; h < kHeads; ++h) s[h] = valid ? __uint_as_float(sr[h]) * args.scale_log2 : -INFINITY;
       // per-head maximum over the 128 tokens of the tile
@@ -306,7 +325,7 @@ paged_decode_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
     for (int h = 0; h < kHeads; ++h)
       l_tot[h] = (red[h] + red[kHeads + h]) + (red[2 * kHeads + h] + red[3 * kHeads + h]);
     const bool have = ok && n_tiles > 0;
-    if (row < args.group) {
+    if (row < n_heads) {
       float mh = -INFINITY, lh = 0.f;
 #pragma unroll
       for (int h = 0; h < kHeads; ++h)
@@ -324,8 +343,8 @@ paged_decode_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
     }
 #pragma unroll
     for (int h = 0; h < kHeads; ++h) {
-      if (h < args.group)      // a split without tokens writes zeros: the merge multiplies them by a zero weight
-        args.part_acc[((static_cast<size_t>(b) * args.num_q_heads + head0 + h) * args.splits + split) * kHd + row] =
+      if (h < n_heads && row < args.DV)      // a split without tokens writes zeros: the merge multiplies them by a zero weight
+        args.part_acc[((static_cast<size_t>(b) * args.num_q_heads + head0 + h) * args.splits + split) * args.DV + row] =
             have ? __uint_as_float(r[h]) : 0.f;
     }
   }
@@ -343,14 +362,20 @@ paged_decode_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
 extern "C" {
 using namespace mfb;
 
-int mfb_paged_combine(const float* part_acc, const float* part_ml, void* out, int splits, int rows, int hd,
-                      cudaStream_t stream);      // paged_attention.cu
+int mfb_paged_combine_ex(const float* part_acc, const float* part_ml, void* out, int splits, int rows, int hd, int Hq,
+                         const int* cu_q, const float* sink, cudaStream_t stream);      // paged_attention.cu
 
-// 1 when the tensor-core kernel serves these shapes (bf16 cache, head dim 128, at most 16 query heads per KV head,
-// block size 16 / 32 / 64 / 128).
+// 1 when the tensor-core kernel serves these shapes (bf16 cache): sizes are multiples of 8 up to 128, the block size is
+// 16, 32, 64 or 128. Any number of query heads per KV head: a CTA takes 16 of them.
+int mfb_paged_decode_tc_supported_ex(int Hq, int Hkv, int D, int DV, int block_size) {
+  if (Hkv < 1 || Hq < 1 || Hq % Hkv || D < 8 || DV < 8 || D > 128 || DV > 128 || D % 8 || DV % 8) return 0;
+  return (block_size == 16 || block_size == 32 || block_size == 64 || block_size == 128) ? 1 : 0;
+}
+
+// The head-dim-128 subset with at most 16 query heads per KV head.
 int mfb_paged_decode_tc_supported(int Hq, int Hkv, int hd, int block_size) {
   if (hd != 128 || Hkv < 1 || Hq % Hkv || Hq / Hkv > pdt::kHeads) return 0;
-  return (block_size == 16 || block_size == 32 || block_size == 64 || block_size == 128) ? 1 : 0;
+  return mfb_paged_decode_tc_supported_ex(Hq, Hkv, hd, hd, block_size);
 }
 
 // Number of sequence splits that fills the GPU for B sequences of up to max_len tokens.
@@ -368,30 +393,36 @@ int mfb_paged_decode_tc_splits(int B, int Hkv, int max_len) {
   return best;
 }
 
-// q [B, Hq, 128] bf16, caches [num_blocks, block_size, Hkv, 128] bf16, out [B, Hq, 128] bf16; scratch as for
-// mfb_paged_decode_attention (mfb_paged_decode_scratch_bytes with the same splits).
-int mfb_paged_decode_attention_tc(const void* q, const void* key_cache, const void* value_cache, const int* block_tables,
-                                  const int* context_lens, void* out, void* scratch, int splits, int B, int Hq, int Hkv,
-                                  int num_blocks, int block_size, int max_blocks, float scale, int* status,
-                                  cudaStream_t stream) {
-  if (!mfb_paged_decode_tc_supported(Hq, Hkv, 128, block_size) || splits < 1 || num_blocks < 1) {
-    mfb_host::set_error("paged_decode_tc: unsupported Hq=%d Hkv=%d block_size=%d splits=%d", Hq, Hkv, block_size, splits);
+// q [rows, Hq, D] bf16, caches [num_blocks, block_size, Hkv, D | DV] bf16, out [rows, Hq, DV] bf16; scratch as for
+// mfb_paged_decode_attention (mfb_paged_decode_scratch_bytes(B, Hq, DV, splits)). cu_q null: row b belongs to sequence b
+// (rows == B); else [B + 1] row boundaries of a ragged batch, of which only the sequences with one row are computed and
+// written. chunk > 0: keys of the query's own chunk of positions only. sink: [Hq] fp32 or null, adds exp(sink) to the
+// softmax denominator.
+int mfb_paged_decode_attention_tc_ex(const void* q, const void* key_cache, const void* value_cache, const int* block_tables,
+                                     const int* context_lens, const int* cu_q, const float* sink, void* out, void* scratch,
+                                     int splits, int rows, int B, int Hq, int Hkv, int D, int DV, int num_blocks,
+                                     int block_size, int max_blocks, int chunk, float scale, int* status,
+                                     cudaStream_t stream) {
+  if (!mfb_paged_decode_tc_supported_ex(Hq, Hkv, D, DV, block_size) || splits < 1 || num_blocks < 1 || (!cu_q && rows != B)) {
+    mfb_host::set_error("paged_decode_tc: unsupported Hq=%d Hkv=%d D=%d DV=%d block_size=%d splits=%d", Hq, Hkv, D, DV,
+                        block_size, splits);
     return 1;
   }
-  if (B <= 0) return 0;
+  if (B <= 0 || rows <= 0) return 0;
   CUtensorMap tQ, tK, tV;
   int rc;
   const CUtensorMapDataType BF = CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
-  const uint64_t rows = (uint64_t)num_blocks * block_size, pitch = (uint64_t)Hkv * pdt::kHd;
-  if ((rc = mfb_host::make_tmap_2d(&tQ, q, 2, BF, (uint64_t)B * Hq, pdt::kHd, pdt::kHd, pdt::kHeads, 64))) return 20 + rc;
-  if ((rc = mfb_host::make_tmap_2d(&tK, key_cache, 2, BF, rows, pitch, pitch, block_size, 64))) return 30 + rc;
-  if ((rc = mfb_host::make_tmap_2d(&tV, value_cache, 2, BF, rows, pitch, pitch, block_size, 64))) return 40 + rc;
+  const uint64_t slots = (uint64_t)num_blocks * block_size, kp = (uint64_t)Hkv * D, vp = (uint64_t)Hkv * DV;
+  if ((rc = mfb_host::make_tmap_2d(&tQ, q, 2, BF, (uint64_t)rows * Hq, D, D, pdt::kHeads, 64))) return 20 + rc;
+  if ((rc = mfb_host::make_tmap_2d(&tK, key_cache, 2, BF, slots, kp, kp, block_size, 64))) return 30 + rc;
+  if ((rc = mfb_host::make_tmap_2d(&tV, value_cache, 2, BF, slots, vp, vp, block_size, 64))) return 40 + rc;
   pdt::Args a;
-  a.block_tables = block_tables; a.context_lens = context_lens; a.max_blocks = max_blocks; a.block_size = block_size;
-  a.num_q_heads = Hq; a.num_kv_heads = Hkv; a.group = Hq / Hkv; a.splits = splits;
+  a.block_tables = block_tables; a.context_lens = context_lens; a.cu_q = cu_q; a.max_blocks = max_blocks;
+  a.block_size = block_size; a.num_q_heads = Hq; a.num_kv_heads = Hkv; a.group = Hq / Hkv; a.splits = splits;
+  a.D = D; a.DV = DV; a.chunk = chunk; a.head_blocks = (a.group + pdt::kHeads - 1) / pdt::kHeads;
   a.scale_log2 = scale * 1.4426950408889634f;
   a.part_acc = reinterpret_cast<float*>(scratch);
-  a.part_ml = a.part_acc + static_cast<size_t>(B) * Hq * splits * pdt::kHd;
+  a.part_ml = a.part_acc + static_cast<size_t>(B) * Hq * splits * DV;
   a.status = status;
   static bool attr_set = false;
   if (!attr_set) {
@@ -401,10 +432,20 @@ int mfb_paged_decode_attention_tc(const void* q, const void* key_cache, const vo
     }
     attr_set = true;
   }
-  dim3 grid(splits, Hkv, B);
+  dim3 grid(splits, Hkv * a.head_blocks, B);
   pdt::paged_decode_tc_kernel<<<grid, pdt::kThreads, pdt::kSmem, stream>>>(tQ, tK, tV, a);
   if (cudaGetLastError() != cudaSuccess) { mfb_host::set_error("paged_decode_tc: launch failed"); return 11; }
-  return mfb_paged_combine(a.part_acc, a.part_ml, out, splits, B * Hq, pdt::kHd, stream);
+  return mfb_paged_combine_ex(a.part_acc, a.part_ml, out, splits, B * Hq, DV, Hq, cu_q, sink, stream);
+}
+
+// q [B, Hq, 128], caches [num_blocks, block_size, Hkv, 128], out [B, Hq, 128]: one row per sequence, no chunks, no sink.
+int mfb_paged_decode_attention_tc(const void* q, const void* key_cache, const void* value_cache, const int* block_tables,
+                                  const int* context_lens, void* out, void* scratch, int splits, int B, int Hq, int Hkv,
+                                  int num_blocks, int block_size, int max_blocks, float scale, int* status,
+                                  cudaStream_t stream) {
+  return mfb_paged_decode_attention_tc_ex(q, key_cache, value_cache, block_tables, context_lens, nullptr, nullptr, out, scratch,
+                                          splits, B, B, Hq, Hkv, pdt::kHd, pdt::kHd, num_blocks, block_size, max_blocks, 0,
+                                          scale, status, stream);
 }
 
 }  // extern "C"

@@ -1,0 +1,508 @@
+// Prefill attention of a ragged batch over a paged bf16 cache on the tensor cores (sm_100a, tcgen05 + TMA), grouped-query
+// attention with query / key size and value size up to 128 each (multiples of 8), optional chunked mask and softmax sink.
+//
+// Sequence b brings the rows cu_q[b] .. cu_q[b + 1] - 1 of q; its keys and values, those rows included, are in the cache
+// already, so a whole prompt, a later portion of a prompt and any mix of sequences are the same problem: row r of the
+// portion sits at position context_lens[b] - q_len + r and sees keys up to itself, with `chunk` > 0 only those of its
+// own chunk of `chunk` positions (counted from position 0). `sink` [Hq] adds exp(sink_h) to the denominator.
+//
+// The tensor-core pipeline is the one of flash_attention_fwd2.cu: a CTA owns up to 256 query rows of one head as two
+// 128-row tiles that share the key / value tiles; every tile has a softmax warpgroup; P goes back into tensor memory
+// and is read from there by the P V product. What differs:
+//   - work comes as a list of (sequence, first row of a 256-row pair); only key tiles that some row of a tile sees are
+//     visited, from the chunk of its first row to its last row;
+//   - K / V tiles (128 consecutive positions) are assembled from the sequence's pages, one TMA box per page and 64
+//     columns; pages past the end of the sequence repeat the tile's first page and are masked;
+//   - head sizes are padded to 64 or 128 columns: q is read through a three-dimensional map that fills the columns past
+//     the head with zeros, so whatever a K box holds there does not count; columns of V past the head reach only
+//     columns of the result that are not stored;
+//   - the result is staged in shared memory and written row by row: a portion may end anywhere.
+//
+// Roles (320 threads): warp 0 TMA producer, warp 1 MMA issuer + TMEM owner, warps 2..5 softmax of tile A, warps 6..9
+// softmax of tile B. Every wait is bounded (common.cuh).
+#include "common.cuh"
+
+namespace mfb {
+namespace ppt {
+
+constexpr int kThreads = 320;
+constexpr int kTile = 128;
+constexpr int kSubBytes = kTile * 128;     // [128 rows][128 B] swizzled sub-tile (64 bf16 columns)
+constexpr float kRescaleThreshold = 8.0f;  // log2 units
+
+struct Args {
+  const int* work;           // [n_work, 2]: sequence, first row of the pair inside the portion
+  const int* cu_q;           // [B + 1]
+  const int* block_tables;   // [B, max_blocks]
+  const int* context_lens;   // [B]
+  const float* sink;         // [Hq] or null
+  __nv_bfloat16* out;        // [T, Hq, DV]
+  int num_q_heads, group, D, DV, block_size, max_blocks, chunk;
+  float scale_log2;
+  int* status;
+};
+
+__device__ __forceinline__ float ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ uint64_t pack2(float lo, float hi) {
+  uint64_t r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(lo), "f"(hi));
+  return r;
+}
+__device__ __forceinline__ void unpack2(uint64_t v, float& lo, float& hi) {
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(v));
+}
+__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
+  uint64_t d;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+  return d;
+}
+__device__ __forceinline__ uint64_t add2(uint64_t a, uint64_t b) {
+  uint64_t d;
+  asm("add.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+  return d;
+}
+__device__ __forceinline__ float fmax3(float a, float b, float c) {
+  float d;
+  asm("max.f32 %0, %1, %2, %3;" : "=f"(d) : "f"(a), "f"(b), "f"(c));
+  return d;
+}
+__device__ __forceinline__ void tmem_st_32x32b_x32(uint32_t taddr, const uint32_t* r) {
+  asm volatile(
+      "tcgen05.st.sync.aligned.32x32b.x32.b32 [%0], "
+      "{%1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15, %16,"
+      " %17, %18, %19, %20, %21, %22, %23, %24, %25, %26, %27, %28, %29, %30, %31, %32};\n"
+      ::"r"(taddr), "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]), "r"(r[7]),
+        "r"(r[8]), "r"(r[9]), "r"(r[10]), "r"(r[11]), "r"(r[12]), "r"(r[13]), "r"(r[14]), "r"(r[15]),
+        "r"(r[16]), "r"(r[17]), "r"(r[18]), "r"(r[19]), "r"(r[20]), "r"(r[21]), "r"(r[22]), "r"(r[23]),
+        "r"(r[24]), "r"(r[25]), "r"(r[26]), "r"(r[27]), "r"(r[28]), "r"(r[29]), "r"(r[30]), "r"(r[31])
+      : "memory");
+}
+
+// HQ: padded query / key size, HV: padded value size (64 or 128)
+template <int HQ, int HV>
+__global__ void __launch_bounds__(kThreads, 1)
+paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
+                        const __grid_constant__ CUtensorMap tmV, const Args args) {
+  constexpr int QB = HQ / 64, VB = HV / 64;          // 64-column sub-tiles
+  constexpr int kQBytes = QB * kSubBytes, kVBytes = VB * kSubBytes;
+  constexpr int kStage = kQBytes > kVBytes ? kQBytes : kVBytes;   // a Q tile's buffer also stages its result
+  extern __shared__ uint8_t smem_raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) &
+                                             ~static_cast<uintptr_t>(1023));
+  uint8_t* sQ = smem;                         // 2 tiles (A, B)
+  uint8_t* sK = sQ + 2 * kStage;              // 2 stages
+  uint8_t* sV = sK + 2 * kQBytes;             // 2 stages
+  uint64_t* bars = reinterpret_cast<uint64_t*>(sV + 2 * kVBytes);
+  uint64_t* q_full = bars;          // 1
+  uint64_t* k_full = bars + 1;      // 2
+  uint64_t* k_empty = bars + 3;     // 2
+  uint64_t* v_full = bars + 5;      // 2
+  uint64_t* v_empty = bars + 7;     // 2
+  uint64_t* s_full = bars + 9;      // 2: S of tile A / B complete
+  uint64_t* p_ready = bars + 11;    // 2: P of tile A / B written (128 arrivals)
+  uint64_t* pv_done = bars + 13;    // 2: P V of tile A / B complete
+  uint32_t* tmem_holder = reinterpret_cast<uint32_t*>(bars + 15);
+  volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_holder + 1);
+
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int head = static_cast<int>(blockIdx.x) % args.num_q_heads;
+  const int item = static_cast<int>(blockIdx.x) / args.num_q_heads;
+  const int b = args.work[2 * item], pair_row = args.work[2 * item + 1];
+  const int q0 = args.cu_q[b];
+  const int q_len = args.cu_q[b + 1] - q0;
+  const int len = args.context_lens[b];
+  const int pos0 = len - q_len;                      // position of the portion's first row
+  const int kv_head = head / args.group;
+  int n_kv_x[2], lo_x[2], rows_x[2];   // tile x: rows_x[x] rows, key tiles lo_x[x] .. n_kv_x[x] - 1
+#pragma unroll
+  for (int x = 0; x < 2; ++x) {
+    const int r0 = pair_row + x * kTile;
+    int rows = q_len - r0;
+    rows = rows < 0 ? 0 : (rows > kTile ? kTile : rows);
+    rows_x[x] = rows;
+    const int first = pos0 + r0;
+    lo_x[x] = (rows > 0 && args.chunk > 0) ? (first - first % args.chunk) / kTile : 0;
+    n_kv_x[x] = rows > 0 ? (first + rows - 1) / kTile + 1 : 0;
+  }
+  const int n_kv = n_kv_x[0] > n_kv_x[1] ? n_kv_x[0] : n_kv_x[1];
+  const int lo = lo_x[0];              // positions grow with the rows: tile A starts first
+
+  if (threadIdx.x == 0) {
+    *abort_flag = 0;
+    mbar_init(smem_u32(q_full), 1);
+    for (int s = 0; s < 2; ++s) {
+      mbar_init(smem_u32(&k_full[s]), 1);
+      mbar_init(smem_u32(&k_empty[s]), 1);
+      mbar_init(smem_u32(&v_full[s]), 1);
+      mbar_init(smem_u32(&v_empty[s]), 1);
+      mbar_init(smem_u32(&s_full[s]), 1);
+      mbar_init(smem_u32(&p_ready[s]), 128);
+      mbar_init(smem_u32(&pv_done[s]), 1);
+    }
+    fence_barrier_init();
+    tma_prefetch_desc(&tmQ);
+    tma_prefetch_desc(&tmK);
+    tma_prefetch_desc(&tmV);
+  }
+  if (warp == 1) {
+    tmem_alloc(smem_u32(tmem_holder), 512);
+    tmem_relinquish();
+  }
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem_base = *tmem_holder;
+  // S_A +0, S_B +128, O_A +256, O_B +384; P_X lives in the first 64 columns of S_X
+  if (warp == 0) {
+    // ------------------------------ TMA producer ------------------------------
+    if (lane == 0 && n_kv > 0) {
+      const uint32_t qb = smem_u32(q_full);
+      const int n_tiles_here = rows_x[1] > 0 ? 2 : 1;
+      mbar_expect_tx(qb, n_tiles_here * kQBytes);
+      for (int x = 0; x < n_tiles_here; ++x)
+        for (int c = 0; c < QB; ++c)
+          tma_load_3d(smem_u32(sQ) + x * kStage + c * kSubBytes, &tmQ, qb, c * 64, head, q0 + pair_row + x * kTile);
+      const int bs = args.block_size;
+      const int pages = kTile / bs;
+      const int* table = args.block_tables + static_cast<size_t>(b) * args.max_blocks;
+      const int kcol = kv_head * args.D, vcol = kv_head * args.DV;
+      bool ok = true;
+      for (int j = lo; j < n_kv && ok; ++j) {
+        const int st = (j - lo) & 1;
+        const uint32_t ph = ((j - lo) >> 1) & 1;
+        const int tok0 = j * kTile;
+        const int first_page = table[tok0 / bs];
+        ok = mbar_wait(smem_u32(&k_empty[st]), ph ^ 1, abort_flag, args.status, kStatusWaitTimeoutProducer);
+        if (!ok) break;
+        const uint32_t kb = smem_u32(&k_full[st]);
+        mbar_expect_tx(kb, kQBytes);
+        const uint32_t kd = smem_u32(sK + st * kQBytes);
+        for (int i = 0; i < pages; ++i) {
+          const int pg = tok0 + i * bs < len ? table[tok0 / bs + i] : first_page;
+          for (int c = 0; c < QB; ++c) tma_load_2d(kd + c * kSubBytes + i * bs * 128, &tmK, kb, kcol + c * 64, pg * bs);
+        }
+        ok = mbar_wait(smem_u32(&v_empty[st]), ph ^ 1, abort_flag, args.status, kStatusWaitTimeoutProducer);
+        if (!ok) break;
+        const uint32_t vb = smem_u32(&v_full[st]);
+        mbar_expect_tx(vb, kVBytes);
+        const uint32_t vd = smem_u32(sV + st * kVBytes);
+        for (int i = 0; i < pages; ++i) {
+          const int pg = tok0 + i * bs < len ? table[tok0 / bs + i] : first_page;
+          for (int c = 0; c < VB; ++c) tma_load_2d(vd + c * kSubBytes + i * bs * 128, &tmV, vb, vcol + c * 64, pg * bs);
+        }
+      }
+    }
+    __syncwarp();
+  } else if (warp == 1) {
+    // ------------------------------ MMA issuer ------------------------------
+    if (lane == 0 && n_kv > 0) {
+      constexpr uint32_t IDESC_QK = umma_idesc_bf16(kTile, kTile, 0, 0);  // A = Q K-major (smem), B = K K-major
+      constexpr uint32_t IDESC_PV = umma_idesc_bf16(kTile, HV, 0, 1);     // A = P (tensor memory), B = V MN-major
+      auto issue_qk = [&](int x, int j) {
+        const uint32_t qa = smem_u32(sQ) + x * kStage;
+        const uint32_t ka = smem_u32(sK) + ((j - lo) & 1) * kQBytes;
+#pragma unroll
+        for (int k = 0; k < HQ / 16; ++k) {
+          const uint32_t off = (k >> 2) * kSubBytes + (k & 3) * 32;
+          umma_f16_ss(tmem_base + x * kTile, umma_desc_kmajor_sw128(qa + off), umma_desc_kmajor_sw128(ka + off),
+                      IDESC_QK, k > 0 ? 1u : 0u);
+        }
+        umma_commit(smem_u32(&s_full[x]));
+      };
+      bool ok = mbar_wait(smem_u32(q_full), 0, abort_flag, args.status, kStatusWaitTimeoutMma);
+      auto active = [&](int x, int j) { return j >= lo_x[x] && j < n_kv_x[x]; };
+      if (ok) {
+        ok = mbar_wait(smem_u32(&k_full[0]), 0, abort_flag, args.status, kStatusWaitTimeoutMma);
+        if (ok) {
+          tc_fence_after();
+          if (active(0, lo)) issue_qk(0, lo);
+          if (active(1, lo)) issue_qk(1, lo);
+          umma_commit(smem_u32(&k_empty[0]));
+        }
+      }
+      for (int j = lo; j < n_kv && ok; ++j) {
+        const int st = (j - lo) & 1;
+        const uint32_t ph = ((j - lo) >> 1) & 1;
+        ok = mbar_wait(smem_u32(&v_full[st]), ph, abort_flag, args.status, kStatusWaitTimeoutMma);
+        if (!ok) break;
+        bool k_next_waited = false;
+#pragma unroll
+        for (int x = 0; x < 2; ++x) {
+          const bool pv_now = active(x, j), qk_next = active(x, j + 1);
+          if (pv_now) {
+            ok = mbar_wait(smem_u32(&p_ready[x]), (j - lo_x[x]) & 1, abort_flag, args.status, kStatusWaitTimeoutMma);
+            if (!ok) break;
+            tc_fence_after();
+            const uint32_t va = smem_u32(sV) + st * kVBytes;
+            const uint32_t p_tmem = tmem_base + x * kTile;          // bf16 pairs: 8 columns per 16 keys
+            const uint32_t o_tmem = tmem_base + 256 + x * kTile;
+#pragma unroll
+            for (int k = 0; k < kTile / 16; ++k) {
+              const uint64_t b_desc = umma_desc_mnmajor_sw128(va + k * 16 * 128, kSubBytes);
+              umma_f16_ts(o_tmem, p_tmem + k * 8, b_desc, IDESC_PV, (j > lo_x[x] || k > 0) ? 1u : 0u);
+            }
+            umma_commit(smem_u32(&pv_done[x]));
+          }
+          if (qk_next) {
+            if (!k_next_waited) {
+              ok = mbar_wait(smem_u32(&k_full[(j + 1 - lo) & 1]), ((j + 1 - lo) >> 1) & 1, abort_flag, args.status,
+                             kStatusWaitTimeoutMma);
+              if (!ok) break;
+              tc_fence_after();
+              k_next_waited = true;
+            }
+            issue_qk(x, j + 1);   // overwrites S_X / P_X: executes behind the P V product issued just above
+          }
+        }
+        if (!ok) break;
+        umma_commit(smem_u32(&v_empty[st]));
+        if (k_next_waited) umma_commit(smem_u32(&k_empty[(j + 1 - lo) & 1]));
+      }
+    }
+    __syncwarp();
+  } else {
+    // ------------------------------ softmax warpgroups ------------------------------
+    const int x = (warp - 2) >> 2;                 // 0 = tile A, 1 = tile B
+    const int ew = warp & 3;                       // TMEM lane quarter of this warp
+    const int row = ew * 32 + lane;
+    const uint32_t lane_base = static_cast<uint32_t>(ew * 32) << 16;
+    const uint32_t s_tmem = tmem_base + x * kTile + lane_base;
+    const uint32_t o_tmem = tmem_base + 256 + x * kTile + lane_base;
+    const uint32_t bar_and = 2 + x;
+    const int my_n = n_kv_x[x], my_lo = lo_x[x];
+    const int my_pos = pos0 + pair_row + x * kTile + row;
+    const int my_first = args.chunk > 0 ? my_pos - my_pos % args.chunk : 0;   // first key this row may see
+    float m_used = -INFINITY, l_sum = 0.f;
+    bool ok = true;
+    const uint64_t scale2 = pack2(args.scale_log2, args.scale_log2);
+    for (int j = my_lo; j < my_n; ++j) {
+      ok = mbar_wait(smem_u32(&s_full[x]), (j - my_lo) & 1, abort_flag, args.status, kStatusWaitTimeoutEpilogue);
+      if (!ok) break;
+      tc_fence_after();
+      // columns [col_lo, col_hi] of this key tile are visible to the row (none, if the range is empty)
+      const int col_lo = my_first - j * kTile;
+      const int col_hi = my_pos - j * kTile;
+      const bool masked = __any_sync(0xffffffffu, col_lo > 0 || col_hi < kTile - 1);
+      // pass 1: row maximum (four independent chains of three-input maxima); the scores are not kept
+      float mxs[4];
+      {
+        uint32_t sr[kTile];
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+          uint32_t (&r)[32] = *reinterpret_cast<uint32_t(*)[32]>(&sr[c * 32]);
+          tmem_ld_32x32b_x32(s_tmem + c * 32, r);
+        }
+        tmem_ld_wait();
+        float* s = reinterpret_cast<float*>(sr);
+        if (masked) {
+#pragma unroll
+          for (int i = 0; i < kTile; ++i)
+            if (i > col_hi || i < col_lo) s[i] = -INFINITY;
+        }
+#pragma unroll
+        for (int a = 0; a < 4; ++a) {
+          float m = s[a * 32];
+#pragma unroll
+          for (int i = 1; i + 1 < 32; i += 2) m = fmax3(m, s[a * 32 + i], s[a * 32 + i + 1]);
+          mxs[a] = fmaxf(m, s[a * 32 + 31]);
+        }
+      }
+      float mx = fmaxf(fmaxf(mxs[0], mxs[1]), fmaxf(mxs[2], mxs[3]));
+      mx *= args.scale_log2;
+      float alpha = 1.f;
+      if (j == my_lo) {
+        m_used = mx;                               // -inf when this row sees nothing in its tile's first key tile
+      } else if (mx > m_used + kRescaleThreshold) {
+        alpha = ex2(m_used - mx);                  // 0 when nothing was accumulated yet
+        m_used = mx;
+      }
+      if (j > my_lo && __any_sync(0xffffffffu, alpha != 1.f)) {
+        // S(j) is complete, so every earlier P V product has finished; the next one waits for p_ready below:
+        // nobody else touches O now
+#pragma unroll
+        for (int c = 0; c < HV / 16; ++c) {
+          uint32_t r[16];
+          tmem_ld_32x32b_x16(o_tmem + c * 16, r);
+          tmem_ld_wait();
+#pragma unroll
+          for (int i = 0; i < 16; ++i) r[i] = __float_as_uint(__uint_as_float(r[i]) * alpha);
+          tmem_st_32x32b_x16(o_tmem + c * 16, r);
+        }
+      }
+      const float neg_m = (m_used == -INFINITY) ? 0.f : -m_used;
+      const uint64_t negm2 = pack2(neg_m, neg_m);
+      uint64_t rs2[4] = {0, 0, 0, 0};
+      // exp2 of the scaled, shifted scores two at a time; P goes back as bf16 pairs, 64 score columns (32 packed
+      // registers) per store, into the first 64 columns of this tile's S buffer
+#pragma unroll
+      for (int h = 0; h < 2; ++h) {
+        // pass 2: 64 scores at a time; the second half is read before the first half's P overwrites columns 0..31
+        uint32_t sr[64];
+        {
+          uint32_t (&ra)[32] = *reinterpret_cast<uint32_t(*)[32]>(&sr[0]);
+          uint32_t (&rb)[32] = *reinterpret_cast<uint32_t(*)[32]>(&sr[32]);
+          tmem_ld_32x32b_x32(s_tmem + h * 64, ra);
+          tmem_ld_32x32b_x32(s_tmem + h * 64 + 32, rb);
+          tmem_ld_wait();
+        }
+        float* s = reinterpret_cast<float*>(sr);
+        if (masked) {
+#pragma unroll
+          for (int i = 0; i < 64; ++i)
+            if (h * 64 + i > col_hi || h * 64 + i < col_lo) s[i] = -INFINITY;
+        }
+        uint32_t pk[32];
+#pragma unroll
+        for (int i = 0; i < 32; ++i) {
+          float t0, t1;
+          unpack2(fma2(pack2(s[2 * i], s[2 * i + 1]), scale2, negm2), t0, t1);
+          const float e0 = ex2(t0), e1 = ex2(t1);
+          rs2[i & 3] = add2(rs2[i & 3], pack2(e0, e1));
+          pk[i] = pack_bf16x2(e0, e1);
+        }
+        tmem_st_32x32b_x32(s_tmem + h * 32, pk);
+      }
+      float r0, r1, r2, r3;
+      unpack2(add2(rs2[0], rs2[1]), r0, r1);
+      unpack2(add2(rs2[2], rs2[3]), r2, r3);
+      l_sum = l_sum * alpha + ((r0 + r1) + (r2 + r3));
+      tmem_st_wait();
+      tc_fence_before();
+      mbar_arrive(smem_u32(&p_ready[x]));
+    }
+    if (my_n > 0) {
+      if (ok) ok = mbar_wait(smem_u32(&pv_done[x]), (my_n - 1 - my_lo) & 1, abort_flag, args.status, kStatusWaitTimeoutEpilogue);
+      // one decision for the whole warpgroup (a thread that gave up above still arrives here)
+      ok = named_bar_and(bar_and, 128, ok);
+      if (ok) {
+        tc_fence_after();
+        // the sink joins the denominator on the scale of the sum; an enormous sink overflows to a zero weight of the keys
+        const float den = args.sink ? l_sum + ex2(args.sink[head] * 1.4426950408889634f - m_used) : l_sum;
+        const float inv_l = 1.f / den;
+        // every MMA that read Q_X has completed: its shared memory now stages the warp's 32 rows
+        uint8_t* stage = sQ + x * kStage;
+        uint8_t* orow = stage + row * 128;
+#pragma unroll
+        for (int c = 0; c < HV / 32; ++c) {
+          uint32_t r[32];
+          tmem_ld_32x32b_x32(o_tmem + c * 32, r);
+          tmem_ld_wait();
+#pragma unroll
+          for (int q = 0; q < 4; ++q) {
+            const int chunk = c * 4 + q;
+            uint4 v = make_uint4(
+                pack_bf16x2(__uint_as_float(r[q * 8 + 0]) * inv_l, __uint_as_float(r[q * 8 + 1]) * inv_l),
+                pack_bf16x2(__uint_as_float(r[q * 8 + 2]) * inv_l, __uint_as_float(r[q * 8 + 3]) * inv_l),
+                pack_bf16x2(__uint_as_float(r[q * 8 + 4]) * inv_l, __uint_as_float(r[q * 8 + 5]) * inv_l),
+                pack_bf16x2(__uint_as_float(r[q * 8 + 6]) * inv_l, __uint_as_float(r[q * 8 + 7]) * inv_l));
+            *reinterpret_cast<uint4*>(orow + (chunk >> 3) * kSubBytes + (((chunk & 7) ^ (row & 7)) << 4)) = v;
+          }
+        }
+        __syncwarp();
+        const int rows = rows_x[x] - ew * 32;           // valid rows of this warp (may be negative)
+        const int vecs = args.DV / 8;
+        __nv_bfloat16* obase = args.out + (static_cast<size_t>(q0 + pair_row + x * kTile + ew * 32) * args.num_q_heads + head) * args.DV;
+        for (int i = lane; i < 32 * (HV / 8); i += 32) {
+          const int rr = i / (HV / 8), c = i % (HV / 8);
+          if (rr < rows && c < vecs) {
+            const int srow = ew * 32 + rr;
+            const uint4 v = *reinterpret_cast<const uint4*>(stage + srow * 128 + (c >> 3) * kSubBytes + (((c & 7) ^ (srow & 7)) << 4));
+            *reinterpret_cast<uint4*>(obase + static_cast<size_t>(rr) * args.num_q_heads * args.DV + c * 8) = v;
+          }
+        }
+      }
+    }
+  }
+  tc_fence_before();
+  __syncthreads();
+  if (warp == 1) {
+    tc_fence_after();
+    tmem_dealloc(tmem_base, 512);
+  }
+}
+
+// three-dimensional map of q [T, Hq, D]: box of 128 tokens x 1 head x 64 columns; columns past D read as zero
+int make_q_map(CUtensorMap* out, const void* q, uint64_t T, uint64_t Hq, uint64_t D) {
+  mfb_host::EncodeTiledFn enc = mfb_host::get_encode_tiled();
+  if (!enc) { mfb_host::set_error("cuTensorMapEncodeTiled entry point not available"); return 1; }
+  if ((reinterpret_cast<uintptr_t>(q) & 15) || (D * 2) % 16) { mfb_host::set_error("paged_prefill_tc: q not aligned"); return 2; }
+  cuuint64_t gdim[3] = {D, Hq, T};
+  cuuint64_t gstride[2] = {D * 2, Hq * D * 2};
+  cuuint32_t box[3] = {64, 1, kTile};
+  cuuint32_t estr[3] = {1, 1, 1};
+  const CUresult r = enc(out, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(q), gdim, gstride, box, estr,
+                         CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+                         CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  if (r != CUDA_SUCCESS) { mfb_host::set_error("paged_prefill_tc: tensor map of q failed (%d)", (int)r); return 3; }
+  return 0;
+}
+
+template <int HQ, int HV>
+int launch(const CUtensorMap& tQ, const CUtensorMap& tK, const CUtensorMap& tV, const Args& a, int grid, cudaStream_t stream) {
+  constexpr int QBYTES = HQ / 64 * kSubBytes, VBYTES = HV / 64 * kSubBytes;
+  constexpr int STAGE = QBYTES > VBYTES ? QBYTES : VBYTES;
+  constexpr int SMEM = 2 * STAGE + 2 * QBYTES + 2 * VBYTES + 16 * 8 + 16 + 1024;
+  static_assert(SMEM <= 232448, "shared memory budget exceeded");
+  auto kern = paged_prefill_tc_kernel<HQ, HV>;
+  static bool attr_set = false;
+  if (!attr_set) {
+    if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM) != cudaSuccess) {
+      mfb_host::set_error("paged_prefill_tc: cannot raise the shared memory limit");
+      return 10;
+    }
+    attr_set = true;
+  }
+  kern<<<grid, kThreads, SMEM, stream>>>(tQ, tK, tV, a);
+  if (cudaGetLastError() != cudaSuccess) { mfb_host::set_error("paged_prefill_tc: launch failed"); return 11; }
+  return 0;
+}
+
+}  // namespace ppt
+}  // namespace mfb
+
+extern "C" {
+using namespace mfb;
+
+// 1 when the kernel serves these shapes (bf16): sizes are multiples of 8 up to 128, the block size divides 128.
+int mfb_paged_prefill_tc_supported(int Hq, int Hkv, int D, int DV, int block_size) {
+  if (Hkv < 1 || Hq < 1 || Hq % Hkv || D < 8 || DV < 8 || D > 128 || DV > 128 || D % 8 || DV % 8) return 0;
+  return (block_size == 16 || block_size == 32 || block_size == 64 || block_size == 128) ? 1 : 0;
+}
+
+// q [T, Hq, D], caches [num_blocks, block_size, Hkv, D | DV], out [T, Hq, DV], all bf16. work [n_work, 2] int32: (sequence,
+// first row of a 256-row pair inside its portion), for every pair of every sequence whose rows this launch computes.
+int mfb_paged_prefill_tc(const void* q, const void* key_cache, const void* value_cache, const int* work, int n_work,
+                         const int* cu_q, const int* block_tables, const int* context_lens, const float* sink, void* out, int T,
+                         int Hq, int Hkv, int D, int DV, int num_blocks, int block_size, int max_blocks, int chunk, float scale,
+                         int* status, cudaStream_t stream) {
+  if (!mfb_paged_prefill_tc_supported(Hq, Hkv, D, DV, block_size) || num_blocks < 1 || T < 1) {
+    mfb_host::set_error("paged_prefill_tc: unsupported Hq=%d Hkv=%d D=%d DV=%d block_size=%d", Hq, Hkv, D, DV, block_size);
+    return 1;
+  }
+  if (n_work <= 0) return 0;
+  CUtensorMap tQ, tK, tV;
+  int rc;
+  const CUtensorMapDataType BF = CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
+  const uint64_t rows = (uint64_t)num_blocks * block_size;
+  if ((rc = mfb_host::make_tmap_2d(&tK, key_cache, 2, BF, rows, (uint64_t)Hkv * D, (uint64_t)Hkv * D, block_size, 64))) return 30 + rc;
+  if ((rc = mfb_host::make_tmap_2d(&tV, value_cache, 2, BF, rows, (uint64_t)Hkv * DV, (uint64_t)Hkv * DV, block_size, 64))) return 40 + rc;
+  if ((rc = ppt::make_q_map(&tQ, q, T, Hq, D))) return 20 + rc;
+  ppt::Args a;
+  a.work = work; a.cu_q = cu_q; a.block_tables = block_tables; a.context_lens = context_lens; a.sink = sink;
+  a.out = reinterpret_cast<__nv_bfloat16*>(out);
+  a.num_q_heads = Hq; a.group = Hq / Hkv; a.D = D; a.DV = DV; a.block_size = block_size; a.max_blocks = max_blocks;
+  a.chunk = chunk; a.scale_log2 = scale * 1.4426950408889634f; a.status = status;
+  const int grid = n_work * Hq;
+  if (D > 64) {
+    if (DV > 64) return ppt::launch<128, 128>(tQ, tK, tV, a, grid, stream);
+    return ppt::launch<128, 64>(tQ, tK, tV, a, grid, stream);
+  }
+  if (DV > 64) return ppt::launch<64, 128>(tQ, tK, tV, a, grid, stream);
+  return ppt::launch<64, 64>(tQ, tK, tV, a, grid, stream);
+}
+
+}  // extern "C"

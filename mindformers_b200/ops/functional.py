@@ -147,6 +147,9 @@ def gemm(a: torch.Tensor, b: torch.Tensor, *, a_mn: bool = False, b_mn: bool = F
         else:
             out.copy_(res)
         return out
+    if K % 8 and not a_mn and not b_mn:          # operand rows must be multiples of 16 bytes
+        a, b = F.pad(a, (0, -K % 8)), F.pad(b, (0, -K % 8))
+        K = a.shape[1]
     if not _aligned(a):
         a = a.contiguous()
     if not _aligned(b):
@@ -154,7 +157,9 @@ def gemm(a: torch.Tensor, b: torch.Tensor, *, a_mn: bool = False, b_mn: bool = F
     if out is None:
         if accumulate:
             raise ValueError("gemm: accumulate needs an output tensor")
-        out = torch.empty((M, N), dtype=out_dtype, device=a.device)
+        per = 16 // out_dtype.itemsize               # so must the rows of the result: a padded pitch where N is not
+        out = torch.empty((M, N + -N % per), dtype=out_dtype, device=a.device)[:, :N] if N % per else \
+            torch.empty((M, N), dtype=out_dtype, device=a.device)
     elif not _aligned(out) or out.shape != (M, N):
         raise ValueError("gemm: output must be a 16-byte aligned [M,N] tensor with unit inner stride")
     mode = _OUT_MODES[(out.dtype, bool(accumulate))]

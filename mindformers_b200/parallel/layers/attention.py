@@ -36,6 +36,8 @@ class AttnMeta:
     doc_tables: Optional[tuple] = None    # (doc_start, doc_end) int32 [B, S], built once per forward from the above
     cache: Optional[object] = None        # inference.KVCacheContext for paged attention
     kv_carry: Optional[object] = None     # modules.seq_pipe.KVCarry: keys / values of the earlier sequence chunks
+    layer_run: Optional[int] = None       # position of the running layer in the stack (its cache; layers that share
+                                          # weights run more than once)
     cp_rank_positions: bool = False       # positions already hold the context-parallel offsets
 
 

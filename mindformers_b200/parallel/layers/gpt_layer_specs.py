@@ -17,7 +17,8 @@ from .mlp import MLP
 from .moe import GroupedMLP, MoELayer, SharedExpertMLP, TopKRouter
 from .mtp import MultiTokenPredictionBlock, MultiTokenPredictionLayer
 from .norm import build_norm
-from .transformer_layer import TransformerLayer, TransformerLayerSubmodules
+from .ragged_attention import RaggedSelfAttention
+from .transformer_layer import OutputNormTransformerLayer, TransformerLayer, TransformerLayerSubmodules
 
 
 def get_moe_module_spec(num_experts: Optional[int] = None, moe_grouped_gemm: bool = True) -> ModuleSpec:
@@ -53,8 +54,22 @@ def get_gpt_layer_local_spec(num_experts: Optional[int] = None, moe_grouped_gemm
         post_attn_layernorm=norm if sandwich_norm else None, post_mlp_layernorm=norm if sandwich_norm else None))
 
 
+def get_output_norm_layer_spec(config) -> ModuleSpec:
+    """Spec of one layer whose sub-layer outputs are normalised; a layer without a feed-forward has
+    ``ffn_hidden_size == 0``."""
+    norm = ModuleSpec(module=build_norm)
+    ff = bool(config.ffn_hidden_size)
+    return ModuleSpec(module=OutputNormTransformerLayer, submodules=TransformerLayerSubmodules(
+        self_attention=ModuleSpec(module=RaggedSelfAttention), mlp=get_mlp_module_spec() if ff else None,
+        post_attn_layernorm=norm, post_mlp_layernorm=norm if ff else None))
+
+
 def get_gpt_layer_spec_for_config(config, is_moe: bool) -> ModuleSpec:
     """``get_gpt_layer_local_spec`` with the switches taken from a ``TransformerConfig``."""
+    if config.norm_placement == "output":
+        if is_moe or not config.ragged_attention:
+            raise ValueError("output-normalised layers are built with ragged attention and a dense feed-forward")
+        return get_output_norm_layer_spec(config)
     return get_gpt_layer_local_spec(
         num_experts=config.num_moe_experts if is_moe else None, moe_grouped_gemm=True,
         qk_layernorm=bool(getattr(config, "qk_layernorm", False)),
@@ -65,6 +80,9 @@ def get_gpt_layer_spec_for_config(config, is_moe: bool) -> ModuleSpec:
 def get_gpt_decoder_block_spec(config) -> List[ModuleSpec]:
     """One layer spec per layer of the whole model: dense or MoE after ``config.moe_layer_pattern()``
     (``first_k_dense_replace`` wins over ``moe_layer_freq``). A pipeline stage picks its own layers from the list."""
+    if config.layer_overrides:
+        return [get_gpt_layer_spec_for_config(config.for_layer(i), bool(flag))
+                for i, flag in enumerate(config.moe_layer_pattern())]
     dense = get_gpt_layer_spec_for_config(config, False)
     moe = get_gpt_layer_spec_for_config(config, True) if config.num_moe_experts else None
     return [moe if flag else dense for flag in config.moe_layer_pattern()]

@@ -17,6 +17,7 @@ from typing import Optional
 import torch
 import torch.nn as nn
 
+from ...ops import stream
 from .. import mappings as M
 from .. import parallel_state as ps
 from .attention import AttnMeta
@@ -96,6 +97,9 @@ class GPTModel(nn.Module):
     def logits(self, hidden):
         """Vocab-sharded logits ``[T, V/tp]`` of hidden states ``[T(/tp under SP), H]``."""
         w = self._output_weight()
+        cap = self.config.logit_softcap
+        if cap:          # fp32 accumulators -> cap * tanh(x / cap), element-wise (a vocabulary shard needs no other rank)
+            return stream.linear(hidden, w, act="softcap", cap=float(cap))
         y, _ = self.output_layer(hidden, weight=w)
         return y
 

@@ -10,9 +10,10 @@ import torch.nn as nn
 import torch.nn.functional as F
 
 from ...ops import functional as Fn
+from ...ops import stream
 from .tensor_parallel import ColumnParallelLinear, RowParallelLinear
 
-_ACT = {"gelu": F.gelu, "silu": F.silu, "swiglu": F.silu, "relu": F.relu,
+_ACT = {"relu2": stream.relu2, "gelu": F.gelu, "silu": F.silu, "swiglu": F.silu, "relu": F.relu,
         "fast_gelu": lambda x: F.gelu(x, approximate="tanh"), "gelu_tanh": lambda x: F.gelu(x, approximate="tanh")}
 
 
@@ -43,6 +44,10 @@ class MLP(nn.Module):
                                             is_expert=is_expert)
 
     def forward(self, hidden):
+        if self.act_name == "relu2" and not self.gated and self.linear_fc1.tp == 1 and self.linear_fc1.bias is None \
+                and self.linear_fc1.weight is not None and hidden.dim() == 2 and not torch.is_grad_enabled():
+            # a few rows: the activation runs in the epilogue of the up projection
+            return self.linear_fc2(stream.linear(hidden, self.linear_fc1.weight, act="relu2"))
         x, _ = self.linear_fc1(hidden)
         if self.gated and self.act_name in ("silu", "swiglu"):
             x = Fn.swiglu(x)

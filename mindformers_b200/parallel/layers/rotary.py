@@ -105,6 +105,32 @@ class YarnRotaryEmbedding(RotaryEmbedding):
         self.register_buffer("sin", (ang.sin() * self.mscale).contiguous().to(device), persistent=False)
 
 
+class RotaryFrequencies(nn.Module):
+    """Rotation frequencies for kernels that evaluate the angles themselves (``position * freqs[i]`` in fp32): ``freqs
+    [dim / 2]`` and the ``amplitude`` that multiplies cos and sin. There is no table, hence no longest position.
+
+    ``scaling`` None: ``base^(-2i/dim)``. ``{"type": "yarn", "factor", "original_max_position_embeddings", "beta_fast",
+    "beta_slow"}``: dimensions that turn more than ``beta_fast`` times over the original context keep their frequency,
+    those that turn less than ``beta_slow`` times are slowed down by ``factor``, with a linear ramp in between, and the
+    amplitude is ``0.1 ln(factor) + 1``. Computed in double precision, stored in fp32."""
+
+    def __init__(self, dim: int, base: float = 10000.0, scaling: Optional[dict] = None, device=None):
+        super().__init__()
+        freqs = base ** (-torch.arange(0, dim, 2, dtype=torch.float64) / dim)
+        self.amplitude = 1.0
+        if scaling:
+            kind = scaling.get("rope_type", scaling.get("type"))
+            if kind != "yarn":
+                raise ValueError(f"unsupported rotary scaling {kind!r}")
+            factor = float(scaling["factor"])
+            lo, hi = yarn_find_correction_range(float(scaling.get("beta_fast", 32.0)), float(scaling.get("beta_slow", 1.0)),
+                                                dim, base, float(scaling["original_max_position_embeddings"]))
+            ramp = ((torch.arange(dim // 2, dtype=torch.float64) - lo) / max(hi - lo, 0.001)).clamp(0, 1)
+            freqs = freqs / factor * ramp + freqs * (1 - ramp)
+            self.amplitude = 0.1 * math.log(factor) + 1.0
+        self.register_buffer("freqs", freqs.float().contiguous().to(device), persistent=False)
+
+
 def get_rope(config, max_positions: Optional[int] = None, head_dim: Optional[int] = None, device=None):
     """Build the rotary table a model configuration asks for."""
     maxp = max_positions or max(config.max_position_embeddings, config.seq_length)

@@ -18,6 +18,7 @@ import torch.nn as nn
 from torch.utils.checkpoint import checkpoint
 
 from .. import parallel_state as ps
+from ...ops import stream
 from ..spec_utils import build_module
 from .attention import AttnMeta
 from .moe import MoELayer
@@ -101,6 +102,43 @@ class TransformerLayer(nn.Module):
         return self._dropout(mlp_out), residual, aux
 
 
+class OutputNormTransformerLayer(nn.Module):
+    """Layer with a 32-bit residual stream and norms on the sub-layer OUTPUTS only: ``x <- x + scale1 * norm1(attention(x))``,
+    then ``x <- x + scale2 * norm2(mlp(x))`` (no second half without an ``mlp``; no scales without ``config.layer_scale``).
+    A serving layer: projection bias, norm, scale and residual add are one kernel (``ops/stream.py::add_normed``).
+
+    ``forward(pending, residual, ...)`` takes and returns the stream twice: ``pending`` in the activation dtype (the next
+    sub-layer's input) and ``residual`` in fp32 (None before the first layer)."""
+
+    stream_in_residual = True      # the result is ``residual`` alone; nothing is left to be added
+
+    def __init__(self, config, layer_number: int = 1, submodules: Optional[TransformerLayerSubmodules] = None):
+        super().__init__()
+        self.config, self.layer_number = config, layer_number
+        self.self_attention = build_module(submodules.self_attention, config, layer_number)
+        self.post_attn_layernorm = build_module(submodules.post_attn_layernorm, config)
+        self.mlp = build_module(submodules.mlp, config) if submodules.mlp is not None else None
+        self.post_mlp_layernorm = build_module(submodules.post_mlp_layernorm, config) if self.mlp is not None else None
+
+        def scale():
+            ref = self.post_attn_layernorm.weight
+            return nn.Parameter(torch.ones_like(ref)) if config.layer_scale else None
+        self.register_parameter("attn_layer_scale", scale())
+        self.register_parameter("mlp_layer_scale", scale() if self.mlp is not None else None)
+
+    def _add(self, residual, pending, y, bias, norm, scale):
+        return stream.add_normed(pending if residual is None else residual, y, bias, norm.weight, getattr(norm, "bias", None),
+                                 scale, norm.eps, hasattr(norm, "bias"), inplace=residual is not None)
+
+    def forward(self, pending, residual, rotary, meta: AttnMeta):
+        y, bias = self.self_attention(pending, rotary, meta)
+        pending, residual = self._add(residual, pending, y, bias, self.post_attn_layernorm, self.attn_layer_scale)
+        if self.mlp is not None:
+            y, bias = self.mlp(pending)
+            pending, residual = self._add(residual, pending, y, bias, self.post_mlp_layernorm, self.mlp_layer_scale)
+        return pending, residual, None
+
+
 def pipeline_layer_split(num_layers: int, pp: int, vpp: int = 1, offset=0) -> List[List[List[int]]]:
     """Layer ids of every (pp stage, virtual chunk). ``offset`` adds/removes layers per stage
     (list of pp values, or vpp lists of pp values), as the reference's ``LayerSetting`` does."""
@@ -170,10 +208,16 @@ class TransformerBlock(nn.Module):
         layer_specs = get_gpt_decoder_block_spec(config)      # one spec per layer of the whole model
         from ..init_method import module_rng
         built = []
-        for i in self.layer_ids:
+        owners = [config.shares_weights_with(i) for i in self.layer_ids]
+        if any(o not in self.layer_ids for o in owners):
+            raise NotImplementedError("layers that share weights must be on one pipeline stage")
+        own_ids = [i for i, o in zip(self.layer_ids, owners) if o == i]
+        for i in own_ids:
             with module_rng(base_seed, 100 + i, dev):     # a layer's initial weights depend on its number only
-                built.append(build_module(layer_specs[i], config, layer_number=i + 1))
-        self.layers = StageLayers(self.layer_ids, built)
+                built.append(build_module(layer_specs[i], config.for_layer(i), layer_number=i + 1))
+        self.layers = StageLayers(own_ids, built)
+        # the layers in running order: a layer that shares weights is its owner's module once more
+        self.run_order = [own_ids.index(o) for o in owners]
         self.final_layernorm = build_norm(config) if post_process else None
         self.recompute = bool(config.recompute) if not isinstance(config.recompute, (list, tuple)) else True
         self._recompute_layers = self._resolve_recompute(config.recompute)
@@ -190,6 +234,16 @@ class TransformerBlock(nn.Module):
     # selectively recomputed layer runs twice, whatever the patterns say, because nothing else is cheap
     _DEFAULT_SELECT = (r"mlp\.mul", r"mlp\.activation_func\.silu", r"mlp\.shared_experts\.mul",
                        r"mlp\.shared_experts\.activation_func\.silu", r".*\.norm")
+
+    @property
+    def num_runs(self) -> int:
+        """Layer runs of this stage (each has a cache of its own); above ``len(layers)`` when layers share weights."""
+        return len(self.run_order)
+
+    def cache_shapes(self):
+        """``(kv heads, key size, value size)`` per layer run, or None for attention without per-layer cache shapes."""
+        shapes = [getattr(self.layers[at].self_attention, "cache_shape", None) for at in self.run_order]
+        return [s() for s in shapes] if shapes and all(s is not None for s in shapes) else None
 
     def _setup_selective_recompute_and_offload(self, config):
         from ..recompute import ActivationOffloader, mark_recompute_modules
@@ -246,13 +300,14 @@ class TransformerBlock(nn.Module):
         return 0
 
     def forward(self, hidden, rotary, meta: AttnMeta):
-        pending, residual = hidden, None
+        pending, residual, layer = hidden, None, None
         aux_total = None
         training = self.training and torch.is_grad_enabled()
         if training and self._offload is not None:
             self._offload.prune()
-        for idx, layer in enumerate(self.layers):
-            run = layer
+        for idx, at in enumerate(self.run_order):
+            layer = run = self.layers[at]
+            meta.layer_run = self.layer_ids[idx]
             if self.params_ready_hook is not None:
                 self.params_ready_hook(self.layer_ids[idx])
             if training and self.grads_final_hook is not None and pending.requires_grad:
@@ -273,7 +328,11 @@ class TransformerBlock(nn.Module):
                 pending, residual, aux = run(pending, residual, rotary, meta)
             if aux is not None:
                 aux_total = aux if aux_total is None else aux_total + aux
-        if self.final_layernorm is not None:
+        if getattr(layer, "stream_in_residual", False):
+            norm = self.final_layernorm
+            out = residual if norm is None else stream.norm_stream(residual, norm.weight, getattr(norm, "bias", None), norm.eps,
+                                                                   hasattr(norm, "bias"))
+        elif self.final_layernorm is not None:
             if residual is None:
                 out = self.final_layernorm(pending)
             else:

@@ -8,6 +8,7 @@ dtype fields hold ``torch.dtype`` values after ``__post_init__``.
 """
 from __future__ import annotations
 
+import copy
 import dataclasses
 from dataclasses import dataclass, field
 from typing import Callable, List, Optional, Union
@@ -126,6 +127,20 @@ class TransformerConfig(ModelParallelConfig):
     untie_embeddings_and_output_weights: bool = True
     tie_word_embeddings: bool = False
     post_process: bool = True
+    # ---- layers that differ from one another, output-normalised stacks ----
+    # per layer, the fields of this configuration that differ (``for_layer``); None: all layers are alike
+    layer_overrides: Optional[List[dict]] = None
+    # per layer, the index of the layer whose weights it uses (its own index: weights of its own); None: no sharing
+    layer_sharing: Optional[List[int]] = None
+    norm_placement: str = "input"           # "input": pre-norm; "output": x + scale * norm(sublayer(x)), fp32 stream
+    layer_scale: bool = False               # per-channel scale of every (normalised) sub-layer output
+    ragged_attention: bool = False          # RaggedSelfAttention: whole, cut and mixed sequences in one paged call
+    v_channels: Optional[int] = None        # value size per head (default: kv_channels)
+    rotary_dim: Optional[int] = None        # rotated dimensions per head (default: kv_channels * rotary_percent)
+    add_attention_output_bias: bool = False
+    attention_chunk_size: int = 0           # > 0: a position sees its own chunk of that many positions only
+    attention_sink: bool = False            # learned per-head term in the softmax denominator
+    logit_softcap: Optional[float] = None   # logits <- cap * tanh(logits / cap), fp32
     # ---- init ----
     init_method: Optional[Callable] = None
     output_layer_init_method: Optional[Callable] = None
@@ -306,6 +321,14 @@ class TransformerConfig(ModelParallelConfig):
                 self.moe_aux_loss_coeff = float(self.aux_loss_factors[self.aux_loss_types.index("expert")])
         elif self.expert_model_parallel_size > 1:
             raise ValueError("expert_model_parallel_size > 1 needs num_moe_experts")
+        if self.norm_placement not in ("input", "output"):
+            raise ValueError(f"norm_placement must be 'input' or 'output', got {self.norm_placement!r}")
+        for name in ("layer_overrides", "layer_sharing"):
+            val = getattr(self, name)
+            if val is not None and len(val) != self.num_layers:
+                raise ValueError(f"{name} must have num_layers ({self.num_layers}) entries, got {len(val)}")
+        if self.layer_sharing and any(self.layer_sharing[j] != j or j > i for i, j in enumerate(self.layer_sharing)):
+            raise ValueError("layer_sharing must name an earlier layer that has weights of its own")
         if self.tie_word_embeddings:
             self.untie_embeddings_and_output_weights = False
         if self.use_scaled_init and self.num_layers:
@@ -325,6 +348,22 @@ class TransformerConfig(ModelParallelConfig):
     @property
     def head_dim(self) -> int:
         return self.kv_channels
+
+    def for_layer(self, index: int) -> "TransformerConfig":
+        """The configuration of layer ``index``: this one with the layer's overrides (a copy; the initialisers and
+        dynamic attributes such as ``device`` are kept)."""
+        if not self.layer_overrides:
+            return self
+        out = copy.copy(self)
+        for key, value in self.layer_overrides[index].items():
+            if not hasattr(out, key):
+                raise ValueError(f"layer {index}: unknown configuration field {key!r}")
+            setattr(out, key, value)
+        return out
+
+    def shares_weights_with(self, index: int) -> int:
+        """The layer that owns the weights layer ``index`` runs with."""
+        return index if not self.layer_sharing else int(self.layer_sharing[index])
 
     def moe_layer_pattern(self) -> List[int]:
         """1 for MoE layers, 0 for dense layers (``first_k_dense_replace`` wins over ``moe_layer_freq``)."""

@@ -11,7 +11,9 @@ One iteration (``step()``):
 2. waiting requests are admitted while a slot is free and the block pool can hold their prompt (first come, first
    served; a request that was preempted re-enters with the tokens it had produced, so its cache is recomputed);
 3. if requests were admitted, one prefill call runs their prompts (long prompts in chunks of ``max_prefill_tokens``);
-   otherwise one decode call advances every running request by a token — before it, the newest requests are
+   models whose attention takes ragged batches (``config.ragged_attention``) run MIXED steps instead: one call with the
+   next token of every decoding request and portions of the waiting prompts, ``max_prefill_tokens`` tokens in all, so
+   that a long prompt does not hold up the running requests. Otherwise one decode call advances every running request by a token — before it, the newest requests are
    preempted while the pool cannot give every running request the block its next token may need;
    When every running request decodes greedily (or at one common temperature without top-k / top-p / penalties) and
    shares its stop tokens, the decode call is a BURST instead (``decode_burst`` steps, default 8): the step was
@@ -20,6 +22,9 @@ One iteration (``step()``):
    the tokens are read back once. Requests that finish inside a burst stop there; new arrivals wait for its end;
 4. the next token of every request that was served is chosen (greedy, or temperature / top-k / top-p / penalties with
    a per-request seeded generator), stop conditions are checked and the ``on_token`` callbacks are called.
+
+``attach`` / ``advance`` / ``detach`` drive the same slots, cache and model call with batches chosen by the caller (given
+tokens, logits back, nothing sampled).
 
 With several tensor-parallel ranks every rank runs the same engine: rank 0 owns the queue and broadcasts the requests
 it admits and aborts each iteration; everything else is a deterministic function of those, and the logits are
@@ -128,12 +133,10 @@ class ServingEngine:
         cfg = model.config
         self.max_num_seqs = int(max_num_seqs)
         self.max_model_len = int(max_model_len or getattr(cfg, "seq_length", 2048))
-        self.ctx, self.tables = model._set_kv_cache(self.max_num_seqs, self.max_model_len, num_blocks)
-        if num_blocks:        # an explicit pool size over-subscribes the slots: rebuild the tables around it
-            from ..inference.block_manager import BlockTables
-            from ..inference.paged_attention import KVCacheContext  # noqa: F401  (the cache itself was sized by the model)
-            if int(num_blocks) < self.tables.pool.num_blocks:
-                self.tables = BlockTables(int(num_blocks), self.tables.block_size, self.max_model_len)
+        # an explicit pool size over-subscribes the slots: the cache has exactly that many blocks
+        self.ctx, self.tables = model._set_kv_cache(self.max_num_seqs, self.max_model_len, num_blocks,
+                                                    exact_blocks=bool(num_blocks))
+        self.mixed_steps = bool(getattr(cfg, "ragged_attention", False))
         self.tables.init_cache_engine(self.max_num_seqs)
         self.block_size = self.tables.block_size
         self.max_prefill_tokens = int(max_prefill_tokens)
@@ -149,7 +152,7 @@ class ServingEngine:
         self._stop = False
         self._thread: Optional[threading.Thread] = None
         self.finished_metrics: Deque[Dict[str, float]] = deque(maxlen=4096)
-        self.counters = {"requests": 0, "finished": 0, "aborted": 0, "preempted": 0, "prefill_tokens": 0,
+        self.counters = {"mixed_steps": 0, "requests": 0, "finished": 0, "aborted": 0, "preempted": 0, "prefill_tokens": 0,
                          "decode_tokens": 0, "steps": 0, "bursts": 0}
         self._by_id: Dict[str, Request] = {}
 
@@ -251,7 +254,8 @@ class ServingEngine:
             req = self.waiting[0]
             slot = self._free_slot()
             n = len(req.tokens)
-            if slot is None or self._blocks_for(n + 1) > self.tables.pool.num_free or (admitted and n > budget):
+            if slot is None or self._blocks_for(n + 1) > self.tables.pool.num_free \
+                    or (admitted and n > budget and not self.mixed_steps):
                 break
             self.waiting.popleft()
             req.slot = slot
@@ -267,25 +271,122 @@ class ServingEngine:
             eng = self.tables.engines[slot]
             eng.blocks.extend(self.tables.pool.allocate(need - len(eng.blocks)))
         served: List[Request] = []
-        if admitted:
+        if self.mixed_steps and any(r is not None and len(r.tokens) - r.cached > 1 for r in self.running):
+            served = self._mixed_step()
+        elif admitted and not self.mixed_steps:
             served = self._prefill(admitted)
         else:
             live = [r for r in self.running if r is not None]
             if not live:
                 return []
-            # every running request may need one more block for the token of this step
-            def short():
-                need = sum(1 for r in self.running if r is not None
-                           and self._blocks_for(r.cached + 1) > len(self.tables.engines[r.slot].blocks))
-                return need > self.tables.pool.num_free
-            while short() and len(self._admit_order) > 1:
-                self._preempt(self._admit_order[-1])
+            self._make_room()
             burst = self._burst_length()
             if burst >= 2:
                 return self._decode_burst(burst)
             served = self._decode()
         self._choose_tokens(served)
         return served
+
+    def _make_room(self):
+        """Every running request may need one more block for the token of this step: preempt the newest while the pool
+        cannot give them all one."""
+        def short():
+            need = sum(1 for r in self.running if r is not None
+                       and self._blocks_for(r.cached + 1) > len(self.tables.engines[r.slot].blocks))
+            return need > self.tables.pool.num_free
+        while short() and len(self._admit_order) > 1:
+            self._preempt(self._admit_order[-1])
+
+    # ---- one model call over the slots ------------------------------------------------------------------------------
+    def _call(self, work: Dict[int, List[int]], starts: Dict[int, int],
+              want: Optional[Dict[int, List[int]]] = None) -> Dict[int, torch.Tensor]:
+        """Run the new tokens of the slots in ``work`` (they start at position ``starts[slot]``) as one batch. Returns the
+        logits of every slot's last token, or with ``want`` those of the named new tokens, ``[len(want[slot]), V]``.
+        One token for each: the decode step over all slots; anything else: one ragged call."""
+        B = self.max_num_seqs
+        active = [i in work for i in range(B)]
+        at = [starts.get(i, 0) for i in range(B)]
+        if all(len(t) == 1 for t in work.values()) and (want is None or any(want.values())):
+            logits = self.model._forward_step([work.get(i, [0]) for i in range(B)], at, self.ctx, self.tables, False, active)
+            return {i: logits[i] if want is None else logits[i:i + 1][[0] * len(want[i])] for i in work}
+        rows: Dict[int, List[int]] = {}
+        flat = 0
+        for i in sorted(work):
+            rows[i] = [flat + len(work[i]) - 1] if want is None else [flat + k for k in want[i]]
+            flat += len(work[i])
+        order = [r for i in sorted(work) for r in rows[i]]
+        logits = self.model._forward_step([work.get(i, []) for i in range(B)], at, self.ctx, self.tables, True, active,
+                                          rows=order)
+        out, flat = {}, 0
+        for i in sorted(work):
+            part = logits[flat:flat + len(rows[i])] if rows[i] else None
+            out[i] = part[0] if want is None else part
+            flat += len(rows[i])
+        return out
+
+    def _mixed_step(self) -> List[Request]:
+        """One call with the next token of every decoding request and, within ``max_prefill_tokens``, portions of the
+        prompts that are not in the cache yet (in admission order)."""
+        self._make_room()
+        self.counters["mixed_steps"] += 1
+        live = list(self._admit_order)
+        work: Dict[int, List[int]] = {r.slot: [r.tokens[-1]] for r in live if len(r.tokens) - r.cached == 1}
+        room = max(1, self.max_prefill_tokens - len(work))
+        for r in live:
+            rest = len(r.tokens) - r.cached
+            if rest > 1 and room > 0:
+                work[r.slot] = r.tokens[r.cached:r.cached + room]
+                room -= len(work[r.slot])
+        logits = self._call(work, {r.slot: r.cached for r in live})
+        served = []
+        for r in live:
+            n = len(work.get(r.slot, ()))
+            if not n:
+                continue
+            self.counters["decode_tokens" if r.output and len(r.tokens) - r.cached == 1 else "prefill_tokens"] += n
+            r.cached += n
+            if r.cached == len(r.tokens):
+                r._logits = logits[r.slot]
+                served.append(r)
+        return served
+
+    # ---- batches chosen by the caller --------------------------------------------------------------------------------
+    def attach(self, request_id: str) -> Request:
+        """Take a slot for a sequence that ``advance`` feeds."""
+        slot = self._free_slot()
+        if slot is None:
+            raise RuntimeError(f"all {self.max_num_seqs} slots are taken")
+        if request_id in self._by_id:
+            raise ValueError(f"request {request_id!r} is live already")
+        req = Request(request_id, [], SamplingParams())
+        req.slot = slot
+        self.running[slot] = self._by_id[request_id] = req
+        self._admit_order.append(req)
+        self.counters["requests"] += 1
+        return req
+
+    @torch.no_grad()
+    def advance(self, work: Dict[str, List[int]], want: Dict[str, List[int]]) -> Dict[str, Optional[torch.Tensor]]:
+        """Run the next tokens of attached sequences as one batch; returns, per request, the logits of the new tokens that
+        ``want`` names (``[n, V]``; None for none)."""
+        reqs = {rid: self._by_id[rid] for rid in work}
+        for rid, r in reqs.items():
+            if r.cached + len(work[rid]) > self.max_model_len:
+                raise ValueError(f"request {rid!r} exceeds max_model_len {self.max_model_len}")
+        tokens = {reqs[rid].slot: list(t) for rid, t in work.items() if len(t)}
+        if not tokens:
+            return {rid: None for rid in work}
+        got = self._call(tokens, {r.slot: r.cached for r in reqs.values()},
+                         {reqs[rid].slot: list(want.get(rid, ())) for rid in work if len(work[rid])})
+        for rid, r in reqs.items():
+            r.prompt.extend(work[rid])
+            r.cached += len(work[rid])
+        self.counters["steps"] += 1
+        return {rid: got.get(r.slot) for rid, r in reqs.items()}
+
+    def detach(self, request_id: str):
+        """Give an attached sequence's slot and cache blocks back."""
+        self._release(self._by_id[request_id], "detached")
 
     # ---- decode bursts on the device --------------------------------------------------------------------------------
     def _stop_ids(self, r: Request):
