@@ -72,8 +72,9 @@ class KVCacheContext:
         self.cu_q = None              # python list of cumulative q lengths
         self.layer_offset = 0
         self.cu_q_dev = None          # int32 [B+1]: cu_q on the device (ragged caches, prefill steps)
-        self.prefill_work_dev = None  # int32 [n, 2]: work list of the ragged prefill kernel
-        self.n_prefill_work = self.n_single_rows = 0
+        self.prefill_work = {}        # work lists of the ragged prefill kernel, made when a layer needs them
+        self.q_lens_host = self.context_lens_host = ()
+        self.n_long_rows = self.n_single_rows = 0     # sequences with several new rows / with one
 
     def set_step(self, *, is_prefill, block_tables, slot_mapping, context_lens, q_seq_lens, device):
         self.is_prefill = is_prefill
@@ -87,11 +88,10 @@ class KVCacheContext:
             cu.append(cu[-1] + n)
         self.cu_q = cu
         if self.ragged and is_prefill:
-            from .ragged_attention import prefill_work
-            work = prefill_work(q, [int(x) for x in context_lens])
-            self.n_prefill_work, self.n_single_rows = len(work), sum(n == 1 for n in q)
-            flat = torch.tensor(cu + [x for item in work for x in item], dtype=torch.int32).to(device)   # one copy
-            self.cu_q_dev, self.prefill_work_dev = flat[: len(cu)], flat[len(cu):]
+            self.q_lens_host, self.context_lens_host = q, [int(x) for x in context_lens]
+            self.n_long_rows, self.n_single_rows = sum(n > 1 for n in q), sum(n == 1 for n in q)
+            self.cu_q_dev = torch.tensor(cu, dtype=torch.int32).to(device)
+            self.prefill_work = {}
         # sequences without new tokens in this step (finished prompts of a chunked prefill, idle serving slots) have
         # no row of their own: one entry per sequence that has tokens
         self.last_token_index = torch.as_tensor([c - 1 for c, n in zip(cu[1:], q) if n > 0], dtype=torch.int64,

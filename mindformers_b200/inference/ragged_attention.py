@@ -14,18 +14,32 @@ import torch
 
 from ..ops import _lib
 
-PAIR_ROWS = 256          # query rows of one work item of the prefill kernel
+TILE = 128               # query rows of a tile of the prefill kernel
 
 
-def prefill_work(q_lens, context_lens):
-    """Work list of the prefill kernel: ``[(sequence, first row of a 256-row pair)]`` of every sequence with more than one
-    new row, the pairs that reach furthest into their sequence first (they have the most keys)."""
+def prefill_work(q_lens, context_lens, chunk: int = 0):
+    """Work list of the prefill kernel: ``[(sequence, first row of a 128-row tile)]`` of every sequence with more than one
+    new row, the tiles that see the most key tiles first."""
     items = []
     for b, (n, ctx) in enumerate(zip(q_lens, context_lens)):
         if n > 1:
-            items += [(min(int(ctx) - n + r + PAIR_ROWS, int(ctx)), b, r) for r in range(0, n, PAIR_ROWS)]
+            for r in range(0, n, TILE):
+                first, last = ctx - n + r, min(ctx - n + r + TILE, ctx) - 1
+                lo = first - first % chunk if chunk > 0 else 0
+                items.append((last // TILE - lo // TILE, b, r))
     items.sort(key=lambda t: -t[0])
     return [(b, r) for _, b, r in items]
+
+
+def _work_on_device(cache, chunk: int):
+    """The step's work list for ``chunk`` as an int32 device tensor, made once per step (layers with the same chunk share
+    it)."""
+    work = cache.prefill_work.get(chunk)
+    if work is None:
+        items = prefill_work(cache.q_lens_host, cache.context_lens_host, chunk)
+        work = torch.tensor(items, dtype=torch.int32).to(cache.block_tables.device)
+        cache.prefill_work[chunk] = work
+    return work
 
 
 def _reference(q, cache, layer, scale, chunk, sink):
@@ -82,9 +96,9 @@ def ragged_attention(q: torch.Tensor, cache, layer: int, scale: float, chunk: in
         _lib.count_launch()
         return out.view(T, Hq * DV)
     status = _lib.status_word(q.device).data_ptr()
-    if ragged and cache.n_prefill_work:
-        rc = lib.mfb_paged_prefill_tc(q.data_ptr(), kc.data_ptr(), vc.data_ptr(), cache.prefill_work_dev.data_ptr(),
-                                      cache.n_prefill_work, cu, tables, lens, snk, out.data_ptr(), T, Hq, Hkv, D, DV, nb, bs,
+    if ragged and cache.n_long_rows:
+        work = _work_on_device(cache, int(chunk))
+        rc = lib.mfb_paged_prefill_tc(q.data_ptr(), kc.data_ptr(), vc.data_ptr(), work.data_ptr(), work.shape[0], cu, tables, lens, snk, out.data_ptr(), T, Hq, Hkv, D, DV, nb, bs,
                                       max_blocks, int(chunk), float(scale), status, _lib.stream_ptr())
         _lib.check(rc, "mfb_paged_prefill_tc")
         _lib.count_launch()

@@ -6,10 +6,13 @@
 // portion sits at position context_lens[b] - q_len + r and sees keys up to itself, with `chunk` > 0 only those of its
 // own chunk of `chunk` positions (counted from position 0). `sink` [Hq] adds exp(sink_h) to the denominator.
 //
-// The tensor-core pipeline is the one of flash_attention_fwd2.cu: a CTA owns up to 256 query rows of one head as two
-// 128-row tiles that share the key / value tiles; every tile has a softmax warpgroup; P goes back into tensor memory
-// and is read from there by the P V product. What differs:
-//   - work comes as a list of (sequence, first row of a 256-row pair); only key tiles that some row of a tile sees are
+// The tensor-core pipeline is the one of flash_attention_fwd2.cu (P goes back into tensor memory and is read from there
+// by the P V product), with one 128-row query tile per CTA and one stage of K and of V: a CTA then takes half of an SM's
+// tensor memory and at most half of its shared memory, and two of them share an SM. While one waits for its products or
+// its softmax the other works, and the start and the end of a CTA run under the products of its neighbour, which is what
+// counts when a tile sees few keys (chunks, short portions). K of the next key tile loads during the softmax of this one,
+// V during the scores and the softmax, so one stage of each is enough. What else differs:
+//   - work comes as a list of (sequence, first row of the tile); only key tiles that some row of the tile sees are
 //     visited, from the chunk of its first row to its last row;
 //   - K / V tiles (128 consecutive positions) are assembled from the sequence's pages, one TMA box per page and 64
 //     columns; pages past the end of the sequence repeat the tile's first page and are masked;
@@ -18,20 +21,19 @@
 //     columns of the result that are not stored;
 //   - the result is staged in shared memory and written row by row: a portion may end anywhere.
 //
-// Roles (320 threads): warp 0 TMA producer, warp 1 MMA issuer + TMEM owner, warps 2..5 softmax of tile A, warps 6..9
-// softmax of tile B. Every wait is bounded (common.cuh).
+// Roles (192 threads): warp 0 TMA producer, warp 1 MMA issuer + TMEM owner, warps 2..5 softmax. Every wait is bounded (common.cuh).
 #include "common.cuh"
 
 namespace mfb {
 namespace ppt {
 
-constexpr int kThreads = 320;
+constexpr int kThreads = 192;
 constexpr int kTile = 128;
 constexpr int kSubBytes = kTile * 128;     // [128 rows][128 B] swizzled sub-tile (64 bf16 columns)
 constexpr float kRescaleThreshold = 8.0f;  // log2 units
 
 struct Args {
-  const int* work;           // [n_work, 2]: sequence, first row of the pair inside the portion
+  const int* work;           // [n_work, 2]: sequence, first row of the tile inside the portion
   const int* cu_q;           // [B + 1]
   const int* block_tables;   // [B, max_blocks]
   const int* context_lens;   // [B]
@@ -84,7 +86,7 @@ __device__ __forceinline__ void tmem_st_32x32b_x32(uint32_t taddr, const uint32_
 
 // HQ: padded query / key size, HV: padded value size (64 or 128)
 template <int HQ, int HV>
-__global__ void __launch_bounds__(kThreads, 1)
+__global__ void __launch_bounds__(kThreads, 2)
 paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                         const __grid_constant__ CUtensorMap tmV, const Args args) {
   constexpr int QB = HQ / 64, VB = HV / 64;          // 64-column sub-tiles
@@ -93,103 +95,80 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) &
                                              ~static_cast<uintptr_t>(1023));
-  uint8_t* sQ = smem;                         // 2 tiles (A, B)
-  uint8_t* sK = sQ + 2 * kStage;              // 2 stages
-  uint8_t* sV = sK + 2 * kQBytes;             // 2 stages
-  uint64_t* bars = reinterpret_cast<uint64_t*>(sV + 2 * kVBytes);
-  uint64_t* q_full = bars;          // 1
-  uint64_t* k_full = bars + 1;      // 2
-  uint64_t* k_empty = bars + 3;     // 2
-  uint64_t* v_full = bars + 5;      // 2
-  uint64_t* v_empty = bars + 7;     // 2
-  uint64_t* s_full = bars + 9;      // 2: S of tile A / B complete
-  uint64_t* p_ready = bars + 11;    // 2: P of tile A / B written (128 arrivals)
-  uint64_t* pv_done = bars + 13;    // 2: P V of tile A / B complete
-  uint32_t* tmem_holder = reinterpret_cast<uint32_t*>(bars + 15);
+  uint8_t* sQ = smem;
+  uint8_t* sK = sQ + kStage;
+  uint8_t* sV = sK + kQBytes;
+  uint64_t* bars = reinterpret_cast<uint64_t*>(sV + kVBytes);
+  uint64_t* q_full = bars;
+  uint64_t* k_full = bars + 1;
+  uint64_t* k_empty = bars + 2;
+  uint64_t* v_full = bars + 3;
+  uint64_t* v_empty = bars + 4;
+  uint64_t* s_full = bars + 5;      // S complete
+  uint64_t* p_ready = bars + 6;     // P written (128 arrivals)
+  uint64_t* pv_done = bars + 7;     // P V complete
+  uint32_t* tmem_holder = reinterpret_cast<uint32_t*>(bars + 8);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_holder + 1);
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int head = static_cast<int>(blockIdx.x) % args.num_q_heads;
   const int item = static_cast<int>(blockIdx.x) / args.num_q_heads;
-  const int b = args.work[2 * item], pair_row = args.work[2 * item + 1];
-  const int q0 = args.cu_q[b];
-  const int q_len = args.cu_q[b + 1] - q0;
+  const int b = args.work[2 * item], row0 = args.work[2 * item + 1];
+  const int q0 = args.cu_q[b] + row0;                // the tile's first row of q
   const int len = args.context_lens[b];
-  const int pos0 = len - q_len;                      // position of the portion's first row
+  const int rows = args.cu_q[b + 1] - q0 < kTile ? args.cu_q[b + 1] - q0 : kTile;
+  const int pos0 = len - (args.cu_q[b + 1] - q0);    // its position
   const int kv_head = head / args.group;
-  int n_kv_x[2], lo_x[2], rows_x[2];   // tile x: rows_x[x] rows, key tiles lo_x[x] .. n_kv_x[x] - 1
-#pragma unroll
-  for (int x = 0; x < 2; ++x) {
-    const int r0 = pair_row + x * kTile;
-    int rows = q_len - r0;
-    rows = rows < 0 ? 0 : (rows > kTile ? kTile : rows);
-    rows_x[x] = rows;
-    const int first = pos0 + r0;
-    lo_x[x] = (rows > 0 && args.chunk > 0) ? (first - first % args.chunk) / kTile : 0;
-    n_kv_x[x] = rows > 0 ? (first + rows - 1) / kTile + 1 : 0;
-  }
-  const int n_kv = n_kv_x[0] > n_kv_x[1] ? n_kv_x[0] : n_kv_x[1];
-  const int lo = lo_x[0];              // positions grow with the rows: tile A starts first
+  // key tiles lo .. n_kv - 1
+  const int lo = args.chunk > 0 ? (pos0 - pos0 % args.chunk) / kTile : 0;
+  const int n_kv = rows > 0 ? (pos0 + rows - 1) / kTile + 1 : 0;
 
   if (threadIdx.x == 0) {
     *abort_flag = 0;
-    mbar_init(smem_u32(q_full), 1);
-    for (int s = 0; s < 2; ++s) {
-      mbar_init(smem_u32(&k_full[s]), 1);
-      mbar_init(smem_u32(&k_empty[s]), 1);
-      mbar_init(smem_u32(&v_full[s]), 1);
-      mbar_init(smem_u32(&v_empty[s]), 1);
-      mbar_init(smem_u32(&s_full[s]), 1);
-      mbar_init(smem_u32(&p_ready[s]), 128);
-      mbar_init(smem_u32(&pv_done[s]), 1);
-    }
+    for (int i = 0; i < 8; ++i) mbar_init(smem_u32(&bars[i]), &bars[i] == p_ready ? 128 : 1);
     fence_barrier_init();
     tma_prefetch_desc(&tmQ);
     tma_prefetch_desc(&tmK);
     tma_prefetch_desc(&tmV);
   }
   if (warp == 1) {
-    tmem_alloc(smem_u32(tmem_holder), 512);
+    tmem_alloc(smem_u32(tmem_holder), 256);
     tmem_relinquish();
   }
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
   const uint32_t tmem_base = *tmem_holder;
-  // S_A +0, S_B +128, O_A +256, O_B +384; P_X lives in the first 64 columns of S_X
+  const uint32_t tmem_S = tmem_base, tmem_O = tmem_base + kTile;   // P lives in the first 64 columns of S
   if (warp == 0) {
     // ------------------------------ TMA producer ------------------------------
     if (lane == 0 && n_kv > 0) {
       const uint32_t qb = smem_u32(q_full);
-      const int n_tiles_here = rows_x[1] > 0 ? 2 : 1;
-      mbar_expect_tx(qb, n_tiles_here * kQBytes);
-      for (int x = 0; x < n_tiles_here; ++x)
-        for (int c = 0; c < QB; ++c)
-          tma_load_3d(smem_u32(sQ) + x * kStage + c * kSubBytes, &tmQ, qb, c * 64, head, q0 + pair_row + x * kTile);
+      mbar_expect_tx(qb, kQBytes);
+      for (int c = 0; c < QB; ++c) tma_load_3d(smem_u32(sQ) + c * kSubBytes, &tmQ, qb, c * 64, head, q0);
       const int bs = args.block_size;
       const int pages = kTile / bs;
       const int* table = args.block_tables + static_cast<size_t>(b) * args.max_blocks;
       const int kcol = kv_head * args.D, vcol = kv_head * args.DV;
       bool ok = true;
       for (int j = lo; j < n_kv && ok; ++j) {
-        const int st = (j - lo) & 1;
-        const uint32_t ph = ((j - lo) >> 1) & 1;
+        const uint32_t ph = (j - lo) & 1;
         const int tok0 = j * kTile;
         const int first_page = table[tok0 / bs];
-        ok = mbar_wait(smem_u32(&k_empty[st]), ph ^ 1, abort_flag, args.status, kStatusWaitTimeoutProducer);
+        ok = mbar_wait(smem_u32(k_empty), ph ^ 1, abort_flag, args.status, kStatusWaitTimeoutProducer);
         if (!ok) break;
-        const uint32_t kb = smem_u32(&k_full[st]);
+        const uint32_t kb = smem_u32(k_full);
         mbar_expect_tx(kb, kQBytes);
-        const uint32_t kd = smem_u32(sK + st * kQBytes);
+        const uint32_t kd = smem_u32(sK);
         for (int i = 0; i < pages; ++i) {
           const int pg = tok0 + i * bs < len ? table[tok0 / bs + i] : first_page;
           for (int c = 0; c < QB; ++c) tma_load_2d(kd + c * kSubBytes + i * bs * 128, &tmK, kb, kcol + c * 64, pg * bs);
         }
-        ok = mbar_wait(smem_u32(&v_empty[st]), ph ^ 1, abort_flag, args.status, kStatusWaitTimeoutProducer);
+        ok = mbar_wait(smem_u32(v_empty), ph ^ 1, abort_flag, args.status, kStatusWaitTimeoutProducer);
         if (!ok) break;
-        const uint32_t vb = smem_u32(&v_full[st]);
+        const uint32_t vb = smem_u32(v_full);
         mbar_expect_tx(vb, kVBytes);
-        const uint32_t vd = smem_u32(sV + st * kVBytes);
+        const uint32_t vd = smem_u32(sV);
         for (int i = 0; i < pages; ++i) {
           const int pg = tok0 + i * bs < len ? table[tok0 / bs + i] : first_page;
           for (int c = 0; c < VB; ++c) tma_load_2d(vd + c * kSubBytes + i * bs * 128, &tmV, vb, vcol + c * 64, pg * bs);
@@ -202,85 +181,53 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
     if (lane == 0 && n_kv > 0) {
       constexpr uint32_t IDESC_QK = umma_idesc_bf16(kTile, kTile, 0, 0);  // A = Q K-major (smem), B = K K-major
       constexpr uint32_t IDESC_PV = umma_idesc_bf16(kTile, HV, 0, 1);     // A = P (tensor memory), B = V MN-major
-      auto issue_qk = [&](int x, int j) {
-        const uint32_t qa = smem_u32(sQ) + x * kStage;
-        const uint32_t ka = smem_u32(sK) + ((j - lo) & 1) * kQBytes;
-#pragma unroll
-        for (int k = 0; k < HQ / 16; ++k) {
-          const uint32_t off = (k >> 2) * kSubBytes + (k & 3) * 32;
-          umma_f16_ss(tmem_base + x * kTile, umma_desc_kmajor_sw128(qa + off), umma_desc_kmajor_sw128(ka + off),
-                      IDESC_QK, k > 0 ? 1u : 0u);
-        }
-        umma_commit(smem_u32(&s_full[x]));
-      };
+      const uint32_t qa = smem_u32(sQ), ka = smem_u32(sK), va = smem_u32(sV);
       bool ok = mbar_wait(smem_u32(q_full), 0, abort_flag, args.status, kStatusWaitTimeoutMma);
-      auto active = [&](int x, int j) { return j >= lo_x[x] && j < n_kv_x[x]; };
-      if (ok) {
-        ok = mbar_wait(smem_u32(&k_full[0]), 0, abort_flag, args.status, kStatusWaitTimeoutMma);
-        if (ok) {
+      for (int j = lo; j <= n_kv && ok; ++j) {
+        if (j > lo) {
+          // ---- O += P(j - 1) V(j - 1) ----
+          const uint32_t ph = (j - 1 - lo) & 1;
+          ok = mbar_wait(smem_u32(v_full), ph, abort_flag, args.status, kStatusWaitTimeoutMma);
+          if (ok) ok = mbar_wait(smem_u32(p_ready), ph, abort_flag, args.status, kStatusWaitTimeoutMma);
+          if (!ok) break;
           tc_fence_after();
-          if (active(0, lo)) issue_qk(0, lo);
-          if (active(1, lo)) issue_qk(1, lo);
-          umma_commit(smem_u32(&k_empty[0]));
-        }
-      }
-      for (int j = lo; j < n_kv && ok; ++j) {
-        const int st = (j - lo) & 1;
-        const uint32_t ph = ((j - lo) >> 1) & 1;
-        ok = mbar_wait(smem_u32(&v_full[st]), ph, abort_flag, args.status, kStatusWaitTimeoutMma);
-        if (!ok) break;
-        bool k_next_waited = false;
 #pragma unroll
-        for (int x = 0; x < 2; ++x) {
-          const bool pv_now = active(x, j), qk_next = active(x, j + 1);
-          if (pv_now) {
-            ok = mbar_wait(smem_u32(&p_ready[x]), (j - lo_x[x]) & 1, abort_flag, args.status, kStatusWaitTimeoutMma);
-            if (!ok) break;
-            tc_fence_after();
-            const uint32_t va = smem_u32(sV) + st * kVBytes;
-            const uint32_t p_tmem = tmem_base + x * kTile;          // bf16 pairs: 8 columns per 16 keys
-            const uint32_t o_tmem = tmem_base + 256 + x * kTile;
-#pragma unroll
-            for (int k = 0; k < kTile / 16; ++k) {
-              const uint64_t b_desc = umma_desc_mnmajor_sw128(va + k * 16 * 128, kSubBytes);
-              umma_f16_ts(o_tmem, p_tmem + k * 8, b_desc, IDESC_PV, (j > lo_x[x] || k > 0) ? 1u : 0u);
-            }
-            umma_commit(smem_u32(&pv_done[x]));
-          }
-          if (qk_next) {
-            if (!k_next_waited) {
-              ok = mbar_wait(smem_u32(&k_full[(j + 1 - lo) & 1]), ((j + 1 - lo) >> 1) & 1, abort_flag, args.status,
-                             kStatusWaitTimeoutMma);
-              if (!ok) break;
-              tc_fence_after();
-              k_next_waited = true;
-            }
-            issue_qk(x, j + 1);   // overwrites S_X / P_X: executes behind the P V product issued just above
-          }
+          for (int k = 0; k < kTile / 16; ++k)           // bf16 pairs: 8 columns of P per 16 keys
+            umma_f16_ts(tmem_O, tmem_S + k * 8, umma_desc_mnmajor_sw128(va + k * 16 * 128, kSubBytes), IDESC_PV,
+                        (j - 1 > lo || k > 0) ? 1u : 0u);
+          umma_commit(smem_u32(pv_done));
+          umma_commit(smem_u32(v_empty));
         }
-        if (!ok) break;
-        umma_commit(smem_u32(&v_empty[st]));
-        if (k_next_waited) umma_commit(smem_u32(&k_empty[(j + 1 - lo) & 1]));
+        if (j < n_kv) {
+          // ---- S = Q K(j)^T: overwrites S / P, executes behind the P V product issued just above ----
+          ok = mbar_wait(smem_u32(k_full), (j - lo) & 1, abort_flag, args.status, kStatusWaitTimeoutMma);
+          if (!ok) break;
+          tc_fence_after();
+#pragma unroll
+          for (int k = 0; k < HQ / 16; ++k) {
+            const uint32_t off = (k >> 2) * kSubBytes + (k & 3) * 32;
+            umma_f16_ss(tmem_S, umma_desc_kmajor_sw128(qa + off), umma_desc_kmajor_sw128(ka + off), IDESC_QK, k > 0 ? 1u : 0u);
+          }
+          umma_commit(smem_u32(s_full));
+          umma_commit(smem_u32(k_empty));
+        }
       }
     }
     __syncwarp();
   } else {
-    // ------------------------------ softmax warpgroups ------------------------------
-    const int x = (warp - 2) >> 2;                 // 0 = tile A, 1 = tile B
+    // ------------------------------ softmax warpgroup ------------------------------
     const int ew = warp & 3;                       // TMEM lane quarter of this warp
     const int row = ew * 32 + lane;
     const uint32_t lane_base = static_cast<uint32_t>(ew * 32) << 16;
-    const uint32_t s_tmem = tmem_base + x * kTile + lane_base;
-    const uint32_t o_tmem = tmem_base + 256 + x * kTile + lane_base;
-    const uint32_t bar_and = 2 + x;
-    const int my_n = n_kv_x[x], my_lo = lo_x[x];
-    const int my_pos = pos0 + pair_row + x * kTile + row;
+    const uint32_t s_tmem = tmem_S + lane_base;
+    const uint32_t o_tmem = tmem_O + lane_base;
+    const int my_pos = pos0 + row;
     const int my_first = args.chunk > 0 ? my_pos - my_pos % args.chunk : 0;   // first key this row may see
     float m_used = -INFINITY, l_sum = 0.f;
     bool ok = true;
     const uint64_t scale2 = pack2(args.scale_log2, args.scale_log2);
-    for (int j = my_lo; j < my_n; ++j) {
-      ok = mbar_wait(smem_u32(&s_full[x]), (j - my_lo) & 1, abort_flag, args.status, kStatusWaitTimeoutEpilogue);
+    for (int j = lo; j < n_kv; ++j) {
+      ok = mbar_wait(smem_u32(s_full), (j - lo) & 1, abort_flag, args.status, kStatusWaitTimeoutEpilogue);
       if (!ok) break;
       tc_fence_after();
       // columns [col_lo, col_hi] of this key tile are visible to the row (none, if the range is empty)
@@ -314,13 +261,13 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
       float mx = fmaxf(fmaxf(mxs[0], mxs[1]), fmaxf(mxs[2], mxs[3]));
       mx *= args.scale_log2;
       float alpha = 1.f;
-      if (j == my_lo) {
+      if (j == lo) {
         m_used = mx;                               // -inf when this row sees nothing in its tile's first key tile
       } else if (mx > m_used + kRescaleThreshold) {
         alpha = ex2(m_used - mx);                  // 0 when nothing was accumulated yet
         m_used = mx;
       }
-      if (j > my_lo && __any_sync(0xffffffffu, alpha != 1.f)) {
+      if (j > lo && __any_sync(0xffffffffu, alpha != 1.f)) {
         // S(j) is complete, so every earlier P V product has finished; the next one waits for p_ready below:
         // nobody else touches O now
 #pragma unroll
@@ -372,19 +319,19 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
       l_sum = l_sum * alpha + ((r0 + r1) + (r2 + r3));
       tmem_st_wait();
       tc_fence_before();
-      mbar_arrive(smem_u32(&p_ready[x]));
+      mbar_arrive(smem_u32(p_ready));
     }
-    if (my_n > 0) {
-      if (ok) ok = mbar_wait(smem_u32(&pv_done[x]), (my_n - 1 - my_lo) & 1, abort_flag, args.status, kStatusWaitTimeoutEpilogue);
+    if (n_kv > 0) {
+      if (ok) ok = mbar_wait(smem_u32(pv_done), (n_kv - 1 - lo) & 1, abort_flag, args.status, kStatusWaitTimeoutEpilogue);
       // one decision for the whole warpgroup (a thread that gave up above still arrives here)
-      ok = named_bar_and(bar_and, 128, ok);
+      ok = named_bar_and(2, 128, ok);
       if (ok) {
         tc_fence_after();
         // the sink joins the denominator on the scale of the sum; an enormous sink overflows to a zero weight of the keys
         const float den = args.sink ? l_sum + ex2(args.sink[head] * 1.4426950408889634f - m_used) : l_sum;
         const float inv_l = 1.f / den;
-        // every MMA that read Q_X has completed: its shared memory now stages the warp's 32 rows
-        uint8_t* stage = sQ + x * kStage;
+        // every MMA that read Q has completed: its shared memory now stages the warp's 32 rows
+        uint8_t* stage = sQ;
         uint8_t* orow = stage + row * 128;
 #pragma unroll
         for (int c = 0; c < HV / 32; ++c) {
@@ -403,12 +350,12 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
           }
         }
         __syncwarp();
-        const int rows = rows_x[x] - ew * 32;           // valid rows of this warp (may be negative)
+        const int my_rows = rows - ew * 32;             // valid rows of this warp (may be negative)
         const int vecs = args.DV / 8;
-        __nv_bfloat16* obase = args.out + (static_cast<size_t>(q0 + pair_row + x * kTile + ew * 32) * args.num_q_heads + head) * args.DV;
+        __nv_bfloat16* obase = args.out + (static_cast<size_t>(q0 + ew * 32) * args.num_q_heads + head) * args.DV;
         for (int i = lane; i < 32 * (HV / 8); i += 32) {
           const int rr = i / (HV / 8), c = i % (HV / 8);
-          if (rr < rows && c < vecs) {
+          if (rr < my_rows && c < vecs) {
             const int srow = ew * 32 + rr;
             const uint4 v = *reinterpret_cast<const uint4*>(stage + srow * 128 + (c >> 3) * kSubBytes + (((c & 7) ^ (srow & 7)) << 4));
             *reinterpret_cast<uint4*>(obase + static_cast<size_t>(rr) * args.num_q_heads * args.DV + c * 8) = v;
@@ -421,7 +368,7 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
   __syncthreads();
   if (warp == 1) {
     tc_fence_after();
-    tmem_dealloc(tmem_base, 512);
+    tmem_dealloc(tmem_base, 256);
   }
 }
 
@@ -445,8 +392,8 @@ template <int HQ, int HV>
 int launch(const CUtensorMap& tQ, const CUtensorMap& tK, const CUtensorMap& tV, const Args& a, int grid, cudaStream_t stream) {
   constexpr int QBYTES = HQ / 64 * kSubBytes, VBYTES = HV / 64 * kSubBytes;
   constexpr int STAGE = QBYTES > VBYTES ? QBYTES : VBYTES;
-  constexpr int SMEM = 2 * STAGE + 2 * QBYTES + 2 * VBYTES + 16 * 8 + 16 + 1024;
-  static_assert(SMEM <= 232448, "shared memory budget exceeded");
+  constexpr int SMEM = STAGE + QBYTES + VBYTES + 8 * 8 + 16 + 1024;
+  static_assert(2 * SMEM <= 232448, "shared memory budget exceeded");
   auto kern = paged_prefill_tc_kernel<HQ, HV>;
   static bool attr_set = false;
   if (!attr_set) {
@@ -474,7 +421,7 @@ int mfb_paged_prefill_tc_supported(int Hq, int Hkv, int D, int DV, int block_siz
 }
 
 // q [T, Hq, D], caches [num_blocks, block_size, Hkv, D | DV], out [T, Hq, DV], all bf16. work [n_work, 2] int32: (sequence,
-// first row of a 256-row pair inside its portion), for every pair of every sequence whose rows this launch computes.
+// first row of a 128-row tile inside its portion), for all rows of every sequence that this launch computes.
 int mfb_paged_prefill_tc(const void* q, const void* key_cache, const void* value_cache, const int* work, int n_work,
                          const int* cu_q, const int* block_tables, const int* context_lens, const float* sink, void* out, int T,
                          int Hq, int Hkv, int D, int DV, int num_blocks, int block_size, int max_blocks, int chunk, float scale,

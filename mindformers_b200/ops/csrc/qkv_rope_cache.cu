@@ -142,6 +142,126 @@ __global__ void __launch_bounds__(kThreads) qkv_rope_cache_kernel(const Args a) 
   }
 }
 
+// eight neighbours (16-byte aligned)
+__device__ __forceinline__ void ld8(const float* p, float (&v)[8]) {
+  const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
+  v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+}
+__device__ __forceinline__ void ld8(const __nv_bfloat16* p, float (&v)[8]) {
+  const uint4 u = *reinterpret_cast<const uint4*>(p);
+  const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&u);
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const float2 f = __bfloat1622float2(h[i]);
+    v[2 * i] = f.x; v[2 * i + 1] = f.y;
+  }
+}
+__device__ __forceinline__ void st8(float* p, const float (&v)[8]) {
+  *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+  *reinterpret_cast<float4*>(p + 4) = make_float4(v[4], v[5], v[6], v[7]);
+}
+__device__ __forceinline__ void st8(__nv_bfloat16* p, const float (&v)[8]) {
+  *reinterpret_cast<uint4*>(p) = make_uint4(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]), pack_bf16x2(v[4], v[5]),
+                                            pack_bf16x2(v[6], v[7]));
+}
+
+// Head sizes 32, 64, 128 and 256 with neighbouring pairs: LPH = D / 8 lanes hold a head, eight dimensions (four pairs)
+// each, so that a head is one 16-byte access per lane and a CTA works on 256 / LPH heads at a time.
+template <typename T, int LPH>
+__global__ void __launch_bounds__(kThreads) qkv_rope_cache_vec_kernel(const Args a) {
+  extern __shared__ float sh[];
+  constexpr int D = 8 * LPH, GROUPS = kThreads / LPH;
+  const long long t = blockIdx.x;
+  const int half = a.rot / 2;
+  float* sh_cos = sh;
+  float* sh_sin = sh + half;
+  const int slot = a.slots[t];
+  const float pos = static_cast<float>(a.positions[t]);
+  const int sub = threadIdx.x / LPH, e = (threadIdx.x % LPH) * 8;
+  const T* row = reinterpret_cast<const T*>(a.qkv) + t * a.ld_qkv;
+  const T* bias = reinterpret_cast<const T*>(a.bias);
+  // the first head of every group is on its way while the angles are evaluated
+  float x[8];
+  if (sub < a.H + a.G) ld8(row + (long long)sub * D + e, x);
+  for (int i = threadIdx.x; i < half; i += kThreads) {
+    float s, c;
+    sincosf(pos * a.freqs[i], &s, &c);
+    sh_cos[i] = c * a.amplitude;
+    sh_sin[i] = s * a.amplitude;
+  }
+  __syncthreads();
+  const int n_heads = a.H + a.G;
+  for (int h0 = 0; h0 < n_heads; h0 += GROUPS) {
+    const int h = h0 + sub;
+    const bool on = h < n_heads;              // the shuffles below name every lane of the warp
+    const bool is_q = h < a.H;
+    float cur[8];
+#pragma unroll
+    for (int i = 0; i < 8; ++i) cur[i] = on ? x[i] : 0.f;
+    if (h + GROUPS < n_heads) ld8(row + (long long)(h + GROUPS) * D + e, x);
+    if (on && bias) {
+      float b[8];
+      ld8(bias + (long long)h * D + e, b);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) cur[i] += b[i];
+    }
+    const T* nw = reinterpret_cast<const T*>(is_q ? a.q_norm : a.k_norm);
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) ss = fmaf(cur[i], cur[i], ss);
+#pragma unroll
+    for (int o = LPH / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    if (!on || (!is_q && slot < 0)) continue;
+    if (nw) {
+      const float rstd = 1.f / sqrtf(ss / D + a.eps);
+      float w[8];
+      ld8(nw + e, w);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) cur[i] = cur[i] * rstd * w[i];
+    }
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int p = e / 2 + i;
+      if (p < half) {
+        const float c = sh_cos[p], s = sh_sin[p];
+        const float u = cur[2 * i], v = cur[2 * i + 1];
+        cur[2 * i] = u * c - v * s;
+        cur[2 * i + 1] = v * c + u * s;
+      }
+    }
+    T* dst = is_q ? reinterpret_cast<T*>(a.q_out) + (t * a.H + h) * D
+                  : reinterpret_cast<T*>(a.key_cache) + ((long long)slot * a.G + (h - a.H)) * D;
+    st8(dst + e, cur);
+  }
+  if (slot >= 0) {
+    const int n = a.G * a.DV;
+    const long long off = (long long)n_heads * D;
+    T* dst = reinterpret_cast<T*>(a.value_cache) + (long long)slot * n;
+    for (int i = threadIdx.x * 8; i < n; i += kThreads * 8) {
+      float v[8];
+      ld8(row + off + i, v);
+      if (bias) {
+        float b[8];
+        ld8(bias + off + i, b);
+#pragma unroll
+        for (int k = 0; k < 8; ++k) v[k] += b[k];
+      }
+      st8(dst + i, v);
+    }
+  }
+}
+
+template <typename T>
+bool launch_vec(const Args& a, int T_rows, size_t smem, cudaStream_t stream) {
+  switch (a.D) {
+    case 32: qkv_rope_cache_vec_kernel<T, 4><<<T_rows, kThreads, smem, stream>>>(a); return true;
+    case 64: qkv_rope_cache_vec_kernel<T, 8><<<T_rows, kThreads, smem, stream>>>(a); return true;
+    case 128: qkv_rope_cache_vec_kernel<T, 16><<<T_rows, kThreads, smem, stream>>>(a); return true;
+    case 256: qkv_rope_cache_vec_kernel<T, 32><<<T_rows, kThreads, smem, stream>>>(a); return true;
+    default: return false;
+  }
+}
+
 bool al(const void* p, int n) { return (reinterpret_cast<uintptr_t>(p) & (n - 1)) == 0; }
 
 }  // namespace qrc
@@ -168,6 +288,14 @@ int mfb_qkv_rope_cache(const void* qkv, long long ld_qkv, const void* bias, cons
   a.paired = (D % 2 == 0 && (G * DV) % 2 == 0 && ld_qkv % 2 == 0 && qrc::al(qkv, two) && qrc::al(bias, two) &&
               qrc::al(q_out, two) && qrc::al(key_cache, two) && qrc::al(value_cache, two)) ? 1 : 0;
   const size_t smem = (size_t)rot * sizeof(float);
+  const bool vec = interleaved && (G * DV) % 8 == 0 && ld_qkv % 8 == 0 && qrc::al(qkv, 16) && qrc::al(bias, 16) &&
+                   qrc::al(q_norm, 16) && qrc::al(k_norm, 16) && qrc::al(q_out, 16) && qrc::al(key_cache, 16) &&
+                   qrc::al(value_cache, 16);
+  const bool done = vec && (f32 ? qrc::launch_vec<float>(a, T, smem, stream) : qrc::launch_vec<__nv_bfloat16>(a, T, smem, stream));
+  if (done) {
+    if (cudaGetLastError() != cudaSuccess) { mfb_host::set_error("qkv_rope_cache: launch failed"); return 2; }
+    return 0;
+  }
   if (f32) qrc::qkv_rope_cache_kernel<float><<<T, qrc::kThreads, smem, stream>>>(a);
   else qrc::qkv_rope_cache_kernel<__nv_bfloat16><<<T, qrc::kThreads, smem, stream>>>(a);
   if (cudaGetLastError() != cudaSuccess) { mfb_host::set_error("qkv_rope_cache: launch failed"); return 2; }

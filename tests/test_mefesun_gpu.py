@@ -92,7 +92,7 @@ def test_linear_with_activation(dtype, M, N, K, act):
 
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("H,G,D,DV,rot", [(4, 2, 64, 64, 64), (6, 2, 40, 24, 16), (5, 1, 128, 128, 96), (3, 3, 20, 36, 12),
-                                          (2, 1, 144, 12, 144), (8, 8, 16, 16, 0), (2, 2, 7, 5, 4)])
+                                          (2, 1, 144, 12, 144), (34, 9, 64, 32, 40), (17, 1, 256, 8, 256), (70, 2, 32, 4, 6), (8, 8, 16, 16, 0), (2, 2, 7, 5, 4)])
 @pytest.mark.parametrize("interleaved", [True, False])
 def test_qkv_rope_cache(dtype, H, G, D, DV, rot, interleaved):
     T, bs, blocks, eps = 9, 16, 5, 1e-3
