@@ -8,6 +8,7 @@ from __future__ import annotations
 
 import copy
 
+from ..parallel.transformer_config_utils import ALIASES
 from ..tools.register import MindFormerModuleType, MindFormerRegister
 from .configuration_utils import PretrainedConfig
 from .modeling_utils import PreTrainedModel
@@ -192,25 +193,33 @@ class MefesunConfig(PretrainedConfig):
                 beta_fast=float(scaling["fast"]), beta_slow=float(scaling["slow"])),
             ffn_hidden_size=int(mlp["ff"]) if mlp else 0)
 
+    def _owner(self, i: int) -> int:
+        """The layer whose weights layer ``i`` runs with."""
+        for _ in self.layers:
+            j = self.layers[i].get("weights_of")
+            if j is None:
+                return i
+            i = int(j)
+        raise ValueError("weights_of: layers name one another in a circle")
+
     def to_transformer_dict(self) -> dict:
         d = {k: v for k, v in self.to_dict().items()
              if k not in ("architecture", "layers", "norm", "vocab", "width", "mlp", "mixer")}
         fields = [self._layer_fields(i, layer) for i, layer in enumerate(self.layers)]
-        owners = []
-        for i, layer in enumerate(self.layers):
-            j = layer.get("weights_of")
-            owners.append(i if j is None else owners[int(j)])
-        d.update({k: v for k, v in fields[0].items() if k != "rope_scaling"})
+        owners = [self._owner(i) for i in range(len(fields))]
         d.setdefault("seq_length", max(int(f["rope_scaling"]["factor"] * f["rope_scaling"]["original_max_position_embeddings"])
                                        if f["rope_scaling"] else 4096 for f in fields))
         d.setdefault("max_position_embeddings", d["seq_length"])
-        d.update(vocab_size=int(self.vocab), hidden_size=int(self.width), num_layers=len(fields), layer_overrides=fields,
+        own = {k: v for k, v in fields[0].items() if k != "rope_scaling"}
+        own.update(vocab_size=int(self.vocab), hidden_size=int(self.width), num_layers=len(fields), layer_overrides=fields,
                  layer_sharing=owners, layernorm_epsilon=float(self.norm["eps"]), normalization="LayerNorm",
                  norm_placement="output", layer_scale=True, fp32_residual_connection=True, ragged_attention=True,
                  qk_layernorm=True, add_qkv_bias=True, add_attention_output_bias=True, attention_sink=True,
                  rotary_interleaved=True, gated_linear_unit=False, hidden_act="relu2", position_embedding_type="none",
                  tie_word_embeddings=True, logit_softcap=float(self.logit_softcap) if self.logit_softcap else None)
-        return d
+        # other spellings of what the design's own keys describe do not apply
+        d = {k: v for k, v in d.items() if ALIASES.get(k, (k,))[0] not in own}
+        return dict(d, **own)
 
 
 for _legacy in (True, False):

@@ -53,6 +53,12 @@ PRESETS = {
         rope_interleave=True,
         rope_scaling=dict(type="yarn", factor=40.0, beta_fast=32.0, beta_slow=1.0, mscale=1.0, mscale_all_dim=1.0,
                           original_max_position_embeddings=4096)),
+    "tiny_mefesun": dict(
+        model_type="mefesun", vocab=1024, width=256, norm=dict(eps=1e-6), logit_softcap=30.0,
+        layers=[dict(type="attention",
+                     mixer=dict(heads=8, kv_heads=2, dim=32, vdim=32, scale=32 ** -0.5, mask=dict(size=128),
+                                rot=dict(base=10000.0, dims=32, scaling=dict(factor=4.0, original=256, fast=32.0, slow=1.0))),
+                     mlp=dict(kind="dense", ff=768)) for _ in range(2)]),
     "tiny_llama": dict(
         model_type="llama", num_hidden_layers=2, hidden_size=256, num_attention_heads=4, num_key_value_heads=2,
         intermediate_size=688, vocab_size=1024, rms_norm_eps=1e-5, rope_theta=10000.0,

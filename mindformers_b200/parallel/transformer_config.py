@@ -327,8 +327,8 @@ class TransformerConfig(ModelParallelConfig):
             val = getattr(self, name)
             if val is not None and len(val) != self.num_layers:
                 raise ValueError(f"{name} must have num_layers ({self.num_layers}) entries, got {len(val)}")
-        if self.layer_sharing and any(self.layer_sharing[j] != j or j > i for i, j in enumerate(self.layer_sharing)):
-            raise ValueError("layer_sharing must name an earlier layer that has weights of its own")
+        if self.layer_sharing and any(self.layer_sharing[j] != j for j in self.layer_sharing):
+            raise ValueError("layer_sharing must name layers that have weights of their own")
         if self.tie_word_embeddings:
             self.untie_embeddings_and_output_weights = False
         if self.use_scaled_init and self.num_layers:

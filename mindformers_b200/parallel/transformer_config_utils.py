@@ -108,6 +108,8 @@ for _target, _aliases, _fn in _TABLE:
     for _a in _aliases:
         _ALIAS[_a] = (_target, _fn)
 
+ALIASES = _ALIAS          # spelling -> (field, transform)
+
 # keys that a model configuration may carry without a TransformerConfig counterpart
 DEFAULT_WHITE_KEYS = {
     # resolved into model_parallel / context_parallel before the model is built (core/context.py)

@@ -161,12 +161,14 @@ def main(argv=None):
     ap.add_argument("--num_blocks", type=int, default=None)
     ap.add_argument("--max_prefill_tokens", type=int, default=8192)
     ap.add_argument("--model_name", default=None)
+    ap.add_argument("--tokenizer", default=None, help="tokenizer directory (default: --model_dir), or 'byte'")
+    ap.add_argument("--dtype", default=None, help="bfloat16 (default) or float32")
     a = ap.parse_args(argv)
     import uvicorn
 
     from ..models import AutoModelForCausalLM, AutoTokenizer
-    model = AutoModelForCausalLM.from_pretrained(a.model_dir)
-    tokenizer = AutoTokenizer.from_pretrained(a.model_dir)
+    model = AutoModelForCausalLM.from_pretrained(a.model_dir, **({"dtype": a.dtype} if a.dtype else {}))
+    tokenizer = AutoTokenizer.from_pretrained(a.tokenizer or a.model_dir)
     engine = ServingEngine(model, a.max_num_seqs, a.max_model_len, a.num_blocks, a.max_prefill_tokens,
                            eos_token_id=getattr(tokenizer, "eos_token_id", None))
     app = build_app(engine, tokenizer, a.model_name or a.model_dir.rstrip("/").split("/")[-1])

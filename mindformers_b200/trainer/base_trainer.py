@@ -353,9 +353,15 @@ class BaseTrainer:
         from ..models import build_tokenizer
         from ..pipeline import pipeline
         self.config = config
-        model = network if network is not None else build_network(config.get("model") or {})
         path = config.get("load_checkpoint") or config.get("pretrained_model_dir")
-        if path and network is None:
+        section = config.get("model") or {}
+        whole = network is None and not section.get("model_config") and os.path.isfile(os.path.join(str(path), "config.json"))
+        if whole:                        # no ``model.model_config``: the directory's config.json describes the model
+            from ..models import AutoModel
+            model = AutoModel.from_pretrained(path, strict=True)
+        else:
+            model = network if network is not None else build_network(section)
+        if path and network is None and not whole:
             model.load_weights(path, strict=False)
         if network is None and hasattr(model, "apply_quantization_config"):
             # ``model.model_config.quantization_config`` or a top-level ``quantization_config`` section of the YAML

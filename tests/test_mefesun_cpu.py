@@ -50,6 +50,11 @@ def test_config_resolves_by_architecture_and_describes_every_layer(checkpoint):
             mix["heads"], mix["kv_heads"], mix["dim"], mix["vdim"], mix["mask"]["size"], mix["rot"]["dims"])
         assert c.softmax_scale == mix["scale"] and c.ffn_hidden_size == (layer["mlp"]["ff"] if layer["mlp"] else 0)
     assert m.model.decoder.layers[1].mlp is None
+    loop = [dict(cfg["layers"][0], weights_of=1), dict(cfg["layers"][0], weights_of=0)]
+    with pytest.raises(ValueError, match="circle"):
+        MefesunConfig(**dict(cfg, layers=loop)).to_transformer_dict()
+    ahead = [dict(cfg["layers"][0], weights_of=1), cfg["layers"][0]]
+    assert MefesunConfig(**dict(cfg, layers=ahead)).to_transformer_dict()["layer_sharing"] == [1, 1]
     with pytest.raises(ValueError, match="unknown mixer"):
         MefesunConfig(**dict(cfg, layers=[dict(cfg["layers"][0], type="other")])).to_transformer_dict()
 
@@ -177,6 +182,21 @@ def test_greedy_generation_through_generate_and_the_engine(checkpoint, model):
         assert engine.counters["mixed_steps"] >= 3 and engine.stats()["free_blocks"] == engine.stats()["total_blocks"]
     beams = model.generate(prompts[:1], max_new_tokens=4, num_beams=2, do_sample=False, eos_token_id=None)
     assert len(beams[0]) == len(prompts[0]) + 4
+
+
+def test_command_line_predict(checkpoint, tmp_path):
+    """``run_mindformer.py --run_mode predict`` on a model directory: greedy text of the plain implementation."""
+    path, cfg, w = checkpoint
+    yaml = tmp_path / "p.yaml"
+    yaml.write_text("run_mode: predict\nuse_parallel: false\nuse_legacy: false\noutput_dir: " + str(tmp_path) + "\n"
+                    "trainer: {type: CausalLanguageModelingTrainer, model_name: Mefesun}\n"
+                    "processor: {tokenizer: {type: ByteTokenizer}}\n")
+    root = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
+    env = dict(os.environ, CUDA_VISIBLE_DEVICES="")
+    res = subprocess.run([sys.executable, os.path.join(root, "run_mindformer.py"), "--config", str(yaml), "--run_mode", "predict",
+                          "--pretrained_model_dir", path, "--predict_data", "abc", "--save_file", str(tmp_path / "out.txt")],
+                         capture_output=True, text=True, timeout=300, env=env, cwd=str(tmp_path))
+    assert res.returncode == 0 and "abc" in (tmp_path / "out.txt").read_text(), res.stdout[-1500:] + res.stderr[-3000:]
 
 
 def test_sampling_is_seeded(model):
