@@ -18,26 +18,36 @@ TILE = 128               # query rows of a tile of the prefill kernel
 
 
 def prefill_work(q_lens, context_lens, chunk: int = 0):
-    """Work list of the prefill kernel: ``[(sequence, first row of a 128-row tile)]`` of every sequence with more than one
-    new row, the tiles that see the most key tiles first."""
-    items = []
+    """Work list of the prefill kernel: ``[(sequence, first row of q, rows, position of the first row)]``, a 128-row tile
+    each, of every sequence with more than one new row; the tiles that see the most key tiles come first."""
+    items, q0 = [], 0
     for b, (n, ctx) in enumerate(zip(q_lens, context_lens)):
-        if n > 1:
-            for r in range(0, n, TILE):
-                first, last = ctx - n + r, min(ctx - n + r + TILE, ctx) - 1
-                lo = first - first % chunk if chunk > 0 else 0
-                items.append((last // TILE - lo // TILE, b, r))
-    items.sort(key=lambda t: -t[0])
-    return [(b, r) for _, b, r in items]
+        for r in range(0, n if n > 1 else 0, TILE):
+            pos, rows = ctx - n + r, min(TILE, n - r)
+            lo = pos - pos % chunk if chunk > 0 else 0
+            items.append((lo // TILE - (pos + rows - 1) // TILE, (b, q0 + r, rows, pos)))
+        q0 += n
+    items.sort(key=lambda t: t[0])
+    return [item for _, item in items]
+
+
+# mean key tiles per query tile up to which the kernel's persistent form is used (``set_persistent_prefill`` fixes it)
+_PERSISTENT_UP_TO = 8.0
+
+
+def set_persistent_prefill(up_to: float) -> None:
+    global _PERSISTENT_UP_TO
+    _PERSISTENT_UP_TO = float(up_to)
 
 
 def _work_on_device(cache, chunk: int):
-    """The step's work list for ``chunk`` as an int32 device tensor, made once per step (layers with the same chunk share
-    it)."""
+    """The step's work list for ``chunk`` as an int32 device tensor, and whether the persistent form of the kernel runs it;
+    made once per step (layers with the same chunk share it)."""
     work = cache.prefill_work.get(chunk)
     if work is None:
         items = prefill_work(cache.q_lens_host, cache.context_lens_host, chunk)
-        work = torch.tensor(items, dtype=torch.int32).to(cache.block_tables.device)
+        keys = sum((p + n - 1) // TILE - (p - p % chunk if chunk > 0 else 0) // TILE + 1 for _, _, n, p in items)
+        work = (torch.tensor(items, dtype=torch.int32).to(cache.block_tables.device), keys <= _PERSISTENT_UP_TO * len(items))
         cache.prefill_work[chunk] = work
     return work
 
@@ -97,9 +107,10 @@ def ragged_attention(q: torch.Tensor, cache, layer: int, scale: float, chunk: in
         return out.view(T, Hq * DV)
     status = _lib.status_word(q.device).data_ptr()
     if ragged and cache.n_long_rows:
-        work = _work_on_device(cache, int(chunk))
-        rc = lib.mfb_paged_prefill_tc(q.data_ptr(), kc.data_ptr(), vc.data_ptr(), work.data_ptr(), work.shape[0], cu, tables, lens, snk, out.data_ptr(), T, Hq, Hkv, D, DV, nb, bs,
-                                      max_blocks, int(chunk), float(scale), status, _lib.stream_ptr())
+        work, persistent = _work_on_device(cache, int(chunk))
+        rc = lib.mfb_paged_prefill_tc(q.data_ptr(), kc.data_ptr(), vc.data_ptr(), work.data_ptr(), work.shape[0], int(persistent),
+                                      tables, snk, out.data_ptr(), T, Hq, Hkv, D, DV, nb, bs, max_blocks, int(chunk),
+                                      float(scale), status, _lib.stream_ptr())
         _lib.check(rc, "mfb_paged_prefill_tc")
         _lib.count_launch()
     if not ragged or cache.n_single_rows:

@@ -142,7 +142,7 @@ def _declare(lib):
     sig("mfb_paged_decode_tc_supported_ex", [I, I, I, I, I])
     sig("mfb_paged_decode_attention_tc_ex", [P] * 9 + [I] * 11 + [F, P, P])
     sig("mfb_paged_prefill_tc_supported", [I, I, I, I, I])
-    sig("mfb_paged_prefill_tc", [P, P, P, P, I, P, P, P, P, P] + [I] * 9 + [F, P, P])
+    sig("mfb_paged_prefill_tc", [P, P, P, P, I, I, P, P, P] + [I] * 9 + [F, P, P])
     sig("mfb_paged_attention_any", [P] * 8 + [I] * 9 + [F, I, P])
     sig("mfb_qkv_rope_cache", [P, L, P, P, P, F, P, F, I, I, P, P, P, P, P, I, I, I, I, I, I, P])
     sig("mfb_add_normed", [P, L, P, P, P, P, P, I, P, P, I, I, I, F, I, P])

@@ -8,20 +8,23 @@
 //
 // The tensor-core pipeline is the one of flash_attention_fwd2.cu (P goes back into tensor memory and is read from there
 // by the P V product), with one 128-row query tile per CTA and one stage of K and of V: a CTA then takes half of an SM's
-// tensor memory and at most half of its shared memory, and two of them share an SM. While one waits for its products or
-// its softmax the other works, and the start and the end of a CTA run under the products of its neighbour, which is what
-// counts when a tile sees few keys (chunks, short portions). K of the next key tile loads during the softmax of this one,
-// V during the scores and the softmax, so one stage of each is enough. What else differs:
-//   - work comes as a list of (sequence, first row of the tile); only key tiles that some row of the tile sees are
-//     visited, from the chunk of its first row to its last row;
+// tensor memory and at most half of its shared memory, and two of them share an SM: while one waits for its products or
+// its softmax the other works. K of the next key tile loads during the softmax of this one, V during the scores and the
+// softmax, so one stage of each is enough. A CTA's roles run through all of its tiles (see the launcher): the
+// loads and the first scores of a tile run under the last softmax and the output of the one before, which is what counts
+// when a tile sees few keys (chunks, short portions). What else differs:
+//   - work comes as a list of (sequence, first row of q, rows, position of the first row), one entry per query tile; only
+//     key tiles that some row of the tile sees are visited, from the chunk of its first row to its last row;
 //   - K / V tiles (128 consecutive positions) are assembled from the sequence's pages, one TMA box per page and 64
 //     columns; pages past the end of the sequence repeat the tile's first page and are masked;
 //   - head sizes are padded to 64 or 128 columns: q is read through a three-dimensional map that fills the columns past
 //     the head with zeros, so whatever a K box holds there does not count; columns of V past the head reach only
 //     columns of the result that are not stored;
-//   - the result is staged in shared memory and written row by row: a portion may end anywhere.
+//   - the result is written row by row: a portion may end anywhere.
 //
 // Roles (192 threads): warp 0 TMA producer, warp 1 MMA issuer + TMEM owner, warps 2..5 softmax. Every wait is bounded (common.cuh).
+#include <type_traits>
+
 #include "common.cuh"
 
 namespace mfb {
@@ -33,10 +36,9 @@ constexpr int kSubBytes = kTile * 128;     // [128 rows][128 B] swizzled sub-til
 constexpr float kRescaleThreshold = 8.0f;  // log2 units
 
 struct Args {
-  const int* work;           // [n_work, 2]: sequence, first row of the tile inside the portion
-  const int* cu_q;           // [B + 1]
+  const int4* work;          // [n_work]: sequence, first row of q, rows, position of the first row
+  int n_items;               // n_work x query heads: item i is tile i / heads of head i % heads
   const int* block_tables;   // [B, max_blocks]
-  const int* context_lens;   // [B]
   const float* sink;         // [Hq] or null
   __nv_bfloat16* out;        // [T, Hq, DV]
   int num_q_heads, group, D, DV, block_size, max_blocks, chunk;
@@ -91,14 +93,14 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
                         const __grid_constant__ CUtensorMap tmV, const Args args) {
   constexpr int QB = HQ / 64, VB = HV / 64;          // 64-column sub-tiles
   constexpr int kQBytes = QB * kSubBytes, kVBytes = VB * kSubBytes;
-  constexpr int kStage = kQBytes > kVBytes ? kQBytes : kVBytes;   // a Q tile's buffer also stages its result
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) &
                                              ~static_cast<uintptr_t>(1023));
   uint8_t* sQ = smem;
-  uint8_t* sK = sQ + kStage;
+  uint8_t* sK = sQ + kQBytes;
   uint8_t* sV = sK + kQBytes;
-  uint64_t* bars = reinterpret_cast<uint64_t*>(sV + kVBytes);
+  uint8_t* sOut = sV + kVBytes;               // 2 KB per softmax warp
+  uint64_t* bars = reinterpret_cast<uint64_t*>(sOut + 4 * 2048);
   uint64_t* q_full = bars;
   uint64_t* k_full = bars + 1;
   uint64_t* k_empty = bars + 2;
@@ -107,25 +109,26 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
   uint64_t* s_full = bars + 5;      // S complete
   uint64_t* p_ready = bars + 6;     // P written (128 arrivals)
   uint64_t* pv_done = bars + 7;     // P V complete
-  uint32_t* tmem_holder = reinterpret_cast<uint32_t*>(bars + 8);
+  uint64_t* q_empty = bars + 8;     // last scores of a query tile complete
+  uint32_t* tmem_holder = reinterpret_cast<uint32_t*>(bars + 9);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_holder + 1);
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int head = static_cast<int>(blockIdx.x) % args.num_q_heads;
-  const int item = static_cast<int>(blockIdx.x) / args.num_q_heads;
-  const int b = args.work[2 * item], row0 = args.work[2 * item + 1];
-  const int q0 = args.cu_q[b] + row0;                // the tile's first row of q
-  const int len = args.context_lens[b];
-  const int rows = args.cu_q[b + 1] - q0 < kTile ? args.cu_q[b + 1] - q0 : kTile;
-  const int pos0 = len - (args.cu_q[b + 1] - q0);    // its position
-  const int kv_head = head / args.group;
-  // key tiles lo .. n_kv - 1
-  const int lo = args.chunk > 0 ? (pos0 - pos0 % args.chunk) / kTile : 0;
-  const int n_kv = rows > 0 ? (pos0 + rows - 1) / kTile + 1 : 0;
+  struct Tile { int b, head, q0, rows, pos0, lo, n_kv; };      // key tiles lo .. n_kv - 1
+  auto tile_of = [&](int item) {
+    const int4 w = args.work[item / args.num_q_heads];
+    Tile t;
+    t.head = item % args.num_q_heads;
+    t.b = w.x; t.q0 = w.y; t.rows = w.z; t.pos0 = w.w;
+    t.lo = args.chunk > 0 ? (t.pos0 - t.pos0 % args.chunk) / kTile : 0;
+    t.n_kv = (t.pos0 + t.rows - 1) / kTile + 1;
+    return t;
+  };
+  const int first_item = static_cast<int>(blockIdx.x), step = static_cast<int>(gridDim.x);
 
   if (threadIdx.x == 0) {
     *abort_flag = 0;
-    for (int i = 0; i < 8; ++i) mbar_init(smem_u32(&bars[i]), &bars[i] == p_ready ? 128 : 1);
+    for (int i = 0; i < 9; ++i) mbar_init(smem_u32(&bars[i]), &bars[i] == p_ready ? 128 : 1);
     fence_barrier_init();
     tma_prefetch_desc(&tmQ);
     tma_prefetch_desc(&tmK);
@@ -142,65 +145,76 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
   const uint32_t tmem_S = tmem_base, tmem_O = tmem_base + kTile;   // P lives in the first 64 columns of S
   if (warp == 0) {
     // ------------------------------ TMA producer ------------------------------
-    if (lane == 0 && n_kv > 0) {
-      const uint32_t qb = smem_u32(q_full);
-      mbar_expect_tx(qb, kQBytes);
-      for (int c = 0; c < QB; ++c) tma_load_3d(smem_u32(sQ) + c * kSubBytes, &tmQ, qb, c * 64, head, q0);
+    if (lane == 0) {
       const int bs = args.block_size;
       const int pages = kTile / bs;
-      const int* table = args.block_tables + static_cast<size_t>(b) * args.max_blocks;
-      const int kcol = kv_head * args.D, vcol = kv_head * args.DV;
+      uint32_t it = 0, n = 0;                      // key tiles and query tiles so far
       bool ok = true;
-      for (int j = lo; j < n_kv && ok; ++j) {
-        const uint32_t ph = (j - lo) & 1;
-        const int tok0 = j * kTile;
-        const int first_page = table[tok0 / bs];
-        ok = mbar_wait(smem_u32(k_empty), ph ^ 1, abort_flag, args.status, kStatusWaitTimeoutProducer);
+      for (int item = first_item; item < args.n_items && ok; item += step, ++n) {
+        const Tile t = tile_of(item);
+        ok = mbar_wait(smem_u32(q_empty), (n & 1) ^ 1, abort_flag, args.status, kStatusWaitTimeoutProducer);
         if (!ok) break;
-        const uint32_t kb = smem_u32(k_full);
-        mbar_expect_tx(kb, kQBytes);
-        const uint32_t kd = smem_u32(sK);
-        for (int i = 0; i < pages; ++i) {
-          const int pg = tok0 + i * bs < len ? table[tok0 / bs + i] : first_page;
-          for (int c = 0; c < QB; ++c) tma_load_2d(kd + c * kSubBytes + i * bs * 128, &tmK, kb, kcol + c * 64, pg * bs);
-        }
-        ok = mbar_wait(smem_u32(v_empty), ph ^ 1, abort_flag, args.status, kStatusWaitTimeoutProducer);
-        if (!ok) break;
-        const uint32_t vb = smem_u32(v_full);
-        mbar_expect_tx(vb, kVBytes);
-        const uint32_t vd = smem_u32(sV);
-        for (int i = 0; i < pages; ++i) {
-          const int pg = tok0 + i * bs < len ? table[tok0 / bs + i] : first_page;
-          for (int c = 0; c < VB; ++c) tma_load_2d(vd + c * kSubBytes + i * bs * 128, &tmV, vb, vcol + c * 64, pg * bs);
+        const uint32_t qb = smem_u32(q_full);
+        mbar_expect_tx(qb, kQBytes);
+        for (int c = 0; c < QB; ++c) tma_load_3d(smem_u32(sQ) + c * kSubBytes, &tmQ, qb, c * 64, t.head, t.q0);
+        const int* table = args.block_tables + static_cast<size_t>(t.b) * args.max_blocks;
+        const int kv_head = t.head / args.group, end = t.pos0 + t.rows;
+        const int kcol = kv_head * args.D, vcol = kv_head * args.DV;
+        for (int j = t.lo; j < t.n_kv; ++j, ++it) {
+          const uint32_t ph = it & 1;
+          const int tok0 = j * kTile;
+          const int first_page = table[tok0 / bs];
+          ok = mbar_wait(smem_u32(k_empty), ph ^ 1, abort_flag, args.status, kStatusWaitTimeoutProducer);
+          if (!ok) break;
+          const uint32_t kb = smem_u32(k_full);
+          mbar_expect_tx(kb, kQBytes);
+          const uint32_t kd = smem_u32(sK);
+          for (int i = 0; i < pages; ++i) {
+            const int pg = tok0 + i * bs < end ? table[tok0 / bs + i] : first_page;
+            for (int c = 0; c < QB; ++c) tma_load_2d(kd + c * kSubBytes + i * bs * 128, &tmK, kb, kcol + c * 64, pg * bs);
+          }
+          ok = mbar_wait(smem_u32(v_empty), ph ^ 1, abort_flag, args.status, kStatusWaitTimeoutProducer);
+          if (!ok) break;
+          const uint32_t vb = smem_u32(v_full);
+          mbar_expect_tx(vb, kVBytes);
+          const uint32_t vd = smem_u32(sV);
+          for (int i = 0; i < pages; ++i) {
+            const int pg = tok0 + i * bs < end ? table[tok0 / bs + i] : first_page;
+            for (int c = 0; c < VB; ++c) tma_load_2d(vd + c * kSubBytes + i * bs * 128, &tmV, vb, vcol + c * 64, pg * bs);
+          }
         }
       }
     }
     __syncwarp();
   } else if (warp == 1) {
     // ------------------------------ MMA issuer ------------------------------
-    if (lane == 0 && n_kv > 0) {
+    if (lane == 0) {
       constexpr uint32_t IDESC_QK = umma_idesc_bf16(kTile, kTile, 0, 0);  // A = Q K-major (smem), B = K K-major
       constexpr uint32_t IDESC_PV = umma_idesc_bf16(kTile, HV, 0, 1);     // A = P (tensor memory), B = V MN-major
       const uint32_t qa = smem_u32(sQ), ka = smem_u32(sK), va = smem_u32(sV);
-      bool ok = mbar_wait(smem_u32(q_full), 0, abort_flag, args.status, kStatusWaitTimeoutMma);
-      for (int j = lo; j <= n_kv && ok; ++j) {
-        if (j > lo) {
-          // ---- O += P(j - 1) V(j - 1) ----
-          const uint32_t ph = (j - 1 - lo) & 1;
-          ok = mbar_wait(smem_u32(v_full), ph, abort_flag, args.status, kStatusWaitTimeoutMma);
-          if (ok) ok = mbar_wait(smem_u32(p_ready), ph, abort_flag, args.status, kStatusWaitTimeoutMma);
-          if (!ok) break;
-          tc_fence_after();
+      uint32_t it = 0, n = 0;
+      bool ok = true, first_key = true;          // first_key: the pending P V product starts its query tile's sum
+      // O (+)= P V of key tile it - 1
+      auto issue_pv = [&]() {
+        const uint32_t ph = (it - 1) & 1;
+        ok = mbar_wait(smem_u32(v_full), ph, abort_flag, args.status, kStatusWaitTimeoutMma);
+        if (ok) ok = mbar_wait(smem_u32(p_ready), ph, abort_flag, args.status, kStatusWaitTimeoutMma);
+        if (!ok) return;
+        tc_fence_after();
 #pragma unroll
-          for (int k = 0; k < kTile / 16; ++k)           // bf16 pairs: 8 columns of P per 16 keys
-            umma_f16_ts(tmem_O, tmem_S + k * 8, umma_desc_mnmajor_sw128(va + k * 16 * 128, kSubBytes), IDESC_PV,
-                        (j - 1 > lo || k > 0) ? 1u : 0u);
-          umma_commit(smem_u32(pv_done));
-          umma_commit(smem_u32(v_empty));
-        }
-        if (j < n_kv) {
+        for (int k = 0; k < kTile / 16; ++k)           // bf16 pairs: 8 columns of P per 16 keys
+          umma_f16_ts(tmem_O, tmem_S + k * 8, umma_desc_mnmajor_sw128(va + k * 16 * 128, kSubBytes), IDESC_PV,
+                      (!first_key || k > 0) ? 1u : 0u);
+        umma_commit(smem_u32(pv_done));
+        umma_commit(smem_u32(v_empty));
+      };
+      for (int item = first_item; item < args.n_items && ok; item += step, ++n) {
+        const Tile t = tile_of(item);
+        for (int j = t.lo; j < t.n_kv; ++j) {
+          if (it > 0) issue_pv();
+          if (ok && j == t.lo) ok = mbar_wait(smem_u32(q_full), n & 1, abort_flag, args.status, kStatusWaitTimeoutMma);
           // ---- S = Q K(j)^T: overwrites S / P, executes behind the P V product issued just above ----
-          ok = mbar_wait(smem_u32(k_full), (j - lo) & 1, abort_flag, args.status, kStatusWaitTimeoutMma);
+          if (ok) ok = mbar_wait(smem_u32(k_full), it & 1, abort_flag, args.status, kStatusWaitTimeoutMma);
           if (!ok) break;
           tc_fence_after();
 #pragma unroll
@@ -210,8 +224,12 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
           }
           umma_commit(smem_u32(s_full));
           umma_commit(smem_u32(k_empty));
+          if (j == t.n_kv - 1) umma_commit(smem_u32(q_empty));
+          first_key = j == t.lo;
+          ++it;
         }
       }
+      if (ok && it > 0) issue_pv();
     }
     __syncwarp();
   } else {
@@ -221,147 +239,175 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
     const uint32_t lane_base = static_cast<uint32_t>(ew * 32) << 16;
     const uint32_t s_tmem = tmem_S + lane_base;
     const uint32_t o_tmem = tmem_O + lane_base;
-    const int my_pos = pos0 + row;
-    const int my_first = args.chunk > 0 ? my_pos - my_pos % args.chunk : 0;   // first key this row may see
-    float m_used = -INFINITY, l_sum = 0.f;
     bool ok = true;
     const uint64_t scale2 = pack2(args.scale_log2, args.scale_log2);
-    for (int j = lo; j < n_kv; ++j) {
-      ok = mbar_wait(smem_u32(s_full), (j - lo) & 1, abort_flag, args.status, kStatusWaitTimeoutEpilogue);
-      if (!ok) break;
-      tc_fence_after();
-      // columns [col_lo, col_hi] of this key tile are visible to the row (none, if the range is empty)
-      const int col_lo = my_first - j * kTile;
-      const int col_hi = my_pos - j * kTile;
-      const bool masked = __any_sync(0xffffffffu, col_lo > 0 || col_hi < kTile - 1);
-      // pass 1: row maximum (four independent chains of three-input maxima); the scores are not kept
-      float mxs[4];
-      {
-        uint32_t sr[kTile];
+    uint32_t it = 0;
+    for (int item = first_item; item < args.n_items; item += step) {
+      const Tile t = tile_of(item);
+      const int lo = t.lo, n_kv = t.n_kv;
+      const int my_pos = t.pos0 + row;
+      const int my_first = args.chunk > 0 ? my_pos - my_pos % args.chunk : 0;   // first key this row may see
+      float m_used = -INFINITY, l_sum = 0.f;
+      for (int j = lo; j < n_kv; ++j, ++it) {
+        ok = mbar_wait(smem_u32(s_full), it & 1, abort_flag, args.status, kStatusWaitTimeoutEpilogue);
+        if (!ok) break;
+        tc_fence_after();
+        // columns [col_lo, col_hi] of this key tile are visible to the row (none, if the range is empty)
+        const int col_lo = my_first - j * kTile;
+        const int col_hi = my_pos - j * kTile;
+        // the bounds grow with the row: blocks of columns that every row of the warp sees need no mask, and halves that
+        // no row sees no exponentials
+        const int hi_min = __shfl_sync(0xffffffffu, col_hi, 0), hi_max = __shfl_sync(0xffffffffu, col_hi, 31);
+        const int lo_min = __shfl_sync(0xffffffffu, col_lo, 0), lo_max = __shfl_sync(0xffffffffu, col_lo, 31);
+        // the softmax of one key tile, compiled twice: tiles that every row of the warp sees whole carry no masking code
+        auto softmax_tile = [&](auto mask_tag) {
+          constexpr bool MASK = decltype(mask_tag)::value;
+          // pass 1: row maximum (four independent chains of three-input maxima); the scores are not kept
+          float mxs[4];
+          {
+            uint32_t sr[kTile];
 #pragma unroll
-        for (int c = 0; c < 4; ++c) {
-          uint32_t (&r)[32] = *reinterpret_cast<uint32_t(*)[32]>(&sr[c * 32]);
-          tmem_ld_32x32b_x32(s_tmem + c * 32, r);
-        }
-        tmem_ld_wait();
-        float* s = reinterpret_cast<float*>(sr);
-        if (masked) {
+            for (int c = 0; c < 4; ++c) {
+              uint32_t (&r)[32] = *reinterpret_cast<uint32_t(*)[32]>(&sr[c * 32]);
+              tmem_ld_32x32b_x32(s_tmem + c * 32, r);
+            }
+            tmem_ld_wait();
+            float* s = reinterpret_cast<float*>(sr);
 #pragma unroll
-          for (int i = 0; i < kTile; ++i)
-            if (i > col_hi || i < col_lo) s[i] = -INFINITY;
-        }
+            for (int a = 0; a < 4; ++a) {
+              if (MASK && hi_min < a * 32 + 31) {
 #pragma unroll
-        for (int a = 0; a < 4; ++a) {
-          float m = s[a * 32];
+                for (int i = a * 32; i < a * 32 + 32; ++i)
+                  if (i > col_hi) s[i] = -INFINITY;
+              }
+              if (MASK && lo_max > a * 32) {
 #pragma unroll
-          for (int i = 1; i + 1 < 32; i += 2) m = fmax3(m, s[a * 32 + i], s[a * 32 + i + 1]);
-          mxs[a] = fmaxf(m, s[a * 32 + 31]);
-        }
+                for (int i = a * 32; i < a * 32 + 32; ++i)
+                  if (i < col_lo) s[i] = -INFINITY;
+              }
+              float m = s[a * 32];
+#pragma unroll
+              for (int i = 1; i + 1 < 32; i += 2) m = fmax3(m, s[a * 32 + i], s[a * 32 + i + 1]);
+              mxs[a] = fmaxf(m, s[a * 32 + 31]);
+            }
+          }
+          float mx = fmaxf(fmaxf(mxs[0], mxs[1]), fmaxf(mxs[2], mxs[3]));
+          mx *= args.scale_log2;
+          float alpha = 1.f;
+          if (j == lo) {
+            m_used = mx;                               // -inf when this row sees nothing in its tile's first key tile
+          } else if (mx > m_used + kRescaleThreshold) {
+            alpha = ex2(m_used - mx);                  // 0 when nothing was accumulated yet
+            m_used = mx;
+          }
+          if (j > lo && __any_sync(0xffffffffu, alpha != 1.f)) {
+            // S(j) is complete, so every earlier P V product has finished; the next one waits for p_ready below:
+            // nobody else touches O now
+#pragma unroll
+            for (int c = 0; c < HV / 16; ++c) {
+              uint32_t r[16];
+              tmem_ld_32x32b_x16(o_tmem + c * 16, r);
+              tmem_ld_wait();
+#pragma unroll
+              for (int i = 0; i < 16; ++i) r[i] = __float_as_uint(__uint_as_float(r[i]) * alpha);
+              tmem_st_32x32b_x16(o_tmem + c * 16, r);
+            }
+          }
+          const float neg_m = (m_used == -INFINITY) ? 0.f : -m_used;
+          const uint64_t negm2 = pack2(neg_m, neg_m);
+          uint64_t rs2[4] = {0, 0, 0, 0};
+          // exp2 of the scaled, shifted scores two at a time; P goes back as bf16 pairs, 64 score columns (32 packed
+          // registers) per store, into the first 64 columns of this tile's S buffer
+#pragma unroll
+          for (int h = 0; h < 2; ++h) {
+            // pass 2: 64 scores at a time; the second half is read before the first half's P overwrites columns 0..31
+            if (MASK && (hi_max < h * 64 || lo_min > h * 64 + 63)) {
+              uint32_t zero[32];
+#pragma unroll
+              for (int i = 0; i < 32; ++i) zero[i] = 0u;
+              tmem_st_32x32b_x32(s_tmem + h * 32, zero);
+              continue;
+            }
+            uint32_t sr[64];
+            {
+              uint32_t (&ra)[32] = *reinterpret_cast<uint32_t(*)[32]>(&sr[0]);
+              uint32_t (&rb)[32] = *reinterpret_cast<uint32_t(*)[32]>(&sr[32]);
+              tmem_ld_32x32b_x32(s_tmem + h * 64, ra);
+              tmem_ld_32x32b_x32(s_tmem + h * 64 + 32, rb);
+              tmem_ld_wait();
+            }
+            float* s = reinterpret_cast<float*>(sr);
+#pragma unroll
+            for (int a = 0; a < 2; ++a) {
+              if (MASK && hi_min < h * 64 + a * 32 + 31) {
+#pragma unroll
+                for (int i = a * 32; i < a * 32 + 32; ++i)
+                  if (h * 64 + i > col_hi) s[i] = -INFINITY;
+              }
+              if (MASK && lo_max > h * 64 + a * 32) {
+#pragma unroll
+                for (int i = a * 32; i < a * 32 + 32; ++i)
+                  if (h * 64 + i < col_lo) s[i] = -INFINITY;
+              }
+            }
+            uint32_t pk[32];
+#pragma unroll
+            for (int i = 0; i < 32; ++i) {
+              float t0, t1;
+              unpack2(fma2(pack2(s[2 * i], s[2 * i + 1]), scale2, negm2), t0, t1);
+              const float e0 = ex2(t0), e1 = ex2(t1);
+              rs2[i & 3] = add2(rs2[i & 3], pack2(e0, e1));
+              pk[i] = pack_bf16x2(e0, e1);
+            }
+            tmem_st_32x32b_x32(s_tmem + h * 32, pk);
+          }
+          float r0, r1, r2, r3;
+          unpack2(add2(rs2[0], rs2[1]), r0, r1);
+          unpack2(add2(rs2[2], rs2[3]), r2, r3);
+          l_sum = l_sum * alpha + ((r0 + r1) + (r2 + r3));
+        };
+        if (lo_max > 0 || hi_min < kTile - 1) softmax_tile(std::true_type{});
+        else softmax_tile(std::false_type{});
+        tmem_st_wait();
+        tc_fence_before();
+        mbar_arrive(smem_u32(p_ready));
       }
-      float mx = fmaxf(fmaxf(mxs[0], mxs[1]), fmaxf(mxs[2], mxs[3]));
-      mx *= args.scale_log2;
-      float alpha = 1.f;
-      if (j == lo) {
-        m_used = mx;                               // -inf when this row sees nothing in its tile's first key tile
-      } else if (mx > m_used + kRescaleThreshold) {
-        alpha = ex2(m_used - mx);                  // 0 when nothing was accumulated yet
-        m_used = mx;
-      }
-      if (j > lo && __any_sync(0xffffffffu, alpha != 1.f)) {
-        // S(j) is complete, so every earlier P V product has finished; the next one waits for p_ready below:
-        // nobody else touches O now
-#pragma unroll
-        for (int c = 0; c < HV / 16; ++c) {
-          uint32_t r[16];
-          tmem_ld_32x32b_x16(o_tmem + c * 16, r);
-          tmem_ld_wait();
-#pragma unroll
-          for (int i = 0; i < 16; ++i) r[i] = __float_as_uint(__uint_as_float(r[i]) * alpha);
-          tmem_st_32x32b_x16(o_tmem + c * 16, r);
-        }
-      }
-      const float neg_m = (m_used == -INFINITY) ? 0.f : -m_used;
-      const uint64_t negm2 = pack2(neg_m, neg_m);
-      uint64_t rs2[4] = {0, 0, 0, 0};
-      // exp2 of the scaled, shifted scores two at a time; P goes back as bf16 pairs, 64 score columns (32 packed
-      // registers) per store, into the first 64 columns of this tile's S buffer
-#pragma unroll
-      for (int h = 0; h < 2; ++h) {
-        // pass 2: 64 scores at a time; the second half is read before the first half's P overwrites columns 0..31
-        uint32_t sr[64];
-        {
-          uint32_t (&ra)[32] = *reinterpret_cast<uint32_t(*)[32]>(&sr[0]);
-          uint32_t (&rb)[32] = *reinterpret_cast<uint32_t(*)[32]>(&sr[32]);
-          tmem_ld_32x32b_x32(s_tmem + h * 64, ra);
-          tmem_ld_32x32b_x32(s_tmem + h * 64 + 32, rb);
-          tmem_ld_wait();
-        }
-        float* s = reinterpret_cast<float*>(sr);
-        if (masked) {
-#pragma unroll
-          for (int i = 0; i < 64; ++i)
-            if (h * 64 + i > col_hi || h * 64 + i < col_lo) s[i] = -INFINITY;
-        }
-        uint32_t pk[32];
-#pragma unroll
-        for (int i = 0; i < 32; ++i) {
-          float t0, t1;
-          unpack2(fma2(pack2(s[2 * i], s[2 * i + 1]), scale2, negm2), t0, t1);
-          const float e0 = ex2(t0), e1 = ex2(t1);
-          rs2[i & 3] = add2(rs2[i & 3], pack2(e0, e1));
-          pk[i] = pack_bf16x2(e0, e1);
-        }
-        tmem_st_32x32b_x32(s_tmem + h * 32, pk);
-      }
-      float r0, r1, r2, r3;
-      unpack2(add2(rs2[0], rs2[1]), r0, r1);
-      unpack2(add2(rs2[2], rs2[3]), r2, r3);
-      l_sum = l_sum * alpha + ((r0 + r1) + (r2 + r3));
-      tmem_st_wait();
-      tc_fence_before();
-      mbar_arrive(smem_u32(p_ready));
-    }
-    if (n_kv > 0) {
-      if (ok) ok = mbar_wait(smem_u32(pv_done), (n_kv - 1 - lo) & 1, abort_flag, args.status, kStatusWaitTimeoutEpilogue);
+      if (ok) ok = mbar_wait(smem_u32(pv_done), (it - 1) & 1, abort_flag, args.status, kStatusWaitTimeoutEpilogue);
       // one decision for the whole warpgroup (a thread that gave up above still arrives here)
       ok = named_bar_and(2, 128, ok);
-      if (ok) {
-        tc_fence_after();
-        // the sink joins the denominator on the scale of the sum; an enormous sink overflows to a zero weight of the keys
-        const float den = args.sink ? l_sum + ex2(args.sink[head] * 1.4426950408889634f - m_used) : l_sum;
-        const float inv_l = 1.f / den;
-        // every MMA that read Q has completed: its shared memory now stages the warp's 32 rows
-        uint8_t* stage = sQ;
-        uint8_t* orow = stage + row * 128;
+      if (!ok) break;
+      tc_fence_after();
+      // the sink joins the denominator on the scale of the sum; an enormous sink overflows to a zero weight of the keys
+      const float den = args.sink ? l_sum + ex2(args.sink[t.head] * 1.4426950408889634f - m_used) : l_sum;
+      const float inv_l = 1.f / den;
+      // 32 columns at a time through 2 KB of shared memory per warp, so that a store covers 64 bytes of eight rows each
+      uint8_t* stage = sOut + ew * 2048;
+      __nv_bfloat16* obase = args.out + (static_cast<size_t>(t.q0 + ew * 32) * args.num_q_heads + t.head) * args.DV;
 #pragma unroll
-        for (int c = 0; c < HV / 32; ++c) {
-          uint32_t r[32];
-          tmem_ld_32x32b_x32(o_tmem + c * 32, r);
-          tmem_ld_wait();
+      for (int c = 0; c < HV / 32; ++c) {
+        uint32_t r[32];
+        tmem_ld_32x32b_x32(o_tmem + c * 32, r);
+        tmem_ld_wait();
 #pragma unroll
-          for (int q = 0; q < 4; ++q) {
-            const int chunk = c * 4 + q;
-            uint4 v = make_uint4(
-                pack_bf16x2(__uint_as_float(r[q * 8 + 0]) * inv_l, __uint_as_float(r[q * 8 + 1]) * inv_l),
-                pack_bf16x2(__uint_as_float(r[q * 8 + 2]) * inv_l, __uint_as_float(r[q * 8 + 3]) * inv_l),
-                pack_bf16x2(__uint_as_float(r[q * 8 + 4]) * inv_l, __uint_as_float(r[q * 8 + 5]) * inv_l),
-                pack_bf16x2(__uint_as_float(r[q * 8 + 6]) * inv_l, __uint_as_float(r[q * 8 + 7]) * inv_l));
-            *reinterpret_cast<uint4*>(orow + (chunk >> 3) * kSubBytes + (((chunk & 7) ^ (row & 7)) << 4)) = v;
-          }
+        for (int q = 0; q < 4; ++q)
+          *reinterpret_cast<uint4*>(stage + lane * 64 + ((q ^ ((lane >> 1) & 3)) << 4)) = make_uint4(
+              pack_bf16x2(__uint_as_float(r[q * 8 + 0]) * inv_l, __uint_as_float(r[q * 8 + 1]) * inv_l),
+              pack_bf16x2(__uint_as_float(r[q * 8 + 2]) * inv_l, __uint_as_float(r[q * 8 + 3]) * inv_l),
+              pack_bf16x2(__uint_as_float(r[q * 8 + 4]) * inv_l, __uint_as_float(r[q * 8 + 5]) * inv_l),
+              pack_bf16x2(__uint_as_float(r[q * 8 + 6]) * inv_l, __uint_as_float(r[q * 8 + 7]) * inv_l));
+        __syncwarp();
+        const int col = c * 32 + (lane & 3) * 8;
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const int rr = i * 8 + (lane >> 2);
+          if (ew * 32 + rr < t.rows && col < args.DV)
+            *reinterpret_cast<uint4*>(obase + static_cast<size_t>(rr) * args.num_q_heads * args.DV + col) =
+                *reinterpret_cast<const uint4*>(stage + rr * 64 + (((lane & 3) ^ ((rr >> 1) & 3)) << 4));
         }
         __syncwarp();
-        const int my_rows = rows - ew * 32;             // valid rows of this warp (may be negative)
-        const int vecs = args.DV / 8;
-        __nv_bfloat16* obase = args.out + (static_cast<size_t>(q0 + ew * 32) * args.num_q_heads + head) * args.DV;
-        for (int i = lane; i < 32 * (HV / 8); i += 32) {
-          const int rr = i / (HV / 8), c = i % (HV / 8);
-          if (rr < my_rows && c < vecs) {
-            const int srow = ew * 32 + rr;
-            const uint4 v = *reinterpret_cast<const uint4*>(stage + srow * 128 + (c >> 3) * kSubBytes + (((c & 7) ^ (srow & 7)) << 4));
-            *reinterpret_cast<uint4*>(obase + static_cast<size_t>(rr) * args.num_q_heads * args.DV + c * 8) = v;
-          }
-        }
       }
+      // O is read: the next tile's first P V product, which overwrites it, waits for this warpgroup's next p_ready
+      tc_fence_before();
     }
   }
   tc_fence_before();
@@ -389,10 +435,9 @@ int make_q_map(CUtensorMap* out, const void* q, uint64_t T, uint64_t Hq, uint64_
 }
 
 template <int HQ, int HV>
-int launch(const CUtensorMap& tQ, const CUtensorMap& tK, const CUtensorMap& tV, const Args& a, int grid, cudaStream_t stream) {
+int launch(const CUtensorMap& tQ, const CUtensorMap& tK, const CUtensorMap& tV, const Args& a, int max_ctas, cudaStream_t stream) {
   constexpr int QBYTES = HQ / 64 * kSubBytes, VBYTES = HV / 64 * kSubBytes;
-  constexpr int STAGE = QBYTES > VBYTES ? QBYTES : VBYTES;
-  constexpr int SMEM = STAGE + QBYTES + VBYTES + 8 * 8 + 16 + 1024;
+  constexpr int SMEM = 2 * QBYTES + VBYTES + 4 * 2048 + 9 * 8 + 16 + 1024;
   static_assert(2 * SMEM <= 232448, "shared memory budget exceeded");
   auto kern = paged_prefill_tc_kernel<HQ, HV>;
   static bool attr_set = false;
@@ -403,6 +448,7 @@ int launch(const CUtensorMap& tQ, const CUtensorMap& tK, const CUtensorMap& tV, 
     }
     attr_set = true;
   }
+  const int grid = a.n_items < max_ctas ? a.n_items : max_ctas;
   kern<<<grid, kThreads, SMEM, stream>>>(tQ, tK, tV, a);
   if (cudaGetLastError() != cudaSuccess) { mfb_host::set_error("paged_prefill_tc: launch failed"); return 11; }
   return 0;
@@ -420,10 +466,12 @@ int mfb_paged_prefill_tc_supported(int Hq, int Hkv, int D, int DV, int block_siz
   return (block_size == 16 || block_size == 32 || block_size == 64 || block_size == 128) ? 1 : 0;
 }
 
-// q [T, Hq, D], caches [num_blocks, block_size, Hkv, D | DV], out [T, Hq, DV], all bf16. work [n_work, 2] int32: (sequence,
-// first row of a 128-row tile inside its portion), for all rows of every sequence that this launch computes.
-int mfb_paged_prefill_tc(const void* q, const void* key_cache, const void* value_cache, const int* work, int n_work,
-                         const int* cu_q, const int* block_tables, const int* context_lens, const float* sink, void* out, int T,
+// q [T, Hq, D], caches [num_blocks, block_size, Hkv, D | DV], out [T, Hq, DV], all bf16. work [n_work, 4] int32: (sequence,
+// first row of q, 1..128 rows, position of the first row) per query tile, heaviest first; the rows' keys are in the cache.
+// persistent: two CTAs per SM walk over all tiles (for tiles of a few key tiles); else a CTA per query tile and head, which
+// balances tiles of very different lengths better.
+int mfb_paged_prefill_tc(const void* q, const void* key_cache, const void* value_cache, const int* work, int n_work, int persistent,
+                         const int* block_tables, const float* sink, void* out, int T,
                          int Hq, int Hkv, int D, int DV, int num_blocks, int block_size, int max_blocks, int chunk, float scale,
                          int* status, cudaStream_t stream) {
   if (!mfb_paged_prefill_tc_supported(Hq, Hkv, D, DV, block_size) || num_blocks < 1 || T < 1) {
@@ -439,17 +487,17 @@ int mfb_paged_prefill_tc(const void* q, const void* key_cache, const void* value
   if ((rc = mfb_host::make_tmap_2d(&tV, value_cache, 2, BF, rows, (uint64_t)Hkv * DV, (uint64_t)Hkv * DV, block_size, 64))) return 40 + rc;
   if ((rc = ppt::make_q_map(&tQ, q, T, Hq, D))) return 20 + rc;
   ppt::Args a;
-  a.work = work; a.cu_q = cu_q; a.block_tables = block_tables; a.context_lens = context_lens; a.sink = sink;
+  a.work = reinterpret_cast<const int4*>(work); a.n_items = n_work * Hq; a.block_tables = block_tables; a.sink = sink;
   a.out = reinterpret_cast<__nv_bfloat16*>(out);
   a.num_q_heads = Hq; a.group = Hq / Hkv; a.D = D; a.DV = DV; a.block_size = block_size; a.max_blocks = max_blocks;
   a.chunk = chunk; a.scale_log2 = scale * 1.4426950408889634f; a.status = status;
-  const int grid = n_work * Hq;
+  const int max_ctas = persistent ? 2 * 148 : a.n_items;
   if (D > 64) {
-    if (DV > 64) return ppt::launch<128, 128>(tQ, tK, tV, a, grid, stream);
-    return ppt::launch<128, 64>(tQ, tK, tV, a, grid, stream);
+    if (DV > 64) return ppt::launch<128, 128>(tQ, tK, tV, a, max_ctas, stream);
+    return ppt::launch<128, 64>(tQ, tK, tV, a, max_ctas, stream);
   }
-  if (DV > 64) return ppt::launch<64, 128>(tQ, tK, tV, a, grid, stream);
-  return ppt::launch<64, 64>(tQ, tK, tV, a, grid, stream);
+  if (DV > 64) return ppt::launch<64, 128>(tQ, tK, tV, a, max_ctas, stream);
+  return ppt::launch<64, 64>(tQ, tK, tV, a, max_ctas, stream);
 }
 
 }  // extern "C"

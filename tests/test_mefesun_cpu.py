@@ -94,7 +94,8 @@ def test_prefill_work_covers_every_row_once():
     q, ctx = [1, 300, 0, 129, 2], [5, 300, 9, 700, 130]
     for chunk in (0, 64, 200):
         items = prefill_work(q, ctx, chunk)
-        assert sorted(items) == [(1, 0), (1, 128), (1, 256), (3, 0), (3, 128), (4, 0)]
+        assert sorted(items) == [(1, 1, 128, 0), (1, 129, 128, 128), (1, 257, 44, 256), (3, 301, 128, 571), (3, 429, 1, 699),
+                                 (4, 430, 2, 128)]
     assert prefill_work(q, ctx, 0)[0][0] == 3                                # the rows that see the most keys come first
 
 

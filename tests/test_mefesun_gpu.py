@@ -4,6 +4,7 @@ import pytest
 import torch
 
 from mindformers_b200.inference.paged_attention import KVCacheContext
+from mindformers_b200.inference import ragged_attention as ragged
 from mindformers_b200.inference.ragged_attention import ragged_attention
 from mindformers_b200.ops import _lib, stream
 from mindformers_b200.serving import SamplingParams, ServingEngine
@@ -191,10 +192,11 @@ ATTENTION = [(4, 2, 64, 64), (8, 2, 128, 128), (6, 2, 40, 24), (5, 5, 128, 64), 
 
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("H,G,D,DV", ATTENTION)
-@pytest.mark.parametrize("bs", [16, 64])
-def test_ragged_attention(dtype, H, G, D, DV, bs):
+@pytest.mark.parametrize("bs,persistent", [(16, 0), (64, 0), (64, 1000)])
+def test_ragged_attention(dtype, H, G, D, DV, bs, persistent, monkeypatch):
     """Mixed batch: whole prompts, later portions, single rows, a sequence left out; chunks smaller than a key tile, at its
     size and above, that do not divide it, and no chunks at all."""
+    monkeypatch.setattr(ragged, "_PERSISTENT_UP_TO", persistent)
     lens, news = [1, 300, 129, 517, 64, 130, 40], [1, 300, 2, 260, 1, 1, 0]
     for chunk in (0, 21, 64, 128, 200):
         ctx, table, qs, sink, scale, want = attention_case(dtype, H, G, D, DV, bs, chunk, lens, news, seed=chunk)
