@@ -108,6 +108,7 @@ def reverse_name_glm(name: str) -> str:
     return out
 
 
+# Designs whose configuration lists their layers name tensors ``l<i>.*`` beside ``embed`` and ``final.norm``.
 # Mefesun checkpoints: ``l<i>.mix.*`` / ``l<i>.mlp.*`` / ``l<i>.norm1`` ..., a tensor's bias is its name with ``.b``.
 # The last component decides between weight and bias, so the names are mapped one by one (``None``: no suffix).
 _MEFESUN = {
@@ -120,18 +121,18 @@ _MEFESUN = {
 }
 _MEFESUN_TOP = {"embed": "embedding.word_embeddings.weight", "final.norm": "decoder.final_layernorm.weight",
                 "final.norm.b": "decoder.final_layernorm.bias"}
-_MEFESUN_LAYER = re.compile(r"^l(\d+)\.(.+)$")
+_LIST_LAYER = re.compile(r"^l(\d+)\.(.+)$")
 
 
-def is_mefesun_name(name: str) -> bool:
-    return bool(_MEFESUN_LAYER.match(name)) or name in _MEFESUN_TOP
+def is_layer_list_name(name: str) -> bool:
+    return bool(_LIST_LAYER.match(name)) or name in _MEFESUN_TOP
 
 
 def convert_name_mefesun(name: str) -> str:
     """Mefesun key → per-projection framework key."""
     if name in _MEFESUN_TOP:
         return _MEFESUN_TOP[name]
-    m = _MEFESUN_LAYER.match(name)
+    m = _LIST_LAYER.match(name)
     if not m:
         return name
     part, kind = (m[2][:-2], "bias") if m[2].endswith(".b") else (m[2], None)
@@ -170,7 +171,109 @@ def framework_to_mefesun(sd: Dict[str, torch.Tensor], config) -> Dict[str, torch
     return out
 
 
-FAMILIES = ("mefesun", "llama", "qwen2", "qwen2_5", "qwen2_moe", "qwen3", "qwen3_moe", "deepseek_v2", "deepseek_v3",
+# Kukupel checkpoints: tensors that map one to one (suffix of the framework name), then the fused ones.
+_KUKUPEL = {
+    "norm1": "input_layernorm.weight", "norm2": "pre_mlp_layernorm.weight", "mlp.router": "mlp.router.weight",
+    "hc1.in": "mixer_connection.read", "hc1.out": "mixer_connection.write", "hc1.mix": "mixer_connection.mix",
+    "hc2.in": "mlp_connection.read", "hc2.out": "mlp_connection.write", "hc2.mix": "mlp_connection.mix",
+}
+_KUKUPEL_CORE = {"A_log": "a_log", "dt_bias": "dt_bias", "norm": "norm", "a2": "decay_up", "g2": "gate_up"}
+_KUKUPEL_IN = {"q": "q", "k": "k", "v": "v", "gate": "g", "decay_down": "a1", "gate_down": "g1", "beta": "b", "decay": "a"}
+
+
+def _kukupel_layout(config, i: int):
+    """Of layer ``i``: ``(prefix of the delta rule's tensors, its module, [(name, rows)] of the input projection, [(name,
+    columns)] of the output projection)``."""
+    c = config.for_layer(i)
+    H, G, D, DV = c.delta_heads, c.delta_kv_heads, c.delta_key_dim, c.delta_value_dim
+    channel = c.delta_decay == "channel"
+    rows = [("q", G * D), ("k", G * D), ("v", H * DV)]
+    rows += [] if c.delta_gate_rank else [("gate", H * DV)]
+    rows += [("decay_down", c.delta_decay_rank)] if channel else []
+    rows += [("gate_down", c.delta_gate_rank)] if c.delta_gate_rank else []
+    rows += [("beta", H)] + ([] if channel else [("decay", H)])
+    rows = [(_KUKUPEL_IN[n], r) for n, r in rows]
+    if c.mixer != "parallel":
+        return "mix.", "self_attention.core", [("mix." + n, r) for n, r in rows], [("mix.o", H * DV)]
+    a = (c.num_attention_heads, c.num_query_groups, c.kv_channels, c.v_channels or c.kv_channels)
+    left = [("q", a[0] * a[2]), ("k", a[1] * a[2]), ("v", a[1] * a[3])]
+    return ("mix.right.", "self_attention.right", [("mix.left." + n, r) for n, r in left] + [("mix.right." + n, r) for n, r in rows],
+            [("mix.left.o", a[0] * a[3]), ("mix.right.o", H * DV)])
+
+
+def kukupel_to_framework(sd: Dict[str, torch.Tensor], config) -> Dict[str, torch.Tensor]:
+    """Kukupel tensors of any number of whole layers → fused framework parameters (full, unsharded)."""
+    out: Dict[str, torch.Tensor] = {}
+    layers: Dict[int, Dict[str, torch.Tensor]] = {}
+    for name, t in sd.items():
+        m = _LIST_LAYER.match(name)
+        if m:
+            layers.setdefault(int(m[1]), {})[m[2]] = t
+        else:
+            out[_MEFESUN_TOP.get(name, name)] = t
+    for i, own in layers.items():
+        prefix, module, rows, cols = _kukupel_layout(config, i)
+        p, left = f"decoder.layers.{i}.", set(own)
+
+        def take(name):
+            left.discard(name)
+            if name not in own:
+                raise KeyError(f"l{i}.{name} is missing")
+            return own[name]
+        if any(n.startswith("mix.") for n in own):
+            out[p + "self_attention.linear_in.weight"] = torch.cat([take(n) for n, _ in rows], dim=0)
+            out[p + "self_attention.linear_proj.weight"] = torch.cat([take(n) for n, _ in cols], dim=1)
+            out[p + module + ".conv"] = torch.cat([take(f"{prefix}{n}.conv") for n in "qkv"], dim=0).t().contiguous()
+            for n, to in _KUKUPEL_CORE.items():
+                if prefix + n in own:
+                    out[f"{p}{module}.{to}"] = take(prefix + n)
+        n_experts = sum(1 for n in own if re.match(r"^mlp\.e\d+\.gate$", n))
+        if n_experts:
+            w1 = [torch.cat((take(f"mlp.e{e}.gate"), take(f"mlp.e{e}.up")), dim=0).t() for e in range(n_experts)]
+            out[p + "mlp.experts.weight1"] = torch.stack(w1).contiguous()                                      # [E, H, 2F]
+            out[p + "mlp.experts.weight2"] = torch.stack([take(f"mlp.e{e}.down").t() for e in range(n_experts)]).contiguous()
+        for n in sorted(left):
+            if n not in _KUKUPEL:
+                raise KeyError(f"l{i}.{n}: no counterpart in the model")
+            out[p + _KUKUPEL[n]] = own[n]
+    return out
+
+
+def framework_to_kukupel(sd: Dict[str, torch.Tensor], config) -> Dict[str, torch.Tensor]:
+    """Fused framework names → Kukupel tensors."""
+    top = {v: k for k, v in _MEFESUN_TOP.items()}
+    plain, core = {v: k for k, v in _KUKUPEL.items()}, {v: k for k, v in _KUKUPEL_CORE.items()}
+    out: Dict[str, torch.Tensor] = {}
+    for name, t in sd.items():
+        m = re.match(r"^decoder\.layers\.(\d+)\.(.+)$", name)
+        if not m:
+            out[top.get(name, name)] = t
+            continue
+        l, rest = f"l{m[1]}.", m[2]
+        prefix, module, rows, cols = _kukupel_layout(config, int(m[1]))
+        if rest in plain:
+            out[l + plain[rest]] = t
+        elif rest == "self_attention.linear_in.weight":
+            out.update((l + n, piece.contiguous()) for (n, _), piece in zip(rows, torch.split(t, [r for _, r in rows], dim=0)))
+        elif rest == "self_attention.linear_proj.weight":
+            out.update((l + n, piece.contiguous()) for (n, _), piece in zip(cols, torch.split(t, [c for _, c in cols], dim=1)))
+        elif rest == module + ".conv":
+            sizes = [r for n, r in rows if n in (prefix + "q", prefix + "k", prefix + "v")]
+            out.update((f"{l}{prefix}{n}.conv", piece.t().contiguous()) for n, piece in zip("qkv", torch.split(t, sizes, dim=1)))
+        elif rest.startswith(module + "."):
+            out[l + prefix + core[rest[len(module) + 1:]]] = t
+        elif rest == "mlp.experts.weight1":
+            for e in range(t.shape[0]):
+                g, u = t[e].t().chunk(2, dim=0)
+                out[f"{l}mlp.e{e}.gate"], out[f"{l}mlp.e{e}.up"] = g.contiguous(), u.contiguous()
+        elif rest == "mlp.experts.weight2":
+            out.update((f"{l}mlp.e{e}.down", t[e].t().contiguous()) for e in range(t.shape[0]))
+        else:
+            raise KeyError(f"{name}: no counterpart in the checkpoint format")
+    return out
+
+
+FAMILIES = ("mefesun", "kukupel", "llama", "qwen2", "qwen2_5", "qwen2_moe", "qwen3", "qwen3_moe", "deepseek_v2", "deepseek_v3",
             "deepseekv3", "mixtral", "telechat", "glm")
 
 
@@ -412,8 +515,8 @@ def hf_to_framework(hf_sd: Dict[str, torch.Tensor], config, family: str = "llama
             continue
         if dtype is not None and t.is_floating_point():
             t = t.to(dtype)
-        plain[convert_name(name, family)] = t
-    out = fuse_state_dict(plain, config)
+        plain[name if family == "kukupel" else convert_name(name, family)] = t
+    out = kukupel_to_framework(plain, config) if family == "kukupel" else fuse_state_dict(plain, config)
     if keep_fp8 and any_fp8:
         out = requantize_linear_weights(out)
     return out
@@ -451,6 +554,9 @@ def framework_to_hf(sd: Dict[str, torch.Tensor], config, family: str = "llama", 
     if family == "mefesun":
         return {k: (t if dtype is None or not t.is_floating_point() else t.to(dtype)).contiguous()
                 for k, t in framework_to_mefesun(sd, config).items()}
+    if family == "kukupel":
+        return {k: (t if dtype is None or not t.is_floating_point() else t.to(dtype)).contiguous()
+                for k, t in framework_to_kukupel(sd, config).items()}
     for name, t in unfuse_state_dict(sd, config).items():
         if dtype is not None and t.is_floating_point():
             t = t.to(dtype)

@@ -65,6 +65,8 @@ def _speculative_generate(model, prompts, gcfg, max_len, pool_of, draft_len: int
     eos = set(gcfg.eos_ids())
     ctx, tables = model._set_kv_cache(B, max_len + draft_len + 1, getattr(model.config, "num_blocks", None))
     tables.init_cache_engine(B)
+    if ctx.has_state:
+        raise NotImplementedError("rejected drafts are taken back by forgetting cached tokens, which a recurrent state cannot do")
     seqs = [list(p) for p in prompts]
     limits = [max_len if gcfg.max_new_tokens is None else len(p) + gcfg.max_new_tokens for p in prompts]
     pools = [pool_of(i, max_ngram) for i in range(B)]
@@ -152,7 +154,10 @@ def prefix_cache_decoding(model, prompts, gcfg, max_len, **kw):
         for i in range(1, B):
             tables.engines[i].prepare_cache(shared)
             dst = tables.engines[i].blocks[: shared // bs]
+            ctx.copy_state([i], [0])
             for layer in range(len(ctx.key_cache)):
+                if ctx.key_cache[layer] is None:
+                    continue
                 ctx.key_cache[layer][dst] = ctx.key_cache[layer][src]
                 if ctx.value_cache[layer] is not None:
                     ctx.value_cache[layer][dst] = ctx.value_cache[layer][src]

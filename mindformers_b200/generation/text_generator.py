@@ -48,7 +48,8 @@ class GenerationMixin:
             if extra_layers:
                 raise NotImplementedError("draft layers share the cache shapes of the decoder")
             ctx = KVCacheContext(n_layers, num_blocks, block_size, 0, 0, dtype, device, layer_shapes=shapes,
-                                 kv_cache_dtype=getattr(cfg, "kv_cache_dtype", None))
+                                 kv_cache_dtype=getattr(cfg, "kv_cache_dtype", None),
+                                 state_shapes=self.model.decoder.state_shapes(), slots=batch_size)
         elif getattr(cfg, "multi_latent_attention", False):
             ctx = KVCacheContext(n_layers, num_blocks, block_size, 1, 0, dtype, device,
                                  mla_latent_dim=cfg.kv_lora_rank + cfg.qk_pos_emb_head_dim)
@@ -191,6 +192,7 @@ class GenerationMixin:
             bind()
             if state["graph"] is None:
                 # the first call runs eagerly twice on a side stream (lazy allocations, kernel attributes), then captures
+                kept = ctx.save_state()            # the warm-up runs advance recurrent states
                 side = torch.cuda.Stream(device=device)
                 side.wait_stream(torch.cuda.current_stream(device))
                 with torch.cuda.stream(side):
@@ -198,6 +200,7 @@ class GenerationMixin:
                     forward()
                 torch.cuda.current_stream(device).wait_stream(side)
                 torch.cuda.synchronize(device)
+                ctx.restore_state(kept)
                 graph = torch.cuda.CUDAGraph()
                 with torch.cuda.graph(graph):
                     state["out"] = forward()
@@ -272,6 +275,7 @@ class GenerationMixin:
                 entry["captures"] += 1
                 return _Eager
             keep = {k: getattr(st, k).clone() for k in ("tok", "pos", "lens", "slots", "count", "finished", "hist")}
+            kept = ctx.save_state()
             side = torch.cuda.Stream(device=device)
             side.wait_stream(torch.cuda.current_stream(device))
             with torch.cuda.stream(side):
@@ -284,6 +288,7 @@ class GenerationMixin:
                 step()
             for k, v in keep.items():
                 getattr(st, k).copy_(v)
+            ctx.restore_state(kept)
             entry["captures"] += 1
             return graph
 
@@ -580,6 +585,7 @@ class GenerationMixin:
         """Beam ``i`` continues from beam ``src[i]``: copy the cache contents block by block."""
         if src == list(range(len(src))):
             return
+        ctx.copy_state(list(range(len(src))), src)
         dst_blocks, src_blocks = [], []
         for i, j in enumerate(src):
             if i == j:
@@ -589,9 +595,11 @@ class GenerationMixin:
             src_blocks += tables.engines[j].blocks[:n]
         if not dst_blocks:
             return
-        d = torch.tensor(dst_blocks, device=ctx.key_cache[0].device)
-        s = torch.tensor(src_blocks, device=ctx.key_cache[0].device)
         for layer in range(ctx.num_layers):
+            if ctx.key_cache[layer] is None:
+                continue
+            d = torch.tensor(dst_blocks, device=ctx.key_cache[layer].device)
+            s = torch.tensor(src_blocks, device=ctx.key_cache[layer].device)
             ctx.key_cache[layer][d] = ctx.key_cache[layer][s].clone()
             if ctx.value_cache[layer] is not None:
                 ctx.value_cache[layer][d] = ctx.value_cache[layer][s].clone()

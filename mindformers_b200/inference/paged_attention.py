@@ -28,9 +28,16 @@ class KVCacheContext:
 
     def __init__(self, num_layers: int, num_blocks: int, block_size: int, kv_heads: int, head_dim: int,
                  dtype=torch.bfloat16, device="cuda", mla_latent_dim: Optional[int] = None,
-                 kv_cache_dtype: Optional[str] = None, layer_shapes: Optional[list] = None):
+                 kv_cache_dtype: Optional[str] = None, layer_shapes: Optional[list] = None,
+                 state_shapes: Optional[list] = None, slots: int = 0):
         """``layer_shapes``: ``(kv heads, key size, value size)`` of every layer's cache, for models whose layers differ or
-        whose keys and values differ in size; such a cache also carries the step metadata of ragged attention.
+        whose keys and values differ in size (None: the layer caches no keys); such a cache also carries the step metadata
+        of ragged attention.
+
+        ``state_shapes``: per layer None or ``(heads, key size, value size, conv channels, conv taps)``: layers with a
+        recurrent state have, for each of ``slots`` sequences (row b of a batch uses slot b), ``S [heads, key, value]`` in
+        fp32 and a ring of the last conv inputs (``recurrent[layer]``). A sequence that starts at position 0 reads neither,
+        so a slot changes hands without being cleared.
 
         ``kv_cache_dtype="int8"`` stores keys and values as int8 codes with one fp32 scale per token and KV head
         (``key_scale`` / ``value_scale`` ``[num_blocks, block_size, kv_heads]``): half the bytes per cached token, read
@@ -47,8 +54,10 @@ class KVCacheContext:
             if self.int8 or mla_latent_dim or len(layer_shapes) != num_layers:
                 raise ValueError("per-layer cache shapes: one per layer, and no int8 or latent cache")
             rows = (num_blocks, block_size)
-            self.key_cache = [torch.zeros(rows + (h, k), dtype=dtype, device=device) for h, k, _ in layer_shapes]
-            self.value_cache = [torch.zeros(rows + (h, v), dtype=dtype, device=device) for h, _, v in layer_shapes]
+            self.key_cache = [None if s is None else torch.zeros(rows + (s[0], s[1]), dtype=dtype, device=device)
+                              for s in layer_shapes]
+            self.value_cache = [None if s is None else torch.zeros(rows + (s[0], s[2]), dtype=dtype, device=device)
+                                for s in layer_shapes]
         elif self.int8:
             shape = (num_blocks, block_size, kv_heads, head_dim)
             self.key_cache = [torch.zeros(shape, dtype=torch.int8, device=device) for _ in range(num_layers)]
@@ -63,6 +72,9 @@ class KVCacheContext:
             shape = (num_blocks, block_size, kv_heads, head_dim)
             self.key_cache = [torch.zeros(shape, dtype=dtype, device=device) for _ in range(num_layers)]
             self.value_cache = [torch.zeros(shape, dtype=dtype, device=device) for _ in range(num_layers)]
+        self.recurrent = [None if s is None else (torch.zeros((slots,) + tuple(s[:3]), dtype=torch.float32, device=device),
+                                                  torch.zeros((slots, s[4], s[3]), dtype=dtype, device=device))
+                          for s in state_shapes or [None] * num_layers]
         self.is_prefill = True
         self.block_tables = None      # int32 [B, max_blocks]
         self.slot_mapping = None      # int32 [T]
@@ -75,6 +87,26 @@ class KVCacheContext:
         self.prefill_work = {}        # work lists of the ragged prefill kernel, made when a layer needs them
         self.q_lens_host = self.context_lens_host = ()
         self.n_long_rows = self.n_single_rows = 0     # sequences with several new rows / with one
+
+    @property
+    def has_state(self) -> bool:
+        """Whether some layer has a recurrent state: such a step cannot be run twice, nor tokens taken back."""
+        return any(r is not None for r in self.recurrent)
+
+    def save_state(self) -> list:
+        """Copy of the recurrent states (for runs that warm up or capture a step and must leave no trace)."""
+        return [None if r is None else tuple(t.clone() for t in r) for r in self.recurrent]
+
+    def restore_state(self, saved: list):
+        for r, old in zip(self.recurrent, saved):
+            for t, o in zip(r or (), old or ()):
+                t.copy_(o)
+
+    def copy_state(self, dst: List[int], src: List[int]):
+        """Slot ``dst[i]`` continues from what slot ``src[i]`` holds now."""
+        for r in self.recurrent:
+            for t in r or ():
+                t[dst] = t[src].clone()
 
     def set_step(self, *, is_prefill, block_tables, slot_mapping, context_lens, q_seq_lens, device):
         self.is_prefill = is_prefill

@@ -52,14 +52,14 @@ def _work_on_device(cache, chunk: int):
     return work
 
 
-def _reference(q, cache, layer, scale, chunk, sink):
+def _reference(q, cache, layer, scale, chunk, sink, softcap, out, out_scale):
     """Plain PyTorch body for CPU tensors."""
     from .paged_attention import _gather
     B = cache.context_lens.shape[0]
     cu = cache.cu_q if cache.is_prefill else list(range(B + 1))
     lens = cache.context_lens.tolist()
     Hq = q.shape[1]
-    out = q.new_zeros(q.shape[0], Hq, cache.value_cache[layer].shape[-1])
+    out.zero_()
     for b in range(B):
         a, e = cu[b], cu[b + 1]
         if e == a or lens[b] <= 0:
@@ -68,6 +68,8 @@ def _reference(q, cache, layer, scale, chunk, sink):
         v = _gather(cache.value_cache[layer], cache.block_tables[b], lens[b], cache.block_size).float()
         reps = Hq // k.shape[1]
         s = torch.einsum("qhd,khd->hqk", q[a:e].float(), k.repeat_interleave(reps, 1)) * scale
+        if softcap > 0:
+            s = softcap * torch.tanh(s / softcap)
         qp = torch.arange(lens[b] - (e - a), lens[b]).unsqueeze(1)
         kp = torch.arange(lens[b]).unsqueeze(0)
         hide = kp > qp
@@ -77,40 +79,48 @@ def _reference(q, cache, layer, scale, chunk, sink):
         if sink is not None:
             s = torch.cat((s, sink.float()[:, None, None].expand(Hq, e - a, 1)), dim=-1)
         p = torch.softmax(s, dim=-1)[..., :lens[b]]
-        out[a:e] = torch.einsum("hqk,khd->qhd", p, v.repeat_interleave(reps, 1)).to(q.dtype)
+        o = torch.einsum("hqk,khd->qhd", p, v.repeat_interleave(reps, 1)) * out_scale
+        out[a:e] = o.reshape(e - a, -1).to(q.dtype)
     return out
 
 
 def ragged_attention(q: torch.Tensor, cache, layer: int, scale: float, chunk: int = 0,
-                     sink: Optional[torch.Tensor] = None) -> torch.Tensor:
+                     sink: Optional[torch.Tensor] = None, softcap: float = 0.0, out: Optional[torch.Tensor] = None,
+                     out_scale: float = 1.0) -> torch.Tensor:
     """q ``[T, heads, dim]`` of the step's new tokens, whose keys and values are in the cache already → ``[T, heads *
     v_dim]``. ``chunk`` > 0: a position sees its own chunk of that many positions (counted from 0) only. ``sink [heads]``
-    fp32: adds ``exp(sink)`` to the softmax denominator."""
+    fp32: adds ``exp(sink)`` to the softmax denominator. ``softcap`` > 0: scores become ``softcap * tanh(score / softcap)``.
+    ``out``: a matrix (any row pitch that keeps rows on 16 bytes) to write to; the result is multiplied by ``out_scale``."""
     kc, vc = cache.key_cache[layer], cache.value_cache[layer]
     T, Hq, D = q.shape
     Hkv, DV = vc.shape[2], vc.shape[3]
+    softcap = float(softcap or 0.0)
+    if out is None:
+        out = torch.empty((T, Hq * DV), dtype=q.dtype, device=q.device)
+    elif out.dtype != q.dtype or out.shape != (T, Hq * DV) or out.stride(1) != 1:
+        raise TypeError("ragged_attention: out must be a [T, heads * v_dim] matrix of q's dtype with unit column stride")
     if not q.is_cuda:
-        return _reference(q, cache, layer, scale, chunk, sink).view(T, Hq * DV)
+        return _reference(q, cache, layer, scale, chunk, sink, softcap, out, out_scale)
     lib = _lib.get_lib()
     B, max_blocks = cache.block_tables.shape
     ragged = cache.is_prefill
-    out = torch.empty((T, Hq, DV), dtype=q.dtype, device=q.device)
     bs, nb = cache.block_size, kc.shape[0]
     cu = cache.cu_q_dev.data_ptr() if ragged else 0
     tables, lens, snk = cache.block_tables.data_ptr(), cache.context_lens.data_ptr(), _lib.ptr(sink)
-    if q.dtype != torch.bfloat16 or not lib.mfb_paged_prefill_tc_supported(Hq, Hkv, D, DV, bs):
+    if q.dtype != torch.bfloat16 or out.stride(0) % 8 or out.data_ptr() % 16 \
+            or not lib.mfb_paged_prefill_tc_supported(Hq, Hkv, D, DV, bs):
         rc = lib.mfb_paged_attention_any(q.data_ptr(), kc.data_ptr(), vc.data_ptr(), tables, lens, cu, snk, out.data_ptr(), T, B,
-                                         Hq, Hkv, D, DV, bs, max_blocks, int(chunk), float(scale),
-                                         int(q.dtype == torch.float32), _lib.stream_ptr())
+                                         Hq, Hkv, D, DV, bs, max_blocks, int(chunk), float(scale), softcap, out.stride(0),
+                                         float(out_scale), int(q.dtype == torch.float32), _lib.stream_ptr())
         _lib.check(rc, "mfb_paged_attention_any")
         _lib.count_launch()
-        return out.view(T, Hq * DV)
+        return out
     status = _lib.status_word(q.device).data_ptr()
     if ragged and cache.n_long_rows:
         work, persistent = _work_on_device(cache, int(chunk))
         rc = lib.mfb_paged_prefill_tc(q.data_ptr(), kc.data_ptr(), vc.data_ptr(), work.data_ptr(), work.shape[0], int(persistent),
                                       tables, snk, out.data_ptr(), T, Hq, Hkv, D, DV, nb, bs, max_blocks, int(chunk),
-                                      float(scale), status, _lib.stream_ptr())
+                                      float(scale), softcap, out.stride(0), float(out_scale), status, _lib.stream_ptr())
         _lib.check(rc, "mfb_paged_prefill_tc")
         _lib.count_launch()
     if not ragged or cache.n_single_rows:
@@ -129,7 +139,8 @@ def ragged_attention(q: torch.Tensor, cache, layer: int, scale: float, chunk: in
             setattr(cache, name, scratch)
         rc = lib.mfb_paged_decode_attention_tc_ex(
             q.data_ptr(), kc.data_ptr(), vc.data_ptr(), tables, lens, cu, snk, out.data_ptr(), scratch.data_ptr(), splits, T, B,
-            Hq, Hkv, D, DV, nb, bs, max_blocks, int(chunk), float(scale), status, _lib.stream_ptr())
+            Hq, Hkv, D, DV, nb, bs, max_blocks, int(chunk), float(scale), softcap, out.stride(0), float(out_scale), status,
+            _lib.stream_ptr())
         _lib.check(rc, "mfb_paged_decode_attention_tc_ex")
         _lib.count_launch(2)
-    return out.view(T, Hq * DV)
+    return out

@@ -133,6 +133,17 @@ class WeightsLoader:
         return layers, other
 
 
+def tensor_shapes(path: str):
+    """``shape_of(name)`` of a directory (or file) of safetensors: a tensor's shape, None for one it does not hold."""
+    try:
+        loader = WeightsLoader(path)
+    except FileNotFoundError:
+        return lambda name: None
+    shapes = {n: loader.shape(n) for n in loader.keys()}
+    loader.close()
+    return shapes.get
+
+
 def _assign(model, params, buffers, fw: Dict[str, torch.Tensor], used: set, fp8_modules: list, keep_fp8: bool):
     from ..checkpoint.io import _owner_path
     with torch.no_grad():
@@ -165,7 +176,7 @@ def load_weights(model: torch.nn.Module, path: str, family: str = "llama", stric
     layers, other = loader.layer_groups()
     params = dict(model.named_parameters())
     buffers = dict(model.named_buffers())
-    is_hf = any(k.startswith(("model.", "lm_head", "transformer.")) or name_maps.is_mefesun_name(k) for k in loader.keys())
+    is_hf = any(k.startswith(("model.", "lm_head", "transformer.")) or name_maps.is_layer_list_name(k) for k in loader.keys())
     used: set = set()
     fp8_modules: list = []
     peak = 0

@@ -222,7 +222,106 @@ class MefesunConfig(PretrainedConfig):
         return dict(d, **own)
 
 
+class KukupelConfig(PretrainedConfig):
+    """Kukupel: a decoder on several residual streams (hyper-connections) whose layers mix tokens with a gated delta rule,
+    alone (``delta``: one decay per head, silu gate) or beside position-free, soft-capped grouped-query attention
+    (``parallel``: decays per key channel and a sigmoid gate, both low-rank), pre-norm, with mixtures of clamped gated experts
+    whose routing weight multiplies their input, and a tied head.
+
+    Keys of ``config.json``: ``vocab``, ``width``, ``streams``, ``norm.eps`` and ``layers``, a list of ``{"type": "delta",
+    "mixer": {"heads", "kv_heads", "dim", "vdim", "conv"}}`` or ``{"type": "parallel", "mixer": {"left": {"heads",
+    "kv_heads", "dim", "vdim", "scale", "softcap"}, "right": {as delta}, "left_scale", "right_scale"}}``, each with ``"mlp":
+    {"kind": "moe", "router": {"experts", "top"}, "expert": {"ff", "limit"}} | null``. The ranks of the low-rank factors are
+    those of the checkpoint's tensors (``complete_from_checkpoint``), or ``right.decay_rank`` / ``right.gate_rank``, or the
+    value size. Framework keys (``seq_length``, ``block_size``, token ids) may stand beside them."""
+
+    model_type = "kukupel"
+
+    @classmethod
+    def default_values(cls):
+        return dict(architecture="Kukupel", vocab=32000, width=1024, streams=4, norm=dict(eps=1e-6),
+                    layers=KukupelConfig.layer_list("parallel delta delta delta", heads=8, kv_heads=2, dim=128, delta_heads=8,
+                                                    delta_kv_heads=4, delta_dim=128, experts=16, top=2, ff=768),
+                    pad_token_id=0, bos_token_id=None, eos_token_id=None, block_size=64)
+
+    @staticmethod
+    def layer_list(types: str, heads: int, kv_heads: int, dim: int, delta_heads: int, delta_kv_heads: int, delta_dim: int,
+                   experts: int, top: int, ff: int, vdim=None, delta_vdim=None, conv: int = 4, softcap: float = 30.0,
+                   scale=None, scales=(0.5, 0.5), limit: float = 7.0, rank=None):
+        """The ``layers`` list of a model whose layers of one type (``types``, by name) are alike."""
+        delta = dict(heads=delta_heads, kv_heads=delta_kv_heads, dim=delta_dim, vdim=delta_vdim or delta_dim, conv=conv)
+        left = dict(heads=heads, kv_heads=kv_heads, dim=dim, vdim=vdim or dim, scale=scale or dim ** -0.5, softcap=softcap)
+        right = dict(delta, **({} if rank is None else dict(decay_rank=rank, gate_rank=rank)))
+        mixer = {"delta": delta, "parallel": dict(left=left, right=right, left_scale=scales[0], right_scale=scales[1])}
+        mlp = dict(kind="moe", router=dict(experts=experts, top=top), expert=dict(ff=ff, limit=limit))
+        return [dict(type=t, mixer=copy.deepcopy(mixer[t]), mlp=copy.deepcopy(mlp)) for t in types.split()]
+
+    def complete_from_checkpoint(self, shape_of):
+        """Sizes that only the checkpoint gives; ``shape_of(name)`` is a tensor's shape, None for one it does not hold."""
+        for i, layer in enumerate(self.layers):
+            if layer.get("type") == "parallel":
+                for key, name in (("decay_rank", "a1"), ("gate_rank", "g1")):
+                    shape = shape_of(f"l{i}.mix.right.{name}")
+                    if shape is not None:
+                        layer["mixer"]["right"][key] = int(shape[0])
+
+    @staticmethod
+    def _delta_fields(mix: dict, channel: bool) -> dict:
+        rank = int(mix["vdim"])
+        return dict(delta_heads=int(mix["heads"]), delta_kv_heads=int(mix["kv_heads"]), delta_key_dim=int(mix["dim"]),
+                    delta_value_dim=int(mix["vdim"]), delta_conv_taps=int(mix["conv"]),
+                    delta_decay="channel" if channel else "head", delta_gate="sigmoid" if channel else "silu",
+                    delta_decay_rank=int(mix.get("decay_rank") or rank) if channel else 0,
+                    delta_gate_rank=int(mix.get("gate_rank") or rank) if channel else 0)
+
+    @classmethod
+    def _layer_fields(cls, i: int, layer: dict) -> dict:
+        kind, mix, mlp = layer.get("type"), layer["mixer"], layer.get("mlp")
+        if kind == "delta":
+            out = dict(mixer="delta", **cls._delta_fields(mix, False))
+        elif kind == "parallel":
+            a = mix["left"]
+            out = dict(mixer="parallel", parallel_scales=(float(mix["left_scale"]), float(mix["right_scale"])),
+                       num_attention_heads=int(a["heads"]), num_query_groups=int(a["kv_heads"]), kv_channels=int(a["dim"]),
+                       v_channels=int(a["vdim"]), softmax_scale=float(a["scale"]),
+                       attention_softcap=float(a["softcap"]) if a.get("softcap") else None,
+                       **cls._delta_fields(mix["right"], True))
+        else:
+            raise ValueError(f"layer {i}: unknown mixer type {kind!r}")
+        if mlp and mlp.get("kind", "moe") != "moe":
+            raise ValueError(f"layer {i}: unknown feed-forward kind {mlp['kind']!r}")
+        out.update(ffn_hidden_size=0)
+        if mlp:
+            r, e = mlp["router"], mlp["expert"]
+            if not 1 <= int(r["top"]) <= int(r["experts"]):
+                raise ValueError(f"layer {i}: {r['top']} of {r['experts']} experts")
+            out.update(num_moe_experts=int(r["experts"]), moe_router_topk=int(r["top"]), moe_ffn_hidden_size=int(e["ff"]),
+                       moe_activation_limit=float(e["limit"]))
+        return out
+
+    def to_transformer_dict(self) -> dict:
+        d = {k: v for k, v in self.to_dict().items()
+             if k not in ("architecture", "layers", "norm", "vocab", "width", "streams", "mlp", "mixer")}
+        fields = [self._layer_fields(i, layer) for i, layer in enumerate(self.layers)]
+        d.setdefault("seq_length", 32768)                      # no positions enter the model: a bound for buffers alone
+        d.setdefault("max_position_embeddings", d["seq_length"])
+        moe = [1 if f.get("num_moe_experts") else 0 for f in fields]
+        own = dict(num_attention_heads=1, num_query_groups=1, kv_channels=1, ffn_hidden_size=0)       # layers without attention
+        for f in fields:                                       # the stack's own view of what its layers override
+            own.update({k: v for k, v in f.items() if k in own and k != "ffn_hidden_size"})
+        if any(moe):
+            own.update({k: v for k, v in fields[moe.index(1)].items() if k.startswith(("num_moe", "moe_"))}, moe_layer_freq=moe)
+        own.update(vocab_size=int(self.vocab), hidden_size=int(self.width), num_layers=len(fields), layer_overrides=fields,
+                   residual_streams=int(self.streams), layernorm_epsilon=float(self.norm["eps"]), normalization="RMSNorm",
+                   fp32_residual_connection=True, ragged_attention=True, rotary_dim=0, position_embedding_type="none",
+                   moe_activation="clamped_glu", moe_activation_alpha=1.702, moe_apply_probs_on_input=True, norm_topk_prob=False,
+                   moe_router_score_function="sigmoid", moe_router_topk_scaling_factor=1.0, tie_word_embeddings=True)
+        d = {k: v for k, v in d.items() if ALIASES.get(k, (k,))[0] not in own}
+        return dict(d, **own)
+
+
 for _legacy in (True, False):
+    MindFormerRegister.register_cls(KukupelConfig, MindFormerModuleType.CONFIG, alias="KukupelConfig", legacy=_legacy)
     MindFormerRegister.register_cls(MefesunConfig, MindFormerModuleType.CONFIG, alias="MefesunConfig", legacy=_legacy)
 
 LlamaForCausalLM = _model("LlamaForCausalLM", LlamaConfig, "llama")
@@ -238,6 +337,10 @@ MefesunForCausalLM = _model("MefesunForCausalLM", MefesunConfig, "mefesun")
 MefesunForCausalLM.kernel_sources = ("host_util", "elementwise", "gemm_tcgen05", "gemm_tcgen05_2cta", "gemm_bf16_decode",
                                      "output_norm", "qkv_rope_cache", "paged_prefill_tc", "paged_decode_tc",
                                      "paged_attention", "paged_attention_any", "decode_loop")
+KukupelForCausalLM = _model("KukupelForCausalLM", KukupelConfig, "kukupel")
+KukupelForCausalLM.kernel_sources = ("host_util", "elementwise", "gemm_tcgen05", "gemm_tcgen05_2cta", "gemm_bf16_decode",
+                                     "residual_streams", "delta_rule", "qkv_rope_cache", "paged_prefill_tc", "paged_decode_tc",
+                                     "paged_attention", "paged_attention_any", "router", "moe_ep", "moe_any", "decode_loop")
 ChatGLM2ForConditionalGeneration = _model("ChatGLM2ForConditionalGeneration", ChatGLM4Config, "glm")
 
 def _backbone(name, causal_cls):
@@ -307,5 +410,6 @@ MODEL_TYPE_TO_CLASSES = {
     "deepseek_v2": (DeepseekV2Config, DeepseekV2ForCausalLM), "deepseek2": (DeepseekV2Config, DeepseekV2ForCausalLM),
     "qwen2_moe": (Qwen2MoeConfig, Qwen2MoeForCausalLM),
     "telechat": (TelechatConfig, TelechatForCausalLM), "glm": (ChatGLM4Config, ChatGLM2ForConditionalGeneration),
-    "mefesun": (MefesunConfig, MefesunForCausalLM), "chatglm": (ChatGLM4Config, ChatGLM2ForConditionalGeneration),
+    "mefesun": (MefesunConfig, MefesunForCausalLM), "kukupel": (KukupelConfig, KukupelForCausalLM),
+    "chatglm": (ChatGLM4Config, ChatGLM2ForConditionalGeneration),
 }

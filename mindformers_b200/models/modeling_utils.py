@@ -100,6 +100,9 @@ class PreTrainedModel(nn.Module, GenerationMixin, InferModelMixin):
             raise FileNotFoundError(f"{path} does not exist (hub download is not available offline)")
         if config is None:
             config = cls.config_class.from_pretrained(path)
+        if load_weights and hasattr(config, "complete_from_checkpoint"):
+            from ..inference.weights_utils import tensor_shapes
+            config.complete_from_checkpoint(tensor_shapes(path))
         model = cls(config, **kwargs)
         if load_weights:
             try:

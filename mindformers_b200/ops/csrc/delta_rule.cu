@@ -1,0 +1,710 @@
+// Gated delta rule over ragged batches with a recurrent state per sequence slot (sm_100a). Per head, from token to token:
+//
+//   S <- g * S              S [D, DV] fp32; g: one decay per head, or one per head and key channel (rows of S)
+//   u  = beta * (v - S^T k)
+//   S <- S + k u^T
+//   o  = S^T q
+//
+// q, k and v are projections that passed a short causal convolution over time and silu; q and k are unit vectors per head
+// (q also times D^-1/2) and G of them serve H heads. o is normalised over DV, weighted, and gated (silu or sigmoid).
+// Everything from the convolution's result to o is fp32.
+//
+// State of slot b: S [H, D, DV] and the last `taps` inputs of the convolution, a ring in which position p has place
+// p % taps. Slot b belongs to row b of the batch. Nothing has to be cleared when a slot changes hands: a portion that starts
+// at position 0 reads neither S nor the ring, and no position below 0 is ever read.
+//
+// A batch is ragged: sequence b brings the rows cu_q[b] .. cu_q[b + 1] - 1, which end at position context_lens[b] - 1.
+// Portions run as prepare (convolution, unit vectors, decays; one warp per row and head) -> scan (the recurrence) ->
+// gate_out. A decode step (one row per slot) is one kernel, delta_decode.
+//
+// The scan runs token by token in fp32 on the FMA pipes, since the state and all that enters it are 32-bit by design. Columns of
+// S are independent: a CTA takes a range of the columns of one head of one sequence, L lanes share a column, and a thread
+// keeps R rows of C columns in registers for the whole portion, as pairs for the packed fp32 instructions. With
+// a = (g S)^T k and b = (g S)^T q taken in one pass, o = b + u (k . q) needs no second pass over S.
+#include "common.cuh"
+
+namespace mfb {
+namespace dlt {
+
+__device__ __forceinline__ float ld(const float* p) { return *p; }
+__device__ __forceinline__ float ld(const __nv_bfloat16* p) { return __bfloat162float(*p); }
+__device__ __forceinline__ void st(float* p, float v) { *p = v; }
+__device__ __forceinline__ void st(__nv_bfloat16* p, float v) { *p = __float2bfloat16_rn(v); }
+template <int VEC> __device__ __forceinline__ void ldv(const float* p, float (&v)[VEC]) {
+  if constexpr (VEC == 4) {
+    const float4 a = *reinterpret_cast<const float4*>(p);
+    v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
+  } else {
+    v[0] = *p;
+  }
+}
+template <int VEC> __device__ __forceinline__ void ldv(const __nv_bfloat16* p, float (&v)[VEC]) {
+  if constexpr (VEC == 4) {
+    const uint2 u = *reinterpret_cast<const uint2*>(p);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.x));
+    const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.y));
+    v[0] = a.x; v[1] = a.y; v[2] = b.x; v[3] = b.y;
+  } else {
+    v[0] = ld(p);
+  }
+}
+template <int VEC> __device__ __forceinline__ void stv(float* p, const float (&v)[VEC]) {
+  if constexpr (VEC == 4) *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+  else *p = v[0];
+}
+template <int VEC> __device__ __forceinline__ void stv(__nv_bfloat16* p, const float (&v)[VEC]) {
+  if constexpr (VEC == 4) *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]));
+  else st(p, v[0]);
+}
+
+__device__ __forceinline__ float sigmoidf(float x) { return 1.f / (1.f + expf(-x)); }
+__device__ __forceinline__ float siluf(float x) { return x / (1.f + expf(-x)); }
+__device__ __forceinline__ float softplusf(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
+__device__ __forceinline__ float decayf(float a_log, float x) { return expf(-expf(a_log) * softplusf(x)); }
+
+struct Args {
+  const void* x;            // [T, >= 2 G D + H DV] (pitch ld): inputs of the convolution, q | k | v
+  long long ld;
+  const void* b;            // [T, H] (pitch ld): raw beta
+  const void* a;            // raw decay: [T, H] or [T, H D] (pitch ld_a)
+  long long ld_a;
+  const void* gate;         // [T, H DV] (pitch ld_gate)
+  long long ld_gate;
+  const float* conv;        // [taps, 2 G D + H DV], the last row belongs to the current token
+  const float* a_log;       // [H]
+  const float* dt_bias;     // [H] or [H D]
+  const float* norm;        // [DV]
+  void* ring;               // [slots, taps, 2 G D + H DV] type T
+  float* state;             // [slots, H, D, DV]
+  const int* cu_q;          // [B + 1] (portions)
+  const int* context_lens;  // [B]
+  const int* slots;         // [B] cache slot of the row, negative: idle (decode)
+  float* qk;                // scratch [T, G, 2, D]: unit q (scaled), unit k
+  float* v;                 // scratch [T, H, DV]
+  float* beta;              // scratch [T, H, 2]: beta, q . k
+  float* g;                 // scratch [T, H] or [T, H, D]
+  float* o;                 // scratch [T, H, DV]
+  void* out;                // [T, H DV] type T (pitch ld_out)
+  long long ld_out;
+  int T, B, H, G, D, DV, taps, by_channel, gate_silu;
+  float eps, out_scale;
+};
+
+// sequence of row r (the last one that starts at or before it and is not empty there)
+__device__ __forceinline__ int sequence_of(const int* cu_q, int B, int r) {
+  int lo = 0, hi = B - 1;
+  while (lo < hi) {
+    const int mid = (lo + hi + 1) / 2;
+    if (cu_q[mid] <= r) lo = mid; else hi = mid - 1;
+  }
+  return lo;
+}
+
+constexpr int kRun = 8;                // consecutive rows of a warp in `prepare`
+
+// silu(convolution) of channels c .. c + VEC - 1 at row r; `local` rows of the portion lie before r, `pos` is its position
+template <typename T, int VEC>
+__device__ __forceinline__ void conv_silu(const Args& p, const T* ring, long long r, int local, int pos, int c, int C, float (&acc)[VEC]) {
+#pragma unroll
+  for (int i = 0; i < VEC; ++i) acc[i] = 0.f;
+  for (int d = p.taps - 1; d >= 0; --d) {
+    if (d > pos) continue;
+    float xv[VEC], wv[VEC];
+    if (d <= local) ldv<VEC>(reinterpret_cast<const T*>(p.x) + (r - d) * p.ld + c, xv);
+    else ldv<VEC>(ring + (long long)((pos - d) % p.taps) * C + c, xv);
+    ldv<VEC>(p.conv + (long long)(p.taps - 1 - d) * C + c, wv);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) acc[i] = fmaf(xv[i], wv[i], acc[i]);
+  }
+#pragma unroll
+  for (int i = 0; i < VEC; ++i) acc[i] = siluf(acc[i]);
+}
+
+// One warp per unit and run of rows. Units: G (q and k of a key head), H (v of a head), then H (decays of a head's channels)
+// or ceil(H / 32) (decays of 32 heads); the last kind also makes beta.
+template <typename T, int VEC, int NJ>
+__global__ void __launch_bounds__(128) prepare_kernel(const Args p, int units) {
+  const int unit = blockIdx.y * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (unit >= units) return;
+  const int r0 = blockIdx.x * kRun, r1 = min(r0 + kRun, p.T);
+  const int C = 2 * p.G * p.D + p.H * p.DV;
+  int b = sequence_of(p.cu_q, p.B, r0);
+  for (int r = r0; r < r1; ++r) {
+    while (r >= p.cu_q[b + 1]) ++b;
+    const int local = r - p.cu_q[b], pos = p.context_lens[b] - (p.cu_q[b + 1] - r);
+    const T* ring = reinterpret_cast<const T*>(p.ring) + (long long)b * p.taps * C;
+    if (unit < p.G) {
+      float q[NJ][VEC], k[NJ][VEC];
+      float qq = 0.f, kk = 0.f, qk = 0.f;
+#pragma unroll
+      for (int j = 0; j < NJ; ++j) {
+        const int d = (lane + 32 * j) * VEC;
+        if (d < p.D) {
+          conv_silu<T, VEC>(p, ring, r, local, pos, unit * p.D + d, C, q[j]);
+          conv_silu<T, VEC>(p, ring, r, local, pos, (p.G + unit) * p.D + d, C, k[j]);
+#pragma unroll
+          for (int i = 0; i < VEC; ++i) {
+            qq = fmaf(q[j][i], q[j][i], qq);
+            kk = fmaf(k[j][i], k[j][i], kk);
+            qk = fmaf(q[j][i], k[j][i], qk);
+          }
+        }
+      }
+      qq = warp_sum(qq); kk = warp_sum(kk); qk = warp_sum(qk);
+      const float rq = 1.f / sqrtf(qq + 1e-6f) / sqrtf((float)p.D), rk = 1.f / sqrtf(kk + 1e-6f);
+      float* dst = p.qk + ((long long)r * p.G + unit) * 2 * p.D;
+#pragma unroll
+      for (int j = 0; j < NJ; ++j) {
+        const int d = (lane + 32 * j) * VEC;
+        if (d < p.D) {
+#pragma unroll
+          for (int i = 0; i < VEC; ++i) { q[j][i] *= rq; k[j][i] *= rk; }
+          stv<VEC>(dst + d, q[j]);
+          stv<VEC>(dst + p.D + d, k[j]);
+        }
+      }
+      const int reps = p.H / p.G;
+      for (int i = lane; i < reps; i += 32) p.beta[((long long)r * p.H + unit * reps + i) * 2 + 1] = qk * rq * rk;
+    } else if (unit < p.G + p.H) {
+      const int h = unit - p.G;
+#pragma unroll
+      for (int j = 0; j < NJ; ++j) {
+        const int d = (lane + 32 * j) * VEC;
+        if (d < p.DV) {
+          float v[VEC];
+          conv_silu<T, VEC>(p, ring, r, local, pos, 2 * p.G * p.D + h * p.DV + d, C, v);
+          stv<VEC>(p.v + ((long long)r * p.H + h) * p.DV + d, v);
+        }
+      }
+    } else {
+      const int i0 = unit - p.G - p.H;
+      const T* a = reinterpret_cast<const T*>(p.a) + r * p.ld_a;
+      const T* bb = reinterpret_cast<const T*>(p.b) + r * p.ld;
+      if (p.by_channel) {
+        const float al = p.a_log[i0];
+        for (int d = lane; d < p.D; d += 32) {
+          const int c = i0 * p.D + d;
+          p.g[(long long)r * p.H * p.D + c] = decayf(al, ld(a + c) + p.dt_bias[c]);
+        }
+        if (lane == 0) p.beta[((long long)r * p.H + i0) * 2] = sigmoidf(ld(bb + i0));
+      } else {
+        const int h = i0 * 32 + lane;
+        if (h < p.H) {
+          p.g[(long long)r * p.H + h] = decayf(p.a_log[h], ld(a + h) + p.dt_bias[h]);
+          p.beta[((long long)r * p.H + h) * 2] = sigmoidf(ld(bb + h));
+        }
+      }
+    }
+  }
+}
+
+// ---- the recurrence -----------------------------------------------------------------------------------------------------
+__device__ __forceinline__ uint64_t pack2(float lo, float hi) {
+  uint64_t r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(lo), "f"(hi));
+  return r;
+}
+__device__ __forceinline__ void unpack2(uint64_t v, float& lo, float& hi) {
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(v));
+}
+__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
+  uint64_t d;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+  return d;
+}
+__device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
+  uint64_t d;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+  return d;
+}
+__device__ __forceinline__ void cp_async(void* dst, const void* src, int bytes16) {
+  const uint32_t d = smem_u32(dst);
+  if (bytes16) asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(d), "l"(src) : "memory");
+  else asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(d), "l"(src) : "memory");
+}
+__device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N> __device__ __forceinline__ void cp_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+
+constexpr int kScanThreads = 128;
+constexpr int kTile = 16;              // tokens staged at a time (two buffers)
+
+template <int R, int L, int C>
+struct ScanShape {
+  static constexpr int DP = R * L;                          // padded key size
+  static constexpr int kCols = kScanThreads / L * C;        // columns of a CTA
+};
+
+template <int R, int L, int C, bool CH>
+constexpr int scan_smem() {
+  using S = ScanShape<R, L, C>;
+  return 2 * kTile * (2 * S::DP + (CH ? S::DP : 4) + S::kCols + 4) * (int)sizeof(float);
+}
+
+// R rows of C columns per thread, L lanes per column; CH: decays per key channel. vec: D, DV and the scratch rows allow
+// 16-byte copies.
+template <typename T, int R, int L, int C, bool CH>
+__global__ void __launch_bounds__(kScanThreads) scan_kernel(const Args p, int vec) {
+  using S = ScanShape<R, L, C>;
+  constexpr int DP = S::DP, COLS = S::kCols, GW = CH ? DP : 4, GROUPS = kScanThreads / L;
+  const int b = blockIdx.z, h = blockIdx.y, col0 = blockIdx.x * COLS;
+  const int r0 = p.cu_q[b], n = p.cu_q[b + 1] - r0;
+  if (n <= 0) return;
+  const int end = p.context_lens[b], start = end - n;
+  const int D = p.D, DV = p.DV, H = p.H, kvh = h / (H / p.G);
+  if (blockIdx.x == 0 && h == 0) {
+    // the convolution's inputs of the last positions (`prepare`, which read the old ones, has finished)
+    const int ch = 2 * p.G * D + H * DV, keep = min(n, p.taps);
+    T* ring = reinterpret_cast<T*>(p.ring) + (long long)b * p.taps * ch;
+    for (int i = 0; i < keep; ++i) {
+      const int pos = end - keep + i;
+      const T* src = reinterpret_cast<const T*>(p.x) + (long long)(r0 + n - keep + i) * p.ld;
+      for (int c = threadIdx.x; c < ch; c += kScanThreads) ring[(long long)(pos % p.taps) * ch + c] = src[c];
+    }
+  }
+  extern __shared__ __align__(16) float sh[];
+  float* s_qk = sh;                                  // [2][kTile][q DP | k DP]
+  float* s_g = s_qk + 2 * kTile * 2 * DP;            // [2][kTile][GW]
+  float* s_v = s_g + 2 * kTile * GW;                 // [2][kTile][COLS]
+  float* s_b = s_v + 2 * kTile * COLS;               // [2][kTile][4]: beta, q . k
+  for (int i = threadIdx.x; i < 2 * kTile * (2 * DP + GW); i += kScanThreads) sh[i] = 0.f;      // the padding stays zero
+  __syncthreads();
+  const int ln = threadIdx.x % L, grp = threadIdx.x / L;
+
+  const int w = vec ? 4 : 1;                         // floats per copy
+  auto stage = [&](int tile) {
+    const int buf = tile & 1, t0 = tile * kTile, m = min(kTile, n - t0);
+    const int nq = 2 * D / w;
+    for (int i = threadIdx.x; i < m * nq; i += kScanThreads) {
+      const int t = i / nq, e = (i - t * nq) * w;
+      const int at = e < D ? e : DP + e - D;
+      cp_async(s_qk + (buf * kTile + t) * 2 * DP + at, p.qk + ((long long)(r0 + t0 + t) * p.G + kvh) * 2 * D + e, vec);
+    }
+    if (CH) {
+      const int ng = D / w;
+      for (int i = threadIdx.x; i < m * ng; i += kScanThreads) {
+        const int t = i / ng, e = (i - t * ng) * w;
+        cp_async(s_g + (buf * kTile + t) * GW + e, p.g + ((long long)(r0 + t0 + t) * H + h) * D + e, vec);
+      }
+    } else {
+      for (int t = threadIdx.x; t < m; t += kScanThreads)
+        cp_async(s_g + (buf * kTile + t) * GW, p.g + (long long)(r0 + t0 + t) * H + h, 0);
+    }
+    const int left = min(COLS, DV - col0), nv = left / w;
+    for (int i = threadIdx.x; i < m * nv; i += kScanThreads) {
+      const int t = i / nv, e = (i - t * nv) * w;
+      cp_async(s_v + (buf * kTile + t) * COLS + e, p.v + ((long long)(r0 + t0 + t) * H + h) * DV + col0 + e, vec);
+    }
+    for (int i = threadIdx.x; i < 2 * m; i += kScanThreads)
+      cp_async(s_b + (buf * kTile + (i >> 1)) * 4 + (i & 1), p.beta + ((long long)(r0 + t0 + (i >> 1)) * H + h) * 2 + (i & 1), 0);
+    cp_commit();
+  };
+
+  // rows of a thread: (i * L + ln) * 4 .. + 3 for i < R / 4, as pairs
+  uint64_t s[C][R / 2];
+  float* state = p.state + ((long long)b * H + h) * D * DV;
+#pragma unroll
+  for (int c = 0; c < C; ++c) {
+    const int col = col0 + grp + GROUPS * c;
+#pragma unroll
+    for (int i = 0; i < R / 2; ++i) {
+      float v[2];
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const int row = ((i >> 1) * L + ln) * 4 + (i & 1) * 2 + e;
+        v[e] = (start > 0 && row < D && col < DV) ? state[(long long)row * DV + col] : 0.f;
+      }
+      s[c][i] = pack2(v[0], v[1]);
+    }
+  }
+  const int tiles = (n + kTile - 1) / kTile;
+  stage(0);
+  for (int tile = 0; tile < tiles; ++tile) {
+    if (tile + 1 < tiles) {
+      stage(tile + 1);
+      cp_wait<1>();
+    } else {
+      cp_wait<0>();
+    }
+    __syncthreads();
+    const int buf = tile & 1, m = min(kTile, n - tile * kTile);
+    float* orow = p.o + ((long long)(r0 + tile * kTile) * H + h) * DV;
+    for (int t = 0; t < m; ++t) {
+      const float* qp = s_qk + (buf * kTile + t) * 2 * DP + ln * 4;
+      const float* kp = qp + DP;
+      const float* gp = s_g + (buf * kTile + t) * GW;
+      const float* vp = s_v + (buf * kTile + t) * COLS;
+      const float beta = s_b[(buf * kTile + t) * 4], qk = s_b[(buf * kTile + t) * 4 + 1];
+      uint64_t a2[C], b2[C];
+#pragma unroll
+      for (int c = 0; c < C; ++c) a2[c] = b2[c] = 0;
+      uint64_t k2[R / 2];
+#pragma unroll
+      for (int i = 0; i < R / 4; ++i) {
+        const ulonglong2 q4 = *reinterpret_cast<const ulonglong2*>(qp + i * L * 4);
+        const ulonglong2 k4 = *reinterpret_cast<const ulonglong2*>(kp + i * L * 4);
+        k2[2 * i] = k4.x; k2[2 * i + 1] = k4.y;
+        if (CH) {
+          const ulonglong2 g4 = *reinterpret_cast<const ulonglong2*>(gp + ln * 4 + i * L * 4);
+#pragma unroll
+          for (int c = 0; c < C; ++c) {
+            s[c][2 * i] = mul2(s[c][2 * i], g4.x);
+            s[c][2 * i + 1] = mul2(s[c][2 * i + 1], g4.y);
+          }
+        }
+#pragma unroll
+        for (int c = 0; c < C; ++c) {
+          a2[c] = fma2(s[c][2 * i], k4.x, a2[c]);
+          b2[c] = fma2(s[c][2 * i], q4.x, b2[c]);
+          a2[c] = fma2(s[c][2 * i + 1], k4.y, a2[c]);
+          b2[c] = fma2(s[c][2 * i + 1], q4.y, b2[c]);
+        }
+      }
+      float ga = 1.f;
+      if (!CH) ga = gp[0];
+      const uint64_t g2 = pack2(ga, ga);
+#pragma unroll
+      for (int c = 0; c < C; ++c) {
+        float x, y, a, bq;
+        unpack2(a2[c], x, y); a = x + y;
+        unpack2(b2[c], x, y); bq = x + y;
+#pragma unroll
+        for (int d = L / 2; d > 0; d >>= 1) {
+          a += __shfl_xor_sync(0xffffffffu, a, d);
+          bq += __shfl_xor_sync(0xffffffffu, bq, d);
+        }
+        const float u = beta * (vp[grp + GROUPS * c] - ga * a);
+        const int col = col0 + grp + GROUPS * c;
+        if (ln == c % L && col < DV) orow[(long long)t * H * DV + col] = fmaf(u, qk, ga * bq);
+        const uint64_t u2 = pack2(u, u);
+#pragma unroll
+        for (int i = 0; i < R / 2; ++i) s[c][i] = fma2(k2[i], u2, CH ? s[c][i] : mul2(s[c][i], g2));
+      }
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int c = 0; c < C; ++c) {
+    const int col = col0 + grp + GROUPS * c;
+#pragma unroll
+    for (int i = 0; i < R / 2; ++i) {
+      float v[2];
+      unpack2(s[c][i], v[0], v[1]);
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const int row = ((i >> 1) * L + ln) * 4 + (i & 1) * 2 + e;
+        if (row < D && col < DV) state[(long long)row * DV + col] = v[e];
+      }
+    }
+  }
+}
+
+// ---- norm and gate of the read-out: a warp per row and head -----------------------------------------------------------------
+template <typename T, int VEC, int NJ>
+__global__ void __launch_bounds__(128) gate_out_kernel(const Args p) {
+  const long long item = (long long)blockIdx.x * 4 + (threadIdx.x >> 5);
+  if (item >= (long long)p.T * p.H) return;
+  const int lane = threadIdx.x & 31;
+  const long long r = item / p.H;
+  const int h = (int)(item - r * p.H);
+  const float* o = p.o + item * p.DV;
+  const T* gate = reinterpret_cast<const T*>(p.gate) + r * p.ld_gate + h * p.DV;
+  T* out = reinterpret_cast<T*>(p.out) + r * p.ld_out + h * p.DV;
+  float v[NJ][VEC];
+  float ss = 0.f;
+#pragma unroll
+  for (int j = 0; j < NJ; ++j) {
+    const int d = (lane + 32 * j) * VEC;
+    if (d < p.DV) {
+      ldv<VEC>(o + d, v[j]);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) ss = fmaf(v[j][i], v[j][i], ss);
+    }
+  }
+  const float rstd = 1.f / sqrtf(warp_sum(ss) / p.DV + p.eps) * p.out_scale;
+#pragma unroll
+  for (int j = 0; j < NJ; ++j) {
+    const int d = (lane + 32 * j) * VEC;
+    if (d < p.DV) {
+      float w[VEC], z[VEC];
+      ldv<VEC>(p.norm + d, w);
+      ldv<VEC>(gate + d, z);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) v[j][i] = v[j][i] * rstd * w[i] * (p.gate_silu ? siluf(z[i]) : sigmoidf(z[i]));
+      stv<VEC>(out + d, v[j]);
+    }
+  }
+}
+
+// ---- decode: one row per slot, one CTA per head ---------------------------------------------------------------------------------
+// Threads form TY row groups of TX lanes; a lane holds four neighbouring columns of NR rows. D * DV <= 4 NT NR.
+template <typename T, int NT, int NR>
+__global__ void __launch_bounds__(NT) delta_decode_kernel(const Args p, int tx_log2) {
+  const int h = blockIdx.x, b = blockIdx.y;
+  const int D = p.D, DV = p.DV, H = p.H, reps = H / p.G, kvh = h / reps;
+  T* out = reinterpret_cast<T*>(p.out) + (long long)b * p.ld_out + h * DV;
+  if (p.slots[b] < 0) {                        // idle slot: the state stays, the row is defined
+    for (int i = threadIdx.x; i < DV; i += NT) st(out + i, 0.f);
+    return;
+  }
+  const int pos = p.context_lens[b] - 1;
+  const int TX = 1 << tx_log2, TY = NT >> tx_log2, tx = threadIdx.x & (TX - 1), ty = threadIdx.x >> tx_log2;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  float* state = p.state + ((long long)b * H + h) * D * DV;
+  const int col = tx * 4;
+  float4 s[NR];
+#pragma unroll
+  for (int i = 0; i < NR; ++i) {
+    const int row = ty + TY * i;
+    s[i] = (pos > 0 && row < D && col < DV) ? *reinterpret_cast<const float4*>(state + (long long)row * DV + col)
+                                            : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+  extern __shared__ __align__(16) float sh[];
+  float* s_u = sh;                             // [DV] (16-byte aligned: DV is a multiple of 4)
+  float* s_q = s_u + DV;                       // [D]
+  float* s_k = s_q + D;                        // [D]
+  float* s_v = s_k + D;                        // [DV], later o
+  float* s_g = s_v + DV;                       // [D]
+  float* s_red = s_g + D;                      // [NT / 32] + 2 x [TY][4 TX]
+  const int C = 2 * p.G * D + H * DV;
+  T* ring = reinterpret_cast<T*>(p.ring) + (long long)b * p.taps * C;
+  const T* x = reinterpret_cast<const T*>(p.x) + (long long)b * p.ld;
+  for (int i = threadIdx.x; i < 2 * D + DV; i += NT) {
+    const int c = i < D ? kvh * D + i : (i < 2 * D ? (p.G + kvh) * D + i - D : 2 * p.G * D + h * DV + i - 2 * D);
+    float v[1];
+    conv_silu<T, 1>(p, ring, b, 0, pos, c, C, v);
+    s_q[i] = v[0];
+    // the ring has a place for the current input that no token up to this one reads: heads that share q and k do not race
+    if (i >= 2 * D || h % reps == 0) ring[(long long)(pos % p.taps) * C + c] = x[c];
+  }
+  const T* a = reinterpret_cast<const T*>(p.a) + (long long)b * p.ld_a;
+  const float al = p.a_log[h];
+  if (p.by_channel) {
+    for (int i = threadIdx.x; i < D; i += NT) s_g[i] = decayf(al, ld(a + h * D + i) + p.dt_bias[h * D + i]);
+  } else {
+    const float g = decayf(al, ld(a + h) + p.dt_bias[h]);
+    for (int i = threadIdx.x; i < D; i += NT) s_g[i] = g;
+  }
+  const float beta = sigmoidf(ld(reinterpret_cast<const T*>(p.b) + (long long)b * p.ld + h));
+  __syncthreads();
+  float qq = 0.f, kk = 0.f, qk = 0.f;
+  for (int i = lane; i < D; i += 32) {
+    qq = fmaf(s_q[i], s_q[i], qq);
+    kk = fmaf(s_k[i], s_k[i], kk);
+    qk = fmaf(s_q[i], s_k[i], qk);
+  }
+  qq = warp_sum(qq); kk = warp_sum(kk); qk = warp_sum(qk);
+  const float rq = 1.f / sqrtf(qq + 1e-6f) / sqrtf((float)D), rk = 1.f / sqrtf(kk + 1e-6f);
+  float av[4] = {0.f, 0.f, 0.f, 0.f}, bv[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+  for (int i = 0; i < NR; ++i) {
+    const int row = ty + TY * i;
+    if (row < D) {
+      const float g = s_g[row], k = s_k[row] * rk, q = s_q[row] * rq;
+      s[i].x *= g; s[i].y *= g; s[i].z *= g; s[i].w *= g;
+      av[0] = fmaf(s[i].x, k, av[0]); av[1] = fmaf(s[i].y, k, av[1]); av[2] = fmaf(s[i].z, k, av[2]); av[3] = fmaf(s[i].w, k, av[3]);
+      bv[0] = fmaf(s[i].x, q, bv[0]); bv[1] = fmaf(s[i].y, q, bv[1]); bv[2] = fmaf(s[i].z, q, bv[2]); bv[3] = fmaf(s[i].w, q, bv[3]);
+    }
+  }
+  float* red_a = s_red + NT / 32;
+  float* red_b = red_a + NT * 4;
+#pragma unroll
+  for (int i = 0; i < 4; ++i) { red_a[ty * TX * 4 + col + i] = av[i]; red_b[ty * TX * 4 + col + i] = bv[i]; }
+  __syncthreads();
+  float ss = 0.f;
+  for (int c = threadIdx.x; c < DV; c += NT) {
+    float sa = 0.f, sb = 0.f;
+    for (int y = 0; y < TY; ++y) { sa += red_a[y * TX * 4 + c]; sb += red_b[y * TX * 4 + c]; }
+    const float u = beta * (s_v[c] - sa);
+    const float o = fmaf(u, qk * rq * rk, sb);
+    s_u[c] = u;
+    s_v[c] = o;
+    ss = fmaf(o, o, ss);
+  }
+  ss = warp_sum(ss);
+  if (lane == 0) s_red[warp] = ss;
+  __syncthreads();
+  if (col < DV) {
+    const float4 u = *reinterpret_cast<const float4*>(s_u + col);
+#pragma unroll
+    for (int i = 0; i < NR; ++i) {
+      const int row = ty + TY * i;
+      if (row < D) {
+        const float k = s_k[row] * rk;
+        *reinterpret_cast<float4*>(state + (long long)row * DV + col) =
+            make_float4(fmaf(k, u.x, s[i].x), fmaf(k, u.y, s[i].y), fmaf(k, u.z, s[i].z), fmaf(k, u.w, s[i].w));
+      }
+    }
+  }
+  float tot = 0.f;
+#pragma unroll
+  for (int i = 0; i < NT / 32; ++i) tot += s_red[i];
+  const float rstd = 1.f / sqrtf(tot / DV + p.eps) * p.out_scale;
+  const T* gate = reinterpret_cast<const T*>(p.gate) + (long long)b * p.ld_gate + h * DV;
+  for (int c = threadIdx.x; c < DV; c += NT) {
+    const float z = ld(gate + c);
+    st(out + c, s_v[c] * rstd * p.norm[c] * (p.gate_silu ? siluf(z) : sigmoidf(z)));
+  }
+}
+
+// ---- launchers --------------------------------------------------------------------------------------------------------------------
+bool al(const void* p, int bytes) { return (reinterpret_cast<uintptr_t>(p) & (bytes - 1)) == 0; }
+
+int fail(const char* what) {
+  if (cudaGetLastError() != cudaSuccess) { mfb_host::set_error("delta_rule: launch of %s failed", what); return 2; }
+  return 0;
+}
+
+template <typename T>
+int prepare(const Args& p, cudaStream_t stream) {
+  const int units = p.G + p.H + (p.by_channel ? p.H : (p.H + 31) / 32);
+  dim3 grid((p.T + kRun - 1) / kRun, (units + 3) / 4);
+  const int es = sizeof(T), C = 2 * p.G * p.D + p.H * p.DV;
+  const bool vec = p.D % 4 == 0 && p.DV % 4 == 0 && p.ld % 4 == 0 && C % 4 == 0 && al(p.x, 4 * es) && al(p.ring, 4 * es) &&
+                   al(p.conv, 16) && al(p.qk, 16) && al(p.v, 16);
+  const int m = p.D > p.DV ? p.D : p.DV;
+  if (vec) {
+    if (m <= 128) prepare_kernel<T, 4, 1><<<grid, 128, 0, stream>>>(p, units);
+    else prepare_kernel<T, 4, 4><<<grid, 128, 0, stream>>>(p, units);
+  } else {
+    if (m <= 128) prepare_kernel<T, 1, 4><<<grid, 128, 0, stream>>>(p, units);
+    else prepare_kernel<T, 1, 16><<<grid, 128, 0, stream>>>(p, units);
+  }
+  return fail("prepare");
+}
+
+template <typename T, int R, int L, int C, bool CH>
+int scan_one(const Args& p, int vec, cudaStream_t stream) {
+  auto kern = scan_kernel<T, R, L, C, CH>;
+  constexpr int smem = scan_smem<R, L, C, CH>();
+  static bool set = false;
+  if (!set) {
+    if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) {
+      mfb_host::set_error("delta_rule: cannot raise the shared memory limit");
+      return 10;
+    }
+    set = true;
+  }
+  constexpr int cols = ScanShape<R, L, C>::kCols;
+  dim3 grid((p.DV + cols - 1) / cols, p.H, p.B);
+  kern<<<grid, kScanThreads, smem, stream>>>(p, vec);
+  return fail("scan");
+}
+
+template <typename T, bool CH>
+int scan(const Args& p, cudaStream_t stream) {
+  const int vec = p.D % 4 == 0 && p.DV % 4 == 0 && al(p.qk, 16) && al(p.v, 16) && al(p.g, 16) ? 1 : 0;
+  if (p.D <= 32) return scan_one<T, 8, 4, 2, CH>(p, vec, stream);
+  if (p.D <= 64) return scan_one<T, 16, 4, 2, CH>(p, vec, stream);
+  if (p.D <= 128) return scan_one<T, 32, 4, 2, CH>(p, vec, stream);
+  if (p.D <= 256) return scan_one<T, 32, 8, 2, CH>(p, vec, stream);
+  return scan_one<T, 32, 16, 2, CH>(p, vec, stream);
+}
+
+template <typename T>
+int gate_out(const Args& p, cudaStream_t stream) {
+  const long long items = (long long)p.T * p.H;
+  const unsigned grid = (unsigned)((items + 3) / 4);
+  const int es = sizeof(T);
+  const bool vec = p.DV % 4 == 0 && p.ld_gate % 4 == 0 && p.ld_out % 4 == 0 && al(p.o, 16) && al(p.norm, 16) &&
+                   al(p.gate, 4 * es) && al(p.out, 4 * es);
+  if (vec) {
+    if (p.DV <= 128) gate_out_kernel<T, 4, 1><<<grid, 128, 0, stream>>>(p);
+    else gate_out_kernel<T, 4, 4><<<grid, 128, 0, stream>>>(p);
+  } else {
+    if (p.DV <= 128) gate_out_kernel<T, 1, 4><<<grid, 128, 0, stream>>>(p);
+    else gate_out_kernel<T, 1, 16><<<grid, 128, 0, stream>>>(p);
+  }
+  return fail("gate_out");
+}
+
+int tx_log2_of(int DV) {
+  int l = 0;
+  while ((4 << l) < DV) ++l;
+  return l;
+}
+
+template <typename T, int NT, int NR>
+int decode_one(const Args& p, cudaStream_t stream) {
+  const int l = tx_log2_of(p.DV);
+  const size_t smem = (size_t)(3 * p.D + 2 * p.DV + NT / 32 + 2 * NT * 4) * sizeof(float) + 16;
+  delta_decode_kernel<T, NT, NR><<<dim3(p.H, p.B), NT, smem, stream>>>(p, l);
+  return fail("decode");
+}
+
+// rows per thread with nt threads
+int decode_rows(int D, int DV, int nt) {
+  const int ty = nt >> tx_log2_of(DV);
+  return ty < 1 ? 1 << 20 : (D + ty - 1) / ty;
+}
+
+template <typename T>
+int decode(const Args& p, cudaStream_t stream) {
+  const int n256 = decode_rows(p.D, p.DV, 256);
+  if (n256 <= 4) return decode_one<T, 256, 4>(p, stream);
+  if (n256 <= 8) return decode_one<T, 256, 8>(p, stream);
+  if (n256 <= 16) return decode_one<T, 256, 16>(p, stream);
+  return decode_one<T, 512, 16>(p, stream);
+}
+
+int check(const Args& p) {
+  if (p.T < 0 || p.B < 1 || p.H < 1 || p.G < 1 || p.H % p.G || p.D < 1 || p.DV < 1 || p.D > 512 || p.DV > 512 || p.taps < 1 ||
+      p.H > 65535 || p.B > 65535) {
+    mfb_host::set_error("delta_rule: T=%d B=%d H=%d G=%d D=%d DV=%d taps=%d", p.T, p.B, p.H, p.G, p.D, p.DV, p.taps);
+    return 1;
+  }
+  return 0;
+}
+
+}  // namespace dlt
+}  // namespace mfb
+
+extern "C" {
+using namespace mfb;
+
+// 1 when a decode step runs in one kernel (else it runs as portions of one row)
+int mfb_delta_decode_supported(int D, int DV) {
+  return DV % 4 == 0 && D <= 512 && DV <= 512 && dlt::decode_rows(D, DV, 512) <= 16 ? 1 : 0;
+}
+
+// floats of scratch for T rows
+long long mfb_delta_scratch_floats(int T, int H, int G, int D, int DV, int by_channel) {
+  auto up = [](long long n) { return (n + 3) / 4 * 4; };
+  return up((long long)T * G * 2 * D) + 2 * up((long long)T * H * DV) + up((long long)T * H * 2) + up((long long)T * H * (by_channel ? D : 1));
+}
+
+// The whole mixer core (see the file header). f32: the activations (x, b, a, gate, ring, out) are fp32, else bf16. cu_q null: a
+// decode step of B rows, idle where slots < 0. scratch: mfb_delta_scratch_floats (portions only, 16-byte aligned).
+int mfb_delta_rule(const void* x, long long ld, const void* b, const void* a, long long ld_a, const void* gate, long long ld_gate,
+                   const float* conv, const float* a_log, const float* dt_bias, const float* norm, void* ring, float* state,
+                   const int* cu_q, const int* context_lens, const int* slots, float* scratch, void* out, long long ld_out,
+                   int T, int B, int H, int G, int D, int DV, int taps, int by_channel, int gate_silu, float eps, float out_scale,
+                   int f32, cudaStream_t stream) {
+  dlt::Args p;
+  p.x = x; p.ld = ld; p.b = b; p.a = a; p.ld_a = ld_a; p.gate = gate; p.ld_gate = ld_gate; p.conv = conv; p.a_log = a_log;
+  p.dt_bias = dt_bias; p.norm = norm; p.ring = ring; p.state = state; p.cu_q = cu_q; p.context_lens = context_lens;
+  p.slots = slots; p.out = out; p.ld_out = ld_out; p.T = T; p.B = B; p.H = H; p.G = G; p.D = D; p.DV = DV; p.taps = taps;
+  p.by_channel = by_channel; p.gate_silu = gate_silu; p.eps = eps; p.out_scale = out_scale;
+  if (dlt::check(p)) return 1;
+  if (T == 0) return 0;
+  if (!cu_q) {
+    if (!mfb_delta_decode_supported(D, DV) || T != B || !dlt::al(state, 16)) {
+      mfb_host::set_error("delta_rule: decode step of %d rows, %d slots, D=%d DV=%d", T, B, D, DV);
+      return 1;
+    }
+    return f32 ? dlt::decode<float>(p, stream) : dlt::decode<__nv_bfloat16>(p, stream);
+  }
+  auto up = [](long long n) { return (n + 3) / 4 * 4; };
+  p.qk = scratch;
+  p.v = p.qk + up((long long)T * G * 2 * D);
+  p.o = p.v + up((long long)T * H * DV);
+  p.beta = p.o + up((long long)T * H * DV);
+  p.g = p.beta + up((long long)T * H * 2);
+  int rc = f32 ? dlt::prepare<float>(p, stream) : dlt::prepare<__nv_bfloat16>(p, stream);
+  if (rc) return rc;
+  if (f32) rc = by_channel ? dlt::scan<float, true>(p, stream) : dlt::scan<float, false>(p, stream);
+  else rc = by_channel ? dlt::scan<__nv_bfloat16, true>(p, stream) : dlt::scan<__nv_bfloat16, false>(p, stream);
+  if (rc) return rc;
+  return f32 ? dlt::gate_out<float>(p, stream) : dlt::gate_out<__nv_bfloat16>(p, stream);
+}
+
+}  // extern "C"

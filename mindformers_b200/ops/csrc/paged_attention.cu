@@ -235,10 +235,11 @@ paged_decode_split_kernel(const __nv_bfloat16* __restrict__ q,        // [B, Hq,
 
 // out[row, h, :] = merge over splits of (acc, max, sum). With cu_q [B + 1] the result of sequence b goes to row cu_q[b],
 // and only sequences with exactly one row are written; otherwise row b. sink [Hq] (or null) adds exp(sink_h) to the
-// denominator.
+// denominator. Rows of out lie ld_out elements apart; the result is multiplied by out_scale.
 __global__ void paged_combine_kernel(const float* __restrict__ part_acc, const float* __restrict__ part_ml,
                                      __nv_bfloat16* __restrict__ out, int splits, int hd, int Hq,
-                                     const int* __restrict__ cu_q, const float* __restrict__ sink) {
+                                     const int* __restrict__ cu_q, const float* __restrict__ sink, long long ld_out,
+                                     float out_scale) {
   const size_t bh = blockIdx.x;
   const int b = blockIdx.x / Hq, h = blockIdx.x - b * Hq;
   size_t row = b;
@@ -258,7 +259,7 @@ __global__ void paged_combine_kernel(const float* __restrict__ part_acc, const f
     num += w * part_acc[(bh * splits + s2) * hd + d];
     den += w * part_ml[(bh * splits + s2) * 2 + 1];
   }
-  out[(row * Hq + h) * hd + d] = __float2bfloat16(den > 0.f ? num / den : 0.f);
+  out[row * ld_out + (size_t)h * hd + d] = __float2bfloat16(den > 0.f ? out_scale * num / den : 0.f);
 }
 
 // out[t, :] = cache[slot(t), :] gathered through the block table: token i of sequence b for i < lens[b],
@@ -379,10 +380,12 @@ int mfb_paged_decode_attention_ex(const void* q, const void* key_cache, const vo
       part_ml, Hq, Hkv, block_size, max_blocks, chunk, scale)
   if (hd == 128) {
     if (i8) MFB_PA_LAUNCH(128, true); else MFB_PA_LAUNCH(128, false);
-    paged_combine_kernel<<<B * Hq, 128, 0, stream>>>(part_acc, part_ml, (__nv_bfloat16*)out, splits, 128, Hq, nullptr, nullptr);
+    paged_combine_kernel<<<B * Hq, 128, 0, stream>>>(part_acc, part_ml, (__nv_bfloat16*)out, splits, 128, Hq, nullptr, nullptr,
+                                                 (long long)Hq * 128, 1.f);
   } else {
     if (i8) MFB_PA_LAUNCH(64, true); else MFB_PA_LAUNCH(64, false);
-    paged_combine_kernel<<<B * Hq, 64, 0, stream>>>(part_acc, part_ml, (__nv_bfloat16*)out, splits, 64, Hq, nullptr, nullptr);
+    paged_combine_kernel<<<B * Hq, 64, 0, stream>>>(part_acc, part_ml, (__nv_bfloat16*)out, splits, 64, Hq, nullptr, nullptr,
+                                                (long long)Hq * 64, 1.f);
   }
 #undef MFB_PA_LAUNCH
   return cudaGetLastError() == cudaSuccess ? 0 : 2;
@@ -390,10 +393,10 @@ int mfb_paged_decode_attention_ex(const void* q, const void* key_cache, const vo
 
 // Merge of the `splits` partial results of every (sequence, query head): rows = sequences x Hq, hd up to 1024 columns.
 int mfb_paged_combine_ex(const float* part_acc, const float* part_ml, void* out, int splits, int rows, int hd, int Hq,
-                         const int* cu_q, const float* sink, cudaStream_t stream) {
+                         const int* cu_q, const float* sink, long long ld_out, float out_scale, cudaStream_t stream) {
   if (hd < 1 || hd > 1024 || Hq < 1) { mfb_host::set_error("paged_combine: head dim %d", hd); return 1; }
   paged_combine_kernel<<<rows, (hd + 31) / 32 * 32, 0, stream>>>(part_acc, part_ml, (__nv_bfloat16*)out, splits, hd, Hq, cu_q,
-                                                                sink);
+                                                                sink, ld_out, out_scale);
   return cudaGetLastError() == cudaSuccess ? 0 : 2;
 }
 

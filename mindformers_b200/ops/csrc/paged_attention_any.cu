@@ -4,7 +4,7 @@
 // A batch is ragged: sequence b brings the rows cu_q[b] .. cu_q[b + 1] - 1, its last tokens, which are already in the
 // cache; row r sits at position context_lens[b] - (cu_q[b + 1] - r). Keys are visible up to the row's own position, and
 // with `chunk` > 0 only inside the row's chunk of `chunk` positions counted from 0. `sink` [Hq] adds exp(sink_h) to the
-// softmax denominator of head h (no key, no value, not scaled).
+// softmax denominator of head h (no key, no value, not scaled). `softcap` > 0 bounds the scores: softcap * tanh(score / softcap).
 //
 // One CTA of four warps per (row, query head): a warp takes every fourth key, its lanes split the head dimension; the
 // warps' online softmax states are merged through shared memory in a fixed order. All arithmetic is fp32.
@@ -27,7 +27,8 @@ __global__ void __launch_bounds__(kWarps * 32)
 paged_attention_any_kernel(const T* __restrict__ q, const T* __restrict__ key_cache, const T* __restrict__ value_cache,
                            const int* __restrict__ block_tables, const int* __restrict__ context_lens,
                            const int* __restrict__ cu_q, const float* __restrict__ sink, T* __restrict__ out, int B, int Hq,
-                           int Hkv, int D, int DV, int block_size, int max_blocks, int chunk, float scale) {
+                           int Hkv, int D, int DV, int block_size, int max_blocks, int chunk, float scale, float softcap,
+                           long long ld_out, float out_scale) {
   const int r = blockIdx.x, h = blockIdx.y;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   int b, pos;
@@ -67,6 +68,7 @@ paged_attention_any_kernel(const T* __restrict__ q, const T* __restrict__ key_ca
       if (d < D) s = fmaf(qr[i], ld(kp + d), s);
     }
     s = warp_sum(s);
+    if (softcap > 0.f) s = softcap * tanhf(s / softcap);
     const float m_new = fmaxf(m, s);
     const float alpha = expf(m - m_new), p = expf(s - m_new);
     l = l * alpha + p;
@@ -93,25 +95,25 @@ paged_attention_any_kernel(const T* __restrict__ q, const T* __restrict__ key_ca
     wgt[w] = sh_m[w] == -INFINITY ? 0.f : expf(sh_m[w] - mx);
     den += wgt[w] * sh_l[w];
   }
-  const float inv = den > 0.f ? 1.f / den : 0.f;
+  const float inv = den > 0.f ? out_scale / den : 0.f;
   for (int d = threadIdx.x; d < DV; d += kWarps * 32) {
     float num = 0.f;
 #pragma unroll
     for (int w = 0; w < kWarps; ++w) num += wgt[w] * sh_acc[w][d];
-    st(out + ((size_t)r * Hq + h) * DV + d, num * inv);
+    st(out + r * ld_out + (size_t)h * DV + d, num * inv);
   }
 }
 
 template <typename T>
 int launch(const void* q, const void* kc, const void* vc, const int* bt, const int* cl, const int* cu, const float* sink,
            void* out, int rows, int B, int Hq, int Hkv, int D, int DV, int bs, int mb, int chunk, float scale,
-           cudaStream_t stream) {
+           float softcap, long long ld_out, float out_scale, cudaStream_t stream) {
   dim3 grid(rows, Hq);
   const int n = ((D > DV ? D : DV) + 31) / 32;
 #define MFB_PAA(N_)                                                                                                   \
   paged_attention_any_kernel<T, N_><<<grid, kWarps * 32, 0, stream>>>((const T*)q, (const T*)kc, (const T*)vc, bt, cl, \
                                                                       cu, sink, (T*)out, B, Hq, Hkv, D, DV, bs, mb,   \
-                                                                      chunk, scale)
+                                                                      chunk, scale, softcap, ld_out, out_scale)
   if (n <= 2) MFB_PAA(2); else if (n <= 4) MFB_PAA(4); else if (n <= 8) MFB_PAA(8); else MFB_PAA(16);
 #undef MFB_PAA
   if (cudaGetLastError() != cudaSuccess) { mfb_host::set_error("paged_attention_any: launch failed"); return 2; }
@@ -124,12 +126,13 @@ int launch(const void* q, const void* kc, const void* vc, const int* bt, const i
 extern "C" {
 using namespace mfb;
 
-// q [rows, Hq, D], caches [num_blocks, block_size, Hkv, D | DV], out [rows, Hq, DV]: fp32 (f32 = 1) or bf16. cu_q [B + 1]
-// (device) or null: one row per sequence. chunk <= 0: no chunks; sink: [Hq] fp32 or null.
+// q [rows, Hq, D], caches [num_blocks, block_size, Hkv, D | DV], out [rows, Hq, DV] (rows ld_out apart): fp32 (f32 = 1) or bf16. cu_q [B + 1]
+// (device) or null: one row per sequence. chunk <= 0: no chunks; sink: [Hq] fp32 or null. softcap > 0: scores become
+// softcap * tanh(score / softcap). Rows of out lie ld_out elements apart; the result is multiplied by out_scale.
 int mfb_paged_attention_any(const void* q, const void* key_cache, const void* value_cache, const int* block_tables,
                             const int* context_lens, const int* cu_q, const float* sink, void* out, int rows, int B, int Hq,
-                            int Hkv, int D, int DV, int block_size, int max_blocks, int chunk, float scale, int f32,
-                            cudaStream_t stream) {
+                            int Hkv, int D, int DV, int block_size, int max_blocks, int chunk, float scale, float softcap,
+                            long long ld_out, float out_scale, int f32, cudaStream_t stream) {
   if (rows <= 0 || B <= 0) return 0;
   if (Hkv < 1 || Hq < 1 || Hq % Hkv || Hq > 65535 || D < 1 || DV < 1 || D > 32 * paa::kMaxPerLane ||
       DV > 32 * paa::kMaxPerLane || block_size < 1 || (!cu_q && rows != B)) {
@@ -138,9 +141,9 @@ int mfb_paged_attention_any(const void* q, const void* key_cache, const void* va
     return 1;
   }
   return f32 ? paa::launch<float>(q, key_cache, value_cache, block_tables, context_lens, cu_q, sink, out, rows, B, Hq, Hkv, D,
-                                  DV, block_size, max_blocks, chunk, scale, stream)
+                                  DV, block_size, max_blocks, chunk, scale, softcap, ld_out, out_scale, stream)
              : paa::launch<__nv_bfloat16>(q, key_cache, value_cache, block_tables, context_lens, cu_q, sink, out, rows, B, Hq,
-                                          Hkv, D, DV, block_size, max_blocks, chunk, scale, stream);
+                                          Hkv, D, DV, block_size, max_blocks, chunk, scale, softcap, ld_out, out_scale, stream);
 }
 
 }  // extern "C"

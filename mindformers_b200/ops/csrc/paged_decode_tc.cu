@@ -48,6 +48,7 @@ struct Args {
   int max_blocks, block_size, num_q_heads, num_kv_heads, group, splits;
   int D, DV, chunk, head_blocks;   // head_blocks: CTAs of up to 16 query heads per KV head
   float scale_log2;
+  float cap_log2, cap_scale;       // soft cap of the scores in log2 units (0: none) and scale / cap
   float* part_acc;           // [B, Hq, splits, DV] unnormalised
   float* part_ml;            // [B, Hq, splits, 2]: running max (log2 units), sum
   int* status;
@@ -57,6 +58,14 @@ __device__ __forceinline__ float ex2(float x) {
   float y;
   asm volatile("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
+}
+
+// cap * tanh(x) from exp(2 |x|): the error stays at a few 1e-7 of the cap
+__device__ __forceinline__ float capped(float x, float cap) {
+  const float e = ex2(fabsf(x) * 2.8853900817779268f);
+  float r;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(e + 1.f));
+  return copysignf(cap * fmaf(-2.f, r, 1.f), x);
 }
 
 __global__ void __launch_bounds__(kThreads, 2)
@@ -254,6 +263,11 @@ paged_decode_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       const bool valid = tok < len && tok >= first_tok;
 #pragma unroll
       for (int h = 0; h < kHeads; ++h) s[h] = valid ? __uint_as_float(sr[h]) * args.scale_log2 : -INFINITY;
+      if (args.cap_log2 > 0.f && valid) {
+#pragma unroll
+        for (int h = 0; h < kHeads; ++h)
+          if (h < n_heads) s[h] = capped(__uint_as_float(sr[h]) * args.cap_scale, args.cap_log2);
+      }
       // per-head maximum over the 128 tokens of the tile
 #pragma unroll
       for (int h = 0; h < kHeads; ++h) {
@@ -363,7 +377,8 @@ extern "C" {
 using namespace mfb;
 
 int mfb_paged_combine_ex(const float* part_acc, const float* part_ml, void* out, int splits, int rows, int hd, int Hq,
-                         const int* cu_q, const float* sink, cudaStream_t stream);      // paged_attention.cu
+                         const int* cu_q, const float* sink, long long ld_out, float out_scale,
+                         cudaStream_t stream);      // paged_attention.cu
 
 // 1 when the tensor-core kernel serves these shapes (bf16 cache): sizes are multiples of 8 up to 128, the block size is
 // 16, 32, 64 or 128. Any number of query heads per KV head: a CTA takes 16 of them.
@@ -397,12 +412,13 @@ int mfb_paged_decode_tc_splits(int B, int Hkv, int max_len) {
 // mfb_paged_decode_attention (mfb_paged_decode_scratch_bytes(B, Hq, DV, splits)). cu_q null: row b belongs to sequence b
 // (rows == B); else [B + 1] row boundaries of a ragged batch, of which only the sequences with one row are computed and
 // written. chunk > 0: keys of the query's own chunk of positions only. sink: [Hq] fp32 or null, adds exp(sink) to the
-// softmax denominator.
+// softmax denominator. softcap > 0: scores become softcap * tanh(score / softcap). Rows of out lie ld_out elements apart; the
+// result is multiplied by out_scale.
 int mfb_paged_decode_attention_tc_ex(const void* q, const void* key_cache, const void* value_cache, const int* block_tables,
                                      const int* context_lens, const int* cu_q, const float* sink, void* out, void* scratch,
                                      int splits, int rows, int B, int Hq, int Hkv, int D, int DV, int num_blocks,
-                                     int block_size, int max_blocks, int chunk, float scale, int* status,
-                                     cudaStream_t stream) {
+                                     int block_size, int max_blocks, int chunk, float scale, float softcap,
+                                     long long ld_out, float out_scale, int* status, cudaStream_t stream) {
   if (!mfb_paged_decode_tc_supported_ex(Hq, Hkv, D, DV, block_size) || splits < 1 || num_blocks < 1 || (!cu_q && rows != B)) {
     mfb_host::set_error("paged_decode_tc: unsupported Hq=%d Hkv=%d D=%d DV=%d block_size=%d splits=%d", Hq, Hkv, D, DV,
                         block_size, splits);
@@ -421,6 +437,8 @@ int mfb_paged_decode_attention_tc_ex(const void* q, const void* key_cache, const
   a.block_size = block_size; a.num_q_heads = Hq; a.num_kv_heads = Hkv; a.group = Hq / Hkv; a.splits = splits;
   a.D = D; a.DV = DV; a.chunk = chunk; a.head_blocks = (a.group + pdt::kHeads - 1) / pdt::kHeads;
   a.scale_log2 = scale * 1.4426950408889634f;
+  a.cap_log2 = softcap > 0.f ? softcap * 1.4426950408889634f : 0.f;
+  a.cap_scale = softcap > 0.f ? scale / softcap : 0.f;
   a.part_acc = reinterpret_cast<float*>(scratch);
   a.part_ml = a.part_acc + static_cast<size_t>(B) * Hq * splits * DV;
   a.status = status;
@@ -435,7 +453,7 @@ int mfb_paged_decode_attention_tc_ex(const void* q, const void* key_cache, const
   dim3 grid(splits, Hkv * a.head_blocks, B);
   pdt::paged_decode_tc_kernel<<<grid, pdt::kThreads, pdt::kSmem, stream>>>(tQ, tK, tV, a);
   if (cudaGetLastError() != cudaSuccess) { mfb_host::set_error("paged_decode_tc: launch failed"); return 11; }
-  return mfb_paged_combine_ex(a.part_acc, a.part_ml, out, splits, B * Hq, DV, Hq, cu_q, sink, stream);
+  return mfb_paged_combine_ex(a.part_acc, a.part_ml, out, splits, B * Hq, DV, Hq, cu_q, sink, ld_out, out_scale, stream);
 }
 
 // q [B, Hq, 128], caches [num_blocks, block_size, Hkv, 128], out [B, Hq, 128]: one row per sequence, no chunks, no sink.
@@ -445,7 +463,7 @@ int mfb_paged_decode_attention_tc(const void* q, const void* key_cache, const vo
                                   cudaStream_t stream) {
   return mfb_paged_decode_attention_tc_ex(q, key_cache, value_cache, block_tables, context_lens, nullptr, nullptr, out, scratch,
                                           splits, B, B, Hq, Hkv, pdt::kHd, pdt::kHd, num_blocks, block_size, max_blocks, 0,
-                                          scale, status, stream);
+                                          scale, 0.f, (long long)Hq * pdt::kHd, 1.f, status, stream);
 }
 
 }  // extern "C"

@@ -4,7 +4,8 @@
 // Sequence b brings the rows cu_q[b] .. cu_q[b + 1] - 1 of q; its keys and values, those rows included, are in the cache
 // already, so a whole prompt, a later portion of a prompt and any mix of sequences are the same problem: row r of the
 // portion sits at position context_lens[b] - q_len + r and sees keys up to itself, with `chunk` > 0 only those of its
-// own chunk of `chunk` positions (counted from position 0). `sink` [Hq] adds exp(sink_h) to the denominator.
+// own chunk of `chunk` positions (counted from position 0). `sink` [Hq] adds exp(sink_h) to the denominator. A soft cap
+// bounds the scores (cap * tanh(score / cap)).
 //
 // The tensor-core pipeline is the one of flash_attention_fwd2.cu (P goes back into tensor memory and is read from there
 // by the P V product), with one 128-row query tile per CTA and one stage of K and of V: a CTA then takes half of an SM's
@@ -43,6 +44,9 @@ struct Args {
   __nv_bfloat16* out;        // [T, Hq, DV]
   int num_q_heads, group, D, DV, block_size, max_blocks, chunk;
   float scale_log2;
+  float cap_log2, cap_scale;   // soft cap of the scores in log2 units (CAP kernels) and scale / cap
+  long long ld_out;
+  float out_scale;
   int* status;
 };
 
@@ -50,6 +54,13 @@ __device__ __forceinline__ float ex2(float x) {
   float y;
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
+}
+// cap * tanh(x) from exp(2 |x|): the error stays at a few 1e-7 of the cap
+__device__ __forceinline__ float capped(float x, float cap) {
+  const float e = ex2(fabsf(x) * 2.8853900817779268f);
+  float r;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(e + 1.f));
+  return copysignf(cap * fmaf(-2.f, r, 1.f), x);
 }
 __device__ __forceinline__ uint64_t pack2(float lo, float hi) {
   uint64_t r;
@@ -62,6 +73,11 @@ __device__ __forceinline__ void unpack2(uint64_t v, float& lo, float& hi) {
 __device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
   uint64_t d;
   asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+  return d;
+}
+__device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
+  uint64_t d;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
   return d;
 }
 __device__ __forceinline__ uint64_t add2(uint64_t a, uint64_t b) {
@@ -86,8 +102,18 @@ __device__ __forceinline__ void tmem_st_32x32b_x32(uint32_t taddr, const uint32_
       : "memory");
 }
 
-// HQ: padded query / key size, HV: padded value size (64 or 128)
-template <int HQ, int HV>
+// tanh(x) / x as a polynomial in z = x^2 on |x| <= kPolyReach (Chebyshev interpolation of degree 4 on [0, kPolyReach^2]:
+// relative error 7.4e-8). It runs on the FMA pipes two scores at a time, which leaves the exponentials to the softmax.
+constexpr float kPolyReach = 0.6f;
+__device__ __forceinline__ uint64_t tanh_ratio2(uint64_t z) {
+  const uint64_t c0 = pack2(0.999999926f, 0.999999926f), c1 = pack2(-0.33332302f, -0.33332302f),
+                 c2 = pack2(0.133100644f, 0.133100644f), c3 = pack2(-0.0520966534f, -0.0520966534f),
+                 c4 = pack2(0.0154687513f, 0.0154687513f);
+  return fma2(fma2(fma2(fma2(c4, z, c3), z, c2), z, c1), z, c0);
+}
+
+// HQ: padded query / key size, HV: padded value size (64 or 128); CAP: scores are soft-capped
+template <int HQ, int HV, bool CAP>
 __global__ void __launch_bounds__(kThreads, 2)
 paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                         const __grid_constant__ CUtensorMap tmV, const Args args) {
@@ -292,7 +318,8 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
             }
           }
           float mx = fmaxf(fmaxf(mxs[0], mxs[1]), fmaxf(mxs[2], mxs[3]));
-          mx *= args.scale_log2;
+          if (!CAP) mx *= args.scale_log2;
+          else if (mx != -INFINITY) mx = capped(mx * args.cap_scale, args.cap_log2);      // the cap keeps the order
           float alpha = 1.f;
           if (j == lo) {
             m_used = mx;                               // -inf when this row sees nothing in its tile's first key tile
@@ -337,6 +364,24 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
               tmem_ld_wait();
             }
             float* s = reinterpret_cast<float*>(sr);
+            if constexpr (CAP) {
+              // scores in log2 units: by the polynomial where every score of the warp is within its reach
+              float am = 0.f;
+#pragma unroll
+              for (int i = 0; i < 64; ++i) am = fmaxf(am, fabsf(s[i]));
+              if (__all_sync(0xffffffffu, am * args.cap_scale <= kPolyReach)) {
+                const uint64_t cs2 = pack2(args.cap_scale, args.cap_scale);
+#pragma unroll
+                for (int i = 0; i < 32; ++i) {
+                  const uint64_t v = pack2(s[2 * i], s[2 * i + 1]);
+                  const uint64_t x = mul2(v, cs2);
+                  unpack2(mul2(mul2(v, scale2), tanh_ratio2(mul2(x, x))), s[2 * i], s[2 * i + 1]);
+                }
+              } else {
+#pragma unroll
+                for (int i = 0; i < 64; ++i) s[i] = capped(s[i] * args.cap_scale, args.cap_log2);
+              }
+            }
 #pragma unroll
             for (int a = 0; a < 2; ++a) {
               if (MASK && hi_min < h * 64 + a * 32 + 31) {
@@ -354,7 +399,8 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
 #pragma unroll
             for (int i = 0; i < 32; ++i) {
               float t0, t1;
-              unpack2(fma2(pack2(s[2 * i], s[2 * i + 1]), scale2, negm2), t0, t1);
+              const uint64_t v = pack2(s[2 * i], s[2 * i + 1]);
+              unpack2(CAP ? add2(v, negm2) : fma2(v, scale2, negm2), t0, t1);
               const float e0 = ex2(t0), e1 = ex2(t1);
               rs2[i & 3] = add2(rs2[i & 3], pack2(e0, e1));
               pk[i] = pack_bf16x2(e0, e1);
@@ -379,10 +425,10 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
       tc_fence_after();
       // the sink joins the denominator on the scale of the sum; an enormous sink overflows to a zero weight of the keys
       const float den = args.sink ? l_sum + ex2(args.sink[t.head] * 1.4426950408889634f - m_used) : l_sum;
-      const float inv_l = 1.f / den;
+      const float inv_l = args.out_scale / den;
       // 32 columns at a time through 2 KB of shared memory per warp, so that a store covers 64 bytes of eight rows each
       uint8_t* stage = sOut + ew * 2048;
-      __nv_bfloat16* obase = args.out + (static_cast<size_t>(t.q0 + ew * 32) * args.num_q_heads + t.head) * args.DV;
+      __nv_bfloat16* obase = args.out + (t.q0 + ew * 32) * args.ld_out + static_cast<size_t>(t.head) * args.DV;
 #pragma unroll
       for (int c = 0; c < HV / 32; ++c) {
         uint32_t r[32];
@@ -401,7 +447,7 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
         for (int i = 0; i < 4; ++i) {
           const int rr = i * 8 + (lane >> 2);
           if (ew * 32 + rr < t.rows && col < args.DV)
-            *reinterpret_cast<uint4*>(obase + static_cast<size_t>(rr) * args.num_q_heads * args.DV + col) =
+            *reinterpret_cast<uint4*>(obase + rr * args.ld_out + col) =
                 *reinterpret_cast<const uint4*>(stage + rr * 64 + (((lane & 3) ^ ((rr >> 1) & 3)) << 4));
         }
         __syncwarp();
@@ -434,12 +480,12 @@ int make_q_map(CUtensorMap* out, const void* q, uint64_t T, uint64_t Hq, uint64_
   return 0;
 }
 
-template <int HQ, int HV>
+template <int HQ, int HV, bool CAP>
 int launch(const CUtensorMap& tQ, const CUtensorMap& tK, const CUtensorMap& tV, const Args& a, int max_ctas, cudaStream_t stream) {
   constexpr int QBYTES = HQ / 64 * kSubBytes, VBYTES = HV / 64 * kSubBytes;
   constexpr int SMEM = 2 * QBYTES + VBYTES + 4 * 2048 + 9 * 8 + 16 + 1024;
   static_assert(2 * SMEM <= 232448, "shared memory budget exceeded");
-  auto kern = paged_prefill_tc_kernel<HQ, HV>;
+  auto kern = paged_prefill_tc_kernel<HQ, HV, CAP>;
   static bool attr_set = false;
   if (!attr_set) {
     if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM) != cudaSuccess) {
@@ -469,16 +515,21 @@ int mfb_paged_prefill_tc_supported(int Hq, int Hkv, int D, int DV, int block_siz
 // q [T, Hq, D], caches [num_blocks, block_size, Hkv, D | DV], out [T, Hq, DV], all bf16. work [n_work, 4] int32: (sequence,
 // first row of q, 1..128 rows, position of the first row) per query tile, heaviest first; the rows' keys are in the cache.
 // persistent: two CTAs per SM walk over all tiles (for tiles of a few key tiles); else a CTA per query tile and head, which
-// balances tiles of very different lengths better.
+// balances tiles of very different lengths better. softcap > 0: scores become softcap * tanh(score / softcap). Rows of out lie
+// ld_out elements apart; the result is multiplied by out_scale.
 int mfb_paged_prefill_tc(const void* q, const void* key_cache, const void* value_cache, const int* work, int n_work, int persistent,
                          const int* block_tables, const float* sink, void* out, int T,
                          int Hq, int Hkv, int D, int DV, int num_blocks, int block_size, int max_blocks, int chunk, float scale,
-                         int* status, cudaStream_t stream) {
+                         float softcap, long long ld_out, float out_scale, int* status, cudaStream_t stream) {
   if (!mfb_paged_prefill_tc_supported(Hq, Hkv, D, DV, block_size) || num_blocks < 1 || T < 1) {
     mfb_host::set_error("paged_prefill_tc: unsupported Hq=%d Hkv=%d D=%d DV=%d block_size=%d", Hq, Hkv, D, DV, block_size);
     return 1;
   }
   if (n_work <= 0) return 0;
+  if (ld_out % 8 || (reinterpret_cast<uintptr_t>(out) & 15)) {
+    mfb_host::set_error("paged_prefill_tc: rows of the result must start on 16 bytes");
+    return 1;
+  }
   CUtensorMap tQ, tK, tV;
   int rc;
   const CUtensorMapDataType BF = CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
@@ -491,13 +542,19 @@ int mfb_paged_prefill_tc(const void* q, const void* key_cache, const void* value
   a.out = reinterpret_cast<__nv_bfloat16*>(out);
   a.num_q_heads = Hq; a.group = Hq / Hkv; a.D = D; a.DV = DV; a.block_size = block_size; a.max_blocks = max_blocks;
   a.chunk = chunk; a.scale_log2 = scale * 1.4426950408889634f; a.status = status;
+  a.cap_log2 = softcap > 0.f ? softcap * 1.4426950408889634f : 0.f;
+  a.cap_scale = softcap > 0.f ? scale / softcap : 0.f;
+  a.ld_out = ld_out; a.out_scale = out_scale;
   const int max_ctas = persistent ? 2 * 148 : a.n_items;
+#define MFB_PPT(HQ_, HV_) \
+  return softcap > 0.f ? ppt::launch<HQ_, HV_, true>(tQ, tK, tV, a, max_ctas, stream) : ppt::launch<HQ_, HV_, false>(tQ, tK, tV, a, max_ctas, stream)
   if (D > 64) {
-    if (DV > 64) return ppt::launch<128, 128>(tQ, tK, tV, a, max_ctas, stream);
-    return ppt::launch<128, 64>(tQ, tK, tV, a, max_ctas, stream);
+    if (DV > 64) MFB_PPT(128, 128);
+    MFB_PPT(128, 64);
   }
-  if (DV > 64) return ppt::launch<64, 128>(tQ, tK, tV, a, max_ctas, stream);
-  return ppt::launch<64, 64>(tQ, tK, tV, a, max_ctas, stream);
+  if (DV > 64) MFB_PPT(64, 128);
+  MFB_PPT(64, 64);
+#undef MFB_PPT
 }
 
 }  // extern "C"

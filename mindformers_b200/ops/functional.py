@@ -229,19 +229,31 @@ def _pair_workspace(device) -> torch.Tensor:
 
 
 def grouped_gemm(a: torch.Tensor, b: torch.Tensor, block_group: torch.Tensor, num_blocks: torch.Tensor,
-                 *, b_mn: bool = False, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+                 *, b_mn: bool = False, out: Optional[torch.Tensor] = None, group_offsets: Optional[torch.Tensor] = None,
+                 seg_fill: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Ragged-M grouped GEMM for MoE experts.
 
     ``a``: ``[R, K]`` rows sorted by expert, every expert segment padded to a multiple of 128 rows.
     ``b``: ``[G, N, K]`` (or ``[G, K, N]`` when ``b_mn``). ``block_group[i]`` = expert of the i-th
-    128-row block; ``num_blocks`` = device scalar with the number of blocks in use.
+    128-row block; ``num_blocks`` = device scalar with the number of blocks in use. With ``group_offsets`` and ``seg_fill``
+    (rows in use per expert) padding rows may be left undefined.
     """
     G = b.shape[0]
     R, K = a.shape
     N = b.shape[2] if b_mn else b.shape[1]
     if out is None:
         out = torch.empty((R, N), dtype=a.dtype, device=a.device)
-    if not (_on_gpu(a) and _GEMM_BACKEND == "tcgen05" and a.dtype == torch.bfloat16):
+    tc = _GEMM_BACKEND == "tcgen05" and a.dtype == torch.bfloat16
+    if _on_gpu(a) and b_mn and a.dtype == b.dtype and a.dtype in (torch.bfloat16, torch.float32) \
+            and (not tc or K % 64 or N % 8) and a.is_contiguous() and b.is_contiguous() and out.is_contiguous():
+        # 32-bit experts and sizes that the tensor-core kernel does not take
+        rc = _lib.get_lib().mfb_grouped_gemm_any(
+            a.data_ptr(), b.data_ptr(), out.data_ptr(), R, N, K, block_group.data_ptr(), num_blocks.data_ptr(),
+            _lib.ptr(group_offsets), _lib.ptr(seg_fill), int(a.dtype == torch.float32), _lib.stream_ptr())
+        _lib.check(rc, "mfb_grouped_gemm_any")
+        _lib.count_launch()
+        return out
+    if not (_on_gpu(a) and tc):
         nb = int(num_blocks.item())
         bg = block_group[:nb].tolist()
         out.zero_()
@@ -486,6 +498,27 @@ def swiglu(x: torch.Tensor) -> torch.Tensor:
 # =================================================================================================
 # RoPE (applied in place to the leading heads of a packed [T, heads, hd] buffer)
 # =================================================================================================
+def clamped_glu(x: torch.Tensor, limit: float, alpha: float, plan=None) -> torch.Tensor:
+    """``g * sigmoid(alpha g) * (u + 1)`` of ``x [R, 2F]`` = gate | up, ``g = min(gate, limit)``, ``u = clamp(up, -limit,
+    limit)``, computed in fp32. ``plan``: a permutation plan whose unused rows are skipped (left undefined). No gradients."""
+    R, F_ = x.shape[0], x.shape[1] // 2
+    if not _on_gpu(x):
+        g, u = x.float().chunk(2, dim=-1)
+        g, u = g.clamp(max=limit), u.clamp(-limit, limit)
+        return (g * torch.sigmoid(alpha * g) * (u + 1)).to(x.dtype)
+    if torch.is_grad_enabled() and x.requires_grad:
+        raise NotImplementedError("clamped_glu has no backward pass")
+    if x.dtype not in (torch.bfloat16, torch.float32) or not x.is_contiguous():
+        raise TypeError("clamped_glu needs a contiguous bfloat16 or float32 matrix")
+    y = torch.empty((R, F_), dtype=x.dtype, device=x.device)
+    p = [None] * 4 if plan is None else [plan.block_group, plan.num_blocks, plan.group_offsets, getattr(plan, "seg_fill", None)]
+    rc = _lib.get_lib().mfb_clamped_glu(x.data_ptr(), y.data_ptr(), R, F_, float(limit), float(alpha), *(_lib.ptr(t) for t in p),
+                                        int(x.dtype == torch.float32), _lib.stream_ptr())
+    _lib.check(rc, "mfb_clamped_glu")
+    _lib.count_launch()
+    return y
+
+
 def rope_reference(x, cos, sin, positions, n_heads, rot, interleaved=False):
     """x: [T, heads_total, hd]; rotates the first n_heads heads. cos/sin: [max_pos, rot/2] fp32."""
     T = x.shape[0]

@@ -1,4 +1,4 @@
-"""Serving ops of decoders that keep a 32-bit residual stream and normalise the OUTPUT of their sub-layers.
+"""Serving ops of decoders that keep a 32-bit residual stream (or several) beside 16-bit activations.
 
 Like the ops of ``functional.py`` every op has two bodies: the sm_100a kernel, always taken for CUDA tensors (bf16 or
 fp32), and a plain PyTorch body for CPU tensors. They are inference ops: no gradients.
@@ -79,6 +79,40 @@ def norm_stream(x: torch.Tensor, w: torch.Tensor, b: Optional[torch.Tensor], eps
     _lib.check(rc, "mfb_norm_stream")
     _lib.count_launch()
     return y
+
+
+def residual_streams(x: torch.Tensor, n: int, y: Optional[torch.Tensor], mix: Optional[torch.Tensor],
+                     write: Optional[torch.Tensor], read: Optional[torch.Tensor], w: torch.Tensor, eps: float,
+                     keep: bool = True) -> Tuple[torch.Tensor, Optional[torch.Tensor]]:
+    """One step of ``n`` fp32 residual streams: ``x_t <- sum_s mix[s, t] x_s + write[t] y`` (without ``y``: no update), then
+    the next sub-layer's input ``rms_norm(sum_t read[t] x_t) * w`` (``read`` None: the sum of the streams).
+
+    ``x``: the streams ``[T, n, W]`` fp32 (updated in place) or, before the first update, the embedding ``[T, W]`` in the dtype
+    of ``w``, to which all streams are equal. Returns ``(input [T, W], streams)``; ``keep=False`` drops the streams, and
+    without an update they are ``x`` itself."""
+    embedded = x.dim() == 2
+    T, W, dtype = x.shape[0], x.shape[-1], w.dtype
+    if not x.is_cuda:
+        xs = x.float()[:, None].expand(T, n, W) if embedded else x
+        if y is not None:
+            xs = torch.einsum("sd,tsw->tdw", mix, xs) + write[:, None] * y.float()[:, None]
+        u = xs.sum(1) if read is None else (read[:, None] * xs).sum(1)
+        return norm_reference(u, w, None, eps, False).to(dtype), (x if y is None else xs if keep else None)
+    _check_dtype(dtype)
+    if x.dtype != (dtype if embedded else torch.float32) or not x.is_contiguous() or not (embedded or x.shape[1] == n) \
+            or (y is not None and (y.dtype != dtype or y.shape != (T, W) or y.stride(1) != 1)):
+        raise TypeError("residual_streams: fp32 streams (or the embedding) and a sub-layer output in the activation dtype expected")
+    _typed(mix, write, read, dtype=torch.float32)
+    h = torch.empty((T, W), dtype=dtype, device=x.device)
+    out = None
+    if y is not None and keep:
+        out = torch.empty((T, n, W), dtype=torch.float32, device=x.device) if embedded else x
+    rc = _lib.get_lib().mfb_residual_streams(
+        x.data_ptr(), int(embedded), _lib.ptr(y), 0 if y is None else y.stride(0), _lib.ptr(mix), _lib.ptr(write), _lib.ptr(read),
+        w.data_ptr(), _lib.ptr(out), h.data_ptr(), T, n, W, float(eps), int(dtype == torch.float32), _lib.stream_ptr())
+    _lib.check(rc, "mfb_residual_streams")
+    _lib.count_launch()
+    return h, (x if y is None else out)
 
 
 def relu2(x: torch.Tensor) -> torch.Tensor:

@@ -86,6 +86,17 @@ def linear_all_reduce(x, w):
     return fused_tp.gemm_all_reduce(x, w)
 
 
+def moe_local_enabled(config, x: torch.Tensor) -> bool:
+    """Forward-only calls on one rank that the exchange does not serve (32-bit activations, other widths)."""
+    from . import fused_moe
+    return not _FORCE_OFF and fused_moe.local_supported(config, x)
+
+
+def moe_local(layer, hidden, probs, ids):
+    from . import fused_moe
+    return fused_moe.moe_local(layer, hidden, probs, ids)
+
+
 def moe_dispatch_experts_combine(layer, hidden, probs, ids):
     from . import fused_moe
     return fused_moe.moe_dispatch_experts_combine(layer, hidden, probs, ids)

@@ -256,7 +256,7 @@ class _Dispatch(torch.autograd.Function):
     """``x [T,H]`` → expert input rows of this rank ``[rows, H]`` (permute + send)."""
 
     @staticmethod
-    def forward(ctx, x, ids, ex: MoEExchange, st: _PlanState, layer_key):
+    def forward(ctx, x, ids, ex: MoEExchange, st: _PlanState, layer_key, weights=None):
         x = x.contiguous()
         T = x.shape[0]
         if ex.world > 1:
@@ -264,7 +264,7 @@ class _Dispatch(torch.autograd.Function):
         else:
             xin = torch.empty(st.rows, ex.H, dtype=torch.bfloat16, device=x.device)
             ptrs = ex.local_ptrs(xin)
-        ex.scatter(st, x, ids, ptrs, zero_pad=not str(layer_key).startswith("nograd"))
+        ex.scatter(st, x, ids, ptrs, weights=weights, zero_pad=not str(layer_key).startswith("nograd"))
         ex.barrier(1)
         ctx.ex, ctx.st, ctx.T = ex, st, T
         ctx.save_for_backward(ids)
@@ -283,14 +283,14 @@ class _Dispatch(torch.autograd.Function):
             ptrs = ex.local_ptrs(dxin)
         dx, _ = ex.gather(st, T, ids, ptrs)
         ex.release_slot(*st.slot)
-        return dx, None, None, None, None
+        return dx, None, None, None, None, None
 
 
 class _Combine(torch.autograd.Function):
     """Expert output rows ``[rows, H]`` + ``probs [T,k]`` → ``[T,H]`` (receive + weighted unpermute)."""
 
     @staticmethod
-    def forward(ctx, y, probs, ids, ex: MoEExchange, st: _PlanState, layer_key):
+    def forward(ctx, y, probs, ids, ex: MoEExchange, st: _PlanState, layer_key, unweighted=False):
         T = probs.shape[0]
         probs = probs.contiguous().float()
         if ex.world > 1:
@@ -300,7 +300,7 @@ class _Combine(torch.autograd.Function):
         else:
             yout, ptrs = y.contiguous(), None
             ptrs = ex.local_ptrs(yout)
-        out, _ = ex.gather(st, T, ids, ptrs, weights=probs)
+        out, _ = ex.gather(st, T, ids, ptrs, weights=None if unweighted else probs)
         ctx.ex, ctx.st, ctx.T, ctx.ptrs = ex, st, T, ptrs
         ctx.save_for_backward(ids, probs, yout)
         return out
@@ -321,12 +321,43 @@ class _Combine(torch.autograd.Function):
         ex.barrier(1)
         # peers overwrite dy_ws only after this rank has passed the barrier of this layer's dispatch backward,
         # which comes after the expert GEMMs that consume it
-        return dy, dots, None, None, None, None
+        return dy, dots, None, None, None, None, None
 
 
 def supported(config, hidden: torch.Tensor) -> bool:
     return (hidden.is_cuda and hidden.dtype == torch.bfloat16 and hidden.dim() == 2 and hidden.shape[1] % 8 == 0
             and config.num_moe_experts <= 512 and ps.get_expert_model_parallel_world_size() <= 8)
+
+
+def local_supported(config, hidden: torch.Tensor) -> bool:
+    """One rank, forward only, any width, bf16 or fp32."""
+    return (hidden.is_cuda and hidden.dtype in (torch.bfloat16, torch.float32) and hidden.dim() == 2 and not torch.is_grad_enabled()
+            and config.num_moe_experts <= 512 and ps.get_expert_model_parallel_world_size() == 1)
+
+
+def moe_local(layer, hidden: torch.Tensor, probs: torch.Tensor, ids: torch.Tensor) -> torch.Tensor:
+    """Router outputs → combined expert outputs on one rank: the exchange's permutation plan with kernels for every width
+    and for 32-bit activations (``ops/csrc/moe_any.cu``)."""
+    cfg = layer.config
+    ex = MoEExchange.get(cfg)
+    ids, hidden, probs = ids.contiguous(), hidden.contiguous(), probs.contiguous().float()
+    T, H = hidden.shape
+    st = ex.plan(ids, T)
+    f32 = int(hidden.dtype == torch.float32)
+    on_input = bool(cfg.moe_apply_probs_on_input)
+    rows = torch.empty((st.rows, H), dtype=hidden.dtype, device=hidden.device)
+    rc = ex.lib.mfb_moe_scatter_any(hidden.data_ptr(), ids.data_ptr(), st.rank_in_e.data_ptr(), st.write_base.data_ptr(),
+                                    probs.data_ptr() if on_input else None, rows.data_ptr(), st.dest_row.data_ptr(), T, ex.k, H,
+                                    st.rows, f32, _lib.stream_ptr())
+    _lib.check(rc, "mfb_moe_scatter_any")
+    layer.last_tokens_per_expert = st.counts
+    y = layer.experts(rows, st.plan)
+    out = torch.empty_like(hidden)
+    rc = ex.lib.mfb_moe_gather_any(y.data_ptr(), st.dest_row.data_ptr(), None if on_input else probs.data_ptr(), out.data_ptr(), T,
+                                   ex.k, H, f32, _lib.stream_ptr())
+    _lib.check(rc, "mfb_moe_gather_any")
+    _lib.count_launch(2)
+    return out
 
 
 def moe_dispatch_experts_combine(layer, hidden: torch.Tensor, probs: torch.Tensor, ids: torch.Tensor) -> torch.Tensor:
@@ -341,10 +372,14 @@ def moe_dispatch_experts_combine(layer, hidden: torch.Tensor, probs: torch.Tenso
     slot = ex.acquire_slot(layer_key)
     st.slot = (layer_key, slot)
     key = f"{layer_key}.{slot}"
-    xin = apply_fn(_Dispatch, hidden, ids, ex, st, key)
+    on_input = bool(layer.config.moe_apply_probs_on_input)
+    if on_input and needs_grad:
+        raise NotImplementedError("routing weights on the experts' input have no backward pass")
+    weights = probs.contiguous().float() if on_input else None
+    xin = apply_fn(_Dispatch, hidden, ids, ex, st, key, weights)
     layer.last_tokens_per_expert = st.counts
     y = layer.experts(xin, st.plan)
-    out = apply_fn(_Combine, y, probs, ids, ex, st, key)
+    out = apply_fn(_Combine, y, probs, ids, ex, st, key, on_input)
     if not needs_grad:
         ex.release_slot(*st.slot)
     return out

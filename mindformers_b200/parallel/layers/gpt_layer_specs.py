@@ -13,12 +13,14 @@ from typing import List, Optional
 
 from ..spec_utils import ModuleSpec
 from .attention import CrossAttention, MLASelfAttention, MLASelfAttentionMegatron, SelfAttention
+from .delta_rule import GatedDeltaMixer, ParallelMixer
 from .mlp import MLP
 from .moe import GroupedMLP, MoELayer, SharedExpertMLP, TopKRouter
 from .mtp import MultiTokenPredictionBlock, MultiTokenPredictionLayer
 from .norm import build_norm
 from .ragged_attention import RaggedSelfAttention
-from .transformer_layer import OutputNormTransformerLayer, TransformerLayer, TransformerLayerSubmodules
+from .transformer_layer import (OutputNormTransformerLayer, StreamTransformerLayer, TransformerLayer,
+                                TransformerLayerSubmodules)
 
 
 def get_moe_module_spec(num_experts: Optional[int] = None, moe_grouped_gemm: bool = True) -> ModuleSpec:
@@ -64,8 +66,25 @@ def get_output_norm_layer_spec(config) -> ModuleSpec:
         post_attn_layernorm=norm, post_mlp_layernorm=norm if ff else None))
 
 
+_MIXERS = {"attention": RaggedSelfAttention, "delta": GatedDeltaMixer, "parallel": ParallelMixer}
+
+
+def get_stream_layer_spec(config, is_moe: bool) -> ModuleSpec:
+    """Spec of one layer on several residual streams: ``config.mixer``, then an MoE or dense feed-forward (none with
+    ``ffn_hidden_size == 0``)."""
+    norm = ModuleSpec(module=build_norm)
+    mlp = get_mlp_module_spec(config.num_moe_experts if is_moe else None) if is_moe or config.ffn_hidden_size else None
+    return ModuleSpec(module=StreamTransformerLayer, submodules=TransformerLayerSubmodules(
+        input_layernorm=norm, self_attention=ModuleSpec(module=_MIXERS[config.mixer]), mlp=mlp,
+        pre_mlp_layernorm=norm if mlp is not None else None))
+
+
 def get_gpt_layer_spec_for_config(config, is_moe: bool) -> ModuleSpec:
     """``get_gpt_layer_local_spec`` with the switches taken from a ``TransformerConfig``."""
+    if config.residual_streams:
+        if config.norm_placement != "input" or not config.ragged_attention or config.normalization != "RMSNorm":
+            raise ValueError("layers on residual streams are pre-norm layers with RMS norms and ragged attention")
+        return get_stream_layer_spec(config, is_moe)
     if config.norm_placement == "output":
         if is_moe or not config.ragged_attention:
             raise ValueError("output-normalised layers are built with ragged attention and a dense feed-forward")

@@ -238,6 +238,12 @@ class GroupedMLP(nn.Module):
 
     w1_fp8 = w2_fp8 = w1_scale_inv = w2_scale_inv = None
 
+    def _activate(self, h, plan):
+        cfg = self.config
+        if cfg.moe_activation == "clamped_glu":
+            return Fn.clamped_glu(h, cfg.moe_activation_limit, cfg.moe_activation_alpha, plan)
+        return Fn.swiglu(h)
+
     def quantize_fp8_(self) -> bool:
         """Inference: replace the bf16 expert weights by block-scaled fp8 ones (``[E, out, in]`` e4m3 with one fp32
         scale per 128 x 128 block, the DeepSeek-V3 checkpoint format)."""
@@ -260,10 +266,14 @@ class GroupedMLP(nn.Module):
                       group_offsets=getattr(plan, "group_offsets", None), seg_fill=getattr(plan, "seg_fill", None))
             xq, sa = Fn.quantize_act_1x128(x)
             h = Fn.fp8_gemm(xq, sa, self.w1_fp8, self.w1_scale_inv, **kw)
-            hq, sh = Fn.quantize_act_1x128(Fn.swiglu(h))
+            hq, sh = Fn.quantize_act_1x128(self._activate(h, None))
             return Fn.fp8_gemm(hq, sh, self.w2_fp8, self.w2_scale_inv, **kw)
+        if not torch.is_grad_enabled() and getattr(plan, "seg_fill", None) is not None:
+            kw = dict(b_mn=True, group_offsets=plan.group_offsets, seg_fill=plan.seg_fill)
+            h = Fn.grouped_gemm(x, self.weight1, plan.block_group, plan.num_blocks, **kw)
+            return Fn.grouped_gemm(self._activate(h, plan), self.weight2, plan.block_group, plan.num_blocks, **kw)
         h = apply_fn(_GroupedLinearFn, x, self.weight1, plan.block_group, plan.num_blocks, plan.group_offsets)
-        h = Fn.swiglu(h)
+        h = self._activate(h, plan)
         return apply_fn(_GroupedLinearFn, h, self.weight2, plan.block_group, plan.num_blocks, plan.group_offsets)
 
 
@@ -403,8 +413,15 @@ class MoELayer(nn.Module):
         from .. import fused_comm
         if not self.staged and fused_comm.moe_enabled(self.config, hidden):
             out = fused_comm.moe_dispatch_experts_combine(self, hidden, probs, ids)
+        elif not self.staged and fused_comm.moe_local_enabled(self.config, hidden):
+            out = fused_comm.moe_local(self, hidden, probs, ids)
         else:
             x, plan, ctx = self.dispatcher.dispatch(hidden, ids)
+            if self.config.moe_apply_probs_on_input:
+                if ctx[0] != "local":
+                    raise NotImplementedError("routing weights on the experts' input need the fused exchange across ranks")
+                x[plan.dest] = (x[plan.dest].float() * probs.reshape(-1, 1)).to(x.dtype)
+                probs = torch.ones_like(probs)
             y = self.experts(x, plan)
             out = self.dispatcher.combine(y, plan, ctx, probs.to(hidden.dtype))
         if with_shared and self.shared_experts is not None:

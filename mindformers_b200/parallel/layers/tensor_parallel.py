@@ -234,7 +234,8 @@ class RowParallelLinear(_Fp8WeightMixin, nn.Module):
 
     def __init__(self, input_size: int, output_size: int, *, config, init_method: Callable = None,
                  bias: bool = False, input_is_parallel: bool = True, skip_bias_add: bool = False,
-                 is_expert: bool = False, delay_allreduce: bool = False):
+                 is_expert: bool = False, delay_allreduce: bool = False, partition_sections=None):
+        """``partition_sections``: the input columns are these sections, each split over the ranks."""
         super().__init__()
         self.config = config
         self.tp = 1 if is_expert and config.expert_tensor_parallel_size == 1 else ps.get_tensor_model_parallel_world_size()
@@ -250,8 +251,9 @@ class RowParallelLinear(_Fp8WeightMixin, nn.Module):
         init = init_method or default_init(config.output_layer_init_std)
         self.weight = _init_weight((output_size, self.input_size_per_partition), init, config.params_dtype, dev,
                                    partition_dim=1, full_shape=(output_size, input_size), rank=self.rank,
-                                   world=self.tp)
+                                   world=self.tp, sections=partition_sections)
         _mark_tp(self.weight, self.tp > 1, 1)
+        self.weight.partition_sections = tuple(partition_sections) if partition_sections else None
         if bias:
             self.bias = nn.Parameter(torch.zeros(output_size, dtype=config.params_dtype, device=dev))
             _mark_tp(self.bias, False, -1)

@@ -139,6 +139,70 @@ class OutputNormTransformerLayer(nn.Module):
         return pending, residual, None
 
 
+class StreamConnection(nn.Module):
+    """How one sub-layer is tied to ``n`` residual streams: its input is ``sum_s read[s] x_s``, and its output ``y`` enters as
+    ``x_t <- sum_s mix[s, t] x_s + write[t] y``. fp32."""
+
+    def __init__(self, n: int, device=None):
+        super().__init__()
+        def param(t):
+            return nn.Parameter(t.to(device))
+        self.read = param(torch.full((n,), 1.0 / n))
+        self.write = param(torch.ones(n))
+        self.mix = param(torch.eye(n))
+
+
+@dataclass
+class ResidualStreams:
+    """The streams ``x`` (``[T, n, W]`` fp32, or the embedding before the first update) and the connection of the sub-layer
+    whose output has not entered them yet."""
+    x: torch.Tensor
+    link: Optional[StreamConnection] = None
+
+
+class StreamTransformerLayer(nn.Module):
+    """Pre-norm layer on several fp32 residual streams (hyper-connections): mixer, then a feed-forward (dense or MoE; none
+    without an ``mlp``), each with a ``StreamConnection``. A serving layer: between two sub-layers, the update of the
+    streams, the next read and its norm are one kernel (``ops/stream.py::residual_streams``), across layers too, since the
+    output of a layer's last sub-layer stays pending."""
+
+    residual_streams = True       # ``residual`` is a ``ResidualStreams`` that still lacks ``pending``
+
+    def __init__(self, config, layer_number: int = 1, submodules: Optional[TransformerLayerSubmodules] = None):
+        super().__init__()
+        self.config, self.layer_number = config, layer_number
+        dev = getattr(config, "device", None)
+        self.input_layernorm = build_module(submodules.input_layernorm, config)
+        self.self_attention = build_module(submodules.self_attention, config, layer_number)
+        self.mixer_connection = StreamConnection(config.residual_streams, dev)
+        self.mlp = self.pre_mlp_layernorm = self.mlp_connection = None
+        if submodules.mlp is not None:
+            mlp_cls = getattr(submodules.mlp, "module", submodules.mlp)
+            self.is_moe = isinstance(mlp_cls, type) and issubclass(mlp_cls, MoELayer)
+            self.pre_mlp_layernorm = build_module(submodules.pre_mlp_layernorm, config)
+            self.mlp = build_module(submodules.mlp, config, layer_number) if self.is_moe else build_module(submodules.mlp, config)
+            self.mlp_connection = StreamConnection(config.residual_streams, dev)
+
+    def _enter(self, pending, streams: ResidualStreams, link: StreamConnection, norm):
+        """Let ``pending`` enter the streams; returns the input of the sub-layer behind ``link`` and the streams it leaves."""
+        old = streams.link
+        h, x = stream.residual_streams(streams.x, self.config.residual_streams, pending if old is not None else None,
+                                       None if old is None else old.mix, None if old is None else old.write, link.read,
+                                       norm.weight, norm.eps)
+        return h, ResidualStreams(x, link)
+
+    def forward(self, pending, residual: Optional[ResidualStreams], rotary, meta: AttnMeta):
+        if residual is None:                       # the embedding: every stream is equal to it
+            residual = ResidualStreams(pending)
+        h, residual = self._enter(pending, residual, self.mixer_connection, self.input_layernorm)
+        pending, _ = self.self_attention(h, rotary, meta)
+        aux = None
+        if self.mlp is not None:
+            h, residual = self._enter(pending, residual, self.mlp_connection, self.pre_mlp_layernorm)
+            pending, aux = self.mlp(h)
+        return pending, residual, aux if self.mlp is not None and self.is_moe else None
+
+
 def pipeline_layer_split(num_layers: int, pp: int, vpp: int = 1, offset=0) -> List[List[List[int]]]:
     """Layer ids of every (pp stage, virtual chunk). ``offset`` adds/removes layers per stage
     (list of pp values, or vpp lists of pp values), as the reference's ``LayerSetting`` does."""
@@ -241,9 +305,15 @@ class TransformerBlock(nn.Module):
         return len(self.run_order)
 
     def cache_shapes(self):
-        """``(kv heads, key size, value size)`` per layer run, or None for attention without per-layer cache shapes."""
+        """``(kv heads, key size, value size)`` per layer run (None: it caches no keys), or None for attention without
+        per-layer cache shapes."""
         shapes = [getattr(self.layers[at].self_attention, "cache_shape", None) for at in self.run_order]
         return [s() for s in shapes] if shapes and all(s is not None for s in shapes) else None
+
+    def state_shapes(self):
+        """Per layer run the recurrent state's shape (``KVCacheContext``) or None; None when no layer has one."""
+        shapes = [getattr(self.layers[at].self_attention, "state_shape", lambda: None)() for at in self.run_order]
+        return shapes if any(s is not None for s in shapes) else None
 
     def _setup_selective_recompute_and_offload(self, config):
         from ..recompute import ActivationOffloader, mark_recompute_modules
@@ -328,7 +398,13 @@ class TransformerBlock(nn.Module):
                 pending, residual, aux = run(pending, residual, rotary, meta)
             if aux is not None:
                 aux_total = aux if aux_total is None else aux_total + aux
-        if getattr(layer, "stream_in_residual", False):
+        if getattr(layer, "residual_streams", False):
+            norm, old = self.final_layernorm, residual.link
+            if norm is None:
+                raise NotImplementedError("residual streams stay on one pipeline stage")
+            out, _ = stream.residual_streams(residual.x, old.read.numel(), pending, old.mix, old.write, None, norm.weight,
+                                             norm.eps, keep=False)
+        elif getattr(layer, "stream_in_residual", False):
             norm = self.final_layernorm
             out = residual if norm is None else stream.norm_stream(residual, norm.weight, getattr(norm, "bias", None), norm.eps,
                                                                    hasattr(norm, "bias"))

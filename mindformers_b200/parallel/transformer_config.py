@@ -133,12 +133,26 @@ class TransformerConfig(ModelParallelConfig):
     # per layer, the index of the layer whose weights it uses (its own index: weights of its own); None: no sharing
     layer_sharing: Optional[List[int]] = None
     norm_placement: str = "input"           # "input": pre-norm; "output": x + scale * norm(sublayer(x)), fp32 stream
+    residual_streams: int = 0               # > 0: that many fp32 streams with learned reads, writes and mixing (pre-norm)
+    mixer: str = "attention"                # with residual_streams: "attention", "delta" (gated delta rule) or "parallel"
+                                            # (attention beside a gated delta rule, both on the same input)
+    parallel_scales: Optional[tuple] = None  # weights of the two outputs of a parallel mixer
+    delta_heads: int = 0                    # gated delta rule: value heads,
+    delta_kv_heads: int = 0                 #   query / key heads (each serves delta_heads / delta_kv_heads value heads),
+    delta_key_dim: int = 0                  #   sizes per head,
+    delta_value_dim: int = 0
+    delta_conv_taps: int = 4                #   taps of the short convolutions,
+    delta_decay: str = "head"               #   decays per "head" or per key "channel" (from a low-rank projection),
+    delta_decay_rank: int = 0
+    delta_gate: str = "silu"                #   gate of the read-out, "silu" or "sigmoid", and
+    delta_gate_rank: int = 0                #   its rank (0: one full projection)
     layer_scale: bool = False               # per-channel scale of every (normalised) sub-layer output
     ragged_attention: bool = False          # RaggedSelfAttention: whole, cut and mixed sequences in one paged call
     v_channels: Optional[int] = None        # value size per head (default: kv_channels)
     rotary_dim: Optional[int] = None        # rotated dimensions per head (default: kv_channels * rotary_percent)
     add_attention_output_bias: bool = False
     attention_chunk_size: int = 0           # > 0: a position sees its own chunk of that many positions only
+    attention_softcap: Optional[float] = None   # attention scores <- cap * tanh(scores / cap), fp32
     attention_sink: bool = False            # learned per-head term in the softmax denominator
     logit_softcap: Optional[float] = None   # logits <- cap * tanh(logits / cap), fp32
     # ---- init ----
@@ -213,7 +227,10 @@ class TransformerConfig(ModelParallelConfig):
     moe_pad_expert_input_to_capacity: bool = False
     moe_token_drop_policy: str = "probs"
     moe_permute_fusion: bool = True
-    moe_apply_probs_on_input: bool = False
+    moe_apply_probs_on_input: bool = False  # the routing weight multiplies the expert's input, not its output
+    moe_activation: str = "swiglu"          # "swiglu" or "clamped_glu": g sigmoid(alpha g) (u + 1), g and u clamped
+    moe_activation_limit: float = 7.0       #   at this limit (g from above only)
+    moe_activation_alpha: float = 1.702
     moe_token_dispatcher_type: str = "alltoall"
     use_allgather_dispatcher: bool = False
     kv_cache_dtype: Optional[str] = None    # "int8": paged KV cache in int8 with per-token, per-head scales
@@ -321,6 +338,10 @@ class TransformerConfig(ModelParallelConfig):
                 self.moe_aux_loss_coeff = float(self.aux_loss_factors[self.aux_loss_types.index("expert")])
         elif self.expert_model_parallel_size > 1:
             raise ValueError("expert_model_parallel_size > 1 needs num_moe_experts")
+        if self.mixer not in ("attention", "delta", "parallel") or self.delta_decay not in ("head", "channel") \
+                or self.delta_gate not in ("silu", "sigmoid") or self.moe_activation not in ("swiglu", "clamped_glu"):
+            raise ValueError(f"unknown mixer {self.mixer!r}, decay {self.delta_decay!r}, gate {self.delta_gate!r} or expert "
+                             f"activation {self.moe_activation!r}")
         if self.norm_placement not in ("input", "output"):
             raise ValueError(f"norm_placement must be 'input' or 'output', got {self.norm_placement!r}")
         for name in ("layer_overrides", "layer_sharing"):
