@@ -114,10 +114,11 @@ def main():
     ap.add_argument("--no-numerics-check", action="store_true")
     ap.add_argument("--tp", type=int, default=None)
     ap.add_argument("--recompute", type=int, default=0, help="recompute the activations of the first N layers in backward")
-    ap.add_argument("--config", default="llama8b", choices=["llama8b", "qwen3_moe", "qwen25_cp", "mefesun_serving"],
+    ap.add_argument("--config", default="llama8b", choices=["llama8b", "qwen3_moe", "qwen25_cp", "mefesun_serving", "kukupel_serving"],
                     help="llama8b: the headline (Llama-3.1-8B, TP2+SP x DP); qwen3_moe: Qwen3-30B-A3B, expert parallel = N, "
                          "micro batch 1; qwen25_cp: Qwen2.5-7B, one sequence of --seq-len tokens, context parallel = N; "
-                         "mefesun_serving: prefill and decode throughput of Mefesun beside Qwen3 at equal size (one GPU)")
+                         "mefesun_serving: prefill and decode throughput of Mefesun beside Qwen3 at equal size (one GPU); "
+                         "kukupel_serving: the same of Kukupel beside Qwen3-MoE")
     args = ap.parse_args()
     if args.config == "qwen3_moe" and args.model == "llama3_1_8b":
         args.model = "qwen3_30b_a3b"
@@ -128,12 +129,15 @@ def main():
         args.seqs_per_gpu = 1
     if args.impl == "reference":
         return reference_arm(args)
-    if args.config == "mefesun_serving":
+    if args.config in ("mefesun_serving", "kukupel_serving"):
         import torch
 
-        from benchmarks.bench_ragged_serving import main as serving
+        if args.config == "mefesun_serving":
+            from benchmarks.bench_ragged_serving import main as serving
+        else:
+            from benchmarks.bench_recurrent_serving import main as serving
         if args.gpus != 1:
-            raise SystemExit("--config mefesun_serving runs on one GPU")
+            raise SystemExit(f"--config {args.config} runs on one GPU")
         torch.cuda.set_device(0)
         sampler = ClockSampler(0)
         sampler.start()

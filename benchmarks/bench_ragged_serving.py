@@ -120,6 +120,7 @@ class Table:
         t_mem, t_math = nbytes / self.hbm * 1e3, flop / self.flops * 1e3
         self.rows.append({"kernel": what, "model": model, "ms": round(ms, 4),
                           "of_" + self.source: round(max(t_mem, t_math) / ms, 3), "bound": "hbm" if t_mem >= t_math else "tensor"})
+        return self.rows[-1]
 
 
 def step_meta(ctx, tables, batch, new, context):

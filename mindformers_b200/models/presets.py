@@ -59,6 +59,15 @@ PRESETS = {
                      mixer=dict(heads=8, kv_heads=2, dim=32, vdim=32, scale=32 ** -0.5, mask=dict(size=128),
                                 rot=dict(base=10000.0, dims=32, scaling=dict(factor=4.0, original=256, fast=32.0, slow=1.0))),
                      mlp=dict(kind="dense", ff=768)) for _ in range(2)]),
+    "tiny_kukupel": dict(
+        model_type="kukupel", vocab=1024, width=256, streams=4, norm=dict(eps=1e-6),
+        layers=[dict(type="parallel",
+                     mixer=dict(left=dict(heads=8, kv_heads=2, dim=32, vdim=32, scale=32 ** -0.5, softcap=30.0),
+                                right=dict(heads=4, kv_heads=2, dim=64, vdim=64, conv=4, decay_rank=32, gate_rank=32),
+                                left_scale=0.5, right_scale=0.5),
+                     mlp=dict(kind="moe", router=dict(experts=8, top=2), expert=dict(ff=256, limit=7.0))),
+                dict(type="delta", mixer=dict(heads=4, kv_heads=2, dim=64, vdim=64, conv=4),
+                     mlp=dict(kind="moe", router=dict(experts=8, top=2), expert=dict(ff=256, limit=7.0)))]),
     "tiny_llama": dict(
         model_type="llama", num_hidden_layers=2, hidden_size=256, num_attention_heads=4, num_key_value_heads=2,
         intermediate_size=688, vocab_size=1024, rms_norm_eps=1e-5, rope_theta=10000.0,

@@ -12,6 +12,7 @@ needs no host-side sizes. All index tensors are built on the device.
 """
 from __future__ import annotations
 
+import copy
 from typing import Optional, Tuple
 
 import torch
@@ -375,6 +376,9 @@ class MoELayer(nn.Module):
         if getattr(config, "enable_deredundency", False):
             kind = "deredundency"
         self.expert_tp = getattr(self.experts, "etp", 1) > 1
+        if config.moe_apply_probs_on_input:               # the dispatcher moves weighted copies, one expert each
+            config = copy.copy(config)
+            config.moe_router_topk = 1
         self.staged = kind != "alltoall" or self.expert_tp or bool(getattr(config, "use_pad_tokens", False))
         if self.staged:
             from .moe_dispatchers import StagedTokenDispatcher
@@ -416,14 +420,17 @@ class MoELayer(nn.Module):
         elif not self.staged and fused_comm.moe_local_enabled(self.config, hidden):
             out = fused_comm.moe_local(self, hidden, probs, ids)
         else:
-            x, plan, ctx = self.dispatcher.dispatch(hidden, ids)
-            if self.config.moe_apply_probs_on_input:
-                if ctx[0] != "local":
-                    raise NotImplementedError("routing weights on the experts' input need the fused exchange across ranks")
-                x[plan.dest] = (x[plan.dest].float() * probs.reshape(-1, 1)).to(x.dtype)
-                probs = torch.ones_like(probs)
+            T, k = ids.shape
+            if self.config.moe_apply_probs_on_input:      # every weighted copy is a token of its own
+                copies = (hidden.repeat_interleave(k, 0).float() * probs.reshape(-1, 1)).to(hidden.dtype)
+                x, plan, ctx = self.dispatcher.dispatch(copies, ids.reshape(-1, 1))
+                probs = torch.ones_like(probs.reshape(-1, 1))
+            else:
+                x, plan, ctx = self.dispatcher.dispatch(hidden, ids)
             y = self.experts(x, plan)
             out = self.dispatcher.combine(y, plan, ctx, probs.to(hidden.dtype))
+            if self.config.moe_apply_probs_on_input:
+                out = out.view(T, k, -1).float().sum(1).to(hidden.dtype)
         if with_shared and self.shared_experts is not None:
             out = out + self.shared_experts(hidden)
         return out, aux

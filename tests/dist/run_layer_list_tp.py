@@ -1,4 +1,4 @@
-"""Two tensor-parallel gloo ranks serve a Mefesun checkpoint in portions; every rank compares with the expected logits."""
+"""Two tensor-parallel gloo ranks serve a checkpoint in portions; every rank compares with the expected logits."""
 import os
 import sys
 

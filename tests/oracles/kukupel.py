@@ -200,6 +200,8 @@ def random_weights(cfg, seed=0, ranks=(12, 20), decay=(-3.0, 1.0)):
         H, G, D, DV = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
         for name, rows in (("q", G * D), ("k", G * D), ("v", H * DV)):
             w[p + name], w[p + name + ".conv"] = mat(rows, W, 1.5), vec((rows, m["conv"]), 0.2, 0.5)
+        # keys that resemble the queries, so that no read-out is a sum that nearly cancels before it is normalised
+        w[p + "k"], w[p + "k.conv"] = 0.4 * w[p + "k"] + w[p + "q"], w[p + "q.conv"] + 0.1 * w[p + "k.conv"]
         w[p + "b"], w[p + "A_log"], w[p + "norm"] = mat(H, W), vec(H, 0.0, 0.7), vec(DV, 1.0)
         if by_channel:
             w[p + "a1"], w[p + "a2"], w[p + "dt_bias"] = mat(ranks[0], W), mat(H * D, ranks[0]), vec(H * D, *decay)

@@ -259,7 +259,7 @@ def test_tensor_parallel_ranks_give_the_same_logits(tmp_path):
     path = cases.write_checkpoint(tmp_path / "m", cfg, w)
     toks = cases.tokens(50, cfg["vocab"], seed=1)
     torch.save(cases.expected(cfg, w, toks), tmp_path / "want.pt")
-    script = os.path.join(os.path.dirname(os.path.abspath(__file__)), "dist", "run_mefesun_tp.py")
+    script = os.path.join(os.path.dirname(os.path.abspath(__file__)), "dist", "run_layer_list_tp.py")
     res = subprocess.run([sys.executable, "-m", "torch.distributed.run", "--nnodes=1", "--nproc-per-node", "2", "--master-addr",
                           "127.0.0.1", "--master-port", "29671", script, path, str(tmp_path / "want.pt")],
                          capture_output=True, text=True, timeout=300)

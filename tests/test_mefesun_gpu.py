@@ -3,7 +3,6 @@ whole prompts, portions, decoding, mixed batches with pages and slots used again
 import pytest
 import torch
 
-from mindformers_b200.inference.paged_attention import KVCacheContext
 from mindformers_b200.inference import ragged_attention as ragged
 from mindformers_b200.inference.ragged_attention import ragged_attention
 from mindformers_b200.ops import _lib, stream
@@ -11,6 +10,7 @@ from mindformers_b200.serving import SamplingParams, ServingEngine
 from mindformers_b200.serving.trace import build_engine
 
 from oracles import cases, mefesun
+from oracles.paged import attention_case
 
 pytestmark = pytest.mark.gpu
 DEV = "cuda"
@@ -140,50 +140,6 @@ def test_qkv_rope_cache(dtype, H, G, D, DV, rot, interleaved):
             assert rel(kf[slots[t]], wk[t]) < tol(dtype, 5e-3) and rel(vf[slots[t]], wv[t]) < tol(dtype)
     untouched = [s for s in range(blocks * bs) if s not in slots.tolist()]
     assert bool((kf[untouched] == 7).all()) and bool((vf[untouched] == 7).all())
-
-
-def attention_case(dtype, H, G, D, DV, bs, chunk, lens, news, seed=0, sink_scale=1.0, spots=()):
-    """A paged cache with shuffled pages and the step's queries. ``spots``: (sequence, query position, key position) whose
-    score is made to stand out (it decides the row where it is visible, and nothing where it is hidden)."""
-    B = len(lens)
-    g = torch.Generator().manual_seed(seed)
-    per = [-(-n // bs) for n in lens]
-    width = max(per) + 2
-    total = sum(per) + 3
-    perm = torch.randperm(total, generator=g).tolist()
-    ctx = KVCacheContext(1, total, bs, 0, 0, dtype, DEV, layer_shapes=[(G, D, DV)])
-    table = torch.full((B, width), -1, dtype=torch.int32)
-    scale = 1.3 * D ** -0.5
-    qs, ks, vs = [], [], []
-    for b in range(B):
-        for i in range(per[b]):
-            table[b, i] = perm.pop()
-        k = torch.randn(lens[b], G, D, generator=g)
-        v = torch.randn(lens[b], G, DV, generator=g)
-        q = torch.randn(news[b], H, D, generator=g)
-        for sb, qp, kp in spots:
-            if sb == b:
-                r = qp - (lens[b] - news[b])
-                k[kp] = q[r].view(G, H // G, D).mean(1) * 6
-        qs.append(q.to(dtype)); ks.append(k.to(dtype)); vs.append(v.to(dtype))
-    stale = torch.randn(ctx.key_cache[0].shape, generator=g).to(dtype)           # pages hold other requests' old rows
-    ctx.key_cache[0].copy_(stale * 5)
-    ctx.value_cache[0].copy_(torch.randn(ctx.value_cache[0].shape, generator=g).to(dtype) * 5)
-    for b in range(B):
-        for t in range(lens[b]):
-            at = (int(table[b, t // bs]), t % bs)
-            ctx.key_cache[0][at] = ks[b][t].to(DEV)
-            ctx.value_cache[0][at] = vs[b][t].to(DEV)
-    sink = torch.randn(H, generator=g) * sink_scale + 1
-    want = []
-    for b in range(B):
-        n, m = lens[b], news[b]
-        reps = H // G
-        s = torch.einsum("qhd,khd->hqk", qs[b].double(), ks[b].double().repeat_interleave(reps, 1)) * scale
-        mask = mefesun.chunk_mask(n, chunk if chunk else n)[n - m:]
-        p = mefesun.softmax_with_sink(s, mask, sink.double())
-        want.append(torch.einsum("hqk,khd->qhd", p, vs[b].double().repeat_interleave(reps, 1)))
-    return ctx, table, qs, sink, scale, torch.cat(want).reshape(sum(news), H * DV)
 
 
 ATTENTION = [(4, 2, 64, 64), (8, 2, 128, 128), (6, 2, 40, 24), (5, 5, 128, 64), (3, 1, 64, 128), (20, 1, 24, 40), (3, 1, 20, 36),
