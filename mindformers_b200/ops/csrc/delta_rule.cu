@@ -21,6 +21,8 @@
 // S are independent: a CTA takes a range of the columns of one head of one sequence, L lanes share a column, and a thread
 // keeps R rows of C columns in registers for the whole portion, as pairs for the packed fp32 instructions. With
 // a = (g S)^T k and b = (g S)^T q taken in one pass, o = b + u (k . q) needs no second pass over S.
+#include <type_traits>
+
 #include "common.cuh"
 
 namespace mfb {
@@ -120,28 +122,94 @@ __device__ __forceinline__ void conv_silu(const Args& p, const T* ring, long lon
   for (int i = 0; i < VEC; ++i) acc[i] = siluf(acc[i]);
 }
 
+// The same for four neighbouring channels of a run of rows and at most four taps, in registers: the run's inputs are fetched
+// ahead, a window holds the three before the current one, and the weights stay.
+template <typename T>
+struct ConvRun {
+  typedef typename std::conditional<sizeof(T) == 2, uint2, float4>::type Raw;
+  Raw x[kRun];
+  float w[4][4], before[3][4];          // w[d]: weight of the input d rows back
+  __device__ __forceinline__ static void unpack(const Raw& r, float (&v)[4]) { ldv<4>(reinterpret_cast<const T*>(&r), v); }
+  __device__ __forceinline__ void open(const Args& p, int r0, int c, int C) {
+#pragma unroll
+    for (int i = 0; i < kRun; ++i)
+      if (r0 + i < p.T) x[i] = *reinterpret_cast<const Raw*>(reinterpret_cast<const T*>(p.x) + (long long)(r0 + i) * p.ld + c);
+#pragma unroll
+    for (int d = 0; d < 4; ++d) {
+      if (d < p.taps) ldv<4>(p.conv + (long long)(p.taps - 1 - d) * C + c, w[d]);
+      else { w[d][0] = w[d][1] = w[d][2] = w[d][3] = 0.f; }
+    }
+  }
+  // the inputs before row r (first of the run or of its sequence)
+  __device__ __forceinline__ void rewind(const Args& p, const T* ring, long long r, int local, int pos, int c, int C) {
+#pragma unroll
+    for (int d = 1; d < 4; ++d) {
+      if (d < p.taps && d <= pos) {
+        if (d <= local) ldv<4>(reinterpret_cast<const T*>(p.x) + (r - d) * p.ld + c, before[d - 1]);
+        else ldv<4>(ring + (long long)((pos - d) % p.taps) * C + c, before[d - 1]);
+      } else {
+        before[d - 1][0] = before[d - 1][1] = before[d - 1][2] = before[d - 1][3] = 0.f;
+      }
+    }
+  }
+  __device__ __forceinline__ void next(const Raw& raw, float (&out)[4]) {
+    float cur[4];
+    unpack(raw, cur);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      float a = fmaf(before[2][i], w[3][i], before[1][i] * w[2][i]);
+      a = fmaf(cur[i], w[0][i], fmaf(before[0][i], w[1][i], a));
+      before[2][i] = before[1][i]; before[1][i] = before[0][i]; before[0][i] = cur[i];
+      out[i] = siluf(a);
+    }
+  }
+};
+
 // One warp per unit and run of rows. Units: G (q and k of a key head), H (v of a head), then H (decays of a head's channels)
-// or ceil(H / 32) (decays of 32 heads); the last kind also makes beta.
-template <typename T, int VEC, int NJ>
+// or ceil(H / 32) (decays of 32 heads); the last kind also makes beta. FAST: VEC 4, heads up to 128, at most four taps.
+template <typename T, int VEC, int NJ, bool FAST>
 __global__ void __launch_bounds__(128) prepare_kernel(const Args p, int units) {
   const int unit = blockIdx.y * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   if (unit >= units) return;
   const int r0 = blockIdx.x * kRun, r1 = min(r0 + kRun, p.T);
   const int C = 2 * p.G * p.D + p.H * p.DV;
   int b = sequence_of(p.cu_q, p.B, r0);
-  for (int r = r0; r < r1; ++r) {
+  const bool is_qk = unit < p.G, is_v = !is_qk && unit < p.G + p.H;
+  ConvRun<T> ca, cb;
+  const int h = unit - p.G, dl = lane * 4;
+  const int c0 = is_qk ? unit * p.D + dl : 2 * p.G * p.D + h * p.DV + dl, c1 = (p.G + unit) * p.D + dl;
+  const bool on = is_qk ? dl < p.D : dl < p.DV;
+  if constexpr (FAST) {
+    if ((is_qk || is_v) && on) ca.open(p, r0, c0, C);
+    if (is_qk && on) cb.open(p, r0, c1, C);
+  }
+#pragma unroll
+  for (int ri = 0; ri < kRun; ++ri) {
+    const int r = r0 + ri;
+    if (r >= r1) break;
     while (r >= p.cu_q[b + 1]) ++b;
     const int local = r - p.cu_q[b], pos = p.context_lens[b] - (p.cu_q[b + 1] - r);
     const T* ring = reinterpret_cast<const T*>(p.ring) + (long long)b * p.taps * C;
-    if (unit < p.G) {
+    if constexpr (FAST) {
+      if ((is_qk || is_v) && on && (ri == 0 || local == 0)) {
+        ca.rewind(p, ring, r, local, pos, c0, C);
+        if (is_qk) cb.rewind(p, ring, r, local, pos, c1, C);
+      }
+    }
+    if (is_qk) {
       float q[NJ][VEC], k[NJ][VEC];
       float qq = 0.f, kk = 0.f, qk = 0.f;
 #pragma unroll
       for (int j = 0; j < NJ; ++j) {
         const int d = (lane + 32 * j) * VEC;
         if (d < p.D) {
-          conv_silu<T, VEC>(p, ring, r, local, pos, unit * p.D + d, C, q[j]);
-          conv_silu<T, VEC>(p, ring, r, local, pos, (p.G + unit) * p.D + d, C, k[j]);
+          if constexpr (FAST) {
+            ca.next(ca.x[ri], q[j]);
+            cb.next(cb.x[ri], k[j]);
+          } else {
+            conv_silu<T, VEC>(p, ring, r, local, pos, unit * p.D + d, C, q[j]);
+            conv_silu<T, VEC>(p, ring, r, local, pos, (p.G + unit) * p.D + d, C, k[j]);
+          }
 #pragma unroll
           for (int i = 0; i < VEC; ++i) {
             qq = fmaf(q[j][i], q[j][i], qq);
@@ -165,14 +233,14 @@ __global__ void __launch_bounds__(128) prepare_kernel(const Args p, int units) {
       }
       const int reps = p.H / p.G;
       for (int i = lane; i < reps; i += 32) p.beta[((long long)r * p.H + unit * reps + i) * 2 + 1] = qk * rq * rk;
-    } else if (unit < p.G + p.H) {
-      const int h = unit - p.G;
+    } else if (is_v) {
 #pragma unroll
       for (int j = 0; j < NJ; ++j) {
         const int d = (lane + 32 * j) * VEC;
         if (d < p.DV) {
           float v[VEC];
-          conv_silu<T, VEC>(p, ring, r, local, pos, 2 * p.G * p.D + h * p.DV + d, C, v);
+          if constexpr (FAST) ca.next(ca.x[ri], v);
+          else conv_silu<T, VEC>(p, ring, r, local, pos, 2 * p.G * p.D + h * p.DV + d, C, v);
           stv<VEC>(p.v + ((long long)r * p.H + h) * p.DV + d, v);
         }
       }
@@ -188,10 +256,10 @@ __global__ void __launch_bounds__(128) prepare_kernel(const Args p, int units) {
         }
         if (lane == 0) p.beta[((long long)r * p.H + i0) * 2] = sigmoidf(ld(bb + i0));
       } else {
-        const int h = i0 * 32 + lane;
-        if (h < p.H) {
-          p.g[(long long)r * p.H + h] = decayf(p.a_log[h], ld(a + h) + p.dt_bias[h]);
-          p.beta[((long long)r * p.H + h) * 2] = sigmoidf(ld(bb + h));
+        const int hh = i0 * 32 + lane;
+        if (hh < p.H) {
+          p.g[(long long)r * p.H + hh] = decayf(p.a_log[hh], ld(a + hh) + p.dt_bias[hh]);
+          p.beta[((long long)r * p.H + hh) * 2] = sigmoidf(ld(bb + hh));
         }
       }
     }
@@ -217,35 +285,58 @@ __device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
   asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
   return d;
 }
-__device__ __forceinline__ void cp_async(void* dst, const void* src, int bytes16) {
-  const uint32_t d = smem_u32(dst);
-  if (bytes16) asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(d), "l"(src) : "memory");
-  else asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(d), "l"(src) : "memory");
-}
-__device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-template <int N> __device__ __forceinline__ void cp_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+constexpr int kComputeThreads = 128;
+constexpr int kFeedWarps = 2;          // warps that load and prepare the vectors of the pairs ahead
+constexpr int kScanThreads = kComputeThreads + 32 * kFeedWarps;
+constexpr int kPairs = 4;              // pairs of tokens per stage (two stages)
+constexpr int kTile = 2 * kPairs;
 
-constexpr int kScanThreads = 128;
-constexpr int kTile = 16;              // tokens staged at a time (two buffers)
-
-template <int R, int L, int C>
+// vectors of a pair of tokens in a stage: with decays per channel k1 g1, q1 g1, k2 g1 g2, q2 g1 g2, k1 g2, k2, g1 g2; with one
+// decay k1, q1, k2, q2
+template <int R, int L, int C, bool CH>
 struct ScanShape {
   static constexpr int DP = R * L;                          // padded key size
-  static constexpr int kCols = kScanThreads / L * C;        // columns of a CTA
+  static constexpr int kGroups = kComputeThreads / L;
+  static constexpr int kCols = kGroups * C;                 // columns of a CTA
+  static constexpr int kVecs = CH ? 7 : 4;
+  static constexpr int kStage = kPairs * (kVecs * DP + 2 * kCols + 8);      // floats; 8: beta1, q1 k1, beta2, q2 k2, c, q2 k1, g1, g2
 };
 
-template <int R, int L, int C, bool CH>
-constexpr int scan_smem() {
-  using S = ScanShape<R, L, C>;
-  return 2 * kTile * (2 * S::DP + (CH ? S::DP : 4) + S::kCols + 4) * (int)sizeof(float);
+// sum over the L lanes of a column group of N values per lane; lane l is left with values l, l + L, ... (N / L of them), or,
+// where N < L, with value l N / L: halves are exchanged as long as a lane holds more than one
+template <int N, int L>
+__device__ __forceinline__ void reduce_scatter(float (&v)[N], int ln) {
+  int n = N;
+#pragma unroll
+  for (int d = L / 2; d > 0; d >>= 1) {
+    if (n > 1) {
+      n /= 2;
+      const bool up = ln & d;
+#pragma unroll
+      for (int i = 0; i < N / 2; ++i) {
+        if (i < n) {
+          const float keep = up ? v[i + n] : v[i], give = up ? v[i] : v[i + n];
+          v[i] = keep + __shfl_xor_sync(0xffffffffu, give, d);
+        }
+      }
+    } else {
+      v[0] += __shfl_xor_sync(0xffffffffu, v[0], d);
+    }
+  }
 }
 
-// R rows of C columns per thread, L lanes per column; CH: decays per key channel. vec: D, DV and the scratch rows allow
-// 16-byte copies.
+// Two tokens at a time. With S the state before them, A1 = S^T (g1 k1), A2 = S^T (g1 g2 k2) and B1, B2 the same of q:
+//   u1 = beta1 (v1 - A1)                 o1 = B1 + (q1 . k1) u1
+//   u2 = beta2 (v2 - A2 - c u1)          o2 = B2 + (q2 . g2 k1) u1 + (q2 . k2) u2        c = k2 . g2 k1
+//   S <- g1 g2 S + (g2 k1) u1^T + k2 u2^T
+// which is the same recurrence with seven instead of eight operations per element and pair, and one instead of two points at
+// which the lanes of a column wait for one another. R rows of C columns per thread, L lanes per column; CH: decays per key
+// channel. vec: D, DV and the scratch rows allow 16-byte accesses. While the compute warps work on one stage of pairs, the
+// feed warps fetch and prepare the next.
 template <typename T, int R, int L, int C, bool CH>
-__global__ void __launch_bounds__(kScanThreads) scan_kernel(const Args p, int vec) {
-  using S = ScanShape<R, L, C>;
-  constexpr int DP = S::DP, COLS = S::kCols, GW = CH ? DP : 4, GROUPS = kScanThreads / L;
+__global__ void __launch_bounds__(kScanThreads, 2) scan_kernel(const Args p, int vec) {
+  using S = ScanShape<R, L, C, CH>;
+  constexpr int DP = S::DP, COLS = S::kCols, GROUPS = S::kGroups, VECS = S::kVecs;
   const int b = blockIdx.z, h = blockIdx.y, col0 = blockIdx.x * COLS;
   const int r0 = p.cu_q[b], n = p.cu_q[b + 1] - r0;
   if (n <= 0) return;
@@ -261,44 +352,111 @@ __global__ void __launch_bounds__(kScanThreads) scan_kernel(const Args p, int ve
       for (int c = threadIdx.x; c < ch; c += kScanThreads) ring[(long long)(pos % p.taps) * ch + c] = src[c];
     }
   }
-  extern __shared__ __align__(16) float sh[];
-  float* s_qk = sh;                                  // [2][kTile][q DP | k DP]
-  float* s_g = s_qk + 2 * kTile * 2 * DP;            // [2][kTile][GW]
-  float* s_v = s_g + 2 * kTile * GW;                 // [2][kTile][COLS]
-  float* s_b = s_v + 2 * kTile * COLS;               // [2][kTile][4]: beta, q . k
-  for (int i = threadIdx.x; i < 2 * kTile * (2 * DP + GW); i += kScanThreads) sh[i] = 0.f;      // the padding stays zero
-  __syncthreads();
-  const int ln = threadIdx.x % L, grp = threadIdx.x / L;
+  extern __shared__ __align__(16) float sh[];        // [2][kStage]: vectors of the pairs, v, scalars
+  const int lane = threadIdx.x & 31;
+  const int tiles = (n + kTile - 1) / kTile;
 
-  const int w = vec ? 4 : 1;                         // floats per copy
-  auto stage = [&](int tile) {
-    const int buf = tile & 1, t0 = tile * kTile, m = min(kTile, n - t0);
-    const int nq = 2 * D / w;
-    for (int i = threadIdx.x; i < m * nq; i += kScanThreads) {
-      const int t = i / nq, e = (i - t * nq) * w;
-      const int at = e < D ? e : DP + e - D;
-      cp_async(s_qk + (buf * kTile + t) * 2 * DP + at, p.qk + ((long long)(r0 + t0 + t) * p.G + kvh) * 2 * D + e, vec);
-    }
-    if (CH) {
-      const int ng = D / w;
-      for (int i = threadIdx.x; i < m * ng; i += kScanThreads) {
-        const int t = i / ng, e = (i - t * ng) * w;
-        cp_async(s_g + (buf * kTile + t) * GW + e, p.g + ((long long)(r0 + t0 + t) * H + h) * D + e, vec);
+  if (threadIdx.x >= kComputeThreads) {
+    // ------------------------------ feed ------------------------------
+    constexpr int NJ = (DP + 127) / 128, PW = kPairs / kFeedWarps, VN = (2 * COLS + 127) / 128;
+    const int fw = (threadIdx.x - kComputeThreads) >> 5;
+    float k[PW][2][NJ][4], q[PW][2][NJ][4], g[PW][2][CH ? NJ : 1][4], v[PW][VN][4];
+    float2 sc[PW];                                   // lane 0: beta, q k of token 1; lane 1: of token 2
+    float gs[PW];                                    // and its decay (without CH)
+    auto four = [&](const float* src, int at, int size, float fill, float (&o)[4]) {
+      if (at + 3 < size && vec) { ldv<4>(src + at, o); return; }
+#pragma unroll
+      for (int e = 0; e < 4; ++e) o[e] = at + e < size ? src[at + e] : fill;
+    };
+    auto fetch = [&](int tile) {
+#pragma unroll
+      for (int w = 0; w < PW; ++w) {
+        const int t0 = tile * kTile + 2 * (fw + w * kFeedWarps);
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          const bool there = t0 + e < n;             // an odd last token is paired with one that changes nothing
+          const long long row = r0 + (there ? t0 + e : n - 1);
+          const float* src = p.qk + (row * p.G + kvh) * 2 * D;
+#pragma unroll
+          for (int j = 0; j < NJ; ++j) {
+            const int d = (lane + 32 * j) * 4;
+            four(src, d, there ? D : 0, 0.f, q[w][e][j]);
+            four(src + D, d, there ? D : 0, 0.f, k[w][e][j]);
+            if constexpr (CH) four(p.g + (row * H + h) * D, d, there ? D : 0, 1.f, g[w][e][j]);
+          }
+        }
+#pragma unroll
+        for (int i = 0; i < VN; ++i) {
+          const int at = (lane + 32 * i) * 4, e = at / COLS, c = at % COLS;
+          if (e < 2) four(p.v + ((long long)(r0 + min(t0 + e, n - 1)) * H + h) * DV, col0 + c, DV, 0.f, v[w][i]);
+        }
+        if (lane < 2) {
+          const bool there = t0 + lane < n;
+          const long long at = (long long)(r0 + (there ? t0 + lane : n - 1)) * H + h;
+          sc[w] = there ? *reinterpret_cast<const float2*>(p.beta + at * 2) : make_float2(0.f, 0.f);
+          gs[w] = !CH && there ? p.g[at] : 1.f;
+        }
       }
-    } else {
-      for (int t = threadIdx.x; t < m; t += kScanThreads)
-        cp_async(s_g + (buf * kTile + t) * GW, p.g + (long long)(r0 + t0 + t) * H + h, 0);
+    };
+    auto put = [&](int tile) {
+      float* stage = sh + (tile & 1) * S::kStage;
+#pragma unroll
+      for (int w = 0; w < PW; ++w) {
+        const int j2 = fw + w * kFeedWarps;
+        float* vecs = stage + j2 * VECS * DP;
+        float kk = 0.f, qk = 0.f;
+#pragma unroll
+        for (int j = 0; j < NJ; ++j) {
+          const int d = (lane + 32 * j) * 4;
+          if (d < DP) {
+            float o[7][4];
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+              const float k1 = k[w][0][j][e], q1 = q[w][0][j][e], k2 = k[w][1][j][e], q2 = q[w][1][j][e];
+              float w1 = k1;
+              if constexpr (CH) {
+                const float g1 = g[w][0][j][e], g2 = g[w][1][j][e], gg = g1 * g2;
+                w1 = k1 * g2;
+                o[0][e] = k1 * g1; o[1][e] = q1 * g1; o[2][e] = k2 * gg; o[3][e] = q2 * gg;
+                o[4][e] = w1; o[5][e] = k2; o[6][e] = gg;
+              } else {
+                o[0][e] = k1; o[1][e] = q1; o[2][e] = k2; o[3][e] = q2;
+              }
+              kk = fmaf(k2, w1, kk);
+              qk = fmaf(q2, w1, qk);
+            }
+#pragma unroll
+            for (int x = 0; x < VECS; ++x) stv<4>(vecs + x * DP + d, o[x]);
+          }
+        }
+        kk = warp_sum(kk);
+        qk = warp_sum(qk);
+        float* vs = stage + kPairs * VECS * DP + j2 * 2 * COLS;
+#pragma unroll
+        for (int i = 0; i < VN; ++i) {
+          const int at = (lane + 32 * i) * 4;
+          if (at < 2 * COLS) stv<4>(vs + at, v[w][i]);
+        }
+        float* ss = stage + kPairs * (VECS * DP + 2 * COLS) + j2 * 8;
+        const float g2 = __shfl_sync(0xffffffffu, gs[w], 1);
+        if (lane < 2) { ss[2 * lane] = sc[w].x; ss[2 * lane + 1] = sc[w].y; ss[6 + lane] = gs[w]; }
+        if (lane == 0) { ss[4] = CH ? kk : kk * g2; ss[5] = CH ? qk : qk * g2; }
+      }
+    };
+    fetch(0);
+    put(0);
+    if (tiles > 1) fetch(1);
+    __syncthreads();
+    for (int tile = 0; tile < tiles; ++tile) {
+      if (tile + 1 < tiles) put(tile + 1);
+      if (tile + 2 < tiles) fetch(tile + 2);
+      __syncthreads();
     }
-    const int left = min(COLS, DV - col0), nv = left / w;
-    for (int i = threadIdx.x; i < m * nv; i += kScanThreads) {
-      const int t = i / nv, e = (i - t * nv) * w;
-      cp_async(s_v + (buf * kTile + t) * COLS + e, p.v + ((long long)(r0 + t0 + t) * H + h) * DV + col0 + e, vec);
-    }
-    for (int i = threadIdx.x; i < 2 * m; i += kScanThreads)
-      cp_async(s_b + (buf * kTile + (i >> 1)) * 4 + (i & 1), p.beta + ((long long)(r0 + t0 + (i >> 1)) * H + h) * 2 + (i & 1), 0);
-    cp_commit();
-  };
+    return;
+  }
 
+  // ------------------------------ compute ------------------------------
+  const int ln = threadIdx.x % L, grp = threadIdx.x / L;
   // rows of a thread: (i * L + ln) * 4 .. + 3 for i < R / 4, as pairs
   uint64_t s[C][R / 2];
   float* state = p.state + ((long long)b * H + h) * D * DV;
@@ -316,68 +474,93 @@ __global__ void __launch_bounds__(kScanThreads) scan_kernel(const Args p, int ve
       s[c][i] = pack2(v[0], v[1]);
     }
   }
-  const int tiles = (n + kTile - 1) / kTile;
-  stage(0);
+  // after the exchange of partial sums a lane computes one column (C <= L), or C / L of them
+  constexpr int OWN = C > L ? C / L : 1;
+  __syncthreads();
   for (int tile = 0; tile < tiles; ++tile) {
-    if (tile + 1 < tiles) {
-      stage(tile + 1);
-      cp_wait<1>();
-    } else {
-      cp_wait<0>();
-    }
-    __syncthreads();
-    const int buf = tile & 1, m = min(kTile, n - tile * kTile);
+    const float* stage = sh + (tile & 1) * S::kStage;
+    const int m = min(kTile, n - tile * kTile);
     float* orow = p.o + ((long long)(r0 + tile * kTile) * H + h) * DV;
-    for (int t = 0; t < m; ++t) {
-      const float* qp = s_qk + (buf * kTile + t) * 2 * DP + ln * 4;
-      const float* kp = qp + DP;
-      const float* gp = s_g + (buf * kTile + t) * GW;
-      const float* vp = s_v + (buf * kTile + t) * COLS;
-      const float beta = s_b[(buf * kTile + t) * 4], qk = s_b[(buf * kTile + t) * 4 + 1];
-      uint64_t a2[C], b2[C];
+    for (int j = 0; 2 * j < m; ++j) {
+      const float* vec1 = stage + j * VECS * DP + ln * 4;
+      uint64_t acc[C][4];
 #pragma unroll
-      for (int c = 0; c < C; ++c) a2[c] = b2[c] = 0;
-      uint64_t k2[R / 2];
+      for (int c = 0; c < C; ++c)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) acc[c][e] = 0;
 #pragma unroll
       for (int i = 0; i < R / 4; ++i) {
-        const ulonglong2 q4 = *reinterpret_cast<const ulonglong2*>(qp + i * L * 4);
-        const ulonglong2 k4 = *reinterpret_cast<const ulonglong2*>(kp + i * L * 4);
-        k2[2 * i] = k4.x; k2[2 * i + 1] = k4.y;
-        if (CH) {
-          const ulonglong2 g4 = *reinterpret_cast<const ulonglong2*>(gp + ln * 4 + i * L * 4);
+        const ulonglong2 k1 = *reinterpret_cast<const ulonglong2*>(vec1 + i * L * 4);
+        const ulonglong2 q1 = *reinterpret_cast<const ulonglong2*>(vec1 + DP + i * L * 4);
+        const ulonglong2 k2 = *reinterpret_cast<const ulonglong2*>(vec1 + 2 * DP + i * L * 4);
+        const ulonglong2 q2 = *reinterpret_cast<const ulonglong2*>(vec1 + 3 * DP + i * L * 4);
 #pragma unroll
-          for (int c = 0; c < C; ++c) {
-            s[c][2 * i] = mul2(s[c][2 * i], g4.x);
-            s[c][2 * i + 1] = mul2(s[c][2 * i + 1], g4.y);
-          }
+        for (int c = 0; c < C; ++c) {
+          acc[c][0] = fma2(s[c][2 * i], k1.x, acc[c][0]);
+          acc[c][1] = fma2(s[c][2 * i], q1.x, acc[c][1]);
+          acc[c][2] = fma2(s[c][2 * i], k2.x, acc[c][2]);
+          acc[c][3] = fma2(s[c][2 * i], q2.x, acc[c][3]);
         }
 #pragma unroll
         for (int c = 0; c < C; ++c) {
-          a2[c] = fma2(s[c][2 * i], k4.x, a2[c]);
-          b2[c] = fma2(s[c][2 * i], q4.x, b2[c]);
-          a2[c] = fma2(s[c][2 * i + 1], k4.y, a2[c]);
-          b2[c] = fma2(s[c][2 * i + 1], q4.y, b2[c]);
+          acc[c][0] = fma2(s[c][2 * i + 1], k1.y, acc[c][0]);
+          acc[c][1] = fma2(s[c][2 * i + 1], q1.y, acc[c][1]);
+          acc[c][2] = fma2(s[c][2 * i + 1], k2.y, acc[c][2]);
+          acc[c][3] = fma2(s[c][2 * i + 1], q2.y, acc[c][3]);
         }
       }
-      float ga = 1.f;
-      if (!CH) ga = gp[0];
-      const uint64_t g2 = pack2(ga, ga);
+      const float* ss = stage + kPairs * (VECS * DP + 2 * COLS) + j * 8;
+      const float4 bb = *reinterpret_cast<const float4*>(ss), cg = *reinterpret_cast<const float4*>(ss + 4);
+      const float g1 = CH ? 1.f : cg.z, g12 = CH ? 1.f : cg.z * cg.w;
+      float sums[4][C];
+#pragma unroll
+      for (int c = 0; c < C; ++c)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          float x, y;
+          unpack2(acc[c][e], x, y);
+          sums[e][c] = x + y;
+        }
+#pragma unroll
+      for (int e = 0; e < 4; ++e) reduce_scatter<C, L>(sums[e], ln);
+      // this lane's column(s)
+      float u1[OWN], u2[OWN];
+#pragma unroll
+      for (int o = 0; o < OWN; ++o) {
+        const int c = C > L ? ln * OWN + o : (ln * C) / L;
+        const int lc = grp + GROUPS * c, col = col0 + lc;
+        const float* vp = stage + kPairs * VECS * DP + j * 2 * COLS + lc;
+        u1[o] = bb.x * (vp[0] - g1 * sums[0][o]);
+        u2[o] = bb.z * (vp[COLS] - g12 * sums[2][o] - cg.x * u1[o]);
+        if (col < DV && (C >= L || ln % (L / C) == 0)) {
+          orow[(long long)(2 * j) * H * DV + col] = fmaf(u1[o], bb.y, g1 * sums[1][o]);
+          if (2 * j + 1 < m) orow[(long long)(2 * j + 1) * H * DV + col] = fmaf(u2[o], bb.w, fmaf(cg.y, u1[o], g12 * sums[3][o]));
+        }
+        if (!CH) u1[o] *= cg.w;
+      }
+      const uint64_t g2 = pack2(g12, g12);
+      const float* w1p = CH ? vec1 + 4 * DP : vec1;
+      const float* w2p = CH ? vec1 + 5 * DP : vec1 + 2 * DP;
+      const float* gp = vec1 + 6 * DP;
+      uint64_t x1[C], x2[C];
 #pragma unroll
       for (int c = 0; c < C; ++c) {
-        float x, y, a, bq;
-        unpack2(a2[c], x, y); a = x + y;
-        unpack2(b2[c], x, y); bq = x + y;
+        const int src = (lane & ~(L - 1)) + (C > L ? c / OWN : c * (L / C));
+        const float y1 = __shfl_sync(0xffffffffu, u1[C > L ? c % OWN : 0], src), y2 = __shfl_sync(0xffffffffu, u2[C > L ? c % OWN : 0], src);
+        x1[c] = pack2(y1, y1);
+        x2[c] = pack2(y2, y2);
+      }
 #pragma unroll
-        for (int d = L / 2; d > 0; d >>= 1) {
-          a += __shfl_xor_sync(0xffffffffu, a, d);
-          bq += __shfl_xor_sync(0xffffffffu, bq, d);
+      for (int i = 0; i < R / 4; ++i) {
+        const ulonglong2 w1 = *reinterpret_cast<const ulonglong2*>(w1p + i * L * 4);
+        const ulonglong2 w2 = *reinterpret_cast<const ulonglong2*>(w2p + i * L * 4);
+        ulonglong2 g4;
+        if (CH) g4 = *reinterpret_cast<const ulonglong2*>(gp + i * L * 4);
+#pragma unroll
+        for (int c = 0; c < C; ++c) {
+          s[c][2 * i] = fma2(w2.x, x2[c], fma2(w1.x, x1[c], mul2(s[c][2 * i], CH ? g4.x : g2)));
+          s[c][2 * i + 1] = fma2(w2.y, x2[c], fma2(w1.y, x1[c], mul2(s[c][2 * i + 1], CH ? g4.y : g2)));
         }
-        const float u = beta * (vp[grp + GROUPS * c] - ga * a);
-        const int col = col0 + grp + GROUPS * c;
-        if (ln == c % L && col < DV) orow[(long long)t * H * DV + col] = fmaf(u, qk, ga * bq);
-        const uint64_t u2 = pack2(u, u);
-#pragma unroll
-        for (int i = 0; i < R / 2; ++i) s[c][i] = fma2(k2[i], u2, CH ? s[c][i] : mul2(s[c][i], g2));
       }
     }
     __syncthreads();
@@ -436,19 +619,53 @@ __global__ void __launch_bounds__(128) gate_out_kernel(const Args p) {
 }
 
 // ---- decode: one row per slot, one CTA per head ---------------------------------------------------------------------------------
-// Threads form TY row groups of TX lanes; a lane holds four neighbouring columns of NR rows. D * DV <= 4 NT NR.
-template <typename T, int NT, int NR>
-__global__ void __launch_bounds__(NT) delta_decode_kernel(const Args p, int tx_log2) {
-  const int h = blockIdx.x, b = blockIdx.y;
+// Threads form TY row groups of TX lanes; a lane holds four neighbouring columns of NR rows. D * DV <= 4 NT NR. FAST (at most
+// four taps, 2 D + DV <= NI NT, D and DV <= NT): every input is on its way before the first one is used, the state last, so that
+// a CTA waits for memory once.
+template <typename T, int NT, int NR, int NI, bool FAST>
+__global__ void __launch_bounds__(NT, NR > 8 && NT > 256 ? 1 : 2) delta_decode_kernel(const Args p, int tx_log2) {
+  const int h = blockIdx.x, b = blockIdx.y, tid = threadIdx.x;
+  const int slot = p.slots[b], pos = p.context_lens[b] - 1;
   const int D = p.D, DV = p.DV, H = p.H, reps = H / p.G, kvh = h / reps;
   T* out = reinterpret_cast<T*>(p.out) + (long long)b * p.ld_out + h * DV;
-  if (p.slots[b] < 0) {                        // idle slot: the state stays, the row is defined
-    for (int i = threadIdx.x; i < DV; i += NT) st(out + i, 0.f);
+  if (slot < 0) {                              // idle slot: the state stays, the row is defined
+    for (int i = tid; i < DV; i += NT) st(out + i, 0.f);
     return;
   }
-  const int pos = p.context_lens[b] - 1;
-  const int TX = 1 << tx_log2, TY = NT >> tx_log2, tx = threadIdx.x & (TX - 1), ty = threadIdx.x >> tx_log2;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int TX = 1 << tx_log2, TY = NT >> tx_log2, tx = tid & (TX - 1), ty = tid >> tx_log2;
+  const int warp = tid >> 5, lane = tid & 31;
+  const int C = 2 * p.G * D + H * DV, items = 2 * D + DV;
+  T* ring = reinterpret_cast<T*>(p.ring) + (long long)b * p.taps * C;
+  const T* x = reinterpret_cast<const T*>(p.x) + (long long)b * p.ld;
+  const T* a = reinterpret_cast<const T*>(p.a) + (long long)b * p.ld_a;
+  const T* gate = reinterpret_cast<const T*>(p.gate) + (long long)b * p.ld_gate + h * DV;
+  auto channel = [&](int i) {
+    return i < D ? kvh * D + i : (i < 2 * D ? (p.G + kvh) * D + i - D : 2 * p.G * D + h * DV + i - 2 * D);
+  };
+  T xr[NI][4], ar, zr, br = reinterpret_cast<const T*>(p.b)[(long long)b * p.ld + h];
+  st(&ar, 0.f); st(&zr, 0.f);
+  float wr[NI][4], dt = 0.f, nw = 0.f;
+  const float al = p.a_log[h];
+  if constexpr (FAST) {
+#pragma unroll
+    for (int j = 0; j < NI; ++j) {
+      const int i = tid + NT * j, c = i < items ? channel(i) : 0;
+#pragma unroll
+      for (int d = 0; d < 4; ++d) {
+        st(&xr[j][d], 0.f);
+        wr[j][d] = 0.f;
+        if (i < items && d < p.taps && d <= pos) {
+          xr[j][d] = d == 0 ? x[c] : ring[(long long)((pos - d) % p.taps) * C + c];
+          wr[j][d] = p.conv[(long long)(p.taps - 1 - d) * C + c];
+        }
+      }
+    }
+    if (tid < D) {
+      ar = a[p.by_channel ? h * D + tid : h];
+      dt = p.dt_bias[p.by_channel ? h * D + tid : h];
+    }
+    if (tid < DV) { zr = gate[tid]; nw = p.norm[tid]; }
+  }
   float* state = p.state + ((long long)b * H + h) * D * DV;
   const int col = tx * 4;
   float4 s[NR];
@@ -465,26 +682,34 @@ __global__ void __launch_bounds__(NT) delta_decode_kernel(const Args p, int tx_l
   float* s_v = s_k + D;                        // [DV], later o
   float* s_g = s_v + DV;                       // [D]
   float* s_red = s_g + D;                      // [NT / 32] + 2 x [TY][4 TX]
-  const int C = 2 * p.G * D + H * DV;
-  T* ring = reinterpret_cast<T*>(p.ring) + (long long)b * p.taps * C;
-  const T* x = reinterpret_cast<const T*>(p.x) + (long long)b * p.ld;
-  for (int i = threadIdx.x; i < 2 * D + DV; i += NT) {
-    const int c = i < D ? kvh * D + i : (i < 2 * D ? (p.G + kvh) * D + i - D : 2 * p.G * D + h * DV + i - 2 * D);
-    float v[1];
-    conv_silu<T, 1>(p, ring, b, 0, pos, c, C, v);
-    s_q[i] = v[0];
-    // the ring has a place for the current input that no token up to this one reads: heads that share q and k do not race
-    if (i >= 2 * D || h % reps == 0) ring[(long long)(pos % p.taps) * C + c] = x[c];
-  }
-  const T* a = reinterpret_cast<const T*>(p.a) + (long long)b * p.ld_a;
-  const float al = p.a_log[h];
-  if (p.by_channel) {
-    for (int i = threadIdx.x; i < D; i += NT) s_g[i] = decayf(al, ld(a + h * D + i) + p.dt_bias[h * D + i]);
+  // the ring has a place for the current input that no token up to this one reads: heads that share q and k do not race
+  if constexpr (FAST) {
+#pragma unroll
+    for (int j = 0; j < NI; ++j) {
+      const int i = tid + NT * j;
+      if (i < items) {
+        float acc = 0.f;
+#pragma unroll
+        for (int d = 3; d >= 0; --d) acc = fmaf(ld(&xr[j][d]), wr[j][d], acc);
+        s_q[i] = siluf(acc);
+        if (i >= 2 * D || h % reps == 0) ring[(long long)(pos % p.taps) * C + channel(i)] = xr[j][0];
+      }
+    }
+    if (tid < D) s_g[tid] = decayf(al, ld(&ar) + dt);
   } else {
-    const float g = decayf(al, ld(a + h) + p.dt_bias[h]);
-    for (int i = threadIdx.x; i < D; i += NT) s_g[i] = g;
+    for (int i = tid; i < items; i += NT) {
+      const int c = channel(i);
+      float v[1];
+      conv_silu<T, 1>(p, ring, b, 0, pos, c, C, v);
+      s_q[i] = v[0];
+      if (i >= 2 * D || h % reps == 0) ring[(long long)(pos % p.taps) * C + c] = x[c];
+    }
+    for (int i = tid; i < D; i += NT) {
+      const int c = p.by_channel ? h * D + i : h;
+      s_g[i] = decayf(al, ld(a + c) + p.dt_bias[c]);
+    }
   }
-  const float beta = sigmoidf(ld(reinterpret_cast<const T*>(p.b) + (long long)b * p.ld + h));
+  const float beta = sigmoidf(ld(&br));
   __syncthreads();
   float qq = 0.f, kk = 0.f, qk = 0.f;
   for (int i = lane; i < D; i += 32) {
@@ -511,7 +736,7 @@ __global__ void __launch_bounds__(NT) delta_decode_kernel(const Args p, int tx_l
   for (int i = 0; i < 4; ++i) { red_a[ty * TX * 4 + col + i] = av[i]; red_b[ty * TX * 4 + col + i] = bv[i]; }
   __syncthreads();
   float ss = 0.f;
-  for (int c = threadIdx.x; c < DV; c += NT) {
+  for (int c = tid; c < DV; c += NT) {
     float sa = 0.f, sb = 0.f;
     for (int y = 0; y < TY; ++y) { sa += red_a[y * TX * 4 + c]; sb += red_b[y * TX * 4 + c]; }
     const float u = beta * (s_v[c] - sa);
@@ -539,10 +764,9 @@ __global__ void __launch_bounds__(NT) delta_decode_kernel(const Args p, int tx_l
 #pragma unroll
   for (int i = 0; i < NT / 32; ++i) tot += s_red[i];
   const float rstd = 1.f / sqrtf(tot / DV + p.eps) * p.out_scale;
-  const T* gate = reinterpret_cast<const T*>(p.gate) + (long long)b * p.ld_gate + h * DV;
-  for (int c = threadIdx.x; c < DV; c += NT) {
-    const float z = ld(gate + c);
-    st(out + c, s_v[c] * rstd * p.norm[c] * (p.gate_silu ? siluf(z) : sigmoidf(z)));
+  for (int c = tid; c < DV; c += NT) {
+    const float z = FAST ? ld(&zr) : ld(gate + c), w = FAST ? nw : p.norm[c];
+    st(out + c, s_v[c] * rstd * w * (p.gate_silu ? siluf(z) : sigmoidf(z)));
   }
 }
 
@@ -562,20 +786,18 @@ int prepare(const Args& p, cudaStream_t stream) {
   const bool vec = p.D % 4 == 0 && p.DV % 4 == 0 && p.ld % 4 == 0 && C % 4 == 0 && al(p.x, 4 * es) && al(p.ring, 4 * es) &&
                    al(p.conv, 16) && al(p.qk, 16) && al(p.v, 16);
   const int m = p.D > p.DV ? p.D : p.DV;
-  if (vec) {
-    if (m <= 128) prepare_kernel<T, 4, 1><<<grid, 128, 0, stream>>>(p, units);
-    else prepare_kernel<T, 4, 4><<<grid, 128, 0, stream>>>(p, units);
-  } else {
-    if (m <= 128) prepare_kernel<T, 1, 4><<<grid, 128, 0, stream>>>(p, units);
-    else prepare_kernel<T, 1, 16><<<grid, 128, 0, stream>>>(p, units);
-  }
+  if (vec && m <= 128 && p.taps <= 4) prepare_kernel<T, 4, 1, true><<<grid, 128, 0, stream>>>(p, units);
+  else if (vec) prepare_kernel<T, 4, 4, false><<<grid, 128, 0, stream>>>(p, units);
+  else prepare_kernel<T, 1, 16, false><<<grid, 128, 0, stream>>>(p, units);
   return fail("prepare");
 }
 
 template <typename T, int R, int L, int C, bool CH>
 int scan_one(const Args& p, int vec, cudaStream_t stream) {
+  using S = ScanShape<R, L, C, CH>;
   auto kern = scan_kernel<T, R, L, C, CH>;
-  constexpr int smem = scan_smem<R, L, C, CH>();
+  constexpr int smem = 2 * S::kStage * (int)sizeof(float);
+  static_assert(smem <= 227 * 1024, "shared memory budget exceeded");
   static bool set = false;
   if (!set) {
     if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) {
@@ -584,8 +806,7 @@ int scan_one(const Args& p, int vec, cudaStream_t stream) {
     }
     set = true;
   }
-  constexpr int cols = ScanShape<R, L, C>::kCols;
-  dim3 grid((p.DV + cols - 1) / cols, p.H, p.B);
+  dim3 grid((p.DV + S::kCols - 1) / S::kCols, p.H, p.B);
   kern<<<grid, kScanThreads, smem, stream>>>(p, vec);
   return fail("scan");
 }
@@ -593,11 +814,11 @@ int scan_one(const Args& p, int vec, cudaStream_t stream) {
 template <typename T, bool CH>
 int scan(const Args& p, cudaStream_t stream) {
   const int vec = p.D % 4 == 0 && p.DV % 4 == 0 && al(p.qk, 16) && al(p.v, 16) && al(p.g, 16) ? 1 : 0;
-  if (p.D <= 32) return scan_one<T, 8, 4, 2, CH>(p, vec, stream);
-  if (p.D <= 64) return scan_one<T, 16, 4, 2, CH>(p, vec, stream);
-  if (p.D <= 128) return scan_one<T, 32, 4, 2, CH>(p, vec, stream);
-  if (p.D <= 256) return scan_one<T, 32, 8, 2, CH>(p, vec, stream);
-  return scan_one<T, 32, 16, 2, CH>(p, vec, stream);
+  if (p.D <= 32) return scan_one<T, 8, 4, 4, CH>(p, vec, stream);
+  if (p.D <= 64) return scan_one<T, 8, 8, 4, CH>(p, vec, stream);
+  if (p.D <= 128) return scan_one<T, 16, 8, 4, CH>(p, vec, stream);
+  if (p.D <= 256) return scan_one<T, 16, 16, 4, CH>(p, vec, stream);
+  return scan_one<T, 16, 32, 4, CH>(p, vec, stream);
 }
 
 template <typename T>
@@ -623,11 +844,13 @@ int tx_log2_of(int DV) {
   return l;
 }
 
-template <typename T, int NT, int NR>
+template <typename T, int NT, int NR, int NI>
 int decode_one(const Args& p, cudaStream_t stream) {
   const int l = tx_log2_of(p.DV);
   const size_t smem = (size_t)(3 * p.D + 2 * p.DV + NT / 32 + 2 * NT * 4) * sizeof(float) + 16;
-  delta_decode_kernel<T, NT, NR><<<dim3(p.H, p.B), NT, smem, stream>>>(p, l);
+  const bool fast = p.taps <= 4 && 2 * p.D + p.DV <= NI * NT && p.D <= NT && p.DV <= NT;
+  if (fast) delta_decode_kernel<T, NT, NR, NI, true><<<dim3(p.H, p.B), NT, smem, stream>>>(p, l);
+  else delta_decode_kernel<T, NT, NR, NI, false><<<dim3(p.H, p.B), NT, smem, stream>>>(p, l);
   return fail("decode");
 }
 
@@ -640,10 +863,10 @@ int decode_rows(int D, int DV, int nt) {
 template <typename T>
 int decode(const Args& p, cudaStream_t stream) {
   const int n256 = decode_rows(p.D, p.DV, 256);
-  if (n256 <= 4) return decode_one<T, 256, 4>(p, stream);
-  if (n256 <= 8) return decode_one<T, 256, 8>(p, stream);
-  if (n256 <= 16) return decode_one<T, 256, 16>(p, stream);
-  return decode_one<T, 512, 16>(p, stream);
+  if (n256 <= 4) return decode_one<T, 256, 4, 2>(p, stream);
+  if (n256 <= 8) return decode_one<T, 256, 8, 2>(p, stream);
+  if (n256 <= 16) return decode_one<T, 512, 8, 1>(p, stream);
+  return decode_one<T, 512, 16, 2>(p, stream);
 }
 
 int check(const Args& p) {
