@@ -14,13 +14,12 @@
 // at position 0 reads neither S nor the ring, and no position below 0 is ever read.
 //
 // A batch is ragged: sequence b brings the rows cu_q[b] .. cu_q[b + 1] - 1, which end at position context_lens[b] - 1.
-// Portions run as prepare (convolution, unit vectors, decays; one warp per row and head) -> scan (the recurrence) ->
-// gate_out. A decode step (one row per slot) is one kernel, delta_decode.
+// Portions run as prepare (convolutions, unit vectors) and decays -> scan (the recurrence) -> gate_out. A decode step (one row
+// per slot) is one kernel, delta_decode.
 //
-// The scan runs token by token in fp32 on the FMA pipes, since the state and all that enters it are 32-bit by design. Columns of
+// The scan walks the tokens in fp32 on the FMA pipes, since the state and all that enters it are 32-bit by design. Columns of
 // S are independent: a CTA takes a range of the columns of one head of one sequence, L lanes share a column, and a thread
-// keeps R rows of C columns in registers for the whole portion, as pairs for the packed fp32 instructions. With
-// a = (g S)^T k and b = (g S)^T q taken in one pass, o = b + u (k . q) needs no second pass over S.
+// keeps R rows of C columns in registers for the whole portion, as pairs for the packed fp32 instructions.
 #include <type_traits>
 
 #include "common.cuh"
@@ -59,6 +58,7 @@ template <int VEC> __device__ __forceinline__ void stv(__nv_bfloat16* p, const f
   else st(p, v[0]);
 }
 
+// (an overflowing exponential gives a quotient of zero)
 __device__ __forceinline__ float sigmoidf(float x) { return 1.f / (1.f + expf(-x)); }
 __device__ __forceinline__ float siluf(float x) { return x / (1.f + expf(-x)); }
 __device__ __forceinline__ float softplusf(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
@@ -83,7 +83,7 @@ struct Args {
   const int* slots;         // [B] cache slot of the row, negative: idle (decode)
   float* qk;                // scratch [T, G, 2, D]: unit q (scaled), unit k
   float* v;                 // scratch [T, H, DV]
-  float* beta;              // scratch [T, H, 2]: beta, q . k
+  float* beta;              // scratch [T, H]
   float* g;                 // scratch [T, H] or [T, H, D]
   float* o;                 // scratch [T, H, DV]
   void* out;                // [T, H DV] type T (pitch ld_out)
@@ -165,23 +165,31 @@ struct ConvRun {
   }
 };
 
-// One warp per unit and run of rows. Units: G (q and k of a key head), H (v of a head), then H (decays of a head's channels)
-// or ceil(H / 32) (decays of 32 heads); the last kind also makes beta. FAST: VEC 4, heads up to 128, at most four taps.
+// One warp per unit and run of rows; units: G heads of q and G of k (made unit vectors, q also scaled), H heads of v. FAST: VEC
+// 4, heads up to 128, at most four taps.
 template <typename T, int VEC, int NJ, bool FAST>
-__global__ void __launch_bounds__(128) prepare_kernel(const Args p, int units) {
+__global__ void __launch_bounds__(128) prepare_kernel(const Args p) {
   const int unit = blockIdx.y * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-  if (unit >= units) return;
+  if (unit >= 2 * p.G + p.H) return;
   const int r0 = blockIdx.x * kRun, r1 = min(r0 + kRun, p.T);
   const int C = 2 * p.G * p.D + p.H * p.DV;
+  const bool is_q = unit < p.G, is_v = unit >= 2 * p.G;
+  const int size = is_v ? p.DV : p.D, c0 = is_v ? 2 * p.G * p.D + (unit - 2 * p.G) * p.DV : unit * p.D;
+  float* dst;
+  long long pitch;
+  if (is_v) {
+    pitch = (long long)p.H * p.DV;
+    dst = p.v + (unit - 2 * p.G) * p.DV;
+  } else {
+    pitch = (long long)p.G * 2 * p.D;
+    dst = p.qk + (is_q ? unit * 2 : (unit - p.G) * 2 + 1) * p.D;
+  }
+  const float scale = is_q ? 1.f / sqrtf((float)p.D) : 1.f;
   int b = sequence_of(p.cu_q, p.B, r0);
-  const bool is_qk = unit < p.G, is_v = !is_qk && unit < p.G + p.H;
-  ConvRun<T> ca, cb;
-  const int h = unit - p.G, dl = lane * 4;
-  const int c0 = is_qk ? unit * p.D + dl : 2 * p.G * p.D + h * p.DV + dl, c1 = (p.G + unit) * p.D + dl;
-  const bool on = is_qk ? dl < p.D : dl < p.DV;
+  ConvRun<T> run;
+  const bool on = lane * 4 < size;
   if constexpr (FAST) {
-    if ((is_qk || is_v) && on) ca.open(p, r0, c0, C);
-    if (is_qk && on) cb.open(p, r0, c1, C);
+    if (on) run.open(p, r0, c0 + lane * 4, C);
   }
 #pragma unroll
   for (int ri = 0; ri < kRun; ++ri) {
@@ -191,77 +199,54 @@ __global__ void __launch_bounds__(128) prepare_kernel(const Args p, int units) {
     const int local = r - p.cu_q[b], pos = p.context_lens[b] - (p.cu_q[b + 1] - r);
     const T* ring = reinterpret_cast<const T*>(p.ring) + (long long)b * p.taps * C;
     if constexpr (FAST) {
-      if ((is_qk || is_v) && on && (ri == 0 || local == 0)) {
-        ca.rewind(p, ring, r, local, pos, c0, C);
-        if (is_qk) cb.rewind(p, ring, r, local, pos, c1, C);
+      if (on && (ri == 0 || local == 0)) run.rewind(p, ring, r, local, pos, c0 + lane * 4, C);
+    }
+    float v[NJ][VEC];
+    float ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < NJ; ++j) {
+      const int d = (lane + 32 * j) * VEC;
+      if (d < size) {
+        if constexpr (FAST) run.next(run.x[ri], v[j]);
+        else conv_silu<T, VEC>(p, ring, r, local, pos, c0 + d, C, v[j]);
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) ss = fmaf(v[j][i], v[j][i], ss);
       }
     }
-    if (is_qk) {
-      float q[NJ][VEC], k[NJ][VEC];
-      float qq = 0.f, kk = 0.f, qk = 0.f;
+    float f = 1.f;
+    if (!is_v) f = scale / sqrtf(warp_sum(ss) + 1e-6f);
 #pragma unroll
-      for (int j = 0; j < NJ; ++j) {
-        const int d = (lane + 32 * j) * VEC;
-        if (d < p.D) {
-          if constexpr (FAST) {
-            ca.next(ca.x[ri], q[j]);
-            cb.next(cb.x[ri], k[j]);
-          } else {
-            conv_silu<T, VEC>(p, ring, r, local, pos, unit * p.D + d, C, q[j]);
-            conv_silu<T, VEC>(p, ring, r, local, pos, (p.G + unit) * p.D + d, C, k[j]);
-          }
+    for (int j = 0; j < NJ; ++j) {
+      const int d = (lane + 32 * j) * VEC;
+      if (d < size) {
 #pragma unroll
-          for (int i = 0; i < VEC; ++i) {
-            qq = fmaf(q[j][i], q[j][i], qq);
-            kk = fmaf(k[j][i], k[j][i], kk);
-            qk = fmaf(q[j][i], k[j][i], qk);
-          }
-        }
+        for (int i = 0; i < VEC; ++i) v[j][i] *= f;
+        stv<VEC>(dst + r * pitch + d, v[j]);
       }
-      qq = warp_sum(qq); kk = warp_sum(kk); qk = warp_sum(qk);
-      const float rq = 1.f / sqrtf(qq + 1e-6f) / sqrtf((float)p.D), rk = 1.f / sqrtf(kk + 1e-6f);
-      float* dst = p.qk + ((long long)r * p.G + unit) * 2 * p.D;
+    }
+  }
+}
+
+// beta [T, H] and the decays [T, H] or [T, H, D], VEC channels per thread
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256) decay_kernel(const Args p) {
+  const int per = p.by_channel ? p.D / VEC : 1;
+  const long long n = (long long)p.T * p.H * per;
+  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x) {
+    const long long rh = i / per, r = rh / p.H;
+    const int h = (int)(rh - r * p.H), d = (int)(i - rh * per) * VEC;
+    if (d == 0) p.beta[rh] = sigmoidf(ld(reinterpret_cast<const T*>(p.b) + r * p.ld + h));
+    const T* a = reinterpret_cast<const T*>(p.a) + r * p.ld_a;
+    if (p.by_channel) {
+      float v[VEC], t[VEC];
+      ldv<VEC>(a + h * p.D + d, v);
+      ldv<VEC>(p.dt_bias + h * p.D + d, t);
+      const float al = p.a_log[h];
 #pragma unroll
-      for (int j = 0; j < NJ; ++j) {
-        const int d = (lane + 32 * j) * VEC;
-        if (d < p.D) {
-#pragma unroll
-          for (int i = 0; i < VEC; ++i) { q[j][i] *= rq; k[j][i] *= rk; }
-          stv<VEC>(dst + d, q[j]);
-          stv<VEC>(dst + p.D + d, k[j]);
-        }
-      }
-      const int reps = p.H / p.G;
-      for (int i = lane; i < reps; i += 32) p.beta[((long long)r * p.H + unit * reps + i) * 2 + 1] = qk * rq * rk;
-    } else if (is_v) {
-#pragma unroll
-      for (int j = 0; j < NJ; ++j) {
-        const int d = (lane + 32 * j) * VEC;
-        if (d < p.DV) {
-          float v[VEC];
-          if constexpr (FAST) ca.next(ca.x[ri], v);
-          else conv_silu<T, VEC>(p, ring, r, local, pos, 2 * p.G * p.D + h * p.DV + d, C, v);
-          stv<VEC>(p.v + ((long long)r * p.H + h) * p.DV + d, v);
-        }
-      }
+      for (int e = 0; e < VEC; ++e) v[e] = decayf(al, v[e] + t[e]);
+      stv<VEC>(p.g + rh * p.D + d, v);
     } else {
-      const int i0 = unit - p.G - p.H;
-      const T* a = reinterpret_cast<const T*>(p.a) + r * p.ld_a;
-      const T* bb = reinterpret_cast<const T*>(p.b) + r * p.ld;
-      if (p.by_channel) {
-        const float al = p.a_log[i0];
-        for (int d = lane; d < p.D; d += 32) {
-          const int c = i0 * p.D + d;
-          p.g[(long long)r * p.H * p.D + c] = decayf(al, ld(a + c) + p.dt_bias[c]);
-        }
-        if (lane == 0) p.beta[((long long)r * p.H + i0) * 2] = sigmoidf(ld(bb + i0));
-      } else {
-        const int hh = i0 * 32 + lane;
-        if (hh < p.H) {
-          p.g[(long long)r * p.H + hh] = decayf(p.a_log[hh], ld(a + hh) + p.dt_bias[hh]);
-          p.beta[((long long)r * p.H + hh) * 2] = sigmoidf(ld(bb + hh));
-        }
-      }
+      p.g[rh] = decayf(p.a_log[h], ld(a + h) + p.dt_bias[h]);
     }
   }
 }
@@ -361,8 +346,7 @@ __global__ void __launch_bounds__(kScanThreads, 2) scan_kernel(const Args p, int
     constexpr int NJ = (DP + 127) / 128, PW = kPairs / kFeedWarps, VN = (2 * COLS + 127) / 128;
     const int fw = (threadIdx.x - kComputeThreads) >> 5;
     float k[PW][2][NJ][4], q[PW][2][NJ][4], g[PW][2][CH ? NJ : 1][4], v[PW][VN][4];
-    float2 sc[PW];                                   // lane 0: beta, q k of token 1; lane 1: of token 2
-    float gs[PW];                                    // and its decay (without CH)
+    float bs[PW], gs[PW];                            // lanes 0 and 1: beta and decay (without CH) of the two tokens
     auto four = [&](const float* src, int at, int size, float fill, float (&o)[4]) {
       if (at + 3 < size && vec) { ldv<4>(src + at, o); return; }
 #pragma unroll
@@ -393,7 +377,7 @@ __global__ void __launch_bounds__(kScanThreads, 2) scan_kernel(const Args p, int
         if (lane < 2) {
           const bool there = t0 + lane < n;
           const long long at = (long long)(r0 + (there ? t0 + lane : n - 1)) * H + h;
-          sc[w] = there ? *reinterpret_cast<const float2*>(p.beta + at * 2) : make_float2(0.f, 0.f);
+          bs[w] = there ? p.beta[at] : 0.f;
           gs[w] = !CH && there ? p.g[at] : 1.f;
         }
       }
@@ -404,7 +388,7 @@ __global__ void __launch_bounds__(kScanThreads, 2) scan_kernel(const Args p, int
       for (int w = 0; w < PW; ++w) {
         const int j2 = fw + w * kFeedWarps;
         float* vecs = stage + j2 * VECS * DP;
-        float kk = 0.f, qk = 0.f;
+        float kk = 0.f, qk = 0.f, own1 = 0.f, own2 = 0.f;
 #pragma unroll
         for (int j = 0; j < NJ; ++j) {
           const int d = (lane + 32 * j) * 4;
@@ -424,6 +408,8 @@ __global__ void __launch_bounds__(kScanThreads, 2) scan_kernel(const Args p, int
               }
               kk = fmaf(k2, w1, kk);
               qk = fmaf(q2, w1, qk);
+              own1 = fmaf(q1, k1, own1);
+              own2 = fmaf(q2, k2, own2);
             }
 #pragma unroll
             for (int x = 0; x < VECS; ++x) stv<4>(vecs + x * DP + d, o[x]);
@@ -431,6 +417,8 @@ __global__ void __launch_bounds__(kScanThreads, 2) scan_kernel(const Args p, int
         }
         kk = warp_sum(kk);
         qk = warp_sum(qk);
+        own1 = warp_sum(own1);
+        own2 = warp_sum(own2);
         float* vs = stage + kPairs * VECS * DP + j2 * 2 * COLS;
 #pragma unroll
         for (int i = 0; i < VN; ++i) {
@@ -439,7 +427,7 @@ __global__ void __launch_bounds__(kScanThreads, 2) scan_kernel(const Args p, int
         }
         float* ss = stage + kPairs * (VECS * DP + 2 * COLS) + j2 * 8;
         const float g2 = __shfl_sync(0xffffffffu, gs[w], 1);
-        if (lane < 2) { ss[2 * lane] = sc[w].x; ss[2 * lane + 1] = sc[w].y; ss[6 + lane] = gs[w]; }
+        if (lane < 2) { ss[2 * lane] = bs[w]; ss[2 * lane + 1] = lane ? own2 : own1; ss[6 + lane] = gs[w]; }
         if (lane == 0) { ss[4] = CH ? kk : kk * g2; ss[5] = CH ? qk : qk * g2; }
       }
     };
@@ -780,16 +768,26 @@ int fail(const char* what) {
 
 template <typename T>
 int prepare(const Args& p, cudaStream_t stream) {
-  const int units = p.G + p.H + (p.by_channel ? p.H : (p.H + 31) / 32);
-  dim3 grid((p.T + kRun - 1) / kRun, (units + 3) / 4);
+  dim3 grid((p.T + kRun - 1) / kRun, (2 * p.G + p.H + 3) / 4);
   const int es = sizeof(T), C = 2 * p.G * p.D + p.H * p.DV;
   const bool vec = p.D % 4 == 0 && p.DV % 4 == 0 && p.ld % 4 == 0 && C % 4 == 0 && al(p.x, 4 * es) && al(p.ring, 4 * es) &&
                    al(p.conv, 16) && al(p.qk, 16) && al(p.v, 16);
   const int m = p.D > p.DV ? p.D : p.DV;
-  if (vec && m <= 128 && p.taps <= 4) prepare_kernel<T, 4, 1, true><<<grid, 128, 0, stream>>>(p, units);
-  else if (vec) prepare_kernel<T, 4, 4, false><<<grid, 128, 0, stream>>>(p, units);
-  else prepare_kernel<T, 1, 16, false><<<grid, 128, 0, stream>>>(p, units);
+  if (vec && m <= 128 && p.taps <= 4) prepare_kernel<T, 4, 1, true><<<grid, 128, 0, stream>>>(p);
+  else if (vec) prepare_kernel<T, 4, 4, false><<<grid, 128, 0, stream>>>(p);
+  else prepare_kernel<T, 1, 16, false><<<grid, 128, 0, stream>>>(p);
   return fail("prepare");
+}
+
+template <typename T>
+int decays(const Args& p, cudaStream_t stream) {
+  const bool vec = p.by_channel && p.D % 4 == 0 && p.ld_a % 4 == 0 && al(p.a, 4 * sizeof(T)) && al(p.dt_bias, 16) && al(p.g, 16);
+  const long long n = (long long)p.T * p.H * (p.by_channel ? p.D / (vec ? 4 : 1) : 1);
+  long long blocks = (n + 255) / 256;
+  if (blocks > 148 * 16) blocks = 148 * 16;
+  if (vec) decay_kernel<T, 4><<<(unsigned)blocks, 256, 0, stream>>>(p);
+  else decay_kernel<T, 1><<<(unsigned)blocks, 256, 0, stream>>>(p);
+  return fail("decays");
 }
 
 template <typename T, int R, int L, int C, bool CH>
@@ -816,7 +814,11 @@ int scan(const Args& p, cudaStream_t stream) {
   const int vec = p.D % 4 == 0 && p.DV % 4 == 0 && al(p.qk, 16) && al(p.v, 16) && al(p.g, 16) ? 1 : 0;
   if (p.D <= 32) return scan_one<T, 8, 4, 4, CH>(p, vec, stream);
   if (p.D <= 64) return scan_one<T, 8, 8, 4, CH>(p, vec, stream);
-  if (p.D <= 128) return scan_one<T, 16, 8, 4, CH>(p, vec, stream);
+  if (p.D <= 128) {
+    // few sequences and heads: half as many columns per CTA give twice as many CTAs
+    if ((long long)p.B * p.H * ((p.DV + 63) / 64) <= 148) return scan_one<T, 8, 16, 4, CH>(p, vec, stream);
+    return scan_one<T, 16, 8, 4, CH>(p, vec, stream);
+  }
   if (p.D <= 256) return scan_one<T, 16, 16, 4, CH>(p, vec, stream);
   return scan_one<T, 16, 32, 4, CH>(p, vec, stream);
 }
@@ -863,9 +865,9 @@ int decode_rows(int D, int DV, int nt) {
 template <typename T>
 int decode(const Args& p, cudaStream_t stream) {
   const int n256 = decode_rows(p.D, p.DV, 256);
-  if (n256 <= 4) return decode_one<T, 256, 4, 2>(p, stream);
+  if (n256 <= 4 && decode_rows(p.D, p.DV, 128) <= 8) return decode_one<T, 128, 8, 2>(p, stream);
   if (n256 <= 8) return decode_one<T, 256, 8, 2>(p, stream);
-  if (n256 <= 16) return decode_one<T, 512, 8, 1>(p, stream);
+  if (n256 <= 16) return decode_one<T, 256, 16, 2>(p, stream);
   return decode_one<T, 512, 16, 2>(p, stream);
 }
 
@@ -892,7 +894,7 @@ int mfb_delta_decode_supported(int D, int DV) {
 // floats of scratch for T rows
 long long mfb_delta_scratch_floats(int T, int H, int G, int D, int DV, int by_channel) {
   auto up = [](long long n) { return (n + 3) / 4 * 4; };
-  return up((long long)T * G * 2 * D) + 2 * up((long long)T * H * DV) + up((long long)T * H * 2) + up((long long)T * H * (by_channel ? D : 1));
+  return up((long long)T * G * 2 * D) + 2 * up((long long)T * H * DV) + up((long long)T * H) + up((long long)T * H * (by_channel ? D : 1));
 }
 
 // The whole mixer core (see the file header). f32: the activations (x, b, a, gate, ring, out) are fp32, else bf16. cu_q null: a
@@ -921,8 +923,9 @@ int mfb_delta_rule(const void* x, long long ld, const void* b, const void* a, lo
   p.v = p.qk + up((long long)T * G * 2 * D);
   p.o = p.v + up((long long)T * H * DV);
   p.beta = p.o + up((long long)T * H * DV);
-  p.g = p.beta + up((long long)T * H * 2);
+  p.g = p.beta + up((long long)T * H);
   int rc = f32 ? dlt::prepare<float>(p, stream) : dlt::prepare<__nv_bfloat16>(p, stream);
+  if (!rc) rc = f32 ? dlt::decays<float>(p, stream) : dlt::decays<__nv_bfloat16>(p, stream);
   if (rc) return rc;
   if (f32) rc = by_channel ? dlt::scan<float, true>(p, stream) : dlt::scan<float, false>(p, stream);
   else rc = by_channel ? dlt::scan<__nv_bfloat16, true>(p, stream) : dlt::scan<__nv_bfloat16, false>(p, stream);

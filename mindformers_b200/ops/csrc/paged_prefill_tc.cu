@@ -45,6 +45,7 @@ struct Args {
   int num_q_heads, group, D, DV, block_size, max_blocks, chunk;
   float scale_log2;
   float cap_log2, cap_scale;   // soft cap of the scores in log2 units (CAP kernels) and scale / cap
+  float cap_poly[5];           // capped score (log2 units) = s * polynomial in s^2, for |s| * cap_scale <= kPolyReach
   long long ld_out;
   float out_scale;
   int* status;
@@ -102,15 +103,11 @@ __device__ __forceinline__ void tmem_st_32x32b_x32(uint32_t taddr, const uint32_
       : "memory");
 }
 
-// tanh(x) / x as a polynomial in z = x^2 on |x| <= kPolyReach (Chebyshev interpolation of degree 4 on [0, kPolyReach^2]:
-// relative error 7.4e-8). It runs on the FMA pipes two scores at a time, which leaves the exponentials to the softmax.
+// tanh(x) / x as a polynomial in x^2 on |x| <= kPolyReach (Chebyshev interpolation of degree 4 on [0, kPolyReach^2]: relative
+// error 7.4e-8). It runs on the FMA pipes two scores at a time, which leaves the exponentials to the softmax; the launcher
+// folds the scales into the coefficients.
 constexpr float kPolyReach = 0.6f;
-__device__ __forceinline__ uint64_t tanh_ratio2(uint64_t z) {
-  const uint64_t c0 = pack2(0.999999926f, 0.999999926f), c1 = pack2(-0.33332302f, -0.33332302f),
-                 c2 = pack2(0.133100644f, 0.133100644f), c3 = pack2(-0.0520966534f, -0.0520966534f),
-                 c4 = pack2(0.0154687513f, 0.0154687513f);
-  return fma2(fma2(fma2(fma2(c4, z, c3), z, c2), z, c1), z, c0);
-}
+constexpr float kTanhRatio[5] = {0.999999926f, -0.33332302f, 0.133100644f, -0.0520966534f, 0.0154687513f};
 
 // HQ: padded query / key size, HV: padded value size (64 or 128); CAP: scores are soft-capped
 template <int HQ, int HV, bool CAP>
@@ -365,21 +362,23 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
             }
             float* s = reinterpret_cast<float*>(sr);
             if constexpr (CAP) {
-              // scores in log2 units: by the polynomial where every score of the warp is within its reach
+              // capped, shifted scores: by the polynomial where every score of the warp is within its reach
               float am = 0.f;
 #pragma unroll
-              for (int i = 0; i < 64; ++i) am = fmaxf(am, fabsf(s[i]));
+              for (int i = 0; i < 32; ++i) am = fmax3(am, fabsf(s[2 * i]), fabsf(s[2 * i + 1]));
               if (__all_sync(0xffffffffu, am * args.cap_scale <= kPolyReach)) {
-                const uint64_t cs2 = pack2(args.cap_scale, args.cap_scale);
+                uint64_t c[5];
+#pragma unroll
+                for (int k = 0; k < 5; ++k) c[k] = pack2(args.cap_poly[k], args.cap_poly[k]);
 #pragma unroll
                 for (int i = 0; i < 32; ++i) {
                   const uint64_t v = pack2(s[2 * i], s[2 * i + 1]);
-                  const uint64_t x = mul2(v, cs2);
-                  unpack2(mul2(mul2(v, scale2), tanh_ratio2(mul2(x, x))), s[2 * i], s[2 * i + 1]);
+                  const uint64_t z = mul2(v, v);
+                  unpack2(fma2(v, fma2(fma2(fma2(fma2(c[4], z, c[3]), z, c[2]), z, c[1]), z, c[0]), negm2), s[2 * i], s[2 * i + 1]);
                 }
               } else {
 #pragma unroll
-                for (int i = 0; i < 64; ++i) s[i] = capped(s[i] * args.cap_scale, args.cap_log2);
+                for (int i = 0; i < 64; ++i) s[i] = capped(s[i] * args.cap_scale, args.cap_log2) + neg_m;
               }
             }
 #pragma unroll
@@ -399,8 +398,8 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
 #pragma unroll
             for (int i = 0; i < 32; ++i) {
               float t0, t1;
-              const uint64_t v = pack2(s[2 * i], s[2 * i + 1]);
-              unpack2(CAP ? add2(v, negm2) : fma2(v, scale2, negm2), t0, t1);
+              if constexpr (CAP) { t0 = s[2 * i]; t1 = s[2 * i + 1]; }
+              else unpack2(fma2(pack2(s[2 * i], s[2 * i + 1]), scale2, negm2), t0, t1);
               const float e0 = ex2(t0), e1 = ex2(t1);
               rs2[i & 3] = add2(rs2[i & 3], pack2(e0, e1));
               pk[i] = pack_bf16x2(e0, e1);
@@ -544,6 +543,8 @@ int mfb_paged_prefill_tc(const void* q, const void* key_cache, const void* value
   a.chunk = chunk; a.scale_log2 = scale * 1.4426950408889634f; a.status = status;
   a.cap_log2 = softcap > 0.f ? softcap * 1.4426950408889634f : 0.f;
   a.cap_scale = softcap > 0.f ? scale / softcap : 0.f;
+  float power = a.scale_log2;
+  for (int k = 0; k < 5; ++k, power *= a.cap_scale * a.cap_scale) a.cap_poly[k] = ppt::kTanhRatio[k] * power;
   a.ld_out = ld_out; a.out_scale = out_scale;
   const int max_ctas = persistent ? 2 * 148 : a.n_items;
 #define MFB_PPT(HQ_, HV_) \

@@ -134,7 +134,7 @@ def delta_rule(x: torch.Tensor, b: torch.Tensor, a: torch.Tensor, gate: torch.Te
         buf = torch.empty(need, dtype=torch.float32, device=x.device)
         scratch = buf.data_ptr()
     _launch(lib, x, b, a, gate, w, s, ring, S, cu, cache.context_lens, cache.slot_mapping, scratch, out, T, B, eps, out_scale)
-    _lib.count_launch(1 if decode else 3)
+    _lib.count_launch(1 if decode else 4)
     return out
 
 
@@ -162,7 +162,7 @@ def _decode_as_portions(x, b, a, gate, w, s, state, cache, eps, out, out_scale):
                       device=x.device)
     lens = cache.context_lens.clamp(min=1)
     _launch(lib, x, b, a, gate, w, s, ring, S, cu.data_ptr(), lens, cache.slot_mapping, buf.data_ptr(), out, B, B, eps, out_scale)
-    _lib.count_launch(3)
+    _lib.count_launch(4)
     S[:B].copy_(torch.where(idle[:, None, None, None], keep[0], S[:B]))
     ring[:B].copy_(torch.where(idle[:, None, None], keep[1], ring[:B]))
     return out
