@@ -121,6 +121,8 @@ _MEFESUN = {
 }
 _MEFESUN_TOP = {"embed": "embedding.word_embeddings.weight", "final.norm": "decoder.final_layernorm.weight",
                 "final.norm.b": "decoder.final_layernorm.bias"}
+_GAVATAR_TOP = {"embed": "embedding.word_embeddings.weight", "final.norm": "decoder.final_layernorm.weight",
+                "head": "output_layer.weight", "loop.step": "decoder.loop_step"}
 _LIST_LAYER = re.compile(r"^l(\d+)\.(.+)$")
 
 
@@ -227,11 +229,7 @@ def kukupel_to_framework(sd: Dict[str, torch.Tensor], config) -> Dict[str, torch
             for n, to in _KUKUPEL_CORE.items():
                 if prefix + n in own:
                     out[f"{p}{module}.{to}"] = take(prefix + n)
-        n_experts = sum(1 for n in own if re.match(r"^mlp\.e\d+\.gate$", n))
-        if n_experts:
-            w1 = [torch.cat((take(f"mlp.e{e}.gate"), take(f"mlp.e{e}.up")), dim=0).t() for e in range(n_experts)]
-            out[p + "mlp.experts.weight1"] = torch.stack(w1).contiguous()                                      # [E, H, 2F]
-            out[p + "mlp.experts.weight2"] = torch.stack([take(f"mlp.e{e}.down").t() for e in range(n_experts)]).contiguous()
+        out.update((p + n, t) for n, t in _stack_experts(own, take).items())
         for n in sorted(left):
             if n not in _KUKUPEL:
                 raise KeyError(f"l{i}.{n}: no counterpart in the model")
@@ -262,18 +260,14 @@ def framework_to_kukupel(sd: Dict[str, torch.Tensor], config) -> Dict[str, torch
             out.update((f"{l}{prefix}{n}.conv", piece.t().contiguous()) for n, piece in zip("qkv", torch.split(t, sizes, dim=1)))
         elif rest.startswith(module + "."):
             out[l + prefix + core[rest[len(module) + 1:]]] = t
-        elif rest == "mlp.experts.weight1":
-            for e in range(t.shape[0]):
-                g, u = t[e].t().chunk(2, dim=0)
-                out[f"{l}mlp.e{e}.gate"], out[f"{l}mlp.e{e}.up"] = g.contiguous(), u.contiguous()
-        elif rest == "mlp.experts.weight2":
-            out.update((f"{l}mlp.e{e}.down", t[e].t().contiguous()) for e in range(t.shape[0]))
+        elif rest.startswith("mlp.experts.weight"):
+            out.update((l + n, piece) for n, piece in _unstack_experts(rest, t).items())
         else:
             raise KeyError(f"{name}: no counterpart in the checkpoint format")
     return out
 
 
-FAMILIES = ("mefesun", "kukupel", "llama", "qwen2", "qwen2_5", "qwen2_moe", "qwen3", "qwen3_moe", "deepseek_v2", "deepseek_v3",
+FAMILIES = ("mefesun", "kukupel", "gavatar", "llama", "qwen2", "qwen2_5", "qwen2_moe", "qwen3", "qwen3_moe", "deepseek_v2", "deepseek_v3",
             "deepseekv3", "mixtral", "telechat", "glm")
 
 
@@ -497,6 +491,116 @@ def weight_dequant(weight: torch.Tensor, scale_inv: torch.Tensor, block: int = 1
     return (weight.float() * s).to(torch.bfloat16)
 
 
+# Gavatar checkpoints: tensors that map one to one, and per mixer those whose rows are stacked into one parameter.
+_GAVATAR = {
+    "norm1": "input_layernorm.weight", "norm1b": "post_attn_layernorm.weight", "norm2": "pre_mlp_layernorm.weight",
+    "norm2b": "post_mlp_layernorm.weight", "shift": "token_shift", "mlp.router": "mlp.router.weight",
+    "mlp.router.b": "mlp.router.bias", "mix.o": "self_attention.linear_proj.weight",
+}
+_GAVATAR_MIXER = {
+    "attention": {"mix.talk": "self_attention.talk"},
+    "latent": {"mix.dq.norm": "self_attention.q_latent_norm.weight", "mix.dkv.norm": "self_attention.kv_latent_norm.weight",
+               "mix.uq": "self_attention.linear_q_up.weight", "mix.sink": "self_attention.sink"},
+    "matrix_memory": {"mix.i.b": "self_attention.input_bias", "mix.f.b": "self_attention.forget_bias",
+                      "mix.norm": "self_attention.norm"},
+}
+
+
+def _gavatar_layout(config, i: int):
+    """Of layer ``i``: the tensors that map one to one, and ``{parameter: [(tensor, rows)]}`` of the stacked ones."""
+    c = config.for_layer(i)
+    H, D = c.num_attention_heads, c.kv_channels
+    DV = c.v_channels or D
+    if c.mixer == "attention":
+        qkv = [("q", H * D), ("k", c.num_query_groups * D), ("v", c.num_query_groups * DV)]
+        stacked = {"linear_qkv.weight": qkv + [("g", H * DV)], "qkv_bias": [(n + ".b", r) for n, r in qkv]}
+    elif c.mixer == "latent":
+        stacked = {"linear_in.weight": [("dq", c.q_lora_rank), ("dkv", c.kv_lora_rank), ("g", H)],
+                   "linear_kv_up.weight": [("uk", H * D), ("uv", H * DV)]}
+    else:
+        H, D, DV = c.memory_heads, c.memory_key_dim, c.memory_value_dim
+        stacked = {"linear_in.weight": [("q", H * D), ("k", H * D), ("v", H * DV), ("g", H * DV), ("i", H), ("f", H)]}
+    return dict(_GAVATAR, **_GAVATAR_MIXER[c.mixer]), {"self_attention." + p: [("mix." + n, r) for n, r in rows]
+                                                       for p, rows in stacked.items()}
+
+
+def _stack_experts(own: Dict[str, torch.Tensor], take) -> Dict[str, torch.Tensor]:
+    """``mlp.e<i>.gate / up / down`` of one layer → ``weight1 [E, H, 2F]``, ``weight2 [E, F, H]``."""
+    n = sum(1 for name in own if re.match(r"^mlp\.e\d+\.gate$", name))
+    if not n:
+        return {}
+    w1 = [torch.cat((take(f"mlp.e{e}.gate"), take(f"mlp.e{e}.up")), dim=0).t() for e in range(n)]
+    return {"mlp.experts.weight1": torch.stack(w1).contiguous(),
+            "mlp.experts.weight2": torch.stack([take(f"mlp.e{e}.down").t() for e in range(n)]).contiguous()}
+
+
+def _unstack_experts(name: str, t: torch.Tensor) -> Dict[str, torch.Tensor]:
+    if name.endswith("weight2"):
+        return {f"mlp.e{e}.down": t[e].t().contiguous() for e in range(t.shape[0])}
+    out = {}
+    for e in range(t.shape[0]):
+        g, u = t[e].t().chunk(2, dim=0)
+        out[f"mlp.e{e}.gate"], out[f"mlp.e{e}.up"] = g.contiguous(), u.contiguous()
+    return out
+
+
+def gavatar_to_framework(sd: Dict[str, torch.Tensor], config) -> Dict[str, torch.Tensor]:
+    """Gavatar tensors of any number of whole layers → fused framework parameters."""
+    out: Dict[str, torch.Tensor] = {}
+    layers: Dict[int, Dict[str, torch.Tensor]] = {}
+    for name, t in sd.items():
+        m = _LIST_LAYER.match(name)
+        if m:
+            layers.setdefault(int(m[1]), {})[m[2]] = t
+        else:
+            out[_GAVATAR_TOP.get(name, name)] = t
+    for i, own in layers.items():
+        p, left = f"decoder.layers.{i}.", set(own)
+        plain, stacked = _gavatar_layout(config, i)
+
+        def take(name):
+            left.discard(name)
+            if name not in own:
+                raise KeyError(f"l{i}.{name} is missing")
+            return own[name]
+        for to, rows in stacked.items():
+            out[p + to] = torch.cat([take(n) for n, _ in rows], dim=0)
+        out.update((p + n, t) for n, t in _stack_experts(own, take).items())
+        for n in sorted(left):
+            if n not in plain:
+                raise KeyError(f"l{i}.{n}: no counterpart in the model")
+            out[p + plain[n]] = own[n]
+    return out
+
+
+def framework_to_gavatar(sd: Dict[str, torch.Tensor], config) -> Dict[str, torch.Tensor]:
+    """Fused framework names → Gavatar tensors."""
+    top = {v: k for k, v in _GAVATAR_TOP.items()}
+    out: Dict[str, torch.Tensor] = {}
+    for name, t in sd.items():
+        m = re.match(r"^decoder\.layers\.(\d+)\.(.+)$", name)
+        if not m:
+            out[top.get(name, name)] = t
+            continue
+        l, rest = f"l{m[1]}.", m[2]
+        plain, stacked = _gavatar_layout(config, int(m[1]))
+        back = {v: k for k, v in plain.items()}
+        if rest in back:
+            out[l + back[rest]] = t
+        elif rest in stacked:
+            rows = stacked[rest]
+            out.update((l + n, piece.contiguous()) for (n, _), piece in zip(rows, torch.split(t, [r for _, r in rows], dim=0)))
+        elif rest.startswith("mlp.experts.weight"):
+            out.update((l + n, piece) for n, piece in _unstack_experts(rest, t).items())
+        else:
+            raise KeyError(f"{name}: no counterpart in the checkpoint format")
+    return out
+
+
+# families whose tensors are renamed and fused layer by layer, by the layer's own configuration
+_BY_LAYER = {"kukupel": (kukupel_to_framework, framework_to_kukupel), "gavatar": (gavatar_to_framework, framework_to_gavatar)}
+
+
 def hf_to_framework(hf_sd: Dict[str, torch.Tensor], config, family: str = "llama", dtype=None,
                     keep_fp8: bool = False) -> Dict[str, torch.Tensor]:
     """Full conversion of an HF state dict (fp8 block-scaled weights are dequantised unless ``keep_fp8``)."""
@@ -515,8 +619,8 @@ def hf_to_framework(hf_sd: Dict[str, torch.Tensor], config, family: str = "llama
             continue
         if dtype is not None and t.is_floating_point():
             t = t.to(dtype)
-        plain[name if family == "kukupel" else convert_name(name, family)] = t
-    out = kukupel_to_framework(plain, config) if family == "kukupel" else fuse_state_dict(plain, config)
+        plain[name if family in _BY_LAYER else convert_name(name, family)] = t
+    out = _BY_LAYER[family][0](plain, config) if family in _BY_LAYER else fuse_state_dict(plain, config)
     if keep_fp8 and any_fp8:
         out = requantize_linear_weights(out)
     return out
@@ -554,9 +658,9 @@ def framework_to_hf(sd: Dict[str, torch.Tensor], config, family: str = "llama", 
     if family == "mefesun":
         return {k: (t if dtype is None or not t.is_floating_point() else t.to(dtype)).contiguous()
                 for k, t in framework_to_mefesun(sd, config).items()}
-    if family == "kukupel":
+    if family in _BY_LAYER:
         return {k: (t if dtype is None or not t.is_floating_point() else t.to(dtype)).contiguous()
-                for k, t in framework_to_kukupel(sd, config).items()}
+                for k, t in _BY_LAYER[family][1](sd, config).items()}
     for name, t in unfuse_state_dict(sd, config).items():
         if dtype is not None and t.is_floating_point():
             t = t.to(dtype)

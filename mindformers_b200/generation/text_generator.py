@@ -49,7 +49,8 @@ class GenerationMixin:
                 raise NotImplementedError("draft layers share the cache shapes of the decoder")
             ctx = KVCacheContext(n_layers, num_blocks, block_size, 0, 0, dtype, device, layer_shapes=shapes,
                                  kv_cache_dtype=getattr(cfg, "kv_cache_dtype", None),
-                                 state_shapes=self.model.decoder.state_shapes(), slots=batch_size)
+                                 state_shapes=self.model.decoder.state_shapes(), slots=batch_size,
+                                 carry_width=self.model.decoder.carry_width())
         elif getattr(cfg, "multi_latent_attention", False):
             ctx = KVCacheContext(n_layers, num_blocks, block_size, 1, 0, dtype, device,
                                  mla_latent_dim=cfg.kv_lora_rank + cfg.qk_pos_emb_head_dim)

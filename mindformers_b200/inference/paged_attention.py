@@ -29,15 +29,17 @@ class KVCacheContext:
     def __init__(self, num_layers: int, num_blocks: int, block_size: int, kv_heads: int, head_dim: int,
                  dtype=torch.bfloat16, device="cuda", mla_latent_dim: Optional[int] = None,
                  kv_cache_dtype: Optional[str] = None, layer_shapes: Optional[list] = None,
-                 state_shapes: Optional[list] = None, slots: int = 0):
+                 state_shapes: Optional[list] = None, slots: int = 0, carry_width: int = 0):
         """``layer_shapes``: ``(kv heads, key size, value size)`` of every layer's cache, for models whose layers differ or
-        whose keys and values differ in size (None: the layer caches no keys); such a cache also carries the step metadata
-        of ragged attention.
+        whose keys and values differ in size (None: the layer caches no keys; value size 0: the layer's values are its keys);
+        such a cache also carries the step metadata of ragged attention.
 
-        ``state_shapes``: per layer None or ``(heads, key size, value size, conv channels, conv taps)``: layers with a
-        recurrent state have, for each of ``slots`` sequences (row b of a batch uses slot b), ``S [heads, key, value]`` in
-        fp32 and a ring of the last conv inputs (``recurrent[layer]``). A sequence that starts at position 0 reads neither,
-        so a slot changes hands without being cleared.
+        ``state_shapes``: per layer None, ``(heads, key size, value size, conv channels, conv taps)`` or a list of shapes.
+        Layers with a recurrent state have, for each of ``slots`` sequences (row b of a batch uses slot b), ``S [heads, key,
+        value]`` in fp32 and a ring of the last conv inputs, or one fp32 tensor per listed shape (``recurrent[layer]``).
+        ``carry_width``: every layer has a vector of that many fp32 values per slot that goes from one token to the next
+        (``carry [layers, slots, width]``; ``carry_before`` is its value before a prefill step). A sequence that starts at
+        position 0 reads none of them, so a slot changes hands without being cleared.
 
         ``kv_cache_dtype="int8"`` stores keys and values as int8 codes with one fp32 scale per token and KV head
         (``key_scale`` / ``value_scale`` ``[num_blocks, block_size, kv_heads]``): half the bytes per cached token, read
@@ -56,7 +58,7 @@ class KVCacheContext:
             rows = (num_blocks, block_size)
             self.key_cache = [None if s is None else torch.zeros(rows + (s[0], s[1]), dtype=dtype, device=device)
                               for s in layer_shapes]
-            self.value_cache = [None if s is None else torch.zeros(rows + (s[0], s[2]), dtype=dtype, device=device)
+            self.value_cache = [None if s is None or not s[2] else torch.zeros(rows + (s[0], s[2]), dtype=dtype, device=device)
                                 for s in layer_shapes]
         elif self.int8:
             shape = (num_blocks, block_size, kv_heads, head_dim)
@@ -72,9 +74,17 @@ class KVCacheContext:
             shape = (num_blocks, block_size, kv_heads, head_dim)
             self.key_cache = [torch.zeros(shape, dtype=dtype, device=device) for _ in range(num_layers)]
             self.value_cache = [torch.zeros(shape, dtype=dtype, device=device) for _ in range(num_layers)]
-        self.recurrent = [None if s is None else (torch.zeros((slots,) + tuple(s[:3]), dtype=torch.float32, device=device),
-                                                  torch.zeros((slots, s[4], s[3]), dtype=dtype, device=device))
-                          for s in state_shapes or [None] * num_layers]
+
+        def state(s):
+            if s is None:
+                return None
+            if isinstance(s, list):
+                return tuple(torch.zeros((slots,) + tuple(x), dtype=torch.float32, device=device) for x in s)
+            return (torch.zeros((slots,) + tuple(s[:3]), dtype=torch.float32, device=device),
+                    torch.zeros((slots, s[4], s[3]), dtype=dtype, device=device))
+        self.recurrent = [state(s) for s in state_shapes or [None] * num_layers]
+        self.carry = torch.zeros((num_layers, slots, carry_width), dtype=torch.float32, device=device) if carry_width else None
+        self.carry_before = torch.zeros_like(self.carry) if carry_width else None
         self.is_prefill = True
         self.block_tables = None      # int32 [B, max_blocks]
         self.slot_mapping = None      # int32 [T]
@@ -91,22 +101,24 @@ class KVCacheContext:
     @property
     def has_state(self) -> bool:
         """Whether some layer has a recurrent state: such a step cannot be run twice, nor tokens taken back."""
-        return any(r is not None for r in self.recurrent)
+        return self.carry is not None or any(r is not None for r in self.recurrent)
+
+    def _states(self) -> list:
+        """Every state tensor, slots first."""
+        return [t for r in self.recurrent for t in r or ()] + ([] if self.carry is None else [self.carry.transpose(0, 1)])
 
     def save_state(self) -> list:
         """Copy of the recurrent states (for runs that warm up or capture a step and must leave no trace)."""
-        return [None if r is None else tuple(t.clone() for t in r) for r in self.recurrent]
+        return [t.clone() for t in self._states()]
 
     def restore_state(self, saved: list):
-        for r, old in zip(self.recurrent, saved):
-            for t, o in zip(r or (), old or ()):
-                t.copy_(o)
+        for t, old in zip(self._states(), saved):
+            t.copy_(old)
 
     def copy_state(self, dst: List[int], src: List[int]):
         """Slot ``dst[i]`` continues from what slot ``src[i]`` holds now."""
-        for r in self.recurrent:
-            for t in r or ():
-                t[dst] = t[src].clone()
+        for t in self._states():
+            t[dst] = t[src].clone()
 
     def set_step(self, *, is_prefill, block_tables, slot_mapping, context_lens, q_seq_lens, device):
         self.is_prefill = is_prefill
@@ -119,6 +131,8 @@ class KVCacheContext:
         for n in q:
             cu.append(cu[-1] + n)
         self.cu_q = cu
+        if self.carry is not None and is_prefill:
+            self.carry_before.copy_(self.carry)
         if self.ragged and is_prefill:
             self.q_lens_host, self.context_lens_host = q, [int(x) for x in context_lens]
             self.n_long_rows, self.n_single_rows = sum(n > 1 for n in q), sum(n == 1 for n in q)

@@ -111,7 +111,7 @@ class ModelRunner:
         if mla:
             self.kv_heads, self.head_dim, width = 1, cfg.kv_lora_rank + cfg.qk_pos_emb_head_dim, cfg.kv_lora_rank + cfg.qk_pos_emb_head_dim
             per_block = self.n_layers * self.block_size * width * first.element_size()
-        elif self.model.model.decoder.state_shapes():
+        elif self.model.model.decoder.state_shapes() or self.model.model.decoder.carry_width():
             raise NotImplementedError("models with recurrent layers keep a state per sequence slot, which this interface (block "
                                       "tables and slot mappings without sequence slots) cannot name: use serving.ServingEngine")
         elif shapes is not None:

@@ -320,7 +320,93 @@ class KukupelConfig(PretrainedConfig):
         return dict(d, **own)
 
 
+class GavatarConfig(PretrainedConfig):
+    """Gavatar: a decoder on one fp32 stream with norms (weights around zero) on both sides of every sub-layer, a token shift in
+    front of every mixer, scaled embeddings plus sinusoidal position vectors, and a block of layers that runs several times. Its
+    mixers are sliding-window grouped-query attention with unit-norm queries, keys and values whose softmax weights are mixed over
+    heads (``attention``), sliding-window latent attention with a softmax sink (``latent_attention``), both position-free and
+    gated, and a matrix memory (``mlstm``); its feed-forwards are mixtures of SwiGLU experts with biased router logits.
+
+    Keys of ``config.json``: ``vocab``, ``width``, ``norm.eps``, ``embedding.scale``, ``loop`` (``{"start", "stop", "times"}`` or
+    null) and ``layers``, a list of ``{"type": "attention", "mixer": {"heads", "kv_heads", "dim", "vdim", "scale", "mask":
+    {"size"}}}``, ``{"type": "latent_attention", "mixer": {"heads", "dim", "vdim", "q_rank", "kv_rank", "scale", "mask":
+    {"size"}}}`` or ``{"type": "mlstm", "mixer": {"heads", "dim", "vdim", "gate_cap"}}``, each with ``"mlp": {"kind": "moe",
+    "router": {"experts", "top"}, "expert": {"ff"}} | null``. Framework keys (``seq_length``, ``block_size``, token ids) may
+    stand beside them."""
+
+    model_type = "gavatar"
+
+    @classmethod
+    def default_values(cls):
+        return dict(architecture="Gavatar", vocab=32000, width=1024, norm=dict(eps=1e-6), embedding=dict(scale=1.0), loop=None,
+                    layers=GavatarConfig.layer_list("latent_attention mlstm attention", heads=8, kv_heads=2, dim=128, rank=256,
+                                                    window=1024, memory_heads=4, memory_dim=128, experts=16, top=2, ff=768),
+                    pad_token_id=0, bos_token_id=None, eos_token_id=None, block_size=64)
+
+    @staticmethod
+    def layer_list(types: str, heads: int, kv_heads: int, dim: int, rank: int, window: int, memory_heads: int, memory_dim: int,
+                   experts: int, top: int, ff: int, vdim=None, q_rank=None, memory_vdim=None, scale=None, gate_cap: float = 15.0):
+        """The ``layers`` list of a model whose layers of one type (``types``, by name) are alike."""
+        common = dict(heads=heads, dim=dim, vdim=vdim or dim, scale=scale or dim ** -0.5, mask=dict(size=window))
+        mixer = {"attention": dict(common, kv_heads=kv_heads),
+                 "latent_attention": dict(common, q_rank=q_rank or rank, kv_rank=rank),
+                 "mlstm": dict(heads=memory_heads, dim=memory_dim, vdim=memory_vdim or memory_dim, gate_cap=gate_cap)}
+        mlp = dict(kind="moe", router=dict(experts=experts, top=top), expert=dict(ff=ff))
+        return [dict(type=t, mixer=copy.deepcopy(mixer[t]), mlp=copy.deepcopy(mlp)) for t in types.split()]
+
+    @staticmethod
+    def _layer_fields(i: int, layer: dict) -> dict:
+        kind, mix, mlp = layer.get("type"), layer["mixer"], layer.get("mlp")
+        if kind in ("attention", "latent_attention"):
+            out = dict(num_attention_heads=int(mix["heads"]), kv_channels=int(mix["dim"]), v_channels=int(mix["vdim"]),
+                       softmax_scale=float(mix["scale"]), attention_window=int((mix.get("mask") or {}).get("size") or 0))
+            if kind == "attention":
+                out.update(mixer="attention", num_query_groups=int(mix["kv_heads"]), add_qkv_bias=True, qk_unit_norm=True,
+                           value_unit_norm=True, attention_talk=True, attention_output_gate="channel")
+            else:
+                out.update(mixer="latent", num_query_groups=int(mix["heads"]), q_lora_rank=int(mix["q_rank"]),
+                           kv_lora_rank=int(mix["kv_rank"]), attention_sink=True, attention_output_gate="head")
+        elif kind == "mlstm":
+            out = dict(mixer="matrix_memory", memory_heads=int(mix["heads"]), memory_key_dim=int(mix["dim"]),
+                       memory_value_dim=int(mix["vdim"]), memory_gate_cap=float(mix["gate_cap"]))
+        else:
+            raise ValueError(f"layer {i}: unknown mixer type {kind!r}")
+        if mlp and mlp.get("kind", "moe") != "moe":
+            raise ValueError(f"layer {i}: unknown feed-forward kind {mlp['kind']!r}")
+        out.update(ffn_hidden_size=0)
+        if mlp:
+            r, e = mlp["router"], mlp["expert"]
+            if not 1 <= int(r["top"]) <= int(r["experts"]):
+                raise ValueError(f"layer {i}: {r['top']} of {r['experts']} experts")
+            out.update(num_moe_experts=int(r["experts"]), moe_router_topk=int(r["top"]), moe_ffn_hidden_size=int(e["ff"]))
+        return out
+
+    def to_transformer_dict(self) -> dict:
+        d = {k: v for k, v in self.to_dict().items()
+             if k not in ("architecture", "layers", "norm", "vocab", "width", "embedding", "loop", "mlp", "mixer")}
+        fields = [self._layer_fields(i, layer) for i, layer in enumerate(self.layers)]
+        d.setdefault("seq_length", 32768)                      # position vectors have no longest position: a bound for buffers
+        d.setdefault("max_position_embeddings", d["seq_length"])
+        moe = [1 if f.get("num_moe_experts") else 0 for f in fields]
+        own = dict(num_attention_heads=1, num_query_groups=1, kv_channels=1, ffn_hidden_size=0)       # layers without attention
+        for f in fields:                                       # the stack's own view of what its layers override
+            own.update({k: v for k, v in f.items() if k in own and k != "ffn_hidden_size"})
+        if any(moe):
+            own.update({k: v for k, v in fields[moe.index(1)].items() if k.startswith(("num_moe", "moe_"))}, moe_layer_freq=moe)
+        loop = self.loop
+        own.update(vocab_size=int(self.vocab), hidden_size=int(self.width), num_layers=len(fields), layer_overrides=fields,
+                   layer_loop=(int(loop["start"]), int(loop["stop"]), int(loop["times"])) if loop else None,
+                   layernorm_epsilon=float(self.norm["eps"]), normalization="RMSNorm", layernorm_zero_centered_gamma=True,
+                   norm_placement="both", token_shift=True, fp32_residual_connection=True, ragged_attention=True, rotary_dim=0,
+                   position_embedding_type="sinusoidal", embedding_scale=float(self.embedding["scale"]),
+                   moe_router_score_function="softmax", norm_topk_prob=True, moe_router_logit_bias=True,
+                   moe_router_topk_scaling_factor=1.0, tie_word_embeddings=False)
+        d = {k: v for k, v in d.items() if ALIASES.get(k, (k,))[0] not in own}
+        return dict(d, **own)
+
+
 for _legacy in (True, False):
+    MindFormerRegister.register_cls(GavatarConfig, MindFormerModuleType.CONFIG, alias="GavatarConfig", legacy=_legacy)
     MindFormerRegister.register_cls(KukupelConfig, MindFormerModuleType.CONFIG, alias="KukupelConfig", legacy=_legacy)
     MindFormerRegister.register_cls(MefesunConfig, MindFormerModuleType.CONFIG, alias="MefesunConfig", legacy=_legacy)
 
@@ -341,6 +427,11 @@ KukupelForCausalLM = _model("KukupelForCausalLM", KukupelConfig, "kukupel")
 KukupelForCausalLM.kernel_sources = ("host_util", "elementwise", "gemm_tcgen05", "gemm_tcgen05_2cta", "gemm_bf16_decode",
                                      "residual_streams", "delta_rule", "qkv_rope_cache", "paged_prefill_tc", "paged_decode_tc",
                                      "paged_attention", "paged_attention_any", "router", "moe_ep", "moe_any", "decode_loop")
+GavatarForCausalLM = _model("GavatarForCausalLM", GavatarConfig, "gavatar")
+GavatarForCausalLM.kernel_sources = ("host_util", "elementwise", "gemm_tcgen05", "gemm_tcgen05_2cta", "gemm_bf16_decode",
+                                     "sandwich_norm", "head_mix", "matrix_memory", "qkv_rope_cache", "paged_prefill_tc",
+                                     "paged_decode_tc", "paged_attention", "paged_attention_any", "latent_decode", "router", "moe_ep",
+                                     "moe_any", "decode_loop")
 ChatGLM2ForConditionalGeneration = _model("ChatGLM2ForConditionalGeneration", ChatGLM4Config, "glm")
 
 def _backbone(name, causal_cls):
@@ -411,5 +502,6 @@ MODEL_TYPE_TO_CLASSES = {
     "qwen2_moe": (Qwen2MoeConfig, Qwen2MoeForCausalLM),
     "telechat": (TelechatConfig, TelechatForCausalLM), "glm": (ChatGLM4Config, ChatGLM2ForConditionalGeneration),
     "mefesun": (MefesunConfig, MefesunForCausalLM), "kukupel": (KukupelConfig, KukupelForCausalLM),
+    "gavatar": (GavatarConfig, GavatarForCausalLM),
     "chatglm": (ChatGLM4Config, ChatGLM2ForConditionalGeneration),
 }

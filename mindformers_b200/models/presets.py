@@ -68,6 +68,15 @@ PRESETS = {
                      mlp=dict(kind="moe", router=dict(experts=8, top=2), expert=dict(ff=256, limit=7.0))),
                 dict(type="delta", mixer=dict(heads=4, kv_heads=2, dim=64, vdim=64, conv=4),
                      mlp=dict(kind="moe", router=dict(experts=8, top=2), expert=dict(ff=256, limit=7.0)))]),
+    "tiny_gavatar": dict(
+        model_type="gavatar", vocab=1024, width=256, norm=dict(eps=1e-6), embedding=dict(scale=8.0), loop=dict(start=0, stop=2, times=2),
+        layers=[dict(type="latent_attention",
+                     mixer=dict(heads=4, dim=64, vdim=64, q_rank=96, kv_rank=160, scale=0.125, mask=dict(size=128)),
+                     mlp=dict(kind="moe", router=dict(experts=8, top=2), expert=dict(ff=256))),
+                dict(type="mlstm", mixer=dict(heads=4, dim=32, vdim=64, gate_cap=15.0),
+                     mlp=dict(kind="moe", router=dict(experts=8, top=2), expert=dict(ff=256))),
+                dict(type="attention", mixer=dict(heads=8, kv_heads=2, dim=32, vdim=32, scale=32 ** -0.5, mask=dict(size=128)),
+                     mlp=dict(kind="moe", router=dict(experts=8, top=2), expert=dict(ff=256)))]),
     "tiny_llama": dict(
         model_type="llama", num_hidden_layers=2, hidden_size=256, num_attention_heads=4, num_key_value_heads=2,
         intermediate_size=688, vocab_size=1024, rms_norm_eps=1e-5, rope_theta=10000.0,

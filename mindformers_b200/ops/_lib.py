@@ -140,19 +140,30 @@ def _declare(lib):
     sig("mfb_gemm_w8a8", [P, P, P, P, P, P, I, I, I, L, L, L, P, P])
     sig("mfb_quant_act_int8", [P, L, P, L, P, P, L, I, P])
     sig("mfb_paged_decode_tc_supported_ex", [I, I, I, I, I])
-    sig("mfb_paged_decode_attention_tc_ex", [P] * 9 + [I] * 11 + [F, F, L, F, P, P])
+    sig("mfb_paged_decode_attention_tc_ex", [P] * 9 + [I] * 13 + [F, F, L, F, P, P])
     sig("mfb_paged_prefill_tc_supported", [I, I, I, I, I])
-    sig("mfb_paged_prefill_tc", [P, P, P, P, I, I, P, P, P] + [I] * 9 + [F, F, L, F, P, P])
-    sig("mfb_paged_attention_any", [P] * 8 + [I] * 9 + [F, F, L, F, I, P])
+    sig("mfb_paged_prefill_tc", [P, P, P, P, I, I, P, P, P] + [I] * 11 + [L, L, F, F, L, F, P, P])
+    sig("mfb_paged_attention_any", [P] * 8 + [I] * 11 + [F, F, L, F, I, P])
     sig("mfb_residual_streams", [P, I, P, L, P, P, P, P, P, P, I, I, I, F, I, P])
+    sig("mfb_embed_stream", [P, P, P, P, P, I, I, I, F, I, P])
+    sig("mfb_normed_step", [P, P, L] + [P] * 11 + [I] * 4 + [F, I, P])
+    sig("mfb_latent_norm_cache", [P, L, P, P, F, P, P, P, I, I, I, I, P])
+    sig("mfb_gate_heads", [P, L, P, L, I, I, I, I, P])
+    sig("mfb_talk_mix", [P, P, P, L, P, I, I, I, I, I, P])
+    sig("mfb_matrix_memory_scratch_floats", [I] * 5, L)
+    sig("mfb_matrix_memory", [P, L] + [P] * 11 + [I] * 6 + [F, F, I, P])
+    sig("mfb_latent_decode_supported", [I, I])
+    sig("mfb_latent_decode_splits", [I, I, I])
+    sig("mfb_latent_decode_scratch_bytes", [I] * 4, L)
+    sig("mfb_latent_decode", [P] * 7 + [I] * 8 + [F, P, P])
     sig("mfb_delta_decode_supported", [I, I])
     sig("mfb_delta_scratch_floats", [I] * 6, L)
     sig("mfb_delta_rule", [P, L, P, P, L, P, L] + [P] * 11 + [L] + [I] * 9 + [F, F, I, P])
-    sig("mfb_clamped_glu", [P, P, I, I, F, F, P, P, P, P, I, P])
+    sig("mfb_clamped_glu", [P, P, I, I, F, F, F, P, P, P, P, I, P])
     sig("mfb_moe_scatter_any", [P] * 7 + [I] * 5 + [P])
     sig("mfb_moe_gather_any", [P] * 4 + [I] * 4 + [P])
     sig("mfb_grouped_gemm_any", [P, P, P, I, I, I, P, P, P, P, I, P])
-    sig("mfb_qkv_rope_cache", [P, L, P, P, P, F, P, F, I, I, P, P, P, P, P, I, I, I, I, I, I, P])
+    sig("mfb_qkv_rope_cache", [P, L, P, P, P, F, P, F, I, I, P, P, P, P, P, I, I, I, I, I, I, I, P])
     sig("mfb_add_normed", [P, L, P, P, P, P, P, I, P, P, I, I, I, F, I, P])
     sig("mfb_norm_stream", [P, P, P, P, I, I, I, F, I, P])
     sig("mfb_relu2", [P, P, L, I, L, I, P])

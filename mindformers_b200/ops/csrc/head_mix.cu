@@ -1,0 +1,181 @@
+// Small steps around attention (sm_100a, bf16 or fp32):
+//
+//   latent_norm_cache:  RMS norms of the query latent and of the key / value latent, the latter into the paged cache
+//   gate_heads:         x <- x * sigmoid(gate), a gate per column or per group of neighbouring columns
+//   talk_mix:           softmax weights mixed over heads, after the products with the values: head h of the result is
+//                       sum_g talk[h, g] o[g, own key / value head of h], times sigmoid(gate)
+#include "common.cuh"
+
+namespace mfb {
+namespace hmx {
+
+__device__ __forceinline__ float ld(const float* p) { return *p; }
+__device__ __forceinline__ float ld(const __nv_bfloat16* p) { return __bfloat162float(*p); }
+__device__ __forceinline__ void st(float* p, float v) { *p = v; }
+__device__ __forceinline__ void st(__nv_bfloat16* p, float v) { *p = __float2bfloat16_rn(v); }
+__device__ __forceinline__ float2 ld2(const float* p) { return *reinterpret_cast<const float2*>(p); }
+__device__ __forceinline__ float2 ld2(const __nv_bfloat16* p) { return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p)); }
+__device__ __forceinline__ void st2(float* p, float a, float b) { *reinterpret_cast<float2*>(p) = make_float2(a, b); }
+__device__ __forceinline__ void st2(__nv_bfloat16* p, float a, float b) { *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(a, b); }
+__device__ __forceinline__ float sigmoid(float z) { return 1.f / (1.f + __expf(-z)); }
+
+// one CTA of two warpgroups' worth of warps per token: the first half norms the query latent, the second the other one
+template <typename T>
+__global__ void __launch_bounds__(256)
+latent_norm_cache_kernel(const T* __restrict__ proj, long long ld_proj, const T* __restrict__ q_norm, const T* __restrict__ kv_norm,
+                         float eps, const int* __restrict__ slots, T* __restrict__ q, T* __restrict__ cache, int Q, int R) {
+  __shared__ float red[8];
+  const long long t = blockIdx.x;
+  const int half = threadIdx.x >> 7, tid = threadIdx.x & 127;
+  const int n = half ? R : Q;
+  const T* src = proj + t * ld_proj + (half ? Q : 0);
+  float ss = 0.f;
+  for (int i = tid; i < n; i += 128) {
+    const float v = ld(src + i);
+    ss = fmaf(v, v, ss);
+  }
+  ss = warp_sum(ss);
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
+  __syncthreads();
+  const float* r = red + half * 4;
+  const float rstd = 1.f / sqrtf(((r[0] + r[1]) + (r[2] + r[3])) / n + eps);
+  const int slot = slots[t];
+  if (half && slot < 0) return;
+  const T* w = half ? kv_norm : q_norm;
+  T* dst = half ? cache + (long long)slot * R : q + t * Q;
+  for (int i = tid; i < n; i += 128) st(dst + i, ld(src + i) * rstd * ld(w + i));
+}
+
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256)
+gate_heads_kernel(T* __restrict__ x, long long ld_x, const T* __restrict__ gate, long long ld_g, long long T_rows, int n, int per) {
+  const int nv = n / VEC;
+  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < T_rows * nv; i += (long long)gridDim.x * blockDim.x) {
+    const long long t = i / nv;
+    const int c = (int)(i % nv) * VEC;
+    T* p = x + t * ld_x + c;
+    const T* g = gate + t * ld_g;
+    if constexpr (VEC == 2) {
+      const float2 v = ld2(p);
+      st2(p, v.x * sigmoid(ld(g + c / per)), v.y * sigmoid(ld(g + (c + 1) / per)));
+    } else {
+      st(p, ld(p) * sigmoid(ld(g + c / per)));
+    }
+  }
+}
+
+constexpr int kAcc = 8;
+
+// a thread keeps up to eight result heads of one key / value head for VEC columns; the matrix lies in shared memory
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256)
+talk_mix_kernel(const T* __restrict__ o, const float* __restrict__ talk, const T* __restrict__ gate, long long ld_g, T* __restrict__ y,
+                int H, int G, int DV, int in_smem) {
+  extern __shared__ float sh[];
+  const long long t = blockIdx.x;
+  if (in_smem) {
+    for (int i = threadIdx.x; i < H * H; i += blockDim.x) sh[i] = talk[i];
+    __syncthreads();
+  }
+  const float* tm = in_smem ? sh : talk;
+  const int group = H / G, blocks = (group + kAcc - 1) / kAcc, nv = DV / VEC;
+  const T* src = o + t * H * G * DV;
+  for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < G * blocks * nv; i += gridDim.y * blockDim.x) {
+    const int d = (i % nv) * VEC, kb = i / nv, kv = kb / blocks, h0 = kv * group + (kb % blocks) * kAcc;
+    const int m = min(kAcc, kv * group + group - h0);
+    float acc[kAcc][VEC];
+#pragma unroll
+    for (int j = 0; j < kAcc; ++j)
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) acc[j][e] = 0.f;
+    for (int g = 0; g < H; ++g) {
+      float v[VEC];
+      const T* p = src + ((long long)g * G + kv) * DV + d;
+      if constexpr (VEC == 2) { const float2 f = ld2(p); v[0] = f.x; v[1] = f.y; }
+      else v[0] = ld(p);
+#pragma unroll
+      for (int j = 0; j < kAcc; ++j)
+        if (j < m) {
+          const float w = tm[(h0 + j) * H + g];
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) acc[j][e] = fmaf(w, v[e], acc[j][e]);
+        }
+    }
+#pragma unroll
+    for (int j = 0; j < kAcc; ++j)
+      if (j < m) {
+        const long long col = (long long)(h0 + j) * DV + d;
+        float r[VEC];
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) r[e] = gate ? acc[j][e] * sigmoid(ld(gate + t * ld_g + col + e)) : acc[j][e];
+        T* dst = y + t * H * DV + col;
+        if constexpr (VEC == 2) st2(dst, r[0], r[1]);
+        else st(dst, r[0]);
+      }
+  }
+}
+
+bool al(const void* p, int n) { return (reinterpret_cast<uintptr_t>(p) & (n - 1)) == 0; }
+
+}  // namespace hmx
+}  // namespace mfb
+
+extern "C" {
+using namespace mfb;
+
+// proj [T, >= Q + R] (rows ld_proj apart): query latent | key / value latent; q [T, Q]; cache rows [.., R] at slots[t] (< 0: not
+// written). f32 = 1: all fp32, else bf16.
+int mfb_latent_norm_cache(const void* proj, long long ld_proj, const void* q_norm, const void* kv_norm, float eps, const int* slots,
+                          void* q, void* cache, int T, int Q, int R, int f32, cudaStream_t stream) {
+  if (T <= 0) return 0;
+  if (Q < 1 || R < 1 || ld_proj < Q + R) { mfb_host::set_error("latent_norm_cache: Q=%d R=%d", Q, R); return 1; }
+  using bf = __nv_bfloat16;
+  if (f32) hmx::latent_norm_cache_kernel<float><<<T, 256, 0, stream>>>((const float*)proj, ld_proj, (const float*)q_norm, (const float*)kv_norm, eps, slots, (float*)q, (float*)cache, Q, R);
+  else hmx::latent_norm_cache_kernel<bf><<<T, 256, 0, stream>>>((const bf*)proj, ld_proj, (const bf*)q_norm, (const bf*)kv_norm, eps, slots, (bf*)q, (bf*)cache, Q, R);
+  return cudaGetLastError() == cudaSuccess ? 0 : 2;
+}
+
+// x [T, n] *= sigmoid(gate [T, m]) with m a divisor of n: n / m neighbouring columns share a gate.
+int mfb_gate_heads(void* x, long long ld_x, const void* gate, long long ld_g, int T, int n, int m, int f32, cudaStream_t stream) {
+  if (T <= 0) return 0;
+  if (n < 1 || m < 1 || n % m) { mfb_host::set_error("gate_heads: n=%d m=%d", n, m); return 1; }
+  const bool vec = n % 2 == 0 && ld_x % 2 == 0 && hmx::al(x, f32 ? 8 : 4);
+  const long long items = (long long)T * (vec ? n / 2 : n);
+  const long long want = (items + 255) / 256;
+  const int grid = (int)(want < 148 * 16 ? want : 148 * 16);
+  using bf = __nv_bfloat16;
+  const int per = n / m;
+  if (f32) {
+    if (vec) hmx::gate_heads_kernel<float, 2><<<grid, 256, 0, stream>>>((float*)x, ld_x, (const float*)gate, ld_g, T, n, per);
+    else hmx::gate_heads_kernel<float, 1><<<grid, 256, 0, stream>>>((float*)x, ld_x, (const float*)gate, ld_g, T, n, per);
+  } else {
+    if (vec) hmx::gate_heads_kernel<bf, 2><<<grid, 256, 0, stream>>>((bf*)x, ld_x, (const bf*)gate, ld_g, T, n, per);
+    else hmx::gate_heads_kernel<bf, 1><<<grid, 256, 0, stream>>>((bf*)x, ld_x, (const bf*)gate, ld_g, T, n, per);
+  }
+  return cudaGetLastError() == cudaSuccess ? 0 : 2;
+}
+
+// o [T, H, G, DV], talk [H, H] fp32, gate [T, H DV] (rows ld_g apart) or null -> y [T, H DV].
+int mfb_talk_mix(const void* o, const float* talk, const void* gate, long long ld_g, void* y, int T, int H, int G, int DV, int f32,
+                 cudaStream_t stream) {
+  if (T <= 0) return 0;
+  if (G < 1 || H < 1 || H % G || DV < 1) { mfb_host::set_error("talk_mix: H=%d G=%d DV=%d", H, G, DV); return 1; }
+  const bool vec = DV % 2 == 0 && hmx::al(o, f32 ? 8 : 4) && hmx::al(y, f32 ? 8 : 4);
+  const int in_smem = (size_t)H * H * 4 <= 48 * 1024;
+  const size_t smem = in_smem ? (size_t)H * H * 4 : 0;
+  const int items = G * ((H / G + hmx::kAcc - 1) / hmx::kAcc) * (vec ? DV / 2 : DV);
+  int gy = 1;
+  while ((long long)T * gy < 148 * 4 && gy * 256 < items) ++gy;
+  const dim3 grid(T, gy);
+  using bf = __nv_bfloat16;
+  if (f32) {
+    if (vec) hmx::talk_mix_kernel<float, 2><<<grid, 256, smem, stream>>>((const float*)o, talk, (const float*)gate, ld_g, (float*)y, H, G, DV, in_smem);
+    else hmx::talk_mix_kernel<float, 1><<<grid, 256, smem, stream>>>((const float*)o, talk, (const float*)gate, ld_g, (float*)y, H, G, DV, in_smem);
+  } else {
+    if (vec) hmx::talk_mix_kernel<bf, 2><<<grid, 256, smem, stream>>>((const bf*)o, talk, (const bf*)gate, ld_g, (bf*)y, H, G, DV, in_smem);
+    else hmx::talk_mix_kernel<bf, 1><<<grid, 256, smem, stream>>>((const bf*)o, talk, (const bf*)gate, ld_g, (bf*)y, H, G, DV, in_smem);
+  }
+  return cudaGetLastError() == cudaSuccess ? 0 : 2;
+}
+
+}  // extern "C"

@@ -1,0 +1,420 @@
+// Decode attention over a paged cache of latents, keys and values at once (sm_100a, tcgen05 + TMA), with an optional sliding
+// window and softmax sink. The factors that make keys and values of a latent are absorbed into query and result, so that one
+// decode step is, per sequence and head h with q, c of `rank` numbers (a multiple of 8 up to 512):
+//     s[t]   = scale * <q[h], c[t]>                       max(0, len - window) <= t < len
+//     o[h,:] = sum_t softmax(s)[t] * c[t]                 the sink is one more term of the softmax's denominator
+// The layout is that of mla_decode.cu, which serves one fixed latent width beside rotated columns: a CTA handles (split of the
+// sequence, 16 heads, sequence), the products are transposed so that the tokens fill the 128 rows of the tensor core, and a
+// tile of 128 tokens streams twice through a ring of 32 KB slots (128 latent columns each, the last one possibly half), once
+// for S^T and once, from L2, for O^T. Columns past the rank are zero fill in both operands; the rows of O^T that belong to
+// them are not stored. Two CTAs share an SM.
+//
+// Roles (192 threads): warp 0 TMA producer (block-table lookups), warp 1 MMA issuer + TMEM owner, warps 2..5 softmax / rescale /
+// epilogue. Every wait is bounded (common.cuh). The splits are merged by the combine kernel of paged_attention.cu.
+#include "common.cuh"
+
+namespace mfb {
+namespace latd {
+
+constexpr int kThreads = 192;
+constexpr int kTile = 128;              // tokens per tile
+constexpr int kHeads = 16;              // heads per CTA
+constexpr int kMaxRank = 512;
+constexpr int kSub = kTile * 128;       // [128 tokens][64 columns] swizzled sub-tile, 16 KB
+constexpr int kUnit = 2 * kSub;         // ring slot: a pair of sub-tiles (128 columns)
+constexpr int kSlots = 2;
+constexpr int kPBytes = 2 * kHeads * 128;   // P^T: two [16 heads][64 tokens] K-major sub-tiles
+constexpr int kTmemCols = 256;
+constexpr int kQSub = kHeads * 128;     // [16 heads][64 columns], 2 KB
+constexpr int kQBytes = kMaxRank / 64 * kQSub;
+constexpr float kRescale = 8.0f;
+
+struct Args {
+  const int* block_tables;   // [B, max_blocks]
+  const int* context_lens;   // [B]
+  int max_blocks, block_size, num_heads, splits, rank, window;
+  float scale_log2;
+  float* part_o;             // [B, num_heads, splits, rank] unnormalised
+  float* part_ml;            // [B, num_heads, splits, 2]: running max (log2 units), sum
+  int* status;
+};
+
+__device__ __forceinline__ float ex2(float x) {
+  float y;
+  asm volatile("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
+__global__ void __launch_bounds__(kThreads, 2)
+latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmC, const Args args) {
+  extern __shared__ uint8_t smem_raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) &
+                                             ~static_cast<uintptr_t>(1023));
+  uint8_t* sRing = smem;                               // 2 x 32 KB
+  uint8_t* sP = sRing + kSlots * kUnit;          // 4 KB
+  uint8_t* sQ = sP + kPBytes;                       // 18 KB
+  float* red = reinterpret_cast<float*>(sQ + kQBytes);          // [4 warps][16]
+  uint64_t* bars = reinterpret_cast<uint64_t*>(red + 4 * kHeads);
+  uint64_t* q_full = bars;                  // 1
+  uint64_t* full = bars + 1;                // up to 5
+  uint64_t* empty = bars + 6;               // up to 5
+  uint64_t* s_full = bars + 11;             // 2
+  uint64_t* s_empty = bars + 13;            // 2
+  uint64_t* p_ready = bars + 15;            // 1
+  uint64_t* pv_done = bars + 16;            // 1
+  uint32_t* tmem_holder = reinterpret_cast<uint32_t*>(bars + 17);
+  volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_holder + 1);
+
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int split = blockIdx.x, chunk = blockIdx.y, b = blockIdx.z;
+  const int len = args.context_lens[b];
+  const int first_tok = args.window > 0 && len > args.window ? len - args.window : 0;
+  const int base_tile = first_tok / kTile;
+  const int n_tiles_all = (len + kTile - 1) / kTile - base_tile;
+  const int per = (n_tiles_all + args.splits - 1) / args.splits;
+  const int rel0 = split * per;
+  const int rel1 = (rel0 + per < n_tiles_all) ? rel0 + per : n_tiles_all;
+  const int n_tiles = rel1 > rel0 ? rel1 - rel0 : 0;
+  const int t0 = base_tile + rel0;
+  const int head0 = chunk * kHeads;
+  const int subs = (args.rank + 63) / 64, units = (subs + 1) / 2;      // 64-column sub-tiles, pairs of them
+
+  if (threadIdx.x == 0) {
+    *abort_flag = 0;
+    mbar_init(smem_u32(q_full), 1);
+    for (int s = 0; s < kSlots; ++s) {
+      mbar_init(smem_u32(&full[s]), 1);
+      mbar_init(smem_u32(&empty[s]), 1);
+    }
+    for (int s = 0; s < 2; ++s) {
+      mbar_init(smem_u32(&s_full[s]), 1);
+      mbar_init(smem_u32(&s_empty[s]), 128);
+    }
+    mbar_init(smem_u32(p_ready), 128);
+    mbar_init(smem_u32(pv_done), 1);
+    fence_barrier_init();
+    tma_prefetch_desc(&tmQ);
+    tma_prefetch_desc(&tmC);
+  }
+  if (warp == 1) {
+    tmem_alloc(smem_u32(tmem_holder), kTmemCols);
+    tmem_relinquish();
+  }
+  fence_proxy_async_smem();
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem_base = *tmem_holder;
+  const uint32_t tmem_O = tmem_base;              // 4 blocks of 16 columns, 32 apart
+  const uint32_t tmem_S = tmem_base + 128;        // 2 buffers of 16 columns, 32 apart
+
+  if (warp == 0) {
+    // ------------------------------------ producer ------------------------------------
+    if (lane == 0 && n_tiles > 0) {
+      const uint32_t qb = smem_u32(q_full);
+      mbar_expect_tx(qb, subs * kQSub);
+      for (int c = 0; c < subs; ++c)
+        tma_load_2d(smem_u32(sQ) + c * kQSub, &tmQ, qb, c * 64, b * args.num_heads + head0);
+      const int bs = args.block_size;
+      const int pages = kTile / bs;            // pages per tile (block_size divides 128)
+      const int* table = args.block_tables + static_cast<size_t>(b) * args.max_blocks;
+      uint32_t unit = 0;
+      bool ok = true;
+      for (int j = 0; j < n_tiles && ok; ++j) {
+        const int tok0 = (t0 + j) * kTile;
+        int page_row[8];
+        const int first_page = table[tok0 / bs];
+        for (int i = 0; i < pages; ++i) {
+          // pages past the end of the sequence may be unallocated: read the tile's first page instead (masked)
+          int pg = (tok0 + i * bs < len) ? table[tok0 / bs + i] : first_page;
+          if (pg < 0) pg = first_page;
+          page_row[i] = pg * bs;
+        }
+        // two passes over the tile's pairs: for S^T, then again for O^T
+        for (int u = 0; u < 2 * units && ok; ++u) {
+          const int slot = unit % kSlots;
+          const uint32_t ph = (unit / kSlots) & 1;
+          ok = mbar_wait(smem_u32(&empty[slot]), ph ^ 1, abort_flag, args.status, kStatusWaitTimeoutProducer);
+          if (!ok) break;
+          const uint32_t fb = smem_u32(&full[slot]);
+          const uint32_t dst = smem_u32(sRing + slot * kUnit);
+          const int pair = u < units ? u : u - units;
+          const bool two = 2 * pair + 1 < subs;
+          const int col0 = pair * 128;
+          mbar_expect_tx(fb, two ? kUnit : kSub);
+          for (int i = 0; i < pages; ++i) {
+            tma_load_2d(dst + i * bs * 128, &tmC, fb, col0, page_row[i]);
+            if (two) tma_load_2d(dst + kSub + i * bs * 128, &tmC, fb, col0 + 64, page_row[i]);
+          }
+          ++unit;
+        }
+      }
+    }
+    __syncwarp();
+  } else if (warp == 1) {
+    // ------------------------------------ MMA issuer ------------------------------------
+    if (lane == 0 && n_tiles > 0) {
+      constexpr uint32_t IDESC_S = umma_idesc_bf16(kTile, kHeads, 0, 0);   // A = cache K-major, B = Q K-major
+      constexpr uint32_t IDESC_PV = umma_idesc_bf16(kTile, kHeads, 1, 0);  // A = cache MN-major, B = P^T K-major
+      bool ok = mbar_wait(smem_u32(q_full), 0, abort_flag, args.status, kStatusWaitTimeoutMma);
+      const uint32_t qa = smem_u32(sQ), pa = smem_u32(sP);
+      uint32_t unit = 0;
+      for (int j = 0; j < n_tiles && ok; ++j) {
+        const int sb = j & 1;
+        const uint32_t sph = (j >> 1) & 1;
+        ok = mbar_wait(smem_u32(&s_empty[sb]), sph ^ 1, abort_flag, args.status, kStatusWaitTimeoutMma);
+        if (!ok) break;
+        // ---- S^T = C . Q^T over the pairs of the first pass ----
+        for (int u = 0; u < units && ok; ++u) {
+          const int slot = unit % kSlots;
+          const uint32_t ph = (unit / kSlots) & 1;
+          ok = mbar_wait(smem_u32(&full[slot]), ph, abort_flag, args.status, kStatusWaitTimeoutMma);
+          if (!ok) break;
+          tc_fence_after();
+          const uint32_t ca = smem_u32(sRing + slot * kUnit);
+          const int ksteps = 2 * u + 1 < subs ? 8 : 4;
+          const int qsub0 = 2 * u;
+#pragma unroll
+          for (int k = 0; k < 8; ++k) {
+            if (k < ksteps) {
+              const uint64_t a_desc = umma_desc_kmajor_sw128(ca + (k >> 2) * kSub + (k & 3) * 32);
+              const uint64_t b_desc = umma_desc_kmajor_sw128(qa + (qsub0 + (k >> 2)) * kQSub + (k & 3) * 32);
+              umma_f16_ss(tmem_S + sb * 32, a_desc, b_desc, IDESC_S, (u > 0 || k > 0) ? 1u : 0u);
+            }
+          }
+          umma_commit(smem_u32(&empty[slot]));
+          ++unit;
+        }
+        if (!ok) break;
+        umma_commit(smem_u32(&s_full[sb]));
+        // ---- O^T += C^T . P^T over the pairs of the second pass ----
+        ok = mbar_wait(smem_u32(p_ready), j & 1, abort_flag, args.status, kStatusWaitTimeoutMma);
+        if (!ok) break;
+        for (int m = 0; m < units && ok; ++m) {
+          const int slot = unit % kSlots;
+          const uint32_t ph = (unit / kSlots) & 1;
+          ok = mbar_wait(smem_u32(&full[slot]), ph, abort_flag, args.status, kStatusWaitTimeoutMma);
+          if (!ok) break;
+          tc_fence_after();
+          const uint32_t ca = smem_u32(sRing + slot * kUnit);
+#pragma unroll
+          for (int k = 0; k < kTile / 16; ++k) {
+            const uint64_t a_desc = umma_desc_mnmajor_sw128(ca + k * 16 * 128, kSub);
+            const uint64_t b_desc = umma_desc_kmajor_sw128(pa + (k >> 2) * (kHeads * 128) + (k & 3) * 32);
+            umma_f16_ss(tmem_O + m * 32, a_desc, b_desc, IDESC_PV, (j > 0 || k > 0) ? 1u : 0u);
+          }
+          umma_commit(smem_u32(&empty[slot]));
+          ++unit;
+        }
+        if (!ok) break;
+        umma_commit(smem_u32(pv_done));
+      }
+    }
+    __syncwarp();
+  } else {
+    // ------------------------------------ softmax / epilogue ------------------------------------
+    const int ew = warp & 3;
+    const int row = ew * 32 + lane;                 // token row of S^T, dv row of O^T
+    const uint32_t lane_base = static_cast<uint32_t>(ew * 32) << 16;
+    float m_used[kHeads], l_part[kHeads];
+#pragma unroll
+    for (int h = 0; h < kHeads; ++h) { m_used[h] = -INFINITY; l_part[h] = 0.f; }
+    bool ok = true;
+    for (int j = 0; j < n_tiles; ++j) {
+      const int sb = j & 1;
+      const uint32_t sph = (j >> 1) & 1;
+      ok = mbar_wait(smem_u32(&s_full[sb]), sph, abort_flag, args.status, kStatusWaitTimeoutEpilogue);
+      ok = named_bar_and(2, 128, ok);
+      if (!ok) break;
+      tc_fence_after();
+      uint32_t sr[16];
+      tmem_ld_32x32b_x16(tmem_S + sb * 32 + lane_base, sr);
+      tmem_ld_wait();
+      tc_fence_before();
+      mbar_arrive(smem_u32(&s_empty[sb]));
+      float s[kHeads];
+      const int tok = (t0 + j) * kTile + row;
+      const bool valid = tok < len && tok >= first_tok;
+#pragma unroll
+      for (int h = 0; h < kHeads; ++h) s[h] = valid ? __uint_as_float(sr[h]) * args.scale_log2 : -INFINITY;
+      // per-head maximum over the 128 tokens of the tile
+#pragma unroll
+      for (int h = 0; h < kHeads; ++h) {
+        const float w = warp_max(s[h]);
+        if (lane == 0) red[ew * kHeads + h] = w;
+      }
+      named_bar_sync(1, 128);
+      float alpha[kHeads];
+      bool any_rescale = false;
+#pragma unroll
+      for (int h = 0; h < kHeads; ++h) {
+        const float mx = fmaxf(fmaxf(red[h], red[kHeads + h]), fmaxf(red[2 * kHeads + h], red[3 * kHeads + h]));
+        alpha[h] = 1.f;
+        if (m_used[h] == -INFINITY) {
+          m_used[h] = mx;                           // first tile with a valid token (nothing accumulated yet)
+        } else if (mx > m_used[h] + kRescale) {
+          alpha[h] = ex2(m_used[h] - mx);
+          m_used[h] = mx;
+          any_rescale = true;
+        }
+      }
+#pragma unroll
+      for (int h = 0; h < kHeads; ++h) {
+        const float neg_m = (m_used[h] == -INFINITY) ? 0.f : -m_used[h];
+        s[h] = valid ? ex2(s[h] + neg_m) : 0.f;
+        l_part[h] = l_part[h] * alpha[h] + s[h];
+      }
+      if (j > 0) {
+        // the previous O^T update has completed: P^T may be overwritten and O^T touched
+        ok = mbar_wait(smem_u32(pv_done), (j - 1) & 1, abort_flag, args.status, kStatusWaitTimeoutEpilogue);
+        if (ok && any_rescale) {
+          tc_fence_after();
+          for (int m = 0; m < units; ++m) {
+            uint32_t r[16];
+            tmem_ld_32x32b_x16(tmem_O + lane_base + m * 32, r);
+            tmem_ld_wait();
+#pragma unroll
+            for (int h = 0; h < kHeads; ++h) r[h] = __float_as_uint(__uint_as_float(r[h]) * alpha[h]);
+            tmem_st_32x32b_x16(tmem_O + lane_base + m * 32, r);
+          }
+          tmem_st_wait();
+        }
+      }
+      ok = named_bar_and(2, 128, ok);               // also orders the reads of `red` before the next tile's writes
+      if (!ok) break;
+      // P^T[h][token] as a K-major operand: sub-tile of 64 tokens, row h of 128 bytes, 16-byte chunks swizzled by row
+      {
+        uint8_t* pcol = sP + (row >> 6) * (kHeads * 128) + (row & 7) * 2;
+        const int chunk = (row & 63) >> 3;
+#pragma unroll
+        for (int h = 0; h < kHeads; ++h)
+          *reinterpret_cast<__nv_bfloat16*>(pcol + h * 128 + ((chunk ^ (h & 7)) << 4)) = __float2bfloat16_rn(s[h]);
+      }
+      fence_proxy_async_smem();
+      tc_fence_before();
+      mbar_arrive(smem_u32(p_ready));
+    }
+    if (ok && n_tiles > 0) {
+      ok = mbar_wait(smem_u32(pv_done), (n_tiles - 1) & 1, abort_flag, args.status, kStatusWaitTimeoutEpilogue);
+      ok = named_bar_and(2, 128, ok);
+    }
+    // per-head sums over the 128 token rows
+    float l_tot[kHeads];
+#pragma unroll
+    for (int h = 0; h < kHeads; ++h) {
+      const float w = warp_sum(l_part[h]);
+      if (lane == 0) red[ew * kHeads + h] = w;
+    }
+    named_bar_sync(1, 128);
+#pragma unroll
+    for (int h = 0; h < kHeads; ++h)
+      l_tot[h] = (red[h] + red[kHeads + h]) + (red[2 * kHeads + h] + red[3 * kHeads + h]);
+    const bool have = ok && n_tiles > 0;
+    const size_t first_row = static_cast<size_t>(b) * args.num_heads + head0;
+    if (row < kHeads && head0 + row < args.num_heads) {
+      float mh = -INFINITY, lh = 0.f;
+#pragma unroll
+      for (int h = 0; h < kHeads; ++h)
+        if (h == row) { mh = m_used[h]; lh = l_tot[h]; }
+      if (!have) { mh = -INFINITY; lh = 0.f; }
+      float* ml = args.part_ml + ((first_row + row) * args.splits + split) * 2;
+      ml[0] = mh;
+      ml[1] = lh;
+    }
+    if (have) tc_fence_after();
+    for (int m = 0; m < units; ++m) {
+      uint32_t r[16];
+      if (have) {
+        tmem_ld_32x32b_x16(tmem_O + lane_base + m * 32, r);
+        tmem_ld_wait();
+      }
+      const int col = m * 128 + row;
+#pragma unroll
+      for (int h = 0; h < kHeads; ++h)
+        if (head0 + h < args.num_heads && col < args.rank)      // a split without tokens writes zeros, which the merge weighs by zero
+          args.part_o[((first_row + h) * args.splits + split) * args.rank + col] = have ? __uint_as_float(r[h]) : 0.f;
+    }
+  }
+  tc_fence_before();
+  __syncthreads();
+  if (warp == 1) {
+    tc_fence_after();
+    tmem_dealloc(tmem_base, kTmemCols);
+  }
+}
+
+}  // namespace latd
+}  // namespace mfb
+
+extern "C" {
+using namespace mfb;
+
+int mfb_paged_combine_ex(const float* part_acc, const float* part_ml, void* out, int splits, int rows, int hd, int Hq,
+                         const int* cu_q, const float* sink, long long ld_out, float out_scale,
+                         cudaStream_t stream);      // paged_attention.cu
+
+int mfb_latent_decode_supported(int rank, int block_size) {
+  return rank >= 8 && rank <= latd::kMaxRank && rank % 8 == 0 &&
+                 (block_size == 16 || block_size == 32 || block_size == 64 || block_size == 128)
+             ? 1 : 0;
+}
+
+// Number of sequence splits that fills the GPU for a batch of B sequences of up to max_len visible tokens.
+int mfb_latent_decode_splits(int B, int num_heads, int max_len) {
+  // cost of a choice = waves of CTAs over the 2 x 148 resident CTAs x (tiles per CTA + about one tile of fixed work per CTA)
+  const int chunks = (num_heads + latd::kHeads - 1) / latd::kHeads;
+  const int tiles = (max_len + latd::kTile - 1) / latd::kTile;
+  int best = 1;
+  long long best_cost = -1;
+  for (int s = 1; s <= tiles && s <= 32; ++s) {
+    const long long ctas = static_cast<long long>(B) * chunks * s;
+    const long long waves = (ctas + 295) / 296;
+    const long long cost = waves * ((tiles + s - 1) / s + 1);
+    if (best_cost < 0 || cost < best_cost) { best_cost = cost; best = s; }
+  }
+  return best;
+}
+
+long long mfb_latent_decode_scratch_bytes(int B, int num_heads, int rank, int splits) {
+  return static_cast<long long>(B) * splits * num_heads * (rank + 2) * 4;
+}
+
+// q [B, num_heads, rank] (queries in latent space), cache [num_blocks, block_size, rank], out [B, num_heads, rank], all bf16;
+// block_tables [B, max_blocks]; context_lens [B] counts the tokens in the cache, the new one included; window > 0: only the last
+// `window` of them; sink [num_heads] fp32 or null; scratch: mfb_latent_decode_scratch_bytes.
+int mfb_latent_decode(const void* q, const void* cache, const int* block_tables, const int* context_lens, const float* sink, void* out,
+                      void* scratch, int splits, int B, int num_heads, int rank, int num_blocks, int block_size, int max_blocks,
+                      int window, float scale, int* status, cudaStream_t stream) {
+  if (!mfb_latent_decode_supported(rank, block_size) || num_heads < 1 || splits < 1 || num_blocks < 1 || max_blocks < 1) {
+    mfb_host::set_error("latent_decode: heads=%d rank=%d splits=%d block_size=%d", num_heads, rank, splits, block_size);
+    return 1;
+  }
+  if (B <= 0) return 0;
+  CUtensorMap tQ, tC;
+  int rc;
+  const CUtensorMapDataType BF = CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
+  if ((rc = mfb_host::make_tmap_2d(&tQ, q, 2, BF, (uint64_t)B * num_heads, rank, rank, latd::kHeads, 64))) return 20 + rc;
+  if ((rc = mfb_host::make_tmap_2d(&tC, cache, 2, BF, (uint64_t)num_blocks * block_size, rank, rank, block_size, 64))) return 30 + rc;
+  latd::Args a;
+  a.block_tables = block_tables; a.context_lens = context_lens; a.max_blocks = max_blocks; a.block_size = block_size;
+  a.num_heads = num_heads; a.splits = splits; a.rank = rank; a.window = window; a.scale_log2 = scale * 1.4426950408889634f;
+  a.part_o = reinterpret_cast<float*>(scratch);
+  a.part_ml = a.part_o + static_cast<size_t>(B) * splits * num_heads * rank;
+  a.status = status;
+  constexpr int SMEM = latd::kSlots * latd::kUnit + latd::kPBytes + latd::kQBytes + 4 * latd::kHeads * 4 + 18 * 8 + 16 + 1024;
+  static bool attr_set = false;
+  if (!attr_set) {
+    if (cudaFuncSetAttribute(latd::latent_decode_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM) != cudaSuccess) {
+      mfb_host::set_error("latent_decode: cannot raise shared memory limit");
+      return 10;
+    }
+    attr_set = true;
+  }
+  const dim3 grid(splits, (num_heads + latd::kHeads - 1) / latd::kHeads, B);
+  latd::latent_decode_kernel<<<grid, latd::kThreads, SMEM, stream>>>(tQ, tC, a);
+  if (cudaGetLastError() != cudaSuccess) { mfb_host::set_error("latent_decode: launch failed"); return 11; }
+  return mfb_paged_combine_ex(a.part_o, a.part_ml, out, splits, B * num_heads, rank, num_heads, nullptr, sink,
+                              (long long)num_heads * rank, 1.f, stream);
+}
+
+}  // extern "C"

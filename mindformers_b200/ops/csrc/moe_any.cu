@@ -1,7 +1,7 @@
 // Mixture-of-experts steps for every size and for bf16 or fp32 (sm_100a), on the permutation plan of moe_ep.cu (expert
 // segments padded to blocks of 128 rows):
 //
-//   clamped_glu:       y = g * sigmoid(alpha * g) * (u + 1) with g = min(x[:F], limit), u = clamp(x[F:], -limit, limit)
+//   clamped_glu:       y = g * sigmoid(alpha * g) * (u + shift) with g = min(x[:F], limit), u = clamp(x[F:], -limit, limit)
 //   scatter / gather:  rows of one rank, optionally weighted; the path of 32-bit models and of widths that are not a
 //                      multiple of 8
 //   grouped_gemm_any:  out[rows of expert e] = a[rows of expert e] W[e] with W [E, K, N], fp32 FMA: the path of 32-bit
@@ -31,16 +31,16 @@ __device__ __forceinline__ int rows_in_use(int blk, const int* block_group, cons
   return left < 0 ? 0 : (left > kBlock ? kBlock : left);
 }
 
-__device__ __forceinline__ float glu(float g, float u, float limit, float alpha) {
+__device__ __forceinline__ float glu(float g, float u, float limit, float alpha, float shift) {
   g = fminf(g, limit);
   u = fminf(fmaxf(u, -limit), limit);
-  return g / (1.f + __expf(-alpha * g)) * (u + 1.f);
+  return g / (1.f + __expf(-alpha * g)) * (u + shift);
 }
 
 // grid: (row block, column slice); VEC 8 (bf16, F % 8 == 0) or 1
 template <typename T, int VEC>
 __global__ void __launch_bounds__(256)
-clamped_glu_kernel(const T* __restrict__ x, T* __restrict__ y, int R, int F, float limit, float alpha,
+clamped_glu_kernel(const T* __restrict__ x, T* __restrict__ y, int R, int F, float limit, float alpha, float shift,
                    const int* __restrict__ block_group, const int* __restrict__ num_blocks, const int* __restrict__ offsets,
                    const int* __restrict__ fill) {
   int used = rows_in_use(blockIdx.x, block_group, num_blocks, offsets, fill);
@@ -60,11 +60,11 @@ clamped_glu_kernel(const T* __restrict__ x, T* __restrict__ y, int R, int F, flo
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
         const float2 g = __bfloat1622float2(ga[j]), u = __bfloat1622float2(ub[j]);
-        o[j] = pack_bf16x2(glu(g.x, u.x, limit, alpha), glu(g.y, u.y, limit, alpha));
+        o[j] = pack_bf16x2(glu(g.x, u.x, limit, alpha, shift), glu(g.y, u.y, limit, alpha, shift));
       }
       *reinterpret_cast<uint4*>(y + r * F + c) = make_uint4(o[0], o[1], o[2], o[3]);
     } else {
-      st(y + r * F + c, glu(ld(x + r * 2 * F + c), ld(x + r * 2 * F + F + c), limit, alpha));
+      st(y + r * F + c, glu(ld(x + r * 2 * F + c), ld(x + r * 2 * F + F + c), limit, alpha, shift));
     }
   }
 }
@@ -154,7 +154,7 @@ extern "C" {
 using namespace mfb;
 
 // x [R, 2 F] (gate | up) -> y [R, F]. block_group (with num_blocks) or null; offsets / fill or null: see rows_in_use.
-int mfb_clamped_glu(const void* x, void* y, int R, int F, float limit, float alpha, const int* block_group, const int* num_blocks,
+int mfb_clamped_glu(const void* x, void* y, int R, int F, float limit, float alpha, float shift, const int* block_group, const int* num_blocks,
                     const int* offsets, const int* fill, int f32, cudaStream_t stream) {
   if (R <= 0 || F <= 0) return 0;
   const int blocks = (R + many::kBlock - 1) / many::kBlock;
@@ -163,9 +163,9 @@ int mfb_clamped_glu(const void* x, void* y, int R, int F, float limit, float alp
   if (slices > 64) slices = 64;
   dim3 grid(blocks, (unsigned)slices);
   using bf = __nv_bfloat16;
-  if (f32) many::clamped_glu_kernel<float, 1><<<grid, 256, 0, stream>>>((const float*)x, (float*)y, R, F, limit, alpha, block_group, num_blocks, offsets, fill);
-  else if (vec) many::clamped_glu_kernel<bf, 8><<<grid, 256, 0, stream>>>((const bf*)x, (bf*)y, R, F, limit, alpha, block_group, num_blocks, offsets, fill);
-  else many::clamped_glu_kernel<bf, 1><<<grid, 256, 0, stream>>>((const bf*)x, (bf*)y, R, F, limit, alpha, block_group, num_blocks, offsets, fill);
+  if (f32) many::clamped_glu_kernel<float, 1><<<grid, 256, 0, stream>>>((const float*)x, (float*)y, R, F, limit, alpha, shift, block_group, num_blocks, offsets, fill);
+  else if (vec) many::clamped_glu_kernel<bf, 8><<<grid, 256, 0, stream>>>((const bf*)x, (bf*)y, R, F, limit, alpha, shift, block_group, num_blocks, offsets, fill);
+  else many::clamped_glu_kernel<bf, 1><<<grid, 256, 0, stream>>>((const bf*)x, (bf*)y, R, F, limit, alpha, shift, block_group, num_blocks, offsets, fill);
   return cudaGetLastError() == cudaSuccess ? 0 : 2;
 }
 

@@ -3,7 +3,8 @@
 //
 // A batch is ragged: sequence b brings the rows cu_q[b] .. cu_q[b + 1] - 1, its last tokens, which are already in the
 // cache; row r sits at position context_lens[b] - (cu_q[b + 1] - r). Keys are visible up to the row's own position, and
-// with `chunk` > 0 only inside the row's chunk of `chunk` positions counted from 0. `sink` [Hq] adds exp(sink_h) to the
+// with `chunk` > 0 only inside the row's chunk of `chunk` positions counted from 0, with `window` > 0 only the row's own and
+// the `window` - 1 before it. With `all_values` a head's weights are applied to the values of every KV head. `sink` [Hq] adds exp(sink_h) to the
 // softmax denominator of head h (no key, no value, not scaled). `softcap` > 0 bounds the scores: softcap * tanh(score / softcap).
 //
 // One CTA of four warps per (row, query head): a warp takes every fourth key, its lanes split the head dimension; the
@@ -27,7 +28,7 @@ __global__ void __launch_bounds__(kWarps * 32)
 paged_attention_any_kernel(const T* __restrict__ q, const T* __restrict__ key_cache, const T* __restrict__ value_cache,
                            const int* __restrict__ block_tables, const int* __restrict__ context_lens,
                            const int* __restrict__ cu_q, const float* __restrict__ sink, T* __restrict__ out, int B, int Hq,
-                           int Hkv, int D, int DV, int block_size, int max_blocks, int chunk, float scale, float softcap,
+                           int Hkv, int D, int DV, int block_size, int max_blocks, int chunk, int window, float scale, float softcap,
                            long long ld_out, float out_scale) {
   const int r = blockIdx.x, h = blockIdx.y;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -44,8 +45,9 @@ paged_attention_any_kernel(const T* __restrict__ q, const T* __restrict__ key_ca
     b = r;
     pos = context_lens[b] - 1;
   }
-  const int first = (chunk > 0 && pos >= 0) ? pos - pos % chunk : 0;
-  const int kvh = h / (Hq / Hkv);
+  int first = (chunk > 0 && pos >= 0) ? pos - pos % chunk : 0;
+  if (window > 0 && pos - window + 1 > first) first = pos - window + 1;
+  const int kvh = h / (Hq / Hkv), vheads = gridDim.z, vsel = blockIdx.z, vh = vheads > 1 ? vsel : kvh;
   const int* table = block_tables + (size_t)b * max_blocks;
   const T* qp = q + ((size_t)r * Hq + h) * D;
   float qr[N], acc[N];
@@ -73,7 +75,7 @@ paged_attention_any_kernel(const T* __restrict__ q, const T* __restrict__ key_ca
     const float alpha = expf(m - m_new), p = expf(s - m_new);
     l = l * alpha + p;
     m = m_new;
-    const T* vp = value_cache + (slot * Hkv + kvh) * DV;
+    const T* vp = value_cache + (slot * Hkv + vh) * DV;
 #pragma unroll
     for (int i = 0; i < N; ++i) {
       const int d = lane + 32 * i;
@@ -100,20 +102,20 @@ paged_attention_any_kernel(const T* __restrict__ q, const T* __restrict__ key_ca
     float num = 0.f;
 #pragma unroll
     for (int w = 0; w < kWarps; ++w) num += wgt[w] * sh_acc[w][d];
-    st(out + r * ld_out + (size_t)h * DV + d, num * inv);
+    st(out + r * ld_out + ((size_t)h * vheads + vsel) * DV + d, num * inv);
   }
 }
 
 template <typename T>
 int launch(const void* q, const void* kc, const void* vc, const int* bt, const int* cl, const int* cu, const float* sink,
-           void* out, int rows, int B, int Hq, int Hkv, int D, int DV, int bs, int mb, int chunk, float scale,
+           void* out, int rows, int B, int Hq, int Hkv, int D, int DV, int bs, int mb, int chunk, int window, int all_values, float scale,
            float softcap, long long ld_out, float out_scale, cudaStream_t stream) {
-  dim3 grid(rows, Hq);
+  dim3 grid(rows, Hq, all_values ? Hkv : 1);
   const int n = ((D > DV ? D : DV) + 31) / 32;
 #define MFB_PAA(N_)                                                                                                   \
   paged_attention_any_kernel<T, N_><<<grid, kWarps * 32, 0, stream>>>((const T*)q, (const T*)kc, (const T*)vc, bt, cl, \
                                                                       cu, sink, (T*)out, B, Hq, Hkv, D, DV, bs, mb,   \
-                                                                      chunk, scale, softcap, ld_out, out_scale)
+                                                                      chunk, window, scale, softcap, ld_out, out_scale)
   if (n <= 2) MFB_PAA(2); else if (n <= 4) MFB_PAA(4); else if (n <= 8) MFB_PAA(8); else MFB_PAA(16);
 #undef MFB_PAA
   if (cudaGetLastError() != cudaSuccess) { mfb_host::set_error("paged_attention_any: launch failed"); return 2; }
@@ -127,23 +129,24 @@ extern "C" {
 using namespace mfb;
 
 // q [rows, Hq, D], caches [num_blocks, block_size, Hkv, D | DV], out [rows, Hq, DV] (rows ld_out apart): fp32 (f32 = 1) or bf16. cu_q [B + 1]
-// (device) or null: one row per sequence. chunk <= 0: no chunks; sink: [Hq] fp32 or null. softcap > 0: scores become
+// (device) or null: one row per sequence. chunk <= 0: no chunks; window <= 0: no window; all_values: out [rows, Hq, Hkv, DV];
+// value_cache may be key_cache; sink: [Hq] fp32 or null. softcap > 0: scores become
 // softcap * tanh(score / softcap). Rows of out lie ld_out elements apart; the result is multiplied by out_scale.
 int mfb_paged_attention_any(const void* q, const void* key_cache, const void* value_cache, const int* block_tables,
                             const int* context_lens, const int* cu_q, const float* sink, void* out, int rows, int B, int Hq,
-                            int Hkv, int D, int DV, int block_size, int max_blocks, int chunk, float scale, float softcap,
-                            long long ld_out, float out_scale, int f32, cudaStream_t stream) {
+                            int Hkv, int D, int DV, int block_size, int max_blocks, int chunk, int window, int all_values, float scale,
+                            float softcap, long long ld_out, float out_scale, int f32, cudaStream_t stream) {
   if (rows <= 0 || B <= 0) return 0;
-  if (Hkv < 1 || Hq < 1 || Hq % Hkv || Hq > 65535 || D < 1 || DV < 1 || D > 32 * paa::kMaxPerLane ||
+  if (Hkv < 1 || Hq < 1 || Hq % Hkv || Hq > 65535 || Hkv > 65535 || D < 1 || DV < 1 || D > 32 * paa::kMaxPerLane ||
       DV > 32 * paa::kMaxPerLane || block_size < 1 || (!cu_q && rows != B)) {
     mfb_host::set_error("paged_attention_any: rows=%d B=%d Hq=%d Hkv=%d D=%d DV=%d block_size=%d", rows, B, Hq, Hkv, D, DV,
                         block_size);
     return 1;
   }
   return f32 ? paa::launch<float>(q, key_cache, value_cache, block_tables, context_lens, cu_q, sink, out, rows, B, Hq, Hkv, D,
-                                  DV, block_size, max_blocks, chunk, scale, softcap, ld_out, out_scale, stream)
+                                  DV, block_size, max_blocks, chunk, window, all_values, scale, softcap, ld_out, out_scale, stream)
              : paa::launch<__nv_bfloat16>(q, key_cache, value_cache, block_tables, context_lens, cu_q, sink, out, rows, B, Hq,
-                                          Hkv, D, DV, block_size, max_blocks, chunk, scale, softcap, ld_out, out_scale, stream);
+                                          Hkv, D, DV, block_size, max_blocks, chunk, window, all_values, scale, softcap, ld_out, out_scale, stream);
 }
 
 }  // extern "C"

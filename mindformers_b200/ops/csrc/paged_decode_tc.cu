@@ -2,7 +2,8 @@
 // size and value size up to 128 each (multiples of 8), grouped-query attention (16 query heads of a KV head per CTA).
 //
 // Cache layout: key_cache / value_cache [num_blocks, block_size, kv_heads, D | DV]; a sequence's blocks come from its
-// block table. With `chunk` > 0 only the keys of the query's own chunk of positions (counted from 0) are visited. The
+// block table. With `chunk` > 0 only the keys of the query's own chunk of positions (counted from 0) are visited, with `window`
+// > 0 only the last `window` ones; with `all_values` a query head's weights are applied to the values of every KV head. The
 // tiles are 128 columns wide: q's columns past D are zero fill, so what a K tile holds there does not count, and the
 // value columns past DV reach only result rows that are not stored; 64-column halves that hold no head column are not
 // loaded. A CTA handles (split of the sequence, KV head, sequence) and walks its tokens in tiles of 128. As in
@@ -46,11 +47,12 @@ struct Args {
   const int* context_lens;   // [B]
   const int* cu_q;           // [B + 1] or null: only sequences with exactly one new row are computed, q row cu_q[b]
   int max_blocks, block_size, num_q_heads, num_kv_heads, group, splits;
-  int D, DV, chunk, head_blocks;   // head_blocks: CTAs of up to 16 query heads per KV head
+  int D, DV, chunk, window, head_blocks;   // head_blocks: CTAs of up to 16 query heads per KV head
+  int vheads;                      // value heads per query head: 1 (its own) or all
   float scale_log2;
   float cap_log2, cap_scale;       // soft cap of the scores in log2 units (0: none) and scale / cap
-  float* part_acc;           // [B, Hq, splits, DV] unnormalised
-  float* part_ml;            // [B, Hq, splits, 2]: running max (log2 units), sum
+  float* part_acc;           // [B, Hq, vheads, splits, DV] unnormalised
+  float* part_ml;            // [B, Hq, vheads, splits, 2]: running max (log2 units), sum
   int* status;
 };
 
@@ -91,15 +93,17 @@ paged_decode_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int split = blockIdx.x, b = blockIdx.z;
-  const int kvh = static_cast<int>(blockIdx.y) / args.head_blocks, hb = static_cast<int>(blockIdx.y) % args.head_blocks;
+  const int vsel = static_cast<int>(blockIdx.y) % args.vheads, hy = static_cast<int>(blockIdx.y) / args.vheads;
+  const int kvh = hy / args.head_blocks, hb = hy % args.head_blocks;
   int q_row = b;
   if (args.cu_q) {
     q_row = args.cu_q[b];
     if (args.cu_q[b + 1] - q_row != 1) return;
   }
   const int len = args.context_lens[b];
-  // first visible token: the start of the chunk that holds the query (position len - 1)
-  const int first_tok = (args.chunk > 0 && len > 0) ? len - 1 - (len - 1) % args.chunk : 0;
+  // first visible token: the start of the chunk that holds the query (position len - 1), or of its window
+  int first_tok = (args.chunk > 0 && len > 0) ? len - 1 - (len - 1) % args.chunk : 0;
+  if (args.window > 0 && len - args.window > first_tok) first_tok = len - args.window;
   const int base_tile = first_tok / kTile;
   const int n_tiles_all = (len + kTile - 1) / kTile - base_tile;
   const int per = (n_tiles_all + args.splits - 1) / args.splits;
@@ -173,7 +177,7 @@ paged_decode_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
         }
         ++unit;
       };
-      const int kcol = kvh * args.D, vcol = kvh * args.DV;
+      const int kcol = kvh * args.D, vcol = (args.vheads > 1 ? vsel : kvh) * args.DV;
       load_tile(&tmK, 0, kcol, k_halves);
       for (int j = 0; j < n_tiles && ok; ++j) {
         if (j + 1 < n_tiles) load_tile(&tmK, j + 1, kcol, k_halves);
@@ -345,7 +349,7 @@ paged_decode_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       for (int h = 0; h < kHeads; ++h)
         if (h == row) { mh = m_used[h]; lh = l_tot[h]; }
       if (!have) { mh = -INFINITY; lh = 0.f; }
-      float* ml = args.part_ml + ((static_cast<size_t>(b) * args.num_q_heads + head0 + row) * args.splits + split) * 2;
+      float* ml = args.part_ml + (((static_cast<size_t>(b) * args.num_q_heads + head0 + row) * args.vheads + vsel) * args.splits + split) * 2;
       ml[0] = mh;
       ml[1] = lh;
     }
@@ -358,7 +362,7 @@ paged_decode_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
 #pragma unroll
     for (int h = 0; h < kHeads; ++h) {
       if (h < n_heads && row < args.DV)      // a split without tokens writes zeros: the merge multiplies them by a zero weight
-        args.part_acc[((static_cast<size_t>(b) * args.num_q_heads + head0 + h) * args.splits + split) * args.DV + row] =
+        args.part_acc[(((static_cast<size_t>(b) * args.num_q_heads + head0 + h) * args.vheads + vsel) * args.splits + split) * args.DV + row] =
             have ? __uint_as_float(r[h]) : 0.f;
     }
   }
@@ -409,17 +413,17 @@ int mfb_paged_decode_tc_splits(int B, int Hkv, int max_len) {
 }
 
 // q [rows, Hq, D] bf16, caches [num_blocks, block_size, Hkv, D | DV] bf16, out [rows, Hq, DV] bf16; scratch as for
-// mfb_paged_decode_attention (mfb_paged_decode_scratch_bytes(B, Hq, DV, splits)). cu_q null: row b belongs to sequence b
+// mfb_paged_decode_attention (mfb_paged_decode_scratch_bytes(B, Hq, DV, splits); all_values: Hq Hkv rows of results, no sink). cu_q null: row b belongs to sequence b
 // (rows == B); else [B + 1] row boundaries of a ragged batch, of which only the sequences with one row are computed and
-// written. chunk > 0: keys of the query's own chunk of positions only. sink: [Hq] fp32 or null, adds exp(sink) to the
+// written. chunk > 0: keys of the query's own chunk of positions only; window > 0: the last `window` keys only. sink: [Hq] fp32 or null, adds exp(sink) to the
 // softmax denominator. softcap > 0: scores become softcap * tanh(score / softcap). Rows of out lie ld_out elements apart; the
 // result is multiplied by out_scale.
 int mfb_paged_decode_attention_tc_ex(const void* q, const void* key_cache, const void* value_cache, const int* block_tables,
                                      const int* context_lens, const int* cu_q, const float* sink, void* out, void* scratch,
                                      int splits, int rows, int B, int Hq, int Hkv, int D, int DV, int num_blocks,
-                                     int block_size, int max_blocks, int chunk, float scale, float softcap,
-                                     long long ld_out, float out_scale, int* status, cudaStream_t stream) {
-  if (!mfb_paged_decode_tc_supported_ex(Hq, Hkv, D, DV, block_size) || splits < 1 || num_blocks < 1 || (!cu_q && rows != B)) {
+                                     int block_size, int max_blocks, int chunk, int window, int all_values, float scale,
+                                     float softcap, long long ld_out, float out_scale, int* status, cudaStream_t stream) {
+  if (!mfb_paged_decode_tc_supported_ex(Hq, Hkv, D, DV, block_size) || splits < 1 || num_blocks < 1 || (!cu_q && rows != B) || (all_values && sink)) {
     mfb_host::set_error("paged_decode_tc: unsupported Hq=%d Hkv=%d D=%d DV=%d block_size=%d splits=%d", Hq, Hkv, D, DV,
                         block_size, splits);
     return 1;
@@ -435,12 +439,12 @@ int mfb_paged_decode_attention_tc_ex(const void* q, const void* key_cache, const
   pdt::Args a;
   a.block_tables = block_tables; a.context_lens = context_lens; a.cu_q = cu_q; a.max_blocks = max_blocks;
   a.block_size = block_size; a.num_q_heads = Hq; a.num_kv_heads = Hkv; a.group = Hq / Hkv; a.splits = splits;
-  a.D = D; a.DV = DV; a.chunk = chunk; a.head_blocks = (a.group + pdt::kHeads - 1) / pdt::kHeads;
+  a.D = D; a.DV = DV; a.chunk = chunk; a.window = window; a.vheads = all_values ? Hkv : 1; a.head_blocks = (a.group + pdt::kHeads - 1) / pdt::kHeads;
   a.scale_log2 = scale * 1.4426950408889634f;
   a.cap_log2 = softcap > 0.f ? softcap * 1.4426950408889634f : 0.f;
   a.cap_scale = softcap > 0.f ? scale / softcap : 0.f;
   a.part_acc = reinterpret_cast<float*>(scratch);
-  a.part_ml = a.part_acc + static_cast<size_t>(B) * Hq * splits * DV;
+  a.part_ml = a.part_acc + static_cast<size_t>(B) * Hq * a.vheads * splits * DV;
   a.status = status;
   static bool attr_set = false;
   if (!attr_set) {
@@ -450,10 +454,10 @@ int mfb_paged_decode_attention_tc_ex(const void* q, const void* key_cache, const
     }
     attr_set = true;
   }
-  dim3 grid(splits, Hkv * a.head_blocks, B);
+  dim3 grid(splits, Hkv * a.head_blocks * a.vheads, B);
   pdt::paged_decode_tc_kernel<<<grid, pdt::kThreads, pdt::kSmem, stream>>>(tQ, tK, tV, a);
   if (cudaGetLastError() != cudaSuccess) { mfb_host::set_error("paged_decode_tc: launch failed"); return 11; }
-  return mfb_paged_combine_ex(a.part_acc, a.part_ml, out, splits, B * Hq, DV, Hq, cu_q, sink, ld_out, out_scale, stream);
+  return mfb_paged_combine_ex(a.part_acc, a.part_ml, out, splits, B * Hq * a.vheads, DV, Hq * a.vheads, cu_q, sink, ld_out, out_scale, stream);
 }
 
 // q [B, Hq, 128], caches [num_blocks, block_size, Hkv, 128], out [B, Hq, 128]: one row per sequence, no chunks, no sink.
@@ -462,7 +466,7 @@ int mfb_paged_decode_attention_tc(const void* q, const void* key_cache, const vo
                                   int num_blocks, int block_size, int max_blocks, float scale, int* status,
                                   cudaStream_t stream) {
   return mfb_paged_decode_attention_tc_ex(q, key_cache, value_cache, block_tables, context_lens, nullptr, nullptr, out, scratch,
-                                          splits, B, B, Hq, Hkv, pdt::kHd, pdt::kHd, num_blocks, block_size, max_blocks, 0,
+                                          splits, B, B, Hq, Hkv, pdt::kHd, pdt::kHd, num_blocks, block_size, max_blocks, 0, 0, 0,
                                           scale, 0.f, (long long)Hq * pdt::kHd, 1.f, status, stream);
 }
 

@@ -14,6 +14,10 @@
 // softmax, so one stage of each is enough. A CTA's roles run through all of its tiles (see the launcher): the
 // loads and the first scores of a tile run under the last softmax and the output of the one before, which is what counts
 // when a tile sees few keys (chunks, short portions). What else differs:
+//   - a sliding window (`window` > 0) hides the keys that lie `window` or more positions before the row;
+//   - with `all_values` every query head's weights are applied to the values of every key / value head, one after the other
+//     (items of their own, so that K and q come from L2);
+//   - rows of K and V may lie further apart than their heads fill (slices of one product);
 //   - work comes as a list of (sequence, first row of q, rows, position of the first row), one entry per query tile; only
 //     key tiles that some row of the tile sees are visited, from the chunk of its first row to its last row;
 //   - K / V tiles (128 consecutive positions) are assembled from the sequence's pages, one TMA box per page and 64
@@ -38,11 +42,12 @@ constexpr float kRescaleThreshold = 8.0f;  // log2 units
 
 struct Args {
   const int4* work;          // [n_work]: sequence, first row of q, rows, position of the first row
-  int n_items;               // n_work x query heads: item i is tile i / heads of head i % heads
+  int n_items;               // n_work x query heads x vheads, in this order
   const int* block_tables;   // [B, max_blocks]
   const float* sink;         // [Hq] or null
-  __nv_bfloat16* out;        // [T, Hq, DV]
-  int num_q_heads, group, D, DV, block_size, max_blocks, chunk;
+  __nv_bfloat16* out;        // [T, Hq, vheads, DV]
+  int num_q_heads, group, D, DV, block_size, max_blocks, chunk, window;
+  int vheads;                // value heads per query head: 1 (its own) or all
   float scale_log2;
   float cap_log2, cap_scale;   // soft cap of the scores in log2 units (CAP kernels) and scale / cap
   float cap_poly[5];           // capped score (log2 units) = s * polynomial in s^2, for |s| * cap_scale <= kPolyReach
@@ -137,13 +142,20 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_holder + 1);
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  struct Tile { int b, head, q0, rows, pos0, lo, n_kv; };      // key tiles lo .. n_kv - 1
+  struct Tile { int b, head, vsel, q0, rows, pos0, lo, n_kv; };      // key tiles lo .. n_kv - 1
+  auto first_of = [&](int pos) {            // first position that `pos` sees; does not fall as pos grows
+    int lo = args.chunk > 0 ? pos - pos % args.chunk : 0;
+    if (args.window > 0 && pos - args.window + 1 > lo) lo = pos - args.window + 1;
+    return lo;
+  };
   auto tile_of = [&](int item) {
-    const int4 w = args.work[item / args.num_q_heads];
     Tile t;
+    t.vsel = item % args.vheads;
+    item /= args.vheads;
+    const int4 w = args.work[item / args.num_q_heads];
     t.head = item % args.num_q_heads;
     t.b = w.x; t.q0 = w.y; t.rows = w.z; t.pos0 = w.w;
-    t.lo = args.chunk > 0 ? (t.pos0 - t.pos0 % args.chunk) / kTile : 0;
+    t.lo = first_of(t.pos0) / kTile;
     t.n_kv = (t.pos0 + t.rows - 1) / kTile + 1;
     return t;
   };
@@ -182,7 +194,7 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
         for (int c = 0; c < QB; ++c) tma_load_3d(smem_u32(sQ) + c * kSubBytes, &tmQ, qb, c * 64, t.head, t.q0);
         const int* table = args.block_tables + static_cast<size_t>(t.b) * args.max_blocks;
         const int kv_head = t.head / args.group, end = t.pos0 + t.rows;
-        const int kcol = kv_head * args.D, vcol = kv_head * args.DV;
+        const int kcol = kv_head * args.D, vcol = (args.vheads > 1 ? t.vsel : kv_head) * args.DV;
         for (int j = t.lo; j < t.n_kv; ++j, ++it) {
           const uint32_t ph = it & 1;
           const int tok0 = j * kTile;
@@ -269,7 +281,7 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
       const Tile t = tile_of(item);
       const int lo = t.lo, n_kv = t.n_kv;
       const int my_pos = t.pos0 + row;
-      const int my_first = args.chunk > 0 ? my_pos - my_pos % args.chunk : 0;   // first key this row may see
+      const int my_first = first_of(my_pos);         // first key this row may see
       float m_used = -INFINITY, l_sum = 0.f;
       for (int j = lo; j < n_kv; ++j, ++it) {
         ok = mbar_wait(smem_u32(s_full), it & 1, abort_flag, args.status, kStatusWaitTimeoutEpilogue);
@@ -427,7 +439,7 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
       const float inv_l = args.out_scale / den;
       // 32 columns at a time through 2 KB of shared memory per warp, so that a store covers 64 bytes of eight rows each
       uint8_t* stage = sOut + ew * 2048;
-      __nv_bfloat16* obase = args.out + (t.q0 + ew * 32) * args.ld_out + static_cast<size_t>(t.head) * args.DV;
+      __nv_bfloat16* obase = args.out + (t.q0 + ew * 32) * args.ld_out + static_cast<size_t>(t.head * args.vheads + t.vsel) * args.DV;
 #pragma unroll
       for (int c = 0; c < HV / 32; ++c) {
         uint32_t r[32];
@@ -511,20 +523,26 @@ int mfb_paged_prefill_tc_supported(int Hq, int Hkv, int D, int DV, int block_siz
   return (block_size == 16 || block_size == 32 || block_size == 64 || block_size == 128) ? 1 : 0;
 }
 
-// q [T, Hq, D], caches [num_blocks, block_size, Hkv, D | DV], out [T, Hq, DV], all bf16. work [n_work, 4] int32: (sequence,
+// q [T, Hq, D], caches [num_blocks, block_size, Hkv, D | DV] with rows ld_k / ld_v elements apart, out [T, Hq, DV] (all_values:
+// [T, Hq, Hkv, DV]), all bf16. chunk > 0: a position sees its own chunk only; window > 0: itself and the window - 1 positions
+// before it. work [n_work, 4] int32: (sequence,
 // first row of q, 1..128 rows, position of the first row) per query tile, heaviest first; the rows' keys are in the cache.
 // persistent: two CTAs per SM walk over all tiles (for tiles of a few key tiles); else a CTA per query tile and head, which
 // balances tiles of very different lengths better. softcap > 0: scores become softcap * tanh(score / softcap). Rows of out lie
 // ld_out elements apart; the result is multiplied by out_scale.
 int mfb_paged_prefill_tc(const void* q, const void* key_cache, const void* value_cache, const int* work, int n_work, int persistent,
                          const int* block_tables, const float* sink, void* out, int T,
-                         int Hq, int Hkv, int D, int DV, int num_blocks, int block_size, int max_blocks, int chunk, float scale,
-                         float softcap, long long ld_out, float out_scale, int* status, cudaStream_t stream) {
+                         int Hq, int Hkv, int D, int DV, int num_blocks, int block_size, int max_blocks, int chunk, int window,
+                         int all_values, long long ld_k, long long ld_v, float scale, float softcap, long long ld_out, float out_scale, int* status, cudaStream_t stream) {
   if (!mfb_paged_prefill_tc_supported(Hq, Hkv, D, DV, block_size) || num_blocks < 1 || T < 1) {
     mfb_host::set_error("paged_prefill_tc: unsupported Hq=%d Hkv=%d D=%d DV=%d block_size=%d", Hq, Hkv, D, DV, block_size);
     return 1;
   }
   if (n_work <= 0) return 0;
+  if (ld_k < (long long)Hkv * D || ld_v < (long long)Hkv * DV) {
+    mfb_host::set_error("paged_prefill_tc: row pitches %lld and %lld", ld_k, ld_v);
+    return 1;
+  }
   if (ld_out % 8 || (reinterpret_cast<uintptr_t>(out) & 15)) {
     mfb_host::set_error("paged_prefill_tc: rows of the result must start on 16 bytes");
     return 1;
@@ -533,14 +551,14 @@ int mfb_paged_prefill_tc(const void* q, const void* key_cache, const void* value
   int rc;
   const CUtensorMapDataType BF = CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
   const uint64_t rows = (uint64_t)num_blocks * block_size;
-  if ((rc = mfb_host::make_tmap_2d(&tK, key_cache, 2, BF, rows, (uint64_t)Hkv * D, (uint64_t)Hkv * D, block_size, 64))) return 30 + rc;
-  if ((rc = mfb_host::make_tmap_2d(&tV, value_cache, 2, BF, rows, (uint64_t)Hkv * DV, (uint64_t)Hkv * DV, block_size, 64))) return 40 + rc;
+  if ((rc = mfb_host::make_tmap_2d(&tK, key_cache, 2, BF, rows, (uint64_t)Hkv * D, (uint64_t)ld_k, block_size, 64))) return 30 + rc;
+  if ((rc = mfb_host::make_tmap_2d(&tV, value_cache, 2, BF, rows, (uint64_t)Hkv * DV, (uint64_t)ld_v, block_size, 64))) return 40 + rc;
   if ((rc = ppt::make_q_map(&tQ, q, T, Hq, D))) return 20 + rc;
   ppt::Args a;
-  a.work = reinterpret_cast<const int4*>(work); a.n_items = n_work * Hq; a.block_tables = block_tables; a.sink = sink;
+  a.work = reinterpret_cast<const int4*>(work); a.vheads = all_values ? Hkv : 1; a.n_items = n_work * Hq * a.vheads; a.block_tables = block_tables; a.sink = sink;
   a.out = reinterpret_cast<__nv_bfloat16*>(out);
   a.num_q_heads = Hq; a.group = Hq / Hkv; a.D = D; a.DV = DV; a.block_size = block_size; a.max_blocks = max_blocks;
-  a.chunk = chunk; a.scale_log2 = scale * 1.4426950408889634f; a.status = status;
+  a.chunk = chunk; a.window = window; a.scale_log2 = scale * 1.4426950408889634f; a.status = status;
   a.cap_log2 = softcap > 0.f ? softcap * 1.4426950408889634f : 0.f;
   a.cap_scale = softcap > 0.f ? scale / softcap : 0.f;
   float power = a.scale_log2;

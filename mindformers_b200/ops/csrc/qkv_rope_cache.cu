@@ -1,5 +1,5 @@
 // Between the QKV projection and attention over a paged cache, in one kernel (sm_100a, bf16 or fp32): projection bias,
-// per-head RMS norm of q and k, rotary embedding of q and k, and the write of k and v into the paged cache.
+// per-head RMS norm of q and k (with or without a weight) and of v (without), rotary embedding of q and k, and the write of k and v into the paged cache.
 //
 //   qkv [T, H * D + G * D + G * DV] (row pitch given)  ->  q_out [T, H, D]
 //                                                          key_cache [slots, G, D], value_cache [slots, G, DV]
@@ -47,8 +47,32 @@ struct Args {
   void* key_cache;
   void* value_cache;
   int H, G, D, DV, rot, interleaved, paired;   // paired: neighbours may be accessed two at a time
+  int unit_qk, unit_v;        // norms without a weight
   float amplitude, eps;
 };
+
+// values divided by their root mean square per head, a warp per head; a lane keeps its columns in registers
+template <typename T>
+__device__ __forceinline__ void unit_values(const Args& a, const T* row, const T* bias, long long off, T* dst) {
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  for (int g = warp; g < a.G; g += kThreads / 32) {
+    const T* src = row + off + (long long)g * a.DV;
+    const T* b = bias ? bias + off + (long long)g * a.DV : nullptr;
+    float v[2 * kMaxPairs], ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < 2 * kMaxPairs; ++k) {
+      const int d = lane + 32 * k;
+      v[k] = d < a.DV ? ld(src + d) + (b ? ld(b + d) : 0.f) : 0.f;
+      ss = fmaf(v[k], v[k], ss);
+    }
+    const float rstd = 1.f / sqrtf(warp_sum(ss) / a.DV + a.eps);
+#pragma unroll
+    for (int k = 0; k < 2 * kMaxPairs; ++k) {
+      const int d = lane + 32 * k;
+      if (d < a.DV) st(dst + (long long)g * a.DV + d, v[k] * rstd);
+    }
+  }
+}
 
 template <typename T>
 __global__ void __launch_bounds__(kThreads) qkv_rope_cache_kernel(const Args a) {
@@ -96,7 +120,7 @@ __global__ void __launch_bounds__(kThreads) qkv_rope_cache_kernel(const Args a) 
     }
     const T* nw = reinterpret_cast<const T*>(is_q ? a.q_norm : a.k_norm);
     float rstd = 1.f;
-    if (nw) rstd = 1.f / sqrtf(warp_sum(ss) / D + a.eps);
+    if (nw || a.unit_qk) rstd = 1.f / sqrtf(warp_sum(ss) / D + a.eps);
     T* dst = is_q ? reinterpret_cast<T*>(a.q_out) + (t * a.H + h) * D
                   : reinterpret_cast<T*>(a.key_cache) + ((long long)slot * a.G + (h - a.H)) * D;
 #pragma unroll
@@ -109,6 +133,9 @@ __global__ void __launch_bounds__(kThreads) qkv_rope_cache_kernel(const Args a) 
         if (nw) {
           x = x * rstd * ld(nw + e0);
           if (e1 < D) y = y * rstd * ld(nw + e1);
+        } else {
+          x *= rstd;
+          y *= rstd;
         }
         if (p < half) {
           const float c = sh_cos[p], s = sh_sin[p];
@@ -129,7 +156,9 @@ __global__ void __launch_bounds__(kThreads) qkv_rope_cache_kernel(const Args a) 
     const int n = a.G * a.DV;
     const long long off = (long long)(a.H + a.G) * D;
     T* dst = reinterpret_cast<T*>(a.value_cache) + (long long)slot * n;
-    if (a.paired && n % 2 == 0) {
+    if (a.unit_v) {
+      unit_values(a, row, bias, off, dst);
+    } else if (a.paired && n % 2 == 0) {
       for (int i = threadIdx.x * 2; i < n; i += kThreads * 2) {
         float x, y;
         ld2(row + off + i, x, y);
@@ -212,12 +241,12 @@ __global__ void __launch_bounds__(kThreads) qkv_rope_cache_vec_kernel(const Args
 #pragma unroll
     for (int o = LPH / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
     if (!on || (!is_q && slot < 0)) continue;
-    if (nw) {
+    if (nw || a.unit_qk) {
       const float rstd = 1.f / sqrtf(ss / D + a.eps);
       float w[8];
-      ld8(nw + e, w);
+      if (nw) ld8(nw + e, w);
 #pragma unroll
-      for (int i = 0; i < 8; ++i) cur[i] = cur[i] * rstd * w[i];
+      for (int i = 0; i < 8; ++i) cur[i] = nw ? cur[i] * rstd * w[i] : cur[i] * rstd;
     }
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
@@ -237,6 +266,10 @@ __global__ void __launch_bounds__(kThreads) qkv_rope_cache_vec_kernel(const Args
     const int n = a.G * a.DV;
     const long long off = (long long)n_heads * D;
     T* dst = reinterpret_cast<T*>(a.value_cache) + (long long)slot * n;
+    if (a.unit_v) {
+      unit_values(a, row, bias, off, dst);
+      return;
+    }
     for (int i = threadIdx.x * 8; i < n; i += kThreads * 8) {
       float v[8];
       ld8(row + off + i, v);
@@ -270,13 +303,14 @@ bool al(const void* p, int n) { return (reinterpret_cast<uintptr_t>(p) & (n - 1)
 extern "C" {
 using namespace mfb;
 
-// f32 = 1: all typed tensors are fp32, else bf16. freqs: [rot / 2] fp32; cos and sin are multiplied by `amplitude`.
+// f32 = 1: all typed tensors are fp32, else bf16. unit: bit 0: q and k, bit 1: v are normed without a weight (DV up to 512). freqs: [rot / 2] fp32; cos and sin are multiplied by `amplitude`.
 int mfb_qkv_rope_cache(const void* qkv, long long ld_qkv, const void* bias, const void* q_norm, const void* k_norm, float eps,
                        const float* freqs, float amplitude, int rot, int interleaved, const long long* positions,
                        const int* slots, void* q_out, void* key_cache, void* value_cache, int T, int H, int G, int D, int DV,
-                       int f32, cudaStream_t stream) {
+                       int unit, int f32, cudaStream_t stream) {
   if (T <= 0) return 0;
-  if (H < 1 || G < 1 || D < 1 || DV < 1 || D > 64 * qrc::kMaxPairs || rot < 0 || rot > D || rot % 2) {
+  if (H < 1 || G < 1 || D < 1 || DV < 1 || D > 64 * qrc::kMaxPairs || rot < 0 || rot > D || rot % 2 ||
+      ((unit & 1) && (q_norm || k_norm)) || ((unit & 2) && DV > 64 * qrc::kMaxPairs)) {
     mfb_host::set_error("qkv_rope_cache: H=%d G=%d D=%d DV=%d rot=%d", H, G, D, DV, rot);
     return 1;
   }
@@ -285,6 +319,7 @@ int mfb_qkv_rope_cache(const void* qkv, long long ld_qkv, const void* bias, cons
   a.qkv = qkv; a.ld_qkv = ld_qkv; a.bias = bias; a.q_norm = q_norm; a.k_norm = k_norm; a.freqs = freqs;
   a.positions = positions; a.slots = slots; a.q_out = q_out; a.key_cache = key_cache; a.value_cache = value_cache;
   a.H = H; a.G = G; a.D = D; a.DV = DV; a.rot = rot; a.interleaved = interleaved; a.amplitude = amplitude; a.eps = eps;
+  a.unit_qk = unit & 1; a.unit_v = (unit >> 1) & 1;
   a.paired = (D % 2 == 0 && (G * DV) % 2 == 0 && ld_qkv % 2 == 0 && qrc::al(qkv, two) && qrc::al(bias, two) &&
               qrc::al(q_out, two) && qrc::al(key_cache, two) && qrc::al(value_cache, two)) ? 1 : 0;
   const size_t smem = (size_t)rot * sizeof(float);

@@ -1,8 +1,9 @@
-"""Gated delta rule over ragged batches: short convolutions, unit keys, decays, the recurrence, its norm and gate.
+"""Recurrent mixers over ragged batches: the gated delta rule (short convolutions, unit keys, decays, the recurrence, its norm
+and gate) and the matrix memory (capped log gates, running maximum, memory and normaliser, norm and gate).
 
-``delta_rule`` has two bodies like the ops of ``functional.py``: the sm_100a kernels (``csrc/delta_rule.cu``), always taken
-for CUDA tensors (bf16 or fp32 activations; state and recurrence are fp32), and a plain PyTorch body for CPU tensors. It
-is an inference op: it advances the state in place and has no gradients.
+``delta_rule`` and ``matrix_memory`` have two bodies like the ops of ``functional.py``: the sm_100a kernels (``csrc/delta_rule.cu``, ``csrc/matrix_memory.cu``),
+always taken for CUDA tensors (bf16 or fp32 activations; state and recurrence are fp32), and a plain PyTorch body for CPU
+tensors. They are inference ops: they advance the state in place and have no gradients.
 """
 from __future__ import annotations
 
@@ -165,4 +166,87 @@ def _decode_as_portions(x, b, a, gate, w, s, state, cache, eps, out, out_scale):
     _lib.count_launch(4)
     S[:B].copy_(torch.where(idle[:, None, None, None], keep[0], S[:B]))
     ring[:B].copy_(torch.where(idle[:, None, None], keep[1], ring[:B]))
+    return out
+
+
+# ---- matrix memory ------------------------------------------------------------------------------------------------------------
+@dataclass
+class MemoryShape:
+    heads: int
+    dim: int
+    v_dim: int
+    gate_cap: float
+
+
+def _memory_reference(proj, bi, bf, norm, s: MemoryShape, state, cache, eps, out):
+    H, D, DV, cap = s.heads, s.dim, s.v_dim, s.gate_cap
+    S_all, n_all, m_all = state
+    if not cache.is_prefill:
+        out.zero_()
+    for slot, r0, n, start in _sequences(cache, proj.shape[0]):
+        rows = slice(r0, r0 + n)
+        q, k, v, z, i, f = torch.split(proj[rows].float(), (H * D, H * D, H * DV, H * DV, H, H), dim=1)
+        q, k, v = q.view(n, H, D) * D ** -0.5, k.view(n, H, D), v.view(n, H, DV)
+        i = cap * torch.tanh((i + bi) / cap)
+        f = F.logsigmoid(cap * torch.tanh((f + bf) / cap))
+        S, nv, m = (t[slot].clone() if start > 0 else torch.zeros_like(t[slot]) for t in state)
+        o = torch.empty(n, H, DV)
+        for t in range(n):
+            new = torch.maximum(f[t] + m, i[t])
+            keep, put = torch.exp(f[t] + m - new), torch.exp(i[t] - new)
+            S = keep[:, None, None] * S + (put[:, None] * k[t])[:, :, None] * v[t][:, None]
+            nv = keep[:, None] * nv + put[:, None] * k[t]
+            m = new
+            size = torch.maximum((nv * q[t]).sum(-1).abs(), torch.exp(-m)) + 1e-6
+            o[t] = (S * q[t][:, :, None]).sum(1) / size[:, None]
+        S_all[slot], n_all[slot], m_all[slot] = S, nv, m
+        o = o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + eps) * norm.view(H, DV)
+        out[rows] = (o.reshape(n, H * DV) * torch.sigmoid(z)).to(out.dtype)
+
+
+def matrix_memory(proj: torch.Tensor, input_bias: torch.Tensor, forget_bias: torch.Tensor, norm: torch.Tensor, s: MemoryShape,
+                  state: Tuple[torch.Tensor, torch.Tensor, torch.Tensor], cache, eps: float) -> torch.Tensor:
+    """``proj [T, >= 2 H D + 2 H DV + 2 H]`` (q | k | v | output gate | input gate | forget gate, any row pitch), all of the step's
+    rows in the order of ``cache`` (``KVCacheContext``). Per head, with ``q`` times ``D ** -0.5`` and the log gates ``i = cap
+    tanh((x_i + b_i) / cap)``, ``f = log_sigmoid(cap tanh((x_f + b_f) / cap))``::
+
+        m' = max(f + m, i);  S' = e^(f + m - m') S + e^(i - m') k v^T;  n' the same with k alone
+        o  = S'^T q / (max(|n' . q|, e^(-m')) + 1e-6)
+
+    Returns ``[T, H DV]``: ``o`` RMS-normed per head, times ``norm`` and the sigmoid of the output gate. ``state``: the layer's
+    ``(S [slots, H, D, DV], n [slots, H, D], m [slots, H])`` in fp32, advanced in place."""
+    T, dtype = proj.shape[0], proj.dtype
+    H, D, DV = s.heads, s.dim, s.v_dim
+    out = torch.empty((T, H * DV), dtype=dtype, device=proj.device)
+    if not proj.is_cuda:
+        _memory_reference(proj, input_bias, forget_bias, norm, s, state, cache, eps, out)
+        return out
+    if dtype not in (torch.bfloat16, torch.float32):
+        raise TypeError(f"bfloat16 or float32 activations expected, got {dtype}")
+    _rows(proj, dtype, T, 2 * H * (D + DV) + 2 * H, "proj")
+    S, n, m = state
+    slots = S.shape[0]
+    for t, shape in ((S, (slots, H, D, DV)), (n, (slots, H, D)), (m, (slots, H)), (input_bias, (H,)), (forget_bias, (H,)),
+                     (norm, (H * DV,))):
+        if t.dtype != torch.float32 or tuple(t.shape) != shape or not t.is_contiguous():
+            raise TypeError("matrix_memory: states, biases and the norm's weight are contiguous fp32 tensors of the layer's shape")
+    B = cache.context_lens.numel()
+    if B > slots:
+        raise ValueError("matrix_memory: every sequence needs a state slot")
+    lib = _lib.get_lib()
+    f32 = int(dtype == torch.float32)
+    cu, scratch = 0, 0
+    if cache.is_prefill:
+        cu = cache.cu_q_dev.data_ptr()
+        longest = max(cache.q_lens_host, default=0)
+        buf = torch.empty(lib.mfb_matrix_memory_scratch_floats(T, B, H, D, DV), dtype=torch.float32, device=proj.device)
+        scratch = buf.data_ptr()
+    else:
+        longest = 1
+    rc = lib.mfb_matrix_memory(proj.data_ptr(), proj.stride(0), input_bias.data_ptr(), forget_bias.data_ptr(), norm.data_ptr(),
+                               S.data_ptr(), n.data_ptr(), m.data_ptr(), cu, cache.context_lens.data_ptr(),
+                               cache.slot_mapping.data_ptr(), scratch, out.data_ptr(), T, B, H, D, DV, longest, s.gate_cap, float(eps),
+                               f32, _lib.stream_ptr())
+    _lib.check(rc, "mfb_matrix_memory")
+    _lib.count_launch(2 if cache.is_prefill else 1)
     return out

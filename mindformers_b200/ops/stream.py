@@ -5,6 +5,7 @@ fp32), and a plain PyTorch body for CPU tensors. They are inference ops: no grad
 """
 from __future__ import annotations
 
+from dataclasses import dataclass
 from typing import Optional, Tuple
 
 import torch
@@ -115,6 +116,103 @@ def residual_streams(x: torch.Tensor, n: int, y: Optional[torch.Tensor], mix: Op
     return h, (x if y is None else out)
 
 
+def sinusoidal_frequencies(width: int) -> torch.Tensor:
+    """fp64 ``[ceil(width / 2)]``: frequency i is ``10000 ** (-2 i / width)``."""
+    i = torch.arange((width + 1) // 2, dtype=torch.float64)
+    return torch.pow(torch.tensor(10000.0, dtype=torch.float64), -2.0 * i / width)
+
+
+def embed(ids: torch.Tensor, table: torch.Tensor, scale: float, positions: torch.Tensor,
+          freqs: Optional[torch.Tensor]) -> torch.Tensor:
+    """``scale * table[ids]`` in fp32, plus (with ``freqs``) the position vector whose entries 2i and 2i + 1 are the sine and
+    cosine of ``position * freqs[i]``. The angles are fp64 until they are within one turn."""
+    T, W = ids.numel(), table.shape[1]
+    if not table.is_cuda:
+        x = table[ids].float() * scale
+        if freqs is not None:
+            a = positions.to(torch.float64)[:, None] * freqs[None, :]
+            x = x + torch.stack((torch.sin(a), torch.cos(a)), dim=-1).flatten(1)[:, :W].float()
+        return x
+    _check_dtype(table.dtype)
+    if ids.dtype != torch.int64 or positions.dtype != torch.int64 or positions.numel() != T or not table.is_contiguous() \
+            or not ids.is_contiguous() or (freqs is not None and (freqs.dtype != torch.float64 or freqs.numel() != (W + 1) // 2)):
+        raise TypeError("embed: int64 ids and positions, a contiguous table and fp64 frequencies expected")
+    x = torch.empty((T, W), dtype=torch.float32, device=table.device)
+    rc = _lib.get_lib().mfb_embed_stream(ids.data_ptr(), table.data_ptr(), positions.contiguous().data_ptr(), _lib.ptr(freqs),
+                                         x.data_ptr(), T, W, table.shape[0], float(scale), int(table.dtype == torch.float32),
+                                         _lib.stream_ptr())
+    _lib.check(rc, "mfb_embed_stream")
+    _lib.count_launch()
+    return x
+
+
+@dataclass
+class Carry:
+    """Token shift of one layer run: ``mu [W]`` and the cache that keeps the last token's vector per sequence slot."""
+    mu: torch.Tensor
+    cache: object
+    run: int
+
+
+def _shift_reference(h, carry: Carry):
+    from .recurrent import _sequences
+    cache, out = carry.cache, h.clone()
+    state = cache.carry[carry.run]
+    for slot, r0, n, start in _sequences(cache, h.shape[0]):
+        first = state[slot] if start > 0 else torch.zeros_like(state[slot])
+        before = torch.cat((first[None], h[r0:r0 + n - 1]))
+        out[r0:r0 + n] = h[r0:r0 + n] + (before - h[r0:r0 + n]) * carry.mu.float()
+        state[slot] = h[r0 + n - 1]
+    return out
+
+
+def normed_step(x: torch.Tensor, y: Optional[torch.Tensor], w_in: Optional[torch.Tensor], step: Optional[torch.Tensor],
+                w_out: torch.Tensor, eps: float, zero_centered: bool, carry: Optional[Carry] = None,
+                keep: bool = True) -> Tuple[torch.Tensor, Optional[torch.Tensor]]:
+    """One step of an fp32 residual stream ``x [T, W]`` with norms on both sides of a sub-layer: ``x' = x + rms_norm(y; w_in) +
+    step`` (without ``y`` or ``step``: without that term), then the next sub-layer's input ``h = rms_norm(x'; w_out)``, with
+    ``carry`` shifted by a token: ``h + (h of the sequence's token before - h) * mu`` (zeros before the first token; the last
+    ``h`` of a portion stays in ``cache.carry``). ``zero_centered``: the norms' weights are ``1 + w``.
+
+    Returns ``(h in the dtype of w_out, x')``; ``x`` is not changed; ``keep=False`` drops ``x'``."""
+    T, W, dtype = x.shape[0], x.shape[1], w_out.dtype
+    if not x.is_cuda:
+        one = 1.0 if zero_centered else 0.0
+        if y is not None:
+            x = x + norm_reference(y, w_in.float() + one, None, eps, False)
+        if step is not None:
+            x = x + step.float()
+        h = norm_reference(x, w_out.float() + one, None, eps, False)
+        if carry is not None:
+            h = _shift_reference(h, carry)
+        return h.to(dtype), (x if keep else None)
+    _check_dtype(dtype)
+    _typed(w_in, step, w_out, None if carry is None else carry.mu, dtype=dtype)
+    if x.dtype != torch.float32 or not x.is_contiguous() or (y is not None and (
+            y.dtype != dtype or y.shape != (T, W) or y.stride(1) != 1 or w_in is None)):
+        raise TypeError("normed_step: a contiguous fp32 stream and a sub-layer output in the activation dtype expected")
+    h = torch.empty((T, W), dtype=dtype, device=x.device)
+    same = y is None and step is None
+    out = torch.empty_like(x) if keep and not same else None
+    B, cu, lens, slots, before, after = 0, 0, 0, 0, 0, 0
+    if carry is not None:
+        c = carry.cache
+        state = c.carry[carry.run]
+        B = c.context_lens.numel()
+        if state.dtype != torch.float32 or state.shape[1] != W or not state.is_contiguous() or B > state.shape[0]:
+            raise ValueError("normed_step: the carry does not have the stream's width, or a sequence has no slot")
+        cu = c.cu_q_dev.data_ptr() if c.is_prefill else 0
+        lens, slots, after = c.context_lens.data_ptr(), c.slot_mapping.data_ptr(), state.data_ptr()
+        before = c.carry_before[carry.run].data_ptr() if c.is_prefill else after
+    rc = _lib.get_lib().mfb_normed_step(
+        x.data_ptr(), _lib.ptr(y), 0 if y is None else y.stride(0), _lib.ptr(w_in), _lib.ptr(step), w_out.data_ptr(), _lib.ptr(out),
+        h.data_ptr(), None if carry is None else carry.mu.data_ptr(), before, after, cu, lens, slots, T, W, B, int(zero_centered),
+        float(eps), int(dtype == torch.float32), _lib.stream_ptr())
+    _lib.check(rc, "mfb_normed_step")
+    _lib.count_launch()
+    return h, (x if same else out) if keep else None
+
+
 def relu2(x: torch.Tensor) -> torch.Tensor:
     """``max(x, 0)^2``"""
     if not x.is_cuda or (torch.is_grad_enabled() and x.requires_grad):
@@ -196,9 +294,9 @@ def _rotate_reference(x, positions, freqs, amplitude, rot, interleaved):
 def qkv_rope_cache(qkv: torch.Tensor, bias: Optional[torch.Tensor], q_norm: Optional[torch.Tensor],
                    k_norm: Optional[torch.Tensor], eps: float, freqs: torch.Tensor, amplitude: float, interleaved: bool,
                    positions: torch.Tensor, slots: torch.Tensor, key_cache: torch.Tensor, value_cache: torch.Tensor,
-                   heads: int, kv_heads: int, dim: int, v_dim: int) -> torch.Tensor:
+                   heads: int, kv_heads: int, dim: int, v_dim: int, unit_qk: bool = False, unit_v: bool = False) -> torch.Tensor:
     """Everything between the QKV projection and attention over the paged cache: projection bias, per-head RMS norm of q
-    and k (``None``: no norm), rotation of the first ``2 * len(freqs)`` dimensions by ``position * freqs`` (cos and sin
+    and k (``None``: no norm; ``unit_qk``: a norm without a weight) and of v (``unit_v``, without a weight), rotation of the first ``2 * len(freqs)`` dimensions by ``position * freqs`` (cos and sin
     times ``amplitude``) and the write of k and v into the cache rows ``slots`` (negative: not written).
 
     ``qkv [T, heads * dim + kv_heads * (dim + v_dim)]`` → q ``[T, heads, dim]``."""
@@ -208,10 +306,13 @@ def qkv_rope_cache(qkv: torch.Tensor, bias: Optional[torch.Tensor], q_norm: Opti
         x = qkv.float() if bias is None else qkv.float() + bias.float()
         q, k = x[:, :nq].view(T, heads, dim), x[:, nq:nq + nk].view(T, kv_heads, dim)
         v = x[:, nq + nk:]
-        if q_norm is not None:
-            q = norm_reference(q, q_norm, None, eps, False)
-        if k_norm is not None:
-            k = norm_reference(k, k_norm, None, eps, False)
+        one = torch.ones(())
+        if q_norm is not None or unit_qk:
+            q = norm_reference(q, one if unit_qk else q_norm, None, eps, False)
+        if k_norm is not None or unit_qk:
+            k = norm_reference(k, one if unit_qk else k_norm, None, eps, False)
+        if unit_v:
+            v = norm_reference(v.reshape(T, kv_heads, v_dim), one, None, eps, False).reshape(T, -1)
         q = _rotate_reference(q, positions, freqs, amplitude, rot, interleaved)
         k = _rotate_reference(k, positions, freqs, amplitude, rot, interleaved)
         keep = slots >= 0
@@ -222,13 +323,78 @@ def qkv_rope_cache(qkv: torch.Tensor, bias: Optional[torch.Tensor], q_norm: Opti
     _check_dtype(dtype)
     _typed(bias, q_norm, k_norm, key_cache, value_cache, dtype=dtype)
     if qkv.stride(1) != 1 or qkv.shape[1] != nq + nk + kv_heads * v_dim or positions.dtype != torch.int64 \
-            or slots.dtype != torch.int32 or freqs.dtype != torch.float32 or positions.numel() != T or slots.numel() != T:
+            or slots.dtype != torch.int32 or (unit_qk and (q_norm is not None or k_norm is not None)) or freqs.dtype != torch.float32 or positions.numel() != T or slots.numel() != T:
         raise TypeError("qkv_rope_cache: unexpected shapes or dtypes")
     q = torch.empty((T, heads, dim), dtype=dtype, device=qkv.device)
     rc = _lib.get_lib().mfb_qkv_rope_cache(
         qkv.data_ptr(), qkv.stride(0), _lib.ptr(bias), _lib.ptr(q_norm), _lib.ptr(k_norm), float(eps), freqs.data_ptr(),
         float(amplitude), rot, int(interleaved), positions.data_ptr(), slots.data_ptr(), q.data_ptr(), key_cache.data_ptr(),
-        value_cache.data_ptr(), T, heads, kv_heads, dim, v_dim, int(dtype == torch.float32), _lib.stream_ptr())
+        value_cache.data_ptr(), T, heads, kv_heads, dim, v_dim, int(unit_qk) + 2 * int(unit_v), int(dtype == torch.float32),
+        _lib.stream_ptr())
     _lib.check(rc, "mfb_qkv_rope_cache")
     _lib.count_launch()
     return q
+
+
+def latent_norm_cache(proj: torch.Tensor, q_norm: torch.Tensor, kv_norm: torch.Tensor, eps: float, slots: torch.Tensor,
+                      cache: torch.Tensor) -> torch.Tensor:
+    """Between the down projections of latent attention and what follows: ``proj [T, >= Q + R]`` (query latent | key / value
+    latent, any row pitch) → the RMS-normed query latent ``[T, Q]``; the normed key / value latent goes to the rows ``slots`` of
+    ``cache [.., R]`` (negative: not written)."""
+    T, dtype, Q, R = proj.shape[0], proj.dtype, q_norm.numel(), kv_norm.numel()
+    if not proj.is_cuda:
+        c = norm_reference(proj[:, Q:Q + R], kv_norm, None, eps, False)
+        keep = slots >= 0
+        cache.view(-1, R)[slots[keep].long()] = c[keep].to(cache.dtype)
+        return norm_reference(proj[:, :Q], q_norm, None, eps, False).to(dtype)
+    _check_dtype(dtype)
+    _typed(q_norm, kv_norm, cache, dtype=dtype)
+    if proj.stride(1) != 1 or proj.shape[1] < Q + R or slots.dtype != torch.int32 or slots.numel() != T or cache.shape[-1] != R:
+        raise TypeError("latent_norm_cache: unexpected shapes or dtypes")
+    q = torch.empty((T, Q), dtype=dtype, device=proj.device)
+    rc = _lib.get_lib().mfb_latent_norm_cache(proj.data_ptr(), proj.stride(0), q_norm.data_ptr(), kv_norm.data_ptr(), float(eps),
+                                              slots.data_ptr(), q.data_ptr(), cache.data_ptr(), T, Q, R,
+                                              int(dtype == torch.float32), _lib.stream_ptr())
+    _lib.check(rc, "mfb_latent_norm_cache")
+    _lib.count_launch()
+    return q
+
+
+def gate_heads_(x: torch.Tensor, gate: torch.Tensor) -> torch.Tensor:
+    """``x [T, n]`` times ``sigmoid(gate [T, m])``, in place: a gate per column (m = n) or per n / m neighbouring columns."""
+    T, n = x.shape
+    m = gate.shape[1]
+    if n % m or gate.shape[0] != T:
+        raise ValueError(f"{m} gates for {n} columns")
+    if not x.is_cuda:
+        return x.copy_((x.float().view(T, m, n // m) * torch.sigmoid(gate.float())[..., None]).view(T, n))
+    _check_dtype(x.dtype)
+    if gate.dtype != x.dtype or x.stride(1) != 1 or gate.stride(1) != 1:
+        raise TypeError("gate_heads_: matrices of one dtype with unit column stride expected")
+    rc = _lib.get_lib().mfb_gate_heads(x.data_ptr(), x.stride(0), gate.data_ptr(), gate.stride(0), T, n, m,
+                                       int(x.dtype == torch.float32), _lib.stream_ptr())
+    _lib.check(rc, "mfb_gate_heads")
+    _lib.count_launch()
+    return x
+
+
+def talk_mix(o: torch.Tensor, talk: torch.Tensor, gate: Optional[torch.Tensor]) -> torch.Tensor:
+    """Softmax weights mixed over heads, applied after the products with the values: ``o [T, H, G, DV]`` holds head g's weights
+    on the values of every key / value head; result ``[T, H * DV]``, head h ``sum_g talk[h, g] o[:, g, own head of h]`` times
+    ``sigmoid(gate [T, H * DV])``."""
+    T, H, G, DV = o.shape
+    if not o.is_cuda:
+        own = torch.arange(H) // (H // G)
+        y = torch.einsum("hg,tghv->thv", talk.float(), o.float()[:, :, own])
+        y = y.reshape(T, H * DV)
+        return (y if gate is None else y * torch.sigmoid(gate.float())).to(o.dtype)
+    _check_dtype(o.dtype)
+    if talk.dtype != torch.float32 or talk.shape != (H, H) or not talk.is_contiguous() or not o.is_contiguous() or (
+            gate is not None and (gate.dtype != o.dtype or gate.shape != (T, H * DV) or gate.stride(1) != 1)):
+        raise TypeError("talk_mix: unexpected shapes or dtypes")
+    y = torch.empty((T, H * DV), dtype=o.dtype, device=o.device)
+    rc = _lib.get_lib().mfb_talk_mix(o.data_ptr(), talk.data_ptr(), _lib.ptr(gate), 0 if gate is None else gate.stride(0),
+                                     y.data_ptr(), T, H, G, DV, int(o.dtype == torch.float32), _lib.stream_ptr())
+    _lib.check(rc, "mfb_talk_mix")
+    _lib.count_launch()
+    return y

@@ -38,6 +38,7 @@ class AttnMeta:
     kv_carry: Optional[object] = None     # modules.seq_pipe.KVCarry: keys / values of the earlier sequence chunks
     layer_run: Optional[int] = None       # position of the running layer in the stack (its cache; layers that share
                                           # weights run more than once)
+    loop_step: Optional[torch.Tensor] = None   # vector that enters the residual stream before the running layer
     cp_rank_positions: bool = False       # positions already hold the context-parallel offsets
 
 

@@ -14,12 +14,13 @@ from typing import List, Optional
 from ..spec_utils import ModuleSpec
 from .attention import CrossAttention, MLASelfAttention, MLASelfAttentionMegatron, SelfAttention
 from .delta_rule import GatedDeltaMixer, ParallelMixer
+from .matrix_memory import MatrixMemoryMixer
 from .mlp import MLP
 from .moe import GroupedMLP, MoELayer, SharedExpertMLP, TopKRouter
 from .mtp import MultiTokenPredictionBlock, MultiTokenPredictionLayer
 from .norm import build_norm
-from .ragged_attention import RaggedSelfAttention
-from .transformer_layer import (OutputNormTransformerLayer, StreamTransformerLayer, TransformerLayer,
+from .ragged_attention import RaggedLatentAttention, RaggedSelfAttention
+from .transformer_layer import (OutputNormTransformerLayer, SandwichTransformerLayer, StreamTransformerLayer, TransformerLayer,
                                 TransformerLayerSubmodules)
 
 
@@ -66,7 +67,8 @@ def get_output_norm_layer_spec(config) -> ModuleSpec:
         post_attn_layernorm=norm, post_mlp_layernorm=norm if ff else None))
 
 
-_MIXERS = {"attention": RaggedSelfAttention, "delta": GatedDeltaMixer, "parallel": ParallelMixer}
+_MIXERS = {"attention": RaggedSelfAttention, "latent": RaggedLatentAttention, "delta": GatedDeltaMixer,
+           "matrix_memory": MatrixMemoryMixer, "parallel": ParallelMixer}
 
 
 def get_stream_layer_spec(config, is_moe: bool) -> ModuleSpec:
@@ -79,12 +81,27 @@ def get_stream_layer_spec(config, is_moe: bool) -> ModuleSpec:
         pre_mlp_layernorm=norm if mlp is not None else None))
 
 
+def get_sandwich_layer_spec(config, is_moe: bool) -> ModuleSpec:
+    """Spec of one layer with norms on both sides of its sub-layers: ``config.mixer``, then an MoE or dense feed-forward
+    (none with ``ffn_hidden_size == 0``)."""
+    norm = ModuleSpec(module=build_norm)
+    mlp = get_mlp_module_spec(config.num_moe_experts if is_moe else None) if is_moe or config.ffn_hidden_size else None
+    after = norm if mlp is not None else None
+    return ModuleSpec(module=SandwichTransformerLayer, submodules=TransformerLayerSubmodules(
+        input_layernorm=norm, self_attention=ModuleSpec(module=_MIXERS[config.mixer]), post_attn_layernorm=norm, mlp=mlp,
+        pre_mlp_layernorm=after, post_mlp_layernorm=after))
+
+
 def get_gpt_layer_spec_for_config(config, is_moe: bool) -> ModuleSpec:
     """``get_gpt_layer_local_spec`` with the switches taken from a ``TransformerConfig``."""
     if config.residual_streams:
         if config.norm_placement != "input" or not config.ragged_attention or config.normalization != "RMSNorm":
             raise ValueError("layers on residual streams are pre-norm layers with RMS norms and ragged attention")
         return get_stream_layer_spec(config, is_moe)
+    if config.norm_placement == "both":
+        if not config.ragged_attention or config.normalization != "RMSNorm":
+            raise ValueError("layers with norms on both sides are built with ragged attention and RMS norms")
+        return get_sandwich_layer_spec(config, is_moe)
     if config.norm_placement == "output":
         if is_moe or not config.ragged_attention:
             raise ValueError("output-normalised layers are built with ragged attention and a dense feed-forward")

@@ -37,9 +37,23 @@ class LanguageModelEmbedding(nn.Module):
         self.word_embeddings = VocabParallelEmbedding(config.vocab_size, config.hidden_size, config=config,
                                                       reduce_scatter_embeddings=sp)
         self.sp = sp
+        # an fp32 stream starts from scaled rows plus sinusoidal position vectors
+        self.scale, self.sinusoidal = float(config.embedding_scale), config.position_embedding_type == "sinusoidal"
+        self.stream = self.sinusoidal or self.scale != 1.0
+        if self.stream:
+            if not config.fp32_residual_connection or ps.get_tensor_model_parallel_world_size() > 1:
+                raise NotImplementedError("scaled or sinusoidal embeddings start an fp32 stream on one tensor-parallel rank")
+            self.freqs = stream.sinusoidal_frequencies(config.hidden_size) if self.sinusoidal else None
 
-    def forward(self, input_ids):
-        return self.word_embeddings(input_ids)
+    def forward(self, input_ids, positions=None):
+        if not self.stream:
+            return self.word_embeddings(input_ids)
+        w = self.word_embeddings.weight
+        if self.freqs is not None and self.freqs.device != w.device:
+            self.freqs = self.freqs.to(w.device)
+        if positions is None:
+            positions = torch.arange(input_ids.shape[-1], device=w.device).expand(input_ids.shape)
+        return stream.embed(input_ids.reshape(-1), w, self.scale, positions.reshape(-1), self.freqs)
 
 
 class GPTModel(nn.Module):
@@ -100,6 +114,8 @@ class GPTModel(nn.Module):
         cap = self.config.logit_softcap
         if cap:          # fp32 accumulators -> cap * tanh(x / cap), element-wise (a vocabulary shard needs no other rank)
             return stream.linear(hidden, w, act="softcap", cap=float(cap))
+        if self.config.norm_placement == "both" and ps.get_tensor_model_parallel_world_size() == 1:
+            return stream.linear(hidden, w, out_dtype=torch.float32)
         y, _ = self.output_layer(hidden, weight=w)
         return y
 
@@ -130,7 +146,7 @@ class GPTModel(nn.Module):
             if self.embedding.sp:
                 hidden = M.scatter_to_sequence_parallel_region(hidden)
         elif self.pre_process:
-            hidden = self.embedding(input_ids)
+            hidden = self.embedding(input_ids, meta.positions) if self.embedding.stream else self.embedding(input_ids)
         else:
             hidden = self.input_tensor
         rotary = self.rotary_pos_emb() if self.rotary_pos_emb is not None else None

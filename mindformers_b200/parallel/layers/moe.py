@@ -46,6 +46,8 @@ class TopKRouter(nn.Module):
         self.weight = nn.Parameter(w.to(config.moe_router_dtype))
         self.weight.sequence_parallel = bool(config.sequence_parallel)
         self.weight.no_weight_decay = False
+        self.register_parameter("bias", nn.Parameter(torch.zeros(E, dtype=config.moe_router_dtype, device=dev))
+                                if config.moe_router_logit_bias else None)
         self.topk = config.moe_router_topk
         self.score_fn = config.moe_router_score_function
         if config.moe_router_enable_expert_bias:
@@ -56,7 +58,7 @@ class TopKRouter(nn.Module):
             self.expert_load = None
 
     def gating(self, x):
-        return F.linear(x.to(self.weight.dtype), self.weight).float()
+        return F.linear(x.to(self.weight.dtype), self.weight, self.bias).float()
 
     def _select(self, scores):
         cfg = self.config
@@ -243,6 +245,8 @@ class GroupedMLP(nn.Module):
         cfg = self.config
         if cfg.moe_activation == "clamped_glu":
             return Fn.clamped_glu(h, cfg.moe_activation_limit, cfg.moe_activation_alpha, plan)
+        if h.is_cuda and not torch.is_grad_enabled() and (h.dtype == torch.float32 or getattr(plan, "seg_fill", None) is not None):
+            return Fn.clamped_glu(h, float("inf"), 1.0, plan, shift=0.0)        # padding rows skipped, any width, fp32 too
         return Fn.swiglu(h)
 
     def quantize_fp8_(self) -> bool:

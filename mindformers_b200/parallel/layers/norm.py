@@ -71,4 +71,9 @@ def get_norm(config):
 
 
 def build_norm(config, hidden_size=None, eps=None):
-    return get_norm(config)(config, hidden_size or config.hidden_size, eps or config.layernorm_epsilon)
+    """Norm of the residual width. With ``config.layernorm_zero_centered_gamma`` in a stack with norms on both sides, whose
+    fused step adds the one (``ops/stream.py::normed_step``), the weight is stored around zero."""
+    norm = get_norm(config)(config, hidden_size or config.hidden_size, eps or config.layernorm_epsilon)
+    if config.norm_placement == "both" and config.layernorm_zero_centered_gamma:
+        nn.init.zeros_(norm.weight)
+    return norm

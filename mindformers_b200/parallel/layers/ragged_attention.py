@@ -2,9 +2,11 @@
 
 ``RaggedSelfAttention`` is the serving counterpart of ``SelfAttention`` for models whose attention has one or more of:
 key and value sizes that differ, per-layer sizes and rotary settings, a chunked mask (``attention_chunk_size``), a
-softmax sink (``attention_sink``), soft-capped scores (``attention_softcap``), no rotation at all (``rotary_dim = 0``),
-projection biases folded into the following kernel. Parameter names are those of ``SelfAttention`` plus ``sink [heads]``
-(fp32). ``RaggedAttentionCore`` is what lies between the projections, for mixers that share them with something else. One kernel applies bias, q / k norm and rotation and writes the cache
+softmax sink (``attention_sink``), soft-capped scores (``attention_softcap``), no rotation at all (``rotary_dim = 0``), a
+sliding window (``attention_window``), norms without weights (``qk_unit_norm``, ``value_unit_norm``), weights mixed over heads
+(``attention_talk``), an output gate (``attention_output_gate``), projection biases folded into the following kernel. Parameter
+names are those of ``SelfAttention`` plus ``sink [heads]`` and ``talk [heads, heads]`` (fp32). ``RaggedLatentAttention`` caches
+one latent per token instead of keys and values. ``RaggedAttentionCore`` is what lies between the projections, for mixers that share them with something else. One kernel applies bias, q / k norm and rotation and writes the cache
 (``ops/stream.py::qkv_rope_cache``); one call attends for all sequences of the batch
 (``inference/ragged_attention.py``).
 """
@@ -59,32 +61,57 @@ class RaggedAttentionCore(nn.Module):
         self.scale = config.softmax_scale or 1.0 / math.sqrt(D)
         self.chunk = int(config.attention_chunk_size or 0)
         self.softcap = float(config.attention_softcap or 0.0)
+        self.window = int(config.attention_window or 0)
+        self.unit_qk, self.unit_v = bool(config.qk_unit_norm), bool(config.value_unit_norm)
+        if self.unit_qk and config.qk_layernorm:
+            raise ValueError(f"layer {layer_number}: qk_unit_norm and qk_layernorm exclude one another")
+        if config.attention_talk and tp > 1:
+            raise NotImplementedError("softmax weights mixed over heads need every head on one tensor-parallel rank")
+        self.register_parameter("talk", nn.Parameter(torch.eye(H, dtype=torch.float32, device=dev)) if config.attention_talk else None)
 
     def cache_shape(self):
         """``(kv heads, key size, value size)`` of this rank's cache."""
         return self.nkv, self.dim, self.v_dim
 
-    def attend(self, qkv, bias, meta: AttnMeta, out=None, out_scale: float = 1.0):
+    def attend(self, qkv, bias, meta: AttnMeta, out=None, out_scale: float = 1.0, gate=None):
         """``qkv [T, sum(sections)]`` (this rank's rows; any row pitch) → ``[T, heads * v_dim]`` times ``out_scale``, in ``out``
-        when given."""
+        when given; ``gate``: times its sigmoid."""
         from ...inference.ragged_attention import ragged_attention
         cache, layer = meta.cache, cache_layer(meta, self.layer_number)
         qn = self.q_layernorm.weight if self.q_layernorm is not None else None
         kn = self.k_layernorm.weight if self.k_layernorm is not None else None
         q = stream.qkv_rope_cache(qkv, bias, qn, kn, self.config.layernorm_epsilon, self.rotary.freqs, self.rotary.amplitude,
                                   self.config.rotary_interleaved, meta.positions, cache.slot_mapping,
-                                  cache.key_cache[layer], cache.value_cache[layer], self.nq, self.nkv, self.dim, self.v_dim)
-        return ragged_attention(q, cache, layer, self.scale, self.chunk, self.sink, self.softcap, out, out_scale)
+                                  cache.key_cache[layer], cache.value_cache[layer], self.nq, self.nkv, self.dim, self.v_dim,
+                                  self.unit_qk, self.unit_v)
+        if self.talk is not None:
+            if out is not None or out_scale != 1.0:
+                raise NotImplementedError("softmax weights mixed over heads write a result of their own")
+            o = ragged_attention(q, cache, layer, self.scale, self.chunk, self.sink, self.softcap, window=self.window, all_values=True)
+            return stream.talk_mix(o.view(o.shape[0], self.nq, self.nkv, self.v_dim), self.talk, gate)
+        out = ragged_attention(q, cache, layer, self.scale, self.chunk, self.sink, self.softcap, out, out_scale, self.window)
+        return out if gate is None else stream.gate_heads_(out, gate)
 
 
 class RaggedSelfAttention(RaggedAttentionCore):
-    """Returns ``(output without bias, output bias)``: the step behind the sub-layer adds the bias."""
+    """Returns ``(output without bias, output bias)``: the step behind the sub-layer adds the bias. With an output gate its
+    rows follow those of q, k and v in the input projection, and the bias of q, k and v is a parameter of its own."""
 
     def __init__(self, config, layer_number: int = 1):
         super().__init__(config, layer_number)
-        self.linear_qkv = ColumnParallelLinear(config.hidden_size, sum(self.sections), config=config,
-                                               bias=config.add_qkv_bias or config.add_bias_linear, skip_bias_add=True,
-                                               partition_sections=self.sections)
+        bias = bool(config.add_qkv_bias or config.add_bias_linear)
+        H, tp = config.num_attention_heads, ps.get_tensor_model_parallel_world_size()
+        gates = {None: 0, "head": H, "channel": H * self.v_dim}[config.attention_output_gate]
+        if gates and tp > 1:
+            raise NotImplementedError("gated ragged attention runs on one tensor-parallel rank")
+        sections = self.sections + ((gates,) if gates else ())
+        self.linear_qkv = ColumnParallelLinear(config.hidden_size, sum(sections), config=config, bias=bias and not gates,
+                                               skip_bias_add=True, partition_sections=sections)
+        self.n_qkv = sum(self.sections) // tp if not gates else sum(self.sections)
+        self.gated = gates > 0
+        w = self.linear_qkv.weight
+        self.register_parameter("qkv_bias", nn.Parameter(torch.zeros(sum(self.sections), dtype=w.dtype, device=w.device))
+                                if bias and gates else None)
         self.linear_proj = RowParallelLinear(config.num_attention_heads * self.v_dim, config.hidden_size, config=config,
                                              skip_bias_add=True,
                                              bias=config.add_attention_output_bias or config.add_bias_linear)
@@ -92,4 +119,48 @@ class RaggedSelfAttention(RaggedAttentionCore):
     def forward(self, hidden, rotary, meta: AttnMeta):
         cache_layer(meta, self.layer_number)
         qkv, bias = self.linear_qkv(hidden)
+        if self.gated:
+            return self.linear_proj(self.attend(qkv[:, :self.n_qkv], self.qkv_bias, meta, gate=qkv[:, self.n_qkv:]))
         return self.linear_proj(self.attend(qkv, bias, meta))
+
+
+class RaggedLatentAttention(nn.Module):
+    """Latent attention without positions: queries through a normed latent, keys and values linear in one cached, normed latent
+    of ``kv_lora_rank`` numbers per token. Returns ``(output, None)``. One projection makes the query latent, the key / value
+    latent and the output gates; one kernel norms both latents and writes the cache (``ops/stream.py::latent_norm_cache``)."""
+
+    def __init__(self, config, layer_number: int = 1):
+        super().__init__()
+        if ps.get_tensor_model_parallel_world_size() > 1:
+            raise NotImplementedError("ragged latent attention runs on one tensor-parallel rank")
+        self.layer_number, self.eps = layer_number, config.layernorm_epsilon
+        H, D, DV, Q, R = (config.num_attention_heads, config.kv_channels, config.v_channels or config.kv_channels, config.q_lora_rank,
+                          config.kv_lora_rank)
+        self.heads, self.dim, self.v_dim, self.rank = H, D, DV, R
+        self.scale, self.window = config.softmax_scale or 1.0 / math.sqrt(D), int(config.attention_window or 0)
+        gates = {None: 0, "head": H, "channel": H * DV}[config.attention_output_gate]
+        self.sections = (Q, R) + ((gates,) if gates else ())
+        linear = lambda cols, rows: ColumnParallelLinear(cols, rows, config=config, bias=False)
+        self.linear_in = linear(config.hidden_size, sum(self.sections))
+        self.q_latent_norm, self.kv_latent_norm = RMSNorm(config, Q, self.eps), RMSNorm(config, R, self.eps)
+        self.linear_q_up, self.linear_kv_up = linear(Q, H * D), linear(R, H * (D + DV))
+        dev = self.linear_in.weight.device
+        self.register_parameter("sink", nn.Parameter(torch.zeros(H, dtype=torch.float32, device=dev)) if config.attention_sink else None)
+        self.linear_proj = RowParallelLinear(H * DV, config.hidden_size, config=config)
+
+    def cache_shape(self):
+        return 1, self.rank, 0
+
+    def forward(self, hidden, rotary, meta: AttnMeta):
+        from ...inference.ragged_attention import latent_attention
+        cache, layer = meta.cache, cache_layer(meta, self.layer_number)
+        proj, _ = self.linear_in(hidden)
+        n = sum(self.sections[:2])
+        c = stream.latent_norm_cache(proj[:, :n], self.q_latent_norm.weight, self.kv_latent_norm.weight, self.eps, cache.slot_mapping,
+                                     cache.key_cache[layer])
+        q, _ = self.linear_q_up(c)
+        out = latent_attention(q.view(-1, self.heads, self.dim), cache, layer, self.linear_kv_up.weight, self.v_dim, self.scale,
+                               self.window, self.sink)
+        if len(self.sections) > 2:
+            out = stream.gate_heads_(out, proj[:, n:])
+        return self.linear_proj(out)

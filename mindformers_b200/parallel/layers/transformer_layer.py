@@ -203,6 +203,61 @@ class StreamTransformerLayer(nn.Module):
         return pending, residual, aux if self.mlp is not None and self.is_moe else None
 
 
+@dataclass
+class NormedResidual:
+    """The fp32 stream and the norm through which the pending sub-layer output has yet to enter it (None: nothing pends)."""
+    x: torch.Tensor
+    norm: Any = None
+
+
+class SandwichTransformerLayer(nn.Module):
+    """Layer with an fp32 residual stream and norms on both sides of every sub-layer: ``x <- x + norm_b(mixer(norm_a(x)))``,
+    then the same with the feed-forward (dense or MoE; none without an ``mlp``). With ``config.token_shift`` the mixer reads
+    ``h + (h of the token before - h) * mu``. A serving layer: entering the stream, the next norm and the shift are one kernel
+    (``ops/stream.py::normed_step``), across layers too, since a layer's last output stays pending."""
+
+    normed_residual = True        # ``residual`` is a ``NormedResidual`` that still lacks ``pending``
+
+    def __init__(self, config, layer_number: int = 1, submodules: Optional[TransformerLayerSubmodules] = None):
+        super().__init__()
+        self.config, self.layer_number = config, layer_number
+        self.input_layernorm = build_module(submodules.input_layernorm, config)
+        self.self_attention = build_module(submodules.self_attention, config, layer_number)
+        self.post_attn_layernorm = build_module(submodules.post_attn_layernorm, config)
+        self.register_parameter("token_shift", nn.Parameter(torch.zeros_like(self.input_layernorm.weight))
+                                if config.token_shift else None)
+        self.mlp = self.pre_mlp_layernorm = self.post_mlp_layernorm = None
+        self.is_moe = False
+        if submodules.mlp is not None:
+            mlp_cls = getattr(submodules.mlp, "module", submodules.mlp)
+            self.is_moe = isinstance(mlp_cls, type) and issubclass(mlp_cls, MoELayer)
+            self.pre_mlp_layernorm = build_module(submodules.pre_mlp_layernorm, config)
+            self.mlp = build_module(submodules.mlp, config, layer_number) if self.is_moe else build_module(submodules.mlp, config)
+            self.post_mlp_layernorm = build_module(submodules.post_mlp_layernorm, config)
+
+    def _enter(self, pending, res: NormedResidual, norm, meta: AttnMeta, step=None, shift=None):
+        """Let ``pending`` enter the stream; returns the input of the sub-layer behind ``norm`` and the new stream."""
+        carry = None
+        if shift is not None:
+            if meta.cache is None:
+                raise RuntimeError("token shift serves from a cache: generate() or the serving engine provide one")
+            carry = stream.Carry(shift, meta.cache, meta.layer_run - meta.cache.layer_offset)
+        return stream.normed_step(res.x, pending if res.norm is not None else None, res.norm.weight if res.norm is not None else None,
+                                  step, norm.weight, norm.eps, self.config.layernorm_zero_centered_gamma, carry)
+
+    def forward(self, pending, residual: Optional[NormedResidual], rotary, meta: AttnMeta):
+        if residual is None:
+            residual = NormedResidual(pending)
+        h, x = self._enter(pending, residual, self.input_layernorm, meta, meta.loop_step, self.token_shift)
+        pending, _ = self.self_attention(h, rotary, meta)
+        residual, aux = NormedResidual(x, self.post_attn_layernorm), None
+        if self.mlp is not None:
+            h, x = self._enter(pending, residual, self.pre_mlp_layernorm, meta)
+            pending, aux = self.mlp(h)
+            residual = NormedResidual(x, self.post_mlp_layernorm)
+        return pending, residual, aux if self.is_moe else None
+
+
 def pipeline_layer_split(num_layers: int, pp: int, vpp: int = 1, offset=0) -> List[List[List[int]]]:
     """Layer ids of every (pp stage, virtual chunk). ``offset`` adds/removes layers per stage
     (list of pp values, or vpp lists of pp values), as the reference's ``LayerSetting`` does."""
@@ -280,8 +335,21 @@ class TransformerBlock(nn.Module):
             with module_rng(base_seed, 100 + i, dev):     # a layer's initial weights depend on its number only
                 built.append(build_module(layer_specs[i], config.for_layer(i), layer_number=i + 1))
         self.layers = StageLayers(own_ids, built)
-        # the layers in running order: a layer that shares weights is its owner's module once more
-        self.run_order = [own_ids.index(o) for o in owners]
+        # the layers in running order: a layer that shares weights is its owner's module once more, a looped layer runs in
+        # every pass; every run has a number (``run_ids``), and with it a cache, of its own
+        self.run_order, self.run_ids = [own_ids.index(o) for o in owners], list(self.layer_ids)
+        self.run_steps = [None] * len(self.run_order)
+        self.register_parameter("loop_step", None)
+        if config.layer_loop is not None:
+            if pp * vpp > 1:
+                raise NotImplementedError("looped layers stay on one pipeline stage")
+            runs = config.layer_runs()
+            self.run_order, self.run_ids = [own_ids.index(i) for i, _ in runs], list(range(len(runs)))
+            self.run_steps = [t for _, t in runs]
+            with module_rng(base_seed, 90, dev):
+                self.loop_step = nn.Parameter(torch.empty(int(config.layer_loop[2]), config.hidden_size, dtype=torch.float32,
+                                                          device=dev or ("cuda" if torch.cuda.is_available() else "cpu"))
+                                              .normal_(0.0, config.init_method_std).to(config.params_dtype))
         self.final_layernorm = build_norm(config) if post_process else None
         self.recompute = bool(config.recompute) if not isinstance(config.recompute, (list, tuple)) else True
         self._recompute_layers = self._resolve_recompute(config.recompute)
@@ -314,6 +382,10 @@ class TransformerBlock(nn.Module):
         """Per layer run the recurrent state's shape (``KVCacheContext``) or None; None when no layer has one."""
         shapes = [getattr(self.layers[at].self_attention, "state_shape", lambda: None)() for at in self.run_order]
         return shapes if any(s is not None for s in shapes) else None
+
+    def carry_width(self) -> int:
+        """Width of the vector that every layer run carries from one token of a sequence to the next (0: none)."""
+        return self.config.hidden_size if any(getattr(layer, "token_shift", None) is not None for layer in self.layers) else 0
 
     def _setup_selective_recompute_and_offload(self, config):
         from ..recompute import ActivationOffloader, mark_recompute_modules
@@ -377,12 +449,14 @@ class TransformerBlock(nn.Module):
             self._offload.prune()
         for idx, at in enumerate(self.run_order):
             layer = run = self.layers[at]
-            meta.layer_run = self.layer_ids[idx]
+            meta.layer_run = self.run_ids[idx]
+            if self.loop_step is not None:
+                meta.loop_step = None if self.run_steps[idx] is None else self.loop_step[self.run_steps[idx]]
             if self.params_ready_hook is not None:
-                self.params_ready_hook(self.layer_ids[idx])
+                self.params_ready_hook(self.layers.layer_ids[at])
             if training and self.grads_final_hook is not None and pending.requires_grad:
                 # the gradient of a layer's input is the last thing its backward pass produces
-                def fire(_grad, _cb=self.grads_final_hook, _gid=self.layer_ids[idx]):
+                def fire(_grad, _cb=self.grads_final_hook, _gid=self.layers.layer_ids[at]):
                     _cb(_gid)
                 pending.register_hook(fire)
             if training and self._offload is not None and idx in self._offload_layers:
@@ -404,6 +478,12 @@ class TransformerBlock(nn.Module):
                 raise NotImplementedError("residual streams stay on one pipeline stage")
             out, _ = stream.residual_streams(residual.x, old.read.numel(), pending, old.mix, old.write, None, norm.weight,
                                              norm.eps, keep=False)
+        elif getattr(layer, "normed_residual", False):
+            norm = self.final_layernorm
+            if norm is None:
+                raise NotImplementedError("an fp32 stream with a pending norm stays on one pipeline stage")
+            out, _ = stream.normed_step(residual.x, pending, residual.norm.weight, None, norm.weight, norm.eps,
+                                        self.config.layernorm_zero_centered_gamma, keep=False)
         elif getattr(layer, "stream_in_residual", False):
             norm = self.final_layernorm
             out = residual if norm is None else stream.norm_stream(residual, norm.weight, getattr(norm, "bias", None), norm.eps,

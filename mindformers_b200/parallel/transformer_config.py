@@ -132,10 +132,20 @@ class TransformerConfig(ModelParallelConfig):
     layer_overrides: Optional[List[dict]] = None
     # per layer, the index of the layer whose weights it uses (its own index: weights of its own); None: no sharing
     layer_sharing: Optional[List[int]] = None
-    norm_placement: str = "input"           # "input": pre-norm; "output": x + scale * norm(sublayer(x)), fp32 stream
+    norm_placement: str = "input"           # "input": pre-norm; "output": x + scale * norm(sublayer(x)), fp32 stream;
+                                            # "both": x + norm(sublayer(norm(x))), fp32 stream
+    layer_loop: Optional[tuple] = None      # (start, stop, times): these layers run so many times in a row with the same
+                                            # weights; before pass t a learned vector (row t) is added to the stream
+    token_shift: bool = False               # norm_placement "both": a mixer reads h + (h of the token before - h) * mu
+    embedding_scale: float = 1.0            # factor of the embedding rows (fp32 streams)
     residual_streams: int = 0               # > 0: that many fp32 streams with learned reads, writes and mixing (pre-norm)
-    mixer: str = "attention"                # with residual_streams: "attention", "delta" (gated delta rule) or "parallel"
+    mixer: str = "attention"                # with residual_streams or norm_placement "both": "attention", "latent" (cached
+                                            # latents), "delta" (gated delta rule), "matrix_memory" (mLSTM) or "parallel"
                                             # (attention beside a gated delta rule, both on the same input)
+    memory_heads: int = 0                   # matrix memory: heads, sizes per head and the soft cap of its gates
+    memory_key_dim: int = 0
+    memory_value_dim: int = 0
+    memory_gate_cap: float = 15.0
     parallel_scales: Optional[tuple] = None  # weights of the two outputs of a parallel mixer
     delta_heads: int = 0                    # gated delta rule: value heads,
     delta_kv_heads: int = 0                 #   query / key heads (each serves delta_heads / delta_kv_heads value heads),
@@ -154,6 +164,11 @@ class TransformerConfig(ModelParallelConfig):
     attention_chunk_size: int = 0           # > 0: a position sees its own chunk of that many positions only
     attention_softcap: Optional[float] = None   # attention scores <- cap * tanh(scores / cap), fp32
     attention_sink: bool = False            # learned per-head term in the softmax denominator
+    attention_window: int = 0               # > 0: a position sees itself and the attention_window - 1 positions before it
+    qk_unit_norm: bool = False              # RMS norm of q and k per head without a weight
+    value_unit_norm: bool = False           # RMS norm of the values per head without a weight
+    attention_talk: bool = False            # the softmax weights of the heads are mixed by a learned [heads, heads] matrix
+    attention_output_gate: Optional[str] = None   # sigmoid gate on the heads' outputs, per "channel" or per "head"
     logit_softcap: Optional[float] = None   # logits <- cap * tanh(logits / cap), fp32
     # ---- init ----
     init_method: Optional[Callable] = None
@@ -218,6 +233,7 @@ class TransformerConfig(ModelParallelConfig):
     moe_router_score_function: str = "softmax"
     moe_router_dtype: Union[str, torch.dtype] = "float32"
     moe_router_enable_expert_bias: bool = False
+    moe_router_logit_bias: bool = False     # learned bias of the router's logits (selection and weights)
     moe_router_bias_update_rate: float = 1e-3
     moe_grouped_gemm: bool = True
     moe_aux_loss_coeff: float = 0.0
@@ -338,12 +354,19 @@ class TransformerConfig(ModelParallelConfig):
                 self.moe_aux_loss_coeff = float(self.aux_loss_factors[self.aux_loss_types.index("expert")])
         elif self.expert_model_parallel_size > 1:
             raise ValueError("expert_model_parallel_size > 1 needs num_moe_experts")
-        if self.mixer not in ("attention", "delta", "parallel") or self.delta_decay not in ("head", "channel") \
+        if self.mixer not in ("attention", "latent", "delta", "matrix_memory", "parallel") or self.delta_decay not in ("head", "channel") \
                 or self.delta_gate not in ("silu", "sigmoid") or self.moe_activation not in ("swiglu", "clamped_glu"):
             raise ValueError(f"unknown mixer {self.mixer!r}, decay {self.delta_decay!r}, gate {self.delta_gate!r} or expert "
                              f"activation {self.moe_activation!r}")
-        if self.norm_placement not in ("input", "output"):
-            raise ValueError(f"norm_placement must be 'input' or 'output', got {self.norm_placement!r}")
+        if self.norm_placement not in ("input", "output", "both"):
+            raise ValueError(f"norm_placement must be 'input', 'output' or 'both', got {self.norm_placement!r}")
+        if self.attention_output_gate not in (None, "channel", "head"):
+            raise ValueError(f"attention_output_gate must be None, 'channel' or 'head', got {self.attention_output_gate!r}")
+        if self.layer_loop is not None:
+            start, stop, times = (int(x) for x in self.layer_loop)
+            if not 0 <= start < stop <= self.num_layers or times < 1 or self.layer_sharing:
+                raise ValueError(f"layer_loop {self.layer_loop} of {self.num_layers} layers"
+                                 + (" beside layer_sharing" if self.layer_sharing else ""))
         for name in ("layer_overrides", "layer_sharing"):
             val = getattr(self, name)
             if val is not None and len(val) != self.num_layers:
@@ -385,6 +408,17 @@ class TransformerConfig(ModelParallelConfig):
     def shares_weights_with(self, index: int) -> int:
         """The layer that owns the weights layer ``index`` runs with."""
         return index if not self.layer_sharing else int(self.layer_sharing[index])
+
+    def layer_runs(self) -> List[tuple]:
+        """``(layer, pass)`` of every layer run in order; ``pass`` counts the passes of ``layer_loop`` and is None except for
+        the first layer of a pass."""
+        if self.layer_loop is None:
+            return [(i, None) for i in range(self.num_layers)]
+        start, stop, times = (int(x) for x in self.layer_loop)
+        runs = [(i, None) for i in range(start)]
+        for t in range(times):
+            runs += [(i, t if i == start else None) for i in range(start, stop)]
+        return runs + [(i, None) for i in range(stop, self.num_layers)]
 
     def moe_layer_pattern(self) -> List[int]:
         """1 for MoE layers, 0 for dense layers (``first_k_dense_replace`` wins over ``moe_layer_freq``)."""
