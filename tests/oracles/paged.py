@@ -3,14 +3,14 @@ import torch
 
 from mindformers_b200.inference.paged_attention import KVCacheContext
 
-from . import mefesun
+from . import gavatar, mefesun
 
 
 def attention_case(dtype, H, G, D, DV, bs, chunk, lens, news, seed=0, sink_scale=1.0, spots=(), softcap=0.0, score_scale=1.3,
-                   device="cuda"):
+                   device="cuda", window=0, all_values=False):
     """A paged cache with shuffled pages and the step's queries. ``spots``: (sequence, query position, key position) whose
     score is made to stand out (it decides the row where it is visible, and nothing where it is hidden). With ``softcap`` the scores
-    are capped and there is no sink."""
+    are capped and there is no sink, as with ``all_values`` (every head's weights on the values of every KV head)."""
     B = len(lens)
     g = torch.Generator().manual_seed(seed)
     per = [-(-n // bs) for n in lens]
@@ -49,6 +49,12 @@ def attention_case(dtype, H, G, D, DV, bs, chunk, lens, news, seed=0, sink_scale
         if softcap:
             s = softcap * torch.tanh(s / softcap)
         mask = mefesun.chunk_mask(n, chunk if chunk else n)[n - m:]
-        p = mefesun.softmax_with_sink(s, mask, sink.double() if not softcap else torch.full((H,), -1e30, dtype=torch.float64))
-        want.append(torch.einsum("hqk,khd->qhd", p, vs[b].double().repeat_interleave(reps, 1)))
-    return ctx, table, qs, sink, scale, torch.cat(want).reshape(sum(news), H * DV)
+        if window:
+            mask = mask & gavatar.window_mask(n, window)[n - m:]
+        none = softcap or all_values
+        p = mefesun.softmax_with_sink(s, mask, sink.double() if not none else torch.full((H,), -1e30, dtype=torch.float64))
+        if all_values:
+            want.append(torch.einsum("hqk,kgd->qhgd", p, vs[b].double()))
+        else:
+            want.append(torch.einsum("hqk,khd->qhd", p, vs[b].double().repeat_interleave(reps, 1)))
+    return ctx, table, qs, sink, scale, torch.cat(want).reshape(sum(news), -1)
