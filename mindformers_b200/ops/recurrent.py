@@ -248,5 +248,5 @@ def matrix_memory(proj: torch.Tensor, input_bias: torch.Tensor, forget_bias: tor
                                cache.slot_mapping.data_ptr(), scratch, out.data_ptr(), T, B, H, D, DV, longest, s.gate_cap, float(eps),
                                f32, _lib.stream_ptr())
     _lib.check(rc, "mfb_matrix_memory")
-    _lib.count_launch(2 if cache.is_prefill else 1)
+    _lib.count_launch(3 if cache.is_prefill else 1)
     return out
