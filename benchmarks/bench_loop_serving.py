@@ -48,7 +48,7 @@ def kernel_table(size, prompt_batch=4, prompt=4096, decode_batch=64, context=409
     """Every kernel of a layer of the two models, prefill (``prompt_batch`` prompts) and decode shapes; ``only``: a part of the
     kernels' names."""
     from mindformers_b200.inference.paged_attention import mla_decode_attention
-    from mindformers_b200.inference.ragged_attention import latent_attention, ragged_attention
+    from mindformers_b200.inference.ragged_attention import latent_attention, ragged_attention, talking_attention
     from mindformers_b200.ops import functional as Fn
     from mindformers_b200.ops import recurrent, stream
     from mindformers_b200.parallel.layers.attention import AttnMeta
@@ -97,7 +97,7 @@ def kernel_table(size, prompt_batch=4, prompt=4096, decode_batch=64, context=409
         q = new(T, H, D)
         kv_bytes = B * min(WIN, ctx_len) * G * D * 4 if n == 1 else 0
         talk_flop = seen * H * (4 * D + 2 * H)
-        mixed = lambda: stream.talk_mix(ragged_attention(q, cm, 3, sa.scale, window=WIN, all_values=True).view(T, H, G, D), sa.talk, gate)
+        mixed = lambda: talking_attention(q, cm, 3, sa.scale, sa.talk, gate, WIN)
         add(f"{phase} attention", "gavatar window, mixed weights, gate", mixed, kv_bytes or T * (3 * H + 2 * G) * D * 2,
             talk_flop if n > 1 else 0)
         add(f"{phase} attention", "gavatar kernel, window alone", lambda: ragged_attention(q, cm, 3, sa.scale, window=WIN),

@@ -127,12 +127,13 @@ def _scratch(cache, name: str, need: int, device):
 
 def ragged_attention(q: torch.Tensor, cache, layer: int, scale: float, chunk: int = 0,
                      sink: Optional[torch.Tensor] = None, softcap: float = 0.0, out: Optional[torch.Tensor] = None,
-                     out_scale: float = 1.0, window: int = 0, all_values: bool = False) -> torch.Tensor:
+                     out_scale: float = 1.0, window: int = 0, all_values: bool = False, singles: bool = True) -> torch.Tensor:
     """q ``[T, heads, dim]`` of the step's new tokens, whose keys and values are in the cache already → ``[T, heads *
     v_dim]``. ``chunk`` > 0: a position sees its own chunk of that many positions (counted from 0) only; ``window`` > 0: it sees
     itself and the ``window - 1`` positions before it. ``sink [heads]`` fp32: adds ``exp(sink)`` to the softmax denominator.
     ``softcap`` > 0: scores become ``softcap * tanh(score / softcap)``. ``all_values``: every head's weights are applied to the
     values of every key / value head: ``[T, heads * kv_heads * v_dim]``. A layer without values of its own attends over its keys.
+    ``singles`` False: the result of sequences with one new row in a ragged step may be left undefined.
     ``out``: a matrix (any row pitch that keeps rows on 16 bytes) to write to; the result is multiplied by ``out_scale``."""
     kc, vc = cache.key_cache[layer], _values(cache, layer)
     T, Hq, D = q.shape
@@ -165,7 +166,7 @@ def ragged_attention(q: torch.Tensor, cache, layer: int, scale: float, chunk: in
         work, persistent = _work_on_device(cache, int(chunk), int(window))
         _prefill_tc(lib, q, kc.data_ptr(), Hkv * D, Hkv, nb * bs, vc.data_ptr(), Hkv * DV, work, persistent, cache.block_tables, sink,
                     out, D, DV, bs, chunk, window, all_values, scale, softcap, out_scale)
-    if not ragged or cache.n_single_rows:
+    if not ragged or (cache.n_single_rows and singles):
         reach = max_blocks * bs
         for span in (chunk, window):
             if span > 0:
@@ -180,6 +181,42 @@ def ragged_attention(q: torch.Tensor, cache, layer: int, scale: float, chunk: in
             float(out_scale), status, _lib.stream_ptr())
         _lib.check(rc, "mfb_paged_decode_attention_tc_ex")
         _lib.count_launch(2)
+    return out
+
+
+def talking_attention(q: torch.Tensor, cache, layer: int, scale: float, talk: torch.Tensor, gate: Optional[torch.Tensor] = None,
+                      window: int = 0) -> torch.Tensor:
+    """Attention whose softmax weights are mixed over heads (head h uses ``sum_g talk[h, g] weights_g`` on the values of its own
+    key / value head), times ``sigmoid(gate)``: q ``[T, heads, dim]``, talk ``[heads, heads]`` fp32, gate ``[T, heads * v_dim]`` →
+    ``[T, heads * v_dim]``. Decoded rows are one kernel and its merge; portions apply every head's weights to the values of every
+    key / value head and mix the results."""
+    from ..ops import stream
+    T, H, D = q.shape
+    G, DV = cache.value_cache[layer].shape[2:]
+    lib = _lib.get_lib() if q.is_cuda else None
+    fused = lib is not None and q.dtype == torch.bfloat16 and lib.mfb_paged_talk_decode_supported(H, G, D, DV, cache.block_size)
+    if cache.is_prefill or not fused:
+        o = ragged_attention(q, cache, layer, scale, window=window, all_values=True, singles=not fused)
+        out = stream.talk_mix(o.view(T, H, G, DV), talk, gate)
+        if not fused or not cache.n_single_rows:
+            return out
+    else:
+        out = torch.empty((T, H * DV), dtype=q.dtype, device=q.device)
+    if gate is not None and (gate.dtype != q.dtype or gate.shape != out.shape or gate.stride(1) != 1):
+        raise TypeError("talking_attention: the gate must be a [T, heads * v_dim] matrix of q's dtype with unit column stride")
+    kc, vc = cache.key_cache[layer], cache.value_cache[layer]
+    B, max_blocks = cache.block_tables.shape
+    reach = max_blocks * cache.block_size if window <= 0 else min(max_blocks * cache.block_size, window + 128)
+    splits = lib.mfb_paged_talk_decode_splits(cache.n_single_rows if cache.is_prefill else B, reach)
+    scratch = _scratch(cache, "_ragged_talk_scratch" if cache.is_prefill else "_talk_scratch",
+                       lib.mfb_paged_talk_decode_scratch_bytes(B, H, G, DV, splits), q.device)
+    rc = lib.mfb_paged_talk_decode(q.data_ptr(), kc.data_ptr(), vc.data_ptr(), cache.block_tables.data_ptr(),
+                                   cache.context_lens.data_ptr(), cache.cu_q_dev.data_ptr() if cache.is_prefill else 0, talk.data_ptr(),
+                                   _lib.ptr(gate), 0 if gate is None else gate.stride(0), out.data_ptr(), scratch.data_ptr(), splits, T,
+                                   B, H, G, D, DV, kc.shape[0], cache.block_size, max_blocks, int(window), float(scale),
+                                   _lib.status_word(q.device).data_ptr(), _lib.stream_ptr())
+    _lib.check(rc, "mfb_paged_talk_decode")
+    _lib.count_launch(2)
     return out
 
 

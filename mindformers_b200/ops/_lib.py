@@ -152,6 +152,10 @@ def _declare(lib):
     sig("mfb_talk_mix", [P, P, P, L, P, I, I, I, I, I, P])
     sig("mfb_matrix_memory_scratch_floats", [I] * 5, L)
     sig("mfb_matrix_memory", [P, L] + [P] * 11 + [I] * 6 + [F, F, I, P])
+    sig("mfb_paged_talk_decode_supported", [I] * 5)
+    sig("mfb_paged_talk_decode_splits", [I, I])
+    sig("mfb_paged_talk_decode_scratch_bytes", [I] * 5, L)
+    sig("mfb_paged_talk_decode", [P] * 8 + [L, P, P] + [I] * 11 + [F, P, P])
     sig("mfb_latent_decode_supported", [I, I])
     sig("mfb_latent_decode_splits", [I, I, I])
     sig("mfb_latent_decode_scratch_bytes", [I] * 4, L)

@@ -65,8 +65,8 @@ class RaggedAttentionCore(nn.Module):
         self.unit_qk, self.unit_v = bool(config.qk_unit_norm), bool(config.value_unit_norm)
         if self.unit_qk and config.qk_layernorm:
             raise ValueError(f"layer {layer_number}: qk_unit_norm and qk_layernorm exclude one another")
-        if config.attention_talk and tp > 1:
-            raise NotImplementedError("softmax weights mixed over heads need every head on one tensor-parallel rank")
+        if config.attention_talk and (tp > 1 or self.chunk or self.softcap or config.attention_sink):
+            raise NotImplementedError("softmax weights mixed over heads: one tensor-parallel rank, no chunks, no soft cap, no sink")
         self.register_parameter("talk", nn.Parameter(torch.eye(H, dtype=torch.float32, device=dev)) if config.attention_talk else None)
 
     def cache_shape(self):
@@ -76,7 +76,7 @@ class RaggedAttentionCore(nn.Module):
     def attend(self, qkv, bias, meta: AttnMeta, out=None, out_scale: float = 1.0, gate=None):
         """``qkv [T, sum(sections)]`` (this rank's rows; any row pitch) → ``[T, heads * v_dim]`` times ``out_scale``, in ``out``
         when given; ``gate``: times its sigmoid."""
-        from ...inference.ragged_attention import ragged_attention
+        from ...inference.ragged_attention import ragged_attention, talking_attention
         cache, layer = meta.cache, cache_layer(meta, self.layer_number)
         qn = self.q_layernorm.weight if self.q_layernorm is not None else None
         kn = self.k_layernorm.weight if self.k_layernorm is not None else None
@@ -87,8 +87,7 @@ class RaggedAttentionCore(nn.Module):
         if self.talk is not None:
             if out is not None or out_scale != 1.0:
                 raise NotImplementedError("softmax weights mixed over heads write a result of their own")
-            o = ragged_attention(q, cache, layer, self.scale, self.chunk, self.sink, self.softcap, window=self.window, all_values=True)
-            return stream.talk_mix(o.view(o.shape[0], self.nq, self.nkv, self.v_dim), self.talk, gate)
+            return talking_attention(q, cache, layer, self.scale, self.talk, gate, self.window)
         out = ragged_attention(q, cache, layer, self.scale, self.chunk, self.sink, self.softcap, out, out_scale, self.window)
         return out if gate is None else stream.gate_heads_(out, gate)
 

@@ -6,7 +6,7 @@ import torch
 
 from mindformers_b200.inference import ragged_attention as ragged
 from mindformers_b200.inference.paged_attention import KVCacheContext
-from mindformers_b200.inference.ragged_attention import latent_attention, ragged_attention
+from mindformers_b200.inference.ragged_attention import latent_attention, ragged_attention, talking_attention
 from mindformers_b200.ops import _lib, recurrent, stream
 from mindformers_b200.ops import functional as Fn
 from mindformers_b200.serving import SamplingParams, ServingEngine
@@ -217,6 +217,53 @@ def test_windowed_attention_at_the_edges(dtype, H, G, D, DV, window):
                 row = qp - (lens - news)
                 err = (got[row].double().cpu() - want[row]).norm() / want[row].norm()
                 assert float(err) < tol(dtype, 2e-5, 3e-2), (qp, kp, lens, news)
+    assert _lib.read_status() == 0
+
+
+TALK = [(4, 2, 64, 64), (32, 8, 128, 128), (6, 2, 40, 24), (6, 3, 48, 96), (20, 1, 24, 40), (34, 2, 16, 72), (3, 1, 20, 36),
+        (1, 1, 8, 8), (64, 4, 32, 64), (16, 16, 64, 32), (40, 5, 128, 128), (2, 1, 144, 12)]
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("H,G,D,DV", TALK)
+@pytest.mark.parametrize("window", [1, 100, 128, 5000])
+def test_mixed_weights(dtype, H, G, D, DV, window):
+    """Portions and decoded rows; a gate that lies in a wider matrix."""
+    talk, own = rand(H, H, seed=5) * H ** -0.5 + torch.eye(H), torch.arange(H) // (H // G)
+    for lens, news, bs, ragged_step in (([1, 300, 129, 257, 64, 700, 40], [1, 300, 2, 130, 1, 1, 0], 64, True),
+                                        ([70, 3], [1, 1], 64, True), ([1, 63, 64, 129, 900], [1] * 5, 16, False)):
+        ctx, table, qs, _, scale, o = attention_case(dtype, H, G, D, DV, bs, 0, lens, news, seed=D, window=window, all_values=True,
+                                                     score_scale=4.0)
+        T = sum(news)
+        gate = rand(T, H * DV + 8, seed=6, dtype=dtype)
+        want = torch.einsum("hg,tghv->thv", talk.double(), o.view(T, H, G, DV)[:, :, own]).reshape(T, H * DV)
+        want = want * torch.sigmoid(gate[:, :H * DV].double())
+        ctx.set_step(is_prefill=ragged_step, block_tables=table, slot_mapping=[0] * T, context_lens=lens, q_seq_lens=news, device=DEV)
+        got = talking_attention(torch.cat(qs).to(DEV), ctx, 0, scale, talk.to(DEV), gate.to(DEV)[:, :H * DV], window)
+        err = rows_rel(got, want)
+        assert float(err.max()) < tol(dtype, 2e-5, 3e-2), (ragged_step, lens, int(err.argmax()))
+    assert _lib.read_status() == 0
+
+
+@pytest.mark.parametrize("H,G,D,DV", [(8, 2, 128, 128), (6, 3, 48, 24)])
+@pytest.mark.parametrize("window", [64, 130])
+def test_mixed_weights_at_the_edges(H, G, D, DV, window):
+    """One key that stands out, just inside and just outside the window, decoded and in portions."""
+    talk, own = rand(H, H, seed=5) * H ** -0.5 + torch.eye(H), torch.arange(H) // (H // G)
+    for qp in (399, 383, 300, 128 + window, window, window - 1):
+        for kp in (qp - window + 1, qp - window, qp):
+            for lens, news in ((400, 400), (qp + 1, 2), (qp + 1, 1)):
+                if kp < 0 or kp >= lens:
+                    continue
+                ctx, table, qs, _, scale, o = attention_case(torch.bfloat16, H, G, D, DV, 16, 0, [lens], [news], seed=qp + kp,
+                                                             spots=[(0, qp, kp)], window=window, all_values=True)
+                want = torch.einsum("hg,tghv->thv", talk.double(), o.view(news, H, G, DV)[:, :, own]).reshape(news, H * DV)
+                ctx.set_step(is_prefill=news > 1, block_tables=table, slot_mapping=[0] * news, context_lens=[lens], q_seq_lens=[news],
+                             device=DEV)
+                got = talking_attention(qs[0].to(DEV), ctx, 0, scale, talk.to(DEV), None, window)
+                row = qp - (lens - news)
+                err = (got[row].double().cpu() - want[row]).norm() / want[row].norm()
+                assert float(err) < 3e-2, (qp, kp, lens, news)
     assert _lib.read_status() == 0
 
 
