@@ -64,6 +64,36 @@ gate_heads_kernel(T* __restrict__ x, long long ld_x, const T* __restrict__ gate,
   }
 }
 
+// bf16, eight columns per access; PER8: the eight columns share a gate
+template <bool PER8>
+__global__ void __launch_bounds__(256)
+gate_heads_vec_kernel(__nv_bfloat16* __restrict__ x, long long ld_x, const __nv_bfloat16* __restrict__ gate, long long ld_g, int T_rows,
+                      int n, int per) {
+  const int nv = n / 8;
+  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < (long long)T_rows * nv; i += (long long)gridDim.x * blockDim.x) {
+    const int t = (int)(i / nv), c = (int)(i % nv) * 8;
+    uint4* p = reinterpret_cast<uint4*>(x + t * ld_x + c);
+    uint4 u = *p;
+    __nv_bfloat162* v = reinterpret_cast<__nv_bfloat162*>(&u);
+    const __nv_bfloat16* g = gate + t * ld_g;
+    float s[8];
+    if constexpr (PER8) {
+      s[0] = sigmoid(ld(g + c / per));
+#pragma unroll
+      for (int k = 1; k < 8; ++k) s[k] = s[0];
+    } else {
+#pragma unroll
+      for (int k = 0; k < 8; ++k) s[k] = sigmoid(ld(g + c + k));
+    }
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      const float2 f = __bfloat1622float2(v[k]);
+      v[k] = __floats2bfloat162_rn(f.x * s[2 * k], f.y * s[2 * k + 1]);
+    }
+    *p = u;
+  }
+}
+
 constexpr int kAcc = 8;
 
 // a thread keeps up to eight result heads of one key / value head for VEC columns; the matrix lies in shared memory
@@ -115,6 +145,69 @@ talk_mix_kernel(const T* __restrict__ o, const float* __restrict__ talk, const T
   }
 }
 
+// bf16, DV a multiple of 8, up to GR heads per key / value head at a time: a thread keeps GR result heads of 8 columns. The matrix
+// lies in shared memory transposed, [g][h], so that the weights of a thread's heads are one vector.
+template <int GR>
+__global__ void __launch_bounds__(256)
+talk_mix_vec_kernel(const __nv_bfloat16* __restrict__ o, const float* __restrict__ talk, const __nv_bfloat16* __restrict__ gate,
+                    long long ld_g, __nv_bfloat16* __restrict__ y, long long T, int H, int G, int DV) {
+  extern __shared__ float sh[];
+  const int group = H / G, blocks = (group + GR - 1) / GR, hp = G * blocks * GR;      // heads, every group padded to GR
+  for (int i = threadIdx.x; i < H * hp; i += blockDim.x) {
+    const int g = i / hp, p = i % hp, kv = p / (blocks * GR), r = p % (blocks * GR);
+    sh[i] = r < group ? talk[(kv * group + r) * H + g] : 0.f;
+  }
+  __syncthreads();
+  const int nv = DV / 8, per = G * blocks * nv;
+  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < T * per; i += (long long)gridDim.x * blockDim.x) {
+    const long long t = i / per;
+    const int e = (int)(i % per), d = (e % nv) * 8, kb = e / nv, kv = kb / blocks;
+    const __nv_bfloat16* src = o + t * H * G * DV + kv * DV + d;
+    float acc[GR][8];
+#pragma unroll
+    for (int j = 0; j < GR; ++j)
+#pragma unroll
+      for (int k = 0; k < 8; ++k) acc[j][k] = 0.f;
+#pragma unroll 4
+    for (int g = 0; g < H; ++g) {
+      const uint4 u = *reinterpret_cast<const uint4*>(src + (long long)g * G * DV);
+      const __nv_bfloat162* p2 = reinterpret_cast<const __nv_bfloat162*>(&u);
+      const float* w = sh + g * hp + kb * GR;
+#pragma unroll
+      for (int k = 0; k < 4; ++k) {
+        const float2 f = __bfloat1622float2(p2[k]);
+#pragma unroll
+        for (int j = 0; j < GR; ++j) {
+          acc[j][2 * k] = fmaf(w[j], f.x, acc[j][2 * k]);
+          acc[j][2 * k + 1] = fmaf(w[j], f.y, acc[j][2 * k + 1]);
+        }
+      }
+    }
+#pragma unroll
+    for (int j = 0; j < GR; ++j) {
+      const int r = (kb % blocks) * GR + j;
+      if (r < group) {
+        const long long col = (long long)(kv * group + r) * DV + d;
+        float v[8];
+#pragma unroll
+        for (int k = 0; k < 8; ++k) v[k] = acc[j][k];
+        if (gate) {
+          const uint4 u = *reinterpret_cast<const uint4*>(gate + t * ld_g + col);
+          const __nv_bfloat162* z = reinterpret_cast<const __nv_bfloat162*>(&u);
+#pragma unroll
+          for (int k = 0; k < 4; ++k) {
+            const float2 f = __bfloat1622float2(z[k]);
+            v[2 * k] *= sigmoid(f.x);
+            v[2 * k + 1] *= sigmoid(f.y);
+          }
+        }
+        *reinterpret_cast<uint4*>(y + t * H * DV + col) = make_uint4(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]),
+                                                                     pack_bf16x2(v[4], v[5]), pack_bf16x2(v[6], v[7]));
+      }
+    }
+  }
+}
+
 bool al(const void* p, int n) { return (reinterpret_cast<uintptr_t>(p) & (n - 1)) == 0; }
 
 }  // namespace hmx
@@ -139,6 +232,15 @@ int mfb_latent_norm_cache(const void* proj, long long ld_proj, const void* q_nor
 int mfb_gate_heads(void* x, long long ld_x, const void* gate, long long ld_g, int T, int n, int m, int f32, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (n < 1 || m < 1 || n % m) { mfb_host::set_error("gate_heads: n=%d m=%d", n, m); return 1; }
+  if (!f32 && n % 8 == 0 && ld_x % 8 == 0 && hmx::al(x, 16) && (n / m == 1 || (n / m) % 8 == 0)) {
+    const long long want8 = ((long long)T * (n / 8) + 255) / 256;
+    const int grid8 = (int)(want8 < 148 * 16 ? want8 : 148 * 16);
+    __nv_bfloat16* xp = (__nv_bfloat16*)x;
+    const __nv_bfloat16* gp = (const __nv_bfloat16*)gate;
+    if (n / m == 1) hmx::gate_heads_vec_kernel<false><<<grid8, 256, 0, stream>>>(xp, ld_x, gp, ld_g, T, n, 1);
+    else hmx::gate_heads_vec_kernel<true><<<grid8, 256, 0, stream>>>(xp, ld_x, gp, ld_g, T, n, n / m);
+    return cudaGetLastError() == cudaSuccess ? 0 : 2;
+  }
   const bool vec = n % 2 == 0 && ld_x % 2 == 0 && hmx::al(x, f32 ? 8 : 4);
   const long long items = (long long)T * (vec ? n / 2 : n);
   const long long want = (items + 255) / 256;
@@ -160,6 +262,20 @@ int mfb_talk_mix(const void* o, const float* talk, const void* gate, long long l
                  cudaStream_t stream) {
   if (T <= 0) return 0;
   if (G < 1 || H < 1 || H % G || DV < 1) { mfb_host::set_error("talk_mix: H=%d G=%d DV=%d", H, G, DV); return 1; }
+  if (!f32 && DV % 8 == 0 && hmx::al(o, 16) && hmx::al(y, 16) && (!gate || (hmx::al(gate, 16) && ld_g % 8 == 0))) {
+    const int group = H / G, gr = group <= 1 ? 1 : (group == 2 ? 2 : 4), blocks = (group + gr - 1) / gr;
+    const size_t bytes = (size_t)H * G * blocks * gr * 4;
+    if (bytes <= 48 * 1024) {
+      const long long want = ((long long)T * G * blocks * (DV / 8) + 255) / 256;
+      const int grid = (int)(want < 148 * 8 ? want : 148 * 8);
+      const __nv_bfloat16 *op = (const __nv_bfloat16*)o, *gp = (const __nv_bfloat16*)gate;
+      __nv_bfloat16* yp = (__nv_bfloat16*)y;
+      if (gr == 1) hmx::talk_mix_vec_kernel<1><<<grid, 256, bytes, stream>>>(op, talk, gp, ld_g, yp, T, H, G, DV);
+      else if (gr == 2) hmx::talk_mix_vec_kernel<2><<<grid, 256, bytes, stream>>>(op, talk, gp, ld_g, yp, T, H, G, DV);
+      else hmx::talk_mix_vec_kernel<4><<<grid, 256, bytes, stream>>>(op, talk, gp, ld_g, yp, T, H, G, DV);
+      return cudaGetLastError() == cudaSuccess ? 0 : 2;
+    }
+  }
   const bool vec = DV % 2 == 0 && hmx::al(o, f32 ? 8 : 4) && hmx::al(y, f32 ? 8 : 4);
   const int in_smem = (size_t)H * H * 4 <= 48 * 1024;
   const size_t smem = in_smem ? (size_t)H * H * 4 : 0;

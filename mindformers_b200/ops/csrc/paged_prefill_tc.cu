@@ -15,8 +15,8 @@
 // loads and the first scores of a tile run under the last softmax and the output of the one before, which is what counts
 // when a tile sees few keys (chunks, short portions). What else differs:
 //   - a sliding window (`window` > 0) hides the keys that lie `window` or more positions before the row;
-//   - with `all_values` every query head's weights are applied to the values of every key / value head, one after the other
-//     (items of their own, so that K and q come from L2);
+//   - with `all_values` every query head's weights are applied to the values of every key / value head: by a kernel of its own
+//     (below), with a sink or a soft cap as items of their own;
 //   - rows of K and V may lie further apart than their heads fill (slices of one product);
 //   - work comes as a list of (sequence, first row of q, rows, position of the first row), one entry per query tile; only
 //     key tiles that some row of the tile sees are visited, from the chunk of its first row to its last row;
@@ -475,6 +475,333 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
   }
 }
 
+// ---- every head's weights on the values of every key / value head ---------------------------------------------------------------
+// The products with the values are G times those of ordinary attention, so scores and softmax of a key tile serve NV = 256 / HV
+// value heads at once: their accumulators fill half of tensor memory, two score buffers the other half, and one CTA owns the SM.
+// The scores of key tile j + 1 are computed before the products of tile j with the values, under which their softmax then runs.
+// Eight softmax warps share a query tile: a row belongs to two threads, 64 key columns each, which exchange their maxima (and, at
+// the end, their sums) through shared memory and keep the scores in registers in between; each writes one half of the results.
+//
+// Roles (320 threads): warp 0 TMA producer, warp 1 MMA issuer + TMEM owner, warps 2..9 softmax. Every wait is bounded.
+constexpr int kAvThreads = 320;
+constexpr int kAvRing = 96 * 1024;         // V tiles
+
+template <int HQ, int HV>
+__global__ void __launch_bounds__(kAvThreads, 1)
+paged_prefill_values_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
+                            const __grid_constant__ CUtensorMap tmV, const Args args, const int G) {
+  constexpr int QB = HQ / 64, VB = HV / 64, NV = 256 / HV;
+  constexpr int kQBytes = QB * kSubBytes, kVBytes = VB * kSubBytes, kSlots = kAvRing / kVBytes;
+  extern __shared__ uint8_t smem_raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~static_cast<uintptr_t>(1023));
+  uint8_t* sQ = smem;
+  uint8_t* sK = sQ + kQBytes;                        // two stages
+  uint8_t* sV = sK + 2 * kQBytes;                    // ring
+  uint8_t* sOut = sV + kAvRing;                      // 2 KB per softmax warp
+  float* sMax = reinterpret_cast<float*>(sOut + 8 * 2048);        // [2 tiles][2 halves][128]
+  float* sSum = sMax + 4 * kTile;                    // [2 halves][128]
+  uint64_t* bars = reinterpret_cast<uint64_t*>(sSum + 2 * kTile);
+  uint64_t* q_full = bars;
+  uint64_t* q_empty = bars + 1;
+  uint64_t* k_full = bars + 2;                       // 2
+  uint64_t* k_empty = bars + 4;                      // 2
+  uint64_t* s_full = bars + 6;                       // 2
+  uint64_t* p_ready = bars + 8;
+  uint64_t* pv_done = bars + 9;                      // 2: a tile's softmax may end before the products of the tile before
+  uint64_t* v_full = bars + 11;                      // kSlots
+  uint64_t* v_empty = v_full + kSlots;
+  uint32_t* tmem_holder = reinterpret_cast<uint32_t*>(v_empty + kSlots);
+  volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_holder + 1);
+
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int vblocks = (G + NV - 1) / NV;
+  struct Tile { int b, head, v0, nv, q0, rows, pos0, lo, n_kv; };     // value heads v0 .. v0 + nv - 1, key tiles lo .. n_kv - 1
+  auto first_of = [&](int pos) {
+    int lo = args.chunk > 0 ? pos - pos % args.chunk : 0;
+    if (args.window > 0 && pos - args.window + 1 > lo) lo = pos - args.window + 1;
+    return lo;
+  };
+  auto tile_of = [&](int item) {
+    Tile t;
+    t.v0 = item % vblocks * NV;
+    t.nv = G - t.v0 < NV ? G - t.v0 : NV;
+    item /= vblocks;
+    const int4 w = args.work[item / args.num_q_heads];
+    t.head = item % args.num_q_heads;
+    t.b = w.x; t.q0 = w.y; t.rows = w.z; t.pos0 = w.w;
+    t.lo = first_of(t.pos0) / kTile;
+    t.n_kv = (t.pos0 + t.rows - 1) / kTile + 1;
+    return t;
+  };
+  const int first_item = static_cast<int>(blockIdx.x), step = static_cast<int>(gridDim.x);
+
+  if (threadIdx.x == 0) {
+    *abort_flag = 0;
+    for (int i = 0; i < 11 + 2 * kSlots; ++i) mbar_init(smem_u32(&bars[i]), &bars[i] == p_ready ? 256 : 1);
+    fence_barrier_init();
+    tma_prefetch_desc(&tmQ);
+    tma_prefetch_desc(&tmK);
+    tma_prefetch_desc(&tmV);
+  }
+  if (warp == 1) {
+    tmem_alloc(smem_u32(tmem_holder), 512);
+    tmem_relinquish();
+  }
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem_base = *tmem_holder;
+  const uint32_t tmem_O = tmem_base + 2 * kTile;     // P of a tile lives in the first 64 columns of its scores
+
+  if (warp == 0) {
+    // ------------------------------ TMA producer ------------------------------
+    if (lane == 0) {
+      const int bs = args.block_size, pages = kTile / bs;
+      uint32_t it = 0, n = 0, unit = 0;              // key tiles, query tiles and V tiles so far
+      bool ok = true;
+      for (int item = first_item; item < args.n_items && ok; item += step, ++n) {
+        const Tile t = tile_of(item);
+        ok = mbar_wait(smem_u32(q_empty), (n & 1) ^ 1, abort_flag, args.status, kStatusWaitTimeoutProducer);
+        if (!ok) break;
+        const uint32_t qb = smem_u32(q_full);
+        mbar_expect_tx(qb, kQBytes);
+        for (int c = 0; c < QB; ++c) tma_load_3d(smem_u32(sQ) + c * kSubBytes, &tmQ, qb, c * 64, t.head, t.q0);
+        const int* table = args.block_tables + static_cast<size_t>(t.b) * args.max_blocks;
+        const int end = t.pos0 + t.rows, kcol = t.head / args.group * args.D;
+        auto load = [&](const CUtensorMap* tm, uint32_t dst, uint32_t bar, int j, int col, int subs) {
+          const int tok0 = j * kTile, first_page = table[tok0 / bs];
+          for (int i = 0; i < pages; ++i) {
+            const int pg = tok0 + i * bs < end ? table[tok0 / bs + i] : first_page;
+            for (int c = 0; c < subs; ++c) tma_load_2d(dst + c * kSubBytes + i * bs * 128, tm, bar, col + c * 64, pg * bs);
+          }
+        };
+        auto load_k = [&](int j) {
+          const int st = it & 1;
+          ok = mbar_wait(smem_u32(&k_empty[st]), ((it >> 1) & 1) ^ 1, abort_flag, args.status, kStatusWaitTimeoutProducer);
+          if (!ok) return;
+          mbar_expect_tx(smem_u32(&k_full[st]), kQBytes);
+          load(&tmK, smem_u32(sK) + st * kQBytes, smem_u32(&k_full[st]), j, kcol, QB);
+          ++it;
+        };
+        load_k(t.lo);
+        for (int j = t.lo; j < t.n_kv && ok; ++j) {
+          if (j + 1 < t.n_kv) load_k(j + 1);
+          for (int v = 0; v < t.nv && ok; ++v, ++unit) {
+            const int slot = unit % kSlots;
+            ok = mbar_wait(smem_u32(&v_empty[slot]), ((unit / kSlots) & 1) ^ 1, abort_flag, args.status, kStatusWaitTimeoutProducer);
+            if (!ok) break;
+            mbar_expect_tx(smem_u32(&v_full[slot]), kVBytes);
+            load(&tmV, smem_u32(sV) + slot * kVBytes, smem_u32(&v_full[slot]), j, (t.v0 + v) * args.DV, VB);
+          }
+        }
+      }
+    }
+    __syncwarp();
+  } else if (warp == 1) {
+    // ------------------------------ MMA issuer ------------------------------
+    if (lane == 0) {
+      constexpr uint32_t IDESC_QK = umma_idesc_bf16(kTile, kTile, 0, 0);
+      constexpr uint32_t IDESC_PV = umma_idesc_bf16(kTile, HV, 0, 1);
+      const uint32_t qa = smem_u32(sQ), va0 = smem_u32(sV);
+      uint32_t it = 0, n = 0, unit = 0;
+      bool ok = true, first_key = true;              // first_key: the pending products start their query tile's sums
+      int pending = 0;                               // value heads of the pending products
+      // O(v) (+)= P V(v) of key tile it - 1
+      auto issue_pv = [&]() {
+        ok = mbar_wait(smem_u32(p_ready), (it - 1) & 1, abort_flag, args.status, kStatusWaitTimeoutMma);
+        const uint32_t pa = tmem_base + ((it - 1) & 1) * kTile;
+        for (int v = 0; v < pending && ok; ++v, ++unit) {
+          const int slot = unit % kSlots;
+          ok = mbar_wait(smem_u32(&v_full[slot]), (unit / kSlots) & 1, abort_flag, args.status, kStatusWaitTimeoutMma);
+          if (!ok) return;
+          tc_fence_after();
+#pragma unroll
+          for (int k = 0; k < kTile / 16; ++k)
+            umma_f16_ts(tmem_O + v * HV, pa + k * 8, umma_desc_mnmajor_sw128(va0 + slot * kVBytes + k * 16 * 128, kSubBytes), IDESC_PV,
+                        (!first_key || k > 0) ? 1u : 0u);
+          umma_commit(smem_u32(&v_empty[slot]));
+        }
+        if (ok) umma_commit(smem_u32(&pv_done[(it - 1) & 1]));
+      };
+      for (int item = first_item; item < args.n_items && ok; item += step, ++n) {
+        const Tile t = tile_of(item);
+        for (int j = t.lo; j < t.n_kv && ok; ++j) {
+          if (j == t.lo) ok = mbar_wait(smem_u32(q_full), n & 1, abort_flag, args.status, kStatusWaitTimeoutMma);
+          const int st = it & 1;
+          if (ok) ok = mbar_wait(smem_u32(&k_full[st]), (it >> 1) & 1, abort_flag, args.status, kStatusWaitTimeoutMma);
+          if (!ok) break;
+          tc_fence_after();
+          // these scores overwrite those whose products with the values were issued before the last ones
+          const uint32_t ka = smem_u32(sK) + st * kQBytes;
+#pragma unroll
+          for (int k = 0; k < HQ / 16; ++k) {
+            const uint32_t off = (k >> 2) * kSubBytes + (k & 3) * 32;
+            umma_f16_ss(tmem_base + st * kTile, umma_desc_kmajor_sw128(qa + off), umma_desc_kmajor_sw128(ka + off), IDESC_QK,
+                        k > 0 ? 1u : 0u);
+          }
+          umma_commit(smem_u32(&s_full[st]));
+          umma_commit(smem_u32(&k_empty[st]));
+          if (j == t.n_kv - 1) umma_commit(smem_u32(q_empty));
+          if (it > 0) issue_pv();
+          first_key = j == t.lo;
+          pending = t.nv;
+          ++it;
+        }
+      }
+      if (ok && it > 0) issue_pv();
+    }
+    __syncwarp();
+  } else {
+    // ------------------------------ softmax warpgroups ------------------------------
+    const int ew = warp & 3, half = (warp - 2) >> 2;
+    const int row = ew * 32 + lane;
+    const uint32_t lane_base = static_cast<uint32_t>(ew * 32) << 16;
+    bool ok = true;
+    const uint64_t scale2 = pack2(args.scale_log2, args.scale_log2);
+    uint32_t it = 0;
+    for (int item = first_item; item < args.n_items; item += step) {
+      const Tile t = tile_of(item);
+      const int my_pos = t.pos0 + row, my_first = first_of(my_pos);
+      float m_used = -INFINITY, l_sum = 0.f;
+      for (int j = t.lo; j < t.n_kv; ++j, ++it) {
+        const uint32_t s_tmem = tmem_base + (it & 1) * kTile + lane_base;
+        ok = mbar_wait(smem_u32(&s_full[it & 1]), (it >> 1) & 1, abort_flag, args.status, kStatusWaitTimeoutEpilogue) && ok;
+        tc_fence_after();
+        uint32_t sr[64];
+        {
+          uint32_t (&ra)[32] = *reinterpret_cast<uint32_t(*)[32]>(&sr[0]);
+          uint32_t (&rb)[32] = *reinterpret_cast<uint32_t(*)[32]>(&sr[32]);
+          tmem_ld_32x32b_x32(s_tmem + half * 64, ra);
+          tmem_ld_32x32b_x32(s_tmem + half * 64 + 32, rb);
+          tmem_ld_wait();
+        }
+        float* s = reinterpret_cast<float*>(sr);
+        // columns [col_lo, col_hi] of this half are visible to the row; the bounds grow with the row
+        const int col_lo = my_first - j * kTile - half * 64, col_hi = my_pos - j * kTile - half * 64;
+        if (__shfl_sync(0xffffffffu, col_hi, 0) < 63 || __shfl_sync(0xffffffffu, col_lo, 31) > 0) {
+#pragma unroll
+          for (int i = 0; i < 64; ++i)
+            if (i > col_hi || i < col_lo) s[i] = -INFINITY;
+        }
+        float mxs[4];
+#pragma unroll
+        for (int a = 0; a < 4; ++a) {
+          float m = s[a * 16];
+#pragma unroll
+          for (int i = 1; i + 1 < 16; i += 2) m = fmax3(m, s[a * 16 + i], s[a * 16 + i + 1]);
+          mxs[a] = fmaxf(m, s[a * 16 + 15]);
+        }
+        float* mx_of = sMax + (it & 1) * 2 * kTile;
+        mx_of[half * kTile + row] = fmaxf(fmaxf(mxs[0], mxs[1]), fmaxf(mxs[2], mxs[3])) * args.scale_log2;
+        named_bar_sync(1, 256);                      // both halves have their scores in registers, too
+        const float mx = fmaxf(mx_of[row], mx_of[kTile + row]);
+        float alpha = 1.f;
+        if (j == t.lo) {
+          m_used = mx;
+        } else if (mx > m_used + kRescaleThreshold) {
+          alpha = ex2(m_used - mx);
+          m_used = mx;
+        }
+        if (j > t.lo && __any_sync(0xffffffffu, alpha != 1.f)) {
+          // products up to tile j - 1 have to be complete; the next ones wait for p_ready below
+          ok = mbar_wait(smem_u32(&pv_done[(it - 1) & 1]), ((it - 1) >> 1) & 1, abort_flag, args.status, kStatusWaitTimeoutEpilogue) && ok;
+          tc_fence_after();
+#pragma unroll 1
+          for (int c = 0; c < 8; ++c) {
+            uint32_t r[16];
+            const uint32_t o = tmem_O + lane_base + half * 128 + c * 16;
+            tmem_ld_32x32b_x16(o, r);
+            tmem_ld_wait();
+#pragma unroll
+            for (int i = 0; i < 16; ++i) r[i] = __float_as_uint(__uint_as_float(r[i]) * alpha);
+            tmem_st_32x32b_x16(o, r);
+          }
+        }
+        const float neg_m = m_used == -INFINITY ? 0.f : -m_used;
+        const uint64_t negm2 = pack2(neg_m, neg_m);
+        uint64_t rs2[4] = {0, 0, 0, 0};
+        uint32_t pk[32];
+#pragma unroll
+        for (int i = 0; i < 32; ++i) {
+          float x0, x1;
+          unpack2(fma2(pack2(s[2 * i], s[2 * i + 1]), scale2, negm2), x0, x1);
+          const float e0 = ex2(x0), e1 = ex2(x1);
+          rs2[i & 3] = add2(rs2[i & 3], pack2(e0, e1));
+          pk[i] = pack_bf16x2(e0, e1);
+        }
+        tmem_st_32x32b_x32(s_tmem + half * 32, pk);
+        float r0, r1, r2, r3;
+        unpack2(add2(rs2[0], rs2[1]), r0, r1);
+        unpack2(add2(rs2[2], rs2[3]), r2, r3);
+        l_sum = l_sum * alpha + ((r0 + r1) + (r2 + r3));
+        tmem_st_wait();
+        tc_fence_before();
+        mbar_arrive(smem_u32(p_ready));
+      }
+      ok = mbar_wait(smem_u32(&pv_done[(it - 1) & 1]), ((it - 1) >> 1) & 1, abort_flag, args.status, kStatusWaitTimeoutEpilogue) && ok;
+      sSum[half * kTile + row] = l_sum;
+      ok = named_bar_and(2, 256, ok);
+      if (!ok) break;
+      tc_fence_after();
+      const float inv_l = args.out_scale / (sSum[row] + sSum[kTile + row]);
+      uint8_t* stage = sOut + (half * 4 + ew) * 2048;
+      __nv_bfloat16* obase = args.out + (t.q0 + ew * 32) * args.ld_out + static_cast<size_t>(t.head * G + t.v0) * args.DV;
+#pragma unroll 1
+      for (int c = 0; c < 4; ++c) {
+        const int at = half * 128 + c * 32, v = at / HV, col0 = at % HV;
+        uint32_t r[32];
+        tmem_ld_32x32b_x32(tmem_O + lane_base + at, r);
+        tmem_ld_wait();
+#pragma unroll
+        for (int q = 0; q < 4; ++q)
+          *reinterpret_cast<uint4*>(stage + lane * 64 + ((q ^ ((lane >> 1) & 3)) << 4)) = make_uint4(
+              pack_bf16x2(__uint_as_float(r[q * 8 + 0]) * inv_l, __uint_as_float(r[q * 8 + 1]) * inv_l),
+              pack_bf16x2(__uint_as_float(r[q * 8 + 2]) * inv_l, __uint_as_float(r[q * 8 + 3]) * inv_l),
+              pack_bf16x2(__uint_as_float(r[q * 8 + 4]) * inv_l, __uint_as_float(r[q * 8 + 5]) * inv_l),
+              pack_bf16x2(__uint_as_float(r[q * 8 + 6]) * inv_l, __uint_as_float(r[q * 8 + 7]) * inv_l));
+        __syncwarp();
+        const int col = col0 + (lane & 3) * 8;
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const int rr = i * 8 + (lane >> 2);
+          if (ew * 32 + rr < t.rows && col < args.DV && v < t.nv)
+            *reinterpret_cast<uint4*>(obase + rr * args.ld_out + v * args.DV + col) =
+                *reinterpret_cast<const uint4*>(stage + rr * 64 + (((lane & 3) ^ ((rr >> 1) & 3)) << 4));
+        }
+        __syncwarp();
+      }
+      // O is read: the next query tile's first products, which overwrite it, wait for the warps' next p_ready
+      tc_fence_before();
+    }
+  }
+  tc_fence_before();
+  __syncthreads();
+  if (warp == 1) {
+    tc_fence_after();
+    tmem_dealloc(tmem_base, 512);
+  }
+}
+
+template <int HQ, int HV>
+int launch_values(const CUtensorMap& tQ, const CUtensorMap& tK, const CUtensorMap& tV, Args a, int n_work, int G, cudaStream_t stream) {
+  constexpr int NV = 256 / HV, SLOTS = kAvRing / (HV / 64 * kSubBytes);
+  constexpr int SMEM = 3 * (HQ / 64 * kSubBytes) + kAvRing + 8 * 2048 + 6 * kTile * 4 + (11 + 2 * SLOTS) * 8 + 16 + 1024;
+  static_assert(SMEM <= 232448, "shared memory budget exceeded");
+  auto kern = paged_prefill_values_kernel<HQ, HV>;
+  static bool attr_set = false;
+  if (!attr_set) {
+    if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM) != cudaSuccess) {
+      mfb_host::set_error("paged_prefill_tc: cannot raise the shared memory limit");
+      return 10;
+    }
+    attr_set = true;
+  }
+  a.n_items = n_work * a.num_q_heads * ((G + NV - 1) / NV);
+  kern<<<a.n_items < 148 ? a.n_items : 148, kAvThreads, SMEM, stream>>>(tQ, tK, tV, a, G);
+  if (cudaGetLastError() != cudaSuccess) { mfb_host::set_error("paged_prefill_tc: launch failed"); return 11; }
+  return 0;
+}
+
 // three-dimensional map of q [T, Hq, D]: box of 128 tokens x 1 head x 64 columns; columns past D read as zero
 int make_q_map(CUtensorMap* out, const void* q, uint64_t T, uint64_t Hq, uint64_t D) {
   mfb_host::EncodeTiledFn enc = mfb_host::get_encode_tiled();
@@ -564,6 +891,12 @@ int mfb_paged_prefill_tc(const void* q, const void* key_cache, const void* value
   float power = a.scale_log2;
   for (int k = 0; k < 5; ++k, power *= a.cap_scale * a.cap_scale) a.cap_poly[k] = ppt::kTanhRatio[k] * power;
   a.ld_out = ld_out; a.out_scale = out_scale;
+  if (a.vheads > 1 && !sink && !(softcap > 0.f)) {
+    if (D > 64) return DV > 64 ? ppt::launch_values<128, 128>(tQ, tK, tV, a, n_work, Hkv, stream)
+                               : ppt::launch_values<128, 64>(tQ, tK, tV, a, n_work, Hkv, stream);
+    return DV > 64 ? ppt::launch_values<64, 128>(tQ, tK, tV, a, n_work, Hkv, stream)
+                   : ppt::launch_values<64, 64>(tQ, tK, tV, a, n_work, Hkv, stream);
+  }
   const int max_ctas = persistent ? 2 * 148 : a.n_items;
 #define MFB_PPT(HQ_, HV_) \
   return softcap > 0.f ? ppt::launch<HQ_, HV_, true>(tQ, tK, tV, a, max_ctas, stream) : ppt::launch<HQ_, HV_, false>(tQ, tK, tV, a, max_ctas, stream)

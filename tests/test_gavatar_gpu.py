@@ -154,8 +154,8 @@ def test_latent_norm_and_cache_write(dtype, Q, R):
 
 @pytest.mark.parametrize("dtype", DTYPES)
 def test_output_gates(dtype):
-    for T, n, m in ((3, 96, 96), (5, 96, 8), (4, 33, 11), (700, 512, 4)):
-        x, g = rand(T, n + 4, seed=1, dtype=dtype), rand(T, m + 3, seed=2, dtype=dtype)
+    for T, n, m in ((3, 96, 96), (5, 96, 8), (4, 33, 11), (700, 512, 4), (9, 96, 6), (3, 64, 32)):
+        x, g = rand(T, n + 8, seed=1, dtype=dtype), rand(T, m + 3, seed=2, dtype=dtype)
         wide = x.to(DEV)
         got = stream.gate_heads_(wide[:, :n], g.to(DEV)[:, :m])
         want = x[:, :n].double() * torch.sigmoid(g[:, :m].double()).repeat_interleave(n // m, 1)
