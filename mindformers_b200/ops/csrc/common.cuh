@@ -135,6 +135,20 @@ __device__ __forceinline__ void tma_load_3d(uint32_t smem_dst, const CUtensorMap
       ::"r"(smem_dst), "l"(reinterpret_cast<uint64_t>(m)), "r"(bar), "r"(x), "r"(y), "r"(z)
       : "memory");
 }
+// 128 consecutive tokens of a paged cache as `subs` swizzled sub-tiles of 64 columns (from column `col` on), `sub_bytes` apart in
+// shared memory: one box per page and sub-tile, issued by one lane each, so that neither the block-table lookups nor the issue of
+// the boxes queue up. To be called by a whole warp; the tile has at most 16 boxes. Pages at or past `end` may be unallocated:
+// the tile's first page stands in for them (the caller masks its tokens).
+__device__ __forceinline__ void tma_load_pages(uint32_t smem_dst, uint32_t sub_bytes, const CUtensorMap* m, uint32_t bar,
+                                               const int* table, int block_size, int tok0, int end, int col, int subs) {
+  const int lane = static_cast<int>(lane_id()), pages = 128 / block_size;
+  if (lane < pages * subs) {
+    const int i = lane % pages, c = lane / pages;
+    int pg = table[tok0 / block_size + (tok0 + i * block_size < end ? i : 0)];
+    if (pg < 0) pg = table[tok0 / block_size];
+    tma_load_2d(smem_dst + c * sub_bytes + i * block_size * 128, m, bar, col + c * 64, pg * block_size);
+  }
+}
 __device__ __forceinline__ void tma_store_2d(const CUtensorMap* m, uint32_t smem_src, int32_t x,
                                              int32_t y) {
   asm volatile("cp.async.bulk.tensor.2d.global.shared::cta.bulk_group [%0, {%2, %3}], [%1];"

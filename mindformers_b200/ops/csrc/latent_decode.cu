@@ -109,48 +109,31 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
   const uint32_t tmem_S = tmem_base + 128;        // 2 buffers of 16 columns, 32 apart
 
   if (warp == 0) {
-    // ------------------------------------ producer ------------------------------------
-    if (lane == 0 && n_tiles > 0) {
-      const uint32_t qb = smem_u32(q_full);
-      mbar_expect_tx(qb, subs * kQSub);
-      for (int c = 0; c < subs; ++c)
-        tma_load_2d(smem_u32(sQ) + c * kQSub, &tmQ, qb, c * 64, b * args.num_heads + head0);
-      const int bs = args.block_size;
-      const int pages = kTile / bs;            // pages per tile (block_size divides 128)
+    // ------------------------------------ producer (the whole warp) ------------------------------------
+    if (n_tiles > 0) {
+      if (lane == 0) mbar_expect_tx(smem_u32(q_full), subs * kQSub);
+      __syncwarp();
+      if (lane < subs) tma_load_2d(smem_u32(sQ) + lane * kQSub, &tmQ, smem_u32(q_full), lane * 64, b * args.num_heads + head0);
       const int* table = args.block_tables + static_cast<size_t>(b) * args.max_blocks;
       uint32_t unit = 0;
       bool ok = true;
       for (int j = 0; j < n_tiles && ok; ++j) {
-        const int tok0 = (t0 + j) * kTile;
-        int page_row[8];
-        const int first_page = table[tok0 / bs];
-        for (int i = 0; i < pages; ++i) {
-          // pages past the end of the sequence may be unallocated: read the tile's first page instead (masked)
-          int pg = (tok0 + i * bs < len) ? table[tok0 / bs + i] : first_page;
-          if (pg < 0) pg = first_page;
-          page_row[i] = pg * bs;
-        }
         // two passes over the tile's pairs: for S^T, then again for O^T
         for (int u = 0; u < 2 * units && ok; ++u) {
           const int slot = unit % kSlots;
-          const uint32_t ph = (unit / kSlots) & 1;
-          ok = mbar_wait(smem_u32(&empty[slot]), ph ^ 1, abort_flag, args.status, kStatusWaitTimeoutProducer);
+          ok = mbar_wait(smem_u32(&empty[slot]), ((unit / kSlots) & 1) ^ 1, abort_flag, args.status, kStatusWaitTimeoutProducer);
+          ok = __all_sync(0xffffffffu, ok);
           if (!ok) break;
-          const uint32_t fb = smem_u32(&full[slot]);
-          const uint32_t dst = smem_u32(sRing + slot * kUnit);
           const int pair = u < units ? u : u - units;
-          const bool two = 2 * pair + 1 < subs;
-          const int col0 = pair * 128;
-          mbar_expect_tx(fb, two ? kUnit : kSub);
-          for (int i = 0; i < pages; ++i) {
-            tma_load_2d(dst + i * bs * 128, &tmC, fb, col0, page_row[i]);
-            if (two) tma_load_2d(dst + kSub + i * bs * 128, &tmC, fb, col0 + 64, page_row[i]);
-          }
+          const int two = 2 * pair + 1 < subs ? 2 : 1;
+          if (lane == 0) mbar_expect_tx(smem_u32(&full[slot]), two * kSub);
+          __syncwarp();
+          tma_load_pages(smem_u32(sRing + slot * kUnit), kSub, &tmC, smem_u32(&full[slot]), table, args.block_size, (t0 + j) * kTile,
+                         len, pair * 128, two);
           ++unit;
         }
       }
     }
-    __syncwarp();
   } else if (warp == 1) {
     // ------------------------------------ MMA issuer ------------------------------------
     if (lane == 0 && n_tiles > 0) {

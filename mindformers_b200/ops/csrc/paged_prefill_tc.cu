@@ -179,48 +179,38 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
   const uint32_t tmem_base = *tmem_holder;
   const uint32_t tmem_S = tmem_base, tmem_O = tmem_base + kTile;   // P lives in the first 64 columns of S
   if (warp == 0) {
-    // ------------------------------ TMA producer ------------------------------
-    if (lane == 0) {
-      const int bs = args.block_size;
-      const int pages = kTile / bs;
-      uint32_t it = 0, n = 0;                      // key tiles and query tiles so far
-      bool ok = true;
-      for (int item = first_item; item < args.n_items && ok; item += step, ++n) {
-        const Tile t = tile_of(item);
-        ok = mbar_wait(smem_u32(q_empty), (n & 1) ^ 1, abort_flag, args.status, kStatusWaitTimeoutProducer);
+    // ------------------------------ TMA producer (the whole warp) ------------------------------
+    uint32_t it = 0, n = 0;                          // key tiles and query tiles so far
+    bool ok = true;
+    // wait until a buffer is free; the lanes agree on the outcome
+    auto wait_free = [&](uint64_t* bar, uint32_t parity) {
+      ok = mbar_wait(smem_u32(bar), parity, abort_flag, args.status, kStatusWaitTimeoutProducer);
+      ok = __all_sync(0xffffffffu, ok);
+    };
+    for (int item = first_item; item < args.n_items && ok; item += step, ++n) {
+      const Tile t = tile_of(item);
+      wait_free(q_empty, (n & 1) ^ 1);
+      if (!ok) break;
+      if (lane == 0) mbar_expect_tx(smem_u32(q_full), kQBytes);
+      __syncwarp();
+      if (lane < QB) tma_load_3d(smem_u32(sQ) + lane * kSubBytes, &tmQ, smem_u32(q_full), lane * 64, t.head, t.q0);
+      const int* table = args.block_tables + static_cast<size_t>(t.b) * args.max_blocks;
+      const int kv_head = t.head / args.group, end = t.pos0 + t.rows;
+      const int kcol = kv_head * args.D, vcol = (args.vheads > 1 ? t.vsel : kv_head) * args.DV;
+      for (int j = t.lo; j < t.n_kv; ++j, ++it) {
+        const uint32_t ph = it & 1;
+        wait_free(k_empty, ph ^ 1);
         if (!ok) break;
-        const uint32_t qb = smem_u32(q_full);
-        mbar_expect_tx(qb, kQBytes);
-        for (int c = 0; c < QB; ++c) tma_load_3d(smem_u32(sQ) + c * kSubBytes, &tmQ, qb, c * 64, t.head, t.q0);
-        const int* table = args.block_tables + static_cast<size_t>(t.b) * args.max_blocks;
-        const int kv_head = t.head / args.group, end = t.pos0 + t.rows;
-        const int kcol = kv_head * args.D, vcol = (args.vheads > 1 ? t.vsel : kv_head) * args.DV;
-        for (int j = t.lo; j < t.n_kv; ++j, ++it) {
-          const uint32_t ph = it & 1;
-          const int tok0 = j * kTile;
-          const int first_page = table[tok0 / bs];
-          ok = mbar_wait(smem_u32(k_empty), ph ^ 1, abort_flag, args.status, kStatusWaitTimeoutProducer);
-          if (!ok) break;
-          const uint32_t kb = smem_u32(k_full);
-          mbar_expect_tx(kb, kQBytes);
-          const uint32_t kd = smem_u32(sK);
-          for (int i = 0; i < pages; ++i) {
-            const int pg = tok0 + i * bs < end ? table[tok0 / bs + i] : first_page;
-            for (int c = 0; c < QB; ++c) tma_load_2d(kd + c * kSubBytes + i * bs * 128, &tmK, kb, kcol + c * 64, pg * bs);
-          }
-          ok = mbar_wait(smem_u32(v_empty), ph ^ 1, abort_flag, args.status, kStatusWaitTimeoutProducer);
-          if (!ok) break;
-          const uint32_t vb = smem_u32(v_full);
-          mbar_expect_tx(vb, kVBytes);
-          const uint32_t vd = smem_u32(sV);
-          for (int i = 0; i < pages; ++i) {
-            const int pg = tok0 + i * bs < end ? table[tok0 / bs + i] : first_page;
-            for (int c = 0; c < VB; ++c) tma_load_2d(vd + c * kSubBytes + i * bs * 128, &tmV, vb, vcol + c * 64, pg * bs);
-          }
-        }
+        if (lane == 0) mbar_expect_tx(smem_u32(k_full), kQBytes);
+        __syncwarp();
+        tma_load_pages(smem_u32(sK), kSubBytes, &tmK, smem_u32(k_full), table, args.block_size, j * kTile, end, kcol, QB);
+        wait_free(v_empty, ph ^ 1);
+        if (!ok) break;
+        if (lane == 0) mbar_expect_tx(smem_u32(v_full), kVBytes);
+        __syncwarp();
+        tma_load_pages(smem_u32(sV), kSubBytes, &tmV, smem_u32(v_full), table, args.block_size, j * kTile, end, vcol, VB);
       }
     }
-    __syncwarp();
   } else if (warp == 1) {
     // ------------------------------ MMA issuer ------------------------------
     if (lane == 0) {
@@ -554,49 +544,45 @@ paged_prefill_values_kernel(const __grid_constant__ CUtensorMap tmQ, const __gri
   const uint32_t tmem_O = tmem_base + 2 * kTile;     // P of a tile lives in the first 64 columns of its scores
 
   if (warp == 0) {
-    // ------------------------------ TMA producer ------------------------------
-    if (lane == 0) {
-      const int bs = args.block_size, pages = kTile / bs;
-      uint32_t it = 0, n = 0, unit = 0;              // key tiles, query tiles and V tiles so far
-      bool ok = true;
-      for (int item = first_item; item < args.n_items && ok; item += step, ++n) {
-        const Tile t = tile_of(item);
-        ok = mbar_wait(smem_u32(q_empty), (n & 1) ^ 1, abort_flag, args.status, kStatusWaitTimeoutProducer);
-        if (!ok) break;
-        const uint32_t qb = smem_u32(q_full);
-        mbar_expect_tx(qb, kQBytes);
-        for (int c = 0; c < QB; ++c) tma_load_3d(smem_u32(sQ) + c * kSubBytes, &tmQ, qb, c * 64, t.head, t.q0);
-        const int* table = args.block_tables + static_cast<size_t>(t.b) * args.max_blocks;
-        const int end = t.pos0 + t.rows, kcol = t.head / args.group * args.D;
-        auto load = [&](const CUtensorMap* tm, uint32_t dst, uint32_t bar, int j, int col, int subs) {
-          const int tok0 = j * kTile, first_page = table[tok0 / bs];
-          for (int i = 0; i < pages; ++i) {
-            const int pg = tok0 + i * bs < end ? table[tok0 / bs + i] : first_page;
-            for (int c = 0; c < subs; ++c) tma_load_2d(dst + c * kSubBytes + i * bs * 128, tm, bar, col + c * 64, pg * bs);
-          }
-        };
-        auto load_k = [&](int j) {
-          const int st = it & 1;
-          ok = mbar_wait(smem_u32(&k_empty[st]), ((it >> 1) & 1) ^ 1, abort_flag, args.status, kStatusWaitTimeoutProducer);
-          if (!ok) return;
-          mbar_expect_tx(smem_u32(&k_full[st]), kQBytes);
-          load(&tmK, smem_u32(sK) + st * kQBytes, smem_u32(&k_full[st]), j, kcol, QB);
-          ++it;
-        };
-        load_k(t.lo);
-        for (int j = t.lo; j < t.n_kv && ok; ++j) {
-          if (j + 1 < t.n_kv) load_k(j + 1);
-          for (int v = 0; v < t.nv && ok; ++v, ++unit) {
-            const int slot = unit % kSlots;
-            ok = mbar_wait(smem_u32(&v_empty[slot]), ((unit / kSlots) & 1) ^ 1, abort_flag, args.status, kStatusWaitTimeoutProducer);
-            if (!ok) break;
-            mbar_expect_tx(smem_u32(&v_full[slot]), kVBytes);
-            load(&tmV, smem_u32(sV) + slot * kVBytes, smem_u32(&v_full[slot]), j, (t.v0 + v) * args.DV, VB);
-          }
+    // ------------------------------ TMA producer (the whole warp) ------------------------------
+    uint32_t it = 0, n = 0, unit = 0;                // key tiles, query tiles and V tiles so far
+    bool ok = true;
+    // wait until a buffer is free; the lanes agree on the outcome
+    auto wait_free = [&](uint64_t* bar, uint32_t parity) {
+      ok = mbar_wait(smem_u32(bar), parity, abort_flag, args.status, kStatusWaitTimeoutProducer);
+      ok = __all_sync(0xffffffffu, ok);
+    };
+    for (int item = first_item; item < args.n_items && ok; item += step, ++n) {
+      const Tile t = tile_of(item);
+      wait_free(q_empty, (n & 1) ^ 1);
+      if (!ok) break;
+      if (lane == 0) mbar_expect_tx(smem_u32(q_full), kQBytes);
+      __syncwarp();
+      if (lane < QB) tma_load_3d(smem_u32(sQ) + lane * kSubBytes, &tmQ, smem_u32(q_full), lane * 64, t.head, t.q0);
+      const int* table = args.block_tables + static_cast<size_t>(t.b) * args.max_blocks;
+      const int end = t.pos0 + t.rows, kcol = t.head / args.group * args.D;
+      auto load = [&](const CUtensorMap* tm, uint8_t* dst, uint64_t* full, uint32_t bytes, int j, int col, int subs) {
+        if (lane == 0) mbar_expect_tx(smem_u32(full), bytes);
+        __syncwarp();
+        tma_load_pages(smem_u32(dst), kSubBytes, tm, smem_u32(full), table, args.block_size, j * kTile, end, col, subs);
+      };
+      auto load_k = [&](int j) {
+        const int st = it & 1;
+        wait_free(&k_empty[st], ((it >> 1) & 1) ^ 1);
+        if (!ok) return;
+        load(&tmK, sK + st * kQBytes, &k_full[st], kQBytes, j, kcol, QB);
+        ++it;
+      };
+      load_k(t.lo);
+      for (int j = t.lo; j < t.n_kv && ok; ++j) {
+        if (j + 1 < t.n_kv) load_k(j + 1);
+        for (int v = 0; v < t.nv && ok; ++v, ++unit) {
+          const int slot = unit % kSlots;
+          wait_free(&v_empty[slot], ((unit / kSlots) & 1) ^ 1);
+          if (ok) load(&tmV, sV + slot * kVBytes, &v_full[slot], kVBytes, j, (t.v0 + v) * args.DV, VB);
         }
       }
     }
-    __syncwarp();
   } else if (warp == 1) {
     // ------------------------------ MMA issuer ------------------------------
     if (lane == 0) {
@@ -626,7 +612,10 @@ paged_prefill_values_kernel(const __grid_constant__ CUtensorMap tmQ, const __gri
       for (int item = first_item; item < args.n_items && ok; item += step, ++n) {
         const Tile t = tile_of(item);
         for (int j = t.lo; j < t.n_kv && ok; ++j) {
-          if (j == t.lo) ok = mbar_wait(smem_u32(q_full), n & 1, abort_flag, args.status, kStatusWaitTimeoutMma);
+          if (j == t.lo) {
+            if (it > 0) issue_pv();                  // the last products of the query tile before do not wait for this one's q
+            if (ok) ok = mbar_wait(smem_u32(q_full), n & 1, abort_flag, args.status, kStatusWaitTimeoutMma);
+          }
           const int st = it & 1;
           if (ok) ok = mbar_wait(smem_u32(&k_full[st]), (it >> 1) & 1, abort_flag, args.status, kStatusWaitTimeoutMma);
           if (!ok) break;
@@ -642,7 +631,7 @@ paged_prefill_values_kernel(const __grid_constant__ CUtensorMap tmQ, const __gri
           umma_commit(smem_u32(&s_full[st]));
           umma_commit(smem_u32(&k_empty[st]));
           if (j == t.n_kv - 1) umma_commit(smem_u32(q_empty));
-          if (it > 0) issue_pv();
+          if (j > t.lo) issue_pv();
           first_key = j == t.lo;
           pending = t.nv;
           ++it;

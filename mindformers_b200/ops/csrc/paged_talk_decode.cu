@@ -123,35 +123,27 @@ paged_talk_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
   const uint32_t tmem_S = tmem_O + nv_max * Hp;             // two buffers of `items` blocks of 16 columns
 
   if (warp == 0) {
-    // ------------------------------------ producer ------------------------------------
-    if (lane == 0 && n_tiles > 0) {
-      const uint32_t qb = smem_u32(q_full);
-      mbar_expect_tx(qb, items * k_halves * (kItem * 128));
-      for (int i = 0; i < items; ++i) {
+    // ------------------------------------ producer (the whole warp) ------------------------------------
+    if (n_tiles > 0) {
+      if (lane == 0) mbar_expect_tx(smem_u32(q_full), items * k_halves * (kItem * 128));
+      __syncwarp();
+      for (int x = lane; x < items * k_halves; x += 32) {
+        const int i = x / k_halves, c = x % k_halves;
         const int head0 = (i / args.per_kv) * args.group + (i % args.per_kv) * kItem;
-        for (int c = 0; c < k_halves; ++c)
-          tma_load_2d(smem_u32(sQ) + i * kQItem + c * (kItem * 128), &tmQ, qb, c * 64, q_row * args.H + head0);
+        tma_load_2d(smem_u32(sQ) + i * kQItem + c * (kItem * 128), &tmQ, smem_u32(q_full), c * 64, q_row * args.H + head0);
       }
-      const int bs = args.block_size, pages = kTile / bs;
       const int* table = args.block_tables + static_cast<size_t>(b) * args.max_blocks;
       uint32_t unit = 0;
       bool ok = true;
       auto load_tile = [&](const CUtensorMap* tm, int j, int col0, int halves) {
         const int slot = unit % slots;
-        const uint32_t ph = (unit / slots) & 1;
-        ok = mbar_wait(smem_u32(&empty[slot]), ph ^ 1, abort_flag, args.status, kStatusWaitTimeoutProducer);
+        ok = mbar_wait(smem_u32(&empty[slot]), ((unit / slots) & 1) ^ 1, abort_flag, args.status, kStatusWaitTimeoutProducer);
+        ok = __all_sync(0xffffffffu, ok);
         if (!ok) return;
-        const int tok0 = (t0 + j) * kTile;
-        const int first_page = table[tok0 / bs];
-        const uint32_t fb = smem_u32(&full[slot]), dst = smem_u32(sRing + slot * kUnit);
-        mbar_expect_tx(fb, halves * kSub);
-        for (int i = 0; i < pages; ++i) {
-          // pages past the end of the sequence may be unallocated: read the tile's first page instead (masked)
-          int pg = tok0 + i * bs < len ? table[tok0 / bs + i] : first_page;
-          if (pg < 0) pg = first_page;
-          tma_load_2d(dst + i * bs * 128, tm, fb, col0, pg * bs);
-          if (halves > 1) tma_load_2d(dst + kSub + i * bs * 128, tm, fb, col0 + 64, pg * bs);
-        }
+        if (lane == 0) mbar_expect_tx(smem_u32(&full[slot]), halves * kSub);
+        __syncwarp();
+        tma_load_pages(smem_u32(sRing + slot * kUnit), kSub, tm, smem_u32(&full[slot]), table, args.block_size, (t0 + j) * kTile, len,
+                       col0, halves);
         ++unit;
       };
       for (int g = 0; g < args.G && ok; ++g) load_tile(&tmK, 0, g * args.D, k_halves);
@@ -160,7 +152,6 @@ paged_talk_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
         for (int v = 0; v < nv && ok; ++v) load_tile(&tmV, j, (v0 + v) * args.DV, v_halves);
       }
     }
-    __syncwarp();
   } else if (warp == 1) {
     // ------------------------------------ MMA issuer ------------------------------------
     if (lane == 0 && n_tiles > 0) {
