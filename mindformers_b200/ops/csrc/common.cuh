@@ -234,6 +234,40 @@ __device__ __forceinline__ void umma_f8f6f4_ss(uint32_t d_tmem, uint64_t a_desc,
       : "memory");
 }
 // Arrive on an mbarrier once every tcgen05.mma issued so far by this thread has completed.
+// The same for a whole, converged warp: every lane passes the same operands and one of them (`leader`) issues. Operands that are
+// uniform over the warp stay in uniform registers, so that an issue costs a few cycles; from a branch that one lane takes, each
+// operand has to be moved there first, which takes longer than a 128 x 128 x 16 product.
+__device__ __forceinline__ void umma_f16_ss_warp(bool leader, uint32_t d_tmem, uint64_t a_desc, uint64_t b_desc, uint32_t idesc,
+                                                 uint32_t accumulate) {
+  asm volatile(
+      "{\n\t"
+      ".reg .pred p, q;\n\t"
+      "setp.ne.u32 p, %4, 0;\n\t"
+      "setp.ne.u32 q, %5, 0;\n\t"
+      "@q tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n\t"
+      "}\n" ::"r"(d_tmem), "l"(a_desc), "l"(b_desc), "r"(idesc), "r"(accumulate), "r"((uint32_t)leader)
+      : "memory");
+}
+__device__ __forceinline__ void umma_f16_ts_warp(bool leader, uint32_t d_tmem, uint32_t a_tmem, uint64_t b_desc, uint32_t idesc,
+                                                 uint32_t accumulate) {
+  asm volatile(
+      "{\n\t"
+      ".reg .pred p, q;\n\t"
+      "setp.ne.u32 p, %4, 0;\n\t"
+      "setp.ne.u32 q, %5, 0;\n\t"
+      "@q tcgen05.mma.cta_group::1.kind::f16 [%0], [%1], %2, %3, p;\n\t"
+      "}\n" ::"r"(d_tmem), "r"(a_tmem), "l"(b_desc), "r"(idesc), "r"(accumulate), "r"((uint32_t)leader)
+      : "memory");
+}
+__device__ __forceinline__ void umma_commit_warp(bool leader, uint32_t bar) {
+  asm volatile(
+      "{\n\t"
+      ".reg .pred q;\n\t"
+      "setp.ne.u32 q, %1, 0;\n\t"
+      "@q tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];\n\t"
+      "}\n" ::"r"(bar), "r"((uint32_t)leader)
+      : "memory");
+}
 __device__ __forceinline__ void umma_commit(uint32_t bar) {
   asm volatile("tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];" ::"r"(bar)
                : "memory");

@@ -212,51 +212,54 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
       }
     }
   } else if (warp == 1) {
-    // ------------------------------ MMA issuer ------------------------------
-    if (lane == 0) {
-      constexpr uint32_t IDESC_QK = umma_idesc_bf16(kTile, kTile, 0, 0);  // A = Q K-major (smem), B = K K-major
-      constexpr uint32_t IDESC_PV = umma_idesc_bf16(kTile, HV, 0, 1);     // A = P (tensor memory), B = V MN-major
-      const uint32_t qa = smem_u32(sQ), ka = smem_u32(sK), va = smem_u32(sV);
-      uint32_t it = 0, n = 0;
-      bool ok = true, first_key = true;          // first_key: the pending P V product starts its query tile's sum
-      // O (+)= P V of key tile it - 1
-      auto issue_pv = [&]() {
-        const uint32_t ph = (it - 1) & 1;
-        ok = mbar_wait(smem_u32(v_full), ph, abort_flag, args.status, kStatusWaitTimeoutMma);
-        if (ok) ok = mbar_wait(smem_u32(p_ready), ph, abort_flag, args.status, kStatusWaitTimeoutMma);
-        if (!ok) return;
+    // ------------------------------ MMA issuer (the whole warp, one lane issues) ------------------------------
+    constexpr uint32_t IDESC_QK = umma_idesc_bf16(kTile, kTile, 0, 0);  // A = Q K-major (smem), B = K K-major
+    constexpr uint32_t IDESC_PV = umma_idesc_bf16(kTile, HV, 0, 1);     // A = P (tensor memory), B = V MN-major
+    const bool leader = elect_one();
+    const uint64_t q_desc = umma_desc_kmajor_sw128(smem_u32(sQ)), k_desc = umma_desc_kmajor_sw128(smem_u32(sK));
+    const uint64_t v_desc = umma_desc_mnmajor_sw128(smem_u32(sV), kSubBytes);
+    uint32_t it = 0, n = 0;
+    bool ok = true, first_key = true;                // first_key: the pending P V product starts its query tile's sum
+    auto wait = [&](uint64_t* bar, uint32_t parity) {
+      ok = mbar_wait(smem_u32(bar), parity, abort_flag, args.status, kStatusWaitTimeoutMma);
+      ok = __all_sync(0xffffffffu, ok);
+    };
+    // O (+)= P V of key tile it - 1
+    auto issue_pv = [&]() {
+      const uint32_t ph = (it - 1) & 1;
+      wait(v_full, ph);
+      if (ok) wait(p_ready, ph);
+      if (!ok) return;
+      tc_fence_after();
+#pragma unroll
+      for (int k = 0; k < kTile / 16; ++k)           // bf16 pairs: 8 columns of P per 16 keys
+        umma_f16_ts_warp(leader, tmem_O, tmem_S + k * 8, v_desc + ((k * 16 * 128) >> 4), IDESC_PV, (!first_key || k > 0) ? 1u : 0u);
+      umma_commit_warp(leader, smem_u32(pv_done));
+      umma_commit_warp(leader, smem_u32(v_empty));
+    };
+    for (int item = first_item; item < args.n_items && ok; item += step, ++n) {
+      const Tile t = tile_of(item);
+      for (int j = t.lo; j < t.n_kv; ++j) {
+        if (it > 0) issue_pv();
+        if (ok && j == t.lo) wait(q_full, n & 1);
+        // ---- S = Q K(j)^T: overwrites S / P, executes behind the P V product issued just above ----
+        if (ok) wait(k_full, it & 1);
+        if (!ok) break;
         tc_fence_after();
 #pragma unroll
-        for (int k = 0; k < kTile / 16; ++k)           // bf16 pairs: 8 columns of P per 16 keys
-          umma_f16_ts(tmem_O, tmem_S + k * 8, umma_desc_mnmajor_sw128(va + k * 16 * 128, kSubBytes), IDESC_PV,
-                      (!first_key || k > 0) ? 1u : 0u);
-        umma_commit(smem_u32(pv_done));
-        umma_commit(smem_u32(v_empty));
-      };
-      for (int item = first_item; item < args.n_items && ok; item += step, ++n) {
-        const Tile t = tile_of(item);
-        for (int j = t.lo; j < t.n_kv; ++j) {
-          if (it > 0) issue_pv();
-          if (ok && j == t.lo) ok = mbar_wait(smem_u32(q_full), n & 1, abort_flag, args.status, kStatusWaitTimeoutMma);
-          // ---- S = Q K(j)^T: overwrites S / P, executes behind the P V product issued just above ----
-          if (ok) ok = mbar_wait(smem_u32(k_full), it & 1, abort_flag, args.status, kStatusWaitTimeoutMma);
-          if (!ok) break;
-          tc_fence_after();
-#pragma unroll
-          for (int k = 0; k < HQ / 16; ++k) {
-            const uint32_t off = (k >> 2) * kSubBytes + (k & 3) * 32;
-            umma_f16_ss(tmem_S, umma_desc_kmajor_sw128(qa + off), umma_desc_kmajor_sw128(ka + off), IDESC_QK, k > 0 ? 1u : 0u);
-          }
-          umma_commit(smem_u32(s_full));
-          umma_commit(smem_u32(k_empty));
-          if (j == t.n_kv - 1) umma_commit(smem_u32(q_empty));
-          first_key = j == t.lo;
-          ++it;
+        for (int k = 0; k < HQ / 16; ++k) {
+          constexpr int kSubUnits = kSubBytes >> 4;
+          const int off = (k >> 2) * kSubUnits + (k & 3) * 2;
+          umma_f16_ss_warp(leader, tmem_S, q_desc + off, k_desc + off, IDESC_QK, k > 0 ? 1u : 0u);
         }
+        umma_commit_warp(leader, smem_u32(s_full));
+        umma_commit_warp(leader, smem_u32(k_empty));
+        if (j == t.n_kv - 1) umma_commit_warp(leader, smem_u32(q_empty));
+        first_key = j == t.lo;
+        ++it;
       }
-      if (ok && it > 0) issue_pv();
     }
-    __syncwarp();
+    if (ok && it > 0) issue_pv();
   } else {
     // ------------------------------ softmax warpgroup ------------------------------
     const int ew = warp & 3;                       // TMEM lane quarter of this warp
@@ -584,62 +587,66 @@ paged_prefill_values_kernel(const __grid_constant__ CUtensorMap tmQ, const __gri
       }
     }
   } else if (warp == 1) {
-    // ------------------------------ MMA issuer ------------------------------
-    if (lane == 0) {
-      constexpr uint32_t IDESC_QK = umma_idesc_bf16(kTile, kTile, 0, 0);
-      constexpr uint32_t IDESC_PV = umma_idesc_bf16(kTile, HV, 0, 1);
-      const uint32_t qa = smem_u32(sQ), va0 = smem_u32(sV);
-      uint32_t it = 0, n = 0, unit = 0;
-      bool ok = true, first_key = true;              // first_key: the pending products start their query tile's sums
-      int pending = 0;                               // value heads of the pending products
-      // O(v) (+)= P V(v) of key tile it - 1
-      auto issue_pv = [&]() {
-        ok = mbar_wait(smem_u32(p_ready), (it - 1) & 1, abort_flag, args.status, kStatusWaitTimeoutMma);
-        const uint32_t pa = tmem_base + ((it - 1) & 1) * kTile;
-        for (int v = 0; v < pending && ok; ++v, ++unit) {
-          const int slot = unit % kSlots;
-          ok = mbar_wait(smem_u32(&v_full[slot]), (unit / kSlots) & 1, abort_flag, args.status, kStatusWaitTimeoutMma);
-          if (!ok) return;
-          tc_fence_after();
+    // ------------------------------ MMA issuer (the whole warp, one lane issues) ------------------------------
+    constexpr uint32_t IDESC_QK = umma_idesc_bf16(kTile, kTile, 0, 0);
+    constexpr uint32_t IDESC_PV = umma_idesc_bf16(kTile, HV, 0, 1);
+    const bool leader = elect_one();
+    const uint64_t q_desc = umma_desc_kmajor_sw128(smem_u32(sQ));
+    uint32_t it = 0, n = 0, unit = 0;
+    bool ok = true, first_key = true;                // first_key: the pending products start their query tile's sums
+    int pending = 0;                                 // value heads of the pending products
+    auto wait = [&](uint64_t* bar, uint32_t parity) {
+      ok = mbar_wait(smem_u32(bar), parity, abort_flag, args.status, kStatusWaitTimeoutMma);
+      ok = __all_sync(0xffffffffu, ok);
+    };
+    // O(v) (+)= P V(v) of key tile it - 1
+    auto issue_pv = [&]() {
+      wait(p_ready, (it - 1) & 1);
+      const uint32_t pa = tmem_base + ((it - 1) & 1) * kTile;
+      for (int v = 0; v < pending && ok; ++v, ++unit) {
+        const int slot = unit % kSlots;
+        wait(&v_full[slot], (unit / kSlots) & 1);
+        if (!ok) return;
+        tc_fence_after();
+        const uint64_t v_desc = umma_desc_mnmajor_sw128(smem_u32(sV) + slot * kVBytes, kSubBytes);
+        const uint32_t o = tmem_O + v * HV;
 #pragma unroll
-          for (int k = 0; k < kTile / 16; ++k)
-            umma_f16_ts(tmem_O + v * HV, pa + k * 8, umma_desc_mnmajor_sw128(va0 + slot * kVBytes + k * 16 * 128, kSubBytes), IDESC_PV,
-                        (!first_key || k > 0) ? 1u : 0u);
-          umma_commit(smem_u32(&v_empty[slot]));
-        }
-        if (ok) umma_commit(smem_u32(&pv_done[(it - 1) & 1]));
-      };
-      for (int item = first_item; item < args.n_items && ok; item += step, ++n) {
-        const Tile t = tile_of(item);
-        for (int j = t.lo; j < t.n_kv && ok; ++j) {
-          if (j == t.lo) {
-            if (it > 0) issue_pv();                  // the last products of the query tile before do not wait for this one's q
-            if (ok) ok = mbar_wait(smem_u32(q_full), n & 1, abort_flag, args.status, kStatusWaitTimeoutMma);
-          }
-          const int st = it & 1;
-          if (ok) ok = mbar_wait(smem_u32(&k_full[st]), (it >> 1) & 1, abort_flag, args.status, kStatusWaitTimeoutMma);
-          if (!ok) break;
-          tc_fence_after();
-          // these scores overwrite those whose products with the values were issued before the last ones
-          const uint32_t ka = smem_u32(sK) + st * kQBytes;
-#pragma unroll
-          for (int k = 0; k < HQ / 16; ++k) {
-            const uint32_t off = (k >> 2) * kSubBytes + (k & 3) * 32;
-            umma_f16_ss(tmem_base + st * kTile, umma_desc_kmajor_sw128(qa + off), umma_desc_kmajor_sw128(ka + off), IDESC_QK,
-                        k > 0 ? 1u : 0u);
-          }
-          umma_commit(smem_u32(&s_full[st]));
-          umma_commit(smem_u32(&k_empty[st]));
-          if (j == t.n_kv - 1) umma_commit(smem_u32(q_empty));
-          if (j > t.lo) issue_pv();
-          first_key = j == t.lo;
-          pending = t.nv;
-          ++it;
-        }
+        for (int k = 0; k < kTile / 16; ++k)
+          umma_f16_ts_warp(leader, o, pa + k * 8, v_desc + ((k * 16 * 128) >> 4), IDESC_PV, (!first_key || k > 0) ? 1u : 0u);
+        umma_commit_warp(leader, smem_u32(&v_empty[slot]));
       }
-      if (ok && it > 0) issue_pv();
+      if (ok) umma_commit_warp(leader, smem_u32(&pv_done[(it - 1) & 1]));
+    };
+    for (int item = first_item; item < args.n_items && ok; item += step, ++n) {
+      const Tile t = tile_of(item);
+      for (int j = t.lo; j < t.n_kv && ok; ++j) {
+        if (j == t.lo) {
+          if (it > 0) issue_pv();                    // the last products of the query tile before do not wait for this one's q
+          if (ok) wait(q_full, n & 1);
+        }
+        const int st = it & 1;
+        if (ok) wait(&k_full[st], (it >> 1) & 1);
+        if (!ok) break;
+        tc_fence_after();
+        // these scores overwrite those whose products with the values were issued before the last ones
+        const uint64_t k_desc = umma_desc_kmajor_sw128(smem_u32(sK) + st * kQBytes);
+        const uint32_t s_tmem = tmem_base + st * kTile;
+#pragma unroll
+        for (int k = 0; k < HQ / 16; ++k) {
+          constexpr int kSubUnits = kSubBytes >> 4;
+          const int off = (k >> 2) * kSubUnits + (k & 3) * 2;
+          umma_f16_ss_warp(leader, s_tmem, q_desc + off, k_desc + off, IDESC_QK, k > 0 ? 1u : 0u);
+        }
+        umma_commit_warp(leader, smem_u32(&s_full[st]));
+        umma_commit_warp(leader, smem_u32(&k_empty[st]));
+        if (j == t.n_kv - 1) umma_commit_warp(leader, smem_u32(q_empty));
+        if (j > t.lo) issue_pv();
+        first_key = j == t.lo;
+        pending = t.nv;
+        ++it;
+      }
     }
-    __syncwarp();
+    if (ok && it > 0) issue_pv();
   } else {
     // ------------------------------ softmax warpgroups ------------------------------
     const int ew = warp & 3, half = (warp - 2) >> 2;
