@@ -399,7 +399,7 @@ class GavatarConfig(PretrainedConfig):
                    layernorm_epsilon=float(self.norm["eps"]), normalization="RMSNorm", layernorm_zero_centered_gamma=True,
                    norm_placement="both", token_shift=True, fp32_residual_connection=True, ragged_attention=True, rotary_dim=0,
                    position_embedding_type="sinusoidal", embedding_scale=float(self.embedding["scale"]),
-                   moe_router_score_function="softmax", norm_topk_prob=True, moe_router_logit_bias=True,
+                   moe_router_score_function="softmax", norm_topk_prob=True, moe_router_logit_bias=True, moe_router_dtype="params",
                    moe_router_topk_scaling_factor=1.0, tie_word_embeddings=False)
         d = {k: v for k, v in d.items() if ALIASES.get(k, (k,))[0] not in own}
         return dict(d, **own)

@@ -110,7 +110,7 @@ def _declare(lib):
     sig("mfb_dp_announce", [I, I, I, I, P, P])
     sig("mfb_dp_reduce_bucket", [I, I, I, I, L, L, P, P, P, P, P, I, P, P])
     sig("mfb_dp_adamw_allgather", [I, I, I, L, L, P, P, P, P, P, P, P, P, L, F, F, F, F, F, F, F, F, F, F, P, P])
-    sig("mfb_router_fwd", [P, P, P, P, P, P, I, I, I, I, I, I, I, F, P])
+    sig("mfb_router_fwd", [P, P, P, P, P, P, P, I, I, I, I, I, I, I, F, P])
     sig("mfb_router_bwd", [P, P, P, P, P, I, I, I, I, I, F, P])
     sig("mfb_moe_flag_words", [])
     sig("mfb_moe_rank", [P, I, I, P, P, P])

@@ -135,65 +135,59 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
       }
     }
   } else if (warp == 1) {
-    // ------------------------------------ MMA issuer ------------------------------------
-    if (lane == 0 && n_tiles > 0) {
+    // ------------------------------------ MMA issuer (the whole warp, one lane issues) ------------------------------------
+    if (n_tiles > 0) {
       constexpr uint32_t IDESC_S = umma_idesc_bf16(kTile, kHeads, 0, 0);   // A = cache K-major, B = Q K-major
       constexpr uint32_t IDESC_PV = umma_idesc_bf16(kTile, kHeads, 1, 0);  // A = cache MN-major, B = P^T K-major
-      bool ok = mbar_wait(smem_u32(q_full), 0, abort_flag, args.status, kStatusWaitTimeoutMma);
-      const uint32_t qa = smem_u32(sQ), pa = smem_u32(sP);
+      const bool leader = elect_one();
+      const uint64_t ring_k = umma_desc_kmajor_sw128(smem_u32(sRing)), ring_v = umma_desc_mnmajor_sw128(smem_u32(sRing), kSub);
+      const uint64_t q_desc = umma_desc_kmajor_sw128(smem_u32(sQ)), p_desc = umma_desc_kmajor_sw128(smem_u32(sP));
       uint32_t unit = 0;
+      bool ok = true;
+      auto wait = [&](uint64_t* bar, uint32_t parity) {
+        ok = mbar_wait(smem_u32(bar), parity, abort_flag, args.status, kStatusWaitTimeoutMma);
+        ok = __all_sync(0xffffffffu, ok);
+      };
+      wait(q_full, 0);
       for (int j = 0; j < n_tiles && ok; ++j) {
         const int sb = j & 1;
-        const uint32_t sph = (j >> 1) & 1;
-        ok = mbar_wait(smem_u32(&s_empty[sb]), sph ^ 1, abort_flag, args.status, kStatusWaitTimeoutMma);
-        if (!ok) break;
+        wait(&s_empty[sb], ((j >> 1) & 1) ^ 1);
         // ---- S^T = C . Q^T over the pairs of the first pass ----
         for (int u = 0; u < units && ok; ++u) {
           const int slot = unit % kSlots;
-          const uint32_t ph = (unit / kSlots) & 1;
-          ok = mbar_wait(smem_u32(&full[slot]), ph, abort_flag, args.status, kStatusWaitTimeoutMma);
+          wait(&full[slot], (unit / kSlots) & 1);
           if (!ok) break;
           tc_fence_after();
-          const uint32_t ca = smem_u32(sRing + slot * kUnit);
+          const uint64_t ca = ring_k + slot * (kUnit >> 4), qa = q_desc + 2 * u * (kQSub >> 4);
           const int ksteps = 2 * u + 1 < subs ? 8 : 4;
-          const int qsub0 = 2 * u;
 #pragma unroll
-          for (int k = 0; k < 8; ++k) {
-            if (k < ksteps) {
-              const uint64_t a_desc = umma_desc_kmajor_sw128(ca + (k >> 2) * kSub + (k & 3) * 32);
-              const uint64_t b_desc = umma_desc_kmajor_sw128(qa + (qsub0 + (k >> 2)) * kQSub + (k & 3) * 32);
-              umma_f16_ss(tmem_S + sb * 32, a_desc, b_desc, IDESC_S, (u > 0 || k > 0) ? 1u : 0u);
-            }
-          }
-          umma_commit(smem_u32(&empty[slot]));
+          for (int k = 0; k < 8; ++k)
+            if (k < ksteps)
+              umma_f16_ss_warp(leader, tmem_S + sb * 32, ca + (k >> 2) * (kSub >> 4) + (k & 3) * 2,
+                               qa + (k >> 2) * (kQSub >> 4) + (k & 3) * 2, IDESC_S, (u > 0 || k > 0) ? 1u : 0u);
+          umma_commit_warp(leader, smem_u32(&empty[slot]));
           ++unit;
         }
         if (!ok) break;
-        umma_commit(smem_u32(&s_full[sb]));
+        umma_commit_warp(leader, smem_u32(&s_full[sb]));
         // ---- O^T += C^T . P^T over the pairs of the second pass ----
-        ok = mbar_wait(smem_u32(p_ready), j & 1, abort_flag, args.status, kStatusWaitTimeoutMma);
-        if (!ok) break;
+        wait(p_ready, j & 1);
         for (int m = 0; m < units && ok; ++m) {
           const int slot = unit % kSlots;
-          const uint32_t ph = (unit / kSlots) & 1;
-          ok = mbar_wait(smem_u32(&full[slot]), ph, abort_flag, args.status, kStatusWaitTimeoutMma);
+          wait(&full[slot], (unit / kSlots) & 1);
           if (!ok) break;
           tc_fence_after();
-          const uint32_t ca = smem_u32(sRing + slot * kUnit);
+          const uint64_t ca = ring_v + slot * (kUnit >> 4);
 #pragma unroll
-          for (int k = 0; k < kTile / 16; ++k) {
-            const uint64_t a_desc = umma_desc_mnmajor_sw128(ca + k * 16 * 128, kSub);
-            const uint64_t b_desc = umma_desc_kmajor_sw128(pa + (k >> 2) * (kHeads * 128) + (k & 3) * 32);
-            umma_f16_ss(tmem_O + m * 32, a_desc, b_desc, IDESC_PV, (j > 0 || k > 0) ? 1u : 0u);
-          }
-          umma_commit(smem_u32(&empty[slot]));
+          for (int k = 0; k < kTile / 16; ++k)
+            umma_f16_ss_warp(leader, tmem_O + m * 32, ca + k * ((16 * 128) >> 4), p_desc + (k >> 2) * ((kHeads * 128) >> 4) + (k & 3) * 2,
+                             IDESC_PV, (j > 0 || k > 0) ? 1u : 0u);
+          umma_commit_warp(leader, smem_u32(&empty[slot]));
           ++unit;
         }
-        if (!ok) break;
-        umma_commit(smem_u32(pv_done));
+        if (ok) umma_commit_warp(leader, smem_u32(pv_done));
       }
     }
-    __syncwarp();
   } else {
     // ------------------------------------ softmax / epilogue ------------------------------------
     const int ew = warp & 3;

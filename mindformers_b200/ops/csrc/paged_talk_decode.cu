@@ -153,54 +153,66 @@ paged_talk_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
       }
     }
   } else if (warp == 1) {
-    // ------------------------------------ MMA issuer ------------------------------------
-    if (lane == 0 && n_tiles > 0) {
+    // ------------------------------------ MMA issuer (the whole warp, one lane issues) ------------------------------------
+    if (n_tiles > 0) {
       constexpr uint32_t IDESC_S = umma_idesc_bf16(kTile, kItem, 0, 0);     // A = K tile K-major, B = Q K-major
       const uint32_t idesc_pv = umma_idesc_bf16(kTile, Hp, 1, 0);           // A = V tile MN-major, B = P^T K-major
-      bool ok = mbar_wait(smem_u32(q_full), 0, abort_flag, args.status, kStatusWaitTimeoutMma);
-      const uint32_t qa = smem_u32(sQ);
+      const bool leader = elect_one();
+      const uint64_t ring_k = umma_desc_kmajor_sw128(smem_u32(sRing)), ring_v = umma_desc_mnmajor_sw128(smem_u32(sRing), kSub);
+      const uint64_t q_desc = umma_desc_kmajor_sw128(smem_u32(sQ)), p_desc = umma_desc_kmajor_sw128(smem_u32(sP));
+      const int k_steps = 4 * k_halves;
       uint32_t unit = 0;
-      auto next_unit = [&]() {                              // address of the next tile of the ring, once it is there
+      bool ok = true;
+      auto wait = [&](uint64_t* bar, uint32_t parity) {
+        ok = mbar_wait(smem_u32(bar), parity, abort_flag, args.status, kStatusWaitTimeoutMma);
+        ok = __all_sync(0xffffffffu, ok);
+      };
+      wait(q_full, 0);
+      auto next_unit = [&]() {                              // offset of the next tile of the ring in descriptor units, once it is there
         const int slot = unit % slots;
-        ok = mbar_wait(smem_u32(&full[slot]), (unit / slots) & 1, abort_flag, args.status, kStatusWaitTimeoutMma);
+        wait(&full[slot], (unit / slots) & 1);
         tc_fence_after();
-        return smem_u32(sRing + slot * kUnit);
+        return static_cast<uint64_t>(slot * (kUnit >> 4));
       };
       auto scores = [&](int j) {
         const int sb = j & 1;
-        ok = mbar_wait(smem_u32(&s_empty[sb]), ((j >> 1) & 1) ^ 1, abort_flag, args.status, kStatusWaitTimeoutMma);
+        wait(&s_empty[sb], ((j >> 1) & 1) ^ 1);
         for (int g = 0; g < args.G && ok; ++g) {
-          const uint32_t ka = next_unit();
+          const uint64_t ka = ring_k + next_unit();
           if (!ok) return;
           for (int p = 0; p < args.per_kv; ++p) {
             const int i = g * args.per_kv + p;
-            for (int k = 0; k < 4 * k_halves; ++k)
-              umma_f16_ss(tmem_S + (sb * items + i) * kItem, umma_desc_kmajor_sw128(ka + (k >> 2) * kSub + (k & 3) * 32),
-                          umma_desc_kmajor_sw128(qa + i * kQItem + (k >> 2) * (kItem * 128) + (k & 3) * 32), IDESC_S, k > 0 ? 1u : 0u);
-            umma_commit(smem_u32(&s_full[sb * items + i]));
+            const uint64_t qa = q_desc + i * (kQItem >> 4);
+            const uint32_t s_tmem = tmem_S + (sb * items + i) * kItem;
+#pragma unroll
+            for (int k = 0; k < 8; ++k)
+              if (k < k_steps)
+                umma_f16_ss_warp(leader, s_tmem, ka + (k >> 2) * (kSub >> 4) + (k & 3) * 2,
+                                 qa + (k >> 2) * ((kItem * 128) >> 4) + (k & 3) * 2, IDESC_S, k > 0 ? 1u : 0u);
+            umma_commit_warp(leader, smem_u32(&s_full[sb * items + i]));
           }
-          umma_commit(smem_u32(&empty[unit % slots]));
+          umma_commit_warp(leader, smem_u32(&empty[unit % slots]));
           ++unit;
         }
       };
       if (ok) scores(0);
       for (int j = 0; j < n_tiles && ok; ++j) {
         if (j + 1 < n_tiles) scores(j + 1);
-        if (ok) ok = mbar_wait(smem_u32(p_ready), j & 1, abort_flag, args.status, kStatusWaitTimeoutMma);
-        const uint32_t pa = smem_u32(sP) + (j & 1) * p_buf;
+        if (ok) wait(p_ready, j & 1);
+        const uint64_t pa = p_desc + (j & 1) * (p_buf >> 4);
         for (int v = 0; v < nv && ok; ++v) {
-          const uint32_t va = next_unit();
+          const uint64_t va = ring_v + next_unit();
           if (!ok) break;
+#pragma unroll
           for (int k = 0; k < kTile / 16; ++k)
-            umma_f16_ss(tmem_O + v * Hp, umma_desc_mnmajor_sw128(va + k * 16 * 128, kSub),
-                        umma_desc_kmajor_sw128(pa + (k >> 2) * p_sub + (k & 3) * 32), idesc_pv, (j > 0 || k > 0) ? 1u : 0u);
-          umma_commit(smem_u32(&empty[unit % slots]));
+            umma_f16_ss_warp(leader, tmem_O + v * Hp, va + k * ((16 * 128) >> 4), pa + (k >> 2) * (p_sub >> 4) + (k & 3) * 2, idesc_pv,
+                             (j > 0 || k > 0) ? 1u : 0u);
+          umma_commit_warp(leader, smem_u32(&empty[unit % slots]));
           ++unit;
         }
-        if (ok) umma_commit(smem_u32(pv_done));
+        if (ok) umma_commit_warp(leader, smem_u32(pv_done));
       }
     }
-    __syncwarp();
   } else {
     // ------------------------------------ softmax / epilogue ------------------------------------
     const int ew = warp & 3;

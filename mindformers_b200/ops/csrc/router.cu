@@ -1,6 +1,7 @@
 // Top-k MoE router (sm_100a): score function, optional expert bias, group-limited selection, top-k,
 // renormalisation, scaling and per-expert token counts in one pass; one warp per token.
 //
+//   logits (+ a bias of their own, forward only)
 //   scores = softmax(logits) | sigmoid(logits)                                   [T, E] fp32
 //   sel    = scores (+ bias); with G groups only the best `group_topk` groups stay eligible, a group being
 //            ranked by its best score (no bias) or by the sum of its two best biased scores (bias given)
@@ -33,13 +34,13 @@ __device__ __forceinline__ void warp_argmax(float& v, int& i) {
 }
 
 template <int PER>
-__device__ __forceinline__ void router_scores(const float* __restrict__ row, int E, int lane, bool sigmoid,
-                                              float (&s)[PER]) {
+__device__ __forceinline__ void router_scores(const float* __restrict__ row, const float* __restrict__ logit_bias, int E, int lane,
+                                              bool sigmoid, float (&s)[PER]) {
   float mx = -INFINITY;
 #pragma unroll
   for (int j = 0; j < PER; ++j) {
     const int e = lane + 32 * j;
-    s[j] = e < E ? row[e] : -INFINITY;
+    s[j] = e < E ? (logit_bias ? row[e] + logit_bias[e] : row[e]) : -INFINITY;
     mx = fmaxf(mx, s[j]);
   }
   if (sigmoid) {
@@ -62,14 +63,14 @@ __device__ __forceinline__ void router_scores(const float* __restrict__ row, int
 
 template <int PER>
 __global__ void __launch_bounds__(kRouterWarps * 32)
-router_fwd_kernel(const float* __restrict__ logits, const float* __restrict__ bias, float* __restrict__ probs,
+router_fwd_kernel(const float* __restrict__ logits, const float* __restrict__ logit_bias, const float* __restrict__ bias, float* __restrict__ probs,
                   long long* __restrict__ ids, float* __restrict__ scores_out, float* __restrict__ counts,
                   RouterArgs a) {
   const int lane = threadIdx.x & 31;
   const int t = blockIdx.x * kRouterWarps + (threadIdx.x >> 5);
   if (t >= a.T) return;
   float s[PER], sel[PER];
-  router_scores<PER>(logits + (long long)t * a.E, a.E, lane, a.sigmoid != 0, s);
+  router_scores<PER>(logits + (long long)t * a.E, logit_bias, a.E, lane, a.sigmoid != 0, s);
 #pragma unroll
   for (int j = 0; j < PER; ++j) {
     const int e = lane + 32 * j;
@@ -151,7 +152,7 @@ router_bwd_kernel(const float* __restrict__ logits, const long long* __restrict_
   const int t = blockIdx.x * kRouterWarps + (threadIdx.x >> 5);
   if (t >= a.T) return;
   float s[PER], ds[PER];
-  router_scores<PER>(logits + (long long)t * a.E, a.E, lane, a.sigmoid != 0, s);
+  router_scores<PER>(logits + (long long)t * a.E, nullptr, a.E, lane, a.sigmoid != 0, s);
 #pragma unroll
   for (int j = 0; j < PER; ++j) {
     const int e = lane + 32 * j;
@@ -229,15 +230,15 @@ static int router_check(int T, int E, int k, int groups, int group_topk) {
     else KERNEL<16><<<grid, kRouterWarps * 32, 0, stream>>>(__VA_ARGS__);              \
   } while (0)
 
-// logits [T, E] fp32 (contiguous); bias [E] or null; probs [T, k] fp32; ids [T, k] int64;
+// logits [T, E] fp32 (contiguous); logit_bias [E] or null: added to the logits; bias [E] or null; probs [T, k] fp32; ids [T, k] int64;
 // scores_out [T, E] fp32 or null; counts [E] fp32 or null (incremented, not cleared).
-int mfb_router_fwd(const float* logits, const float* bias, float* probs, long long* ids, float* scores_out,
+int mfb_router_fwd(const float* logits, const float* logit_bias, const float* bias, float* probs, long long* ids, float* scores_out,
                    float* counts, int T, int E, int k, int sigmoid, int norm, int groups, int group_topk,
                    float scale, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (router_check(T, E, k, groups, group_topk)) return 1;
   RouterArgs a{T, E, k, sigmoid, norm, groups, group_topk, scale};
-  MFB_ROUTER_DISPATCH(router_fwd_kernel, logits, bias, probs, ids, scores_out, counts, a);
+  MFB_ROUTER_DISPATCH(router_fwd_kernel, logits, logit_bias, bias, probs, ids, scores_out, counts, a);
   return cudaGetLastError() == cudaSuccess ? 0 : 2;
 }
 

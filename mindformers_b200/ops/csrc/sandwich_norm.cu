@@ -236,7 +236,10 @@ void launch(const Args& a, cudaStream_t stream) {
 template <typename T, int VEC>
 int pick(const Args& a, cudaStream_t stream) {
   const int nvec = a.W / VEC;
-  if (nvec <= 256) launch<T, VEC, 1, 256>(a, stream);
+  // with the shift a CTA's rows follow one another: more threads for fewer columns each
+  if (a.mu && nvec > 256 && nvec <= 512) launch<T, VEC, 1, 512>(a, stream);
+  else if (a.mu && nvec > 512 && nvec <= 1024) launch<T, VEC, 2, 512>(a, stream);
+  else if (nvec <= 256) launch<T, VEC, 1, 256>(a, stream);
   else if (nvec <= 512) launch<T, VEC, 2, 256>(a, stream);
   else if (nvec <= 1024) launch<T, VEC, 4, 256>(a, stream);
   else if (nvec <= 2048) launch<T, VEC, 4, 512>(a, stream);

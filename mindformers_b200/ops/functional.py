@@ -958,13 +958,13 @@ def router_topk_reference(logits, bias, k, sigmoid, norm, scale, groups=0, group
 
 class _RouterFn(torch.autograd.Function):
     @staticmethod
-    def forward(ctx, logits, bias, k, sigmoid, norm, scale, groups, group_topk, need_scores, counts):
+    def forward(ctx, logits, bias, k, sigmoid, norm, scale, groups, group_topk, need_scores, counts, logit_bias=None):
         T, E = logits.shape
         logits = logits.contiguous()
         probs = torch.empty(T, k, dtype=torch.float32, device=logits.device)
         ids = torch.empty(T, k, dtype=torch.int64, device=logits.device)
         scores = torch.empty(T, E, dtype=torch.float32, device=logits.device) if need_scores else None
-        rc = _lib.get_lib().mfb_router_fwd(logits.data_ptr(), _lib.ptr(bias), probs.data_ptr(), ids.data_ptr(),
+        rc = _lib.get_lib().mfb_router_fwd(logits.data_ptr(), _lib.ptr(logit_bias), _lib.ptr(bias), probs.data_ptr(), ids.data_ptr(),
                                            _lib.ptr(scores), _lib.ptr(counts), T, E, k, int(sigmoid), int(norm),
                                            int(groups or 0), int(group_topk or 0), float(scale), _lib.stream_ptr())
         _lib.check(rc, "mfb_router_fwd")
@@ -991,17 +991,22 @@ class _RouterFn(torch.autograd.Function):
                                            float(scale), _lib.stream_ptr())
         _lib.check(rc, "mfb_router_bwd")
         _lib.count_launch()
-        return (dlogits,) + (None,) * 9
+        return (dlogits,) + (None,) * 10
 
 
 def router_topk(logits: torch.Tensor, bias: Optional[torch.Tensor], k: int, *, sigmoid: bool = False, norm: bool = True,
                 scale: float = 1.0, groups: int = 0, group_topk: int = 0, need_scores: bool = False,
-                counts: Optional[torch.Tensor] = None):
+                counts: Optional[torch.Tensor] = None, logit_bias: Optional[torch.Tensor] = None):
     """Fused router: ``(probs [T,k] fp32, ids [T,k] int64, scores [T,E] | None)``; ``counts [E]`` (fp32) is
-    incremented by the number of copies routed to each expert."""
+    incremented by the number of copies routed to each expert. ``logit_bias [E]`` (fp32) is added to the logits, ``bias`` to
+    the scores by which experts are chosen."""
     E = logits.shape[-1]
-    if _on_gpu(logits) and logits.dtype == torch.float32 and E <= 512 and k <= 32 and (not groups or groups <= 32):
-        probs, ids, scores = apply_fn(_RouterFn, logits, bias, k, sigmoid, norm, scale, groups, group_topk, need_scores, counts)
+    fused = _on_gpu(logits) and logits.dtype == torch.float32 and E <= 512 and k <= 32 and (not groups or groups <= 32)
+    if logit_bias is not None and (not fused or torch.is_grad_enabled()):
+        logits, logit_bias = logits.float() + logit_bias, None
+    if fused:
+        probs, ids, scores = apply_fn(_RouterFn, logits, bias, k, sigmoid, norm, scale, groups, group_topk, need_scores, counts,
+                                      logit_bias)
         return probs, ids, (scores if need_scores else None)
     probs, ids, scores = router_topk_reference(logits.float(), bias, k, sigmoid, norm, scale, groups, group_topk)
     if counts is not None:

@@ -328,7 +328,7 @@ def qkv_rope_cache(qkv: torch.Tensor, bias: Optional[torch.Tensor], q_norm: Opti
     q = torch.empty((T, heads, dim), dtype=dtype, device=qkv.device)
     rc = _lib.get_lib().mfb_qkv_rope_cache(
         qkv.data_ptr(), qkv.stride(0), _lib.ptr(bias), _lib.ptr(q_norm), _lib.ptr(k_norm), float(eps), freqs.data_ptr(),
-        float(amplitude), rot, int(interleaved), positions.data_ptr(), slots.data_ptr(), q.data_ptr(), key_cache.data_ptr(),
+        float(amplitude), rot, int(interleaved or not rot), positions.data_ptr(), slots.data_ptr(), q.data_ptr(), key_cache.data_ptr(),
         value_cache.data_ptr(), T, heads, kv_heads, dim, v_dim, int(unit_qk) + 2 * int(unit_v), int(dtype == torch.float32),
         _lib.stream_ptr())
     _lib.check(rc, "mfb_qkv_rope_cache")

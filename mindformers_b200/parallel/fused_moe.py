@@ -28,13 +28,16 @@ BLOCK = 128
 
 
 class _Plan:
-    """What ``GroupedMLP`` needs from a permutation plan (all device tensors)."""
+    """What ``GroupedMLP`` needs from a permutation plan (all device tensors, parts of one zero-filled buffer)."""
 
-    def __init__(self, E_local, rows_cap, dev):
-        self.group_offsets = torch.zeros(E_local + 1, dtype=torch.int32, device=dev)
-        self.seg_fill = torch.zeros(E_local, dtype=torch.int32, device=dev)
-        self.block_group = torch.zeros(rows_cap // BLOCK, dtype=torch.int32, device=dev)
-        self.num_blocks = torch.zeros(1, dtype=torch.int32, device=dev)
+    def __init__(self, E_local, rows_cap, dev, extra: int = 0):
+        sizes = (E_local + 1, E_local, rows_cap // BLOCK, 1, extra)
+        starts = [0]
+        for n in sizes:
+            starts.append(starts[-1] + -(-n // 4) * 4)             # parts start on 16 bytes
+        buf = torch.zeros(starts[-1], dtype=torch.int32, device=dev)
+        self.group_offsets, self.seg_fill, self.block_group, self.num_blocks, self.extra = (
+            buf[a:a + n] for a, n in zip(starts, sizes))
         self.rows = rows_cap
 
 
@@ -247,9 +250,9 @@ class _PlanState:
         self.rank_in_e = torch.empty(n, dtype=torch.int32, device=dev)
         self.counts = torch.empty(ex.E, dtype=torch.int32, device=dev)
         self.write_base = torch.empty(ex.E, dtype=torch.int32, device=dev)
-        self.owner_cap = torch.zeros(8, dtype=torch.int32, device=dev)
         self.dest_row = torch.empty(n, dtype=torch.int32, device=dev)
-        self.plan = _Plan(ex.E_local, rows, dev)
+        self.plan = _Plan(ex.E_local, rows, dev, extra=8)
+        self.owner_cap = self.plan.extra
 
 
 class _Dispatch(torch.autograd.Function):

@@ -21,6 +21,7 @@ import torch.nn as nn
 import torch.nn.functional as F
 
 from ...ops import functional as Fn
+from ...ops import stream
 from .. import mappings as M
 from .. import parallel_state as ps
 from .mlp import MLP
@@ -46,7 +47,7 @@ class TopKRouter(nn.Module):
         self.weight = nn.Parameter(w.to(config.moe_router_dtype))
         self.weight.sequence_parallel = bool(config.sequence_parallel)
         self.weight.no_weight_decay = False
-        self.register_parameter("bias", nn.Parameter(torch.zeros(E, dtype=config.moe_router_dtype, device=dev))
+        self.register_parameter("bias", nn.Parameter(torch.zeros(E, dtype=torch.float32, device=dev))
                                 if config.moe_router_logit_bias else None)
         self.topk = config.moe_router_topk
         self.score_fn = config.moe_router_score_function
@@ -58,7 +59,10 @@ class TopKRouter(nn.Module):
             self.expert_load = None
 
     def gating(self, x):
-        return F.linear(x.to(self.weight.dtype), self.weight, self.bias).float()
+        """Logits without their bias, fp32."""
+        if self.weight.dtype == torch.bfloat16 and x.dtype == torch.bfloat16 and x.is_cuda and not torch.is_grad_enabled():
+            return stream.linear(x, self.weight, out_dtype=torch.float32)
+        return F.linear(x.to(self.weight.dtype), self.weight).float()
 
     def _select(self, scores):
         cfg = self.config
@@ -76,8 +80,9 @@ class TopKRouter(nn.Module):
 
     def forward(self, x: torch.Tensor):
         cfg = self.config
-        logits = self.gating(x)
+        logits, logit_bias = self.gating(x), self.bias
         if cfg.moe_z_loss_coeff:
+            logits, logit_bias = logits if logit_bias is None else logits + logit_bias, None
             z = torch.logsumexp(logits, dim=-1).pow(2).mean() * cfg.moe_z_loss_coeff
         else:
             z = None
@@ -91,7 +96,7 @@ class TopKRouter(nn.Module):
         probs, ids, scores = Fn.router_topk(
             logits, self.expert_bias, self.topk, sigmoid=sig, norm=norm, scale=float(cfg.moe_router_topk_scaling_factor),
             groups=int(cfg.moe_router_num_groups or 0), group_topk=int(cfg.moe_router_group_topk or 0),
-            need_scores=want_aux, counts=counts)
+            need_scores=want_aux, counts=counts, logit_bias=logit_bias)
         aux = None
         if want_aux:
             T = x.shape[0]

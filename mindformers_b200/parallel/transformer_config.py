@@ -231,7 +231,8 @@ class TransformerConfig(ModelParallelConfig):
     moe_router_pre_softmax: bool = False
     moe_router_topk_scaling_factor: Optional[float] = None
     moe_router_score_function: str = "softmax"
-    moe_router_dtype: Union[str, torch.dtype] = "float32"
+    moe_router_dtype: Union[str, torch.dtype] = "float32"   # of the router's weight ("params": params_dtype); 16-bit products
+                                            # are accumulated in, and the logits are, 32-bit
     moe_router_enable_expert_bias: bool = False
     moe_router_logit_bias: bool = False     # learned bias of the router's logits (selection and weights)
     moe_router_bias_update_rate: float = 1e-3
@@ -285,6 +286,8 @@ class TransformerConfig(ModelParallelConfig):
 
     def __post_init__(self):
         self._check_parallel()
+        if self.moe_router_dtype == "params":
+            self.moe_router_dtype = torch.bfloat16 if self.bf16 else self.params_dtype
         for name in ("compute_dtype", "layernorm_compute_dtype", "rotary_dtype", "softmax_compute_dtype",
                      "moe_router_dtype", "params_dtype"):
             setattr(self, name, to_torch_dtype(getattr(self, name)))
