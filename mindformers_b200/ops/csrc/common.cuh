@@ -136,17 +136,36 @@ __device__ __forceinline__ void tma_load_3d(uint32_t smem_dst, const CUtensorMap
       : "memory");
 }
 // 128 consecutive tokens of a paged cache as `subs` swizzled sub-tiles of 64 columns (from column `col` on), `sub_bytes` apart in
-// shared memory: one box per page and sub-tile, issued by one lane each, so that neither the block-table lookups nor the issue of
-// the boxes queue up. To be called by a whole warp; the tile has at most 16 boxes. Pages at or past `end` may be unallocated:
-// the tile's first page stands in for them (the caller masks its tokens).
-__device__ __forceinline__ void tma_load_pages(uint32_t smem_dst, uint32_t sub_bytes, const CUtensorMap* m, uint32_t bar,
-                                               const int* table, int block_size, int tok0, int end, int col, int subs) {
-  const int lane = static_cast<int>(lane_id()), pages = 128 / block_size;
-  if (lane < pages * subs) {
-    const int i = lane % pages, c = lane / pages;
-    int pg = table[tok0 / block_size + (tok0 + i * block_size < end ? i : 0)];
-    if (pg < 0) pg = table[tok0 / block_size];
-    tma_load_2d(smem_dst + c * sub_bytes + i * block_size * 128, m, bar, col + c * 64, pg * block_size);
+// shared memory: one box per page and sub-tile. To be called by a whole, converged warp, of which one lane (`leader`) issues: the
+// operands are uniform over the warp, so they need not be moved to uniform registers one by one, which takes longer than the
+// copy itself. `page` is what tile_page() gave this lane, early enough to hide the lookup.
+__device__ __forceinline__ void tma_load_2d_warp(bool leader, uint32_t smem_dst, const CUtensorMap* m, uint32_t bar, int32_t x,
+                                                 int32_t y) {
+  asm volatile(
+      "{\n\t"
+      ".reg .pred q;\n\t"
+      "setp.ne.u32 q, %5, 0;\n\t"
+      "@q cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4}], [%2];\n\t"
+      "}\n" ::"r"(smem_dst), "l"(reinterpret_cast<uint64_t>(m)), "r"(bar), "r"(x), "r"(y), "r"((uint32_t)leader)
+      : "memory");
+}
+// The page of this lane's part (lane modulo pages per tile) of the 128 tokens from tok0 on. Pages at or past `end` may be
+// unallocated: the tile's first page stands in for them (the caller masks its tokens).
+__device__ __forceinline__ int tile_page(const int* table, int block_size, int tok0, int end) {
+  const int i = static_cast<int>(lane_id()) % (128 / block_size);
+  const int first = table[tok0 / block_size];
+  const int pg = tok0 + i * block_size < end ? table[tok0 / block_size + i] : first;
+  return pg < 0 ? first : pg;
+}
+__device__ __forceinline__ void tma_load_pages(bool leader, uint32_t smem_dst, uint32_t sub_bytes, const CUtensorMap* m, uint32_t bar,
+                                               int page, int block_size, int col, int subs) {
+  const int pages = 128 / block_size;
+  const int lane = static_cast<int>(lane_id());
+  for (int i = 0; i < pages; ++i) {
+    // a warp reduction leaves its result in a uniform register
+    const int row = __reduce_add_sync(0xffffffffu, lane == i ? page : 0) * block_size;
+    for (int c = 0; c < subs; ++c)
+      tma_load_2d_warp(leader, smem_dst + c * sub_bytes + i * block_size * 128, m, bar, col + c * 64, row);
   }
 }
 __device__ __forceinline__ void tma_store_2d(const CUtensorMap* m, uint32_t smem_src, int32_t x,

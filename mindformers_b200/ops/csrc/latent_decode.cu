@@ -109,15 +109,21 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
   const uint32_t tmem_S = tmem_base + 128;        // 2 buffers of 16 columns, 32 apart
 
   if (warp == 0) {
-    // ------------------------------------ producer (the whole warp) ------------------------------------
+    // ------------------------------------ producer (the whole warp, one lane issues) ------------------------------------
     if (n_tiles > 0) {
-      if (lane == 0) mbar_expect_tx(smem_u32(q_full), subs * kQSub);
+      const bool leader = elect_one();
+      if (leader) {
+        mbar_expect_tx(smem_u32(q_full), subs * kQSub);
+        for (int c = 0; c < subs; ++c) tma_load_2d(smem_u32(sQ) + c * kQSub, &tmQ, smem_u32(q_full), c * 64, b * args.num_heads + head0);
+      }
       __syncwarp();
-      if (lane < subs) tma_load_2d(smem_u32(sQ) + lane * kQSub, &tmQ, smem_u32(q_full), lane * 64, b * args.num_heads + head0);
+      const int bs = args.block_size;
       const int* table = args.block_tables + static_cast<size_t>(b) * args.max_blocks;
       uint32_t unit = 0;
       bool ok = true;
+      int page = tile_page(table, bs, t0 * kTile, len);
       for (int j = 0; j < n_tiles && ok; ++j) {
+        const int next = j + 1 < n_tiles ? tile_page(table, bs, (t0 + j + 1) * kTile, len) : 0;
         // two passes over the tile's pairs: for S^T, then again for O^T
         for (int u = 0; u < 2 * units && ok; ++u) {
           const int slot = unit % kSlots;
@@ -126,12 +132,12 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
           if (!ok) break;
           const int pair = u < units ? u : u - units;
           const int two = 2 * pair + 1 < subs ? 2 : 1;
-          if (lane == 0) mbar_expect_tx(smem_u32(&full[slot]), two * kSub);
+          if (leader) mbar_expect_tx(smem_u32(&full[slot]), two * kSub);
           __syncwarp();
-          tma_load_pages(smem_u32(sRing + slot * kUnit), kSub, &tmC, smem_u32(&full[slot]), table, args.block_size, (t0 + j) * kTile,
-                         len, pair * 128, two);
+          tma_load_pages(leader, smem_u32(sRing + slot * kUnit), kSub, &tmC, smem_u32(&full[slot]), page, bs, pair * 128, two);
           ++unit;
         }
+        page = next;
       }
     }
   } else if (warp == 1) {
@@ -214,25 +220,29 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
       const bool valid = tok < len && tok >= first_tok;
 #pragma unroll
       for (int h = 0; h < kHeads; ++h) s[h] = valid ? __uint_as_float(sr[h]) * args.scale_log2 : -INFINITY;
-      // per-head maximum over the 128 tokens of the tile
+      // the heads' maxima change seldom: first only see whether some score is more than 2^8 above its head's
+      bool fine = true;
 #pragma unroll
-      for (int h = 0; h < kHeads; ++h) {
-        const float w = warp_max(s[h]);
-        if (lane == 0) red[ew * kHeads + h] = w;
-      }
-      named_bar_sync(1, 128);
+      for (int h = 0; h < kHeads; ++h) fine = fine && !(s[h] > m_used[h] + kRescale);
+      const bool any_rescale = !named_bar_and(3, 128, fine);
       float alpha[kHeads];
-      bool any_rescale = false;
 #pragma unroll
-      for (int h = 0; h < kHeads; ++h) {
-        const float mx = fmaxf(fmaxf(red[h], red[kHeads + h]), fmaxf(red[2 * kHeads + h], red[3 * kHeads + h]));
-        alpha[h] = 1.f;
-        if (m_used[h] == -INFINITY) {
-          m_used[h] = mx;                           // first tile with a valid token (nothing accumulated yet)
-        } else if (mx > m_used[h] + kRescale) {
-          alpha[h] = ex2(m_used[h] - mx);
-          m_used[h] = mx;
-          any_rescale = true;
+      for (int h = 0; h < kHeads; ++h) alpha[h] = 1.f;
+      if (any_rescale) {
+        // per-head maximum over the 128 tokens of the tile
+#pragma unroll
+        for (int h = 0; h < kHeads; ++h) {
+          const float w = warp_max(s[h]);
+          if (lane == 0) red[ew * kHeads + h] = w;
+        }
+        named_bar_sync(1, 128);
+#pragma unroll
+        for (int h = 0; h < kHeads; ++h) {
+          const float mx = fmaxf(fmaxf(red[h], red[kHeads + h]), fmaxf(red[2 * kHeads + h], red[3 * kHeads + h]));
+          if (mx > m_used[h] + kRescale) {              // or nothing was accumulated yet
+            alpha[h] = m_used[h] == -INFINITY ? 0.f : ex2(m_used[h] - mx);
+            m_used[h] = mx;
+          }
         }
       }
 #pragma unroll

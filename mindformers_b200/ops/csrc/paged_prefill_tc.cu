@@ -179,36 +179,39 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
   const uint32_t tmem_base = *tmem_holder;
   const uint32_t tmem_S = tmem_base, tmem_O = tmem_base + kTile;   // P lives in the first 64 columns of S
   if (warp == 0) {
-    // ------------------------------ TMA producer (the whole warp) ------------------------------
+    // ------------------------------ TMA producer (the whole warp, one lane issues) ------------------------------
+    const bool leader = elect_one();
+    const int bs = args.block_size;
     uint32_t it = 0, n = 0;                          // key tiles and query tiles so far
     bool ok = true;
-    // wait until a buffer is free; the lanes agree on the outcome
-    auto wait_free = [&](uint64_t* bar, uint32_t parity) {
-      ok = mbar_wait(smem_u32(bar), parity, abort_flag, args.status, kStatusWaitTimeoutProducer);
+    // wait until a buffer is free (the lanes agree on the outcome) and announce what goes there
+    auto claim = [&](uint64_t* empty, uint32_t parity, uint64_t* full, uint32_t bytes) {
+      ok = mbar_wait(smem_u32(empty), parity, abort_flag, args.status, kStatusWaitTimeoutProducer);
       ok = __all_sync(0xffffffffu, ok);
+      if (ok && leader) mbar_expect_tx(smem_u32(full), bytes);
+      __syncwarp();
     };
     for (int item = first_item; item < args.n_items && ok; item += step, ++n) {
       const Tile t = tile_of(item);
-      wait_free(q_empty, (n & 1) ^ 1);
-      if (!ok) break;
-      if (lane == 0) mbar_expect_tx(smem_u32(q_full), kQBytes);
-      __syncwarp();
-      if (lane < QB) tma_load_3d(smem_u32(sQ) + lane * kSubBytes, &tmQ, smem_u32(q_full), lane * 64, t.head, t.q0);
       const int* table = args.block_tables + static_cast<size_t>(t.b) * args.max_blocks;
       const int kv_head = t.head / args.group, end = t.pos0 + t.rows;
       const int kcol = kv_head * args.D, vcol = (args.vheads > 1 ? t.vsel : kv_head) * args.DV;
+      int page = tile_page(table, bs, t.lo * kTile, end);
+      claim(q_empty, (n & 1) ^ 1, q_full, kQBytes);
+      if (!ok) break;
+      if (leader)
+        for (int c = 0; c < QB; ++c) tma_load_3d(smem_u32(sQ) + c * kSubBytes, &tmQ, smem_u32(q_full), c * 64, t.head, t.q0);
+      __syncwarp();
       for (int j = t.lo; j < t.n_kv; ++j, ++it) {
         const uint32_t ph = it & 1;
-        wait_free(k_empty, ph ^ 1);
+        claim(k_empty, ph ^ 1, k_full, kQBytes);
         if (!ok) break;
-        if (lane == 0) mbar_expect_tx(smem_u32(k_full), kQBytes);
-        __syncwarp();
-        tma_load_pages(smem_u32(sK), kSubBytes, &tmK, smem_u32(k_full), table, args.block_size, j * kTile, end, kcol, QB);
-        wait_free(v_empty, ph ^ 1);
+        tma_load_pages(leader, smem_u32(sK), kSubBytes, &tmK, smem_u32(k_full), page, bs, kcol, QB);
+        const int next = j + 1 < t.n_kv ? tile_page(table, bs, (j + 1) * kTile, end) : 0;
+        claim(v_empty, ph ^ 1, v_full, kVBytes);
         if (!ok) break;
-        if (lane == 0) mbar_expect_tx(smem_u32(v_full), kVBytes);
-        __syncwarp();
-        tma_load_pages(smem_u32(sV), kSubBytes, &tmV, smem_u32(v_full), table, args.block_size, j * kTile, end, vcol, VB);
+        tma_load_pages(leader, smem_u32(sV), kSubBytes, &tmV, smem_u32(v_full), page, bs, vcol, VB);
+        page = next;
       }
     }
   } else if (warp == 1) {
@@ -547,43 +550,47 @@ paged_prefill_values_kernel(const __grid_constant__ CUtensorMap tmQ, const __gri
   const uint32_t tmem_O = tmem_base + 2 * kTile;     // P of a tile lives in the first 64 columns of its scores
 
   if (warp == 0) {
-    // ------------------------------ TMA producer (the whole warp) ------------------------------
+    // ------------------------------ TMA producer (the whole warp, one lane issues) ------------------------------
+    const bool leader = elect_one();
+    const int bs = args.block_size;
     uint32_t it = 0, n = 0, unit = 0;                // key tiles, query tiles and V tiles so far
     bool ok = true;
-    // wait until a buffer is free; the lanes agree on the outcome
-    auto wait_free = [&](uint64_t* bar, uint32_t parity) {
-      ok = mbar_wait(smem_u32(bar), parity, abort_flag, args.status, kStatusWaitTimeoutProducer);
+    // wait until a buffer is free (the lanes agree on the outcome) and announce what goes there
+    auto claim = [&](uint64_t* empty, uint32_t parity, uint64_t* full, uint32_t bytes) {
+      ok = mbar_wait(smem_u32(empty), parity, abort_flag, args.status, kStatusWaitTimeoutProducer);
       ok = __all_sync(0xffffffffu, ok);
+      if (ok && leader) mbar_expect_tx(smem_u32(full), bytes);
+      __syncwarp();
     };
     for (int item = first_item; item < args.n_items && ok; item += step, ++n) {
       const Tile t = tile_of(item);
-      wait_free(q_empty, (n & 1) ^ 1);
-      if (!ok) break;
-      if (lane == 0) mbar_expect_tx(smem_u32(q_full), kQBytes);
-      __syncwarp();
-      if (lane < QB) tma_load_3d(smem_u32(sQ) + lane * kSubBytes, &tmQ, smem_u32(q_full), lane * 64, t.head, t.q0);
       const int* table = args.block_tables + static_cast<size_t>(t.b) * args.max_blocks;
       const int end = t.pos0 + t.rows, kcol = t.head / args.group * args.D;
-      auto load = [&](const CUtensorMap* tm, uint8_t* dst, uint64_t* full, uint32_t bytes, int j, int col, int subs) {
-        if (lane == 0) mbar_expect_tx(smem_u32(full), bytes);
-        __syncwarp();
-        tma_load_pages(smem_u32(dst), kSubBytes, tm, smem_u32(full), table, args.block_size, j * kTile, end, col, subs);
-      };
-      auto load_k = [&](int j) {
+      int page = tile_page(table, bs, t.lo * kTile, end);
+      claim(q_empty, (n & 1) ^ 1, q_full, kQBytes);
+      if (!ok) break;
+      if (leader)
+        for (int c = 0; c < QB; ++c) tma_load_3d(smem_u32(sQ) + c * kSubBytes, &tmQ, smem_u32(q_full), c * 64, t.head, t.q0);
+      __syncwarp();
+      auto load_k = [&](int pg) {
         const int st = it & 1;
-        wait_free(&k_empty[st], ((it >> 1) & 1) ^ 1);
+        claim(&k_empty[st], ((it >> 1) & 1) ^ 1, &k_full[st], kQBytes);
         if (!ok) return;
-        load(&tmK, sK + st * kQBytes, &k_full[st], kQBytes, j, kcol, QB);
+        tma_load_pages(leader, smem_u32(sK) + st * kQBytes, kSubBytes, &tmK, smem_u32(&k_full[st]), pg, bs, kcol, QB);
         ++it;
       };
-      load_k(t.lo);
+      load_k(page);
       for (int j = t.lo; j < t.n_kv && ok; ++j) {
-        if (j + 1 < t.n_kv) load_k(j + 1);
+        const int next = j + 1 < t.n_kv ? tile_page(table, bs, (j + 1) * kTile, end) : 0;
+        if (j + 1 < t.n_kv) load_k(next);
         for (int v = 0; v < t.nv && ok; ++v, ++unit) {
           const int slot = unit % kSlots;
-          wait_free(&v_empty[slot], ((unit / kSlots) & 1) ^ 1);
-          if (ok) load(&tmV, sV + slot * kVBytes, &v_full[slot], kVBytes, j, (t.v0 + v) * args.DV, VB);
+          claim(&v_empty[slot], ((unit / kSlots) & 1) ^ 1, &v_full[slot], kVBytes);
+          if (ok)
+            tma_load_pages(leader, smem_u32(sV) + slot * kVBytes, kSubBytes, &tmV, smem_u32(&v_full[slot]), page, bs,
+                           (t.v0 + v) * args.DV, VB);
         }
+        page = next;
       }
     }
   } else if (warp == 1) {

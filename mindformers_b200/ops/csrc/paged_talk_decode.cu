@@ -47,7 +47,7 @@ __device__ __forceinline__ float ex2(float x) {
 }
 
 __host__ __device__ constexpr int fixed_bytes(int Hp, int items) {
-  return 2 * 2 * Hp * 128 + items * kQItem + Hp * kTile * 4 + 3 * kMaxHeads * 4 + 2 * 4 * kItem * 4 +
+  return 2 * 2 * Hp * 128 + items * kQItem + Hp * kTile * 4 + 6 * kMaxHeads * 4 +
          (8 + 2 * kMaxSlots + 2 * kMaxItems) * 8 + 16 + 1024;
 }
 
@@ -62,10 +62,10 @@ paged_talk_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
   uint8_t* sP = sRing + slots * kUnit;                      // two buffers of two [Hp heads][64 tokens] sub-tiles
   uint8_t* sQ = sP + 2 * p_buf;
   float* sL = reinterpret_cast<float*>(sQ + items * kQItem);          // [Hp][128] sums per token row
-  float* sM = sL + Hp * kTile;                              // [2][kMaxHeads] running maxima
-  float* sAlpha = sM + 2 * kMaxHeads;                       // [kMaxHeads]
-  float* red = sAlpha + kMaxHeads;                          // [2][4 warps][16]
-  uint64_t* bars = reinterpret_cast<uint64_t*>(red + 2 * 4 * kItem);
+  float* sM = sL + Hp * kTile;                              // [kMaxHeads] running maxima
+  float* sAlpha = sM + kMaxHeads;                           // [kMaxHeads]
+  float* red = sAlpha + kMaxHeads;                          // [4 warps][kMaxHeads]
+  uint64_t* bars = reinterpret_cast<uint64_t*>(red + 4 * kMaxHeads);
   uint64_t* q_full = bars;
   uint64_t* p_ready = bars + 1;
   uint64_t* pv_done = bars + 2;
@@ -123,33 +123,39 @@ paged_talk_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
   const uint32_t tmem_S = tmem_O + nv_max * Hp;             // two buffers of `items` blocks of 16 columns
 
   if (warp == 0) {
-    // ------------------------------------ producer (the whole warp) ------------------------------------
+    // ------------------------------------ producer (the whole warp, one lane issues) ------------------------------------
     if (n_tiles > 0) {
-      if (lane == 0) mbar_expect_tx(smem_u32(q_full), items * k_halves * (kItem * 128));
-      __syncwarp();
-      for (int x = lane; x < items * k_halves; x += 32) {
-        const int i = x / k_halves, c = x % k_halves;
-        const int head0 = (i / args.per_kv) * args.group + (i % args.per_kv) * kItem;
-        tma_load_2d(smem_u32(sQ) + i * kQItem + c * (kItem * 128), &tmQ, smem_u32(q_full), c * 64, q_row * args.H + head0);
+      const bool leader = elect_one();
+      if (leader) {
+        mbar_expect_tx(smem_u32(q_full), items * k_halves * (kItem * 128));
+        for (int i = 0; i < items; ++i) {
+          const int head0 = (i / args.per_kv) * args.group + (i % args.per_kv) * kItem;
+          for (int c = 0; c < k_halves; ++c)
+            tma_load_2d(smem_u32(sQ) + i * kQItem + c * (kItem * 128), &tmQ, smem_u32(q_full), c * 64, q_row * args.H + head0);
+        }
       }
+      __syncwarp();
+      const int bs = args.block_size;
       const int* table = args.block_tables + static_cast<size_t>(b) * args.max_blocks;
       uint32_t unit = 0;
       bool ok = true;
-      auto load_tile = [&](const CUtensorMap* tm, int j, int col0, int halves) {
+      auto load_tile = [&](const CUtensorMap* tm, int page, int col0, int halves) {
         const int slot = unit % slots;
         ok = mbar_wait(smem_u32(&empty[slot]), ((unit / slots) & 1) ^ 1, abort_flag, args.status, kStatusWaitTimeoutProducer);
         ok = __all_sync(0xffffffffu, ok);
         if (!ok) return;
-        if (lane == 0) mbar_expect_tx(smem_u32(&full[slot]), halves * kSub);
+        if (leader) mbar_expect_tx(smem_u32(&full[slot]), halves * kSub);
         __syncwarp();
-        tma_load_pages(smem_u32(sRing + slot * kUnit), kSub, tm, smem_u32(&full[slot]), table, args.block_size, (t0 + j) * kTile, len,
-                       col0, halves);
+        tma_load_pages(leader, smem_u32(sRing + slot * kUnit), kSub, tm, smem_u32(&full[slot]), page, bs, col0, halves);
         ++unit;
       };
-      for (int g = 0; g < args.G && ok; ++g) load_tile(&tmK, 0, g * args.D, k_halves);
+      int page = tile_page(table, bs, t0 * kTile, len);
+      for (int g = 0; g < args.G && ok; ++g) load_tile(&tmK, page, g * args.D, k_halves);
       for (int j = 0; j < n_tiles && ok; ++j) {
-        for (int g = 0; g < args.G && ok && j + 1 < n_tiles; ++g) load_tile(&tmK, j + 1, g * args.D, k_halves);
-        for (int v = 0; v < nv && ok; ++v) load_tile(&tmV, j, (v0 + v) * args.DV, v_halves);
+        const int next = j + 1 < n_tiles ? tile_page(table, bs, (t0 + j + 1) * kTile, len) : 0;
+        for (int g = 0; g < args.G && ok && j + 1 < n_tiles; ++g) load_tile(&tmK, next, g * args.D, k_halves);
+        for (int v = 0; v < nv && ok; ++v) load_tile(&tmV, page, (v0 + v) * args.DV, v_halves);
+        page = next;
       }
     }
   } else if (warp == 1) {
@@ -219,7 +225,7 @@ paged_talk_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
     const int row = ew * 32 + lane;                         // token row of S^T, value row of O^T
     const uint32_t lane_base = static_cast<uint32_t>(ew * 32) << 16;
     for (int h = 0; h < Hp; ++h) sL[h * kTile + row] = 0.f;
-    if (row < kMaxHeads) sM[row] = sM[kMaxHeads + row] = -INFINITY;
+    if (row < kMaxHeads) sM[row] = -INFINITY;
     named_bar_sync(1, 128);
     bool ok = true;
     for (int j = 0; j < n_tiles && ok; ++j) {
@@ -228,7 +234,8 @@ paged_talk_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
       const bool valid = tok < len && tok >= first_tok;
       uint8_t* pcol = sP + sb * p_buf + (row >> 6) * p_sub + (row & 7) * 2;
       const int cell = (row & 63) >> 3;
-      bool rescale = false;
+      // the heads' maxima change seldom: first only see whether some score is more than 2^8 above its head's
+      bool fine = true;
       for (int i = 0; i < items; ++i) {
         const int head0 = (i / args.per_kv) * args.group + (i % args.per_kv) * kItem;
         const int nh = min(kItem, (i / args.per_kv + 1) * args.group - head0);
@@ -237,36 +244,48 @@ paged_talk_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
         uint32_t sr[kItem];
         tmem_ld_32x32b_x16(tmem_S + (sb * items + i) * kItem + lane_base, sr);
         tmem_ld_wait();
-        float* rd = red + (i & 1) * 4 * kItem;
-        float s[kItem];
 #pragma unroll
         for (int h = 0; h < kItem; ++h)
-          if (h < nh) {
-            s[h] = valid ? __uint_as_float(sr[h]) * args.scale_log2 : -INFINITY;
-            const float w = warp_max(s[h]);
-            if (lane == 0) rd[ew * kItem + h] = w;
-          }
+          if (h < nh) fine = fine && !(valid && __uint_as_float(sr[h]) * args.scale_log2 > sM[head0 + h] + kRescale);
+      }
+      const bool rescale = !named_bar_and(2, 128, fine);
+      if (rescale) {
+        for (int i = 0; i < items; ++i) {
+          const int head0 = (i / args.per_kv) * args.group + (i % args.per_kv) * kItem;
+          const int nh = min(kItem, (i / args.per_kv + 1) * args.group - head0);
+          uint32_t sr[kItem];
+          tmem_ld_32x32b_x16(tmem_S + (sb * items + i) * kItem + lane_base, sr);
+          tmem_ld_wait();
+#pragma unroll
+          for (int h = 0; h < kItem; ++h)
+            if (h < nh) {
+              const float w = warp_max(valid ? __uint_as_float(sr[h]) * args.scale_log2 : -INFINITY);
+              if (lane == 0) red[ew * kMaxHeads + head0 + h] = w;
+            }
+        }
         named_bar_sync(1, 128);
+        if (row < args.H) {
+          const float mx = fmaxf(fmaxf(red[row], red[kMaxHeads + row]), fmaxf(red[2 * kMaxHeads + row], red[3 * kMaxHeads + row]));
+          const float m = sM[row];
+          const bool grown = mx > m + kRescale;             // or nothing was accumulated yet
+          sAlpha[row] = grown ? (m == -INFINITY ? 0.f : ex2(m - mx)) : 1.f;
+          if (grown) sM[row] = mx;
+        }
+        named_bar_sync(1, 128);
+        for (int h = 0; h < args.H; ++h) sL[h * kTile + row] *= sAlpha[h];
+      }
+      for (int i = 0; i < items; ++i) {
+        const int head0 = (i / args.per_kv) * args.group + (i % args.per_kv) * kItem;
+        const int nh = min(kItem, (i / args.per_kv + 1) * args.group - head0);
+        uint32_t sr[kItem];
+        tmem_ld_32x32b_x16(tmem_S + (sb * items + i) * kItem + lane_base, sr);
+        tmem_ld_wait();
 #pragma unroll
         for (int h = 0; h < kItem; ++h)
           if (h < nh) {
             const int head = head0 + h;
-            const float mx = fmaxf(fmaxf(rd[h], rd[kItem + h]), fmaxf(rd[2 * kItem + h], rd[3 * kItem + h]));
-            float m = sM[sb * kMaxHeads + head], alpha = 1.f;
-            if (m == -INFINITY) {
-              m = mx;                                       // first tile with a visible token (nothing accumulated yet)
-            } else if (mx > m + kRescale) {
-              alpha = ex2(m - mx);
-              m = mx;
-              rescale = true;
-            }
-            if (row == 0) {
-              sM[(sb ^ 1) * kMaxHeads + head] = m;
-              sAlpha[head] = alpha;
-            }
-            const float p = valid ? ex2(s[h] - m) : 0.f;
-            float* l = sL + head * kTile + row;
-            *l = *l * alpha + p;
+            const float p = valid ? ex2(fmaf(__uint_as_float(sr[h]), args.scale_log2, -sM[head])) : 0.f;
+            sL[head * kTile + row] += p;
             *reinterpret_cast<__nv_bfloat16*>(pcol + head * 128 + ((cell ^ (head & 7)) << 4)) = __float2bfloat16_rn(p);
           }
       }
@@ -307,7 +326,7 @@ paged_talk_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
         const float sum = warp_sum((l[lane] + l[lane + 32]) + (l[lane + 64] + l[lane + 96]));
         if (lane == 0) {
           float* ml = args.part_ml + ((static_cast<size_t>(b) * args.H + h) * args.splits + split) * 2;
-          ml[0] = have ? sM[(n_tiles & 1) * kMaxHeads + h] : -INFINITY;
+          ml[0] = have ? sM[h] : -INFINITY;
           ml[1] = have ? sum : 0.f;
         }
       }
