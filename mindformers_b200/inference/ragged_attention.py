@@ -273,8 +273,9 @@ def _absorbed(q, cache, layer, w_uk, w_uv, scale, window, sink):
     """Queries through the key factor, attention over the latents themselves, results through the value factor: ``[T, heads *
     v_dim]``."""
     T, H = q.shape[0], q.shape[1]
-    q_lat = torch.bmm(q.transpose(0, 1), w_uk).transpose(0, 1).contiguous()                    # [T, heads, rank]
-    R = q_lat.shape[2]
+    R, DV = w_uk.shape[2], w_uv.shape[1]
+    q_lat = torch.empty((T, H, R), dtype=q.dtype, device=q.device)
+    torch.bmm(q.transpose(0, 1), w_uk, out=q_lat.transpose(0, 1))
     lib = _lib.get_lib() if q.is_cuda else None
     if lib is not None and q.dtype == torch.bfloat16 and not cache.is_prefill \
             and lib.mfb_latent_decode_supported(R, cache.block_size):
@@ -292,7 +293,9 @@ def _absorbed(q, cache, layer, w_uk, w_uv, scale, window, sink):
         _lib.count_launch(2)
     else:
         o_lat = ragged_attention(q_lat, cache, layer, scale, sink=sink, window=window).view(T, H, R)
-    return torch.bmm(o_lat.transpose(0, 1), w_uv.transpose(1, 2)).transpose(0, 1).reshape(T, -1)
+    out = torch.empty((T, H, DV), dtype=q.dtype, device=q.device)
+    torch.bmm(o_lat.transpose(0, 1), w_uv.transpose(1, 2), out=out.transpose(0, 1))
+    return out.view(T, H * DV)
 
 
 def latent_attention(q: torch.Tensor, cache, layer: int, w_kv: torch.Tensor, v_dim: int, scale: float, window: int = 0,

@@ -3,11 +3,14 @@
 // decode step is, per sequence and head h with q, c of `rank` numbers (a multiple of 8 up to 512):
 //     s[t]   = scale * <q[h], c[t]>                       max(0, len - window) <= t < len
 //     o[h,:] = sum_t softmax(s)[t] * c[t]                 the sink is one more term of the softmax's denominator
-// The layout is that of mla_decode.cu, which serves one fixed latent width beside rotated columns: a CTA handles (split of the
-// sequence, 16 heads, sequence), the products are transposed so that the tokens fill the 128 rows of the tensor core, and a
-// tile of 128 tokens streams twice through a ring of 32 KB slots (128 latent columns each, the last one possibly half), once
-// for S^T and once, from L2, for O^T. Columns past the rank are zero fill in both operands; the rows of O^T that belong to
-// them are not stored. Two CTAs share an SM.
+// As in mla_decode.cu, which serves one fixed latent width beside rotated columns, the products are transposed so that the tokens
+// fill the 128 rows of the tensor core, and a CTA takes (split of the sequence, 16 or 32 heads, sequence):
+//     S^T [128 tokens x heads]       = C_tile (A, K-major) . Q^T (B, K-major)
+//     O^T [rank x heads]            += C_tile^T (A, MN-major: the same bytes) . P^T [heads x 128 tokens] (B, K-major)
+// A tile of 128 tokens lies in up to four 32 KB slots of a ring (128 latent columns each, the last one possibly half) from its
+// scores to its last product, so the cache is read once per 32 heads. Where two tiles fit the ring, the scores of the next tile
+// are computed under the softmax of this one. Columns past the rank are zero fill in both operands; the rows of O^T that belong
+// to them are not stored.
 //
 // Roles (192 threads): warp 0 TMA producer (block-table lookups), warp 1 MMA issuer + TMEM owner, warps 2..5 softmax / rescale /
 // epilogue. Every wait is bounded (common.cuh). The splits are merged by the combine kernel of paged_attention.cu.
@@ -18,16 +21,22 @@ namespace latd {
 
 constexpr int kThreads = 192;
 constexpr int kTile = 128;              // tokens per tile
-constexpr int kHeads = 16;              // heads per CTA
 constexpr int kMaxRank = 512;
 constexpr int kSub = kTile * 128;       // [128 tokens][64 columns] swizzled sub-tile, 16 KB
 constexpr int kUnit = 2 * kSub;         // ring slot: a pair of sub-tiles (128 columns)
-constexpr int kSlots = 2;
-constexpr int kPBytes = 2 * kHeads * 128;   // P^T: two [16 heads][64 tokens] K-major sub-tiles
-constexpr int kTmemCols = 256;
-constexpr int kQSub = kHeads * 128;     // [16 heads][64 columns], 2 KB
-constexpr int kQBytes = kMaxRank / 64 * kQSub;
+constexpr int kMaxSlots = 6;
 constexpr float kRescale = 8.0f;
+
+// per number of heads of a CTA: P^T as two [heads][64 tokens] K-major sub-tiles, Q as [heads][64 columns] sub-tiles
+template <int HEADS>
+struct Shape {
+  static constexpr int kPBytes = 2 * HEADS * 128, kQSub = HEADS * 128, kQBytes = kMaxRank / 64 * kQSub;
+  static constexpr int kFixed = kPBytes + kQBytes + 4 * HEADS * 4 + (7 + 2 * kMaxSlots) * 8 + 16 + 1024;
+  static constexpr int kFit = (232448 - kFixed) / kUnit;
+  static constexpr int kSlots = kFit < kMaxSlots ? kFit : kMaxSlots;
+  static constexpr int kSmem = kFixed + kSlots * kUnit;
+  static constexpr int kTmemCols = HEADS <= 16 ? 128 : 256;      // four blocks of O^T and two buffers of S^T
+};
 
 struct Args {
   const int* block_tables;   // [B, max_blocks]
@@ -45,24 +54,28 @@ __device__ __forceinline__ float ex2(float x) {
   return y;
 }
 
-__global__ void __launch_bounds__(kThreads, 2)
+template <int HEADS>
+__global__ void __launch_bounds__(kThreads, 1)
 latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmC, const Args args) {
+  using Sh = Shape<HEADS>;
+  constexpr int kHeads = HEADS, kSlots = Sh::kSlots, kPBytes = Sh::kPBytes, kQSub = Sh::kQSub, kQBytes = Sh::kQBytes;
+  constexpr int kTmemCols = Sh::kTmemCols;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) &
                                              ~static_cast<uintptr_t>(1023));
-  uint8_t* sRing = smem;                               // 2 x 32 KB
-  uint8_t* sP = sRing + kSlots * kUnit;          // 4 KB
-  uint8_t* sQ = sP + kPBytes;                       // 18 KB
-  float* red = reinterpret_cast<float*>(sQ + kQBytes);          // [4 warps][16]
+  uint8_t* sRing = smem;
+  uint8_t* sP = sRing + kSlots * kUnit;
+  uint8_t* sQ = sP + kPBytes;
+  float* red = reinterpret_cast<float*>(sQ + kQBytes);  // [4 warps][heads]
   uint64_t* bars = reinterpret_cast<uint64_t*>(red + 4 * kHeads);
   uint64_t* q_full = bars;                  // 1
-  uint64_t* full = bars + 1;                // up to 5
-  uint64_t* empty = bars + 6;               // up to 5
-  uint64_t* s_full = bars + 11;             // 2
-  uint64_t* s_empty = bars + 13;            // 2
-  uint64_t* p_ready = bars + 15;            // 1
-  uint64_t* pv_done = bars + 16;            // 1
-  uint32_t* tmem_holder = reinterpret_cast<uint32_t*>(bars + 17);
+  uint64_t* p_ready = bars + 1;             // 1
+  uint64_t* pv_done = bars + 2;             // 1
+  uint64_t* s_full = bars + 3;              // 2
+  uint64_t* s_empty = bars + 5;             // 2
+  uint64_t* full = bars + 7;                // kSlots
+  uint64_t* empty = full + kMaxSlots;       // kSlots
+  uint32_t* tmem_holder = reinterpret_cast<uint32_t*>(empty + kMaxSlots);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_holder + 1);
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -105,8 +118,8 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
   __syncthreads();
   tc_fence_after();
   const uint32_t tmem_base = *tmem_holder;
-  const uint32_t tmem_O = tmem_base;              // 4 blocks of 16 columns, 32 apart
-  const uint32_t tmem_S = tmem_base + 128;        // 2 buffers of 16 columns, 32 apart
+  const uint32_t tmem_O = tmem_base;                   // 4 blocks of `heads` columns
+  const uint32_t tmem_S = tmem_base + 4 * kHeads;      // 2 buffers of `heads` columns
 
   if (warp == 0) {
     // ------------------------------------ producer (the whole warp, one lane issues) ------------------------------------
@@ -124,13 +137,11 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
       int page = tile_page(table, bs, t0 * kTile, len);
       for (int j = 0; j < n_tiles && ok; ++j) {
         const int next = j + 1 < n_tiles ? tile_page(table, bs, (t0 + j + 1) * kTile, len) : 0;
-        // two passes over the tile's pairs: for S^T, then again for O^T
-        for (int u = 0; u < 2 * units && ok; ++u) {
+        for (int pair = 0; pair < units && ok; ++pair) {
           const int slot = unit % kSlots;
           ok = mbar_wait(smem_u32(&empty[slot]), ((unit / kSlots) & 1) ^ 1, abort_flag, args.status, kStatusWaitTimeoutProducer);
           ok = __all_sync(0xffffffffu, ok);
           if (!ok) break;
-          const int pair = u < units ? u : u - units;
           const int two = 2 * pair + 1 < subs ? 2 : 1;
           if (leader) mbar_expect_tx(smem_u32(&full[slot]), two * kSub);
           __syncwarp();
@@ -148,50 +159,50 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
       const bool leader = elect_one();
       const uint64_t ring_k = umma_desc_kmajor_sw128(smem_u32(sRing)), ring_v = umma_desc_mnmajor_sw128(smem_u32(sRing), kSub);
       const uint64_t q_desc = umma_desc_kmajor_sw128(smem_u32(sQ)), p_desc = umma_desc_kmajor_sw128(smem_u32(sP));
-      uint32_t unit = 0;
       bool ok = true;
       auto wait = [&](uint64_t* bar, uint32_t parity) {
         ok = mbar_wait(smem_u32(bar), parity, abort_flag, args.status, kStatusWaitTimeoutMma);
         ok = __all_sync(0xffffffffu, ok);
       };
-      wait(q_full, 0);
-      for (int j = 0; j < n_tiles && ok; ++j) {
+      // ---- S^T(j) = C . Q^T over the pairs of the tile, which stay in the ring ----
+      auto scores = [&](int j) {
         const int sb = j & 1;
         wait(&s_empty[sb], ((j >> 1) & 1) ^ 1);
-        // ---- S^T = C . Q^T over the pairs of the first pass ----
         for (int u = 0; u < units && ok; ++u) {
-          const int slot = unit % kSlots;
+          const int unit = j * units + u, slot = unit % kSlots;
           wait(&full[slot], (unit / kSlots) & 1);
-          if (!ok) break;
+          if (!ok) return;
           tc_fence_after();
           const uint64_t ca = ring_k + slot * (kUnit >> 4), qa = q_desc + 2 * u * (kQSub >> 4);
           const int ksteps = 2 * u + 1 < subs ? 8 : 4;
 #pragma unroll
           for (int k = 0; k < 8; ++k)
             if (k < ksteps)
-              umma_f16_ss_warp(leader, tmem_S + sb * 32, ca + (k >> 2) * (kSub >> 4) + (k & 3) * 2,
+              umma_f16_ss_warp(leader, tmem_S + sb * kHeads, ca + (k >> 2) * (kSub >> 4) + (k & 3) * 2,
                                qa + (k >> 2) * (kQSub >> 4) + (k & 3) * 2, IDESC_S, (u > 0 || k > 0) ? 1u : 0u);
-          umma_commit_warp(leader, smem_u32(&empty[slot]));
-          ++unit;
         }
+        if (ok) umma_commit_warp(leader, smem_u32(&s_full[sb]));
+      };
+      wait(q_full, 0);
+      const bool ahead = 2 * units <= kSlots;
+      if (ok && ahead) scores(0);
+      for (int j = 0; j < n_tiles && ok; ++j) {
+        if (!ahead) scores(j);
+        else if (j + 1 < n_tiles) scores(j + 1);
+        // ---- O^T += C^T(j) . P^T(j) ----
+        if (ok) wait(p_ready, j & 1);
         if (!ok) break;
-        umma_commit_warp(leader, smem_u32(&s_full[sb]));
-        // ---- O^T += C^T . P^T over the pairs of the second pass ----
-        wait(p_ready, j & 1);
-        for (int m = 0; m < units && ok; ++m) {
-          const int slot = unit % kSlots;
-          wait(&full[slot], (unit / kSlots) & 1);
-          if (!ok) break;
-          tc_fence_after();
+        tc_fence_after();
+        for (int m = 0; m < units; ++m) {
+          const int slot = (j * units + m) % kSlots;
           const uint64_t ca = ring_v + slot * (kUnit >> 4);
 #pragma unroll
           for (int k = 0; k < kTile / 16; ++k)
-            umma_f16_ss_warp(leader, tmem_O + m * 32, ca + k * ((16 * 128) >> 4), p_desc + (k >> 2) * ((kHeads * 128) >> 4) + (k & 3) * 2,
+            umma_f16_ss_warp(leader, tmem_O + m * kHeads, ca + k * ((16 * 128) >> 4), p_desc + (k >> 2) * ((kHeads * 128) >> 4) + (k & 3) * 2,
                              IDESC_PV, (j > 0 || k > 0) ? 1u : 0u);
           umma_commit_warp(leader, smem_u32(&empty[slot]));
-          ++unit;
         }
-        if (ok) umma_commit_warp(leader, smem_u32(pv_done));
+        umma_commit_warp(leader, smem_u32(pv_done));
       }
     }
   } else {
@@ -210,8 +221,10 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
       ok = named_bar_and(2, 128, ok);
       if (!ok) break;
       tc_fence_after();
-      uint32_t sr[16];
-      tmem_ld_32x32b_x16(tmem_S + sb * 32 + lane_base, sr);
+      uint32_t sr[kHeads];
+#pragma unroll
+      for (int c = 0; c < kHeads; c += 16)
+        tmem_ld_32x32b_x16(tmem_S + sb * kHeads + c + lane_base, *reinterpret_cast<uint32_t(*)[16]>(&sr[c]));
       tmem_ld_wait();
       tc_fence_before();
       mbar_arrive(smem_u32(&s_empty[sb]));
@@ -256,14 +269,16 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
         ok = mbar_wait(smem_u32(pv_done), (j - 1) & 1, abort_flag, args.status, kStatusWaitTimeoutEpilogue);
         if (ok && any_rescale) {
           tc_fence_after();
-          for (int m = 0; m < units; ++m) {
-            uint32_t r[16];
-            tmem_ld_32x32b_x16(tmem_O + lane_base + m * 32, r);
-            tmem_ld_wait();
+          for (int m = 0; m < units; ++m)
 #pragma unroll
-            for (int h = 0; h < kHeads; ++h) r[h] = __float_as_uint(__uint_as_float(r[h]) * alpha[h]);
-            tmem_st_32x32b_x16(tmem_O + lane_base + m * 32, r);
-          }
+            for (int c = 0; c < kHeads; c += 16) {
+              uint32_t r[16];
+              tmem_ld_32x32b_x16(tmem_O + lane_base + m * kHeads + c, r);
+              tmem_ld_wait();
+#pragma unroll
+              for (int h = 0; h < 16; ++h) r[h] = __float_as_uint(__uint_as_float(r[h]) * alpha[c + h]);
+              tmem_st_32x32b_x16(tmem_O + lane_base + m * kHeads + c, r);
+            }
           tmem_st_wait();
         }
       }
@@ -310,16 +325,19 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
     }
     if (have) tc_fence_after();
     for (int m = 0; m < units; ++m) {
-      uint32_t r[16];
-      if (have) {
-        tmem_ld_32x32b_x16(tmem_O + lane_base + m * 32, r);
-        tmem_ld_wait();
-      }
       const int col = m * 128 + row;
 #pragma unroll
-      for (int h = 0; h < kHeads; ++h)
-        if (head0 + h < args.num_heads && col < args.rank)      // a split without tokens writes zeros, which the merge weighs by zero
-          args.part_o[((first_row + h) * args.splits + split) * args.rank + col] = have ? __uint_as_float(r[h]) : 0.f;
+      for (int c = 0; c < kHeads; c += 16) {
+        uint32_t r[16];
+        if (have) {
+          tmem_ld_32x32b_x16(tmem_O + lane_base + m * kHeads + c, r);
+          tmem_ld_wait();
+        }
+#pragma unroll
+        for (int h = 0; h < 16; ++h)
+          if (head0 + c + h < args.num_heads && col < args.rank)      // a split without tokens writes zeros, which the merge weighs by zero
+            args.part_o[((first_row + c + h) * args.splits + split) * args.rank + col] = have ? __uint_as_float(r[h]) : 0.f;
+      }
     }
   }
   tc_fence_before();
@@ -329,6 +347,27 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
     tmem_dealloc(tmem_base, kTmemCols);
   }
 }
+
+
+template <int HEADS>
+int launch(const CUtensorMap& tQ, const CUtensorMap& tC, const Args& a, int B, cudaStream_t stream) {
+  using Sh = Shape<HEADS>;
+  static_assert(Sh::kSlots >= 4, "a tile has up to four pairs");
+  static bool attr_set = false;
+  if (!attr_set) {
+    if (cudaFuncSetAttribute(latent_decode_kernel<HEADS>, cudaFuncAttributeMaxDynamicSharedMemorySize, Sh::kSmem) != cudaSuccess) {
+      mfb_host::set_error("latent_decode: cannot raise shared memory limit");
+      return 10;
+    }
+    attr_set = true;
+  }
+  const dim3 grid(a.splits, (a.num_heads + HEADS - 1) / HEADS, B);
+  latent_decode_kernel<HEADS><<<grid, kThreads, Sh::kSmem, stream>>>(tQ, tC, a);
+  if (cudaGetLastError() != cudaSuccess) { mfb_host::set_error("latent_decode: launch failed"); return 11; }
+  return 0;
+}
+
+int heads_per_cta(int num_heads) { return num_heads > 16 ? 32 : 16; }
 
 }  // namespace latd
 }  // namespace mfb
@@ -348,14 +387,14 @@ int mfb_latent_decode_supported(int rank, int block_size) {
 
 // Number of sequence splits that fills the GPU for a batch of B sequences of up to max_len visible tokens.
 int mfb_latent_decode_splits(int B, int num_heads, int max_len) {
-  // cost of a choice = waves of CTAs over the 2 x 148 resident CTAs x (tiles per CTA + about one tile of fixed work per CTA)
-  const int chunks = (num_heads + latd::kHeads - 1) / latd::kHeads;
+  // cost of a choice = waves of CTAs over the 148 SMs x (tiles per CTA + about one tile of fixed work per CTA)
+  const int per = latd::heads_per_cta(num_heads), chunks = (num_heads + per - 1) / per;
   const int tiles = (max_len + latd::kTile - 1) / latd::kTile;
   int best = 1;
   long long best_cost = -1;
   for (int s = 1; s <= tiles && s <= 32; ++s) {
     const long long ctas = static_cast<long long>(B) * chunks * s;
-    const long long waves = (ctas + 295) / 296;
+    const long long waves = (ctas + 147) / 148;
     const long long cost = waves * ((tiles + s - 1) / s + 1);
     if (best_cost < 0 || cost < best_cost) { best_cost = cost; best = s; }
   }
@@ -380,7 +419,7 @@ int mfb_latent_decode(const void* q, const void* cache, const int* block_tables,
   CUtensorMap tQ, tC;
   int rc;
   const CUtensorMapDataType BF = CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
-  if ((rc = mfb_host::make_tmap_2d(&tQ, q, 2, BF, (uint64_t)B * num_heads, rank, rank, latd::kHeads, 64))) return 20 + rc;
+  if ((rc = mfb_host::make_tmap_2d(&tQ, q, 2, BF, (uint64_t)B * num_heads, rank, rank, latd::heads_per_cta(num_heads), 64))) return 20 + rc;
   if ((rc = mfb_host::make_tmap_2d(&tC, cache, 2, BF, (uint64_t)num_blocks * block_size, rank, rank, block_size, 64))) return 30 + rc;
   latd::Args a;
   a.block_tables = block_tables; a.context_lens = context_lens; a.max_blocks = max_blocks; a.block_size = block_size;
@@ -388,18 +427,8 @@ int mfb_latent_decode(const void* q, const void* cache, const int* block_tables,
   a.part_o = reinterpret_cast<float*>(scratch);
   a.part_ml = a.part_o + static_cast<size_t>(B) * splits * num_heads * rank;
   a.status = status;
-  constexpr int SMEM = latd::kSlots * latd::kUnit + latd::kPBytes + latd::kQBytes + 4 * latd::kHeads * 4 + 18 * 8 + 16 + 1024;
-  static bool attr_set = false;
-  if (!attr_set) {
-    if (cudaFuncSetAttribute(latd::latent_decode_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM) != cudaSuccess) {
-      mfb_host::set_error("latent_decode: cannot raise shared memory limit");
-      return 10;
-    }
-    attr_set = true;
-  }
-  const dim3 grid(splits, (num_heads + latd::kHeads - 1) / latd::kHeads, B);
-  latd::latent_decode_kernel<<<grid, latd::kThreads, SMEM, stream>>>(tQ, tC, a);
-  if (cudaGetLastError() != cudaSuccess) { mfb_host::set_error("latent_decode: launch failed"); return 11; }
+  rc = latd::heads_per_cta(num_heads) == 32 ? latd::launch<32>(tQ, tC, a, B, stream) : latd::launch<16>(tQ, tC, a, B, stream);
+  if (rc) return rc;
   return mfb_paged_combine_ex(a.part_o, a.part_ml, out, splits, B * num_heads, rank, num_heads, nullptr, sink,
                               (long long)num_heads * rank, 1.f, stream);
 }
