@@ -353,14 +353,14 @@ paged_talk_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
   }
 }
 
-constexpr int kParts = 8, kAcc = 8;      // heads g in this many parts; result heads at a time
+constexpr int kParts = 8, kAcc = 8;      // heads g in up to this many parts; result heads at a time
 
-// CTA (key / value head and eight of its result heads, sequence): threads (column of the head, part of the heads g)
-__global__ void __launch_bounds__(1024)
+// CTA (key / value head and eight of its result heads, sequence): threads (four columns of the head, part of the heads g)
+__global__ void __launch_bounds__(256)
 talk_combine_kernel(const float* __restrict__ part_acc, const float* __restrict__ part_ml, const float* __restrict__ talk,
                     const __nv_bfloat16* __restrict__ gate, long long ld_gate, __nv_bfloat16* __restrict__ out, int H, int G, int DV,
                     int splits, int blocks, const int* __restrict__ cu_q) {
-  extern __shared__ float sh[];            // [H][splits] weights, [kParts][kAcc][DV] partial sums
+  extern __shared__ __align__(16) float sh[];        // [parts][kAcc][DV] partial sums, [H][splits] weights
   const int b = blockIdx.y, kv = blockIdx.x / blocks, group = H / G;
   const int h0 = kv * group + (blockIdx.x % blocks) * kAcc, n = min(kAcc, kv * group + group - h0);
   long long row = b;
@@ -368,8 +368,9 @@ talk_combine_kernel(const float* __restrict__ part_acc, const float* __restrict_
     row = cu_q[b];
     if (cu_q[b + 1] - cu_q[b] != 1) return;
   }
-  float* sW = sh;
-  float* sO = sh + H * splits;
+  const int nv = DV / 4, parts = blockDim.x / nv;
+  float* sO = sh;
+  float* sW = sh + parts * kAcc * DV;
   for (int g = threadIdx.x; g < H; g += blockDim.x) {
     const float* ml = part_ml + (static_cast<size_t>(b) * H + g) * splits * 2;
     float M = -INFINITY, L = 0.f;
@@ -384,20 +385,32 @@ talk_combine_kernel(const float* __restrict__ part_acc, const float* __restrict_
     for (int s = 0; s < splits; ++s) sW[g * splits + s] *= inv;
   }
   __syncthreads();
-  const int d = threadIdx.x % DV, part = threadIdx.x / DV, parts = blockDim.x / DV;
+  const int d = (threadIdx.x % nv) * 4, part = threadIdx.x / nv;
   if (part < parts) {
-    float acc[kAcc] = {};
+    float acc[kAcc][4] = {};
     for (int g = part; g < H; g += parts) {
       const float* src = part_acc + ((static_cast<size_t>(b) * H + g) * G + kv) * splits * DV + d;
-      float v = 0.f;
+      float v[4] = {};
 #pragma unroll 4
-      for (int s = 0; s < splits; ++s) v = fmaf(sW[g * splits + s], src[s * DV], v);
+      for (int s = 0; s < splits; ++s) {
+        const float4 x = *reinterpret_cast<const float4*>(src + s * DV);
+        const float w = sW[g * splits + s];
+        v[0] = fmaf(w, x.x, v[0]);
+        v[1] = fmaf(w, x.y, v[1]);
+        v[2] = fmaf(w, x.z, v[2]);
+        v[3] = fmaf(w, x.w, v[3]);
+      }
 #pragma unroll
       for (int i = 0; i < kAcc; ++i)
-        if (i < n) acc[i] = fmaf(talk[(h0 + i) * H + g], v, acc[i]);
+        if (i < n) {
+          const float t = talk[(h0 + i) * H + g];
+#pragma unroll
+          for (int e = 0; e < 4; ++e) acc[i][e] = fmaf(t, v[e], acc[i][e]);
+        }
     }
 #pragma unroll
-    for (int i = 0; i < kAcc; ++i) sO[(part * kAcc + i) * DV + d] = acc[i];
+    for (int i = 0; i < kAcc; ++i)
+      if (i < n) *reinterpret_cast<float4*>(sO + (part * kAcc + i) * DV + d) = make_float4(acc[i][0], acc[i][1], acc[i][2], acc[i][3]);
   }
   __syncthreads();
   for (int i = threadIdx.x; i < n * DV; i += blockDim.x) {
@@ -481,6 +494,10 @@ int mfb_paged_talk_decode(const void* q, const void* key_cache, const void* valu
   a.window = window; a.scale_log2 = scale * 1.4426950408889634f; a.status = status;
   a.part_acc = reinterpret_cast<float*>(scratch);
   a.part_ml = a.part_acc + (size_t)B * H * G * splits * DV;
+  if (reinterpret_cast<uintptr_t>(scratch) & 15) {
+    mfb_host::set_error("paged_talk_decode: the scratch must start on 16 bytes");
+    return 1;
+  }
   static bool attr_set = false;
   if (!attr_set) {
     if (cudaFuncSetAttribute(ptd::paged_talk_decode_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, ptd::kSmemLimit) != cudaSuccess ||
@@ -494,9 +511,9 @@ int mfb_paged_talk_decode(const void* q, const void* key_cache, const void* valu
   ptd::paged_talk_decode_kernel<<<dim3(splits, (G + a.nv - 1) / a.nv, B), ptd::kThreads, smem, stream>>>(tQ, tK, tV, a);
   if (cudaGetLastError() != cudaSuccess) { mfb_host::set_error("paged_talk_decode: launch failed"); return 11; }
   const int blocks = (H / G + ptd::kAcc - 1) / ptd::kAcc;
-  const int parts = 1024 / DV < ptd::kParts ? 1024 / DV : ptd::kParts;
-  const int threads = (parts * DV + 31) / 32 * 32;
-  const size_t csmem = ((size_t)H * splits + (size_t)(threads / DV) * ptd::kAcc * DV) * 4;
+  const int nv = DV / 4, parts = 256 / nv < ptd::kParts ? 256 / nv : ptd::kParts;
+  const int threads = (parts * nv + 31) / 32 * 32;
+  const size_t csmem = ((size_t)H * splits + (size_t)(threads / nv) * ptd::kAcc * DV) * 4;
   ptd::talk_combine_kernel<<<dim3(G * blocks, B), threads, csmem, stream>>>(
       a.part_acc, a.part_ml, talk, (const __nv_bfloat16*)gate, ld_gate, (__nv_bfloat16*)out, H, G, DV, splits, blocks, cu_q);
   return cudaGetLastError() == cudaSuccess ? 0 : 12;
