@@ -5,7 +5,8 @@ Equal size: same width, attention heads, head size, recurrent heads and state si
 layers and vocabulary. Half of Gavatar's layers are latent attention, a quarter each matrix memory and attention; every second
 Kukupel layer is attention beside a gated delta rule, the others have the delta rule alone. Gavatar's attention has a window.
 Model figures are device-timed (CUDA events): prefill is one call over whole prompts, decode the captured step of the device-side
-loop; so are the kernels of a decode step (replayed from a graph). L2 is flushed before every timed kernel; the working set of the model runs exceeds it. Roofline denominators are the
+loop. Kernels of a decode step and element-wise kernels are replayed from a graph, so that the host's launches are not part of
+their time. L2 is flushed before every timed kernel; the working set of the model runs exceeds it. Roofline denominators are the
 measured peaks of ``MEASURED_PEAKS.json``; the recurrences are also put against the nominal rate of the FMA pipes (148 SMs x 128
 lanes at 1965 MHz).
 """
@@ -44,7 +45,7 @@ def gavatar(size, max_len):
 
 
 def captured(fn):
-    """``fn`` as a CUDA graph: decode steps are replayed that way, so the host's launches are not part of what is timed."""
+    """``fn`` as a CUDA graph: the host's launches are not part of what is timed."""
     side = torch.cuda.Stream()
     side.wait_stream(torch.cuda.current_stream())
     with torch.cuda.stream(side):
@@ -76,7 +77,9 @@ def kernel_table(size, prompt_batch=4, prompt=4096, decode_batch=64, context=409
     def add(what, model, fn, *a):
         if only and only not in what:
             return {"ms": 1.0}
-        return out.add(what, model, captured(fn) if what.startswith("decode") else fn, *a)
+        small = what.startswith("decode") or any(w in what for w in ("embedding", "norms", "streams", "cache", "gates"))
+        return out.add(what, model, captured(fn) if small else fn, *a)
+
     m, ku = gavatar(size, 8192), kukupel(size, 8192)
     latl, mem, att = (m.model.decoder.layers[i] for i in (0, 1, 3))
     kpar, kdl = ku.model.decoder.layers[0], ku.model.decoder.layers[1]

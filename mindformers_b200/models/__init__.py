@@ -2,7 +2,8 @@ from .auto import AutoConfig, AutoModel, AutoModelForCausalLM, AutoProcessor, Au
 from .configuration_utils import PretrainedConfig
 from .families import (ChatGLM2ForConditionalGeneration, DeepseekV2Config, DeepseekV2ForCausalLM, DeepseekV3Config,
                        DeepseekV3ForCausalLM, LlamaConfig, Qwen2MoeConfig, Qwen2MoeForCausalLM,
-                       GavatarConfig, GavatarForCausalLM, KukupelConfig, KukupelForCausalLM, LlamaForCausalLM, MefesunConfig, MefesunForCausalLM,
+                       GavatarConfig, GavatarForCausalLM, KukupelConfig, KukupelForCausalLM, LlamaForCausalLM, MefesunConfig,
+                       MefesunForCausalLM,
                        MixtralConfig, MixtralForCausalLM, Qwen2Config, Qwen2ForCausalLM, Qwen3Config,
                        Qwen3ForCausalLM, Qwen3MoeConfig, Qwen3MoeForCausalLM, TelechatConfig, TelechatForCausalLM)
 from .families import ChatGLM2Config

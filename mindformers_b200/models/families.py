@@ -430,7 +430,8 @@ KukupelForCausalLM.kernel_sources = ("host_util", "elementwise", "gemm_tcgen05",
 GavatarForCausalLM = _model("GavatarForCausalLM", GavatarConfig, "gavatar")
 GavatarForCausalLM.kernel_sources = ("host_util", "elementwise", "gemm_tcgen05", "gemm_tcgen05_2cta", "gemm_bf16_decode",
                                      "sandwich_norm", "head_mix", "matrix_memory", "qkv_rope_cache", "paged_prefill_tc",
-                                     "paged_decode_tc", "paged_attention", "paged_attention_any", "paged_talk_decode", "latent_decode", "router", "moe_ep",
+                                     "paged_decode_tc", "paged_attention", "paged_attention_any", "paged_talk_decode",
+                                     "latent_decode", "router", "moe_ep",
                                      "moe_any", "decode_loop")
 ChatGLM2ForConditionalGeneration = _model("ChatGLM2ForConditionalGeneration", ChatGLM4Config, "glm")
 

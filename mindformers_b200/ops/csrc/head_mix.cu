@@ -16,7 +16,9 @@ __device__ __forceinline__ void st(__nv_bfloat16* p, float v) { *p = __float2bfl
 __device__ __forceinline__ float2 ld2(const float* p) { return *reinterpret_cast<const float2*>(p); }
 __device__ __forceinline__ float2 ld2(const __nv_bfloat16* p) { return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p)); }
 __device__ __forceinline__ void st2(float* p, float a, float b) { *reinterpret_cast<float2*>(p) = make_float2(a, b); }
-__device__ __forceinline__ void st2(__nv_bfloat16* p, float a, float b) { *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(a, b); }
+__device__ __forceinline__ void st2(__nv_bfloat16* p, float a, float b) {
+  *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(a, b);
+}
 __device__ __forceinline__ float sigmoid(float z) { return 1.f / (1.f + __expf(-z)); }
 
 // one CTA of two warpgroups' worth of warps per token: the first half norms the query latent, the second the other one
@@ -223,8 +225,10 @@ int mfb_latent_norm_cache(const void* proj, long long ld_proj, const void* q_nor
   if (T <= 0) return 0;
   if (Q < 1 || R < 1 || ld_proj < Q + R) { mfb_host::set_error("latent_norm_cache: Q=%d R=%d", Q, R); return 1; }
   using bf = __nv_bfloat16;
-  if (f32) hmx::latent_norm_cache_kernel<float><<<T, 256, 0, stream>>>((const float*)proj, ld_proj, (const float*)q_norm, (const float*)kv_norm, eps, slots, (float*)q, (float*)cache, Q, R);
-  else hmx::latent_norm_cache_kernel<bf><<<T, 256, 0, stream>>>((const bf*)proj, ld_proj, (const bf*)q_norm, (const bf*)kv_norm, eps, slots, (bf*)q, (bf*)cache, Q, R);
+  if (f32) hmx::latent_norm_cache_kernel<float><<<T, 256, 0, stream>>>((const float*)proj, ld_proj, (const float*)q_norm,
+      (const float*)kv_norm, eps, slots, (float*)q, (float*)cache, Q, R);
+  else hmx::latent_norm_cache_kernel<bf><<<T, 256, 0, stream>>>((const bf*)proj, ld_proj, (const bf*)q_norm, (const bf*)kv_norm,
+      eps, slots, (bf*)q, (bf*)cache, Q, R);
   return cudaGetLastError() == cudaSuccess ? 0 : 2;
 }
 
@@ -285,8 +289,10 @@ int mfb_talk_mix(const void* o, const float* talk, const void* gate, long long l
   const dim3 grid(T, gy);
   using bf = __nv_bfloat16;
   if (f32) {
-    if (vec) hmx::talk_mix_kernel<float, 2><<<grid, 256, smem, stream>>>((const float*)o, talk, (const float*)gate, ld_g, (float*)y, H, G, DV, in_smem);
-    else hmx::talk_mix_kernel<float, 1><<<grid, 256, smem, stream>>>((const float*)o, talk, (const float*)gate, ld_g, (float*)y, H, G, DV, in_smem);
+    if (vec) hmx::talk_mix_kernel<float, 2><<<grid, 256, smem, stream>>>((const float*)o, talk, (const float*)gate, ld_g,
+        (float*)y, H, G, DV, in_smem);
+    else hmx::talk_mix_kernel<float, 1><<<grid, 256, smem, stream>>>((const float*)o, talk, (const float*)gate, ld_g, (float*)y, H,
+        G, DV, in_smem);
   } else {
     if (vec) hmx::talk_mix_kernel<bf, 2><<<grid, 256, smem, stream>>>((const bf*)o, talk, (const bf*)gate, ld_g, (bf*)y, H, G, DV, in_smem);
     else hmx::talk_mix_kernel<bf, 1><<<grid, 256, smem, stream>>>((const bf*)o, talk, (const bf*)gate, ld_g, (bf*)y, H, G, DV, in_smem);

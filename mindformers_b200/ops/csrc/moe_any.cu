@@ -154,7 +154,8 @@ extern "C" {
 using namespace mfb;
 
 // x [R, 2 F] (gate | up) -> y [R, F]. block_group (with num_blocks) or null; offsets / fill or null: see rows_in_use.
-int mfb_clamped_glu(const void* x, void* y, int R, int F, float limit, float alpha, float shift, const int* block_group, const int* num_blocks,
+int mfb_clamped_glu(const void* x, void* y, int R, int F, float limit, float alpha, float shift, const int* block_group,
+                    const int* num_blocks,
                     const int* offsets, const int* fill, int f32, cudaStream_t stream) {
   if (R <= 0 || F <= 0) return 0;
   const int blocks = (R + many::kBlock - 1) / many::kBlock;
@@ -163,17 +164,22 @@ int mfb_clamped_glu(const void* x, void* y, int R, int F, float limit, float alp
   if (slices > 64) slices = 64;
   dim3 grid(blocks, (unsigned)slices);
   using bf = __nv_bfloat16;
-  if (f32) many::clamped_glu_kernel<float, 1><<<grid, 256, 0, stream>>>((const float*)x, (float*)y, R, F, limit, alpha, shift, block_group, num_blocks, offsets, fill);
-  else if (vec) many::clamped_glu_kernel<bf, 8><<<grid, 256, 0, stream>>>((const bf*)x, (bf*)y, R, F, limit, alpha, shift, block_group, num_blocks, offsets, fill);
-  else many::clamped_glu_kernel<bf, 1><<<grid, 256, 0, stream>>>((const bf*)x, (bf*)y, R, F, limit, alpha, shift, block_group, num_blocks, offsets, fill);
+  if (f32) many::clamped_glu_kernel<float, 1><<<grid, 256, 0, stream>>>((const float*)x, (float*)y, R, F, limit, alpha, shift,
+      block_group, num_blocks, offsets, fill);
+  else if (vec) many::clamped_glu_kernel<bf, 8><<<grid, 256, 0, stream>>>((const bf*)x, (bf*)y, R, F, limit, alpha, shift,
+      block_group, num_blocks, offsets, fill);
+  else many::clamped_glu_kernel<bf, 1><<<grid, 256, 0, stream>>>((const bf*)x, (bf*)y, R, F, limit, alpha, shift, block_group,
+      num_blocks, offsets, fill);
   return cudaGetLastError() == cudaSuccess ? 0 : 2;
 }
 
 int mfb_moe_scatter_any(const void* x, const long long* ids, const int* rank_in_e, const int* write_base, const float* weights,
                         void* rows, int* dest_row, int T, int k, int H, int rows_cap, int f32, cudaStream_t stream) {
   if (T <= 0 || k <= 0) return 0;
-  if (f32) many::scatter_kernel<float><<<T * k, 128, 0, stream>>>((const float*)x, ids, rank_in_e, write_base, weights, (float*)rows, dest_row, k, H, rows_cap);
-  else many::scatter_kernel<__nv_bfloat16><<<T * k, 128, 0, stream>>>((const __nv_bfloat16*)x, ids, rank_in_e, write_base, weights, (__nv_bfloat16*)rows, dest_row, k, H, rows_cap);
+  if (f32) many::scatter_kernel<float><<<T * k, 128, 0, stream>>>((const float*)x, ids, rank_in_e, write_base, weights,
+      (float*)rows, dest_row, k, H, rows_cap);
+  else many::scatter_kernel<__nv_bfloat16><<<T * k, 128, 0, stream>>>((const __nv_bfloat16*)x, ids, rank_in_e, write_base, weights,
+      (__nv_bfloat16*)rows, dest_row, k, H, rows_cap);
   return cudaGetLastError() == cudaSuccess ? 0 : 2;
 }
 
@@ -194,8 +200,10 @@ int mfb_grouped_gemm_any(const void* a, const void* w, void* out, int R, int N, 
     return 1;
   }
   dim3 grid((N + many::kTN - 1) / many::kTN, R / many::kTM);
-  if (f32) many::grouped_gemm_kernel<float><<<grid, 256, 0, stream>>>((const float*)a, (const float*)w, (float*)out, R, N, K, block_group, num_blocks, offsets, fill);
-  else many::grouped_gemm_kernel<__nv_bfloat16><<<grid, 256, 0, stream>>>((const __nv_bfloat16*)a, (const __nv_bfloat16*)w, (__nv_bfloat16*)out, R, N, K, block_group, num_blocks, offsets, fill);
+  if (f32) many::grouped_gemm_kernel<float><<<grid, 256, 0, stream>>>((const float*)a, (const float*)w, (float*)out, R, N, K,
+      block_group, num_blocks, offsets, fill);
+  else many::grouped_gemm_kernel<__nv_bfloat16><<<grid, 256, 0, stream>>>((const __nv_bfloat16*)a, (const __nv_bfloat16*)w,
+      (__nv_bfloat16*)out, R, N, K, block_group, num_blocks, offsets, fill);
   return cudaGetLastError() == cudaSuccess ? 0 : 2;
 }
 

@@ -4,8 +4,9 @@
 // A batch is ragged: sequence b brings the rows cu_q[b] .. cu_q[b + 1] - 1, its last tokens, which are already in the
 // cache; row r sits at position context_lens[b] - (cu_q[b + 1] - r). Keys are visible up to the row's own position, and
 // with `chunk` > 0 only inside the row's chunk of `chunk` positions counted from 0, with `window` > 0 only the row's own and
-// the `window` - 1 before it. With `all_values` a head's weights are applied to the values of every KV head. `sink` [Hq] adds exp(sink_h) to the
-// softmax denominator of head h (no key, no value, not scaled). `softcap` > 0 bounds the scores: softcap * tanh(score / softcap).
+// the `window` - 1 before it. With `all_values` a head's weights are applied to the values of every KV head. `sink` [Hq] adds
+// exp(sink_h) to the softmax denominator of head h (no key, no value, not scaled). `softcap` > 0 bounds the scores: softcap *
+// tanh(score / softcap).
 //
 // One CTA of four warps per (row, query head): a warp takes every fourth key, its lanes split the head dimension; the
 // warps' online softmax states are merged through shared memory in a fixed order. All arithmetic is fp32.
@@ -128,10 +129,10 @@ int launch(const void* q, const void* kc, const void* vc, const int* bt, const i
 extern "C" {
 using namespace mfb;
 
-// q [rows, Hq, D], caches [num_blocks, block_size, Hkv, D | DV], out [rows, Hq, DV] (rows ld_out apart): fp32 (f32 = 1) or bf16. cu_q [B + 1]
-// (device) or null: one row per sequence. chunk <= 0: no chunks; window <= 0: no window; all_values: out [rows, Hq, Hkv, DV];
-// value_cache may be key_cache; sink: [Hq] fp32 or null. softcap > 0: scores become
-// softcap * tanh(score / softcap). Rows of out lie ld_out elements apart; the result is multiplied by out_scale.
+// q [rows, Hq, D], caches [num_blocks, block_size, Hkv, D | DV], out [rows, Hq, DV] (rows ld_out apart): fp32 (f32 = 1) or bf16.
+// cu_q [B + 1] (device) or null: one row per sequence. chunk <= 0: no chunks; window <= 0: no window; all_values: out [rows, Hq,
+// Hkv, DV]; value_cache may be key_cache; sink: [Hq] fp32 or null. softcap > 0: scores become softcap * tanh(score / softcap).
+// Rows of out lie ld_out elements apart; the result is multiplied by out_scale.
 int mfb_paged_attention_any(const void* q, const void* key_cache, const void* value_cache, const int* block_tables,
                             const int* context_lens, const int* cu_q, const float* sink, void* out, int rows, int B, int Hq,
                             int Hkv, int D, int DV, int block_size, int max_blocks, int chunk, int window, int all_values, float scale,
@@ -146,7 +147,8 @@ int mfb_paged_attention_any(const void* q, const void* key_cache, const void* va
   return f32 ? paa::launch<float>(q, key_cache, value_cache, block_tables, context_lens, cu_q, sink, out, rows, B, Hq, Hkv, D,
                                   DV, block_size, max_blocks, chunk, window, all_values, scale, softcap, ld_out, out_scale, stream)
              : paa::launch<__nv_bfloat16>(q, key_cache, value_cache, block_tables, context_lens, cu_q, sink, out, rows, B, Hq,
-                                          Hkv, D, DV, block_size, max_blocks, chunk, window, all_values, scale, softcap, ld_out, out_scale, stream);
+                                          Hkv, D, DV, block_size, max_blocks, chunk, window, all_values, scale, softcap, ld_out,
+                                          out_scale, stream);
 }
 
 }  // extern "C"

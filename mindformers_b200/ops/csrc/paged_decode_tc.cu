@@ -413,17 +413,18 @@ int mfb_paged_decode_tc_splits(int B, int Hkv, int max_len) {
 }
 
 // q [rows, Hq, D] bf16, caches [num_blocks, block_size, Hkv, D | DV] bf16, out [rows, Hq, DV] bf16; scratch as for
-// mfb_paged_decode_attention (mfb_paged_decode_scratch_bytes(B, Hq, DV, splits); all_values: Hq Hkv rows of results, no sink). cu_q null: row b belongs to sequence b
-// (rows == B); else [B + 1] row boundaries of a ragged batch, of which only the sequences with one row are computed and
-// written. chunk > 0: keys of the query's own chunk of positions only; window > 0: the last `window` keys only. sink: [Hq] fp32 or null, adds exp(sink) to the
-// softmax denominator. softcap > 0: scores become softcap * tanh(score / softcap). Rows of out lie ld_out elements apart; the
-// result is multiplied by out_scale.
+// mfb_paged_decode_attention (mfb_paged_decode_scratch_bytes(B, Hq, DV, splits); all_values: Hq Hkv rows of results, no sink).
+// cu_q null: row b belongs to sequence b (rows == B); else [B + 1] row boundaries of a ragged batch, of which only the sequences
+// with one row are computed and written. chunk > 0: keys of the query's own chunk of positions only; window > 0: the last
+// `window` keys only. sink: [Hq] fp32 or null, adds exp(sink) to the softmax denominator. softcap > 0: scores become softcap *
+// tanh(score / softcap). Rows of out lie ld_out elements apart; the result is multiplied by out_scale.
 int mfb_paged_decode_attention_tc_ex(const void* q, const void* key_cache, const void* value_cache, const int* block_tables,
                                      const int* context_lens, const int* cu_q, const float* sink, void* out, void* scratch,
                                      int splits, int rows, int B, int Hq, int Hkv, int D, int DV, int num_blocks,
                                      int block_size, int max_blocks, int chunk, int window, int all_values, float scale,
                                      float softcap, long long ld_out, float out_scale, int* status, cudaStream_t stream) {
-  if (!mfb_paged_decode_tc_supported_ex(Hq, Hkv, D, DV, block_size) || splits < 1 || num_blocks < 1 || (!cu_q && rows != B) || (all_values && sink)) {
+  if (!mfb_paged_decode_tc_supported_ex(Hq, Hkv, D, DV, block_size) || splits < 1 || num_blocks < 1 || (!cu_q && rows != B)
+      || (all_values && sink)) {
     mfb_host::set_error("paged_decode_tc: unsupported Hq=%d Hkv=%d D=%d DV=%d block_size=%d splits=%d", Hq, Hkv, D, DV,
                         block_size, splits);
     return 1;
@@ -439,7 +440,8 @@ int mfb_paged_decode_attention_tc_ex(const void* q, const void* key_cache, const
   pdt::Args a;
   a.block_tables = block_tables; a.context_lens = context_lens; a.cu_q = cu_q; a.max_blocks = max_blocks;
   a.block_size = block_size; a.num_q_heads = Hq; a.num_kv_heads = Hkv; a.group = Hq / Hkv; a.splits = splits;
-  a.D = D; a.DV = DV; a.chunk = chunk; a.window = window; a.vheads = all_values ? Hkv : 1; a.head_blocks = (a.group + pdt::kHeads - 1) / pdt::kHeads;
+  a.D = D; a.DV = DV; a.chunk = chunk; a.window = window; a.vheads = all_values ? Hkv : 1;
+  a.head_blocks = (a.group + pdt::kHeads - 1) / pdt::kHeads;
   a.scale_log2 = scale * 1.4426950408889634f;
   a.cap_log2 = softcap > 0.f ? softcap * 1.4426950408889634f : 0.f;
   a.cap_scale = softcap > 0.f ? scale / softcap : 0.f;
@@ -457,7 +459,8 @@ int mfb_paged_decode_attention_tc_ex(const void* q, const void* key_cache, const
   dim3 grid(splits, Hkv * a.head_blocks * a.vheads, B);
   pdt::paged_decode_tc_kernel<<<grid, pdt::kThreads, pdt::kSmem, stream>>>(tQ, tK, tV, a);
   if (cudaGetLastError() != cudaSuccess) { mfb_host::set_error("paged_decode_tc: launch failed"); return 11; }
-  return mfb_paged_combine_ex(a.part_acc, a.part_ml, out, splits, B * Hq * a.vheads, DV, Hq * a.vheads, cu_q, sink, ld_out, out_scale, stream);
+  return mfb_paged_combine_ex(a.part_acc, a.part_ml, out, splits, B * Hq * a.vheads, DV, Hq * a.vheads, cu_q, sink, ld_out,
+      out_scale, stream);
 }
 
 // q [B, Hq, 128], caches [num_blocks, block_size, Hkv, 128], out [B, Hq, 128]: one row per sequence, no chunks, no sink.

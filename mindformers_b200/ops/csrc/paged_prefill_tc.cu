@@ -863,7 +863,8 @@ int mfb_paged_prefill_tc_supported(int Hq, int Hkv, int D, int DV, int block_siz
 int mfb_paged_prefill_tc(const void* q, const void* key_cache, const void* value_cache, const int* work, int n_work, int persistent,
                          const int* block_tables, const float* sink, void* out, int T,
                          int Hq, int Hkv, int D, int DV, int num_blocks, int block_size, int max_blocks, int chunk, int window,
-                         int all_values, long long ld_k, long long ld_v, float scale, float softcap, long long ld_out, float out_scale, int* status, cudaStream_t stream) {
+                         int all_values, long long ld_k, long long ld_v, float scale, float softcap, long long ld_out,
+                         float out_scale, int* status, cudaStream_t stream) {
   if (!mfb_paged_prefill_tc_supported(Hq, Hkv, D, DV, block_size) || num_blocks < 1 || T < 1) {
     mfb_host::set_error("paged_prefill_tc: unsupported Hq=%d Hkv=%d D=%d DV=%d block_size=%d", Hq, Hkv, D, DV, block_size);
     return 1;
@@ -885,7 +886,8 @@ int mfb_paged_prefill_tc(const void* q, const void* key_cache, const void* value
   if ((rc = mfb_host::make_tmap_2d(&tV, value_cache, 2, BF, rows, (uint64_t)Hkv * DV, (uint64_t)ld_v, block_size, 64))) return 40 + rc;
   if ((rc = ppt::make_q_map(&tQ, q, T, Hq, D))) return 20 + rc;
   ppt::Args a;
-  a.work = reinterpret_cast<const int4*>(work); a.vheads = all_values ? Hkv : 1; a.n_items = n_work * Hq * a.vheads; a.block_tables = block_tables; a.sink = sink;
+  a.work = reinterpret_cast<const int4*>(work); a.vheads = all_values ? Hkv : 1; a.n_items = n_work * Hq * a.vheads;
+  a.block_tables = block_tables; a.sink = sink;
   a.out = reinterpret_cast<__nv_bfloat16*>(out);
   a.num_q_heads = Hq; a.group = Hq / Hkv; a.D = D; a.DV = DV; a.block_size = block_size; a.max_blocks = max_blocks;
   a.chunk = chunk; a.window = window; a.scale_log2 = scale * 1.4426950408889634f; a.status = status;

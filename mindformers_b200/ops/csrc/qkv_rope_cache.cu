@@ -1,5 +1,6 @@
 // Between the QKV projection and attention over a paged cache, in one kernel (sm_100a, bf16 or fp32): projection bias,
-// per-head RMS norm of q and k (with or without a weight) and of v (without), rotary embedding of q and k, and the write of k and v into the paged cache.
+// per-head RMS norm of q and k (with or without a weight) and of v (without), rotary embedding of q and k, and the write of k and
+// v into the paged cache.
 //
 //   qkv [T, H * D + G * D + G * DV] (row pitch given)  ->  q_out [T, H, D]
 //                                                          key_cache [slots, G, D], value_cache [slots, G, DV]
@@ -303,7 +304,8 @@ bool al(const void* p, int n) { return (reinterpret_cast<uintptr_t>(p) & (n - 1)
 extern "C" {
 using namespace mfb;
 
-// f32 = 1: all typed tensors are fp32, else bf16. unit: bit 0: q and k, bit 1: v are normed without a weight (DV up to 512). freqs: [rot / 2] fp32; cos and sin are multiplied by `amplitude`.
+// f32 = 1: all typed tensors are fp32, else bf16. unit: bit 0: q and k, bit 1: v are normed without a weight (DV up to 512).
+// freqs: [rot / 2] fp32; cos and sin are multiplied by `amplitude`.
 int mfb_qkv_rope_cache(const void* qkv, long long ld_qkv, const void* bias, const void* q_norm, const void* k_norm, float eps,
                        const float* freqs, float amplitude, int rot, int interleaved, const long long* positions,
                        const int* slots, void* q_out, void* key_cache, void* value_cache, int T, int H, int G, int D, int DV,

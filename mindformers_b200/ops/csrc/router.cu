@@ -63,7 +63,8 @@ __device__ __forceinline__ void router_scores(const float* __restrict__ row, con
 
 template <int PER>
 __global__ void __launch_bounds__(kRouterWarps * 32)
-router_fwd_kernel(const float* __restrict__ logits, const float* __restrict__ logit_bias, const float* __restrict__ bias, float* __restrict__ probs,
+router_fwd_kernel(const float* __restrict__ logits, const float* __restrict__ logit_bias, const float* __restrict__ bias,
+                  float* __restrict__ probs,
                   long long* __restrict__ ids, float* __restrict__ scores_out, float* __restrict__ counts,
                   RouterArgs a) {
   const int lane = threadIdx.x & 31;

@@ -500,7 +500,8 @@ def swiglu(x: torch.Tensor) -> torch.Tensor:
 # =================================================================================================
 def clamped_glu(x: torch.Tensor, limit: float, alpha: float, plan=None, shift: float = 1.0) -> torch.Tensor:
     """``g * sigmoid(alpha g) * (u + shift)`` of ``x [R, 2F]`` = gate | up, ``g = min(gate, limit)``, ``u = clamp(up, -limit,
-    limit)``, computed in fp32 (no limit, ``alpha`` 1 and ``shift`` 0: SwiGLU). ``plan``: a permutation plan whose unused rows are skipped (left undefined). No gradients."""
+    limit)``, computed in fp32 (no limit, ``alpha`` 1 and ``shift`` 0: SwiGLU). ``plan``: a permutation plan whose unused rows are
+    skipped (left undefined). No gradients."""
     R, F_ = x.shape[0], x.shape[1] // 2
     if not _on_gpu(x):
         g, u = x.float().chunk(2, dim=-1)
@@ -512,7 +513,8 @@ def clamped_glu(x: torch.Tensor, limit: float, alpha: float, plan=None, shift: f
         raise TypeError("clamped_glu needs a contiguous bfloat16 or float32 matrix")
     y = torch.empty((R, F_), dtype=x.dtype, device=x.device)
     p = [None] * 4 if plan is None else [plan.block_group, plan.num_blocks, plan.group_offsets, getattr(plan, "seg_fill", None)]
-    rc = _lib.get_lib().mfb_clamped_glu(x.data_ptr(), y.data_ptr(), R, F_, float(limit), float(alpha), float(shift), *(_lib.ptr(t) for t in p),
+    rc = _lib.get_lib().mfb_clamped_glu(x.data_ptr(), y.data_ptr(), R, F_, float(limit), float(alpha), float(shift),
+                                         *(_lib.ptr(t) for t in p),
                                         int(x.dtype == torch.float32), _lib.stream_ptr())
     _lib.check(rc, "mfb_clamped_glu")
     _lib.count_launch()

@@ -1,9 +1,9 @@
 """Recurrent mixers over ragged batches: the gated delta rule (short convolutions, unit keys, decays, the recurrence, its norm
 and gate) and the matrix memory (capped log gates, running maximum, memory and normaliser, norm and gate).
 
-``delta_rule`` and ``matrix_memory`` have two bodies like the ops of ``functional.py``: the sm_100a kernels (``csrc/delta_rule.cu``, ``csrc/matrix_memory.cu``),
-always taken for CUDA tensors (bf16 or fp32 activations; state and recurrence are fp32), and a plain PyTorch body for CPU
-tensors. They are inference ops: they advance the state in place and have no gradients.
+``delta_rule`` and ``matrix_memory`` have two bodies like the ops of ``functional.py``: the sm_100a kernels
+(``csrc/delta_rule.cu``, ``csrc/matrix_memory.cu``), always taken for CUDA tensors (bf16 or fp32 activations; state and
+recurrence are fp32), and a plain PyTorch body for CPU tensors. They are inference ops: they advance the state in place and have no gradients.
 """
 from __future__ import annotations
 

@@ -296,8 +296,8 @@ def qkv_rope_cache(qkv: torch.Tensor, bias: Optional[torch.Tensor], q_norm: Opti
                    positions: torch.Tensor, slots: torch.Tensor, key_cache: torch.Tensor, value_cache: torch.Tensor,
                    heads: int, kv_heads: int, dim: int, v_dim: int, unit_qk: bool = False, unit_v: bool = False) -> torch.Tensor:
     """Everything between the QKV projection and attention over the paged cache: projection bias, per-head RMS norm of q
-    and k (``None``: no norm; ``unit_qk``: a norm without a weight) and of v (``unit_v``, without a weight), rotation of the first ``2 * len(freqs)`` dimensions by ``position * freqs`` (cos and sin
-    times ``amplitude``) and the write of k and v into the cache rows ``slots`` (negative: not written).
+    and k (``None``: no norm; ``unit_qk``: a norm without a weight) and of v (``unit_v``, without a weight), rotation of the
+    first ``2 * len(freqs)`` dimensions by ``position * freqs`` (cos and sin times ``amplitude``) and the write of k and v into the cache rows ``slots`` (negative: not written).
 
     ``qkv [T, heads * dim + kv_heads * (dim + v_dim)]`` → q ``[T, heads, dim]``."""
     T, dtype, rot = qkv.shape[0], qkv.dtype, 2 * freqs.numel()
@@ -323,7 +323,8 @@ def qkv_rope_cache(qkv: torch.Tensor, bias: Optional[torch.Tensor], q_norm: Opti
     _check_dtype(dtype)
     _typed(bias, q_norm, k_norm, key_cache, value_cache, dtype=dtype)
     if qkv.stride(1) != 1 or qkv.shape[1] != nq + nk + kv_heads * v_dim or positions.dtype != torch.int64 \
-            or slots.dtype != torch.int32 or (unit_qk and (q_norm is not None or k_norm is not None)) or freqs.dtype != torch.float32 or positions.numel() != T or slots.numel() != T:
+            or slots.dtype != torch.int32 or (unit_qk and (q_norm is not None or k_norm is not None)) \
+            or freqs.dtype != torch.float32 or positions.numel() != T or slots.numel() != T:
         raise TypeError("qkv_rope_cache: unexpected shapes or dtypes")
     q = torch.empty((T, heads, dim), dtype=dtype, device=qkv.device)
     rc = _lib.get_lib().mfb_qkv_rope_cache(

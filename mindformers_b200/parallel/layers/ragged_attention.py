@@ -6,7 +6,8 @@ softmax sink (``attention_sink``), soft-capped scores (``attention_softcap``), n
 sliding window (``attention_window``), norms without weights (``qk_unit_norm``, ``value_unit_norm``), weights mixed over heads
 (``attention_talk``), an output gate (``attention_output_gate``), projection biases folded into the following kernel. Parameter
 names are those of ``SelfAttention`` plus ``sink [heads]`` and ``talk [heads, heads]`` (fp32). ``RaggedLatentAttention`` caches
-one latent per token instead of keys and values. ``RaggedAttentionCore`` is what lies between the projections, for mixers that share them with something else. One kernel applies bias, q / k norm and rotation and writes the cache
+one latent per token instead of keys and values. ``RaggedAttentionCore`` is what lies between the projections, for mixers that
+share them with something else. One kernel applies bias, q / k norm and rotation and writes the cache
 (``ops/stream.py::qkv_rope_cache``); one call attends for all sequences of the batch
 (``inference/ragged_attention.py``).
 """
