@@ -48,6 +48,54 @@ latent_norm_cache_kernel(const T* __restrict__ proj, long long ld_proj, const T*
   for (int i = tid; i < n; i += 128) st(dst + i, ld(src + i) * rstd * ld(w + i));
 }
 
+// bf16, eight columns per access, a warp per token and latent, which it keeps in registers: latents of up to 32 * 8 * kHold
+constexpr int kHold = 8;
+__global__ void __launch_bounds__(256)
+latent_norm_cache_vec_kernel(const __nv_bfloat16* __restrict__ proj, long long ld_proj, const __nv_bfloat16* __restrict__ q_norm,
+                             const __nv_bfloat16* __restrict__ kv_norm, float eps, const int* __restrict__ slots,
+                             __nv_bfloat16* __restrict__ q, __nv_bfloat16* __restrict__ cache, int T_rows, int Q, int R) {
+  const int unit = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (unit >= 2 * T_rows) return;
+  const long long t = unit >> 1;
+  const bool kv = unit & 1;
+  const int n = kv ? R : Q, slot = slots[t];
+  if (kv && slot < 0) return;
+  const __nv_bfloat16* src = proj + t * ld_proj + (kv ? Q : 0);
+  const __nv_bfloat16* w = kv ? kv_norm : q_norm;
+  uint4 x[kHold];
+#pragma unroll
+  for (int i = 0; i < kHold; ++i) {
+    const int c = (i * 32 + lane) * 8;
+    x[i] = c < n ? *reinterpret_cast<const uint4*>(src + c) : make_uint4(0u, 0u, 0u, 0u);
+  }
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < kHold; ++i) {
+    const __nv_bfloat162* v = reinterpret_cast<const __nv_bfloat162*>(&x[i]);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const float2 f = __bfloat1622float2(v[e]);
+      ss = fmaf(f.x, f.x, fmaf(f.y, f.y, ss));
+    }
+  }
+  const float rstd = 1.f / sqrtf(warp_sum(ss) / n + eps);
+  __nv_bfloat16* dst = kv ? cache + (long long)slot * R : q + t * Q;
+#pragma unroll
+  for (int i = 0; i < kHold; ++i) {
+    const int c = (i * 32 + lane) * 8;
+    if (c >= n) break;
+    const uint4 wu = *reinterpret_cast<const uint4*>(w + c);
+    const __nv_bfloat162* wv = reinterpret_cast<const __nv_bfloat162*>(&wu);
+    __nv_bfloat162* v = reinterpret_cast<__nv_bfloat162*>(&x[i]);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const float2 f = __bfloat1622float2(v[e]), g = __bfloat1622float2(wv[e]);
+      v[e] = __floats2bfloat162_rn(f.x * rstd * g.x, f.y * rstd * g.y);
+    }
+    *reinterpret_cast<uint4*>(dst + c) = x[i];
+  }
+}
+
 template <typename T, int VEC>
 __global__ void __launch_bounds__(256)
 gate_heads_kernel(T* __restrict__ x, long long ld_x, const T* __restrict__ gate, long long ld_g, long long T_rows, int n, int per) {
@@ -225,6 +273,13 @@ int mfb_latent_norm_cache(const void* proj, long long ld_proj, const void* q_nor
   if (T <= 0) return 0;
   if (Q < 1 || R < 1 || ld_proj < Q + R) { mfb_host::set_error("latent_norm_cache: Q=%d R=%d", Q, R); return 1; }
   using bf = __nv_bfloat16;
+  constexpr int most = 32 * 8 * hmx::kHold;
+  if (!f32 && Q % 8 == 0 && R % 8 == 0 && ld_proj % 8 == 0 && Q <= most && R <= most && hmx::al(proj, 16) && hmx::al(q_norm, 16)
+      && hmx::al(kv_norm, 16) && hmx::al(q, 16) && hmx::al(cache, 16)) {
+    hmx::latent_norm_cache_vec_kernel<<<(int)(((long long)T * 2 + 7) / 8), 256, 0, stream>>>(
+        (const bf*)proj, ld_proj, (const bf*)q_norm, (const bf*)kv_norm, eps, slots, (bf*)q, (bf*)cache, T, Q, R);
+    return cudaGetLastError() == cudaSuccess ? 0 : 2;
+  }
   if (f32) hmx::latent_norm_cache_kernel<float><<<T, 256, 0, stream>>>((const float*)proj, ld_proj, (const float*)q_norm,
       (const float*)kv_norm, eps, slots, (float*)q, (float*)cache, Q, R);
   else hmx::latent_norm_cache_kernel<bf><<<T, 256, 0, stream>>>((const bf*)proj, ld_proj, (const bf*)q_norm, (const bf*)kv_norm,

@@ -139,10 +139,10 @@ def test_unit_norms_and_cache_write(dtype, H, G, D, DV):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("Q,R", [(64, 128), (33, 7), (1536, 512)])
-def test_latent_norm_and_cache_write(dtype, Q, R):
+@pytest.mark.parametrize("Q,R,more", [(64, 128, 9), (33, 7, 9), (1536, 512, 8), (264, 72, 16), (8, 2048, 0), (2056, 8, 0)])
+def test_latent_norm_and_cache_write(dtype, Q, R, more):
     T = 4
-    x, qn, kn = rand(T, Q + R + 9, seed=1, dtype=dtype), rand(Q, seed=2, dtype=dtype) + 1, rand(R, seed=3, dtype=dtype) + 1
+    x, qn, kn = rand(T, Q + R + more, seed=1, dtype=dtype), rand(Q, seed=2, dtype=dtype) + 1, rand(R, seed=3, dtype=dtype) + 1
     cache = torch.zeros(6, 1, 1, R, dtype=dtype, device=DEV)
     slots = torch.tensor([5, 0, -1, 2], dtype=torch.int32, device=DEV)
     q = stream.latent_norm_cache(x.to(DEV)[:, :Q + R], qn.to(DEV), kn.to(DEV), 1e-3, slots, cache)
