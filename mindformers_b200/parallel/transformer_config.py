@@ -134,7 +134,7 @@ class TransformerConfig(ModelParallelConfig):
     layer_sharing: Optional[List[int]] = None
     norm_placement: str = "input"           # "input": pre-norm; "output": x + scale * norm(sublayer(x)), fp32 stream;
                                             # "both": x + norm(sublayer(norm(x))), fp32 stream
-    layer_loop: Optional[tuple] = None      # (start, stop, times): these layers run so many times in a row with the same
+    layer_loop: Optional[tuple] = None      # (start, stop, times): these layers are repeated, all passes on one set of
                                             # weights; before pass t a learned vector (row t) is added to the stream
     token_shift: bool = False               # norm_placement "both": a mixer reads h + (h of the token before - h) * mu
     embedding_scale: float = 1.0            # factor of the embedding rows (fp32 streams)

@@ -4,7 +4,7 @@
 
 Steps are JSON objects, one per line of standard input:
 
-    {"step": 0, "entries": [{"id": "a", "tokens": [5, 17, 3], "want": [0, 2]}], "end": []}
+    {"step": 0, "entries": [{"id": "first", "tokens": [12, 7, 40, 9], "want": [1, 3]}], "end": []}
 
 ``entries`` names, per request, its next tokens and the places among them whose logits are wanted; ``end`` the requests
 that are finished after the step. The entries of a step run as one batch on the engine's slots and cache pool
