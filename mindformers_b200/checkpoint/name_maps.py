@@ -123,6 +123,7 @@ _MEFESUN_TOP = {"embed": "embedding.word_embeddings.weight", "final.norm": "deco
                 "final.norm.b": "decoder.final_layernorm.bias"}
 _GAVATAR_TOP = {"embed": "embedding.word_embeddings.weight", "final.norm": "decoder.final_layernorm.weight",
                 "head": "output_layer.weight", "loop.step": "decoder.loop_step"}
+_TOGALORN_TOP = dict(_GAVATAR_TOP, **{"loop.in": "decoder.loop_in"})
 _LIST_LAYER = re.compile(r"^l(\d+)\.(.+)$")
 
 
@@ -267,7 +268,7 @@ def framework_to_kukupel(sd: Dict[str, torch.Tensor], config) -> Dict[str, torch
     return out
 
 
-FAMILIES = ("mefesun", "kukupel", "gavatar", "llama", "qwen2", "qwen2_5", "qwen2_moe", "qwen3", "qwen3_moe", "deepseek_v2", "deepseek_v3",
+FAMILIES = ("mefesun", "kukupel", "gavatar", "togalorn", "llama", "qwen2", "qwen2_5", "qwen2_moe", "qwen3", "qwen3_moe", "deepseek_v2", "deepseek_v3",
             "deepseekv3", "mixtral", "telechat", "glm")
 
 
@@ -597,8 +598,106 @@ def framework_to_gavatar(sd: Dict[str, torch.Tensor], config) -> Dict[str, torch
     return out
 
 
+# Togalorn checkpoints: tensors that map one to one (those of the second table transposed), per mixer
+_TOGALORN = {
+    "norm1": "input_layernorm.weight", "mlp.router": "mlp.router.weight", "mlp.correction": "mlp.router.expert_bias",
+    "mlp.shared.down": "mlp.shared_experts.linear_fc2.weight", "mix.o": "self_attention.linear_proj.weight",
+}
+_TOGALORN_TURNED = {"canon1": "input_conv", "mix.conv": "self_attention.conv"}
+_TOGALORN_MIXER = {
+    "latent": {"mix.dq.norm": "self_attention.q_latent_norm.weight", "mix.dkv.norm": "self_attention.kv_latent_norm.weight",
+               "mix.uq": "self_attention.linear_q_up.weight"},
+    "state_space": {"mix.in": "self_attention.linear_in.weight", "mix.conv.b": "self_attention.conv_bias",
+                    "mix.dt_bias": "self_attention.dt_bias", "mix.A_log": "self_attention.a_log", "mix.D": "self_attention.skip",
+                    "mix.norm": "self_attention.norm"},
+}
+
+
+def _togalorn_layout(c):
+    """Of a layer with configuration ``c``: the tensors that map one to one, and ``{parameter: [(tensor, rows)]}`` of the stacked
+    ones."""
+    stacked = {}
+    if c.mixer == "latent":
+        stacked["self_attention.linear_in.weight"] = [("mix.dq", c.q_lora_rank), ("mix.dkv", c.kv_lora_rank + c.rotary_dim),
+                                                      ("mix.g", c.num_attention_heads * c.v_channels)]
+    if c.num_moe_experts and c.moe_shared_expert_intermediate_size:
+        ff = c.moe_shared_expert_intermediate_size
+        stacked["mlp.shared_experts.linear_fc1.weight"] = [("mlp.shared.gate", ff), ("mlp.shared.up", ff)]
+    return dict(_TOGALORN, **_TOGALORN_MIXER[c.mixer]), stacked
+
+
+def togalorn_to_framework(sd: Dict[str, torch.Tensor], config) -> Dict[str, torch.Tensor]:
+    """Togalorn tensors of any number of whole layers → fused framework parameters."""
+    from ..parallel.layers.ragged_attention import expand_kv_up
+    out: Dict[str, torch.Tensor] = {}
+    layers: Dict[int, Dict[str, torch.Tensor]] = {}
+    for name, t in sd.items():
+        m = _LIST_LAYER.match(name)
+        if m:
+            layers.setdefault(int(m[1]), {})[m[2]] = t
+        else:
+            out[_TOGALORN_TOP.get(name, name)] = t
+    for i, own in layers.items():
+        p, left, c = f"decoder.layers.{i}.", set(own), config.for_layer(i)
+        plain, stacked = _togalorn_layout(c)
+
+        def take(name):
+            left.discard(name)
+            if name not in own:
+                raise KeyError(f"l{i}.{name} is missing")
+            return own[name]
+        for to, rows in stacked.items():
+            if any(n in own for n, _ in rows):
+                out[p + to] = torch.cat([take(n) for n, _ in rows], dim=0)
+        if c.mixer == "latent" and "mix.uk" in own:
+            out[p + "self_attention.linear_kv_up.weight"] = expand_kv_up(take("mix.uk"), take("mix.uv"), c.num_attention_heads,
+                                                                         c.kv_channels, c.rotary_dim)
+        out.update((p + n, t) for n, t in _stack_experts(own, take).items())
+        if "mlp.router" in own and "mlp.correction" not in own:          # a buffer: no parameter would be missed
+            raise KeyError(f"l{i}.mlp.correction is missing")
+        for n in sorted(left):
+            if n in _TOGALORN_TURNED:
+                out[p + _TOGALORN_TURNED[n]] = own[n].t().contiguous()
+            elif n in plain:
+                out[p + plain[n]] = own[n]
+            else:
+                raise KeyError(f"l{i}.{n}: no counterpart in the model")
+    return out
+
+
+def framework_to_togalorn(sd: Dict[str, torch.Tensor], config) -> Dict[str, torch.Tensor]:
+    """Fused framework names → Togalorn tensors."""
+    from ..parallel.layers.ragged_attention import split_kv_up
+    top = {v: k for k, v in _TOGALORN_TOP.items()}
+    turned = {v: k for k, v in _TOGALORN_TURNED.items()}
+    out: Dict[str, torch.Tensor] = {}
+    for name, t in sd.items():
+        m = re.match(r"^decoder\.layers\.(\d+)\.(.+)$", name)
+        if not m:
+            out[top.get(name, name)] = t
+            continue
+        l, rest, c = f"l{m[1]}.", m[2], config.for_layer(int(m[1]))
+        plain, stacked = _togalorn_layout(c)
+        back = {v: k for k, v in plain.items()}
+        if rest in back:
+            out[l + back[rest]] = t
+        elif rest in turned:
+            out[l + turned[rest]] = t.t().contiguous()
+        elif rest in stacked:
+            rows = stacked[rest]
+            out.update((l + n, piece.contiguous()) for (n, _), piece in zip(rows, torch.split(t, [r for _, r in rows], dim=0)))
+        elif rest == "self_attention.linear_kv_up.weight":
+            out[l + "mix.uk"], out[l + "mix.uv"] = split_kv_up(t, c.num_attention_heads, c.kv_channels, c.rotary_dim, c.kv_lora_rank)
+        elif rest.startswith("mlp.experts.weight"):
+            out.update((l + n, piece) for n, piece in _unstack_experts(rest, t).items())
+        else:
+            raise KeyError(f"{name}: no counterpart in the checkpoint format")
+    return out
+
+
 # families whose tensors are renamed and fused layer by layer, by the layer's own configuration
-_BY_LAYER = {"kukupel": (kukupel_to_framework, framework_to_kukupel), "gavatar": (gavatar_to_framework, framework_to_gavatar)}
+_BY_LAYER = {"kukupel": (kukupel_to_framework, framework_to_kukupel), "gavatar": (gavatar_to_framework, framework_to_gavatar),
+             "togalorn": (togalorn_to_framework, framework_to_togalorn)}
 
 
 def hf_to_framework(hf_sd: Dict[str, torch.Tensor], config, family: str = "llama", dtype=None,

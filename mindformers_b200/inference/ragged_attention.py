@@ -270,42 +270,43 @@ def _expansion(cache, window: int):
 
 
 def _absorbed(q, cache, layer, w_uk, w_uv, scale, window, sink):
-    """Queries through the key factor, attention over the latents themselves, results through the value factor: ``[T, heads *
-    v_dim]``."""
+    """Queries through the key factor, attention over the cached rows themselves, results through the value factor, which may act
+    on fewer columns: ``[T, heads * v_dim]``."""
     T, H = q.shape[0], q.shape[1]
-    R, DV = w_uk.shape[2], w_uv.shape[1]
+    R, DV, RV = w_uk.shape[2], w_uv.shape[1], w_uv.shape[2]
     q_lat = torch.empty((T, H, R), dtype=q.dtype, device=q.device)
     torch.bmm(q.transpose(0, 1), w_uk, out=q_lat.transpose(0, 1))
     lib = _lib.get_lib() if q.is_cuda else None
     if lib is not None and q.dtype == torch.bfloat16 and not cache.is_prefill \
-            and lib.mfb_latent_decode_supported(R, cache.block_size):
-        o_lat = torch.empty_like(q_lat)
+            and lib.mfb_latent_decode_supported(R, RV, cache.block_size):
+        o_lat = torch.empty((T, H, RV), dtype=q.dtype, device=q.device)
         B, max_blocks = cache.block_tables.shape
         reach = max_blocks * cache.block_size if window <= 0 else min(max_blocks * cache.block_size, window + 128)
         splits = lib.mfb_latent_decode_splits(B, H, reach)
-        scratch = _scratch(cache, "_latent_scratch", lib.mfb_latent_decode_scratch_bytes(B, H, R, splits), q.device)
+        scratch = _scratch(cache, "_latent_scratch", lib.mfb_latent_decode_scratch_bytes(B, H, RV, splits), q.device)
         kc = cache.key_cache[layer]
         rc = lib.mfb_latent_decode(q_lat.data_ptr(), kc.data_ptr(), cache.block_tables.data_ptr(), cache.context_lens.data_ptr(),
-                                   _lib.ptr(sink), o_lat.data_ptr(), scratch.data_ptr(), splits, B, H, R, kc.shape[0],
+                                   _lib.ptr(sink), o_lat.data_ptr(), scratch.data_ptr(), splits, B, H, R, RV, kc.shape[0],
                                    cache.block_size, max_blocks, int(window), float(scale),
                                    _lib.status_word(q.device).data_ptr(), _lib.stream_ptr())
         _lib.check(rc, "mfb_latent_decode")
         _lib.count_launch(2)
     else:
-        o_lat = ragged_attention(q_lat, cache, layer, scale, sink=sink, window=window).view(T, H, R)
+        o_lat = ragged_attention(q_lat, cache, layer, scale, sink=sink, window=window).view(T, H, R)[:, :, :RV]
     out = torch.empty((T, H, DV), dtype=q.dtype, device=q.device)
     torch.bmm(o_lat.transpose(0, 1), w_uv.transpose(1, 2), out=out.transpose(0, 1))
     return out.view(T, H * DV)
 
 
 def latent_attention(q: torch.Tensor, cache, layer: int, w_kv: torch.Tensor, v_dim: int, scale: float, window: int = 0,
-                     sink: Optional[torch.Tensor] = None) -> torch.Tensor:
+                     sink: Optional[torch.Tensor] = None, v_rank: Optional[int] = None) -> torch.Tensor:
     """q ``[T, heads, dim]`` against cached latents ``[.., 1, rank]``, of which the first ``heads * dim`` rows of ``w_kv [heads *
-    (dim + v_dim), rank]`` make the keys and the others the values → ``[T, heads * v_dim]``. Decoded rows attend over the latents
-    (the factors are absorbed into query and result); portions expand the keys and values that they see, once per call."""
+    (dim + v_dim), rank]`` make the keys and the others the values (of the first ``v_rank`` columns alone, where the cached rows
+    also hold a key part) → ``[T, heads * v_dim]``. Decoded rows attend over the latents (the factors are absorbed into query and
+    result); portions expand the keys and values that they see, once per call."""
     T, H, D = q.shape
     R = w_kv.shape[1]
-    w_uk, w_uv = w_kv[:H * D].view(H, D, R), w_kv[H * D:].view(H, v_dim, R)
+    w_uk, w_uv = w_kv[:H * D].view(H, D, R), w_kv[H * D:].view(H, v_dim, R)[:, :, :v_rank]
     lib = _lib.get_lib() if q.is_cuda else None
     expand = lib is not None and q.dtype == torch.bfloat16 and cache.is_prefill and cache.n_long_rows \
         and lib.mfb_paged_prefill_tc_supported(H, H, D, v_dim, cache.block_size)

@@ -5,7 +5,8 @@ from .families import (ChatGLM2ForConditionalGeneration, DeepseekV2Config, Deeps
                        GavatarConfig, GavatarForCausalLM, KukupelConfig, KukupelForCausalLM, LlamaForCausalLM, MefesunConfig,
                        MefesunForCausalLM,
                        MixtralConfig, MixtralForCausalLM, Qwen2Config, Qwen2ForCausalLM, Qwen3Config,
-                       Qwen3ForCausalLM, Qwen3MoeConfig, Qwen3MoeForCausalLM, TelechatConfig, TelechatForCausalLM)
+                       Qwen3ForCausalLM, Qwen3MoeConfig, Qwen3MoeForCausalLM, TelechatConfig, TelechatForCausalLM,
+                       TogalornConfig, TogalornForCausalLM)
 from .families import ChatGLM2Config
 from .modeling_utils import PreTrainedModel
 from .llama_legacy import LegacyLlamaForCausalLM, LlamaLegacyConfig

@@ -405,7 +405,98 @@ class GavatarConfig(PretrainedConfig):
         return dict(d, **own)
 
 
+class TogalornConfig(PretrainedConfig):
+    """Togalorn: a decoder on one fp32 stream whose layers read one norm, in parts of the width, and run their mixer and their
+    feed-forward side by side, the mixer behind a causal convolution of its input. A block of layers may run several times, each pass
+    starting from a product of the stream and the embedding output. Its mixers are latent attention with a rotated key part for all
+    heads and a gate per channel (``latent_attention``) and a state space with a scalar decay per head (``mamba2``); its
+    feed-forwards are mixtures of clamped gated experts with identity experts and a shared one; the head is untied.
+
+    Keys of ``config.json``: ``vocab``, ``width``, ``norm`` (``{"eps", "groups"}``), ``canon.taps``, ``embedding.scale``, ``loop``
+    (``{"start", "stop", "times"}`` or null) and ``layers``, a list of ``{"type": "latent_attention", "mixer": {"heads", "dim",
+    "rot_dim", "vdim", "q_rank", "kv_rank", "scale", "rot": {"base", "dims"}}}`` or ``{"type": "mamba2", "mixer": {"heads",
+    "vdim", "state", "groups", "conv", "norm_groups"}}``, each with ``"mlp": {"kind": "moe", "router": {"experts", "identity",
+    "top"}, "expert": {"ff", "limit"}, "shared": {"ff", "limit"}} | null``. Framework keys (``seq_length``, ``block_size``, token
+    ids) may stand beside them."""
+
+    model_type = "togalorn"
+
+    @classmethod
+    def default_values(cls):
+        return dict(architecture="Togalorn", vocab=32000, width=1024, norm=dict(eps=1e-6, groups=1), canon=dict(taps=4),
+                    embedding=dict(scale=1.0), loop=None,
+                    layers=TogalornConfig.layer_list("mamba2 mamba2 latent_attention", heads=8, dim=96, rot_dim=32, vdim=128, rank=256,
+                                                     ssm_heads=32, ssm_dim=64, state=128, experts=16, top=2, ff=768),
+                    pad_token_id=0, bos_token_id=None, eos_token_id=None, block_size=64)
+
+    @staticmethod
+    def layer_list(types: str, heads: int, dim: int, rot_dim: int, vdim: int, rank: int, ssm_heads: int, ssm_dim: int, state: int,
+                   experts: int, top: int, ff: int, q_rank=None, base: float = 500000.0, scale=None, ssm_groups: int = 1, conv: int = 4,
+                   norm_groups: int = 1, identity: int = 0, limit: float = 7.0, shared_ff=None, shared_limit=None):
+        """The ``layers`` list of a model whose layers of one type (``types``, by name) are alike."""
+        mixer = {"latent_attention": dict(heads=heads, dim=dim, rot_dim=rot_dim, vdim=vdim, q_rank=q_rank or rank, kv_rank=rank,
+                                          scale=scale or (dim + rot_dim) ** -0.5, rot=dict(base=base, dims=rot_dim)),
+                 "mamba2": dict(heads=ssm_heads, vdim=ssm_dim, state=state, groups=ssm_groups, conv=conv, norm_groups=norm_groups)}
+        mlp = dict(kind="moe", router=dict(experts=experts, identity=identity, top=top), expert=dict(ff=ff, limit=limit),
+                   shared=dict(ff=shared_ff or ff, limit=shared_limit or limit))
+        return [dict(type=t, mixer=copy.deepcopy(mixer[t]), mlp=copy.deepcopy(mlp)) for t in types.split()]
+
+    @staticmethod
+    def _layer_fields(i: int, layer: dict) -> dict:
+        kind, mix, mlp = layer.get("type"), layer["mixer"], layer.get("mlp")
+        if kind == "latent_attention":
+            rot = int(mix["rot_dim"])
+            if int(mix["rot"]["dims"]) != rot:
+                raise ValueError(f"layer {i}: {mix['rot']['dims']} rotated dimensions of a rotated part of {rot}")
+            out = dict(mixer="latent", num_attention_heads=int(mix["heads"]), num_query_groups=int(mix["heads"]),
+                       kv_channels=int(mix["dim"]), v_channels=int(mix["vdim"]), softmax_scale=float(mix["scale"]),
+                       q_lora_rank=int(mix["q_rank"]), kv_lora_rank=int(mix["kv_rank"]), rotary_dim=rot,
+                       rotary_base=float(mix["rot"]["base"]), attention_output_gate="channel")
+        elif kind == "mamba2":
+            out = dict(mixer="state_space", ssm_heads=int(mix["heads"]), ssm_head_dim=int(mix["vdim"]), ssm_state=int(mix["state"]),
+                       ssm_groups=int(mix["groups"]), ssm_conv_taps=int(mix["conv"]), ssm_norm_groups=int(mix["norm_groups"]))
+        else:
+            raise ValueError(f"layer {i}: unknown mixer type {kind!r}")
+        if mlp and mlp.get("kind", "moe") != "moe":
+            raise ValueError(f"layer {i}: unknown feed-forward kind {mlp['kind']!r}")
+        out.update(ffn_hidden_size=0)
+        if mlp:
+            r, e, s = mlp["router"], mlp["expert"], mlp["shared"]
+            identity = int(r.get("identity") or 0)
+            if not 1 <= int(r["top"]) <= int(r["experts"]) + identity:
+                raise ValueError(f"layer {i}: {r['top']} of {r['experts']} + {identity} experts")
+            out.update(num_moe_experts=int(r["experts"]), moe_identity_experts=identity, moe_router_topk=int(r["top"]),
+                       moe_ffn_hidden_size=int(e["ff"]), moe_activation_limit=float(e["limit"]),
+                       moe_shared_expert_intermediate_size=int(s["ff"]), moe_shared_expert_activation_limit=float(s["limit"]))
+        return out
+
+    def to_transformer_dict(self) -> dict:
+        d = {k: v for k, v in self.to_dict().items()
+             if k not in ("architecture", "layers", "norm", "vocab", "width", "embedding", "canon", "loop", "mlp", "mixer")}
+        fields = [self._layer_fields(i, layer) for i, layer in enumerate(self.layers)]
+        d.setdefault("seq_length", 32768)                      # angles are evaluated: a bound for buffers alone
+        d.setdefault("max_position_embeddings", d["seq_length"])
+        moe = [1 if f.get("num_moe_experts") else 0 for f in fields]
+        own = dict(num_attention_heads=1, num_query_groups=1, kv_channels=1, ffn_hidden_size=0)       # layers without attention
+        for f in fields:                                       # the stack's own view of what its layers override
+            own.update({k: v for k, v in f.items() if k in own and k != "ffn_hidden_size"})
+        if any(moe):
+            own.update({k: v for k, v in fields[moe.index(1)].items() if k.startswith(("num_moe", "moe_"))}, moe_layer_freq=moe)
+        loop = self.loop
+        own.update(vocab_size=int(self.vocab), hidden_size=int(self.width), num_layers=len(fields), layer_overrides=fields,
+                   layer_loop=(int(loop["start"]), int(loop["stop"]), int(loop["times"])) if loop else None, loop_input=bool(loop),
+                   layernorm_epsilon=float(self.norm["eps"]), norm_groups=int(self.norm["groups"]), normalization="RMSNorm",
+                   norm_placement="parallel", input_conv_taps=int(self.canon["taps"]), fp32_residual_connection=True,
+                   ragged_attention=True, rotary_interleaved=True, position_embedding_type="none",
+                   embedding_scale=float(self.embedding["scale"]), moe_activation="clamped_glu", moe_activation_alpha=1.702,
+                   moe_router_score_function="softmax", norm_topk_prob=True, moe_router_enable_expert_bias=True,
+                   moe_router_dtype="params", moe_router_topk_scaling_factor=1.0, tie_word_embeddings=False)
+        d = {k: v for k, v in d.items() if ALIASES.get(k, (k,))[0] not in own}
+        return dict(d, **own)
+
+
 for _legacy in (True, False):
+    MindFormerRegister.register_cls(TogalornConfig, MindFormerModuleType.CONFIG, alias="TogalornConfig", legacy=_legacy)
     MindFormerRegister.register_cls(GavatarConfig, MindFormerModuleType.CONFIG, alias="GavatarConfig", legacy=_legacy)
     MindFormerRegister.register_cls(KukupelConfig, MindFormerModuleType.CONFIG, alias="KukupelConfig", legacy=_legacy)
     MindFormerRegister.register_cls(MefesunConfig, MindFormerModuleType.CONFIG, alias="MefesunConfig", legacy=_legacy)
@@ -433,6 +524,11 @@ GavatarForCausalLM.kernel_sources = ("host_util", "elementwise", "gemm_tcgen05",
                                      "paged_decode_tc", "paged_attention", "paged_attention_any", "paged_talk_decode",
                                      "latent_decode", "router", "moe_ep",
                                      "moe_any", "decode_loop")
+TogalornForCausalLM = _model("TogalornForCausalLM", TogalornConfig, "togalorn")
+TogalornForCausalLM.kernel_sources = ("host_util", "elementwise", "gemm_tcgen05", "gemm_tcgen05_2cta", "gemm_bf16_decode",
+                                      "sandwich_norm", "joint_norm", "head_mix", "state_space", "paged_prefill_tc",
+                                      "paged_attention", "paged_attention_any", "paged_decode_tc", "latent_decode", "router", "moe_ep",
+                                      "moe_any", "decode_loop")
 ChatGLM2ForConditionalGeneration = _model("ChatGLM2ForConditionalGeneration", ChatGLM4Config, "glm")
 
 def _backbone(name, causal_cls):
@@ -503,6 +599,6 @@ MODEL_TYPE_TO_CLASSES = {
     "qwen2_moe": (Qwen2MoeConfig, Qwen2MoeForCausalLM),
     "telechat": (TelechatConfig, TelechatForCausalLM), "glm": (ChatGLM4Config, ChatGLM2ForConditionalGeneration),
     "mefesun": (MefesunConfig, MefesunForCausalLM), "kukupel": (KukupelConfig, KukupelForCausalLM),
-    "gavatar": (GavatarConfig, GavatarForCausalLM),
+    "gavatar": (GavatarConfig, GavatarForCausalLM), "togalorn": (TogalornConfig, TogalornForCausalLM),
     "chatglm": (ChatGLM4Config, ChatGLM2ForConditionalGeneration),
 }

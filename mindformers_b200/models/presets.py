@@ -77,6 +77,17 @@ PRESETS = {
                      mlp=dict(kind="moe", router=dict(experts=8, top=2), expert=dict(ff=256))),
                 dict(type="attention", mixer=dict(heads=8, kv_heads=2, dim=32, vdim=32, scale=32 ** -0.5, mask=dict(size=128)),
                      mlp=dict(kind="moe", router=dict(experts=8, top=2), expert=dict(ff=256)))]),
+    "tiny_togalorn": dict(
+        model_type="togalorn", vocab=1024, width=320, norm=dict(eps=1e-6, groups=2), canon=dict(taps=4), embedding=dict(scale=12.0),
+        loop=dict(start=1, stop=3, times=2),
+        layers=[dict(type="mamba2", mixer=dict(heads=10, vdim=64, state=64, groups=2, conv=4, norm_groups=5),
+                     mlp=dict(kind="moe", router=dict(experts=6, identity=2, top=2), expert=dict(ff=192, limit=7.0),
+                              shared=dict(ff=256, limit=5.0))),
+                dict(type="latent_attention",
+                     mixer=dict(heads=5, dim=48, rot_dim=16, vdim=64, q_rank=96, kv_rank=160, scale=0.125, rot=dict(base=1e4, dims=16)),
+                     mlp=dict(kind="moe", router=dict(experts=6, identity=2, top=2), expert=dict(ff=192, limit=7.0),
+                              shared=dict(ff=256, limit=5.0))),
+                dict(type="mamba2", mixer=dict(heads=10, vdim=64, state=64, groups=2, conv=4, norm_groups=5), mlp=None)]),
     "tiny_llama": dict(
         model_type="llama", num_hidden_layers=2, hidden_size=256, num_attention_heads=4, num_key_value_heads=2,
         intermediate_size=688, vocab_size=1024, rms_norm_eps=1e-5, rope_theta=10000.0,

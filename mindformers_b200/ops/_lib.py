@@ -117,7 +117,7 @@ def _declare(lib):
     sig("mfb_moe_plan", [I, I, P, I, I, I] + [P] * 11)
     sig("mfb_moe_scatter", [I] * 7 + [P] * 12)
     sig("mfb_moe_barrier", [I, I, P, I, P, P, P])
-    sig("mfb_moe_gather", [I] * 7 + [P] * 9)
+    sig("mfb_moe_gather", [I] * 7 + [P] * 9 + [L, P, P])
     sig("mfb_flash_attn_fwd_ex", [P, P, P, P, P, I, I, I, I, I, L, L, L, L, I, I, F, P, P])
     sig("mfb_flash_attn_bwd_ex", [P] * 10 + [I, I, I, I, I] + [L] * 8 + [I, I, F, P, P])
     sig("mfb_cp_flag_words", [])
@@ -147,7 +147,11 @@ def _declare(lib):
     sig("mfb_residual_streams", [P, I, P, L, P, P, P, P, P, P, I, I, I, F, I, P])
     sig("mfb_embed_stream", [P, P, P, P, P, I, I, I, F, I, P])
     sig("mfb_normed_step", [P, P, L] + [P] * 11 + [I] * 4 + [F, I, P])
-    sig("mfb_latent_norm_cache", [P, L, P, P, F, P, P, P, I, I, I, I, P])
+    sig("mfb_latent_norm_cache", [P, L, P, P, F] + [P] * 5 + [I] * 5 + [P])
+    sig("mfb_rotate_tail", [P, P, P] + [I] * 5 + [P])
+    sig("mfb_joint_step", [P, P, L, P, L, P, L] + [P] * 11 + [I] * 5 + [F, I, P])
+    sig("mfb_state_space_scratch_floats", [I] * 4, L)
+    sig("mfb_state_space", [P, L] + [P] * 14 + [L] + [I] * 9 + [F, I, P])
     sig("mfb_gate_heads", [P, L, P, L, I, I, I, I, P])
     sig("mfb_talk_mix", [P, P, P, L, P, I, I, I, I, I, P])
     sig("mfb_matrix_memory_scratch_floats", [I] * 5, L)
@@ -156,16 +160,16 @@ def _declare(lib):
     sig("mfb_paged_talk_decode_splits", [I, I])
     sig("mfb_paged_talk_decode_scratch_bytes", [I] * 5, L)
     sig("mfb_paged_talk_decode", [P] * 8 + [L, P, P] + [I] * 11 + [F, P, P])
-    sig("mfb_latent_decode_supported", [I, I])
+    sig("mfb_latent_decode_supported", [I, I, I])
     sig("mfb_latent_decode_splits", [I, I, I])
     sig("mfb_latent_decode_scratch_bytes", [I] * 4, L)
-    sig("mfb_latent_decode", [P] * 7 + [I] * 8 + [F, P, P])
+    sig("mfb_latent_decode", [P] * 7 + [I] * 9 + [F, P, P])
     sig("mfb_delta_decode_supported", [I, I])
     sig("mfb_delta_scratch_floats", [I] * 6, L)
     sig("mfb_delta_rule", [P, L, P, P, L, P, L] + [P] * 11 + [L] + [I] * 9 + [F, F, I, P])
     sig("mfb_clamped_glu", [P, P, I, I, F, F, F, P, P, P, P, I, P])
-    sig("mfb_moe_scatter_any", [P] * 7 + [I] * 5 + [P])
-    sig("mfb_moe_gather_any", [P] * 4 + [I] * 4 + [P])
+    sig("mfb_moe_scatter_any", [P] * 7 + [I] * 6 + [P])
+    sig("mfb_moe_gather_any", [P] * 6 + [L, P] + [I] * 5 + [P])
     sig("mfb_grouped_gemm_any", [P, P, P, I, I, I, P, P, P, P, I, P])
     sig("mfb_qkv_rope_cache", [P, L, P, P, P, F, P, F, I, I, P, P, P, P, P, I, I, I, I, I, I, I, P])
     sig("mfb_add_normed", [P, L, P, P, P, P, P, I, P, P, I, I, I, F, I, P])

@@ -1,6 +1,8 @@
 // Small steps around attention (sm_100a, bf16 or fp32):
 //
-//   latent_norm_cache:  RMS norms of the query latent and of the key / value latent, the latter into the paged cache
+//   latent_norm_cache:  RMS norms of the query latent and of the key / value latent, the latter into the paged cache, followed by a
+//                       key part that is rotated by its position (neighbouring dimensions are pairs)
+//   rotate_tail:        the same rotation of the last dimensions of every query head
 //   gate_heads:         x <- x * sigmoid(gate), a gate per column or per group of neighbouring columns
 //   talk_mix:           softmax weights mixed over heads, after the products with the values: head h of the result is
 //                       sum_g talk[h, g] o[g, own key / value head of h], times sigmoid(gate)
@@ -21,11 +23,21 @@ __device__ __forceinline__ void st2(__nv_bfloat16* p, float a, float b) {
 }
 __device__ __forceinline__ float sigmoid(float z) { return 1.f / (1.f + __expf(-z)); }
 
+// (u, v) turned by the angle position * freq
+__device__ __forceinline__ void rotate(float& u, float& v, long long position, float freq) {
+  float s, c;
+  sincosf(static_cast<float>(position) * freq, &s, &c);
+  const float a = u * c - v * s;
+  v = v * c + u * s;
+  u = a;
+}
+
 // one CTA of two warpgroups' worth of warps per token: the first half norms the query latent, the second the other one
 template <typename T>
 __global__ void __launch_bounds__(256)
 latent_norm_cache_kernel(const T* __restrict__ proj, long long ld_proj, const T* __restrict__ q_norm, const T* __restrict__ kv_norm,
-                         float eps, const int* __restrict__ slots, T* __restrict__ q, T* __restrict__ cache, int Q, int R) {
+                         float eps, const int* __restrict__ slots, T* __restrict__ q, T* __restrict__ cache,
+                         const float* __restrict__ freqs, const long long* __restrict__ positions, int Q, int R, int P) {
   __shared__ float red[8];
   const long long t = blockIdx.x;
   const int half = threadIdx.x >> 7, tid = threadIdx.x & 127;
@@ -44,8 +56,58 @@ latent_norm_cache_kernel(const T* __restrict__ proj, long long ld_proj, const T*
   const int slot = slots[t];
   if (half && slot < 0) return;
   const T* w = half ? kv_norm : q_norm;
-  T* dst = half ? cache + (long long)slot * R : q + t * Q;
+  T* dst = half ? cache + (long long)slot * (R + P) : q + t * Q;
   for (int i = tid; i < n; i += 128) st(dst + i, ld(src + i) * rstd * ld(w + i));
+  if (!half) return;
+  for (int i = tid; i < P / 2; i += 128) {
+    float u = ld(src + R + 2 * i), v = ld(src + R + 2 * i + 1);
+    rotate(u, v, positions[t], freqs[i]);
+    st(dst + R + 2 * i, u);
+    st(dst + R + 2 * i + 1, v);
+  }
+}
+
+// a thread per pair
+template <typename T>
+__global__ void __launch_bounds__(256)
+rotate_tail_kernel(T* __restrict__ x, const float* __restrict__ freqs, const long long* __restrict__ positions, int T_rows, int H,
+                   int D, int P) {
+  const int half = P / 2;
+  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < (long long)T_rows * H * half;
+       i += (long long)gridDim.x * blockDim.x) {
+    const long long head = i / half;
+    const int k = (int)(i % half);
+    T* p = x + head * D + D - P + 2 * k;
+    float u = ld(p), v = ld(p + 1);
+    rotate(u, v, positions[head / H], freqs[k]);
+    st(p, u);
+    st(p + 1, v);
+  }
+}
+
+// bf16, four pairs per thread; the heads of a token that a thread meets share its cosines
+__global__ void __launch_bounds__(256)
+rotate_tail_vec_kernel(__nv_bfloat16* __restrict__ x, const float* __restrict__ freqs, const long long* __restrict__ positions, int H,
+                       int D, int P) {
+  const long long t = blockIdx.x;
+  const int per = P / 8, lanes = blockDim.x / per * per;        // threads in use: whole tails
+  if ((int)threadIdx.x >= lanes) return;
+  const int k = threadIdx.x % per;
+  float c[4], s[4];
+  const float pos = static_cast<float>(positions[t]);
+#pragma unroll
+  for (int i = 0; i < 4; ++i) sincosf(pos * freqs[4 * k + i], &s[i], &c[i]);
+  for (int h = threadIdx.x / per; h < H; h += lanes / per) {
+    uint4* p = reinterpret_cast<uint4*>(x + (t * H + h) * D + D - P + 8 * k);
+    uint4 u = *p;
+    __nv_bfloat162* v = reinterpret_cast<__nv_bfloat162*>(&u);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const float2 f = __bfloat1622float2(v[i]);
+      v[i] = __floats2bfloat162_rn(f.x * c[i] - f.y * s[i], f.y * c[i] + f.x * s[i]);
+    }
+    *p = u;
+  }
 }
 
 // bf16, eight columns per access, a warp per token and latent, which it keeps in registers: latents of up to 32 * 8 * kHold
@@ -53,7 +115,8 @@ constexpr int kHold = 8;
 __global__ void __launch_bounds__(256)
 latent_norm_cache_vec_kernel(const __nv_bfloat16* __restrict__ proj, long long ld_proj, const __nv_bfloat16* __restrict__ q_norm,
                              const __nv_bfloat16* __restrict__ kv_norm, float eps, const int* __restrict__ slots,
-                             __nv_bfloat16* __restrict__ q, __nv_bfloat16* __restrict__ cache, int T_rows, int Q, int R) {
+                             __nv_bfloat16* __restrict__ q, __nv_bfloat16* __restrict__ cache, const float* __restrict__ freqs,
+                             const long long* __restrict__ positions, int T_rows, int Q, int R, int P) {
   const int unit = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   if (unit >= 2 * T_rows) return;
   const long long t = unit >> 1;
@@ -79,7 +142,14 @@ latent_norm_cache_vec_kernel(const __nv_bfloat16* __restrict__ proj, long long l
     }
   }
   const float rstd = 1.f / sqrtf(warp_sum(ss) / n + eps);
-  __nv_bfloat16* dst = kv ? cache + (long long)slot * R : q + t * Q;
+  __nv_bfloat16* dst = kv ? cache + (long long)slot * (R + P) : q + t * Q;
+  if (kv) {
+    for (int i = lane; i < P / 2; i += 32) {
+      float2 f = ld2(src + R + 2 * i);
+      rotate(f.x, f.y, positions[t], freqs[i]);
+      st2(dst + R + 2 * i, f.x, f.y);
+    }
+  }
 #pragma unroll
   for (int i = 0; i < kHold; ++i) {
     const int c = (i * 32 + lane) * 8;
@@ -266,24 +336,46 @@ bool al(const void* p, int n) { return (reinterpret_cast<uintptr_t>(p) & (n - 1)
 extern "C" {
 using namespace mfb;
 
-// proj [T, >= Q + R] (rows ld_proj apart): query latent | key / value latent; q [T, Q]; cache rows [.., R] at slots[t] (< 0: not
-// written). f32 = 1: all fp32, else bf16.
+// proj [T, >= Q + R + P] (rows ld_proj apart): query latent | key / value latent | key part to rotate; q [T, Q]; cache rows [..,
+// R + P] at slots[t] (< 0: not written); freqs [P / 2] and positions [T] (not read with P = 0). f32 = 1: all fp32, else bf16.
 int mfb_latent_norm_cache(const void* proj, long long ld_proj, const void* q_norm, const void* kv_norm, float eps, const int* slots,
-                          void* q, void* cache, int T, int Q, int R, int f32, cudaStream_t stream) {
+                          void* q, void* cache, const float* freqs, const long long* positions, int T, int Q, int R, int P, int f32,
+                          cudaStream_t stream) {
   if (T <= 0) return 0;
-  if (Q < 1 || R < 1 || ld_proj < Q + R) { mfb_host::set_error("latent_norm_cache: Q=%d R=%d", Q, R); return 1; }
+  if (Q < 1 || R < 1 || P < 0 || P % 2 || ld_proj < Q + R + P || (P && (!freqs || !positions))) {
+    mfb_host::set_error("latent_norm_cache: Q=%d R=%d P=%d", Q, R, P);
+    return 1;
+  }
   using bf = __nv_bfloat16;
   constexpr int most = 32 * 8 * hmx::kHold;
-  if (!f32 && Q % 8 == 0 && R % 8 == 0 && ld_proj % 8 == 0 && Q <= most && R <= most && hmx::al(proj, 16) && hmx::al(q_norm, 16)
+  if (!f32 && Q % 8 == 0 && R % 8 == 0 && P % 8 == 0 && ld_proj % 8 == 0 && Q <= most && R <= most && hmx::al(proj, 16) && hmx::al(q_norm, 16)
       && hmx::al(kv_norm, 16) && hmx::al(q, 16) && hmx::al(cache, 16)) {
     hmx::latent_norm_cache_vec_kernel<<<(int)(((long long)T * 2 + 7) / 8), 256, 0, stream>>>(
-        (const bf*)proj, ld_proj, (const bf*)q_norm, (const bf*)kv_norm, eps, slots, (bf*)q, (bf*)cache, T, Q, R);
+        (const bf*)proj, ld_proj, (const bf*)q_norm, (const bf*)kv_norm, eps, slots, (bf*)q, (bf*)cache, freqs,
+        positions, T, Q, R, P);
     return cudaGetLastError() == cudaSuccess ? 0 : 2;
   }
   if (f32) hmx::latent_norm_cache_kernel<float><<<T, 256, 0, stream>>>((const float*)proj, ld_proj, (const float*)q_norm,
-      (const float*)kv_norm, eps, slots, (float*)q, (float*)cache, Q, R);
+      (const float*)kv_norm, eps, slots, (float*)q, (float*)cache, freqs, positions, Q, R, P);
   else hmx::latent_norm_cache_kernel<bf><<<T, 256, 0, stream>>>((const bf*)proj, ld_proj, (const bf*)q_norm, (const bf*)kv_norm,
-      eps, slots, (bf*)q, (bf*)cache, Q, R);
+      eps, slots, (bf*)q, (bf*)cache, freqs, positions, Q, R, P);
+  return cudaGetLastError() == cudaSuccess ? 0 : 2;
+}
+
+// x [T, H, D]: the last P dimensions of every head are rotated in place by positions[t] * freqs.
+int mfb_rotate_tail(void* x, const float* freqs, const long long* positions, int T, int H, int D, int P, int f32, cudaStream_t stream) {
+  if (T <= 0 || P == 0) return 0;
+  if (H < 1 || P < 0 || P % 2 || P > D) { mfb_host::set_error("rotate_tail: H=%d D=%d P=%d", H, D, P); return 1; }
+  if (!f32 && P % 8 == 0 && D % 8 == 0 && P <= 8 * 256 && hmx::al(x, 16)) {
+    const long long want = (long long)H * (P / 8);
+    const int threads = want < 256 ? (int)((want + 31) / 32 * 32) : 256;
+    hmx::rotate_tail_vec_kernel<<<T, threads, 0, stream>>>((__nv_bfloat16*)x, freqs, positions, H, D, P);
+    return cudaGetLastError() == cudaSuccess ? 0 : 2;
+  }
+  const long long want = ((long long)T * H * (P / 2) + 255) / 256;
+  const int grid = (int)(want < 148 * 16 ? want : 148 * 16);
+  if (f32) hmx::rotate_tail_kernel<float><<<grid, 256, 0, stream>>>((float*)x, freqs, positions, T, H, D, P);
+  else hmx::rotate_tail_kernel<__nv_bfloat16><<<grid, 256, 0, stream>>>((__nv_bfloat16*)x, freqs, positions, T, H, D, P);
   return cudaGetLastError() == cudaSuccess ? 0 : 2;
 }
 

@@ -1,13 +1,14 @@
 // Decode attention over a paged cache of latents, keys and values at once (sm_100a, tcgen05 + TMA), with an optional sliding
 // window and softmax sink. The factors that make keys and values of a latent are absorbed into query and result, so that one
-// decode step is, per sequence and head h with q, c of `rank` numbers (a multiple of 8 up to 512):
+// decode step is, per sequence and head h with q, c of `rank` numbers (a multiple of 8 up to 576), of which the first `v_rank` (up to
+// 512) make the values and the others only keys (a key part with positions, shared by the heads):
 //     s[t]   = scale * <q[h], c[t]>                       max(0, len - window) <= t < len
-//     o[h,:] = sum_t softmax(s)[t] * c[t]                 the sink is one more term of the softmax's denominator
+//     o[h,:] = sum_t softmax(s)[t] * c[t][:v_rank]        the sink is one more term of the softmax's denominator
 // As in mla_decode.cu, which serves one fixed latent width beside rotated columns, the products are transposed so that the tokens
 // fill the 128 rows of the tensor core, and a CTA takes (split of the sequence, 16 or 32 heads, sequence):
 //     S^T [128 tokens x heads]       = C_tile (A, K-major) . Q^T (B, K-major)
 //     O^T [rank x heads]            += C_tile^T (A, MN-major: the same bytes) . P^T [heads x 128 tokens] (B, K-major)
-// A tile of 128 tokens lies in up to four 32 KB slots of a ring (128 latent columns each, the last one possibly half) from its
+// A tile of 128 tokens lies in up to five 32 KB slots of a ring (128 latent columns each, the last one possibly half) from its
 // scores to its last product, so the cache is read once per 32 heads. Where two tiles fit the ring, the scores of the next tile
 // are computed under the softmax of this one. Columns past the rank are zero fill in both operands; the rows of O^T that belong
 // to them are not stored.
@@ -21,7 +22,7 @@ namespace latd {
 
 constexpr int kThreads = 192;
 constexpr int kTile = 128;              // tokens per tile
-constexpr int kMaxRank = 512;
+constexpr int kMaxRank = 576, kMaxVRank = 512;
 constexpr int kSub = kTile * 128;       // [128 tokens][64 columns] swizzled sub-tile, 16 KB
 constexpr int kUnit = 2 * kSub;         // ring slot: a pair of sub-tiles (128 columns)
 constexpr int kMaxSlots = 6;
@@ -41,9 +42,9 @@ struct Shape {
 struct Args {
   const int* block_tables;   // [B, max_blocks]
   const int* context_lens;   // [B]
-  int max_blocks, block_size, num_heads, splits, rank, window;
+  int max_blocks, block_size, num_heads, splits, rank, v_rank, window;
   float scale_log2;
-  float* part_o;             // [B, num_heads, splits, rank] unnormalised
+  float* part_o;             // [B, num_heads, splits, v_rank] unnormalised
   float* part_ml;            // [B, num_heads, splits, 2]: running max (log2 units), sum
   int* status;
 };
@@ -91,6 +92,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
   const int t0 = base_tile + rel0;
   const int head0 = chunk * kHeads;
   const int subs = (args.rank + 63) / 64, units = (subs + 1) / 2;      // 64-column sub-tiles, pairs of them
+  const int v_units = (args.v_rank + 127) / 128;                       // pairs that hold values
 
   if (threadIdx.x == 0) {
     *abort_flag = 0;
@@ -196,10 +198,12 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
         for (int m = 0; m < units; ++m) {
           const int slot = (j * units + m) % kSlots;
           const uint64_t ca = ring_v + slot * (kUnit >> 4);
+          if (m < v_units) {
 #pragma unroll
-          for (int k = 0; k < kTile / 16; ++k)
-            umma_f16_ss_warp(leader, tmem_O + m * kHeads, ca + k * ((16 * 128) >> 4), p_desc + (k >> 2) * ((kHeads * 128) >> 4) + (k & 3) * 2,
-                             IDESC_PV, (j > 0 || k > 0) ? 1u : 0u);
+            for (int k = 0; k < kTile / 16; ++k)
+              umma_f16_ss_warp(leader, tmem_O + m * kHeads, ca + k * ((16 * 128) >> 4), p_desc + (k >> 2) * ((kHeads * 128) >> 4) + (k & 3) * 2,
+                               IDESC_PV, (j > 0 || k > 0) ? 1u : 0u);
+          }
           umma_commit_warp(leader, smem_u32(&empty[slot]));
         }
         umma_commit_warp(leader, smem_u32(pv_done));
@@ -269,7 +273,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
         ok = mbar_wait(smem_u32(pv_done), (j - 1) & 1, abort_flag, args.status, kStatusWaitTimeoutEpilogue);
         if (ok && any_rescale) {
           tc_fence_after();
-          for (int m = 0; m < units; ++m)
+          for (int m = 0; m < v_units; ++m)
 #pragma unroll
             for (int c = 0; c < kHeads; c += 16) {
               uint32_t r[16];
@@ -324,7 +328,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
       ml[1] = lh;
     }
     if (have) tc_fence_after();
-    for (int m = 0; m < units; ++m) {
+    for (int m = 0; m < v_units; ++m) {
       const int col = m * 128 + row;
 #pragma unroll
       for (int c = 0; c < kHeads; c += 16) {
@@ -335,8 +339,8 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
         }
 #pragma unroll
         for (int h = 0; h < 16; ++h)
-          if (head0 + c + h < args.num_heads && col < args.rank)      // a split without tokens writes zeros, which the merge weighs by zero
-            args.part_o[((first_row + c + h) * args.splits + split) * args.rank + col] = have ? __uint_as_float(r[h]) : 0.f;
+          if (head0 + c + h < args.num_heads && col < args.v_rank)    // a split without tokens writes zeros, which the merge weighs by zero
+            args.part_o[((first_row + c + h) * args.splits + split) * args.v_rank + col] = have ? __uint_as_float(r[h]) : 0.f;
       }
     }
   }
@@ -352,7 +356,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
 template <int HEADS>
 int launch(const CUtensorMap& tQ, const CUtensorMap& tC, const Args& a, int B, cudaStream_t stream) {
   using Sh = Shape<HEADS>;
-  static_assert(Sh::kSlots >= 4, "a tile has up to four pairs");
+  static_assert(Sh::kSlots >= (kMaxRank + 127) / 128, "a tile lies in the ring as a whole");
   static bool attr_set = false;
   if (!attr_set) {
     if (cudaFuncSetAttribute(latent_decode_kernel<HEADS>, cudaFuncAttributeMaxDynamicSharedMemorySize, Sh::kSmem) != cudaSuccess) {
@@ -379,8 +383,8 @@ int mfb_paged_combine_ex(const float* part_acc, const float* part_ml, void* out,
                          const int* cu_q, const float* sink, long long ld_out, float out_scale,
                          cudaStream_t stream);      // paged_attention.cu
 
-int mfb_latent_decode_supported(int rank, int block_size) {
-  return rank >= 8 && rank <= latd::kMaxRank && rank % 8 == 0 &&
+int mfb_latent_decode_supported(int rank, int v_rank, int block_size) {
+  return v_rank >= 8 && v_rank <= latd::kMaxVRank && v_rank % 8 == 0 && rank >= v_rank && rank <= latd::kMaxRank && rank % 8 == 0 &&
                  (block_size == 16 || block_size == 32 || block_size == 64 || block_size == 128)
              ? 1 : 0;
 }
@@ -401,18 +405,18 @@ int mfb_latent_decode_splits(int B, int num_heads, int max_len) {
   return best;
 }
 
-long long mfb_latent_decode_scratch_bytes(int B, int num_heads, int rank, int splits) {
-  return static_cast<long long>(B) * splits * num_heads * (rank + 2) * 4;
+long long mfb_latent_decode_scratch_bytes(int B, int num_heads, int v_rank, int splits) {
+  return static_cast<long long>(B) * splits * num_heads * (v_rank + 2) * 4;
 }
 
-// q [B, num_heads, rank] (queries in latent space), cache [num_blocks, block_size, rank], out [B, num_heads, rank], all bf16;
+// q [B, num_heads, rank] (queries in latent space), cache [num_blocks, block_size, rank], out [B, num_heads, v_rank], all bf16;
 // block_tables [B, max_blocks]; context_lens [B] counts the tokens in the cache, the new one included; window > 0: only the last
 // `window` of them; sink [num_heads] fp32 or null; scratch: mfb_latent_decode_scratch_bytes.
 int mfb_latent_decode(const void* q, const void* cache, const int* block_tables, const int* context_lens, const float* sink, void* out,
-                      void* scratch, int splits, int B, int num_heads, int rank, int num_blocks, int block_size, int max_blocks,
+                      void* scratch, int splits, int B, int num_heads, int rank, int v_rank, int num_blocks, int block_size, int max_blocks,
                       int window, float scale, int* status, cudaStream_t stream) {
-  if (!mfb_latent_decode_supported(rank, block_size) || num_heads < 1 || splits < 1 || num_blocks < 1 || max_blocks < 1) {
-    mfb_host::set_error("latent_decode: heads=%d rank=%d splits=%d block_size=%d", num_heads, rank, splits, block_size);
+  if (!mfb_latent_decode_supported(rank, v_rank, block_size) || num_heads < 1 || splits < 1 || num_blocks < 1 || max_blocks < 1) {
+    mfb_host::set_error("latent_decode: heads=%d rank=%d v_rank=%d splits=%d block_size=%d", num_heads, rank, v_rank, splits, block_size);
     return 1;
   }
   if (B <= 0) return 0;
@@ -423,14 +427,14 @@ int mfb_latent_decode(const void* q, const void* cache, const int* block_tables,
   if ((rc = mfb_host::make_tmap_2d(&tC, cache, 2, BF, (uint64_t)num_blocks * block_size, rank, rank, block_size, 64))) return 30 + rc;
   latd::Args a;
   a.block_tables = block_tables; a.context_lens = context_lens; a.max_blocks = max_blocks; a.block_size = block_size;
-  a.num_heads = num_heads; a.splits = splits; a.rank = rank; a.window = window; a.scale_log2 = scale * 1.4426950408889634f;
+  a.num_heads = num_heads; a.splits = splits; a.rank = rank; a.v_rank = v_rank; a.window = window; a.scale_log2 = scale * 1.4426950408889634f;
   a.part_o = reinterpret_cast<float*>(scratch);
-  a.part_ml = a.part_o + static_cast<size_t>(B) * splits * num_heads * rank;
+  a.part_ml = a.part_o + static_cast<size_t>(B) * splits * num_heads * v_rank;
   a.status = status;
   rc = latd::heads_per_cta(num_heads) == 32 ? latd::launch<32>(tQ, tC, a, B, stream) : latd::launch<16>(tQ, tC, a, B, stream);
   if (rc) return rc;
-  return mfb_paged_combine_ex(a.part_o, a.part_ml, out, splits, B * num_heads, rank, num_heads, nullptr, sink,
-                              (long long)num_heads * rank, 1.f, stream);
+  return mfb_paged_combine_ex(a.part_o, a.part_ml, out, splits, B * num_heads, v_rank, num_heads, nullptr, sink,
+                              (long long)num_heads * v_rank, 1.f, stream);
 }
 
 }  // extern "C"

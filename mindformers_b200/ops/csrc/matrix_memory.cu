@@ -13,7 +13,7 @@
 //                  head's S in registers
 //   finish_kernel: norm, gate and the new n and m of a portion (which other CTAs read until then)
 //   decode_kernel: one row per slot, all in one pass; rows of idle slots (slot_mapping < 0) become zeros
-#include "common.cuh"
+#include "mma_sync.cuh"
 
 namespace mfb {
 namespace mmem {
@@ -287,34 +287,6 @@ __global__ void __launch_bounds__(kDec) decode_kernel(const Args a) {
 // accumulators. q, k and v enter the products as they are (bf16); fp32 factors enter as sums of bf16 numbers: two for S and the
 // weights in the read-out, three for the weighted values that go into S, whose error would stay.
 constexpr int kChunk = 64;
-
-__device__ __forceinline__ void cp16(uint32_t dst, const void* src, int bytes) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(bytes) : "memory");
-}
-__device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-template <int N>
-__device__ __forceinline__ void cp_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
-__device__ __forceinline__ void ldsm4(uint32_t (&r)[4], uint32_t addr) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
-__device__ __forceinline__ void ldsm4t(uint32_t (&r)[4], uint32_t addr) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
-__device__ __forceinline__ void mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
-               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-// two fp32 numbers as a pair of bf16 numbers; they become what is left
-__device__ __forceinline__ uint32_t take_bf16(float& x, float& y) {
-  const __nv_bfloat162 h = __floats2bfloat162_rn(x, y);
-  const float2 f = __bfloat1622float2(h);
-  x -= f.x;
-  y -= f.y;
-  return *reinterpret_cast<const uint32_t*>(&h);
-}
 
 // a warp per head, two tokens per lane
 template <typename T>

@@ -74,9 +74,9 @@ template <typename T>
 __global__ void __launch_bounds__(128)
 scatter_kernel(const T* __restrict__ x, const long long* __restrict__ ids, const int* __restrict__ rank_in_e,
                const int* __restrict__ write_base, const float* __restrict__ weights, T* __restrict__ rows,
-               int* __restrict__ dest_row, int k, int H, int rows_cap) {
-  const int c = blockIdx.x;
-  const int row = write_base[ids[c]] + rank_in_e[c];
+               int* __restrict__ dest_row, int k, int H, int E, int rows_cap) {
+  const int c = blockIdx.x, e = (int)ids[c];
+  const int row = e < E ? write_base[e] + rank_in_e[c] : -1;         // copies for identity experts have no row
   const bool ok = row >= 0 && row < rows_cap;
   if (threadIdx.x == 0) dest_row[c] = ok ? row : -1;
   if (!ok) return;
@@ -87,14 +87,17 @@ scatter_kernel(const T* __restrict__ x, const long long* __restrict__ ids, const
 
 template <typename T>
 __global__ void __launch_bounds__(128)
-gather_kernel(const T* __restrict__ rows, const int* __restrict__ dest_row, const float* __restrict__ weights, T* __restrict__ out,
-              int k, int H) {
+gather_kernel(const T* __restrict__ rows, const int* __restrict__ dest_row, const float* __restrict__ weights,
+              const long long* __restrict__ ids, const T* __restrict__ self, const T* __restrict__ extra, long long ld_extra,
+              T* __restrict__ out, int k, int H, int E) {
   const long long t = blockIdx.x;
   for (int i = threadIdx.x; i < H; i += blockDim.x) {
-    float s = 0.f;
+    float s = extra ? ld(extra + t * ld_extra + i) : 0.f;
     for (int j = 0; j < k; ++j) {
       const int r = dest_row[t * k + j];
-      if (r >= 0) s = fmaf(weights ? weights[t * k + j] : 1.f, ld(rows + (long long)r * H + i), s);
+      const float w = weights ? weights[t * k + j] : 1.f;
+      if (r >= 0) s = fmaf(w, ld(rows + (long long)r * H + i), s);
+      else if (self && ids[t * k + j] >= E) s = fmaf(w, ld(self + t * H + i), s);
     }
     st(out + t * H + i, s);
   }
@@ -174,20 +177,24 @@ int mfb_clamped_glu(const void* x, void* y, int R, int F, float limit, float alp
 }
 
 int mfb_moe_scatter_any(const void* x, const long long* ids, const int* rank_in_e, const int* write_base, const float* weights,
-                        void* rows, int* dest_row, int T, int k, int H, int rows_cap, int f32, cudaStream_t stream) {
+                        void* rows, int* dest_row, int T, int k, int H, int E, int rows_cap, int f32, cudaStream_t stream) {
   if (T <= 0 || k <= 0) return 0;
   if (f32) many::scatter_kernel<float><<<T * k, 128, 0, stream>>>((const float*)x, ids, rank_in_e, write_base, weights,
-      (float*)rows, dest_row, k, H, rows_cap);
+      (float*)rows, dest_row, k, H, E, rows_cap);
   else many::scatter_kernel<__nv_bfloat16><<<T * k, 128, 0, stream>>>((const __nv_bfloat16*)x, ids, rank_in_e, write_base, weights,
-      (__nv_bfloat16*)rows, dest_row, k, H, rows_cap);
+      (__nv_bfloat16*)rows, dest_row, k, H, E, rows_cap);
   return cudaGetLastError() == cudaSuccess ? 0 : 2;
 }
 
-int mfb_moe_gather_any(const void* rows, const int* dest_row, const float* weights, void* out, int T, int k, int H, int f32,
-                       cudaStream_t stream) {
+// Copies with ids >= E stand for self [T, H] (null: nothing); extra [T, H] (rows ld_extra apart; null: nothing) is added.
+int mfb_moe_gather_any(const void* rows, const int* dest_row, const float* weights, const long long* ids, const void* self,
+                       const void* extra, long long ld_extra, void* out, int T, int k, int H, int E, int f32, cudaStream_t stream) {
   if (T <= 0) return 0;
-  if (f32) many::gather_kernel<float><<<T, 128, 0, stream>>>((const float*)rows, dest_row, weights, (float*)out, k, H);
-  else many::gather_kernel<__nv_bfloat16><<<T, 128, 0, stream>>>((const __nv_bfloat16*)rows, dest_row, weights, (__nv_bfloat16*)out, k, H);
+  using bf = __nv_bfloat16;
+  if (f32) many::gather_kernel<float><<<T, 128, 0, stream>>>((const float*)rows, dest_row, weights, ids, (const float*)self,
+      (const float*)extra, ld_extra, (float*)out, k, H, E);
+  else many::gather_kernel<bf><<<T, 128, 0, stream>>>((const bf*)rows, dest_row, weights, ids, (const bf*)self, (const bf*)extra,
+      ld_extra, (bf*)out, k, H, E);
   return cudaGetLastError() == cudaSuccess ? 0 : 2;
 }
 

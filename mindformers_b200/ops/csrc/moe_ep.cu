@@ -228,8 +228,9 @@ moe_scatter_kernel(MoeMoveArgs a, const __nv_bfloat16* __restrict__ x) {
     const int t = (int)(c / a.k);
     const int e = (int)a.ids[c];
     const int owner = e / a.E_local;
-    const int row = a.write_base[e] + a.rank_in_e[c];
-    const bool ok = e >= 0 && owner < a.world && row >= 0 && row < a.owner_cap[owner];
+    const bool own = e >= 0 && owner < a.world;      // an identity expert (ids past the experts) has no row
+    const int row = own ? a.write_base[e] + a.rank_in_e[c] : -1;
+    const bool ok = own && row >= 0 && row < a.owner_cap[owner];
     if (lane == 0 && v_lo == 0) a.dest_row[c] = ok ? row : -1;
     if (!ok) continue;
     const uint4* src = reinterpret_cast<const uint4*>(x + (long long)t * a.H);
@@ -296,10 +297,12 @@ __global__ void moe_barrier_kernel(MoeBarrierArgs a) {
   if (threadIdx.x == 0) *a.epoch_ctr = epoch;
 }
 
-// out[t] = sum_j w[t,j] * row(t,j)  (w == null: plain sum); dots[t,j] = <g[t], row(t,j)> when g is given
+// out[t] = sum_j w[t,j] * row(t,j)  (w == null: plain sum) + extra[t]; dots[t,j] = <g[t], row(t,j)> when g is given. Forward only:
+// with `self`, the row of an identity expert (ids past the experts) is self[t].
 __global__ void __launch_bounds__(256)
 moe_gather_kernel(MoeMoveArgs a, __nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict__ g,
-                  float* __restrict__ dots) {
+                  float* __restrict__ dots, const __nv_bfloat16* __restrict__ self, const __nv_bfloat16* __restrict__ extra,
+                  long long ld_extra) {
   const int lane = threadIdx.x & 31;
   const int warps_per_cta = blockDim.x >> 5;
   const long long gw = (long long)blockIdx.x * warps_per_cta + (threadIdx.x >> 5);
@@ -315,6 +318,12 @@ moe_gather_kernel(MoeMoveArgs a, __nv_bfloat16* __restrict__ out, const __nv_bfl
       float acc[8];
 #pragma unroll
       for (int i = 0; i < 8; ++i) acc[i] = 0.f;
+      if (extra && v < vecs) {
+        const uint4 u = *reinterpret_cast<const uint4*>(extra + t * ld_extra + 8 * v);
+        const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&u);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) { const float2 f = __bfloat1622float2(h[i]); acc[2 * i] = f.x; acc[2 * i + 1] = f.y; }
+      }
       for (int j0 = 0; j0 < a.k; j0 += 4) {
         uint4 q[4];
         float w[4];
@@ -329,6 +338,9 @@ moe_gather_kernel(MoeMoveArgs a, __nv_bfloat16* __restrict__ out, const __nv_bfl
             const int owner = (int)a.ids[c] / a.E_local;
             if (row >= 0 && owner >= 0 && owner < a.world && v < vecs) {
               q[u] = moe_ld_cg(a.buf_peer[owner] + (long long)row * a.H + 8 * v);
+              w[u] = a.weights ? a.weights[c] : 1.f;
+            } else if (self && owner >= a.world && v < vecs) {
+              q[u] = *reinterpret_cast<const uint4*>(self + t * a.H + 8 * v);
               w[u] = a.weights ? a.weights[c] : 1.f;
             }
           }
@@ -512,17 +524,20 @@ int mfb_moe_barrier(int world, int rank, int* epoch_ctr, int phase, const long l
 
 int mfb_moe_gather(int world, int rank, int T, int k, int H, int E_local, int rows_cap, void* out,
                    const long long* ids, const int* dest_row, const long long* peer_bufs, const float* weights,
-                   const void* g, float* dots, int* status, cudaStream_t stream) {
+                   const void* g, float* dots, const void* self, const void* extra, long long ld_extra, int* status,
+                   cudaStream_t stream) {
   if (moe_check(world, rank, E_local * world, E_local, H)) return 1;
   for (int p = 0; p < world; ++p)
-    if (!aligned16(reinterpret_cast<const void*>(peer_bufs[p])) || !aligned16(out) || !aligned16(g)) {
-      mfb_host::set_error("moe gather: row buffers, the output and the gradient must be 16-byte aligned");
+    if (!aligned16(reinterpret_cast<const void*>(peer_bufs[p])) || !aligned16(out) || !aligned16(g) || !aligned16(self) ||
+        !aligned16(extra) || ld_extra % 8) {
+      mfb_host::set_error("moe gather: row buffers, the output, the gradient and what is added must be 16-byte aligned");
       return 1;
     }
   MoeMoveArgs a;
   fill_move(&a, world, rank, T, k, H, E_local, rows_cap, ids, nullptr, nullptr, nullptr, peer_bufs, weights,
             const_cast<int*>(dest_row), nullptr, nullptr, status);
-  moe_gather_kernel<<<148 * 4, 256, 0, stream>>>(a, (__nv_bfloat16*)out, (const __nv_bfloat16*)g, dots);
+  moe_gather_kernel<<<148 * 4, 256, 0, stream>>>(a, (__nv_bfloat16*)out, (const __nv_bfloat16*)g, dots, (const __nv_bfloat16*)self,
+                                                (const __nv_bfloat16*)extra, ld_extra);
   return cudaGetLastError() == cudaSuccess ? 0 : 2;
 }
 

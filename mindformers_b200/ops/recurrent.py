@@ -1,9 +1,11 @@
 """Recurrent mixers over ragged batches: the gated delta rule (short convolutions, unit keys, decays, the recurrence, its norm
-and gate) and the matrix memory (capped log gates, running maximum, memory and normaliser, norm and gate).
+and gate), the matrix memory (capped log gates, running maximum, memory and normaliser, norm and gate) and the state space with a
+scalar decay per head (short convolution, step sizes, the recurrence, gate and grouped norm).
 
-``delta_rule`` and ``matrix_memory`` have two bodies like the ops of ``functional.py``: the sm_100a kernels
-(``csrc/delta_rule.cu``, ``csrc/matrix_memory.cu``), always taken for CUDA tensors (bf16 or fp32 activations; state and
-recurrence are fp32), and a plain PyTorch body for CPU tensors. They are inference ops: they advance the state in place and have no gradients.
+``delta_rule``, ``matrix_memory`` and ``state_space`` have two bodies like the ops of ``functional.py``: the sm_100a kernels
+(``csrc/delta_rule.cu``, ``csrc/matrix_memory.cu``, ``csrc/state_space.cu``), always taken for CUDA tensors (bf16 or fp32
+activations; state and recurrence are fp32), and a plain PyTorch body for CPU tensors. They are inference ops: they advance the
+state in place and have no gradients.
 """
 from __future__ import annotations
 
@@ -43,7 +45,7 @@ class DeltaShape:
 
 def _rows(t: torch.Tensor, dtype, rows: int, cols: int, what: str):
     if t.dtype != dtype or t.dim() != 2 or t.shape[0] != rows or t.shape[1] < cols or t.stride(1) != 1:
-        raise TypeError(f"delta_rule: {what} must be a {dtype} matrix of {rows} rows and at least {cols} columns with unit stride")
+        raise TypeError(f"{what} must be a {dtype} matrix of {rows} rows and at least {cols} columns with unit stride")
 
 
 def _sequences(cache, T: int):
@@ -249,4 +251,116 @@ def matrix_memory(proj: torch.Tensor, input_bias: torch.Tensor, forget_bias: tor
                                f32, _lib.stream_ptr())
     _lib.check(rc, "mfb_matrix_memory")
     _lib.count_launch(3 if cache.is_prefill else 1)
+    return out
+
+
+# ---- state space --------------------------------------------------------------------------------------------------------------
+@dataclass
+class StateSpaceWeights:
+    """Per-layer weights beside the projections, all fp32: ``conv [taps, H P + 2 G N]`` (x, B, C channels; the last row belongs to
+    the current token), ``conv_bias``, ``dt_bias [H]``, ``a_log [H]``, ``skip [H]``, ``norm [H P]``."""
+    conv: torch.Tensor
+    conv_bias: torch.Tensor
+    dt_bias: torch.Tensor
+    a_log: torch.Tensor
+    skip: torch.Tensor
+    norm: torch.Tensor
+
+
+@dataclass
+class StateSpaceShape:
+    heads: int
+    head_dim: int
+    state: int
+    groups: int
+    taps: int
+    norm_groups: int
+
+    @property
+    def inner(self) -> int:
+        return self.heads * self.head_dim
+
+    @property
+    def channels(self) -> int:
+        return self.inner + 2 * self.groups * self.state
+
+    @property
+    def columns(self) -> int:
+        """Columns of the input projection: gate, x, B, C, step sizes."""
+        return self.inner + self.channels + self.heads
+
+
+def _state_space_reference(proj, w: StateSpaceWeights, s: StateSpaceShape, state, ring, cache, eps, out):
+    H, P, N, G = s.heads, s.head_dim, s.state, s.groups
+    if not cache.is_prefill:
+        out.zero_()
+    for slot, r0, n, start in _sequences(cache, proj.shape[0]):
+        z, xs, dt = torch.split(proj[r0:r0 + n, :s.columns], (s.inner, s.channels, H), dim=1)
+        before = torch.zeros(s.taps - 1, s.channels, dtype=torch.float32)
+        for d in range(1, s.taps):
+            if start - d >= 0:
+                before[s.taps - 1 - d] = ring[slot, (start - d) % s.taps].float()
+        seq = torch.cat((before, xs.float()))
+        y = F.silu(sum(seq[j:j + n] * w.conv[j] for j in range(s.taps)) + w.conv_bias).to(proj.dtype).float()
+        for p in range(max(start, start + n - s.taps), start + n):
+            ring[slot, p % s.taps] = xs[p - start]
+        x, B, C = y[:, :s.inner].view(n, H, P), y[:, s.inner:s.inner + G * N], y[:, s.inner + G * N:]
+        B, C = (t.view(n, G, N).repeat_interleave(H // G, 1) for t in (B, C))
+        dt = F.softplus(dt.float() + w.dt_bias, threshold=1e9)
+        keep = torch.exp(-torch.exp(w.a_log) * dt)
+        S = state[slot].clone() if start > 0 else torch.zeros(H, N, P)
+        o = torch.empty(n, H, P)
+        for t in range(n):
+            S = keep[t, :, None, None] * S + (dt[t, :, None] * B[t])[:, :, None] * x[t][:, None]
+            o[t] = (S * C[t][:, :, None]).sum(1) + w.skip[:, None] * x[t]
+        state[slot] = S
+        o = (o.reshape(n, s.inner) * F.silu(z.float())).unflatten(1, (s.norm_groups, -1))
+        o = o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + eps)
+        out[r0:r0 + n] = (o.flatten(1) * w.norm).to(out.dtype)
+
+
+def state_space(proj: torch.Tensor, w: StateSpaceWeights, s: StateSpaceShape, state: Tuple[torch.Tensor, torch.Tensor], cache,
+                eps: float) -> torch.Tensor:
+    """``proj [T, >= columns]`` (gate z | x | B | C | raw step size, any row pitch), all of the step's rows in the order of ``cache``
+    (``KVCacheContext``). x, B and C pass a causal convolution per channel and silu; per head (which shares B and C with its
+    group), with ``dt = softplus(raw + dt_bias)``::
+
+        S' = e^(-e^a_log dt) S + dt B x^T,   y = S'^T C + skip x
+
+    Returns ``[T, H P]``: ``y * silu(z)``, RMS-normed in ``norm_groups`` parts, times ``norm``. ``state``: the layer's ``(S [slots,
+    H, N, P] fp32, ring [slots, taps, channels])``, advanced in place."""
+    T, dtype = proj.shape[0], proj.dtype
+    S, ring = state
+    H, P, N = s.heads, s.head_dim, s.state
+    out = torch.empty((T, s.inner), dtype=dtype, device=proj.device)
+    if not proj.is_cuda:
+        _state_space_reference(proj, w, s, S, ring, cache, eps, out)
+        return out
+    if dtype not in (torch.bfloat16, torch.float32):
+        raise TypeError(f"bfloat16 or float32 activations expected, got {dtype}")
+    _rows(proj, dtype, T, s.columns, "proj")
+    slots = S.shape[0]
+    if tuple(S.shape[1:]) != (H, N, P) or S.dtype != torch.float32 or not S.is_contiguous() \
+            or tuple(ring.shape) != (slots, s.taps, s.channels) or ring.dtype != dtype or not ring.is_contiguous():
+        raise TypeError("state_space: the state does not have the layer's shape")
+    for t, n in ((w.conv, s.taps * s.channels), (w.conv_bias, s.channels), (w.dt_bias, H), (w.a_log, H), (w.skip, H), (w.norm, s.inner)):
+        if t.dtype != torch.float32 or t.numel() != n or not t.is_contiguous():
+            raise TypeError("state_space: weights beside the projections are contiguous fp32 tensors")
+    B = cache.context_lens.numel()
+    if B > slots:
+        raise ValueError("state_space: every sequence needs a state slot")
+    lib = _lib.get_lib()
+    cu, scratch, conv_out, pitch, longest = 0, None, None, 0, 1
+    if cache.is_prefill:
+        cu, longest = cache.cu_q_dev.data_ptr(), max(cache.q_lens_host, default=0)
+        scratch = torch.empty(lib.mfb_state_space_scratch_floats(T, H, P, N), dtype=torch.float32, device=proj.device)
+        pitch = s.channels + -s.channels % 8
+        conv_out = torch.empty((T, pitch), dtype=dtype, device=proj.device)
+    rc = lib.mfb_state_space(proj.data_ptr(), proj.stride(0), w.conv.data_ptr(), w.conv_bias.data_ptr(), w.dt_bias.data_ptr(),
+                             w.a_log.data_ptr(), w.skip.data_ptr(), w.norm.data_ptr(), ring.data_ptr(), S.data_ptr(), cu,
+                             cache.context_lens.data_ptr(), cache.slot_mapping.data_ptr(), _lib.ptr(scratch), _lib.ptr(conv_out),
+                             out.data_ptr(), pitch, T, B, H, P, N, s.groups, s.taps, s.norm_groups, longest, float(eps),
+                             int(dtype == torch.float32), _lib.stream_ptr())
+    _lib.check(rc, "mfb_state_space")
+    _lib.count_launch(4 if cache.is_prefill else 2)
     return out

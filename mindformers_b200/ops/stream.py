@@ -213,6 +213,94 @@ def normed_step(x: torch.Tensor, y: Optional[torch.Tensor], w_in: Optional[torch
     return h, (x if same else out) if keep else None
 
 
+@dataclass
+class InputConv:
+    """Causal convolution of one layer run: ``w [taps, W]`` fp32 (the last row meets the current token) and the cache that keeps
+    the last ``taps - 1`` rows per sequence slot."""
+    w: torch.Tensor
+    cache: object
+    run: int
+
+    def rows(self, before: bool = False):
+        """``[slots, taps - 1, W]`` of this run (``before``: as they were before a prefill step)."""
+        t = self.cache.carry_before if before else self.cache.carry
+        taps, W = self.w.shape
+        return None if t is None else t[self.run].view(-1, taps - 1, W)
+
+
+def _input_conv_reference(h, conv: InputConv):
+    from .recurrent import _sequences
+    out, (taps, W) = h.clone(), conv.w.shape
+    state = conv.rows()
+    for slot, r0, n, start in _sequences(conv.cache, h.shape[0]):
+        seq = h[r0:r0 + n]
+        if taps > 1:
+            first = state[slot] if start > 0 else torch.zeros_like(state[slot])
+            seq = torch.cat((first, seq))
+            state[slot] = seq[n:]
+        out[r0:r0 + n] = h[r0:r0 + n] + sum(seq[j:j + n] * conv.w[j] for j in range(taps))
+    return out
+
+
+def grouped_norm_reference(x, w, groups, eps):
+    """fp32 RMS norm of ``groups`` neighbouring parts of the last axis, each by its own root mean square."""
+    parts = x.float().unflatten(-1, (groups, -1))
+    return (parts * torch.rsqrt(parts.pow(2).mean(-1, keepdim=True) + eps)).flatten(-2) * w.float()
+
+
+def joint_step(x: torch.Tensor, ys, base: Optional[torch.Tensor], step: Optional[torch.Tensor], w: Optional[torch.Tensor],
+               groups: int, eps: float, dtype: torch.dtype, conv: Optional[InputConv] = None, want_h: bool = True,
+               keep: bool = True) -> Tuple[Optional[torch.Tensor], Optional[torch.Tensor], Optional[torch.Tensor]]:
+    """One step of an fp32 residual stream ``x [T, W]`` whose sub-layers run side by side: ``x' = x + sum(ys) + base + step``
+    (``ys``: up to two outputs in the activation dtype; ``base [T, W]`` fp32; ``step [W]``; all optional), ``h`` its RMS norm in
+    ``groups`` parts times ``w`` (``w`` None: ``x'`` itself) and, with ``conv``, ``h + conv(h)``: a causal convolution per channel
+    (zeros before the first token; the last rows of a portion stay in ``cache.carry``).
+
+    Returns ``(h, h + conv(h), x')``, the first two in ``dtype``; ``want_h=False`` / ``keep=False`` drop ``h`` / ``x'``. ``x`` is
+    not changed."""
+    T, W = x.shape
+    ys = [y for y in ys if y is not None]
+    if not x.is_cuda:
+        for t in ys + [base, step]:
+            x = x if t is None else x + t.float()
+        h = x if w is None else grouped_norm_reference(x, w, groups, eps)
+        hc = None if conv is None else _input_conv_reference(h, conv).to(dtype)
+        return (h.to(dtype) if want_h else None), hc, (x if keep else None)
+    _check_dtype(dtype)
+    _typed(step, w, dtype=dtype)
+    if x.dtype != torch.float32 or not x.is_contiguous() or len(ys) > 2 or any(
+            y.dtype != dtype or y.shape != (T, W) or y.stride(1) != 1 for y in ys) or (base is not None and (
+            base.dtype != torch.float32 or base.shape != (T, W) or base.stride(1) != 1)):
+        raise TypeError("joint_step: a contiguous fp32 stream and sub-layer outputs in the activation dtype expected")
+    h = torch.empty((T, W), dtype=dtype, device=x.device) if want_h else None
+    hc = torch.empty((T, W), dtype=dtype, device=x.device) if conv is not None else None
+    same = not ys and base is None and step is None
+    out = torch.empty_like(x) if keep and not same else None
+    B, cu, lens, slots, before, after, taps = 0, 0, 0, 0, 0, 0, 0
+    if conv is not None:
+        c, taps = conv.cache, conv.w.shape[0]
+        B = c.context_lens.numel()
+        if conv.w.dtype != torch.float32 or conv.w.shape[1] != W or not conv.w.is_contiguous():
+            raise TypeError("joint_step: the convolution's weights are a contiguous fp32 [taps, W] tensor")
+        cu = c.cu_q_dev.data_ptr() if c.is_prefill else 0
+        lens, slots = c.context_lens.data_ptr(), c.slot_mapping.data_ptr()
+        if taps > 1:
+            state = conv.rows()
+            if B > state.shape[0]:
+                raise ValueError("joint_step: a sequence has no slot")
+            after = state.data_ptr()
+            before = conv.rows(before=True).data_ptr() if c.is_prefill else after
+    y0, y1 = (ys + [None, None])[:2]
+    rc = _lib.get_lib().mfb_joint_step(
+        x.data_ptr(), _lib.ptr(y0), 0 if y0 is None else y0.stride(0), _lib.ptr(y1), 0 if y1 is None else y1.stride(0),
+        _lib.ptr(base), 0 if base is None else base.stride(0), _lib.ptr(step), _lib.ptr(w), _lib.ptr(out), _lib.ptr(h), _lib.ptr(hc),
+        None if conv is None else conv.w.data_ptr(), before, after, cu, lens, slots, T, W, B, int(groups), taps, float(eps),
+        int(dtype == torch.float32), _lib.stream_ptr())
+    _lib.check(rc, "mfb_joint_step")
+    _lib.count_launch()
+    return h, hc, (x if same else out) if keep else None
+
+
 def relu2(x: torch.Tensor) -> torch.Tensor:
     """``max(x, 0)^2``"""
     if not x.is_cuda or (torch.is_grad_enabled() and x.requires_grad):
@@ -338,27 +426,54 @@ def qkv_rope_cache(qkv: torch.Tensor, bias: Optional[torch.Tensor], q_norm: Opti
 
 
 def latent_norm_cache(proj: torch.Tensor, q_norm: torch.Tensor, kv_norm: torch.Tensor, eps: float, slots: torch.Tensor,
-                      cache: torch.Tensor) -> torch.Tensor:
-    """Between the down projections of latent attention and what follows: ``proj [T, >= Q + R]`` (query latent | key / value
-    latent, any row pitch) → the RMS-normed query latent ``[T, Q]``; the normed key / value latent goes to the rows ``slots`` of
-    ``cache [.., R]`` (negative: not written)."""
+                      cache: torch.Tensor, freqs: Optional[torch.Tensor] = None, positions: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Between the down projections of latent attention and what follows: ``proj [T, >= Q + R + P]`` (query latent | key / value
+    latent | key part with positions, any row pitch) → the RMS-normed query latent ``[T, Q]``; the normed key / value latent and,
+    with ``freqs [P / 2]``, the last part rotated (neighbouring dimensions, by ``position * freqs``) go to the rows ``slots`` of
+    ``cache [.., R + P]`` (negative: not written)."""
     T, dtype, Q, R = proj.shape[0], proj.dtype, q_norm.numel(), kv_norm.numel()
+    P = 0 if freqs is None else 2 * freqs.numel()
     if not proj.is_cuda:
         c = norm_reference(proj[:, Q:Q + R], kv_norm, None, eps, False)
+        if P:
+            k = _rotate_reference(proj[:, None, Q + R:Q + R + P].float(), positions, freqs, 1.0, P, True)[:, 0]
+            c = torch.cat((c, k), dim=1)
         keep = slots >= 0
-        cache.view(-1, R)[slots[keep].long()] = c[keep].to(cache.dtype)
+        cache.view(-1, R + P)[slots[keep].long()] = c[keep].to(cache.dtype)
         return norm_reference(proj[:, :Q], q_norm, None, eps, False).to(dtype)
     _check_dtype(dtype)
     _typed(q_norm, kv_norm, cache, dtype=dtype)
-    if proj.stride(1) != 1 or proj.shape[1] < Q + R or slots.dtype != torch.int32 or slots.numel() != T or cache.shape[-1] != R:
+    if proj.stride(1) != 1 or proj.shape[1] < Q + R + P or slots.dtype != torch.int32 or slots.numel() != T \
+            or cache.shape[-1] != R + P or (P and (freqs.dtype != torch.float32 or positions.dtype != torch.int64
+                                                   or positions.numel() != T or not positions.is_contiguous())):
         raise TypeError("latent_norm_cache: unexpected shapes or dtypes")
     q = torch.empty((T, Q), dtype=dtype, device=proj.device)
     rc = _lib.get_lib().mfb_latent_norm_cache(proj.data_ptr(), proj.stride(0), q_norm.data_ptr(), kv_norm.data_ptr(), float(eps),
-                                              slots.data_ptr(), q.data_ptr(), cache.data_ptr(), T, Q, R,
+                                              slots.data_ptr(), q.data_ptr(), cache.data_ptr(), _lib.ptr(freqs),
+                                              _lib.ptr(positions) if P else 0, T, Q, R, P,
                                               int(dtype == torch.float32), _lib.stream_ptr())
     _lib.check(rc, "mfb_latent_norm_cache")
     _lib.count_launch()
     return q
+
+
+def rotate_tail_(x: torch.Tensor, freqs: torch.Tensor, positions: torch.Tensor) -> torch.Tensor:
+    """The last ``2 * len(freqs)`` dimensions of every head of ``x [T, heads, dim]`` rotated by ``position * freqs`` (neighbouring
+    dimensions are pairs), in place."""
+    T, H, D = x.shape
+    P = 2 * freqs.numel()
+    if not x.is_cuda:
+        x[..., D - P:] = _rotate_reference(x[..., D - P:].float(), positions, freqs, 1.0, P, True).to(x.dtype)
+        return x
+    _check_dtype(x.dtype)
+    if not x.is_contiguous() or P > D or freqs.dtype != torch.float32 or positions.dtype != torch.int64 or positions.numel() != T \
+            or not positions.is_contiguous():
+        raise TypeError("rotate_tail_: contiguous heads, fp32 frequencies and int64 positions expected")
+    rc = _lib.get_lib().mfb_rotate_tail(x.data_ptr(), freqs.data_ptr(), positions.data_ptr(), T, H, D, P,
+                                        int(x.dtype == torch.float32), _lib.stream_ptr())
+    _lib.check(rc, "mfb_rotate_tail")
+    _lib.count_launch()
+    return x
 
 
 def gate_heads_(x: torch.Tensor, gate: torch.Tensor) -> torch.Tensor:

@@ -92,11 +92,11 @@ def moe_local_enabled(config, x: torch.Tensor) -> bool:
     return not _FORCE_OFF and fused_moe.local_supported(config, x)
 
 
-def moe_local(layer, hidden, probs, ids):
+def moe_local(layer, hidden, probs, ids, extra=None):
     from . import fused_moe
-    return fused_moe.moe_local(layer, hidden, probs, ids)
+    return fused_moe.moe_local(layer, hidden, probs, ids, extra)
 
 
-def moe_dispatch_experts_combine(layer, hidden, probs, ids):
+def moe_dispatch_experts_combine(layer, hidden, probs, ids, extra=None):
     from . import fused_moe
-    return fused_moe.moe_dispatch_experts_combine(layer, hidden, probs, ids)
+    return fused_moe.moe_dispatch_experts_combine(layer, hidden, probs, ids, extra)

@@ -232,12 +232,14 @@ class MoEExchange:
             _lib.check(rc, "mfb_moe_barrier")
             _lib.count_launch()
 
-    def gather(self, st, T, ids, peer_ptrs, weights=None, g=None):
+    def gather(self, st, T, ids, peer_ptrs, weights=None, g=None, own=None, extra=None):
+        """``own [T, H]``: the rows of copies for identity experts; ``extra [T, H]`` (any row pitch) is added to the result."""
         out = torch.empty(T, self.H, dtype=torch.bfloat16, device=self.dev)
         dots = torch.empty(T, self.k, dtype=torch.float32, device=self.dev) if g is not None else None
         rc = self.lib.mfb_moe_gather(self.world, self.rank, T, self.k, self.H, self.E_local, st.rows, out.data_ptr(),
                                      ids.data_ptr(), st.dest_row.data_ptr(), peer_ptrs, _lib.ptr(weights), _lib.ptr(g),
-                                     _lib.ptr(dots), self.status(), _lib.stream_ptr())
+                                     _lib.ptr(dots), _lib.ptr(own), _lib.ptr(extra), 0 if extra is None else extra.stride(0),
+                                     self.status(), _lib.stream_ptr())
         _lib.check(rc, "mfb_moe_gather")
         _lib.count_launch()
         return out, dots
@@ -293,7 +295,7 @@ class _Combine(torch.autograd.Function):
     """Expert output rows ``[rows, H]`` + ``probs [T,k]`` → ``[T,H]`` (receive + weighted unpermute)."""
 
     @staticmethod
-    def forward(ctx, y, probs, ids, ex: MoEExchange, st: _PlanState, layer_key, unweighted=False):
+    def forward(ctx, y, probs, ids, ex: MoEExchange, st: _PlanState, layer_key, unweighted=False, own=None, extra=None):
         T = probs.shape[0]
         probs = probs.contiguous().float()
         if ex.world > 1:
@@ -303,7 +305,7 @@ class _Combine(torch.autograd.Function):
         else:
             yout, ptrs = y.contiguous(), None
             ptrs = ex.local_ptrs(yout)
-        out, _ = ex.gather(st, T, ids, ptrs, weights=None if unweighted else probs)
+        out, _ = ex.gather(st, T, ids, ptrs, weights=None if unweighted else probs, own=own, extra=extra)
         ctx.ex, ctx.st, ctx.T, ctx.ptrs = ex, st, T, ptrs
         ctx.save_for_backward(ids, probs, yout)
         return out
@@ -324,7 +326,7 @@ class _Combine(torch.autograd.Function):
         ex.barrier(1)
         # peers overwrite dy_ws only after this rank has passed the barrier of this layer's dispatch backward,
         # which comes after the expert GEMMs that consume it
-        return dy, dots, None, None, None, None, None
+        return dy, dots, None, None, None, None, None, None, None
 
 
 def supported(config, hidden: torch.Tensor) -> bool:
@@ -338,9 +340,18 @@ def local_supported(config, hidden: torch.Tensor) -> bool:
             and config.num_moe_experts <= 512 and ps.get_expert_model_parallel_world_size() == 1)
 
 
-def moe_local(layer, hidden: torch.Tensor, probs: torch.Tensor, ids: torch.Tensor) -> torch.Tensor:
+def _self_rows(cfg, hidden: torch.Tensor) -> Optional[torch.Tensor]:
+    """What copies for identity experts stand for (None: the router has no such outputs)."""
+    if not cfg.moe_identity_experts:
+        return None
+    if cfg.moe_apply_probs_on_input:
+        raise NotImplementedError("identity experts beside routing weights on the experts' input")
+    return hidden
+
+
+def moe_local(layer, hidden: torch.Tensor, probs: torch.Tensor, ids: torch.Tensor, extra: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Router outputs → combined expert outputs on one rank: the exchange's permutation plan with kernels for every width
-    and for 32-bit activations (``ops/csrc/moe_any.cu``)."""
+    and for 32-bit activations (``ops/csrc/moe_any.cu``). ``extra [T, H]`` is added to the result."""
     cfg = layer.config
     ex = MoEExchange.get(cfg)
     ids, hidden, probs = ids.contiguous(), hidden.contiguous(), probs.contiguous().float()
@@ -351,20 +362,23 @@ def moe_local(layer, hidden: torch.Tensor, probs: torch.Tensor, ids: torch.Tenso
     rows = torch.empty((st.rows, H), dtype=hidden.dtype, device=hidden.device)
     rc = ex.lib.mfb_moe_scatter_any(hidden.data_ptr(), ids.data_ptr(), st.rank_in_e.data_ptr(), st.write_base.data_ptr(),
                                     probs.data_ptr() if on_input else None, rows.data_ptr(), st.dest_row.data_ptr(), T, ex.k, H,
-                                    st.rows, f32, _lib.stream_ptr())
+                                    ex.E, st.rows, f32, _lib.stream_ptr())
     _lib.check(rc, "mfb_moe_scatter_any")
     layer.last_tokens_per_expert = st.counts
     y = layer.experts(rows, st.plan)
     out = torch.empty_like(hidden)
-    rc = ex.lib.mfb_moe_gather_any(y.data_ptr(), st.dest_row.data_ptr(), None if on_input else probs.data_ptr(), out.data_ptr(), T,
-                                   ex.k, H, f32, _lib.stream_ptr())
+    rc = ex.lib.mfb_moe_gather_any(y.data_ptr(), st.dest_row.data_ptr(), None if on_input else probs.data_ptr(), ids.data_ptr(),
+                                   _lib.ptr(_self_rows(cfg, hidden)), _lib.ptr(extra), 0 if extra is None else extra.stride(0),
+                                   out.data_ptr(), T, ex.k, H, ex.E, f32, _lib.stream_ptr())
     _lib.check(rc, "mfb_moe_gather_any")
     _lib.count_launch(2)
     return out
 
 
-def moe_dispatch_experts_combine(layer, hidden: torch.Tensor, probs: torch.Tensor, ids: torch.Tensor) -> torch.Tensor:
-    """Router outputs → combined expert outputs ``[T, H]`` through the fused exchange."""
+def moe_dispatch_experts_combine(layer, hidden: torch.Tensor, probs: torch.Tensor, ids: torch.Tensor,
+                                 extra: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Router outputs → combined expert outputs ``[T, H]`` through the fused exchange; forward-only calls may have ``extra [T, H]``
+    added to them."""
     ex = MoEExchange.get(layer.config)
     ids = ids.contiguous()
     st = ex.plan(ids, hidden.shape[0])
@@ -378,11 +392,16 @@ def moe_dispatch_experts_combine(layer, hidden: torch.Tensor, probs: torch.Tenso
     on_input = bool(layer.config.moe_apply_probs_on_input)
     if on_input and needs_grad:
         raise NotImplementedError("routing weights on the experts' input have no backward pass")
+    own = _self_rows(layer.config, hidden)
+    if own is not None:
+        if needs_grad:
+            raise NotImplementedError("identity experts have no backward pass")
+        own = own.contiguous()
     weights = probs.contiguous().float() if on_input else None
     xin = apply_fn(_Dispatch, hidden, ids, ex, st, key, weights)
     layer.last_tokens_per_expert = st.counts
     y = layer.experts(xin, st.plan)
-    out = apply_fn(_Combine, y, probs, ids, ex, st, key, on_input)
+    out = apply_fn(_Combine, y, probs, ids, ex, st, key, on_input, own, extra)
     if not needs_grad:
         ex.release_slot(*st.slot)
     return out

@@ -39,6 +39,8 @@ class AttnMeta:
     layer_run: Optional[int] = None       # position of the running layer in the stack (its cache; layers that share
                                           # weights run more than once)
     loop_step: Optional[torch.Tensor] = None   # vector that enters the residual stream before the running layer
+    loop_entry: Optional[tuple] = None    # (matrix [W, W] on the stream, its part from the embedding output [T, W] fp32) of the
+                                          # passes of a loop whose layers start from both
     cp_rank_positions: bool = False       # positions already hold the context-parallel offsets
 
 

@@ -20,8 +20,9 @@ from .moe import GroupedMLP, MoELayer, SharedExpertMLP, TopKRouter
 from .mtp import MultiTokenPredictionBlock, MultiTokenPredictionLayer
 from .norm import build_norm
 from .ragged_attention import RaggedLatentAttention, RaggedSelfAttention
-from .transformer_layer import (OutputNormTransformerLayer, SandwichTransformerLayer, StreamTransformerLayer, TransformerLayer,
-                                TransformerLayerSubmodules)
+from .state_space import StateSpaceMixer
+from .transformer_layer import (OutputNormTransformerLayer, ParallelTransformerLayer, SandwichTransformerLayer,
+                                StreamTransformerLayer, TransformerLayer, TransformerLayerSubmodules)
 
 
 def get_moe_module_spec(num_experts: Optional[int] = None, moe_grouped_gemm: bool = True) -> ModuleSpec:
@@ -68,7 +69,7 @@ def get_output_norm_layer_spec(config) -> ModuleSpec:
 
 
 _MIXERS = {"attention": RaggedSelfAttention, "latent": RaggedLatentAttention, "delta": GatedDeltaMixer,
-           "matrix_memory": MatrixMemoryMixer, "parallel": ParallelMixer}
+           "matrix_memory": MatrixMemoryMixer, "state_space": StateSpaceMixer, "parallel": ParallelMixer}
 
 
 def get_stream_layer_spec(config, is_moe: bool) -> ModuleSpec:
@@ -92,6 +93,14 @@ def get_sandwich_layer_spec(config, is_moe: bool) -> ModuleSpec:
         pre_mlp_layernorm=after, post_mlp_layernorm=after))
 
 
+def get_parallel_layer_spec(config, is_moe: bool) -> ModuleSpec:
+    """Spec of one layer whose sub-layers read one norm: ``config.mixer`` beside an MoE or dense feed-forward (none with
+    ``ffn_hidden_size == 0``)."""
+    mlp = get_mlp_module_spec(config.num_moe_experts if is_moe else None) if is_moe or config.ffn_hidden_size else None
+    return ModuleSpec(module=ParallelTransformerLayer, submodules=TransformerLayerSubmodules(
+        input_layernorm=ModuleSpec(module=build_norm), self_attention=ModuleSpec(module=_MIXERS[config.mixer]), mlp=mlp))
+
+
 def get_gpt_layer_spec_for_config(config, is_moe: bool) -> ModuleSpec:
     """``get_gpt_layer_local_spec`` with the switches taken from a ``TransformerConfig``."""
     if config.residual_streams:
@@ -102,6 +111,10 @@ def get_gpt_layer_spec_for_config(config, is_moe: bool) -> ModuleSpec:
         if not config.ragged_attention or config.normalization != "RMSNorm":
             raise ValueError("layers with norms on both sides are built with ragged attention and RMS norms")
         return get_sandwich_layer_spec(config, is_moe)
+    if config.norm_placement == "parallel":
+        if not config.ragged_attention or config.normalization != "RMSNorm" or config.layernorm_zero_centered_gamma:
+            raise ValueError("layers whose sub-layers run side by side are built with ragged attention and plain RMS norms")
+        return get_parallel_layer_spec(config, is_moe)
     if config.norm_placement == "output":
         if is_moe or not config.ragged_attention:
             raise ValueError("output-normalised layers are built with ragged attention and a dense feed-forward")

@@ -37,9 +37,9 @@ class LanguageModelEmbedding(nn.Module):
         self.word_embeddings = VocabParallelEmbedding(config.vocab_size, config.hidden_size, config=config,
                                                       reduce_scatter_embeddings=sp)
         self.sp = sp
-        # an fp32 stream starts from scaled rows plus sinusoidal position vectors
+        # an fp32 stream starts from scaled rows plus, where configured, sinusoidal position vectors
         self.scale, self.sinusoidal = float(config.embedding_scale), config.position_embedding_type == "sinusoidal"
-        self.stream = self.sinusoidal or self.scale != 1.0
+        self.stream = self.sinusoidal or self.scale != 1.0 or config.norm_placement == "parallel"
         if self.stream:
             if not config.fp32_residual_connection or ps.get_tensor_model_parallel_world_size() > 1:
                 raise NotImplementedError("scaled or sinusoidal embeddings start an fp32 stream on one tensor-parallel rank")
@@ -114,7 +114,7 @@ class GPTModel(nn.Module):
         cap = self.config.logit_softcap
         if cap:          # fp32 accumulators -> cap * tanh(x / cap), element-wise (a vocabulary shard needs no other rank)
             return stream.linear(hidden, w, act="softcap", cap=float(cap))
-        if self.config.norm_placement == "both" and ps.get_tensor_model_parallel_world_size() == 1:
+        if self.config.norm_placement in ("both", "parallel") and ps.get_tensor_model_parallel_world_size() == 1:
             return stream.linear(hidden, w, out_dtype=torch.float32)
         y, _ = self.output_layer(hidden, weight=w)
         return y

@@ -49,12 +49,13 @@ class MLP(nn.Module):
             # a few rows: the activation runs in the epilogue of the up projection
             return self.linear_fc2(stream.linear(hidden, self.linear_fc1.weight, act="relu2"))
         x, _ = self.linear_fc1(hidden)
-        if self.gated and self.act_name in ("silu", "swiglu"):
-            x = Fn.swiglu(x)
-        elif self.gated:
-            g, u = x.chunk(2, dim=-1)
-            x = get_activation(self.act_name)(g) * u
-        else:
-            x = get_activation(self.act_name)(x)
-        out, bias = self.linear_fc2(x)
+        out, bias = self.linear_fc2(self._activate(x))
         return out, bias
+
+    def _activate(self, x):
+        if self.gated and self.act_name in ("silu", "swiglu"):
+            return Fn.swiglu(x)
+        if self.gated:
+            g, u = x.chunk(2, dim=-1)
+            return get_activation(self.act_name)(g) * u
+        return get_activation(self.act_name)(x)

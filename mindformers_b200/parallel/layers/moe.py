@@ -40,7 +40,8 @@ class TopKRouter(nn.Module):
     def __init__(self, config):
         super().__init__()
         self.config = config
-        E, H = config.num_moe_experts, config.hidden_size
+        # the last outputs stand for experts that return their input
+        E, H = config.num_moe_experts + config.moe_identity_experts, config.hidden_size
         dev = getattr(config, "device", None) or ("cuda" if torch.cuda.is_available() else "cpu")
         w = torch.empty(E, H, dtype=torch.float32, device=dev)
         default_init(config.init_method_std)(w)
@@ -86,7 +87,7 @@ class TopKRouter(nn.Module):
             z = torch.logsumexp(logits, dim=-1).pow(2).mean() * cfg.moe_z_loss_coeff
         else:
             z = None
-        E = cfg.num_moe_experts
+        E = self.weight.shape[0]
         want_aux = self.training and bool(cfg.moe_aux_loss_coeff)
         counts = None
         if self.training and (cfg.moe_aux_loss_coeff or self.expert_load is not None):
@@ -288,7 +289,8 @@ class GroupedMLP(nn.Module):
 
 
 class SharedExpertMLP(MLP):
-    """Always-on expert(s); optional sigmoid gate (reference ``shared_experts.py:30-124``)."""
+    """Always-on expert(s); optional sigmoid gate (reference ``shared_experts.py:30-124``). With ``moe_activation``
+    ``"clamped_glu"`` it has that activation, with a limit of its own where one is configured."""
 
     def __init__(self, config):
         super().__init__(config, ffn_hidden_size=config.moe_shared_expert_intermediate_size)
@@ -298,6 +300,13 @@ class SharedExpertMLP(MLP):
             self.gate_weight.sequence_parallel = bool(config.sequence_parallel)
         else:
             self.gate_weight = None
+
+    def _activate(self, x):
+        cfg = self.config
+        if cfg.moe_activation != "clamped_glu":
+            return super()._activate(x)
+        limit = cfg.moe_shared_expert_activation_limit
+        return Fn.clamped_glu(x.contiguous(), cfg.moe_activation_limit if limit is None else limit, cfg.moe_activation_alpha)
 
     def forward(self, hidden):
         out, _ = super().forward(hidden)
@@ -424,12 +433,22 @@ class MoELayer(nn.Module):
     def _forward_local(self, hidden, with_shared: bool = True):
         probs, ids, aux = self.router(hidden)
         from .. import fused_comm
+        with_shared = with_shared and self.shared_experts is not None
+        # forward-only calls add the shared expert where the copies are combined
+        inside = with_shared and not torch.is_grad_enabled()
         if not self.staged and fused_comm.moe_enabled(self.config, hidden):
-            out = fused_comm.moe_dispatch_experts_combine(self, hidden, probs, ids)
+            out = fused_comm.moe_dispatch_experts_combine(self, hidden, probs, ids, self.shared_experts(hidden) if inside else None)
+            with_shared = with_shared and not inside
         elif not self.staged and fused_comm.moe_local_enabled(self.config, hidden):
-            out = fused_comm.moe_local(self, hidden, probs, ids)
+            out = fused_comm.moe_local(self, hidden, probs, ids, self.shared_experts(hidden) if inside else None)
+            with_shared = with_shared and not inside
         else:
             T, k = ids.shape
+            own = None
+            if self.config.moe_identity_experts:          # copies for identity experts travel nowhere
+                at = ids >= self.config.num_moe_experts
+                own = hidden.float() * probs.float().masked_fill(~at, 0.0).sum(-1, keepdim=True)
+                probs, ids = probs.masked_fill(at, 0.0), ids.masked_fill(at, 0)
             if self.config.moe_apply_probs_on_input:      # every weighted copy is a token of its own
                 copies = (hidden.repeat_interleave(k, 0).float() * probs.reshape(-1, 1)).to(hidden.dtype)
                 x, plan, ctx = self.dispatcher.dispatch(copies, ids.reshape(-1, 1))
@@ -440,6 +459,8 @@ class MoELayer(nn.Module):
             out = self.dispatcher.combine(y, plan, ctx, probs.to(hidden.dtype))
             if self.config.moe_apply_probs_on_input:
                 out = out.view(T, k, -1).float().sum(1).to(hidden.dtype)
-        if with_shared and self.shared_experts is not None:
+            if own is not None:
+                out = (out.float() + own).to(hidden.dtype)
+        if with_shared:
             out = out + self.shared_experts(hidden)
         return out, aux

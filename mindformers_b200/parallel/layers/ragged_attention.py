@@ -124,10 +124,31 @@ class RaggedSelfAttention(RaggedAttentionCore):
         return self.linear_proj(self.attend(qkv, bias, meta))
 
 
+def expand_kv_up(w_uk: torch.Tensor, w_uv: torch.Tensor, heads: int, dim: int, rot: int) -> torch.Tensor:
+    """Factors of keys ``[heads * dim, rank]`` and values ``[heads * v_dim, rank]`` → rows that act on a cached latent with a rotated
+    key part of ``rot`` numbers behind it: a head's key rows are followed by ``rot`` unit vectors."""
+    rank = w_uk.shape[1]
+    k = w_uk.new_zeros(heads, dim + rot, rank + rot)
+    k[:, :dim, :rank] = w_uk.view(heads, dim, rank)
+    k[:, dim:, rank:] = torch.eye(rot, dtype=w_uk.dtype, device=w_uk.device)
+    return torch.cat((k.view(-1, rank + rot), torch.nn.functional.pad(w_uv, (0, rot))))
+
+
+def split_kv_up(w: torch.Tensor, heads: int, dim: int, rot: int, rank: int):
+    """Inverse of ``expand_kv_up``: ``(w_uk, w_uv)``."""
+    n = heads * (dim + rot)
+    return w[:n].view(heads, dim + rot, rank + rot)[:, :dim, :rank].reshape(heads * dim, rank), w[n:, :rank].contiguous()
+
+
 class RaggedLatentAttention(nn.Module):
-    """Latent attention without positions: queries through a normed latent, keys and values linear in one cached, normed latent
-    of ``kv_lora_rank`` numbers per token. Returns ``(output, None)``. One projection makes the query latent, the key / value
-    latent and the output gates; one kernel norms both latents and writes the cache (``ops/stream.py::latent_norm_cache``)."""
+    """Latent attention: queries through a normed latent, keys and values linear in one cached, normed latent of
+    ``kv_lora_rank`` numbers per token. With ``rotary_dim`` each head's query has as many dimensions more, which are rotated, and so
+    has its key: one rotated part for all heads, cached behind the latent. Returns ``(output, None)``.
+
+    One projection makes the query latent, the key / value latent, the rotated key part and the output gates; one kernel norms both
+    latents, rotates the key part and writes the cache (``ops/stream.py::latent_norm_cache``). The rows of ``linear_kv_up`` (keys,
+    then values, head by head) act on the whole cached row: those that make a key's rotated part are unit vectors, so that keys of
+    all heads, expanded or absorbed into the queries, are one product."""
 
     def __init__(self, config, layer_number: int = 1):
         super().__init__()
@@ -136,31 +157,42 @@ class RaggedLatentAttention(nn.Module):
         self.layer_number, self.eps = layer_number, config.layernorm_epsilon
         H, D, DV, Q, R = (config.num_attention_heads, config.kv_channels, config.v_channels or config.kv_channels, config.q_lora_rank,
                           config.kv_lora_rank)
-        self.heads, self.dim, self.v_dim, self.rank = H, D, DV, R
-        self.scale, self.window = config.softmax_scale or 1.0 / math.sqrt(D), int(config.attention_window or 0)
+        P = int(config.rotary_dim or 0)
+        if P % 2 or (P and not config.rotary_interleaved):
+            raise ValueError(f"layer {layer_number}: {P} rotary dimensions (an even number of interleaved ones)")
+        self.heads, self.dim, self.v_dim, self.rank, self.rot = H, D + P, DV, R, P
+        self.scale, self.window = config.softmax_scale or 1.0 / math.sqrt(D + P), int(config.attention_window or 0)
         gates = {None: 0, "head": H, "channel": H * DV}[config.attention_output_gate]
-        self.sections = (Q, R) + ((gates,) if gates else ())
+        self.sections = (Q, R + P) + ((gates,) if gates else ())
         linear = lambda cols, rows: ColumnParallelLinear(cols, rows, config=config, bias=False)
         self.linear_in = linear(config.hidden_size, sum(self.sections))
         self.q_latent_norm, self.kv_latent_norm = RMSNorm(config, Q, self.eps), RMSNorm(config, R, self.eps)
-        self.linear_q_up, self.linear_kv_up = linear(Q, H * D), linear(R, H * (D + DV))
+        self.linear_q_up, self.linear_kv_up = linear(Q, H * (D + P)), linear(R + P, H * (D + P + DV))
         dev = self.linear_in.weight.device
+        self.rotary = RotaryFrequencies(P, config.rotary_base, config.rope_scaling, device=dev) if P else None
+        if P:
+            if self.rotary.amplitude != 1.0:
+                raise NotImplementedError("the rotation of latent attention has no amplitude")
+            with torch.no_grad():
+                self.linear_kv_up.weight.copy_(expand_kv_up(*split_kv_up(self.linear_kv_up.weight, H, D, P, R), H, D, P))
         self.register_parameter("sink", nn.Parameter(torch.zeros(H, dtype=torch.float32, device=dev)) if config.attention_sink else None)
         self.linear_proj = RowParallelLinear(H * DV, config.hidden_size, config=config)
 
     def cache_shape(self):
-        return 1, self.rank, 0
+        return 1, self.rank + self.rot, 0
 
     def forward(self, hidden, rotary, meta: AttnMeta):
         from ...inference.ragged_attention import latent_attention
+        freqs = None if self.rotary is None else self.rotary.freqs
         cache, layer = meta.cache, cache_layer(meta, self.layer_number)
         proj, _ = self.linear_in(hidden)
         n = sum(self.sections[:2])
         c = stream.latent_norm_cache(proj[:, :n], self.q_latent_norm.weight, self.kv_latent_norm.weight, self.eps, cache.slot_mapping,
-                                     cache.key_cache[layer])
-        q, _ = self.linear_q_up(c)
-        out = latent_attention(q.view(-1, self.heads, self.dim), cache, layer, self.linear_kv_up.weight, self.v_dim, self.scale,
-                               self.window, self.sink)
+                                     cache.key_cache[layer], freqs, meta.positions)
+        q = self.linear_q_up(c)[0].contiguous().view(-1, self.heads, self.dim)
+        if freqs is not None:
+            q = stream.rotate_tail_(q, freqs, meta.positions)
+        out = latent_attention(q, cache, layer, self.linear_kv_up.weight, self.v_dim, self.scale, self.window, self.sink, self.rank)
         if len(self.sections) > 2:
             out = stream.gate_heads_(out, proj[:, n:])
         return self.linear_proj(out)

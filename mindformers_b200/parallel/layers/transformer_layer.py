@@ -258,6 +258,58 @@ class SandwichTransformerLayer(nn.Module):
         return pending, residual, aux if self.is_moe else None
 
 
+@dataclass
+class JointResidual:
+    """The fp32 stream and the mixer's output that has yet to enter it beside the pending one of the feed-forward."""
+    x: torch.Tensor
+    mixed: Optional[torch.Tensor] = None
+
+
+class ParallelTransformerLayer(nn.Module):
+    """Layer with an fp32 residual stream whose sub-layers read one norm and run side by side: ``x <- x + (mixer(h') + mlp(h))``
+    with ``h`` the RMS norm of ``x`` in ``config.norm_groups`` parts, and ``h' = h + conv(h)``, a causal convolution per channel,
+    with ``config.input_conv_taps`` (else ``h``). The feed-forward is dense, MoE or absent. A serving layer: entering the stream,
+    the next norm and the convolution are one kernel (``ops/stream.py::joint_step``), across layers too, since a layer's outputs
+    stay pending. Before the first layer of a pass of a loop, ``x <- W [x; embedding output] + step`` (``AttnMeta.loop_entry``)."""
+
+    joint_residual = True         # ``residual`` is a ``JointResidual`` that still lacks ``pending``
+
+    def __init__(self, config, layer_number: int = 1, submodules: Optional[TransformerLayerSubmodules] = None):
+        super().__init__()
+        self.config, self.layer_number = config, layer_number
+        self.input_layernorm = build_module(submodules.input_layernorm, config)
+        self.self_attention = build_module(submodules.self_attention, config, layer_number)
+        taps, w = int(config.input_conv_taps or 0), self.input_layernorm.weight
+        self.register_parameter("input_conv", nn.Parameter(torch.empty(taps, w.numel(), dtype=torch.float32, device=w.device)
+                                                           .normal_(0.0, 0.3)) if taps else None)
+        self.mlp, self.is_moe = None, False
+        if submodules.mlp is not None:
+            mlp_cls = getattr(submodules.mlp, "module", submodules.mlp)
+            self.is_moe = isinstance(mlp_cls, type) and issubclass(mlp_cls, MoELayer)
+            self.mlp = build_module(submodules.mlp, config, layer_number) if self.is_moe else build_module(submodules.mlp, config)
+
+    def forward(self, pending, residual: Optional[JointResidual], rotary, meta: AttnMeta):
+        x, ys = (pending, ()) if residual is None else (residual.x, (pending, residual.mixed))
+        norm, base, step = self.input_layernorm, None, meta.loop_step
+        dtype, groups = norm.weight.dtype, self.config.norm_groups
+        if meta.loop_step is not None and meta.loop_entry is not None:
+            w, base = meta.loop_entry
+            x, ys = stream.linear(stream.joint_step(x, ys, None, None, None, 1, 0.0, dtype, keep=False)[0], w,
+                                  out_dtype=torch.float32), ()
+        conv = None
+        if self.input_conv is not None:
+            if meta.cache is None:
+                raise RuntimeError("the convolution serves from a cache: generate() or the serving engine provide one")
+            conv = stream.InputConv(self.input_conv, meta.cache, meta.layer_run - meta.cache.layer_offset)
+        h, mixed, x = stream.joint_step(x, ys, base, step, norm.weight, groups, norm.eps, dtype, conv,
+                                        want_h=conv is None or self.mlp is not None)
+        mixed, _ = self.self_attention(h if conv is None else mixed, rotary, meta)
+        if self.mlp is None:
+            return mixed, JointResidual(x), None
+        pending, aux = self.mlp(h)
+        return pending, JointResidual(x, mixed), aux if self.is_moe else None
+
+
 def pipeline_layer_split(num_layers: int, pp: int, vpp: int = 1, offset=0) -> List[List[List[int]]]:
     """Layer ids of every (pp stage, virtual chunk). ``offset`` adds/removes layers per stage
     (list of pp values, or vpp lists of pp values), as the reference's ``LayerSetting`` does."""
@@ -340,6 +392,7 @@ class TransformerBlock(nn.Module):
         self.run_order, self.run_ids = [own_ids.index(o) for o in owners], list(self.layer_ids)
         self.run_steps = [None] * len(self.run_order)
         self.register_parameter("loop_step", None)
+        self.register_parameter("loop_in", None)
         if config.layer_loop is not None:
             if pp * vpp > 1:
                 raise NotImplementedError("looped layers stay on one pipeline stage")
@@ -347,9 +400,13 @@ class TransformerBlock(nn.Module):
             self.run_order, self.run_ids = [own_ids.index(i) for i, _ in runs], list(range(len(runs)))
             self.run_steps = [t for _, t in runs]
             with module_rng(base_seed, 90, dev):
-                self.loop_step = nn.Parameter(torch.empty(int(config.layer_loop[2]), config.hidden_size, dtype=torch.float32,
-                                                          device=dev or ("cuda" if torch.cuda.is_available() else "cpu"))
-                                              .normal_(0.0, config.init_method_std).to(config.params_dtype))
+                def rand(*shape):
+                    return nn.Parameter(torch.empty(*shape, dtype=torch.float32,
+                                                    device=dev or ("cuda" if torch.cuda.is_available() else "cpu"))
+                                        .normal_(0.0, config.init_method_std).to(config.params_dtype))
+                self.loop_step = rand(int(config.layer_loop[2]), config.hidden_size)
+                if config.loop_input:
+                    self.loop_in = rand(config.hidden_size, 2 * config.hidden_size)
         self.final_layernorm = build_norm(config) if post_process else None
         self.recompute = bool(config.recompute) if not isinstance(config.recompute, (list, tuple)) else True
         self._recompute_layers = self._resolve_recompute(config.recompute)
@@ -384,8 +441,11 @@ class TransformerBlock(nn.Module):
         return shapes if any(s is not None for s in shapes) else None
 
     def carry_width(self) -> int:
-        """Width of the vector that every layer run carries from one token of a sequence to the next (0: none)."""
-        return self.config.hidden_size if any(getattr(layer, "token_shift", None) is not None for layer in self.layers) else 0
+        """Width of the vector that every layer run carries from one token of a sequence to the next (0: none): one row of the
+        width for a token shift, ``taps - 1`` rows for a convolution in front of the mixers."""
+        rows = [1 if getattr(layer, "token_shift", None) is not None else 0 for layer in self.layers]
+        rows += [layer.input_conv.shape[0] - 1 for layer in self.layers if getattr(layer, "input_conv", None) is not None]
+        return self.config.hidden_size * max(rows, default=0)
 
     def _setup_selective_recompute_and_offload(self, config):
         from ..recompute import ActivationOffloader, mark_recompute_modules
@@ -445,6 +505,10 @@ class TransformerBlock(nn.Module):
         pending, residual, layer = hidden, None, None
         aux_total = None
         training = self.training and torch.is_grad_enabled()
+        if self.loop_in is not None:          # the embedding's part of every pass's first product
+            W, w = self.config.hidden_size, self.loop_in
+            x0 = stream.joint_step(hidden, (), None, None, None, 1, 0.0, w.dtype, keep=False)[0]
+            meta.loop_entry = (w[:, :W], stream.linear(x0, w[:, W:], out_dtype=torch.float32))
         if training and self._offload is not None:
             self._offload.prune()
         for idx, at in enumerate(self.run_order):
@@ -484,6 +548,12 @@ class TransformerBlock(nn.Module):
                 raise NotImplementedError("an fp32 stream with a pending norm stays on one pipeline stage")
             out, _ = stream.normed_step(residual.x, pending, residual.norm.weight, None, norm.weight, norm.eps,
                                         self.config.layernorm_zero_centered_gamma, keep=False)
+        elif getattr(layer, "joint_residual", False):
+            norm = self.final_layernorm
+            if norm is None:
+                raise NotImplementedError("an fp32 stream with pending outputs stays on one pipeline stage")
+            out = stream.joint_step(residual.x, (pending, residual.mixed), None, None, norm.weight, self.config.norm_groups, norm.eps,
+                                    norm.weight.dtype, keep=False)[0]
         elif getattr(layer, "stream_in_residual", False):
             norm = self.final_layernorm
             out = residual if norm is None else stream.norm_stream(residual, norm.weight, getattr(norm, "bias", None), norm.eps,

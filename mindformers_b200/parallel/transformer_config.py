@@ -133,15 +133,28 @@ class TransformerConfig(ModelParallelConfig):
     # per layer, the index of the layer whose weights it uses (its own index: weights of its own); None: no sharing
     layer_sharing: Optional[List[int]] = None
     norm_placement: str = "input"           # "input": pre-norm; "output": x + scale * norm(sublayer(x)), fp32 stream;
-                                            # "both": x + norm(sublayer(norm(x))), fp32 stream
+                                            # "both": x + norm(sublayer(norm(x))), fp32 stream; "parallel": x + mixer(h) +
+                                            # mlp(h) with h = norm(x), fp32 stream
+    norm_groups: int = 1                    # norm_placement "parallel": parts of the width with a root mean square each
+    input_conv_taps: int = 0                # norm_placement "parallel": a mixer reads h + conv(h), a causal convolution of
+                                            # that many taps per channel
+    loop_input: bool = False                # layer_loop: a pass starts from a learned [W, 2 W] matrix on the stream and the
+                                            # embedding output
     layer_loop: Optional[tuple] = None      # (start, stop, times): these layers are repeated, all passes on one set of
                                             # weights; before pass t a learned vector (row t) is added to the stream
     token_shift: bool = False               # norm_placement "both": a mixer reads h + (h of the token before - h) * mu
     embedding_scale: float = 1.0            # factor of the embedding rows (fp32 streams)
     residual_streams: int = 0               # > 0: that many fp32 streams with learned reads, writes and mixing (pre-norm)
-    mixer: str = "attention"                # with residual_streams or norm_placement "both": "attention", "latent" (cached
-                                            # latents), "delta" (gated delta rule), "matrix_memory" (mLSTM) or "parallel"
-                                            # (attention beside a gated delta rule, both on the same input)
+    mixer: str = "attention"                # with residual_streams or norm_placement "both" / "parallel": "attention", "latent"
+                                            # (cached latents), "delta" (gated delta rule), "matrix_memory" (mLSTM),
+                                            # "state_space" (Mamba-2) or "parallel" (attention beside a gated delta rule, both
+                                            # on the same input)
+    ssm_heads: int = 0                      # state space: heads,
+    ssm_head_dim: int = 0                   #   channels per head,
+    ssm_state: int = 0                      #   size of the state per channel,
+    ssm_groups: int = 1                     #   groups of heads that share B and C,
+    ssm_conv_taps: int = 4                  #   taps of the short convolution,
+    ssm_norm_groups: int = 1                #   parts of the read-out with a root mean square each
     memory_heads: int = 0                   # matrix memory: heads, sizes per head and the soft cap of its gates
     memory_key_dim: int = 0
     memory_value_dim: int = 0
@@ -234,6 +247,7 @@ class TransformerConfig(ModelParallelConfig):
     moe_router_dtype: Union[str, torch.dtype] = "float32"   # of the router's weight ("params": params_dtype); 16-bit products
                                             # are accumulated in, and the logits are, 32-bit
     moe_router_enable_expert_bias: bool = False
+    moe_identity_experts: int = 0           # the router's last outputs stand for experts that return their input
     moe_router_logit_bias: bool = False     # learned bias of the router's logits (selection and weights)
     moe_router_bias_update_rate: float = 1e-3
     moe_grouped_gemm: bool = True
@@ -248,6 +262,7 @@ class TransformerConfig(ModelParallelConfig):
     moe_activation: str = "swiglu"          # "swiglu" or "clamped_glu": g sigmoid(alpha g) (u + 1), g and u clamped
     moe_activation_limit: float = 7.0       #   at this limit (g from above only)
     moe_activation_alpha: float = 1.702
+    moe_shared_expert_activation_limit: Optional[float] = None   # limit of the shared expert (None: moe_activation_limit)
     moe_token_dispatcher_type: str = "alltoall"
     use_allgather_dispatcher: bool = False
     kv_cache_dtype: Optional[str] = None    # "int8": paged KV cache in int8 with per-token, per-head scales
@@ -340,8 +355,8 @@ class TransformerConfig(ModelParallelConfig):
         if self.num_moe_experts:
             if self.moe_ffn_hidden_size is None:
                 self.moe_ffn_hidden_size = self.ffn_hidden_size
-            if self.moe_router_topk < 1 or self.moe_router_topk > self.num_moe_experts:
-                raise ValueError("moe_router_topk must lie in [1, num_moe_experts]")
+            if self.moe_router_topk < 1 or self.moe_router_topk > self.num_moe_experts + self.moe_identity_experts:
+                raise ValueError("moe_router_topk must lie in [1, num_moe_experts + moe_identity_experts]")
             if self.num_moe_experts % self.expert_model_parallel_size != 0:
                 raise ValueError("num_moe_experts must be a multiple of expert_model_parallel_size")
             if self.moe_router_topk_scaling_factor is None:
@@ -357,12 +372,17 @@ class TransformerConfig(ModelParallelConfig):
                 self.moe_aux_loss_coeff = float(self.aux_loss_factors[self.aux_loss_types.index("expert")])
         elif self.expert_model_parallel_size > 1:
             raise ValueError("expert_model_parallel_size > 1 needs num_moe_experts")
-        if self.mixer not in ("attention", "latent", "delta", "matrix_memory", "parallel") or self.delta_decay not in ("head", "channel") \
+        if self.mixer not in ("attention", "latent", "delta", "matrix_memory", "state_space", "parallel") \
+                or self.delta_decay not in ("head", "channel") \
                 or self.delta_gate not in ("silu", "sigmoid") or self.moe_activation not in ("swiglu", "clamped_glu"):
             raise ValueError(f"unknown mixer {self.mixer!r}, decay {self.delta_decay!r}, gate {self.delta_gate!r} or expert "
                              f"activation {self.moe_activation!r}")
-        if self.norm_placement not in ("input", "output", "both"):
-            raise ValueError(f"norm_placement must be 'input', 'output' or 'both', got {self.norm_placement!r}")
+        if self.norm_placement not in ("input", "output", "both", "parallel"):
+            raise ValueError(f"norm_placement must be 'input', 'output', 'both' or 'parallel', got {self.norm_placement!r}")
+        if self.norm_placement != "parallel" and (self.norm_groups != 1 or self.input_conv_taps or self.loop_input):
+            raise ValueError("norm_groups, input_conv_taps and loop_input belong to norm_placement 'parallel'")
+        if self.norm_groups < 1 or self.hidden_size % self.norm_groups:
+            raise ValueError(f"width {self.hidden_size} does not divide into {self.norm_groups} parts")
         if self.attention_output_gate not in (None, "channel", "head"):
             raise ValueError(f"attention_output_gate must be None, 'channel' or 'head', got {self.attention_output_gate!r}")
         if self.layer_loop is not None:
