@@ -115,11 +115,12 @@ def main():
     ap.add_argument("--tp", type=int, default=None)
     ap.add_argument("--recompute", type=int, default=0, help="recompute the activations of the first N layers in backward")
     ap.add_argument("--config", default="llama8b", choices=["llama8b", "qwen3_moe", "qwen25_cp", "mefesun_serving", "kukupel_serving",
-                                                             "gavatar_serving"],
+                                                             "gavatar_serving", "togalorn_serving"],
                     help="llama8b: the headline (Llama-3.1-8B, TP2+SP x DP); qwen3_moe: Qwen3-30B-A3B, expert parallel = N, "
                          "micro batch 1; qwen25_cp: Qwen2.5-7B, one sequence of --seq-len tokens, context parallel = N; "
                          "mefesun_serving: prefill and decode throughput of Mefesun beside Qwen3 at equal size (one GPU); "
-                         "kukupel_serving: the same of Kukupel beside Qwen3-MoE; gavatar_serving: the same of Gavatar beside Kukupel")
+                         "kukupel_serving: the same of Kukupel beside Qwen3-MoE; gavatar_serving: the same of Gavatar beside Kukupel; "
+                         "togalorn_serving: the same of Togalorn beside Gavatar")
     args = ap.parse_args()
     if args.config == "qwen3_moe" and args.model == "llama3_1_8b":
         args.model = "qwen3_30b_a3b"
@@ -130,13 +131,15 @@ def main():
         args.seqs_per_gpu = 1
     if args.impl == "reference":
         return reference_arm(args)
-    if args.config in ("mefesun_serving", "kukupel_serving", "gavatar_serving"):
+    if args.config in ("mefesun_serving", "kukupel_serving", "gavatar_serving", "togalorn_serving"):
         import torch
 
         if args.config == "mefesun_serving":
             from benchmarks.bench_ragged_serving import main as serving
         elif args.config == "kukupel_serving":
             from benchmarks.bench_recurrent_serving import main as serving
+        elif args.config == "togalorn_serving":
+            from benchmarks.bench_joint_serving import main as serving
         else:
             from benchmarks.bench_loop_serving import main as serving
         if args.gpus != 1:

@@ -21,7 +21,9 @@ __device__ __forceinline__ void st2(float* p, float a, float b) { *reinterpret_c
 __device__ __forceinline__ void st2(__nv_bfloat16* p, float a, float b) {
   *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(a, b);
 }
-__device__ __forceinline__ float sigmoid(float z) { return 1.f / (1.f + __expf(-z)); }
+// 16-bit results take the fast exponential
+template <typename T>
+__device__ __forceinline__ float sigmoid(float z) { return 1.f / (1.f + (sizeof(T) == 2 ? __expf(-z) : expf(-z))); }
 
 // (u, v) turned by the angle position * freq
 __device__ __forceinline__ void rotate(float& u, float& v, long long position, float freq) {
@@ -177,9 +179,9 @@ gate_heads_kernel(T* __restrict__ x, long long ld_x, const T* __restrict__ gate,
     const T* g = gate + t * ld_g;
     if constexpr (VEC == 2) {
       const float2 v = ld2(p);
-      st2(p, v.x * sigmoid(ld(g + c / per)), v.y * sigmoid(ld(g + (c + 1) / per)));
+      st2(p, v.x * sigmoid<T>(ld(g + c / per)), v.y * sigmoid<T>(ld(g + (c + 1) / per)));
     } else {
-      st(p, ld(p) * sigmoid(ld(g + c / per)));
+      st(p, ld(p) * sigmoid<T>(ld(g + c / per)));
     }
   }
 }
@@ -198,12 +200,12 @@ gate_heads_vec_kernel(__nv_bfloat16* __restrict__ x, long long ld_x, const __nv_
     const __nv_bfloat16* g = gate + t * ld_g;
     float s[8];
     if constexpr (PER8) {
-      s[0] = sigmoid(ld(g + c / per));
+      s[0] = sigmoid<__nv_bfloat16>(ld(g + c / per));
 #pragma unroll
       for (int k = 1; k < 8; ++k) s[k] = s[0];
     } else {
 #pragma unroll
-      for (int k = 0; k < 8; ++k) s[k] = sigmoid(ld(g + c + k));
+      for (int k = 0; k < 8; ++k) s[k] = sigmoid<__nv_bfloat16>(ld(g + c + k));
     }
 #pragma unroll
     for (int k = 0; k < 4; ++k) {
@@ -257,7 +259,7 @@ talk_mix_kernel(const T* __restrict__ o, const float* __restrict__ talk, const T
         const long long col = (long long)(h0 + j) * DV + d;
         float r[VEC];
 #pragma unroll
-        for (int e = 0; e < VEC; ++e) r[e] = gate ? acc[j][e] * sigmoid(ld(gate + t * ld_g + col + e)) : acc[j][e];
+        for (int e = 0; e < VEC; ++e) r[e] = gate ? acc[j][e] * sigmoid<T>(ld(gate + t * ld_g + col + e)) : acc[j][e];
         T* dst = y + t * H * DV + col;
         if constexpr (VEC == 2) st2(dst, r[0], r[1]);
         else st(dst, r[0]);
@@ -317,8 +319,8 @@ talk_mix_vec_kernel(const __nv_bfloat16* __restrict__ o, const float* __restrict
 #pragma unroll
           for (int k = 0; k < 4; ++k) {
             const float2 f = __bfloat1622float2(z[k]);
-            v[2 * k] *= sigmoid(f.x);
-            v[2 * k + 1] *= sigmoid(f.y);
+            v[2 * k] *= sigmoid<__nv_bfloat16>(f.x);
+            v[2 * k + 1] *= sigmoid<__nv_bfloat16>(f.y);
           }
         }
         *reinterpret_cast<uint4*>(y + t * H * DV + col) = make_uint4(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]),

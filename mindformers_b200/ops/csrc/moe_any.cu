@@ -31,10 +31,13 @@ __device__ __forceinline__ int rows_in_use(int blk, const int* block_group, cons
   return left < 0 ? 0 : (left > kBlock ? kBlock : left);
 }
 
+// 16-bit results take the fast exponential
+template <typename T>
 __device__ __forceinline__ float glu(float g, float u, float limit, float alpha, float shift) {
   g = fminf(g, limit);
   u = fminf(fmaxf(u, -limit), limit);
-  return g / (1.f + __expf(-alpha * g)) * (u + shift);
+  const float e = sizeof(T) == 2 ? __expf(-alpha * g) : expf(-alpha * g);
+  return g / (1.f + e) * (u + shift);
 }
 
 // grid: (row block, column slice); VEC 8 (bf16, F % 8 == 0) or 1
@@ -60,11 +63,11 @@ clamped_glu_kernel(const T* __restrict__ x, T* __restrict__ y, int R, int F, flo
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
         const float2 g = __bfloat1622float2(ga[j]), u = __bfloat1622float2(ub[j]);
-        o[j] = pack_bf16x2(glu(g.x, u.x, limit, alpha, shift), glu(g.y, u.y, limit, alpha, shift));
+        o[j] = pack_bf16x2(glu<T>(g.x, u.x, limit, alpha, shift), glu<T>(g.y, u.y, limit, alpha, shift));
       }
       *reinterpret_cast<uint4*>(y + r * F + c) = make_uint4(o[0], o[1], o[2], o[3]);
     } else {
-      st(y + r * F + c, glu(ld(x + r * 2 * F + c), ld(x + r * 2 * F + F + c), limit, alpha, shift));
+      st(y + r * F + c, glu<T>(ld(x + r * 2 * F + c), ld(x + r * 2 * F + F + c), limit, alpha, shift));
     }
   }
 }

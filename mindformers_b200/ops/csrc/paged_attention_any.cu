@@ -16,7 +16,7 @@ namespace mfb {
 namespace paa {
 
 constexpr int kWarps = 4;
-constexpr int kMaxPerLane = 16;         // head sizes up to 512
+constexpr int kMaxPerLane = 32;         // head sizes up to 1024
 
 __device__ __forceinline__ float ld(const float* p) { return *p; }
 __device__ __forceinline__ float ld(const __nv_bfloat16* p) { return __bfloat162float(*p); }
@@ -117,7 +117,8 @@ int launch(const void* q, const void* kc, const void* vc, const int* bt, const i
   paged_attention_any_kernel<T, N_><<<grid, kWarps * 32, 0, stream>>>((const T*)q, (const T*)kc, (const T*)vc, bt, cl, \
                                                                       cu, sink, (T*)out, B, Hq, Hkv, D, DV, bs, mb,   \
                                                                       chunk, window, scale, softcap, ld_out, out_scale)
-  if (n <= 2) MFB_PAA(2); else if (n <= 4) MFB_PAA(4); else if (n <= 8) MFB_PAA(8); else MFB_PAA(16);
+  if (n <= 2) MFB_PAA(2); else if (n <= 4) MFB_PAA(4); else if (n <= 8) MFB_PAA(8); 
+  else if (n <= 16) MFB_PAA(16); else MFB_PAA(32);
 #undef MFB_PAA
   if (cudaGetLastError() != cudaSuccess) { mfb_host::set_error("paged_attention_any: launch failed"); return 2; }
   return 0;

@@ -45,14 +45,14 @@ __device__ __forceinline__ void router_scores(const float* __restrict__ row, con
   }
   if (sigmoid) {
 #pragma unroll
-    for (int j = 0; j < PER; ++j) s[j] = (lane + 32 * j) < E ? 1.f / (1.f + __expf(-s[j])) : 0.f;
+    for (int j = 0; j < PER; ++j) s[j] = (lane + 32 * j) < E ? 1.f / (1.f + expf(-s[j])) : 0.f;
     return;
   }
   mx = warp_max(mx);
   float sum = 0.f;
 #pragma unroll
   for (int j = 0; j < PER; ++j) {
-    s[j] = (lane + 32 * j) < E ? __expf(s[j] - mx) : 0.f;
+    s[j] = (lane + 32 * j) < E ? expf(s[j] - mx) : 0.f;
     sum += s[j];
   }
   sum = warp_sum(sum);

@@ -75,6 +75,18 @@ __device__ __forceinline__ void store(float* p, const float (&v)[VEC]) {
   }
 }
 
+// One step of a decay e^a, a <= 0, as s <- most * s + rest * s: with (1, e^a - 1) where the decay is slow, so that the rounding of
+// a factor close to one does not add up over the thousands of tokens that such a state remembers, else with (0, e^a).
+struct Decay {
+  float most, rest;
+  __device__ __forceinline__ explicit Decay(float a) {
+    const bool slow = a > -0.5f;
+    most = slow ? 1.f : 0.f;
+    rest = slow ? expm1f(a) : expf(a);
+  }
+  __device__ __forceinline__ float operator()(float s, float add) const { return fmaf(rest, s, fmaf(most, s, add)); }
+};
+
 struct Args {
   const void* proj;          // [T, >= 2 H P + 2 G N + H]
   long long ld;
@@ -201,13 +213,14 @@ __global__ void __launch_bounds__(kScan) scan_kernel(const Args a) {
   for (int t = 0; t < rows; ++t) {
     const int stage = t & 1;
     const float dt = sdt[stage], x = sx[stage][col];
-    const float keep = expf(rate * dt), v = dt * x;
+    const Decay decay(rate * dt);
+    const float v = dt * x;
     float acc = 0.f;
 #pragma unroll
     for (int j = 0; j < R; ++j) {
       const int r = grp + kGroups * j;
       if (r < N) {
-        s[j] = fmaf(keep, s[j], sb[stage][r] * v);
+        s[j] = decay(s[j], sb[stage][r] * v);
         acc = fmaf(s[j], sc[stage][r], acc);
       }
     }
@@ -263,7 +276,8 @@ __global__ void __launch_bounds__(kDec) decode_kernel(const Args a) {
     sh[i] = y;
   }
   const float dt = softplus(ld(row + a.col_dt() + h) + a.dt_bias[h]);
-  const float keep = expf(-expf(a.a_log[h]) * dt), d = a.d[h];
+  const Decay decay(-expf(a.a_log[h]) * dt);
+  const float d = a.d[h];
   __syncthreads();
   const float* sB = sh;
   const float* sC = sh + N;
@@ -290,7 +304,7 @@ __global__ void __launch_bounds__(kDec) decode_kernel(const Args a) {
         } else load<VEC>(s + (long long)r * P, x);
 #pragma unroll
         for (int e = 0; e < VEC; ++e) {
-          x[e] = fmaf(keep, x[e], sB[r] * v[e]);
+          x[e] = decay(x[e], sB[r] * v[e]);
           acc[e] = fmaf(x[e], sC[r], acc[e]);
         }
         store<VEC>(s + (long long)r * P, x);
@@ -484,11 +498,11 @@ __global__ void __launch_bounds__(128, 2) chunk_kernel(const Args p) {
     const uint8_t* xt = st + 2 * Sh::kCBytes;
     const float4* sg = reinterpret_cast<const float4*>(xt + Sh::kXBytes);
     const float4 last_gate = sg[n - 1];
-    const float keep = __expf(last_gate.x + last_gate.y);
+    const float keep = expf(last_gate.x + last_gate.y);
     if (tid < kChunk) {
       const float4 gt = sg[tid];
-      sW[tid] = tid < n ? gt.z * __expf((last_gate.x - gt.x) + (last_gate.y - gt.y)) : 0.f;
-      sScale[tid] = __expf(gt.x + gt.y);
+      sW[tid] = tid < n ? gt.z * expf((last_gate.x - gt.x) + (last_gate.y - gt.y)) : 0.f;
+      sScale[tid] = expf(gt.x + gt.y);
     }
     // gates of the warp's 16 columns: rows m * 16 + g (+ 8), loaded ahead of the products
     uint32_t z[4][2][2];

@@ -295,7 +295,7 @@ class ParallelTransformerLayer(nn.Module):
         if meta.loop_step is not None and meta.loop_entry is not None:
             w, base = meta.loop_entry
             x, ys = stream.linear(stream.joint_step(x, ys, None, None, None, 1, 0.0, dtype, keep=False)[0], w,
-                                  out_dtype=torch.float32), ()
+                                  out_dtype=torch.float32).contiguous(), ()        # rows of odd widths lie in a padded matrix
         conv = None
         if self.input_conv is not None:
             if meta.cache is None:

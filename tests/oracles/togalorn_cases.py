@@ -46,8 +46,8 @@ CASES = {
     "chosen_experts": config([latent(1, 32, 2, 96, 24, 64, 0.5, 7.0, moe(7, 2, 3, 96)), mamba(1, 96, 32, 1, 1, 1, moe(8, 4, 1, 64)),
                               mamba(8, 64, 64, 8, 4, 8, moe(6, 0, 2, 40))], width=128, vocab=515, groups=1, taps=1, scale=1.0),
     # sizes that no vector access and no tensor-core kernel takes; many taps; a loop of one pass at the end
-    "odd_sizes": config([mamba(3, 7, 5, 1, 6, 1, moe(3, 1, 2, 50, 0.9, 33)), latent(3, 13, 6, 11, 17, 29, 0.4, 20.0, moe(2, 2, 4, 33)),
-                         mamba(6, 5, 20, 3, 3, 2, None), latent(2, 130, 14, 12, 40, 50, 0.1, 90.0, moe(1, 1, 1, 20))], width=105, vocab=77,
+    "odd_sizes": config([mamba(3, 7, 5, 1, 6, 1, moe(3, 1, 4, 50, 0.9, 33)), latent(3, 13, 6, 11, 17, 29, 0.4, 20.0, moe(2, 2, 4, 33)),
+                         mamba(6, 5, 20, 3, 3, 2, None), latent(2, 130, 14, 12, 40, 50, 0.1, 90.0, moe(1, 1, 2, 20))], width=105, vocab=77,
                         groups=3, taps=6, loop=(2, 4, 1)),
 }
 

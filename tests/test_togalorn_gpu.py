@@ -232,8 +232,6 @@ LATENT = [(4, 48, 16, 64, 128), (8, 96, 32, 128, 512), (16, 128, 64, 128, 512), 
 @pytest.mark.parametrize("H,D,P,DV,R", LATENT)
 def test_latent_attention(dtype, H, D, P, DV, R):
     """Expanded portions, absorbed rows and both in one batch."""
-    if R + P > 512 and dtype == torch.float32:
-        pytest.skip("32-bit attention over cached rows of up to 512 numbers")
     for lens, news, bs, ragged_step in (([1, 300, 129, 517, 64, 130, 40], [1, 300, 2, 260, 1, 1, 0], 64, True),
                                         ([70, 3], [1, 1], 64, True), ([200], [90], 16, True), ([1, 63, 64, 129, 700], [1] * 5, 16, False)):
         ctx, table, q, w, scale, want = latent_case(dtype, H, D, P, DV, R, bs, lens, news, seed=R)
@@ -250,8 +248,6 @@ def test_latent_attention(dtype, H, D, P, DV, R):
 @pytest.mark.parametrize("H,D,P,DV,R", [(8, 96, 32, 128, 256), (3, 13, 4, 11, 29), (4, 128, 64, 128, 512)])
 def test_a_far_rotated_key_is_found(dtype, H, D, P, DV, R):
     """One key whose rotated part stands out, at page and tile borders; in a prompt, in a portion of two rows and decoded."""
-    if R + P > 512 and dtype == torch.float32:
-        pytest.skip("32-bit attention over cached rows of up to 512 numbers")
     n, bs = 400, 16
     for qp in (399, 256, 128, 127, 16):
         for kp in (0, 1, 15, 16, 127, 128, qp, qp + 1):
@@ -470,14 +466,12 @@ def fast_oracle():
 
 def sure_rows(cfg, w, toks, dtype):
     """Positions that no close choice of experts reaches."""
-    return torch.ones(len(toks), dtype=torch.bool) if dtype == "float32" else ~tc.close_calls(cfg, w, toks, 2e-3)
+    return torch.ones(len(toks), dtype=torch.bool) if dtype == "float32" else ~tc.close_calls(cfg, w, toks, 1e-2)
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 @pytest.mark.parametrize("name", sorted(tc.CASES))
 def test_logits_do_not_depend_on_the_schedule(checkpoints, name, dtype):
-    if name == "wide_heads" and dtype == "float32":
-        pytest.skip("32-bit attention over cached rows of up to 512 numbers")
     model, cfg, w = checkpoints(name, dtype)
     toks = {f"r{i}": cases.tokens(n, cfg["vocab"], seed=i) for i, n in enumerate((283, 1, 70, 131, 40))}
     want = {r: tc.expected(cfg, w, t) for r, t in toks.items()}
@@ -489,7 +483,7 @@ def test_logits_do_not_depend_on_the_schedule(checkpoints, name, dtype):
         if ok.any():
             err, ref = tc.errors(logits, want[r])[ok], noise[r][ok]
             assert float(err.max()) < max(LIMIT[dtype], 3 * float(ref.max())), (r, what, int(err.argmax()))
-            assert float(err.median()) < max(LIMIT[dtype] / 10, 3 * float(ref.median())), (r, what)
+            assert len(err) < 20 or float(err.median()) < max(LIMIT[dtype] / 10, 3 * float(ref.median())), (r, what)
     whole = [{r: len(t)} for r, t in toks.items()]
     one_by_one = [{"r2": 30}] + [{"r2": 1}] * 40
     cut = [{r: c} for r, t in toks.items() for c in cases.portions(len(t), (2, 37, 1, 64, 3, 65, 2, 2))]
