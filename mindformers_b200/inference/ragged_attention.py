@@ -309,7 +309,7 @@ def latent_attention(q: torch.Tensor, cache, layer: int, w_kv: torch.Tensor, v_d
     w_uk, w_uv = w_kv[:H * D].view(H, D, R), w_kv[H * D:].view(H, v_dim, R)[:, :, :v_rank]
     lib = _lib.get_lib() if q.is_cuda else None
     expand = lib is not None and q.dtype == torch.bfloat16 and cache.is_prefill and cache.n_long_rows \
-        and lib.mfb_paged_prefill_tc_supported(H, H, D, v_dim, cache.block_size)
+        and lib.mfb_paged_prefill_tc_wide_supported(H, H, D, v_dim, cache.block_size)
     if not expand:
         return _absorbed(q, cache, layer, w_uk, w_uv, scale, window, sink)
     from ..ops import functional as Fn

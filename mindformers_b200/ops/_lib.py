@@ -142,6 +142,7 @@ def _declare(lib):
     sig("mfb_paged_decode_tc_supported_ex", [I, I, I, I, I])
     sig("mfb_paged_decode_attention_tc_ex", [P] * 9 + [I] * 13 + [F, F, L, F, P, P])
     sig("mfb_paged_prefill_tc_supported", [I, I, I, I, I])
+    sig("mfb_paged_prefill_tc_wide_supported", [I, I, I, I, I])
     sig("mfb_paged_prefill_tc", [P, P, P, P, I, I, P, P, P] + [I] * 11 + [L, L, F, F, L, F, P, P])
     sig("mfb_paged_attention_any", [P] * 8 + [I] * 11 + [F, F, L, F, I, P])
     sig("mfb_residual_streams", [P, I, P, L, P, P, P, P, P, P, I, I, I, F, I, P])

@@ -444,6 +444,11 @@ __device__ __forceinline__ uint32_t pack_bf16x2(float lo, float hi) {
   __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
   return *reinterpret_cast<uint32_t*>(&v);
 }
+// 1 / sqrt(v), v > 0: the approximation and one step of Newton's method
+__device__ __forceinline__ float inv_sqrt(float v) {
+  const float r = rsqrtf(v);
+  return r * fmaf(-0.5f * v * r, r, 1.5f);
+}
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

@@ -116,6 +116,7 @@ __global__ void __launch_bounds__(THREADS) joint_step_kernel(const Args a) {
       r = max(r0 - (a.taps - 1), a.cu_q[b]);
     }
   }
+  const float inv_part = 1.f / a.part;
   for (; r < r1; ++r) {
     float xv[K][VEC];
     float ss = 0.f;
@@ -138,7 +139,7 @@ __global__ void __launch_bounds__(THREADS) joint_step_kernel(const Args a) {
         }
       }
     }
-    const float rstd = w ? 1.f / sqrtf(block_sum(ss, red, turn) / a.part + a.eps) : 1.f;
+    const float rstd = w ? inv_sqrt(fmaf(block_sum(ss, red, turn), inv_part, a.eps)) : 1.f;
     const bool own = r >= r0;
     bool first = false, last = false, keep = false;
     if constexpr (TM > 0) {

@@ -1,5 +1,5 @@
 // Prefill attention of a ragged batch over a paged bf16 cache on the tensor cores (sm_100a, tcgen05 + TMA), grouped-query
-// attention with query / key size and value size up to 128 each (multiples of 8), optional chunked mask and softmax sink.
+// attention with query / key size up to 192 and value size up to 128 (multiples of 8), optional chunked mask and softmax sink.
 //
 // Sequence b brings the rows cu_q[b] .. cu_q[b + 1] - 1 of q; its keys and values, those rows included, are in the cache
 // already, so a whole prompt, a later portion of a prompt and any mix of sequences are the same problem: row r of the
@@ -22,7 +22,7 @@
 //     key tiles that some row of the tile sees are visited, from the chunk of its first row to its last row;
 //   - K / V tiles (128 consecutive positions) are assembled from the sequence's pages, one TMA box per page and 64
 //     columns; pages past the end of the sequence repeat the tile's first page and are masked;
-//   - head sizes are padded to 64 or 128 columns: q is read through a three-dimensional map that fills the columns past
+//   - head sizes are padded to 64, 128 or 192 columns (192: one CTA per SM): q is read through a three-dimensional map that fills the columns past
 //     the head with zeros, so whatever a K box holds there does not count; columns of V past the head reach only
 //     columns of the result that are not stored;
 //   - the result is written row by row: a portion may end anywhere.
@@ -114,9 +114,9 @@ __device__ __forceinline__ void tmem_st_32x32b_x32(uint32_t taddr, const uint32_
 constexpr float kPolyReach = 0.6f;
 constexpr float kTanhRatio[5] = {0.999999926f, -0.33332302f, 0.133100644f, -0.0520966534f, 0.0154687513f};
 
-// HQ: padded query / key size, HV: padded value size (64 or 128); CAP: scores are soft-capped
+// HQ: padded query / key size (64, 128 or 192), HV: padded value size (64 or 128); CAP: scores are soft-capped
 template <int HQ, int HV, bool CAP>
-__global__ void __launch_bounds__(kThreads, 2)
+__global__ void __launch_bounds__(kThreads, HQ > 128 ? 1 : 2)
 paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                         const __grid_constant__ CUtensorMap tmV, const Args args) {
   constexpr int QB = HQ / 64, VB = HV / 64;          // 64-column sub-tiles
@@ -825,7 +825,7 @@ template <int HQ, int HV, bool CAP>
 int launch(const CUtensorMap& tQ, const CUtensorMap& tK, const CUtensorMap& tV, const Args& a, int max_ctas, cudaStream_t stream) {
   constexpr int QBYTES = HQ / 64 * kSubBytes, VBYTES = HV / 64 * kSubBytes;
   constexpr int SMEM = 2 * QBYTES + VBYTES + 4 * 2048 + 9 * 8 + 16 + 1024;
-  static_assert(2 * SMEM <= 232448, "shared memory budget exceeded");
+  static_assert((HQ > 128 ? 1 : 2) * SMEM <= 232448, "shared memory budget exceeded");
   auto kern = paged_prefill_tc_kernel<HQ, HV, CAP>;
   static bool attr_set = false;
   if (!attr_set) {
@@ -853,6 +853,11 @@ int mfb_paged_prefill_tc_supported(int Hq, int Hkv, int D, int DV, int block_siz
   return (block_size == 16 || block_size == 32 || block_size == 64 || block_size == 128) ? 1 : 0;
 }
 
+// The same for keys of up to 192 numbers, without all_values or a soft cap beyond 128.
+int mfb_paged_prefill_tc_wide_supported(int Hq, int Hkv, int D, int DV, int block_size) {
+  return D <= 192 && D % 8 == 0 ? mfb_paged_prefill_tc_supported(Hq, Hkv, D < 128 ? D : 128, DV, block_size) : 0;
+}
+
 // q [T, Hq, D], caches [num_blocks, block_size, Hkv, D | DV] with rows ld_k / ld_v elements apart, out [T, Hq, DV] (all_values:
 // [T, Hq, Hkv, DV]), all bf16. chunk > 0: a position sees its own chunk only; window > 0: itself and the window - 1 positions
 // before it. work [n_work, 4] int32: (sequence,
@@ -865,7 +870,8 @@ int mfb_paged_prefill_tc(const void* q, const void* key_cache, const void* value
                          int Hq, int Hkv, int D, int DV, int num_blocks, int block_size, int max_blocks, int chunk, int window,
                          int all_values, long long ld_k, long long ld_v, float scale, float softcap, long long ld_out,
                          float out_scale, int* status, cudaStream_t stream) {
-  if (!mfb_paged_prefill_tc_supported(Hq, Hkv, D, DV, block_size) || num_blocks < 1 || T < 1) {
+  if (!mfb_paged_prefill_tc_wide_supported(Hq, Hkv, D, DV, block_size) || (D > 128 && (all_values || softcap > 0.f)) ||
+      num_blocks < 1 || T < 1) {
     mfb_host::set_error("paged_prefill_tc: unsupported Hq=%d Hkv=%d D=%d DV=%d block_size=%d", Hq, Hkv, D, DV, block_size);
     return 1;
   }
@@ -902,9 +908,12 @@ int mfb_paged_prefill_tc(const void* q, const void* key_cache, const void* value
     return DV > 64 ? ppt::launch_values<64, 128>(tQ, tK, tV, a, n_work, Hkv, stream)
                    : ppt::launch_values<64, 64>(tQ, tK, tV, a, n_work, Hkv, stream);
   }
-  const int max_ctas = persistent ? 2 * 148 : a.n_items;
+  const int max_ctas = persistent ? (D > 128 ? 1 : 2) * 148 : a.n_items;
 #define MFB_PPT(HQ_, HV_) \
   return softcap > 0.f ? ppt::launch<HQ_, HV_, true>(tQ, tK, tV, a, max_ctas, stream) : ppt::launch<HQ_, HV_, false>(tQ, tK, tV, a, max_ctas, stream)
+  if (D > 128)
+    return DV > 64 ? ppt::launch<192, 128, false>(tQ, tK, tV, a, max_ctas, stream)
+                   : ppt::launch<192, 64, false>(tQ, tK, tV, a, max_ctas, stream);
   if (D > 64) {
     if (DV > 64) MFB_PPT(128, 128);
     MFB_PPT(128, 64);

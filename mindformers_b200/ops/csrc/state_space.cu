@@ -26,12 +26,17 @@ __device__ __forceinline__ void st(__nv_bfloat16* p, float v) { *p = __float2bfl
 __device__ __forceinline__ float softplus(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
 template <typename T>
 __device__ __forceinline__ float silu(float z) {
-  if constexpr (sizeof(T) == 2) return z / (1.f + __expf(-z));
+  if constexpr (sizeof(T) == 2) return __fdividef(z, 1.f + __expf(-fmaxf(z, -80.f)));      // the quotient's divisor stays in reach
   else return z / (1.f + expf(-z));
 }
 template <int VEC>
 __device__ __forceinline__ void load(const __nv_bfloat16* p, float (&v)[VEC]) {
-  if constexpr (VEC == 8) {
+  if constexpr (VEC == 4) {
+    const uint2 u = *reinterpret_cast<const uint2*>(p);
+    const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.x));
+    const float2 g = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.y));
+    v[0] = f.x; v[1] = f.y; v[2] = g.x; v[3] = g.y;
+  } else if constexpr (VEC == 8) {
     const uint4 u = *reinterpret_cast<const uint4*>(p);
     const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&u);
 #pragma unroll
@@ -56,7 +61,9 @@ __device__ __forceinline__ void load(const float* p, float (&v)[VEC]) {
 }
 template <int VEC>
 __device__ __forceinline__ void store(__nv_bfloat16* p, const float (&v)[VEC]) {
-  if constexpr (VEC == 8) {
+  if constexpr (VEC == 4) {
+    *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]));
+  } else if constexpr (VEC == 8) {
     *reinterpret_cast<uint4*>(p) = make_uint4(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]), pack_bf16x2(v[4], v[5]),
                                               pack_bf16x2(v[6], v[7]));
   } else {
@@ -105,14 +112,15 @@ struct Args {
   void* xbc;                 // [T, C], rows ld_x apart: after convolution and silu
   long long ld_x;
   void* out;                 // [T, H P]
-  int T, B, H, P, N, G, taps, norm_groups, rows;
+  int T, B, H, P, N, G, taps, norm_groups;
+  int rows;                  // rows (convolution) or heads (decode) per CTA
   float eps;
   __host__ __device__ int inner() const { return H * P; }
   __host__ __device__ int channels() const { return H * P + 2 * G * N; }
   __host__ __device__ int col_dt() const { return 2 * H * P + 2 * G * N; }
 };
 
-constexpr int kMaxTaps = 16;
+constexpr int kMaxTaps = 16, kAhead = 4;
 
 // VEC channels per thread, a.rows rows per CTA; TM: bound of the taps (weights are padded with zeros in front)
 template <typename T, int VEC, int TM>
@@ -153,25 +161,38 @@ __global__ void __launch_bounds__(128) conv_kernel(const Args a) {
     }
   };
   restart(r0);
-  for (int r = r0; r < r1; ++r) {
-    if (r >= a.cu_q[b + 1]) {
-      while (r >= a.cu_q[b + 1]) ++b;
-      restart(r);
+  int end = a.cu_q[b + 1];
+  // kAhead rows are on their way at a time
+  float next[kAhead][VEC];
+  for (int r8 = r0; r8 < r1; r8 += kAhead) {
+#pragma unroll
+    for (int u = 0; u < kAhead; ++u)
+      if (r8 + u < r1) load<VEC>(src + (long long)(r8 + u) * a.ld, next[u]);
+#pragma unroll
+    for (int u = 0; u < kAhead; ++u) {
+      const int r = r8 + u;
+      if (r >= r1) break;
+      if (r >= end) {
+        while (r >= a.cu_q[b + 1]) ++b;
+        end = a.cu_q[b + 1];
+        restart(r);
+      }
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) win[TM - 1][i] = next[u][i];
+      float y[VEC];
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) {
+        y[i] = bias[i];
+#pragma unroll
+        for (int j = 0; j < TM; ++j) y[i] = fmaf(w[j][i], win[j][i], y[i]);
+        y[i] = silu<T>(y[i]);
+      }
+      store<VEC>(reinterpret_cast<T*>(a.xbc) + (long long)r * a.ld_x + c, y);
+#pragma unroll
+      for (int j = 0; j + 1 < TM; ++j)
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) win[j][i] = win[j + 1][i];
     }
-    load<VEC>(src + (long long)r * a.ld, win[TM - 1]);
-    float y[VEC];
-#pragma unroll
-    for (int i = 0; i < VEC; ++i) {
-      y[i] = bias[i];
-#pragma unroll
-      for (int j = 0; j < TM; ++j) y[i] = fmaf(w[j][i], win[j][i], y[i]);
-      y[i] = silu<T>(y[i]);
-    }
-    store<VEC>(reinterpret_cast<T*>(a.xbc) + (long long)r * a.ld_x + c, y);
-#pragma unroll
-    for (int j = 0; j + 1 < TM; ++j)
-#pragma unroll
-      for (int i = 0; i < VEC; ++i) win[j][i] = win[j + 1][i];
   }
 }
 
@@ -245,39 +266,39 @@ __global__ void __launch_bounds__(kScan) scan_kernel(const Args a) {
 
 constexpr int kDec = 256;
 
-// CTA (head, slot). VEC columns per thread; the threads of a column block share the rows.
+// CTA (a.rows heads of a group, slot): B and C once for its heads. VEC columns per thread; the threads of a column block share the
+// rows of S.
 template <typename T, int VEC>
 __global__ void __launch_bounds__(kDec) decode_kernel(const Args a) {
-  extern __shared__ float sh[];                    // B [N], C [N], x [P], partial sums [kDec * VEC]
-  const int h = blockIdx.x, b = blockIdx.y, tid = threadIdx.x;
-  const int N = a.N, P = a.P, H = a.H, inner = a.inner(), C = a.channels(), per = H / a.G, g = h / per;
-  T* out = reinterpret_cast<T*>(a.out) + (long long)b * inner + h * P;
+  extern __shared__ float sh[];                    // B [N], C [N], x [heads P], partial sums [heads][kDec * VEC]
+  const int heads = a.rows, h0 = blockIdx.x * heads, b = blockIdx.y, tid = threadIdx.x;
+  const int N = a.N, P = a.P, H = a.H, inner = a.inner(), C = a.channels(), per = H / a.G, g = h0 / per, cols_x = heads * P;
+  T* out = reinterpret_cast<T*>(a.out) + (long long)b * inner + h0 * P;
   if (a.slots[b] < 0) {
-    for (int c = tid; c < P; c += kDec) st(out + c, 0.f);
+    for (int c = tid; c < cols_x; c += kDec) st(out + c, 0.f);
     return;
   }
   const int pos = a.context_lens[b] - 1;
   const bool fresh = pos <= 0;
-  const long long head = (long long)b * H + h;
   const T* row = reinterpret_cast<const T*>(a.proj) + b * a.ld;
   T* ring = reinterpret_cast<T*>(a.ring) + (long long)b * a.taps * C;
-  float* part = sh + 2 * N + P;
-  for (int i = tid; i < 2 * N + P; i += kDec) {
-    const int c = i < N ? inner + g * N + i : i < 2 * N ? inner + a.G * N + g * N + i - N : h * P + i - 2 * N;
+  float* part = sh + 2 * N + cols_x;
+  const int place = pos % a.taps;
+  for (int i = tid; i < 2 * N + cols_x; i += kDec) {
+    const int c = i < N ? inner + g * N + i : i < 2 * N ? inner + a.G * N + g * N + i - N : h0 * P + i - 2 * N;
     const float now = ld(row + inner + c);
     float y = fmaf(a.conv[(long long)(a.taps - 1) * C + c], now, a.conv_b[c]);
-    for (int j = 1; j < a.taps && j <= pos; ++j)
-      y = fmaf(a.conv[(long long)(a.taps - 1 - j) * C + c], ld(ring + (long long)((pos - j) % a.taps) * C + c), y);
-    // the channels of a group's B and C are written by its first head
-    if (i >= 2 * N || h == g * per) st(ring + (long long)(pos % a.taps) * C + c, now);
+    for (int j = 1; j < a.taps && j <= pos; ++j) {
+      const int at = place >= j ? place - j : place - j + a.taps;
+      y = fmaf(a.conv[(long long)(a.taps - 1 - j) * C + c], ld(ring + (long long)at * C + c), y);
+    }
+    // the channels of a group's B and C are written by its first heads
+    if (i >= 2 * N || h0 == g * per) st(ring + (long long)place * C + c, now);
     y = silu<T>(y);
     // what enters the recurrence after the convolution is an activation
     if constexpr (sizeof(T) == 2) y = __bfloat162float(__float2bfloat16_rn(y));
     sh[i] = y;
   }
-  const float dt = softplus(ld(row + a.col_dt() + h) + a.dt_bias[h]);
-  const Decay decay(-expf(a.a_log[h]) * dt);
-  const float d = a.d[h];
   __syncthreads();
   const float* sB = sh;
   const float* sC = sh + N;
@@ -287,63 +308,71 @@ __global__ void __launch_bounds__(kDec) decode_kernel(const Args a) {
   const bool on = grp < groups;
   for (int c0 = 0; c0 < nv; c0 += cols) {
     const int cv = c0 + ci;
-    float acc[VEC];
+    for (int k = 0; k < heads; ++k) {
+      const int h = h0 + k;
+      float acc[VEC];
 #pragma unroll
-    for (int e = 0; e < VEC; ++e) acc[e] = 0.f;
-    if (on && cv < nv) {
-      float v[VEC];
+      for (int e = 0; e < VEC; ++e) acc[e] = 0.f;
+      if (on && cv < nv) {
+        const float dt = softplus(ld(row + a.col_dt() + h) + a.dt_bias[h]);
+        const Decay decay(-expf(a.a_log[h]) * dt);
+        float v[VEC];
 #pragma unroll
-      for (int e = 0; e < VEC; ++e) v[e] = dt * sX[cv * VEC + e];
-      float* s = a.S + head * N * P + (long long)cv * VEC;
+        for (int e = 0; e < VEC; ++e) v[e] = dt * sX[k * P + cv * VEC + e];
+        float* s = a.S + ((long long)b * H + h) * N * P + (long long)cv * VEC;
 #pragma unroll 8
-      for (int r = grp; r < N; r += groups) {
-        float x[VEC];
-        if (fresh) {
+        for (int r = grp; r < N; r += groups) {
+          float x[VEC];
+          if (fresh) {
 #pragma unroll
-          for (int e = 0; e < VEC; ++e) x[e] = 0.f;
-        } else load<VEC>(s + (long long)r * P, x);
+            for (int e = 0; e < VEC; ++e) x[e] = 0.f;
+          } else load<VEC>(s + (long long)r * P, x);
 #pragma unroll
-        for (int e = 0; e < VEC; ++e) {
-          x[e] = decay(x[e], sB[r] * v[e]);
-          acc[e] = fmaf(x[e], sC[r], acc[e]);
+          for (int e = 0; e < VEC; ++e) {
+            x[e] = decay(x[e], sB[r] * v[e]);
+            acc[e] = fmaf(x[e], sC[r], acc[e]);
+          }
+          store<VEC>(s + (long long)r * P, x);
         }
-        store<VEC>(s + (long long)r * P, x);
       }
-    }
 #pragma unroll
-    for (int e = 0; e < VEC; ++e) part[tid * VEC + e] = acc[e];
+      for (int e = 0; e < VEC; ++e) part[(k * kDec + tid) * VEC + e] = acc[e];
+    }
     __syncthreads();
-    for (int c = tid; c < cols * VEC && c0 * VEC + c < P; c += kDec) {
-      float y = d * sX[c0 * VEC + c];
-      for (int k = 0; k < groups; ++k) y += part[k * cols * VEC + c];
-      st(out + c0 * VEC + c, y * silu<T>(ld(row + h * P + c0 * VEC + c)));
+    const int width = min(cols * VEC, P - c0 * VEC);
+    for (int i = tid; i < heads * width; i += kDec) {
+      const int k = i / width, c = i % width, col = k * P + c0 * VEC + c;
+      float y = a.d[h0 + k] * sX[col];
+      for (int j = 0; j < groups; ++j) y += part[k * kDec * VEC + j * cols * VEC + c];
+      st(out + col, y * silu<T>(ld(row + h0 * P + col)));
     }
     __syncthreads();
   }
 }
 
-// CTA per (row, part): RMS norm in place, K accesses of VEC columns per thread. The CTAs behind those move a sequence's last
-// inputs of the convolution into its ring.
+// RMS norm in place: blockDim.x threads per (row, part), K accesses of VEC columns each; a warp each where blockDim.y > 1. The
+// CTAs behind those move a sequence's last inputs of the convolution into its ring.
+constexpr int kRingCols = 512;
 template <typename T, int VEC, int K>
 __global__ void __launch_bounds__(1024) finish_kernel(const Args a) {
   __shared__ float red[32];
-  const long long items = (long long)a.T * a.norm_groups;
+  const unsigned items = (unsigned)(a.T * a.norm_groups), ctas = (items + blockDim.y - 1) / blockDim.y;
   const int inner = a.inner();
-  if ((long long)blockIdx.x >= items) {
-    const int b = (int)(blockIdx.x - items), C = a.channels();
-    const int n = a.cu_q[b + 1] - a.cu_q[b], end = a.context_lens[b];
-    T* ring = reinterpret_cast<T*>(a.ring) + (long long)b * a.taps * C;
-    for (int j = 0; j < min(n, a.taps); ++j) {
-      const T* src = reinterpret_cast<const T*>(a.proj) + (long long)(a.cu_q[b + 1] - 1 - j) * a.ld + inner;
-      T* dst = ring + (long long)((end - 1 - j) % a.taps) * C;
-      for (int c = threadIdx.x; c < C; c += blockDim.x) dst[c] = src[c];
-    }
+  if (blockIdx.x >= ctas) {                           // a CTA per sequence, token and kRingCols channels
+    const int C = a.channels(), slices = (C + kRingCols - 1) / kRingCols;
+    const int i = (int)(blockIdx.x - ctas), c0 = i % slices * kRingCols, j = i / slices % a.taps, b = i / slices / a.taps;
+    if (j >= a.cu_q[b + 1] - a.cu_q[b]) return;
+    const T* src = reinterpret_cast<const T*>(a.proj) + (long long)(a.cu_q[b + 1] - 1 - j) * a.ld + inner;
+    T* dst = reinterpret_cast<T*>(a.ring) + ((long long)b * a.taps + (a.context_lens[b] - 1 - j) % a.taps) * C;
+    for (int c = c0 + threadIdx.y * blockDim.x + threadIdx.x; c < min(C, c0 + kRingCols); c += blockDim.x * blockDim.y) dst[c] = src[c];
     return;
   }
   const int gw = inner / a.norm_groups, nvec = gw / VEC;
-  const long long t = blockIdx.x / a.norm_groups;
-  const int c0 = (int)(blockIdx.x % a.norm_groups) * gw;
-  T* row = reinterpret_cast<T*>(a.out) + t * inner + c0;
+  const unsigned item = blockIdx.x * blockDim.y + threadIdx.y;
+  if (item >= items) return;
+  const unsigned t = item / a.norm_groups;
+  const int c0 = (int)(item % a.norm_groups) * gw;
+  T* row = reinterpret_cast<T*>(a.out) + (long long)t * inner + c0;
   float v[K][VEC], ss = 0.f;
 #pragma unroll
   for (int k = 0; k < K; ++k) {
@@ -361,7 +390,7 @@ __global__ void __launch_bounds__(1024) finish_kernel(const Args a) {
     ss = 0.f;
     for (int w = 0; w < (int)(blockDim.x >> 5); ++w) ss += red[w];
   }
-  const float rstd = 1.f / sqrtf(ss / gw + a.eps);
+  const float rstd = inv_sqrt(ss / gw + a.eps);
 #pragma unroll
   for (int k = 0; k < K; ++k) {
     const int c = threadIdx.x + k * blockDim.x;
@@ -387,24 +416,28 @@ __global__ void __launch_bounds__(1024) finish_kernel(const Args a) {
 constexpr int kChunk = 64;
 
 // a warp per head, two tokens per lane
+constexpr int kGateHeads = 8;
 template <typename T>
-__global__ void __launch_bounds__(256) gates_kernel(const Args a) {
-  extern __shared__ float sh[];                      // [64][H] raw step sizes
-  const int b = blockIdx.y, r0 = a.cu_q[b], rows = a.cu_q[b + 1] - r0, t0 = blockIdx.x * kChunk;
+__global__ void __launch_bounds__(32 * kGateHeads) gates_kernel(const Args a) {
+  __shared__ float sh[kChunk][kGateHeads + 1];       // raw step sizes
+  const int b = blockIdx.y, r0 = a.cu_q[b], rows = a.cu_q[b + 1] - r0, t0 = blockIdx.x * kChunk, h0 = blockIdx.z * kGateHeads;
   if (t0 >= rows) return;
-  const int n = min(kChunk, rows - t0), H = a.H;
-  for (int i = threadIdx.x; i < n * H; i += blockDim.x)
-    sh[i] = ld(reinterpret_cast<const T*>(a.proj) + (long long)(r0 + t0 + i / H) * a.ld + a.col_dt() + i % H);
+  const int n = min(kChunk, rows - t0), heads = min(kGateHeads, a.H - h0);
+  for (int i = threadIdx.x; i < n * kGateHeads; i += blockDim.x) {
+    const int t = i / kGateHeads, k = i % kGateHeads;
+    if (k < heads) sh[t][k] = ld(reinterpret_cast<const T*>(a.proj) + (long long)(r0 + t0 + t) * a.ld + a.col_dt() + h0 + k);
+  }
   __syncthreads();
-  const int lane = threadIdx.x & 31;
-  for (int h = threadIdx.x >> 5; h < H; h += blockDim.x >> 5) {
+  const int lane = threadIdx.x & 31, own = threadIdx.x >> 5;
+  if (own < heads) {
+    const int h = h0 + own;
     const float rate = -expf(a.a_log[h]), bias = a.dt_bias[h];
     float dt[2];
     double f[2];
 #pragma unroll
     for (int e = 0; e < 2; ++e) {
       const int t = 2 * lane + e;
-      dt[e] = t < n ? softplus(sh[t * H + h] + bias) : 0.f;
+      dt[e] = t < n ? softplus(sh[t][own] + bias) : 0.f;
       f[e] = (double)rate * (double)dt[e];
     }
     double sum = f[0] + f[1];
@@ -677,7 +710,7 @@ bool al16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; }
 
 bool chunks_ok(const Args& a) {
   return a.N % 8 == 0 && a.P % 8 == 0 && a.N <= 256 && a.ld % 8 == 0 && a.ld_x % 8 == 0 && al16(a.proj) && al16(a.xbc) &&
-         al16(a.out) && al16(a.gates) && a.H <= 768;
+         al16(a.out) && al16(a.gates);
 }
 
 template <int NP, int STAGES>
@@ -697,13 +730,8 @@ int chunk_launch(const Args& a, cudaStream_t stream) {
 }
 
 int in_chunks(const Args& a, int longest, cudaStream_t stream) {
-  const size_t smem = (size_t)kChunk * a.H * 4;
-  if (smem > 48 * 1024 && cudaFuncSetAttribute(gates_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                               (int)smem) != cudaSuccess) {
-    mfb_host::set_error("state_space: cannot raise the shared memory limit");
-    return 10;
-  }
-  gates_kernel<__nv_bfloat16><<<dim3((longest + kChunk - 1) / kChunk, a.B), 256, smem, stream>>>(a);
+  const dim3 grid((longest + kChunk - 1) / kChunk, a.B, (a.H + kGateHeads - 1) / kGateHeads);
+  gates_kernel<__nv_bfloat16><<<grid, 32 * kGateHeads, 0, stream>>>(a);
   if (a.N <= 32) return chunk_launch<32, 2>(a, stream);
   if (a.N <= 64) return chunk_launch<64, 2>(a, stream);
   if (a.N <= 128) return chunk_launch<128, 2>(a, stream);
@@ -734,33 +762,41 @@ void scan(const Args& a, cudaStream_t stream) {
 template <typename T, int VEC>
 int finish(const Args& a, cudaStream_t stream) {
   const int gw = a.inner() / a.norm_groups, nvec = gw / VEC;
-  const unsigned grid = (unsigned)((long long)a.T * a.norm_groups + (a.cu_q ? a.B : 0));
-  auto threads = [&](int k) { return ((nvec + k - 1) / k + 31) / 32 * 32; };
-  if (nvec <= 256) finish_kernel<T, VEC, 1><<<grid, threads(1), 0, stream>>>(a);
-  else if (nvec <= 1024) finish_kernel<T, VEC, 2><<<grid, threads(2), 0, stream>>>(a);
-  else if (nvec <= 4096) finish_kernel<T, VEC, 4><<<grid, threads(4), 0, stream>>>(a);
-  else if (VEC == 1 && nvec <= 16384) finish_kernel<T, 1, 16><<<grid, threads(16), 0, stream>>>(a);
+  auto go = [&](auto kern, int k) {
+    const int x = ((nvec + k - 1) / k + 31) / 32 * 32, y = x == 32 ? 4 : 1;
+    const long long items = (long long)a.T * a.norm_groups;
+    const long long ring = a.cu_q ? (long long)a.B * a.taps * ((a.channels() + kRingCols - 1) / kRingCols) : 0;
+    kern<<<(unsigned)((items + y - 1) / y + ring), dim3(x, y), 0, stream>>>(a);
+  };
+  if (nvec <= 32) go(finish_kernel<T, VEC, 1>, 1);
+  else if (nvec <= 64) go(finish_kernel<T, VEC, 2>, 2);
+  else if (nvec <= 4096) go(finish_kernel<T, VEC, 4>, 4);
+  else if (VEC == 1 && nvec <= 16384) go(finish_kernel<T, 1, 16>, 16);
   else { mfb_host::set_error("state_space: parts of %d columns", gw); return 1; }
   return 0;
 }
 
 template <typename T>
-int run(const Args& a, int longest, cudaStream_t stream) {
+int run(Args a, int longest, cudaStream_t stream) {
   constexpr int V = 16 / sizeof(T);
   const int C = a.channels();
   if (a.cu_q) {
     const bool vec = a.inner() % V == 0 && C % V == 0 && a.ld % V == 0 && a.ld_x % V == 0 && al16(a.proj) && al16(a.xbc) &&
                      al16(a.ring) && al16(a.conv) && al16(a.conv_b) && C % 4 == 0 && a.taps <= 4;
-    if (vec) conv<T, V>(a, stream);
+    if (vec) conv<T, 4>(a, stream);
     else conv<T, 1>(a, stream);
     if (sizeof(T) == 2 && longest > 0 && chunks_ok(a)) {
       if (int rc = in_chunks(a, longest, stream)) return rc;
     } else scan<T>(a, stream);
   } else {
     const bool vec = a.P % 4 == 0;
-    const size_t smem = (size_t)(2 * a.N + a.P + kDec * (vec ? 4 : 1)) * sizeof(float);
+    auto bytes = [&](int heads) { return (size_t)(2 * a.N + heads * (a.P + kDec * (vec ? 4 : 1))) * sizeof(float); };
+    a.rows = 1;                                       // heads per CTA, as long as the GPU stays full
+    while (a.rows < 4 && (a.H / a.G) % (a.rows * 2) == 0 && a.H / (a.rows * 2) * (long long)a.B >= 148 * 4 &&
+           bytes(a.rows * 2) <= 32 * 1024) a.rows *= 2;
+    const size_t smem = bytes(a.rows);
     if (smem > 48 * 1024) { mfb_host::set_error("state_space: N=%d P=%d", a.N, a.P); return 1; }
-    const dim3 grid(a.H, a.B);
+    const dim3 grid(a.H / a.rows, a.B);
     if (vec) decode_kernel<T, 4><<<grid, kDec, smem, stream>>>(a);
     else decode_kernel<T, 1><<<grid, kDec, smem, stream>>>(a);
   }
