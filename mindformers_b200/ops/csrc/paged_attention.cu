@@ -100,7 +100,9 @@ paged_decode_split_kernel(const __nv_bfloat16* __restrict__ q,        // [B, Hq,
   constexpr int SLOTS = kPaWarps * KPW;
   const int split = blockIdx.x, kvh = blockIdx.y, b = blockIdx.z, splits = gridDim.x;
   const int group = Hq / Hkv;
-  const int ctx = context_lens[b];
+  const int* table = block_tables + (size_t)b * max_blocks;
+  // an idle row of a captured step has a length but no blocks: no keys
+  const int ctx = table[0] < 0 ? 0 : min(context_lens[b], max_blocks * block_size);
   const int k_begin = split * chunk;
   const int k_end = min(ctx, k_begin + chunk);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -108,7 +110,6 @@ paged_decode_split_kernel(const __nv_bfloat16* __restrict__ q,        // [B, Hq,
   const int slot = warp * KPW + sub;
   __shared__ float sh_acc[SLOTS][kPaHeadsPerPass][HD];
   __shared__ float sh_m[SLOTS][kPaHeadsPerPass], sh_l[SLOTS][kPaHeadsPerPass];
-  const int* table = block_tables + (size_t)b * max_blocks;
   const size_t row = (size_t)Hkv * HD;
   const float scale_log2 = scale * 1.4426950408889634f;
   for (int h0 = 0; h0 < group; h0 += kPaHeadsPerPass) {
@@ -140,7 +141,7 @@ paged_decode_split_kernel(const __nv_bfloat16* __restrict__ q,        // [B, Hq,
     using Slice = typename std::conditional<INT8, SliceI8, SliceBf>::type;
     auto fetch = [&](int t0, Slice& s_) {
       const int tk = (t0 + sub < k_end) ? t0 + sub : k_end - 1;
-      const int blk = table[tk / block_size];
+      const int blk = max(table[tk / block_size], 0);          // a block that is missing belongs to a row nobody reads
       const size_t tok = (size_t)blk * block_size + tk % block_size;
       const size_t base = tok * row + (size_t)kvh * HD + dl * 8;
       if constexpr (INT8) {

@@ -851,6 +851,15 @@ def test_int8_kv_cache_write_decode_and_gather(hd, nq, nkv, block):
                                      causal=False)
         assert torch.allclose(out[b].float(), ref[0, 0], rtol=2e-2, atol=2e-2), (b, (out[b].float() - ref[0, 0]).abs().max())
         o += n
+    # an idle row of a captured step has a length but no blocks: zeros, and the others as before
+    idle, again = perm.clone(), torch.empty_like(out)
+    idle[0] = -1
+    rc = lib.mfb_paged_decode_attention_ex(q.data_ptr(), kc.data_ptr(), vc.data_ptr(), cache.key_scale[0].data_ptr(),
+                                           cache.value_scale[0].data_ptr(), idle.data_ptr(), ctx.data_ptr(), again.data_ptr(),
+                                           scratch.data_ptr(), splits, B, nq, nkv, hd, block, max_blocks, hd ** -0.5,
+                                           _lib.stream_ptr())
+    _lib.check(rc, "paged decode int8")
+    assert float(again[0].abs().max()) == 0 and torch.equal(again[1:], out[1:])
 
 
 @pytest.mark.parametrize("T", [1, 7, 16, 17, 32, 33, 64])
